@@ -5,6 +5,9 @@ Three shared objects are produced under ``hartsyinference_b200/lib``:
 * ``libb200_kernels.so``  every ``csrc/kernels/*.cu`` compiled for sm_100a only
   (``-gencode arch=compute_100a,code=sm_100a``); plain C ABI, no PyTorch headers, loaded with
   ctypes and called with raw device pointers and the current CUDA stream.
+  ``libb200_kernels_decoder.so`` is the same library with the sources of ``KERNEL_GROUPS["decoder"]``
+  only: what a language model with per-layer mixers launches (``ensure("decoder")`` builds it where the
+  full library has not been built).
 * ``libb200_runtime.so``  host-side C++ runtime (``csrc/runtime/*.cpp``): safetensors / GGUF
   readers, GGUF block codecs, paged-KV block allocator, continuous-batching scheduler core,
   BPE tokenizer. No CUDA dependency, so it builds and is tested on CPU-only machines.
@@ -41,6 +44,11 @@ NVCC_FLAGS = [
     "--expt-relaxed-constexpr",
     "-diag-suppress", "550,177",
 ]
+# sources that make a smaller library for one kind of model; no source refers to a symbol of another one
+# except the launch switch that gemm_tcgen05.cu defines
+KERNEL_GROUPS = {
+    "decoder": ("gemm_tcgen05", "attention", "delta", "fused_ops", "linear_f32", "moe", "residual_norm", "sampling"),
+}
 CXX_FLAGS = ["-O2", "-std=c++17", "-fPIC", "-Wall", "-Wno-unused-function", "-pthread"]
 
 
@@ -83,10 +91,26 @@ def _save_stamp(stamp: dict) -> None:
     (LIB / "build_stamp.json").write_text(json.dumps(stamp, indent=1))
 
 
-def build_kernels(force: bool = False, verbose: bool = False) -> Path:
-    """Compile every CUDA source for sm_100a and link ``libb200_kernels.so``."""
-    out = LIB / "libb200_kernels.so"
+def group_lib(group: str) -> Path:
+    return LIB / f"libb200_kernels_{group}.so"
+
+
+def ensure(group: str, verbose: bool = False) -> Path:
+    """The full kernels library when it has been built, else the group's own (compiled now if it is
+    missing or older than its sources), and the host runtime."""
+    LIB.mkdir(parents=True, exist_ok=True)
+    build_runtime(verbose=verbose)
+    full = LIB / "libb200_kernels.so"
+    return full if full.exists() else build_kernels(verbose=verbose, group=group)
+
+
+def build_kernels(force: bool = False, verbose: bool = False, group: str = "") -> Path:
+    """Compile every CUDA source (or those of ``group``) for sm_100a and link ``libb200_kernels.so`` (or the
+    group's library)."""
+    out = group_lib(group) if group else LIB / "libb200_kernels.so"
     srcs = sorted((CSRC / "kernels").glob("*.cu"))
+    if group:
+        srcs = [s for s in srcs if s.stem in KERNEL_GROUPS[group]]
     hdrs = sorted((CSRC / "kernels").glob("*.cuh")) + sorted((CSRC / "kernels").glob("*.h"))
     stamp = _load_stamp()
     nvcc = _nvcc()
@@ -111,10 +135,13 @@ def build_kernels(force: bool = False, verbose: bool = False) -> Path:
                 s, d = futs[f]
                 stamp[f"obj:{s.name}"] = d
     link_digest = hashlib.sha256("".join(stamp.get(f"obj:{s.name}", "") for s in srcs).encode()).hexdigest()
-    if force or jobs or not out.exists() or stamp.get("kernels") != link_digest:
-        _run([nvcc, "-shared", "-o", str(out), *[str(o) for o in objs], "-gencode",
+    key = f"kernels:{group}" if group else "kernels"
+    if force or jobs or not out.exists() or stamp.get(key) != link_digest:
+        tmp = out.with_suffix(f".{os.getpid()}.tmp")
+        _run([nvcc, "-shared", "-o", str(tmp), *[str(o) for o in objs], "-gencode",
               "arch=compute_100a,code=sm_100a", "-Xcompiler", "-fPIC"], verbose)
-        stamp["kernels"] = link_digest
+        os.replace(tmp, out)
+        stamp[key] = link_digest
     _save_stamp(stamp)
     return out
 

@@ -13,7 +13,12 @@
 // src/HartsyInference.Cuda/Kernels/lm/flash_attn_f32.cu, flash_attn_f32_split.cu,
 // flash_attn_v2_tf32.cu). Supported per-call options follow the reference's attention oracle
 // (src/HartsyInference.Core/Backends/AttentionReference.cs): GQA, causal, sliding window,
-// logit soft-cap.
+// logit soft-cap. The extended form of both kernels (template flag kExt) adds, each optional: a bias
+// by key distance from a per-head table, a per-head sink score that only enters the denominator,
+// values that are the keys themselves (one page plane), a sigmoid gate on the output, any head size
+// up to 128 that is a multiple of 8, and a row pitch for q. There the probabilities keep 16 bits of
+// mantissa in the PV product (a bf16 head and a bf16 remainder). `attn_rows_kernel` computes the same
+// with plain fp32 arithmetic for models run in 32 bits and for shapes the tensor-core form leaves out.
 //
 // The score and PV products use warp-level mma.sync (m16n8k16, bf16): with one to sixteen query
 // rows per KV head the kernel is bound by KV bandwidth, not by tensor throughput, and a 128-row
@@ -48,7 +53,14 @@ struct AttnParams {
   uint8_t* out_q;               // [seqs][hq * d] or null
   void* out_scale;              // fp32 [seqs][hq], or blocked UE8M0 bytes when sf_tile_rows > 0
   int sf_tile_rows;
+  // extended form only
+  const float* dist_bias;       // [hq][dist_len] added to the score by key distance (last entry beyond it), or null
+  const float* sinks;           // [hq] score of a key without a value, or null
+  const __nv_bfloat16* gate;    // [tokens][gate_ld]: out *= sigmoid(gate), or null
+  long long q_ld, gate_ld;      // row pitches in elements
+  int dist_len, d, shared_kv;   // d: head size as stored; shared_kv: v is k
 };
+constexpr float kLog2e = 1.4426950408889634f;
 
 // Shared-memory tile: [64 tokens][D] bf16, row pitch D * 2 bytes, 16-byte chunks XOR-swizzled with
 // (token & 7) so that ldmatrix rows of consecutive tokens hit different banks.
@@ -61,19 +73,19 @@ __device__ __forceinline__ uint32_t tile_off(int token, int chunk) {
 // shared memory (`pg`, 64 / page entries) an iteration earlier, so no cp.async waits on a
 // dependent global load of the table; page sizes are powers of two (8..64), so token -> (page,
 // offset) is a shift and a mask.
-template <int D>
+template <int D, bool kExt = false>
 __device__ __forceinline__ void load_tile_paged(uint32_t smem_base, const __nv_bfloat16* pool,
                                                 const int* pg, int kv_head, int hkv, int page_shift,
-                                                int tok0, int kv_len) {
+                                                int tok0, int kv_len, int d = D) {
   constexpr int kChunks = D / 8;
   const int page_mask = (1 << page_shift) - 1;
   for (int i = threadIdx.x; i < kTileTokens * kChunks; i += kAttnThreads) {
     const int t = i / kChunks, c = i % kChunks;
-    const bool valid = tok0 + t < kv_len;
+    const bool valid = tok0 + t < kv_len && (!kExt || c * 8 < d);
     const __nv_bfloat16* src = pool;
     if (valid) {
       const long long pgi = pg[t >> page_shift];
-      src = pool + (((pgi * hkv + kv_head) << page_shift) + (t & page_mask)) * D + c * 8;
+      src = pool + (((pgi * hkv + kv_head) << page_shift) + (t & page_mask)) * (kExt ? d : D) + c * 8;
     }
     cp_async_16(smem_base + tile_off<D>(t, c), src, valid);
   }
@@ -122,11 +134,14 @@ struct WarpState {
 // Processes NG groups of 16 tokens starting at tile-local token `t_begin` for this warp.
 //   qf: Q fragments [D/16][4]; row_limit[r]: first masked key position for the thread's row r
 //   (keys >= limit are masked), row_start[r]: first visible key (sliding window).
-template <int D, int NG>
+//   Extended form: row_bias[r] is the row's distance-bias table (the distance of a key is counted back
+//   from row_limit[r] - 1).
+template <int D, int NG, bool kExt = false>
 __device__ __forceinline__ void warp_tile(WarpState<D>& st, const uint32_t (&qf)[D / 16][4],
                                           uint32_t k_smem, uint32_t v_smem, int t_begin,
                                           int tok0, const int (&row_limit)[2],
-                                          const int (&row_start)[2], const AttnParams& p) {
+                                          const int (&row_start)[2], const AttnParams& p,
+                                          const float* const* row_bias = nullptr) {
   const int lane = threadIdx.x & 31;
   const int tq = lane & 3;
   float s[NG * 2][4];
@@ -159,6 +174,10 @@ __device__ __forceinline__ void warp_tile(WarpState<D>& st, const uint32_t (&qf)
       float x = s[nt][j];
       if (p.softcap > 0.f) x = p.softcap * tanhf(x * p.scale / p.softcap) * (p.scale_log2 / p.scale);
       else x *= p.scale_log2;
+      if (kExt && p.dist_bias) {
+        const int dist = min(max(row_limit[r] - 1 - key, 0), p.dist_len - 1);
+        x = fmaf(row_bias[r][dist], kLog2e, x);
+      }
       if (key >= row_limit[r] || key < row_start[r]) x = -INFINITY;
       s[nt][j] = x;
       mx[r] = fmaxf(mx[r], x);
@@ -178,7 +197,7 @@ __device__ __forceinline__ void warp_tile(WarpState<D>& st, const uint32_t (&qf)
     st.m[r] = mnew;
   }
   float rs[2] = {0.f, 0.f};
-  uint32_t pf[NG][4];
+  uint32_t pf[NG][4], pl[kExt ? NG : 1][4];
 #pragma unroll
   for (int nt = 0; nt < NG * 2; ++nt) {
     float e[4];
@@ -191,6 +210,12 @@ __device__ __forceinline__ void warp_tile(WarpState<D>& st, const uint32_t (&qf)
     // from the odd one
     pf[nt >> 1][(nt & 1) * 2 + 0] = pack_bf16x2(e[0], e[1]);
     pf[nt >> 1][(nt & 1) * 2 + 1] = pack_bf16x2(e[2], e[3]);
+    if (kExt) {
+#pragma unroll
+      for (int j = 0; j < 4; ++j) e[j] -= __bfloat162float(__float2bfloat16(e[j]));
+      pl[kExt ? nt >> 1 : 0][(nt & 1) * 2 + 0] = pack_bf16x2(e[0], e[1]);
+      pl[kExt ? nt >> 1 : 0][(nt & 1) * 2 + 1] = pack_bf16x2(e[2], e[3]);
+    }
   }
 #pragma unroll
   for (int r = 0; r < 2; ++r) {
@@ -217,14 +242,22 @@ __device__ __forceinline__ void warp_tile(WarpState<D>& st, const uint32_t (&qf)
       ldmatrix_x4_trans(v_smem + tile_off<D>(token, chunk), b0, b1, b2, b3);
       mma_bf16_16816(st.o[np * 2], pf[gi], b0, b1);
       mma_bf16_16816(st.o[np * 2 + 1], pf[gi], b2, b3);
+      if (kExt) {
+        mma_bf16_16816(st.o[np * 2], pl[kExt ? gi : 0], b0, b1);
+        mma_bf16_16816(st.o[np * 2 + 1], pl[kExt ? gi : 0], b2, b3);
+      }
     }
   }
+}
+
+__device__ __forceinline__ float gate_of(const AttnParams& p, long long token, int head, int c) {
+  return p.gate ? 1.f / (1.f + __expf(-__bfloat162float(p.gate[token * p.gate_ld + head * p.d + c]))) : 1.f;
 }
 
 // ------------------------------------------------------------------------------------------
 // decode
 // ------------------------------------------------------------------------------------------
-template <int D, int kStages>
+template <int D, int kStages, bool kExt = false>
 __global__ void __launch_bounds__(kAttnThreads)
 attn_decode_kernel(const AttnParams p) {
   pdl_wait();
@@ -237,8 +270,10 @@ attn_decode_kernel(const AttnParams p) {
   const int G = p.hq / p.hkv;
   const int kv_len = p.kv_lens[seq];
   const int n_tiles = (kv_len + kTileTokens - 1) / kTileTokens;
-  const int tiles_per_split = (n_tiles + p.splits - 1) / p.splits;
-  const int tile_begin = split * tiles_per_split;
+  const int start_key = p.window > 0 ? max(0, kv_len - p.window) : 0;
+  const int tile0 = start_key / kTileTokens;                    // tiles before the window are not read
+  const int tiles_per_split = (n_tiles - tile0 + p.splits - 1) / p.splits;
+  const int tile_begin = tile0 + split * tiles_per_split;
   const int tile_end = min(n_tiles, tile_begin + tiles_per_split);
   const int* table = p.block_table + static_cast<long long>(seq) * p.max_pages;
   const uint32_t smem_base = smem_u32(smem);
@@ -246,10 +281,18 @@ attn_decode_kernel(const AttnParams p) {
   // Q fragments: row = query head within the group (rows >= G are zero)
   uint32_t qf[D / 16][4];
   {
-    const __nv_bfloat16* qb = p.q + (static_cast<long long>(seq) * p.hq + kvh * G) * D;
+    const int d = kExt ? p.d : D;
+    const __nv_bfloat16* qb = kExt ? p.q + seq * p.q_ld + kvh * G * d : p.q + (static_cast<long long>(seq) * p.hq + kvh * G) * D;
 #pragma unroll
     for (int kk = 0; kk < D / 16; ++kk) {
       const int c0 = kk * 16 + tq * 2;
+      if (kExt) {
+        qf[kk][0] = g < G && c0 < d ? *reinterpret_cast<const uint32_t*>(qb + g * d + c0) : 0u;
+        qf[kk][1] = g + 8 < G && c0 < d ? *reinterpret_cast<const uint32_t*>(qb + (g + 8) * d + c0) : 0u;
+        qf[kk][2] = g < G && c0 + 8 < d ? *reinterpret_cast<const uint32_t*>(qb + g * d + c0 + 8) : 0u;
+        qf[kk][3] = g + 8 < G && c0 + 8 < d ? *reinterpret_cast<const uint32_t*>(qb + (g + 8) * d + c0 + 8) : 0u;
+        continue;
+      }
       qf[kk][0] = g < G ? *reinterpret_cast<const uint32_t*>(qb + g * D + c0) : 0u;
       qf[kk][1] = g + 8 < G ? *reinterpret_cast<const uint32_t*>(qb + (g + 8) * D + c0) : 0u;
       qf[kk][2] = g < G ? *reinterpret_cast<const uint32_t*>(qb + g * D + c0 + 8) : 0u;
@@ -259,13 +302,32 @@ attn_decode_kernel(const AttnParams p) {
   WarpState<D> st;
   st.init();
   const int lim[2] = {kv_len, kv_len};
-  const int start_key = p.window > 0 ? max(0, kv_len - p.window) : 0;
   const int start[2] = {start_key, start_key};
+  const float* row_bias[2] = {nullptr, nullptr};
+  if (kExt) {
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      const int head = kvh * G + min(g + 8 * r, G - 1);
+      if (p.dist_bias) row_bias[r] = p.dist_bias + static_cast<long long>(head) * p.dist_len;
+      if (p.sinks && split == 0 && warp == 0) {       // the sink enters the running sums once
+        st.m[r] = p.sinks[head] * kLog2e;
+        st.l[r] = 1.f;
+      }
+    }
+  }
 
   __shared__ int pg_ring[4][8];
   auto issue = [&](int tile, int stage) {
     if (tile < tile_end) {
       const uint32_t kb = smem_base + stage * 2 * kTileBytes;
+      if (kExt) {
+        load_tile_paged<D, true>(kb, p.k, pg_ring[tile & 3], kvh, p.hkv, p.page_shift, tile * kTileTokens, kv_len, p.d);
+        if (!p.shared_kv)
+          load_tile_paged<D, true>(kb + kTileBytes, p.v, pg_ring[tile & 3], kvh, p.hkv, p.page_shift, tile * kTileTokens,
+                                   kv_len, p.d);
+        cp_async_commit();
+        return;
+      }
       load_tile_paged<D>(kb, p.k, pg_ring[tile & 3], kvh, p.hkv, p.page_shift, tile * kTileTokens, kv_len);
       load_tile_paged<D>(kb + kTileBytes, p.v, pg_ring[tile & 3], kvh, p.hkv, p.page_shift,
                          tile * kTileTokens, kv_len);
@@ -286,7 +348,8 @@ attn_decode_kernel(const AttnParams p) {
     cp_async_wait<kStages - 1>();
     __syncthreads();
     const uint32_t kb = smem_base + stage * 2 * kTileBytes;
-    warp_tile<D, 1>(st, qf, kb, kb + kTileBytes, warp * 16, tile * kTileTokens, lim, start, p);
+    warp_tile<D, 1, kExt>(st, qf, kb, kExt && p.shared_kv ? kb : kb + kTileBytes, warp * 16, tile * kTileTokens, lim, start, p,
+                          row_bias);
     __syncthreads();
     stage = (stage + 1) % kStages;
   }
@@ -325,7 +388,11 @@ attn_decode_kernel(const AttnParams p) {
       ll += sml[(w * 16 + r) * 2 + 1] * f;
     }
     const int head = kvh * G + r;
-    if (p.splits == 1) {
+    if (kExt && p.splits == 1) {
+      if (c < p.d)
+        p.out[(static_cast<long long>(seq) * p.hq + head) * p.d + c] =
+            __float2bfloat16((ll > 0.f ? acc / ll : 0.f) * gate_of(p, seq, head, c));
+    } else if (p.splits == 1) {
       p.out[(static_cast<long long>(seq) * p.hq + head) * D + c] =
           __float2bfloat16(ll > 0.f ? acc / ll : 0.f);
     } else {
@@ -339,7 +406,7 @@ attn_decode_kernel(const AttnParams p) {
   }
 }
 
-template <int D>
+template <int D, bool kExt = false>
 __global__ void attn_combine_kernel(const AttnParams p) {
   pdl_wait();
   pdl_trigger();
@@ -354,6 +421,12 @@ __global__ void attn_combine_kernel(const AttnParams p) {
       const float f = ms == -INFINITY ? 0.f : exp2f(ms - mm);
       acc += p.ws_o[(base + s) * D + c] * f;
       ll += p.ws_ml[(base + s) * 2 + 1] * f;
+    }
+    if (kExt) {
+      if (c < p.d)
+        p.out[(static_cast<long long>(seq) * p.hq + head) * p.d + c] =
+            __float2bfloat16((ll > 0.f ? acc / ll : 0.f) * gate_of(p, seq, head, c));
+      continue;
     }
     const __nv_bfloat16 o = __float2bfloat16(ll > 0.f ? acc / ll : 0.f);
     if (p.out) p.out[(static_cast<long long>(seq) * p.hq + head) * D + c] = o;
@@ -397,7 +470,7 @@ __global__ void attn_combine_kernel(const AttnParams p) {
 // ------------------------------------------------------------------------------------------
 // prefill / full attention
 // ------------------------------------------------------------------------------------------
-template <int D, bool kPaged>
+template <int D, bool kPaged, bool kExt = false>
 __global__ void __launch_bounds__(kAttnThreads)
 attn_prefill_kernel(const AttnParams p) {
   constexpr int kStages = 2;
@@ -418,11 +491,19 @@ attn_prefill_kernel(const AttnParams p) {
   const int row0 = qt * 64 + warp * 16 + g;   // this thread's rows: row0, row0 + 8
   uint32_t qf[D / 16][4];
   {
-    const __nv_bfloat16* qb = p.q + (static_cast<long long>(q_off) * p.hq + head) * D;
-    const long long rs = static_cast<long long>(p.hq) * D;
+    const int d = kExt ? p.d : D;
+    const __nv_bfloat16* qb = kExt ? p.q + q_off * p.q_ld + head * d : p.q + (static_cast<long long>(q_off) * p.hq + head) * D;
+    const long long rs = kExt ? p.q_ld : static_cast<long long>(p.hq) * D;
 #pragma unroll
     for (int kk = 0; kk < D / 16; ++kk) {
       const int c0 = kk * 16 + tq * 2;
+      if (kExt) {
+        qf[kk][0] = row0 < q_len && c0 < d ? *reinterpret_cast<const uint32_t*>(qb + row0 * rs + c0) : 0u;
+        qf[kk][1] = row0 + 8 < q_len && c0 < d ? *reinterpret_cast<const uint32_t*>(qb + (row0 + 8) * rs + c0) : 0u;
+        qf[kk][2] = row0 < q_len && c0 + 8 < d ? *reinterpret_cast<const uint32_t*>(qb + row0 * rs + c0 + 8) : 0u;
+        qf[kk][3] = row0 + 8 < q_len && c0 + 8 < d ? *reinterpret_cast<const uint32_t*>(qb + (row0 + 8) * rs + c0 + 8) : 0u;
+        continue;
+      }
       qf[kk][0] = row0 < q_len ? *reinterpret_cast<const uint32_t*>(qb + row0 * rs + c0) : 0u;
       qf[kk][1] = row0 + 8 < q_len ? *reinterpret_cast<const uint32_t*>(qb + (row0 + 8) * rs + c0) : 0u;
       qf[kk][2] = row0 < q_len ? *reinterpret_cast<const uint32_t*>(qb + row0 * rs + c0 + 8) : 0u;
@@ -437,6 +518,14 @@ attn_prefill_kernel(const AttnParams p) {
     const int pos = ctx + row0 + 8 * r;   // absolute position of the query row
     lim[r] = p.causal ? min(kv_len, pos + 1) : kv_len;
     start[r] = p.window > 0 ? max(0, pos + 1 - p.window) : 0;
+  }
+  const float* row_bias[2] = {nullptr, nullptr};
+  if (kExt) {
+    if (p.dist_bias) row_bias[0] = row_bias[1] = p.dist_bias + static_cast<long long>(head) * p.dist_len;
+    if (p.sinks) {
+      st.m[0] = st.m[1] = p.sinks[head] * kLog2e;
+      st.l[0] = st.l[1] = 1.f;
+    }
   }
   // keys needed by this CTA: up to the last row's position when causal
   const int last_pos = ctx + min(q_len, qt * 64 + 64) - 1;
@@ -455,7 +544,12 @@ attn_prefill_kernel(const AttnParams p) {
   auto issue = [&](int tile, int stage) {
     if (tile < n_tiles) {
       const uint32_t kb = smem_base + stage * 2 * kTileBytes;
-      if (kPaged) {
+      if (kExt) {
+        load_tile_paged<D, true>(kb, p.k, pg_ring[tile & 3], kvh, p.hkv, p.page_shift, tile * kTileTokens, kv_needed, p.d);
+        if (!p.shared_kv)
+          load_tile_paged<D, true>(kb + kTileBytes, p.v, pg_ring[tile & 3], kvh, p.hkv, p.page_shift, tile * kTileTokens,
+                                   kv_needed, p.d);
+      } else if (kPaged) {
         load_tile_paged<D>(kb, p.k, pg_ring[tile & 3], kvh, p.hkv, p.page_shift, tile * kTileTokens, kv_needed);
         load_tile_paged<D>(kb + kTileBytes, p.v, pg_ring[tile & 3], kvh, p.hkv, p.page_shift,
                            tile * kTileTokens, kv_needed);
@@ -481,7 +575,7 @@ attn_prefill_kernel(const AttnParams p) {
     const uint32_t kb = smem_base + stage * 2 * kTileBytes;
     // a warp whose rows all lie before this tile (causal) still runs: masked scores cost nothing
     // in correctness and keep the barrier pattern uniform
-    warp_tile<D, 4>(st, qf, kb, kb + kTileBytes, 0, tile * kTileTokens, lim, start, p);
+    warp_tile<D, 4, kExt>(st, qf, kb, kExt && p.shared_kv ? kb : kb + kTileBytes, 0, tile * kTileTokens, lim, start, p, row_bias);
     __syncthreads();
     stage ^= 1;
   }
@@ -498,11 +592,124 @@ attn_prefill_kernel(const AttnParams p) {
 #pragma unroll
       for (int i = 0; i < D / 8; ++i) {
         const int c = i * 8 + tq * 2;
+        if (kExt) {
+          if (c < p.d)
+            *reinterpret_cast<uint32_t*>(p.out + (static_cast<long long>(q_off + row) * p.hq + head) * p.d + c) =
+                pack_bf16x2(st.o[i][2 * r] * inv * gate_of(p, q_off + row, head, c),
+                            st.o[i][2 * r + 1] * inv * gate_of(p, q_off + row, head, c + 1));
+          continue;
+        }
         *reinterpret_cast<uint32_t*>(ob + row * rs + c) =
             pack_bf16x2(st.o[i][2 * r] * inv, st.o[i][2 * r + 1] * inv);
       }
     }
   }
+}
+
+// ------------------------------------------------------------------------------------------
+// plain form: one warp per (token, head), 32 keys at a time, fp32 arithmetic throughout
+// ------------------------------------------------------------------------------------------
+struct AttnRowsParams {
+  const void *q, *k, *v, *gate;
+  void* out;
+  const int *block_table, *kv_lens, *cu_q;
+  const float *dist_bias, *sinks;
+  long long q_ld, gate_ld;
+  int tokens, seqs, hq, hkv, d, page, max_pages, window, dist_len;
+  float scale, softcap;
+};
+constexpr int kRowsMaxD = 512;
+
+__device__ __forceinline__ float as_f32(float v) { return v; }
+__device__ __forceinline__ float as_f32(__nv_bfloat16 v) { return __bfloat162float(v); }
+
+template <typename T>
+__global__ void __launch_bounds__(128) attn_rows_kernel(const AttnRowsParams p) {
+  pdl_wait();
+  pdl_trigger();
+  __shared__ float qs[4][kRowsMaxD];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int t = blockIdx.x * 4 + warp, head = blockIdx.y;
+  if (t >= p.tokens) return;
+  int seq = t, first = t, q_len = 1;
+  if (p.cu_q) {
+    int lo = 0, hi = p.seqs - 1;
+    while (lo < hi) {
+      const int mid = (lo + hi + 1) >> 1;
+      if (p.cu_q[mid] <= t) lo = mid; else hi = mid - 1;
+    }
+    seq = lo;
+    first = p.cu_q[seq];
+    q_len = p.cu_q[seq + 1] - first;
+  }
+  const int pos = p.kv_lens[seq] - q_len + (t - first);      // -1 for an empty sequence: no keys
+  const int begin = p.window > 0 ? max(0, pos + 1 - p.window) : 0;
+  const int kvh = head / (p.hq / p.hkv);
+  const int* table = p.block_table + static_cast<long long>(seq) * p.max_pages;
+  const T* q = static_cast<const T*>(p.q) + t * p.q_ld + head * p.d;
+  for (int c = lane; c < p.d; c += 32) qs[warp][c] = as_f32(q[c]);
+  __syncwarp();
+  float m = p.sinks ? p.sinks[head] : -INFINITY, l = p.sinks ? 1.f : 0.f;
+  float o[kRowsMaxD / 32];
+#pragma unroll
+  for (int i = 0; i < kRowsMaxD / 32; ++i) o[i] = 0.f;
+  for (int j0 = begin; j0 <= pos; j0 += 32) {
+    const int j = j0 + lane;
+    long long at = 0;
+    float s = -INFINITY;
+    if (j <= pos) {
+      at = ((static_cast<long long>(table[j / p.page]) * p.hkv + kvh) * p.page + j % p.page) * p.d;
+      const T* kr = static_cast<const T*>(p.k) + at;
+      float a = 0.f;
+      for (int c = 0; c < p.d; ++c) a += qs[warp][c] * as_f32(kr[c]);
+      s = a * p.scale;
+      if (p.softcap > 0.f) s = p.softcap * tanhf(s / p.softcap);
+      if (p.dist_bias) s += p.dist_bias[static_cast<long long>(head) * p.dist_len + min(pos - j, p.dist_len - 1)];
+    }
+    const float mn = fmaxf(m, warp_max(s));
+    const float f = m == -INFINITY ? 0.f : expf(m - mn);
+    const float e = s == -INFINITY ? 0.f : expf(s - mn);
+    l = l * f + warp_sum(e);
+    m = mn;
+#pragma unroll
+    for (int i = 0; i < kRowsMaxD / 32; ++i) o[i] *= f;
+    const int n = min(32, pos - j0 + 1);
+    for (int jj = 0; jj < n; ++jj) {
+      const float w = __shfl_sync(0xffffffffu, e, jj);
+      const T* vr = static_cast<const T*>(p.v) + __shfl_sync(0xffffffffu, at, jj);
+#pragma unroll
+      for (int i = 0; i < kRowsMaxD / 32; ++i)
+        if (lane + i * 32 < p.d) o[i] += w * as_f32(vr[lane + i * 32]);
+    }
+  }
+  T* out = static_cast<T*>(p.out) + (static_cast<long long>(t) * p.hq + head) * p.d;
+  const T* gate = p.gate ? static_cast<const T*>(p.gate) + t * p.gate_ld + head * p.d : nullptr;
+#pragma unroll
+  for (int i = 0; i < kRowsMaxD / 32; ++i) {
+    const int c = lane + i * 32;
+    if (c < p.d) {
+      float y = l > 0.f ? o[i] / l : 0.f;
+      if (gate) y *= 1.f / (1.f + expf(-as_f32(gate[c])));
+      out[c] = static_cast<T>(y);
+    }
+  }
+}
+
+// Rows of keys (and values) into their pages: [tokens][ld] -> [pages][hkv][page][row], 16 bytes per thread
+__global__ void kv_store_kernel(const uint8_t* __restrict__ k, const uint8_t* __restrict__ v, uint8_t* __restrict__ kc,
+                                uint8_t* __restrict__ vc, const long long* __restrict__ slots, int tokens, int hkv,
+                                int row_vecs, int page, long long ld_bytes) {
+  pdl_wait();
+  pdl_trigger();
+  const long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x;
+  if (i >= static_cast<long long>(tokens) * hkv * row_vecs) return;
+  const int c = static_cast<int>(i % row_vecs), h = static_cast<int>(i / row_vecs % hkv);
+  const long long t = i / row_vecs / hkv, slot = slots[t];
+  if (slot < 0) return;
+  const long long src = t * ld_bytes + (static_cast<long long>(h) * row_vecs + c) * 16;
+  const long long dst = (((slot / page) * hkv + h) * page + slot % page) * row_vecs + c;
+  reinterpret_cast<uint4*>(kc)[dst] = *reinterpret_cast<const uint4*>(k + src);
+  if (v) reinterpret_cast<uint4*>(vc)[dst] = *reinterpret_cast<const uint4*>(v + src);
 }
 
 }  // namespace b200
@@ -644,5 +851,105 @@ B200_API int b200_attn_prefill(const void* q, const void* k, const void* v, void
   }
 #undef LAUNCH_PREFILL
   cudaError_t e = cudaGetLastError();
+  return e == cudaSuccess ? 0 : -static_cast<int>(e) - 300;
+}
+
+// Extended attention over pages (see the header comment). cu_q null: one query token per sequence.
+// q [tokens][q_ld] (head h at h * d), out [tokens][hq * d]. v_cache null: the values are the keys.
+// exact != 0: plain fp32 kernel, tensors are fp32 when f32 is set and bf16 otherwise; exact == 0: the
+// tensor-core kernels (bf16, d <= 128, at most 16 query heads per key head at decode; returns -6 for
+// what they do not take). splits / workspace: decode only, as in b200_attn_decode (with the head size
+// rounded up to 64 or 128).
+B200_API int b200_attn_biased(const void* q, const void* k_cache, const void* v_cache, void* out, const int* block_table,
+                              const int* kv_lens, const int* cu_q, int tokens, int seqs, int max_q_len, int hq, int hkv, int d,
+                              int page, int max_pages, int splits, void* workspace, float scale, float softcap, int window,
+                              const float* dist_bias, int dist_len, const float* sinks, const void* gate, long long gate_ld,
+                              long long q_ld, int exact, int f32, cudaStream_t stream) {
+  if (tokens <= 0 || seqs <= 0) return 0;
+  if (d % 8 || d < 8 || d > kRowsMaxD || hq % hkv || q_ld % 8 || (gate && gate_ld % 8) || (dist_bias && dist_len < 1)) return -2;
+  if (f32 && !exact) return -6;
+  if (exact) {
+    AttnRowsParams p{q, k_cache, v_cache ? v_cache : k_cache, gate, out, block_table, kv_lens, cu_q, dist_bias, sinks,
+                     q_ld, gate_ld, tokens, seqs, hq, hkv, d, page, max_pages, window, dist_len, scale, softcap};
+    const dim3 grid((tokens + 3) / 4, hq);
+    const cudaError_t e = f32 ? launch_pdl(attn_rows_kernel<float>, grid, dim3(128), 0, stream, p)
+                              : launch_pdl(attn_rows_kernel<__nv_bfloat16>, grid, dim3(128), 0, stream, p);
+    return e == cudaSuccess ? 0 : -static_cast<int>(e) - 300;
+  }
+  if (d > 128 || (!cu_q && hq / hkv > 16)) return -6;
+  AttnParams p{};
+  p.q = static_cast<const __nv_bfloat16*>(q);
+  p.k = static_cast<const __nv_bfloat16*>(k_cache);
+  p.v = static_cast<const __nv_bfloat16*>(v_cache ? v_cache : k_cache);
+  p.shared_kv = v_cache == nullptr;
+  p.out = static_cast<__nv_bfloat16*>(out);
+  p.block_table = block_table;
+  p.kv_lens = kv_lens;
+  p.cu_q = cu_q;
+  p.seqs = seqs; p.hq = hq; p.hkv = hkv; p.max_pages = max_pages; p.page = page;
+  p.page_shift = page == 8 ? 3 : page == 16 ? 4 : page == 32 ? 5 : page == 64 ? 6 : -1;
+  if (p.page_shift < 0) return -4;
+  p.causal = 1;
+  p.window = window;
+  p.scale = scale;
+  p.scale_log2 = scale * kLog2e;
+  p.softcap = softcap;
+  p.dist_bias = dist_bias; p.dist_len = dist_len; p.sinks = sinks;
+  p.gate = static_cast<const __nv_bfloat16*>(gate);
+  p.gate_ld = gate_ld; p.q_ld = q_ld; p.d = d;
+  p.splits = cu_q || splits < 1 ? 1 : splits;
+  const int dd = d <= 64 ? 64 : 128;
+  if (cu_q) {
+    if (max_q_len <= 0) return 0;
+    const dim3 grid((max_q_len + 63) / 64, hq, seqs);
+    const int smem = 2 * 2 * kTileTokens * dd * 2;
+    static PerDeviceOnce once[2];
+    if (dd == 128) {
+      if (once[1].first_time()) cudaFuncSetAttribute(attn_prefill_kernel<128, true, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+      attn_prefill_kernel<128, true, true><<<grid, kAttnThreads, smem, stream>>>(p);
+    } else {
+      if (once[0].first_time()) cudaFuncSetAttribute(attn_prefill_kernel<64, true, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+      attn_prefill_kernel<64, true, true><<<grid, kAttnThreads, smem, stream>>>(p);
+    }
+    const cudaError_t e = cudaGetLastError();
+    return e == cudaSuccess ? 0 : -static_cast<int>(e) - 300;
+  }
+  if (p.splits > 1) {
+    if (!workspace) return -5;
+    p.ws_o = static_cast<float*>(workspace);
+    p.ws_ml = p.ws_o + static_cast<long long>(seqs) * hq * p.splits * dd;
+  }
+  const dim3 grid(seqs, hkv, p.splits);
+  // the ring doubles as the buffer of the four warps' partial results
+  const int ring = 2 * 2 * kTileTokens * dd * 2, merge = 4 * 16 * (dd + 2) * 4, smem = ring > merge ? ring : merge;
+  static PerDeviceOnce once[2];
+  cudaError_t e;
+  if (dd == 128) {
+    if (once[1].first_time()) cudaFuncSetAttribute(attn_decode_kernel<128, 2, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    e = launch_pdl(attn_decode_kernel<128, 2, true>, grid, dim3(kAttnThreads), smem, stream, p);
+  } else {
+    if (once[0].first_time()) cudaFuncSetAttribute(attn_decode_kernel<64, 2, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    e = launch_pdl(attn_decode_kernel<64, 2, true>, grid, dim3(kAttnThreads), smem, stream, p);
+  }
+  if (e != cudaSuccess) return -static_cast<int>(e) - 300;
+  if (p.splits > 1) {
+    if (dd == 128) e = launch_pdl(attn_combine_kernel<128, true>, dim3(seqs, hq), dim3(128), 0, stream, p);
+    else e = launch_pdl(attn_combine_kernel<64, true>, dim3(seqs, hq), dim3(64), 0, stream, p);
+    if (e != cudaSuccess) return -static_cast<int>(e) - 400;
+  }
+  return 0;
+}
+
+// k (and v, may be null) rows [tokens][ld] with hkv heads of d values of esz bytes -> page pools
+B200_API int b200_kv_store(const void* k, const void* v, void* k_cache, void* v_cache, const long long* slots, int tokens,
+                           int hkv, int d, int page, long long ld, int esz, cudaStream_t stream) {
+  if (tokens <= 0) return 0;
+  if (d * esz % 16 || ld * esz % 16 || ((reinterpret_cast<uintptr_t>(k) | reinterpret_cast<uintptr_t>(v)) & 15)) return -2;
+  const int vecs = d * esz / 16;
+  const long long total = static_cast<long long>(tokens) * hkv * vecs;
+  const cudaError_t e = launch_pdl(kv_store_kernel, dim3(static_cast<unsigned>((total + 255) / 256)), dim3(256), 0, stream,
+                                   static_cast<const uint8_t*>(k), static_cast<const uint8_t*>(v),
+                                   static_cast<uint8_t*>(k_cache), static_cast<uint8_t*>(v_cache), slots, tokens, hkv, vecs,
+                                   page, ld * esz);
   return e == cudaSuccess ? 0 : -static_cast<int>(e) - 300;
 }

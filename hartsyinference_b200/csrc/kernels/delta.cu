@@ -1,0 +1,598 @@
+// Gated delta-rule mixer with one decay per head and key channel.
+//
+// Per head, with a state S [dk][dv] that is carried in fp32 from token to token of a sequence:
+//   S <- diag(g) S;   u = beta (v - S^T k);   S <- S + k u^T;   o = S^T q
+//   y = o / rms(o) * w * sigmoid(gate)
+// q, k, v come from projections through a short causal convolution and silu; q and k are made unit
+// vectors; g = exp(-A softplus(z + dt_bias)); several heads can share one q / k head.
+//
+//  * delta_prep     one warp per (token, head slice): convolution + silu, unit norms, decay, beta.
+//                   At decode it also advances the convolution state (the last taps - 1 inputs).
+//  * delta_tail     convolution state after a portion of a prompt.
+//  * delta_scan     portions of prompts: the columns of S are independent, so a block takes 32 of
+//                   them (a thread keeps two columns of an eighth of the rows in registers) and walks
+//                   over the tokens, which are staged through shared memory. The result does not
+//                   depend on where a prompt is cut: the same operations run in the same order.
+//  * delta_gate     the output norm and gate of a scanned portion, one warp per (token, head).
+//  * delta_step     decode: one block per (sequence, head) reads the state once, applies the update,
+//                   writes it back and emits the normed, gated output.
+//
+// State lives in slots, [slots][heads][dk][dv] fp32 and [slots][taps - 1][channels]; a sequence whose
+// portion starts at position 0 starts from zeros whatever its slot held before, a negative slot is
+// computed from zeros and stored nowhere (padding rows of a captured decode batch).
+#include "common.cuh"
+
+namespace b200 {
+
+typedef unsigned long long f32x2;   // two packed fp32 values
+
+__device__ __forceinline__ f32x2 pack2(float a, float b) {
+  f32x2 r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+  return r;
+}
+__device__ __forceinline__ void unpack2(f32x2 v, float& a, float& b) {
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(v));
+}
+__device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
+  f32x2 r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
+  f32x2 r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+__device__ __forceinline__ float sum2(f32x2 v) {
+  float a, b;
+  unpack2(v, a, b);
+  return a + b;
+}
+
+__device__ __forceinline__ void copy_async_16(uint32_t dst, const void* src, bool valid) {
+  const int sz = valid ? 16 : 0;
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(sz) : "memory");
+}
+__device__ __forceinline__ void copy_async_4(uint32_t dst, const void* src, bool valid) {
+  const int sz = valid ? 4 : 0;
+  asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;" ::"r"(dst), "l"(src), "r"(sz) : "memory");
+}
+
+template <typename T>
+__device__ __forceinline__ void ld4(const T* p, float (&v)[4]);
+template <>
+__device__ __forceinline__ void ld4<float>(const float* p, float (&v)[4]) {
+  const float4 a = *reinterpret_cast<const float4*>(p);
+  v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+}
+template <>
+__device__ __forceinline__ void ld4<__nv_bfloat16>(const __nv_bfloat16* p, float (&v)[4]) {
+  const uint2 raw = *reinterpret_cast<const uint2*>(p);
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+  const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+  v[0] = a.x; v[1] = a.y; v[2] = b.x; v[3] = b.y;
+}
+template <typename T>
+__device__ __forceinline__ void st4(T* p, const float (&v)[4]);
+template <>
+__device__ __forceinline__ void st4<float>(float* p, const float (&v)[4]) {
+  *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+}
+template <>
+__device__ __forceinline__ void st4<__nv_bfloat16>(__nv_bfloat16* p, const float (&v)[4]) {
+  *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]));
+}
+__device__ __forceinline__ float ld1(const float* p) { return *p; }
+__device__ __forceinline__ float ld1(const __nv_bfloat16* p) { return __bfloat162float(*p); }
+__device__ __forceinline__ float sigmoid_f32(float x) { return 1.f / (1.f + expf(-x)); }
+
+// exp(-y). The decays of a sequence multiply up over thousands of tokens, so near 1 the value is formed from
+// exp(-y) - 1, which leaves one unbiased rounding.
+__device__ __forceinline__ float decay_of(float y) { return y < 0.5f ? 1.f + expm1f(-y) : expf(-y); }
+
+struct DeltaParams {
+  const void* proj;          // [T][ldp]: q (hk * dk) | k (hk * dk) | v (h * dv) | ..., beta logits at b_off
+  const void* z;             // [T][ldz]: decay logits (h * dk), then output gate logits (h * dv) at gate_off
+  const float* conv_w;       // [channels][taps]
+  const float* a;            // [h] decay rate exp(A_log)
+  const float* dt_bias;      // [h * dk]
+  void* conv_state;          // [slots][taps - 1][channels]
+  float* state;              // [slots][h][dk][dv]
+  const __nv_bfloat16* norm_w;   // [dv]
+  const int* positions;      // [T]
+  const int* cu_q;           // [seqs + 1]; null: one token per sequence
+  const int* slots;          // [seqs]
+  float *q, *k, *v, *g, *beta, *o;   // scratch: [T][hk * dk] x 2, [T][h * dv], [T][h * dk], [T][h], [T][h * dv]
+  void* out;                 // [T][h * dv]
+  long long ldp, ldz;
+  int tokens, seqs, h, hk, dk, dv, taps, b_off, gate_off, dv_true;
+  float q_scale, eps;
+};
+
+__device__ __forceinline__ int seq_of_token(const int* cu, int seqs, int t) {
+  int lo = 0, hi = seqs - 1;
+  while (lo < hi) {
+    const int mid = (lo + hi + 1) >> 1;
+    if (cu[mid] <= t) lo = mid; else hi = mid - 1;
+  }
+  return lo;
+}
+
+constexpr int kDeltaMaxDk = 256;
+
+// grid: (ceil(T / 8), 2 hk + 2 h); 256 threads, warp w handles token 8 * blockIdx.x + w
+template <typename T>
+__global__ void __launch_bounds__(256) delta_prep_kernel(const DeltaParams p) {
+  pdl_wait();
+  pdl_trigger();
+  const int t = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (t >= p.tokens) return;
+  const T* row = static_cast<const T*>(p.proj) + static_cast<long long>(t) * p.ldp;
+  int slice = blockIdx.y;
+  if (slice >= 2 * p.hk + p.h) {          // decay (and beta) of one head
+    const int head = slice - 2 * p.hk - p.h;
+    const float a = p.a[head];
+    const T* zr = static_cast<const T*>(p.z) + static_cast<long long>(t) * p.ldz + head * p.dk;
+    float* gr = p.g + (static_cast<long long>(t) * p.h + head) * p.dk;
+    for (int e = lane * 4; e < p.dk; e += 128) {
+      float z[4], b[4], g[4];
+      ld4(zr + e, z);
+      ld4(p.dt_bias + head * p.dk + e, b);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const float x = z[j] + b[j];
+        g[j] = decay_of(a * (fmaxf(x, 0.f) + log1pf(expf(-fabsf(x)))));
+      }
+      st4(gr + e, g);
+    }
+    if (lane == 0) p.beta[static_cast<long long>(t) * p.h + head] = sigmoid_f32(ld1(row + p.b_off + head));
+    return;
+  }
+  const bool is_v = slice >= 2 * p.hk;
+  const int d = is_v ? p.dv : p.dk;
+  const int c0 = is_v ? 2 * p.hk * p.dk + (slice - 2 * p.hk) * p.dv : slice * p.dk;
+  const int channels = 2 * p.hk * p.dk + p.h * p.dv;
+  const int tail = p.taps - 1;
+  const int seq = p.cu_q ? seq_of_token(p.cu_q, p.seqs, t) : t;
+  const int first = p.cu_q ? p.cu_q[seq] : t;
+  const int slot = p.slots[seq];
+  const bool carried = slot >= 0 && p.positions[first] > 0;
+  T* st = static_cast<T*>(p.conv_state) + static_cast<long long>(slot < 0 ? 0 : slot) * tail * channels;
+  const bool shift = p.cu_q == nullptr && slot >= 0;
+  float keep[kDeltaMaxDk / 128][4];
+  float sq = 0.f;
+  int it = 0;
+  for (int e = lane * 4; e < d; e += 128, ++it) {
+    float acc[4] = {0.f, 0.f, 0.f, 0.f};
+    for (int j = 0; j < p.taps; ++j) {
+      const int src = t - tail + j;                  // token whose input this tap reads
+      float x[4] = {0.f, 0.f, 0.f, 0.f};
+      if (src >= first) ld4(row + static_cast<long long>(src - t) * p.ldp + c0 + e, x);
+      else if (carried) ld4(st + static_cast<long long>(tail + src - first) * channels + c0 + e, x);
+      // decode: input j becomes row j - 1 of the state (row j has been read already)
+      if (shift && j > 0) st4(st + static_cast<long long>(j - 1) * channels + c0 + e, x);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) acc[i] += x[i] * p.conv_w[(c0 + e + i) * p.taps + j];
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i) acc[i] = acc[i] * sigmoid_f32(acc[i]);
+    if (is_v) {
+      st4(p.v + static_cast<long long>(t) * p.h * p.dv + (c0 - 2 * p.hk * p.dk) + e, acc);
+    } else {
+#pragma unroll
+      for (int n = 0; n < kDeltaMaxDk / 128; ++n)
+        if (n == it)
+#pragma unroll
+          for (int i = 0; i < 4; ++i) keep[n][i] = acc[i];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) sq += acc[i] * acc[i];
+    }
+  }
+  if (is_v) return;
+  sq = warp_sum(sq);
+  const bool is_q = slice < p.hk;
+  const float inv = (is_q ? p.q_scale : 1.f) / sqrtf(sq + 1e-6f);
+  float* dst = (is_q ? p.q + static_cast<long long>(t) * p.hk * p.dk + slice * p.dk
+                     : p.k + static_cast<long long>(t) * p.hk * p.dk + (slice - p.hk) * p.dk);
+#pragma unroll
+  for (int n = 0; n < kDeltaMaxDk / 128; ++n) {
+    const int e = lane * 4 + n * 128;
+    if (e < d) {
+      float v[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) v[i] = keep[n][i] * inv;
+      st4(dst + e, v);
+    }
+  }
+}
+
+// grid: (ceil(channels / 256), seqs)
+template <typename T>
+__global__ void __launch_bounds__(256) delta_tail_kernel(const DeltaParams p) {
+  pdl_wait();
+  pdl_trigger();
+  const int channels = 2 * p.hk * p.dk + p.h * p.dv;
+  const int c = blockIdx.x * 256 + threadIdx.x, seq = blockIdx.y;
+  const int slot = p.slots[seq];
+  if (c >= channels || slot < 0) return;
+  const int first = p.cu_q[seq], len = p.cu_q[seq + 1] - first, tail = p.taps - 1;
+  if (len <= 0) return;
+  const bool carried = p.positions[first] > 0;
+  T* st = static_cast<T*>(p.conv_state) + static_cast<long long>(slot) * tail * channels + c;
+  const T* x = static_cast<const T*>(p.proj) + static_cast<long long>(first) * p.ldp + c;
+  for (int j = 0; j < tail; ++j) {
+    const int src = len - tail + j;      // row j + len of the old state when negative
+    T v = static_cast<T>(0.f);
+    if (src >= 0) v = x[static_cast<long long>(src) * p.ldp];
+    else if (carried) v = st[static_cast<long long>(tail + src) * channels];
+    st[static_cast<long long>(j) * channels] = v;
+  }
+}
+
+constexpr int kScanTokens = 16;     // tokens per staging buffer
+constexpr int kScanCols = 32;       // columns of S per block
+
+// grid: (ceil(dv / 32), h, seqs), 128 threads. dk = 32 * NR. Lane: rows i * 32 + (lane % 8) * 4 + 0..3
+// of columns 2 * (lane / 8), + 1 of the warp's eight.
+template <int NR>
+__global__ void __launch_bounds__(128) delta_scan_kernel(const DeltaParams p) {
+  pdl_wait();
+  pdl_trigger();
+  constexpr int DK = NR * 32;
+  constexpr int kTok = 3 * DK + kScanCols + 4;      // floats per staged token: k, q, g, v, beta
+  extern __shared__ __align__(16) float sm[];
+  const int head = blockIdx.y, seq = blockIdx.z, tid = threadIdx.x;
+  const int warp = tid >> 5, lane = tid & 31, rg = lane & 7;
+  const int col0 = blockIdx.x * kScanCols, lc = warp * 8 + (lane >> 3) * 2, col = col0 + lc;
+  const int first = p.cu_q ? p.cu_q[seq] : seq;
+  const int len = p.cu_q ? p.cu_q[seq + 1] - first : 1;
+  if (len <= 0) return;
+  const int slot = p.slots[seq];
+  const bool carried = slot >= 0 && p.positions[first] > 0;
+  const bool live = col < p.dv;
+  const int kh = head / (p.h / p.hk);
+  float* sp = p.state + (static_cast<long long>(slot < 0 ? 0 : slot) * p.h + head) * DK * p.dv + col;
+
+  f32x2 s0[NR * 2], s1[NR * 2];       // two columns, row pairs
+#pragma unroll
+  for (int i = 0; i < NR; ++i)
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      float2 a = make_float2(0.f, 0.f), b = a;
+      if (carried && live) {
+        const float* rp = sp + static_cast<long long>(i * 32 + rg * 4 + j * 2) * p.dv;
+        a = *reinterpret_cast<const float2*>(rp);
+        b = *reinterpret_cast<const float2*>(rp + p.dv);
+      }
+      s0[i * 2 + j] = pack2(a.x, b.x);
+      s1[i * 2 + j] = pack2(a.y, b.y);
+    }
+
+  auto stage = [&](int t0, int buf) {
+    float* base = sm + buf * kScanTokens * kTok;
+    const int n = min(kScanTokens, len - t0);
+    constexpr int kVec = DK / 4;
+    for (int i = tid; i < n * 3 * kVec; i += 128) {
+      const int tk = i / (3 * kVec), r = i - tk * (3 * kVec), which = r / kVec, c = (r - which * kVec) * 4;
+      const long long t = first + t0 + tk;
+      const float* src = which == 0 ? p.k + (t * p.hk + kh) * DK + c
+                       : which == 1 ? p.q + (t * p.hk + kh) * DK + c : p.g + (t * p.h + head) * DK + c;
+      copy_async_16(smem_u32(base + tk * kTok + which * DK + c), src, true);
+    }
+    for (int i = tid; i < n * (kScanCols / 4); i += 128) {
+      const int tk = i / (kScanCols / 4), c = (i % (kScanCols / 4)) * 4;
+      const long long t = first + t0 + tk;
+      const bool ok = col0 + c < p.dv;
+      copy_async_16(smem_u32(base + tk * kTok + 3 * DK + c), ok ? p.v + (t * p.h + head) * p.dv + col0 + c : p.v, ok);
+    }
+    if (tid < n) {
+      const long long t = first + t0 + tid;
+      copy_async_4(smem_u32(base + tid * kTok + 3 * DK + kScanCols), p.beta + t * p.h + head, true);
+    }
+  };
+  auto commit = [] { asm volatile("cp.async.commit_group;" ::: "memory"); };
+
+  stage(0, 0);
+  commit();
+  int buf = 0;
+  for (int t0 = 0; t0 < len; t0 += kScanTokens, buf ^= 1) {
+    if (t0 + kScanTokens < len) stage(t0 + kScanTokens, buf ^ 1);
+    commit();
+    asm volatile("cp.async.wait_group 1;" ::: "memory");
+    __syncthreads();
+    const int n = min(kScanTokens, len - t0);
+    const float* base = sm + buf * kScanTokens * kTok;
+    float* op = p.o + (static_cast<long long>(first + t0) * p.h + head) * p.dv + col;
+#pragma unroll 2
+    for (int tk = 0; tk < n; ++tk) {
+      const float* tb = base + tk * kTok;
+      f32x2 kk[NR * 2];
+      f32x2 a0 = 0, a1 = 0, b0 = 0, b1 = 0;
+#pragma unroll
+      for (int i = 0; i < NR; ++i) {
+        const ulonglong2 kv = *reinterpret_cast<const ulonglong2*>(tb + i * 32 + rg * 4);
+        const ulonglong2 gv = *reinterpret_cast<const ulonglong2*>(tb + 2 * DK + i * 32 + rg * 4);
+        kk[i * 2] = kv.x;
+        kk[i * 2 + 1] = kv.y;
+        s0[i * 2] = mul2(s0[i * 2], gv.x);
+        s1[i * 2] = mul2(s1[i * 2], gv.x);
+        s0[i * 2 + 1] = mul2(s0[i * 2 + 1], gv.y);
+        s1[i * 2 + 1] = mul2(s1[i * 2 + 1], gv.y);
+        a0 = fma2(s0[i * 2], kv.x, a0);
+        a1 = fma2(s1[i * 2], kv.x, a1);
+        b0 = fma2(s0[i * 2 + 1], kv.y, b0);
+        b1 = fma2(s1[i * 2 + 1], kv.y, b1);
+      }
+      float r0 = sum2(a0) + sum2(b0), r1 = sum2(a1) + sum2(b1);
+#pragma unroll
+      for (int o = 1; o < 8; o <<= 1) {
+        r0 += __shfl_xor_sync(0xffffffffu, r0, o);
+        r1 += __shfl_xor_sync(0xffffffffu, r1, o);
+      }
+      const float2 v = *reinterpret_cast<const float2*>(tb + 3 * DK + lc);
+      const float beta = tb[3 * DK + kScanCols];
+      const float u0 = beta * (v.x - r0), u1 = beta * (v.y - r1);
+      const f32x2 uu0 = pack2(u0, u0), uu1 = pack2(u1, u1);
+      a0 = a1 = b0 = b1 = 0;
+#pragma unroll
+      for (int i = 0; i < NR; ++i) {
+        const ulonglong2 qv = *reinterpret_cast<const ulonglong2*>(tb + DK + i * 32 + rg * 4);
+        s0[i * 2] = fma2(kk[i * 2], uu0, s0[i * 2]);
+        s1[i * 2] = fma2(kk[i * 2], uu1, s1[i * 2]);
+        s0[i * 2 + 1] = fma2(kk[i * 2 + 1], uu0, s0[i * 2 + 1]);
+        s1[i * 2 + 1] = fma2(kk[i * 2 + 1], uu1, s1[i * 2 + 1]);
+        a0 = fma2(s0[i * 2], qv.x, a0);
+        a1 = fma2(s1[i * 2], qv.x, a1);
+        b0 = fma2(s0[i * 2 + 1], qv.y, b0);
+        b1 = fma2(s1[i * 2 + 1], qv.y, b1);
+      }
+      r0 = sum2(a0) + sum2(b0);
+      r1 = sum2(a1) + sum2(b1);
+#pragma unroll
+      for (int o = 1; o < 8; o <<= 1) {
+        r0 += __shfl_xor_sync(0xffffffffu, r0, o);
+        r1 += __shfl_xor_sync(0xffffffffu, r1, o);
+      }
+      if (rg == 0 && live) *reinterpret_cast<float2*>(op + static_cast<long long>(tk) * p.h * p.dv) = make_float2(r0, r1);
+    }
+    __syncthreads();
+  }
+  if (slot >= 0 && live) {
+#pragma unroll
+    for (int i = 0; i < NR; ++i)
+#pragma unroll
+      for (int j = 0; j < 2; ++j) {
+        float2 a, b;
+        unpack2(s0[i * 2 + j], a.x, b.x);
+        unpack2(s1[i * 2 + j], a.y, b.y);
+        float* rp = sp + static_cast<long long>(i * 32 + rg * 4 + j * 2) * p.dv;
+        *reinterpret_cast<float2*>(rp) = a;
+        *reinterpret_cast<float2*>(rp + p.dv) = b;
+      }
+  }
+}
+
+// One warp per (token, head): out = o / rms(o) * w * sigmoid(gate)
+template <typename T>
+__global__ void __launch_bounds__(256) delta_gate_kernel(const DeltaParams p) {
+  pdl_wait();
+  pdl_trigger();
+  const long long w = static_cast<long long>(blockIdx.x) * 8 + (threadIdx.x >> 5);
+  const int lane = threadIdx.x & 31;
+  if (w >= static_cast<long long>(p.tokens) * p.h) return;
+  const int head = static_cast<int>(w % p.h);
+  const long long t = w / p.h;
+  const float* o = p.o + w * p.dv;
+  float sq = 0.f;
+  for (int e = lane * 4; e < p.dv; e += 128) {
+    float v[4];
+    ld4(o + e, v);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) sq += v[i] * v[i];
+  }
+  const float inv = 1.f / sqrtf(warp_sum(sq) / p.dv_true + p.eps);
+  const T* gr = static_cast<const T*>(p.z) + t * p.ldz + p.gate_off + head * p.dv;
+  T* out = static_cast<T*>(p.out) + w * p.dv;
+  for (int e = lane * 4; e < p.dv; e += 128) {
+    float v[4], g[4], n[4];
+    ld4(o + e, v);
+    ld4(gr + e, g);
+    ld4(p.norm_w + e, n);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) v[i] = v[i] * inv * n[i] * sigmoid_f32(g[i]);
+    st4(out + e, v);
+  }
+}
+
+// Decode. grid: (h, seqs); threads = (dv / 4) * ceil(dk / NRT): thread (cg, rg) owns four columns of
+// NRT rows. Dynamic shared memory: (3 dk + (rgs + 1) dv + 32) floats.
+constexpr int kStepThreads = 768;   // most threads of a decode block; larger heads are scanned
+
+template <typename T, int NRT>
+__global__ void __launch_bounds__(kStepThreads) delta_step_kernel(const DeltaParams p) {
+  extern __shared__ __align__(16) float sm[];
+  const int head = blockIdx.x, seq = blockIdx.y, tid = threadIdx.x;
+  const int cgs = p.dv >> 2, cg = tid % cgs, rg = tid / cgs, rgs = blockDim.x / cgs;
+  const bool worker = rg < rgs;
+  const int slot = p.slots[seq];
+  const bool carried = slot >= 0 && p.positions[seq] > 0;
+  float4* sp = reinterpret_cast<float4*>(p.state + (static_cast<long long>(slot < 0 ? 0 : slot) * p.h + head) * p.dk * p.dv) + cg;
+  // the state was last written by an earlier step, not by the kernel right before this one: its load
+  // does not have to wait for that kernel
+  float4 s[NRT];
+#pragma unroll
+  for (int i = 0; i < NRT; ++i) {
+    const int r = rg * NRT + i;
+    s[i] = carried && worker && r < p.dk ? sp[static_cast<long long>(r) * cgs] : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  pdl_wait();
+  pdl_trigger();
+  float *ks = sm, *qs = sm + p.dk, *gs = sm + 2 * p.dk, *us = sm + 3 * p.dk, *part = us + p.dv, *red = part + rgs * p.dv;
+  const int kh = head / (p.h / p.hk);
+  const long long kb = (static_cast<long long>(seq) * p.hk + kh) * p.dk, gb = (static_cast<long long>(seq) * p.h + head) * p.dk;
+  for (int i = tid; i < p.dk; i += blockDim.x) {
+    ks[i] = p.k[kb + i];
+    qs[i] = p.q[kb + i];
+    gs[i] = p.g[gb + i];
+  }
+  __syncthreads();
+  if (worker) {
+    float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int i = 0; i < NRT; ++i) {
+      const int r = rg * NRT + i;
+      if (r < p.dk) {
+        const float g = gs[r], k = ks[r];
+        s[i].x *= g; s[i].y *= g; s[i].z *= g; s[i].w *= g;
+        a.x += s[i].x * k; a.y += s[i].y * k; a.z += s[i].z * k; a.w += s[i].w * k;
+      }
+    }
+    reinterpret_cast<float4*>(part + rg * p.dv)[cg] = a;
+  }
+  __syncthreads();
+  const long long ob = (static_cast<long long>(seq) * p.h + head) * p.dv;
+  for (int c = tid; c < p.dv; c += blockDim.x) {
+    float m = 0.f;
+    for (int r = 0; r < rgs; ++r) m += part[r * p.dv + c];
+    us[c] = p.beta[static_cast<long long>(seq) * p.h + head] * (p.v[ob + c] - m);
+  }
+  __syncthreads();
+  if (worker) {
+    const float4 u = reinterpret_cast<const float4*>(us)[cg];
+    float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int i = 0; i < NRT; ++i) {
+      const int r = rg * NRT + i;
+      if (r < p.dk) {
+        const float k = ks[r], q = qs[r];
+        s[i].x += k * u.x; s[i].y += k * u.y; s[i].z += k * u.z; s[i].w += k * u.w;
+        a.x += s[i].x * q; a.y += s[i].y * q; a.z += s[i].z * q; a.w += s[i].w * q;
+        if (slot >= 0) sp[static_cast<long long>(r) * cgs] = s[i];
+      }
+    }
+    reinterpret_cast<float4*>(part + rg * p.dv)[cg] = a;
+  }
+  __syncthreads();
+  // blockDim >= dv: one thread per output value
+  float o = 0.f;
+  if (tid < p.dv)
+    for (int r = 0; r < rgs; ++r) o += part[r * p.dv + tid];
+  float sq = warp_sum(tid < p.dv ? o * o : 0.f);
+  if ((tid & 31) == 0) red[tid >> 5] = sq;
+  __syncthreads();
+  if (tid < p.dv) {
+    sq = 0.f;
+    for (int i = 0; i * 32 < p.dv; ++i) sq += red[i];
+    const float gate = ld1(static_cast<const T*>(p.z) + seq * p.ldz + p.gate_off + head * p.dv + tid);
+    const float y = o / sqrtf(sq / p.dv_true + p.eps) * __bfloat162float(p.norm_w[tid]) * sigmoid_f32(gate);
+    static_cast<T*>(p.out)[ob + tid] = static_cast<T>(y);
+  }
+}
+
+template <int NR>
+cudaError_t launch_scan(const DeltaParams& p, cudaStream_t stream) {
+  const int smem = 2 * kScanTokens * (3 * NR * 32 + kScanCols + 4) * 4;
+  static PerDeviceOnce once;
+  if (once.first_time()) cudaFuncSetAttribute(delta_scan_kernel<NR>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+  return launch_pdl(delta_scan_kernel<NR>, dim3((p.dv + kScanCols - 1) / kScanCols, p.h, p.seqs), dim3(128), smem, stream, p);
+}
+
+template <typename T, int NRT>
+cudaError_t launch_step(const DeltaParams& p, int threads, cudaStream_t stream) {
+  const int rgs = threads / (p.dv / 4);
+  const int smem = (3 * p.dk + (rgs + 1) * p.dv + 32) * 4;
+  static PerDeviceOnce once;
+  if (once.first_time()) cudaFuncSetAttribute(delta_step_kernel<T, NRT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024);
+  return launch_pdl(delta_step_kernel<T, NRT>, dim3(p.h, p.seqs), dim3(threads), smem, stream, p);
+}
+
+template <typename T>
+int delta_impl(const DeltaParams& p, cudaStream_t stream) {
+  const bool decode = p.cu_q == nullptr;
+  cudaError_t e = launch_pdl(delta_prep_kernel<T>, dim3((p.tokens + 7) / 8, 2 * p.hk + 2 * p.h), dim3(256), 0, stream, p);
+  if (e != cudaSuccess) return -static_cast<int>(e) - 300;
+  if (decode) {
+    const int cgs = p.dv / 4;
+    int nrt = 8;
+    int threads = cgs * ((p.dk + nrt - 1) / nrt);
+    while (nrt > 2 && threads < 128) { nrt /= 2; threads = cgs * ((p.dk + nrt - 1) / nrt); }
+    if (threads < p.dv) threads = p.dv;
+    threads = (threads + 31) / 32 * 32;
+    if (threads <= kStepThreads) {
+      switch (nrt) {
+        case 8: e = launch_step<T, 8>(p, threads, stream); break;
+        case 4: e = launch_step<T, 4>(p, threads, stream); break;
+        default: e = launch_step<T, 2>(p, threads, stream); break;
+      }
+      return e == cudaSuccess ? 0 : -static_cast<int>(e) - 300;
+    }
+  } else {
+    if (p.taps > 1) {
+      const int channels = 2 * p.hk * p.dk + p.h * p.dv;
+      e = launch_pdl(delta_tail_kernel<T>, dim3((channels + 255) / 256, p.seqs), dim3(256), 0, stream, p);
+      if (e != cudaSuccess) return -static_cast<int>(e) - 300;
+    }
+  }
+  switch (p.dk / 32) {
+    case 1: e = launch_scan<1>(p, stream); break;
+    case 2: e = launch_scan<2>(p, stream); break;
+    case 3: e = launch_scan<3>(p, stream); break;
+    case 4: e = launch_scan<4>(p, stream); break;
+    case 5: e = launch_scan<5>(p, stream); break;
+    case 6: e = launch_scan<6>(p, stream); break;
+    case 7: e = launch_scan<7>(p, stream); break;
+    default: e = launch_scan<8>(p, stream); break;
+  }
+  if (e != cudaSuccess) return -static_cast<int>(e) - 300;
+  const long long warps = static_cast<long long>(p.tokens) * p.h;
+  e = launch_pdl(delta_gate_kernel<T>, dim3(static_cast<unsigned>((warps + 7) / 8)), dim3(256), 0, stream, p);
+  return e == cudaSuccess ? 0 : -static_cast<int>(e) - 300;
+}
+
+}  // namespace b200
+
+using namespace b200;
+
+// fp32 scratch of one call, in bytes (q, k, v, g, beta, o)
+B200_API long long b200_delta_workspace_bytes(int tokens, int h, int hk, int dk, int dv) {
+  const long long per = 2ll * hk * dk + 2ll * h * dv + static_cast<long long>(h) * dk + (h + 3) / 4 * 4;
+  return per * tokens * 4;
+}
+
+// Number of kernels one call launches (for the launch count)
+B200_API int b200_delta_launches(int decode, int taps, int dk, int dv) {
+  if (decode) return (dv / 4) * ((dk + 7) / 8) <= kStepThreads && dv <= kStepThreads ? 2 : 3;
+  return taps > 1 ? 4 : 3;
+}
+
+// See the header comment and DeltaParams. dk (<= 256) a multiple of 32, dv a multiple of 8; dk_true /
+// dv_true are the sizes before padding (the q scale and the output norm use them; padded channels
+// carry zeros). cu_q null: one token per sequence (decode).
+B200_API int b200_delta(const void* proj, const void* z, const float* conv_w, const float* a, const float* dt_bias,
+                        void* conv_state, void* state, const void* norm_w, const int* positions, const int* cu_q,
+                        const int* slots, void* workspace, void* out, int tokens, int seqs, int h, int hk, int dk, int dv,
+                        int dk_true, int dv_true, int taps, long long ldp, int b_off, long long ldz, int gate_off, float eps,
+                        int f32, cudaStream_t stream) {
+  if (tokens <= 0 || seqs <= 0) return 0;
+  if (dk % 32 || dk < 32 || dk > kDeltaMaxDk || dv % 8 || dv < 8 || dv > 1024 || hk < 1 || h % hk || taps < 1) return -2;
+  if (ldp % 8 || ldz % 8 || gate_off % 8 || seqs > 65535 || h > 65535) return -2;
+  if (!cu_q && tokens != seqs) return -2;
+  DeltaParams p{};
+  p.proj = proj; p.z = z; p.conv_w = conv_w; p.a = a; p.dt_bias = dt_bias;
+  p.conv_state = conv_state; p.state = static_cast<float*>(state); p.norm_w = static_cast<const __nv_bfloat16*>(norm_w);
+  p.positions = positions; p.cu_q = cu_q; p.slots = slots;
+  p.out = out; p.ldp = ldp; p.ldz = ldz;
+  p.tokens = tokens; p.seqs = seqs; p.h = h; p.hk = hk; p.dk = dk; p.dv = dv; p.taps = taps; p.b_off = b_off;
+  p.gate_off = gate_off; p.dv_true = dv_true; p.eps = eps;
+  p.q_scale = 1.f / sqrtf(static_cast<float>(dk_true));
+  float* ws = static_cast<float*>(workspace);
+  const long long t = tokens;
+  p.q = ws; ws += t * hk * dk;
+  p.k = ws; ws += t * hk * dk;
+  p.v = ws; ws += t * h * dv;
+  p.g = ws; ws += t * h * dk;
+  p.o = ws; ws += t * h * dv;
+  p.beta = ws;
+  return f32 ? delta_impl<float>(p, stream) : delta_impl<__nv_bfloat16>(p, stream);
+}

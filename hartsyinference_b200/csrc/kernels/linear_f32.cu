@@ -1,0 +1,274 @@
+// Products that keep 32-bit results.
+//
+//  * b200_linear_f32: x (fp32 or bf16) times a bf16 weight, fp32 accumulation and output: the dense
+//    linears of a model that is run in 32 bits. Plain FMA tiles, no reduced-precision mode.
+//  * b200_router: router logits, scores and top-k of a mixture of experts in one kernel. The token
+//    rows of a block sit in shared memory as fp32, a warp takes four experts at a time, the logits
+//    stay in shared memory, and one warp per token turns them into scores and picks the experts.
+//  * b200_pair_linear_f32: one weight matrix per (token, choice) pair, the expert products of the
+//    32-bit mode.
+#include "common.cuh"
+
+namespace b200 {
+
+template <typename T>
+__device__ __forceinline__ float to_f32(T v);
+template <>
+__device__ __forceinline__ float to_f32<float>(float v) { return v; }
+template <>
+__device__ __forceinline__ float to_f32<__nv_bfloat16>(__nv_bfloat16 v) { return __bfloat162float(v); }
+
+// ------------------------------------------------------------------------------------------
+// dense
+// ------------------------------------------------------------------------------------------
+constexpr int kLT = 64, kLK = 16;
+
+template <typename T>
+__global__ void __launch_bounds__(256)
+linear_f32_kernel(const T* __restrict__ x, const __nv_bfloat16* __restrict__ w, const __nv_bfloat16* __restrict__ bias,
+                  float* __restrict__ out, int m, int n, int k, long long ldx, long long ldw, long long ldo) {
+  __shared__ float xs[kLK][kLT + 4], ws[kLK][kLT + 4];
+  const int m0 = blockIdx.y * kLT, n0 = blockIdx.x * kLT;
+  const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
+  float acc[4][4];
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
+  for (int k0 = 0; k0 < k; k0 += kLK) {
+    for (int i = tid; i < kLT * kLK; i += 256) {
+      const int r = i / kLK, c = i % kLK;
+      xs[c][r] = (m0 + r < m && k0 + c < k) ? to_f32(x[(m0 + r) * ldx + k0 + c]) : 0.f;
+      ws[c][r] = (n0 + r < n && k0 + c < k) ? __bfloat162float(w[(n0 + r) * ldw + k0 + c]) : 0.f;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int c = 0; c < kLK; ++c) {
+      const float4 a = *reinterpret_cast<const float4*>(&xs[c][ty * 4]);
+      const float4 b = *reinterpret_cast<const float4*>(&ws[c][tx * 4]);
+      const float av[4] = {a.x, a.y, a.z, a.w}, bv[4] = {b.x, b.y, b.z, b.w};
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] += av[i] * bv[j];
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const int r = m0 + ty * 4 + i;
+    if (r >= m) continue;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int c = n0 + tx * 4 + j;
+      if (c < n) out[r * ldo + c] = acc[i][j] + (bias ? __bfloat162float(bias[c]) : 0.f);
+    }
+  }
+}
+
+// ------------------------------------------------------------------------------------------
+// router
+// ------------------------------------------------------------------------------------------
+struct RouterParams {
+  const void* x;               // [tokens][ldx]
+  const __nv_bfloat16* w;      // [experts][ldw]
+  const float* bias;           // [experts] added to the scores for the choice only (may be null)
+  int* ids;                    // [tokens][top_k]
+  float* wts;                  // [tokens][top_k]
+  int tokens, experts, k, ldx, ldw, top_k, sigmoid, norm_topk;
+  float scale;
+};
+
+constexpr int kRouterExpertsPerWarp = 4;
+
+// kTok tokens per block; k is a multiple of 8. Dynamic shared memory: kTok * (k + experts) floats.
+template <typename T, int kTok>
+__global__ void __launch_bounds__(256) router_kernel(const RouterParams p) {
+  pdl_wait();
+  pdl_trigger();
+  extern __shared__ __align__(16) float sm[];
+  float* xs = sm;                       // [kTok][k]
+  float* lg = sm + kTok * p.k;          // [kTok][experts]
+  const int t0 = blockIdx.x * kTok;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+  for (int i = threadIdx.x; i < kTok * p.k; i += blockDim.x) {
+    const int r = i / p.k, c = i - r * p.k;
+    xs[i] = t0 + r < p.tokens ? to_f32(static_cast<const T*>(p.x)[static_cast<long long>(t0 + r) * p.ldx + c]) : 0.f;
+  }
+  __syncthreads();
+  for (int e0 = warp * kRouterExpertsPerWarp; e0 < p.experts; e0 += warps * kRouterExpertsPerWarp) {
+    float acc[kRouterExpertsPerWarp][kTok];
+#pragma unroll
+    for (int i = 0; i < kRouterExpertsPerWarp; ++i)
+#pragma unroll
+      for (int j = 0; j < kTok; ++j) acc[i][j] = 0.f;
+    for (int c = lane * 8; c < p.k; c += 256) {
+      float wv[kRouterExpertsPerWarp][8];
+#pragma unroll
+      for (int i = 0; i < kRouterExpertsPerWarp; ++i) {
+        const int e = e0 + i < p.experts ? e0 + i : p.experts - 1;
+        const uint4 raw = *reinterpret_cast<const uint4*>(p.w + static_cast<long long>(e) * p.ldw + c);
+        const __nv_bfloat162* b = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+        for (int q = 0; q < 4; ++q) {
+          const float2 f = __bfloat1622float2(b[q]);
+          wv[i][2 * q] = f.x;
+          wv[i][2 * q + 1] = f.y;
+        }
+      }
+#pragma unroll
+      for (int j = 0; j < kTok; ++j) {
+        const float4 a = *reinterpret_cast<const float4*>(xs + j * p.k + c);
+        const float4 b = *reinterpret_cast<const float4*>(xs + j * p.k + c + 4);
+#pragma unroll
+        for (int i = 0; i < kRouterExpertsPerWarp; ++i) {
+          acc[i][j] += a.x * wv[i][0] + a.y * wv[i][1] + a.z * wv[i][2] + a.w * wv[i][3];
+          acc[i][j] += b.x * wv[i][4] + b.y * wv[i][5] + b.z * wv[i][6] + b.w * wv[i][7];
+        }
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < kRouterExpertsPerWarp; ++i)
+#pragma unroll
+      for (int j = 0; j < kTok; ++j) {
+        const float s = warp_sum(acc[i][j]);
+        if (lane == 0 && e0 + i < p.experts) lg[j * p.experts + e0 + i] = s;
+      }
+  }
+  __syncthreads();
+  for (int j = warp; j < kTok; j += warps) {
+    const int t = t0 + j;
+    if (t >= p.tokens) continue;
+    float* row = lg + j * p.experts;
+    if (p.sigmoid) {
+      for (int e = lane; e < p.experts; e += 32) row[e] = 1.f / (1.f + expf(-row[e]));
+    } else {
+      float mx = -INFINITY;
+      for (int e = lane; e < p.experts; e += 32) mx = fmaxf(mx, row[e]);
+      mx = warp_max(mx);
+      float s = 0.f;
+      for (int e = lane; e < p.experts; e += 32) {
+        const float v = expf(row[e] - mx);
+        row[e] = v;
+        s += v;
+      }
+      s = warp_sum(s);
+      for (int e = lane; e < p.experts; e += 32) row[e] /= s;
+    }
+    // top-k by score + bias, ties to the lowest index; a chosen expert's score is stored negated so
+    // that later rounds pass over it (scores are never negative)
+    float wsum = 0.f, my_w = 0.f;
+    int my_id = 0;
+    for (int r = 0; r < p.top_k; ++r) {
+      float best = -INFINITY, raw = 0.f;
+      int idx = 0x7fffffff;
+      for (int e = lane; e < p.experts; e += 32) {
+        const float s = row[e];
+        if (__float_as_uint(s) >> 31) continue;
+        const float v = s + (p.bias ? p.bias[e] : 0.f);
+        if (v > best) { best = v; idx = e; raw = s; }
+      }
+      for (int o = 16; o > 0; o >>= 1) {
+        const float ov = __shfl_xor_sync(0xffffffffu, best, o), orw = __shfl_xor_sync(0xffffffffu, raw, o);
+        const int oi = __shfl_xor_sync(0xffffffffu, idx, o);
+        if (ov > best || (ov == best && oi < idx)) { best = ov; idx = oi; raw = orw; }
+      }
+      if (idx >= p.experts) idx = r < p.experts ? r : 0;      // only with scores that are not numbers
+      if ((idx & 31) == lane) row[idx] = __uint_as_float(__float_as_uint(row[idx]) | 0x80000000u);
+      __syncwarp();
+      if (lane == r) { my_w = raw; my_id = idx; }
+      wsum += raw;
+    }
+    if (lane < p.top_k) {
+      p.ids[static_cast<long long>(t) * p.top_k + lane] = my_id;
+      p.wts[static_cast<long long>(t) * p.top_k + lane] = (p.norm_topk ? my_w / (wsum + 1e-20f) : my_w) * p.scale;
+    }
+  }
+}
+
+template <typename T>
+int launch_router(const RouterParams& p, cudaStream_t stream) {
+  const int limit = 200 * 1024;
+  auto bytes = [&](int tok) { return tok * (p.k + p.experts) * 4; };
+  // enough blocks to cover the machine first, then as many tokens per read of the weights as fit
+  int tok = p.tokens >= 4 * 148 ? 8 : p.tokens >= 2 * 148 ? 4 : p.tokens >= 148 ? 2 : 1;
+  while (tok > 1 && bytes(tok) > limit / 2) tok /= 2;
+  if (bytes(tok) > limit) return -2;
+  auto go = [&](auto kernel, int n, PerDeviceOnce& once) {
+    if (once.first_time()) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, limit);
+    return launch_pdl(kernel, dim3((p.tokens + n - 1) / n), dim3(256), bytes(n), stream, p);
+  };
+  static PerDeviceOnce once[4];
+  cudaError_t e;
+  switch (tok) {
+    case 8: e = go(router_kernel<T, 8>, 8, once[3]); break;
+    case 4: e = go(router_kernel<T, 4>, 4, once[2]); break;
+    case 2: e = go(router_kernel<T, 2>, 2, once[1]); break;
+    default: e = go(router_kernel<T, 1>, 1, once[0]); break;
+  }
+  return e == cudaSuccess ? 0 : -static_cast<int>(e) - 300;
+}
+
+// out[pair][j] = x[pair / div] . w[ids[pair]][j] for ids below `experts` (other pairs are skipped).
+// One warp per output feature, eight features per block.
+__global__ void __launch_bounds__(256)
+pair_linear_f32_kernel(const float* __restrict__ x, const __nv_bfloat16* __restrict__ w, const int* __restrict__ ids,
+                       float* __restrict__ out, int div, int experts, int n, int k, long long ldx, long long ldo) {
+  const int pair = blockIdx.y, e = ids[pair];
+  if (e < 0 || e >= experts) return;
+  const int j = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (j >= n) return;
+  const float* xr = x + static_cast<long long>(pair / div) * ldx;
+  const __nv_bfloat16* wr = w + (static_cast<long long>(e) * n + j) * k;
+  float s = 0.f;
+  for (int c = lane; c < k; c += 32) s += xr[c] * __bfloat162float(wr[c]);
+  s = warp_sum(s);
+  if (lane == 0) out[static_cast<long long>(pair) * ldo + j] = s;
+}
+
+}  // namespace b200
+
+using namespace b200;
+
+B200_API int b200_linear_f32(const void* x, int x_f32, const void* w, const void* bias, void* out, int m, int n, int k,
+                             long long ldx, long long ldw, long long ldo, cudaStream_t stream) {
+  if (m <= 0 || n <= 0) return 0;
+  const dim3 grid((n + kLT - 1) / kLT, (m + kLT - 1) / kLT);
+  if (grid.y > 65535) return -2;
+  const auto* wp = static_cast<const __nv_bfloat16*>(w);
+  const auto* bp = static_cast<const __nv_bfloat16*>(bias);
+  if (x_f32)
+    linear_f32_kernel<float><<<grid, 256, 0, stream>>>(static_cast<const float*>(x), wp, bp, static_cast<float*>(out), m, n, k,
+                                                       ldx, ldw, ldo);
+  else
+    linear_f32_kernel<__nv_bfloat16><<<grid, 256, 0, stream>>>(static_cast<const __nv_bfloat16*>(x), wp, bp,
+                                                               static_cast<float*>(out), m, n, k, ldx, ldw, ldo);
+  return cudaGetLastError() == cudaSuccess ? 0 : -300;
+}
+
+// ids / wts [tokens][top_k] from x [tokens][k] (fp32 or bf16) and the router weight [experts][k] bf16:
+// softmax or sigmoid scores in 32 bits, top-k by score + bias, weights = scores (optionally
+// renormalised) * scale. k a multiple of 8, top_k <= 32.
+B200_API int b200_router(const void* x, int x_f32, const void* w, const float* bias, int* ids, float* wts, int tokens,
+                         int experts, int k, int ldx, int ldw, int top_k, int sigmoid, int norm_topk, float scale,
+                         cudaStream_t stream) {
+  if (tokens <= 0) return 0;
+  if (k % 8 || ldw % 8 || top_k < 1 || top_k > 32 || top_k > experts) return -2;
+  RouterParams p{x, static_cast<const __nv_bfloat16*>(w), bias, ids, wts, tokens, experts, k, ldx, ldw, top_k, sigmoid,
+                 norm_topk, scale};
+  return x_f32 ? launch_router<float>(p, stream) : launch_router<__nv_bfloat16>(p, stream);
+}
+
+B200_API int b200_pair_linear_f32(const void* x, const void* w, const int* ids, void* out, int pairs, int div, int experts,
+                                  int n, int k, long long ldx, long long ldo, cudaStream_t stream) {
+  if (pairs <= 0 || n <= 0) return 0;
+  // the pair index is the grid's second dimension: run longer lists in slices (slices start on a token)
+  const int step = 65535 / div * div;
+  for (int p0 = 0; p0 < pairs; p0 += step) {
+    const int cnt = pairs - p0 < step ? pairs - p0 : step;
+    pair_linear_f32_kernel<<<dim3((n + 7) / 8, cnt), 256, 0, stream>>>(
+        static_cast<const float*>(x) + static_cast<long long>(p0 / div) * ldx, static_cast<const __nv_bfloat16*>(w), ids + p0,
+        static_cast<float*>(out) + static_cast<long long>(p0) * ldo, div, experts, n, k, ldx, ldo);
+  }
+  return cudaGetLastError() == cudaSuccess ? 0 : -300;
+}

@@ -123,6 +123,7 @@ __global__ void moe_route_kernel(const RouteParams p) {
       const float orw = __shfl_xor_sync(0xffffffffu, raw, o);
       if (ov > v || (ov == v && oi < idx)) { v = ov; idx = oi; raw = orw; }
     }
+    if (idx >= p.experts) idx = r < p.experts ? r : 0;   // only with scores that are not numbers
     if ((idx & 31) == lane) sel[idx >> 5] = -INFINITY;   // remove from further rounds
     if (lane == r) { my_w = raw; my_id = idx; }
     wsum += raw;
@@ -249,9 +250,56 @@ __global__ void moe_combine_kernel(const __nv_bfloat16* __restrict__ y, const in
   }
 }
 
+// Clamped gate of an expert: y = g sigmoid(alpha g) (u + 1), g = min(gate, limit), u = clamp(up, +-limit),
+// for x [rows][2 f] = gate | up. With a block list only the rows of the blocks in use are computed.
+template <typename T>
+__device__ __forceinline__ float glu_ld(const T* p) { return static_cast<float>(*p); }
+template <typename T>
+__global__ void __launch_bounds__(256) glu_clamped_kernel(const T* __restrict__ x, T* __restrict__ y, long long rows, int f,
+                                                          float limit, float alpha, const int* __restrict__ dyn_blocks, int cap) {
+  pdl_wait();
+  pdl_trigger();
+  if (dyn_blocks) {
+    const long long used = static_cast<long long>(*dyn_blocks) * cap;
+    rows = used < rows ? used : rows;
+  }
+  const int pairs = f >> 1;
+  const long long total = rows * pairs;
+  for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < total;
+       i += static_cast<long long>(gridDim.x) * blockDim.x) {
+    const long long r = i / pairs;
+    const int c = static_cast<int>(i - r * pairs) * 2;
+    const T* g = x + r * 2 * f + c;
+    float o[2];
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      const float a = fminf(glu_ld(g + j), limit), u = fminf(fmaxf(glu_ld(g + f + j), -limit), limit);
+      o[j] = a / (1.f + expf(-alpha * a)) * (u + 1.f);
+    }
+    y[r * f + c] = static_cast<T>(o[0]);
+    y[r * f + c + 1] = static_cast<T>(o[1]);
+  }
+}
+
 }  // namespace b200
 
 using namespace b200;
+
+// f even. dyn_blocks (may be null): only the first *dyn_blocks * cap rows are in use.
+B200_API int b200_glu_clamped(const void* x, void* y, long long rows, int f, float limit, float alpha, const int* dyn_blocks,
+                              int cap, int f32, cudaStream_t stream) {
+  if (rows <= 0) return 0;
+  if (f % 2) return -2;
+  long long blocks = (rows * (f / 2) + 255) / 256;
+  if (blocks > 148 * 16) blocks = 148 * 16;
+  const cudaError_t e =
+      f32 ? launch_pdl(glu_clamped_kernel<float>, dim3(static_cast<unsigned>(blocks)), dim3(256), 0, stream,
+                       static_cast<const float*>(x), static_cast<float*>(y), rows, f, limit, alpha, dyn_blocks, cap)
+          : launch_pdl(glu_clamped_kernel<__nv_bfloat16>, dim3(static_cast<unsigned>(blocks)), dim3(256), 0, stream,
+                       static_cast<const __nv_bfloat16*>(x), static_cast<__nv_bfloat16*>(y), rows, f, limit, alpha, dyn_blocks,
+                       cap);
+  return e == cudaSuccess ? 0 : -static_cast<int>(e) - 300;
+}
 
 B200_API int b200_moe_route(const void* logits, int logits_bf16, const float* bias, int* topk_ids, float* topk_w, int tokens,
                             int experts, int top_k, int n_group, int topk_group, int sigmoid, int norm_topk,

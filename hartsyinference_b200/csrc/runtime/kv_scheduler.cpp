@@ -1,7 +1,9 @@
 // Paged-KV block allocator and continuous-batching scheduler core (host side, no CUDA).
 //
 // The allocator hands out fixed-size KV pages from a free list, keeps one block table per
-// sequence and reference-counts pages so that a prompt prefix can be shared between sequences.
+// sequence and reference-counts pages so that a prompt prefix can be shared between sequences. For
+// models with recurrent state it also hands out state slots, one per sequence, taken with the first
+// page and given back with the pages (a pre-empted sequence loses both and is recomputed).
 // The scheduler decides, once per engine step, which waiting requests are admitted (prefill, in
 // chunks bounded by a token budget), which running sequences decode, and which running sequence is
 // pre-empted (pages released, request re-queued for recompute) when the pool runs dry.
@@ -27,6 +29,7 @@ namespace {
 struct Seq {
   std::vector<int32_t> blocks;
   int64_t tokens = 0;   // tokens whose KV is stored
+  int32_t slot = -1;    // recurrent-state slot
 };
 
 struct KvAllocator {
@@ -35,6 +38,8 @@ struct KvAllocator {
   std::vector<int32_t> free_list;     // stack: back() is handed out next
   std::vector<int32_t> refcount;
   std::unordered_map<int64_t, Seq> seqs;
+  int32_t num_slots = 0;              // 0: sequences need no slot
+  std::vector<int32_t> free_slots;    // stack
   int32_t fail_after = -1;            // fault injection: the N-th next allocation fails
   std::mutex mu;
 
@@ -66,6 +71,8 @@ struct KvAllocator {
       if (--refcount[b] == 0) free_list.push_back(b);
     s.blocks.clear();
     s.tokens = 0;
+    if (s.slot >= 0) free_slots.push_back(s.slot);
+    s.slot = -1;
   }
 };
 
@@ -119,7 +126,13 @@ B200_API int64_t b200_kv_append(void* h, int64_t seq, int32_t new_tokens) {
   std::lock_guard<std::mutex> g(a->mu);
   Seq& s = a->seqs[seq];
   const int32_t need = a->blocks_needed(s, new_tokens);
+  const bool need_slot = a->num_slots > 0 && s.slot < 0;
+  if (need_slot && a->free_slots.empty()) return -1;
   if (need > 0 && !a->take(s, need)) return -1;
+  if (need_slot) {
+    s.slot = a->free_slots.back();
+    a->free_slots.pop_back();
+  }
   s.tokens += new_tokens;
   return s.tokens;
 }
@@ -129,6 +142,7 @@ B200_API int32_t b200_kv_can_append(void* h, int64_t seq, int32_t new_tokens) {
   auto it = a->seqs.find(seq);
   Seq empty;
   const Seq& s = it == a->seqs.end() ? empty : it->second;
+  if (a->num_slots > 0 && s.slot < 0 && a->free_slots.empty()) return 0;
   return a->blocks_needed(s, new_tokens) <= static_cast<int32_t>(a->free_list.size()) ? 1 : 0;
 }
 // Drop the last tokens of a sequence (speculative-decode rollback); frees whole pages that empty.
@@ -139,6 +153,7 @@ B200_API int64_t b200_kv_truncate(void* h, int64_t seq, int64_t new_len) {
   if (it == a->seqs.end()) return -1;
   Seq& s = it->second;
   if (new_len < 0 || new_len > s.tokens) return -1;
+  if (a->num_slots > 0 && new_len != s.tokens) return -1;   // recurrent state cannot be rolled back
   const size_t keep = static_cast<size_t>((new_len + a->block_size - 1) / a->block_size);
   while (s.blocks.size() > keep) {
     const int32_t b = s.blocks.back();
@@ -162,6 +177,7 @@ B200_API int64_t b200_kv_fork_prefix(void* h, int64_t src, int64_t dst, int64_t 
   std::lock_guard<std::mutex> g(a->mu);
   auto it = a->seqs.find(src);
   if (it == a->seqs.end() || a->seqs.count(dst)) return -1;
+  if (a->num_slots > 0) return -1;                          // the state at the end of the prefix is not kept
   const int64_t pages = std::min<int64_t>(tokens, it->second.tokens) / a->block_size;
   Seq d;
   for (int64_t i = 0; i < pages; ++i) {
@@ -189,6 +205,25 @@ B200_API int32_t b200_kv_block_table(void* h, int64_t seq, int32_t* out, int32_t
   const int32_t n = static_cast<int32_t>(b.size());
   for (int32_t i = 0; i < cap; ++i) out[i] = i < n ? b[static_cast<size_t>(i)] : -1;
   return n;
+}
+// State slots (call before any sequence exists): slots 0..n-1, lowest handed out first.
+B200_API void b200_kv_set_slots(void* h, int32_t n) {
+  auto* a = static_cast<KvAllocator*>(h);
+  std::lock_guard<std::mutex> g(a->mu);
+  a->num_slots = n;
+  a->free_slots.clear();
+  for (int32_t i = n - 1; i >= 0; --i) a->free_slots.push_back(i);
+}
+B200_API int32_t b200_kv_seq_slot(void* h, int64_t seq) {
+  auto* a = static_cast<KvAllocator*>(h);
+  std::lock_guard<std::mutex> g(a->mu);
+  auto it = a->seqs.find(seq);
+  return it == a->seqs.end() ? -1 : it->second.slot;
+}
+B200_API int32_t b200_kv_num_free_slots(void* h) {
+  auto* a = static_cast<KvAllocator*>(h);
+  std::lock_guard<std::mutex> g(a->mu);
+  return static_cast<int32_t>(a->free_slots.size());
 }
 // Fault injection for tests: make the allocation that crosses `after_blocks` more blocks fail once.
 B200_API void b200_kv_inject_failure(void* h, int32_t after_blocks) {

@@ -3,6 +3,12 @@
 One engine step = ask the C++ scheduler core what to run, fill pinned host buffers with the batch
 metadata (token ids, positions, KV slots, block tables, lengths), copy them to the device, run the
 prefill chunk batch and/or the decode batch, sample, read the sampled ids back, update requests.
+Models with per-layer mixers run prompt chunks and decoded tokens of a step as ONE ragged batch
+(a decoded token is a chunk of one); a step with decoded tokens only replays a CUDA graph as for every
+other model. Recurrent models hold one state slot per running sequence (``KvAllocator.seq_slot``).
+
+``replay`` drives the same batches from token ids that the caller brings (no scheduler decisions, no
+sampling) and returns logits.
 
 Counterpart in the reference: ``DynamicBatchScheduler`` (SubmitAsync:153, RunLoopAsync:162-268,
 AdmitAndPrefill:311-383 prefills each request alone, RunDecodeRound:460-483 gathers pages per
@@ -83,12 +89,18 @@ class LLMEngine:
                     budget = int(free * 0.85)
                 else:
                     budget = 512 << 20      # the reference's default pool budget
-            num_pages = max(8, budget // per_page)
+            if getattr(model.cfg, "recurrent", False):
+                budget = max(budget - self.max_batch * model.state_bytes_per_slot(), 0)
+            num_pages = max(8, budget // max(per_page, 1))
             # no point in holding more pages than max_batch full-length sequences can use
             num_pages = min(num_pages, self.max_batch * self.max_pages_per_seq)
         self.num_pages = int(num_pages)
         model.alloc_kv(self.num_pages, self.page)
-        self.kv = KvAllocator(self.num_pages, self.page)
+        self.mixed = bool(getattr(model.cfg, "mixed_layers", False))
+        slots = self.max_batch if getattr(model.cfg, "recurrent", False) else 0
+        if slots:
+            model.alloc_state(slots)
+        self.kv = KvAllocator(self.num_pages, self.page, state_slots=slots)
         self.sched = SchedulerCore(self.kv, self.max_batch, self.prefill_chunk, 0, cap=max(1024, 2 * self.max_batch))
         self.requests: dict[int, Request] = {}
         self._next_id = 1
@@ -106,8 +118,8 @@ class LLMEngine:
         self._ev = (torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)) if self.cuda else None
         pin = self.cuda
         mp = self.max_pages_per_seq
-        cap_tokens = max(self.prefill_chunk, self.max_batch)
-        cap_seqs = max(self.max_batch, 1)
+        cap_tokens = self.prefill_chunk + _bucket(self.max_batch)
+        cap_seqs = _bucket(self.max_batch)
         # pinned host staging, reused every step
         self.h_tokens = torch.zeros(cap_tokens, dtype=torch.int32, pin_memory=pin)
         self.h_positions = torch.zeros(cap_tokens, dtype=torch.int32, pin_memory=pin)
@@ -116,6 +128,8 @@ class LLMEngine:
         self.h_kv_lens = torch.zeros(cap_seqs, dtype=torch.int32, pin_memory=pin)
         self.h_cu_q = torch.zeros(cap_seqs + 1, dtype=torch.int32, pin_memory=pin)
         self.h_rows = torch.zeros(cap_seqs, dtype=torch.int64, pin_memory=pin)
+        self.h_state = torch.full((cap_seqs,), -1, dtype=torch.int32, pin_memory=pin)
+        self._replays: dict[object, int] = {}
         self.h_out = torch.zeros(cap_seqs, dtype=torch.int32, pin_memory=pin)
         self.h_status = torch.zeros(4, dtype=torch.int32, pin_memory=pin)
         # called with [code, kernel, site, detail] when a kernel's bounded wait ran out, before the
@@ -198,23 +212,24 @@ class LLMEngine:
 
     def _fill_table(self, row: int, rid: int) -> None:
         self.kv.block_table_into(rid, self.h_table[row].data_ptr(), self.max_pages_per_seq)
+        if self.kv.state_slots:
+            self.h_state[row] = self.kv.seq_slot(rid)
 
     def _to_device(self, t: torch.Tensor, n: int) -> torch.Tensor:
         v = t[:n]
         self.h2d_bytes_last += v.numel() * v.element_size()
         return v.to(self.device, non_blocking=True) if self.cuda else v.clone()
 
-    def _run_prefill(self, chunks: list[tuple[int, int, int]]) -> list[tuple[Request, int]]:
-        """Runs one batch of prompt chunks. Returns [(request, sampled token)] for requests whose
-        prompt completed in this step."""
+    def _run_chunks(self, chunks: list[tuple[int, int, int]]) -> tuple[torch.Tensor, list[int]]:
+        """Runs one ragged batch of (request, start, count) token runs. Returns the final hidden states
+        of all their rows and the row at which every run ends."""
         page = self.page
         t = 0
-        sample_rows: list[tuple[int, Request]] = []
+        ends: list[int] = []
         max_q = max_kv = 0
         for i, (rid, start, count) in enumerate(chunks):
             req = self.requests[rid]
             toks = self._seq_tokens(req)
-            target = len(req.prompt) + len(req.output) - (1 if req.output else 0)
             self.h_tokens[t:t + count] = torch.tensor(toks[start:start + count], dtype=torch.int32)
             self.h_positions[t:t + count] = self._rope_positions(req, start, count)
             self._fill_table(i, rid)
@@ -224,9 +239,8 @@ class LLMEngine:
             self.h_kv_lens[i] = start + count
             max_q = max(max_q, count)
             max_kv = max(max_kv, start + count)
-            if start + count >= target:
-                sample_rows.append((t + count - 1, req))
             t += count
+            ends.append(t - 1)
         n = len(chunks)
         self.h_cu_q[n] = t
         embeds = None
@@ -250,21 +264,37 @@ class LLMEngine:
                              kv_lens=self._to_device(self.h_kv_lens, n), is_decode=False,
                              cu_q=self._to_device(self.h_cu_q, n + 1), max_q_len=max_q, max_kv_len=max_kv,
                              embeds=embeds, cross_states=self._cross_states([self.requests[rid] for rid, _, _ in chunks]),
-                             positions3=self._positions3(chunks), deepstack=self._deepstack(chunks, t))
-        hidden = self.model.forward_hidden(batch)
+                             positions3=self._positions3(chunks), deepstack=self._deepstack(chunks, t),
+                             state_slots=self._to_device(self.h_state, n) if self.kv.state_slots else None)
+        return self.model.forward_hidden(batch), ends
+
+    def _run_prefill(self, chunks: list[tuple[int, int, int]], decode: Sequence[int] = ()) -> list[tuple[Request, int]]:
+        """Runs one batch of prompt chunks, with the next token of the requests in ``decode`` as further
+        runs of one. Returns [(request, sampled token)] for requests whose prompt completed in this step
+        and for the decoded ones."""
+        runs = list(chunks)
+        for rid in decode:
+            req = self.requests[rid]
+            runs.append((rid, len(req.prompt) + len(req.output) - 1, 1))
+        hidden, ends = self._run_chunks(runs)
+        sample_rows: list[tuple[int, Request]] = []
+        rebuilt: list[Request] = []
+        for i, (rid, start, count) in enumerate(runs):
+            req = self.requests[rid]
+            target = len(req.prompt) + len(req.output) - (1 if req.output else 0)
+            if i >= len(chunks) or (start + count >= target and not req.output):
+                sample_rows.append((ends[i], req))
+            elif start + count >= target:
+                rebuilt.append(req)
         done: list[tuple[Request, int]] = []
-        fresh = [(row, req) for row, req in sample_rows if not req.output]
-        if fresh:
-            rows = torch.tensor([r for r, _ in fresh], dtype=torch.int64)
+        if sample_rows:
+            rows = torch.tensor([r for r, _ in sample_rows], dtype=torch.int64)
             rows_d = rows.to(self.device, non_blocking=True) if self.cuda else rows
             self.h2d_bytes_last += rows.numel() * 8
-            toks = self._sample(hidden[rows_d].contiguous(), [req for _, req in fresh])
-            done = [(req, tok) for (_, req), tok in zip(fresh, toks)]
+            toks = self._sample(hidden[rows_d].contiguous(), [req for _, req in sample_rows])
+            done = [(req, tok) for (_, req), tok in zip(sample_rows, toks)]
         # requests that re-computed their context after a pre-emption continue decoding without sampling
-        for row, req in sample_rows:
-            if req.output:
-                done.append((req, -1))
-        return done
+        return done + [(req, -1) for req in rebuilt]
 
     def _read_tokens(self, dev_tokens: torch.Tensor, n: int) -> list[int]:
         """Sampled ids and the kernels' status word come back in the same synchronising read. A
@@ -355,27 +385,36 @@ class LLMEngine:
             self.h_slots[i] = -1
             self.h_kv_lens[i] = 0
             self.h_table[i].zero_()
+            self.h_state[i] = -1
         return max_kv
 
     def _run_decode(self, rids: list[int]) -> list[int]:
         n = len(rids)
         reqs = [self.requests[r] for r in rids]
         greedy = all(not r.params.needs_logits for r in reqs)
-        if self.use_graphs and greedy and not self._graphs_disabled:
+        if self.use_graphs and (greedy or self.mixed) and not self._graphs_disabled:
             try:
-                return self._run_decode_graph(rids)
+                st, bucket = self._run_decode_graph(rids)
+                if greedy:
+                    return self._read_tokens(st["out"], bucket)[:n]
+                return self._sample(st["hidden"][:n], reqs)
             except HartsyInferenceError:
                 raise
             except Exception as e:  # capture failure -> circuit breaker, fall back to eager
                 self._graphs_disabled = True
                 log.warn(f"[Engine] CUDA graph decode disabled after failure: {e}")
-        max_kv = self._decode_batch_tensors(rids, n)
+        return self._sample(self._run_decode_eager(rids), reqs)
+
+    def _run_decode_eager(self, rids: list[int]) -> torch.Tensor:
+        n = len(rids)
+        reqs = [self.requests[r] for r in rids]
+        self._decode_batch_tensors(rids, n)
         batch = ForwardBatch(tokens=self._to_device(self.h_tokens, n), positions=self._to_device(self.h_positions, n),
                              slot_mapping=self._to_device(self.h_slots, n), block_table=self._to_device(self.h_table, n),
                              kv_lens=self._to_device(self.h_kv_lens, n), is_decode=True, max_kv_len=self.max_model_len,
-                             cross_states=self._cross_states(reqs))
-        hidden = self.model.forward_hidden(batch)
-        return self._sample(hidden, reqs)
+                             cross_states=self._cross_states(reqs),
+                             state_slots=self._to_device(self.h_state, n) if self.kv.state_slots else None)
+        return self.model.forward_hidden(batch)
 
     @staticmethod
     def _rope_positions(req: "Request", start: int, count: int) -> torch.Tensor:
@@ -426,7 +465,9 @@ class LLMEngine:
             return None
         return [r.cross_states for r in reqs]
 
-    def _run_decode_graph(self, rids: list[int]) -> list[int]:
+    def _run_decode_graph(self, rids: list[int]) -> tuple[dict, int]:
+        """Replays the captured decode step of the batch's bucket; its results are in the returned static
+        tensors (``out``: greedy tokens, ``hidden``: final hidden states)."""
         n = len(rids)
         bucket = min(_bucket(n), _bucket(self.max_batch))
         self._decode_batch_tensors(rids, bucket)
@@ -443,8 +484,11 @@ class LLMEngine:
         st["table"].copy_(self.h_table[:bucket], non_blocking=True)
         st["kv_lens"].copy_(self.h_kv_lens[:bucket], non_blocking=True)
         self.h2d_bytes_last += bucket * (4 + 4 + 8 + 4 + 4 * mp)
+        if self.kv.state_slots:
+            st["state"].copy_(self.h_state[:bucket], non_blocking=True)
+            self.h2d_bytes_last += bucket * 4
         graph.replay()
-        return self._read_tokens(st["out"], bucket)[:n]
+        return st, bucket
 
     def _capture(self, bucket: int):
         dev, mp = self.device, self.max_pages_per_seq
@@ -455,6 +499,7 @@ class LLMEngine:
             "table": torch.zeros(bucket, mp, dtype=torch.int32, device=dev),
             "kv_lens": torch.zeros(bucket, dtype=torch.int32, device=dev),
             "out": torch.zeros(bucket, dtype=torch.int32, device=dev),
+            "state": torch.full((bucket,), -1, dtype=torch.int32, device=dev),
         }
         if self.fault_injector is not None:
             self.fault_injector("graph_capture")
@@ -462,9 +507,9 @@ class LLMEngine:
         def run():
             batch = ForwardBatch(tokens=st["tokens"], positions=st["positions"], slot_mapping=st["slots"],
                                  block_table=st["table"], kv_lens=st["kv_lens"], is_decode=True,
-                                 max_kv_len=self.max_model_len)
-            hidden = self.model.forward_hidden(batch)
-            self.model.greedy_tokens(hidden, st["out"])
+                                 max_kv_len=self.max_model_len, state_slots=st["state"] if self.kv.state_slots else None)
+            st["hidden"] = self.model.forward_hidden(batch)
+            self.model.greedy_tokens(st["hidden"], st["out"])
 
         # warm up on a side stream (loads kernels, sizes scratch) before capturing
         s = torch.cuda.Stream(device=dev)
@@ -499,13 +544,14 @@ class LLMEngine:
             if self.fault_injector is not None:
                 self.fault_injector("step")
             new_tokens: dict[int, int] = {}
-            if decode:
+            together = decode if self.mixed and prefill else []       # decoded tokens that join the prompt chunks' batch
+            if decode and not together:
                 toks = self._run_decode(decode)
                 for rid, tok in zip(decode, toks):
                     new_tokens[rid] = tok
             completed_prefill: list[tuple[Request, int]] = []
             if prefill:
-                completed_prefill = self._run_prefill(prefill)
+                completed_prefill = self._run_prefill(prefill, together)
             done_ids = {req.id for req, _ in completed_prefill}
             for rid, _, _ in prefill:
                 if rid not in done_ids:
@@ -568,6 +614,60 @@ class LLMEngine:
         self.run_until_done()
         outs = [self.requests[i].output for i in ids]
         return outs
+
+    # ------------------------------------------------------------------------------- replay
+    def replay(self, entries: Sequence[tuple], end: Sequence[object] = ()) -> Optional[torch.Tensor]:
+        """One step over token ids brought by the caller: ``entries`` = [(key, tokens, want)] are the next
+        tokens of each keyed sequence (created at its first entry) and the places among them whose logits
+        are asked for. All entries form one batch, run by the step's own functions: single tokens of
+        running sequences replay the decode step, anything else is a ragged batch of runs. Sequences in
+        ``end`` then give back their pages and state slots. Returns fp32 logits [wanted, vocab] in the
+        order of the entries, or None. Raises ``KvPoolExhaustedError`` when pool or slots do not suffice."""
+        self.h2d_bytes_last = 0
+        if len(entries) > self.h_kv_lens.numel() or sum(len(e[1]) for e in entries) > self.h_tokens.numel():
+            raise ValueError("more entries or tokens in one step than the engine was made for (max_batch, prefill_chunk)")
+        runs, rows, t = [], [], 0
+        for key, tokens, want in entries:
+            tokens = [int(v) for v in tokens]
+            if not tokens:
+                raise ValueError(f"{key}: an entry needs at least one token")
+            rid = self._replays.get(key)
+            if rid is None:
+                rid = self._replays[key] = self._next_id
+                self._next_id += 1
+                self.requests[rid] = Request(rid, [], SamplingParams(greedy=True), finished=True)     # not the scheduler's
+            req = self.requests[rid]
+            start = len(req.prompt) + len(req.output)
+            if start + len(tokens) > self.max_model_len:
+                raise ValueError(f"{key}: {start + len(tokens)} tokens exceed max_model_len={self.max_model_len}")
+            self.kv.append(rid, len(tokens))
+            # the first token is the "prompt" and the rest its continuation, so that a single next token is a decode step
+            req.output += tokens if start else tokens[1:]
+            req.prompt = req.prompt or tokens[:1]
+            runs.append((rid, start, len(tokens)))
+            rows += [t + int(w) for w in want]
+            t += len(tokens)
+        logits = None
+        if runs:
+            if len(runs) <= self.max_batch and all(start > 0 and count == 1 for _, start, count in runs):
+                rids = [rid for rid, _, _ in runs]
+                if self.use_graphs and not self._graphs_disabled:
+                    hidden = self._run_decode_graph(rids)[0]["hidden"]
+                else:
+                    hidden = self._run_decode_eager(rids)
+            else:
+                hidden, _ = self._run_chunks(runs)
+            if rows:
+                idx = torch.tensor(rows, dtype=torch.int64, device=self.device)
+                logits = self.model.full_logits(hidden[idx].contiguous()).float()
+            if self.cuda:
+                self._read_tokens(torch.zeros(1, dtype=torch.int32, device=self.device), 1)     # waits, and checks the status word
+        for key in end:
+            rid = self._replays.pop(key, None)
+            if rid is not None:
+                self.kv.free(rid)
+                self.requests.pop(rid, None)
+        return logits
 
     def release(self, rid: int) -> Optional[Request]:
         return self.requests.pop(rid, None)

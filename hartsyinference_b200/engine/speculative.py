@@ -78,6 +78,8 @@ def generate_speculative(engine, prompt: Sequence[int], params: Optional[Samplin
     params = params or SamplingParams(greedy=True)
     if params.needs_logits:
         raise ValueError("speculative decoding verifies greedy tokens; use a greedy request")
+    if getattr(engine.model.cfg, "recurrent", False):
+        raise ValueError("speculative decoding rolls rejected tokens back; recurrent state cannot be")
     prompt = list(prompt)
     limit = min(params.max_tokens, engine.max_model_len - len(prompt))
     if limit <= 0:

@@ -564,15 +564,21 @@ class TextService:
                 n = len(ids)
                 dev = m.device
                 pages = (n + 15) // 16
-                saved = m.kv_cache
+                saved, saved_state = m.kv_cache, getattr(m, "mixer_state", None)
                 m.alloc_kv(max(pages, 1), 16)
+                recurrent = getattr(m.cfg, "recurrent", False)
+                if recurrent:
+                    m.alloc_state(1)
                 b = ForwardBatch(tokens=torch.tensor(ids, dtype=torch.int32, device=dev),
                                  positions=torch.arange(n, dtype=torch.int32, device=dev),
                                  slot_mapping=torch.arange(n, dtype=torch.int64, device=dev),
                                  block_table=torch.arange(max(pages, 1), dtype=torch.int32, device=dev)[None],
                                  kv_lens=torch.tensor([n], dtype=torch.int32, device=dev), is_decode=False,
-                                 cu_q=torch.tensor([0, n], dtype=torch.int32, device=dev), max_q_len=n, max_kv_len=n)
-                hid = m.forward_hidden(b).float().mean(0)
+                                 cu_q=torch.tensor([0, n], dtype=torch.int32, device=dev), max_q_len=n, max_kv_len=n,
+                                 state_slots=torch.zeros(1, dtype=torch.int32, device=dev) if recurrent else None)
+                hid = m.forward_hidden(b)[:, :m.cfg.hidden_size].float().mean(0)
                 m.kv_cache = saved
+                if recurrent:
+                    m.mixer_state = saved_state
                 outs.append(torch.nn.functional.normalize(hid, dim=0).cpu())
         return torch.stack(outs)

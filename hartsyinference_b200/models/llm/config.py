@@ -27,6 +27,15 @@ class MoeConfig:
     use_correction_bias: bool = False
     first_dense_layers: int = 0         # leading layers that keep a dense FFN
     shared_gate: bool = False           # shared expert gated by sigmoid(x . w)
+    identity_experts: int = 0           # router outputs past the experts that return their input (no weights)
+    exact_router: bool = False          # router logits and scores in 32 bits
+    glu_limit: float = 0.0              # > 0: clamped expert activation g sigmoid(alpha g) (u + 1), g <= limit, |u| <= limit
+    glu_alpha: float = 1.702
+
+    @property
+    def choices(self) -> int:
+        """Router outputs: experts with weights and those that return their input."""
+        return self.num_experts + self.identity_experts
 
 
 @dataclass(frozen=True)
@@ -37,6 +46,35 @@ class MlaConfig:
     qk_rope_head_dim: int = 0
     v_head_dim: int = 0
     attn_scale: float = 0.0             # > 0 overrides 1/sqrt(nope + rope) (YaRN mscale folded in)
+
+
+@dataclass(frozen=True)
+class MixerSpec:
+    """Token mixer of one layer of a model whose layers differ (``TransformerConfig.layer_specs``)."""
+    kind: str = "attention"             # attention | channel_delta
+    heads: int = 1
+    kv_heads: int = 1
+    dim: int = 64                       # query / key size per head
+    vdim: int = 64                      # value size per head
+    # attention
+    scale: float = 0.0                  # 0 = 1/sqrt(dim)
+    softcap: float = 0.0
+    window: int = 0                     # 0 = unlimited
+    bias_reach: int = 0                 # distance at which the logarithmic bias buckets end (0: no distance bias)
+    bias_rows: int = 32                 # bias table rows of synthetic weights (a checkpoint's table gives its own)
+    shared_kv: bool = False             # the values are the keys
+    qk_bias: bool = False
+    out_gate: bool = False              # output * sigmoid(W_g h)
+    sink: Optional[float] = None        # score of a key without a value
+    # channel_delta
+    conv: int = 0                       # taps of the short convolution
+    rank: int = 0                       # low-rank size of decay and gate in synthetic weights (0 = dim)
+
+
+@dataclass(frozen=True)
+class LayerSpec:
+    mixer: MixerSpec
+    moe: Optional[MoeConfig] = None     # None: no feed-forward in this layer
 
 
 @dataclass(frozen=True)
@@ -109,6 +147,8 @@ class TransformerConfig:
     learned_position_offset: int = 0    # rows skipped at the start of the learned position table (OPT: 2)
     moe: Optional[MoeConfig] = None
     mla: Optional[MlaConfig] = None
+    layer_specs: tuple = ()             # one LayerSpec per layer: mixers of different kinds and sizes around a 32-bit
+                                        # residual stream, norms before and after every sublayer
     bos_token_id: int = 1
     eos_token_ids: tuple = (2,)
 
@@ -128,6 +168,16 @@ class TransformerConfig:
         return self.moe is not None and self.moe.num_experts > 0 and layer >= self.moe.first_dense_layers
 
     @property
+    def mixed_layers(self) -> bool:
+        """Layers described one by one (``layer_specs``): 32-bit residual stream, optional recurrent state."""
+        return bool(self.layer_specs)
+
+    @property
+    def recurrent(self) -> bool:
+        """True when some layer carries a state from token to token (a state slot per sequence)."""
+        return any(ls.mixer.kind == "channel_delta" for ls in self.layer_specs)
+
+    @property
     def general_path(self) -> bool:
         """Architectures whose block structure is outside the fused decode path: they run the same
         kernels through an unfused layer loop."""
@@ -142,6 +192,11 @@ class TransformerConfig:
         graph cannot capture."""
         return not (self.alibi or self.attn_sinks or bool(self.cross_layers))
 
+    @property
+    def fp8_linears_ok(self) -> bool:
+        """False for models that are served with bf16 weights whatever the ``fp8_linears`` flag says."""
+        return not self.mixed_layers
+
     def layer_window(self, layer: int) -> int:
         if self.sliding_window <= 0:
             return 0
@@ -153,6 +208,9 @@ class TransformerConfig:
 
     def param_count(self) -> int:
         h, l = self.hidden_size, self.num_layers
+        if self.layer_specs:
+            from .mixers import spec_param_count
+            return sum(spec_param_count(ls, h) for ls in self.layer_specs) + 2 * self.vocab_size * h + h
         attn = h * (self.q_size + 2 * self.kv_size) + self.q_size * h
         if self.mla is not None:
             m = self.mla
@@ -177,6 +235,8 @@ class TransformerConfig:
         (src/HartsyInference.LLM/Transformer/TensorParallelTransformer.cs:59-108)."""
         if tp <= 1:
             return
+        if self.layer_specs:
+            raise ValueError(f"{self.arch}: models with per-layer mixers are not sharded; load with tp=1")
         if self.num_heads % tp or self.ffn_size % tp:
             raise ValueError(f"heads ({self.num_heads}) and ffn ({self.ffn_size}) must divide by tp={tp}")
         if self.num_kv_heads % tp and tp % self.num_kv_heads:
@@ -224,7 +284,10 @@ def tiny(base: str = "qwen2.5-0.5b", **over: Any) -> TransformerConfig:
 def from_hf_config(d: dict) -> TransformerConfig:
     """Map a Hugging Face ``config.json`` (llama / mistral / qwen2 / qwen3 / gemma 1-3 / granite / olmo2 /
     phi3 / glm / glm4 / starcoder2 / stablelm / cohere / cohere2 / nemotron / gpt_neox / gpt2 / granitemoe / mllama (text) / qwen2_vl - qwen2_5_vl - qwen3_vl (text) / hunyuan_v1_dense / apertus / bloom / gpt_oss / gptj / opt / phi / olmo3 / exaone4 / helium / ernie4_5 / arcee / smollm3 / ministral / seed_oss / minicpm / internlm2 / deepseek_v2-v3 / glm4_moe / dots1 / ernie4_5_moe / hunyuan_v1_moe / cwm / gpt_bigcode / falcon / mixtral /
-    olmoe / qwen2_moe / qwen3_moe families) onto :class:`TransformerConfig`."""
+    olmoe / qwen2_moe / qwen3_moe families, and lududra) onto :class:`TransformerConfig`."""
+    if str(d.get("architecture", "")).lower() == "lududra":
+        from .lududra import lududra_config
+        return lududra_config(d)
     mt = d.get("model_type", "llama")
     if mt == "opt":
         d = {**d, "intermediate_size": d.get("ffn_dim") or 4 * d["hidden_size"], "hidden_act": d.get("activation_function", "relu"),

@@ -94,14 +94,18 @@ def _gemma_sandwich_fix(cfg: TransformerConfig, get: Callable[[str], Optional[to
 
 
 def load_llm(path: str | Path, device: str | torch.device = "cuda", comm: Optional[Comm] = None,
-             fp8: Optional[bool] = None) -> LoadedLLM:
+             fp8: Optional[bool] = None, dtype: torch.dtype = torch.bfloat16) -> LoadedLLM:
+    """``dtype`` float32 loads a model to run in 32 bits, for the architectures that have that form (a
+    ``ValueError`` otherwise)."""
     if str(path).startswith("synthetic:"):
         return _load_synthetic(str(path)[len("synthetic:"):], device, comm, fp8)
     p = Path(path)
     if p.is_file() and p.suffix == ".gguf":
         return _load_gguf(p, device, comm, fp8)
     if p.is_dir() and (p / "config.json").exists():
-        return _load_hf(p, device, comm, fp8)
+        return _load_hf(p, device, comm, fp8, dtype)
+    if dtype != torch.bfloat16:
+        raise ValueError(f"{path}: only checkpoint directories load in {dtype}")
     if p.is_dir():
         ggufs = sorted(p.glob("*.gguf"))
         if ggufs:
@@ -411,7 +415,7 @@ def _llava_names(ck) -> tuple[Callable, Callable]:
     return lm, tower
 
 
-def _load_hf(p: Path, device, comm, fp8) -> LoadedLLM:
+def _load_hf(p: Path, device, comm, fp8, dtype: torch.dtype = torch.bfloat16) -> LoadedLLM:
     from ...assets.lowbit import dequantizing_get
     raw = json.loads((p / "config.json").read_text())
     ck = ShardedCheckpoint(p)
@@ -459,7 +463,7 @@ def _load_hf(p: Path, device, comm, fp8) -> LoadedLLM:
                              get=tower_get, feature_layer=int(raw.get("vision_feature_layer", -2)))
     else:
         cfg = from_hf_config(raw)
-        model = DecoderModel(cfg, device, comm=comm, fp8=_want_fp8(fp8, device), dp_attention=_want_dp_attention(cfg, comm))
+        model = DecoderModel(cfg, device, comm=comm, fp8=_want_fp8(fp8, device), dp_attention=_want_dp_attention(cfg, comm), dtype=dtype)
         model.load_state_dict(standard_names(ck_get, raw))
     tok: Tokenizer
     if (p / "tokenizer.json").exists():

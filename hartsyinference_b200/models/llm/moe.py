@@ -12,6 +12,10 @@ plan: every local expert gets as many blocks of ``cap`` slots as its tokens need
 gate_up GEMM over the blocks in use (one launch) -> GLU -> grouped down GEMM -> ``moe_combine``
 (fixed order, deterministic).
 
+Experts that return their input, 32-bit routing and the clamped activation are fields of ``MoeConfig``;
+models with a 32-bit residual stream take the expert outputs uncombined (``routed_rows``), the norm
+kernel that follows sums them.
+
 Reference behaviour: src/HartsyInference.LLM/Transformer/MoeFeedForward.cs (Route:186-233,
 RouteGroupLimited:240-312, Forward:88-161 with one device-to-host copy of the router logits and
 a per-expert gather / GEMM / scatter-add loop) and src/HartsyInference.LLM/Models/DeepSeekV3Model.cs
@@ -27,7 +31,7 @@ import torch
 from ... import ops
 from ...ops import LinearWeight
 from ...ops import reference as R
-from .config import TransformerConfig
+from .config import MoeConfig, TransformerConfig
 
 _CHUNK = 1024        # tokens per pass: up to 8 runs of 128 tokens share one read of the expert weights
 
@@ -47,15 +51,16 @@ class MoeFeedForward:
     """Callable ``(h [T, H], model) -> [T, H]`` plugged into ``LayerWeights.ffn_module``."""
 
     def __init__(self, cfg: TransformerConfig, weights: MoeWeights, rank: int = 0, world: int = 1,
-                 all_reduce: Optional[Callable[[torch.Tensor], torch.Tensor]] = None):
-        moe = cfg.moe
+                 all_reduce: Optional[Callable[[torch.Tensor], torch.Tensor]] = None, moe: Optional[MoeConfig] = None,
+                 hidden: int = 0):
+        moe = moe if moe is not None else cfg.moe
         assert moe is not None and moe.num_experts % world == 0
         self.cfg, self.moe, self.w = cfg, moe, weights
         self.rank, self.world = rank, world
         self.e_local = moe.num_experts // world
         self.e0 = rank * self.e_local
         self.all_reduce = all_reduce
-        self.hidden = cfg.hidden_size
+        self.hidden = hidden or cfg.hidden_size
         self.ffn = moe.expert_ffn
         self._xs: dict[tuple[int, int], torch.Tensor] = {}     # (capacity, runs) -> dispatch buffer
 
@@ -70,12 +75,43 @@ class MoeFeedForward:
     # ---------------------------------------------------------------------------------- pieces
     def route(self, h: torch.Tensor) -> tuple[torch.Tensor, torch.Tensor]:
         m = self.moe
+        if m.exact_router:
+            return ops.router(h, self.w.router, self.w.router_bias, m.top_k, sigmoid=m.scoring == "sigmoid",
+                              norm_topk=m.norm_topk_prob, scale=m.routed_scaling_factor)
         logits = ops.linear(h, self.w.router)
         if not logits.is_cuda:
             logits = logits.float()
         return ops.moe_route(logits, self.w.router_bias, m.top_k, n_group=m.n_group, topk_group=m.topk_group,
                              sigmoid=m.scoring == "sigmoid", norm_topk=m.norm_topk_prob,
                              scale=m.routed_scaling_factor)
+
+    def _activate(self, gu: torch.Tensor, plan=None) -> torch.Tensor:
+        if self.moe.glu_limit > 0:
+            return ops.glu_clamped(gu, self.moe.glu_limit, self.moe.glu_alpha, plan)
+        return ops.glu(gu, self.cfg.activation)[0]
+
+    def routed_rows(self, h: torch.Tensor) -> "ops.RoutedRows":
+        """Expert outputs of every row of ``h`` (bf16 or fp32) with their slots and weights, for a consumer
+        that combines them (``ops.residual_norm``). Single rank, no shared expert, no token limit."""
+        m, w = self.moe, self.w
+        assert self.world == 1 and w.shared_gate_up is None
+        ids, wts = self.route(h)
+        source = h if m.identity_experts > 0 else None
+        if h.is_cuda and h.dtype == torch.bfloat16:
+            cap = ops.moe_block_capacity(h.shape[0], m.top_k, m.choices)
+            blocks = (h.shape[0] * m.top_k + cap - 1) // cap + self.e_local
+            # rows of slots without a token are computed and never read: they need no value
+            xs = torch.empty(blocks * cap, self.hidden, dtype=h.dtype, device=h.device)
+            plan = ops.moe_dispatch_dynamic(h, ids, 0, self.e_local, cap, xs)
+            gu = ops.grouped_linear_dynamic(xs, w.gate_up, self.e_local, plan)
+            y = ops.grouped_linear_dynamic(self._activate(gu, plan), w.down, self.e_local, plan)
+            return ops.RoutedRows(y, plan.slot_of, ids, wts, source, m.num_experts)
+        # 32-bit products (and CPU tensors): one product per (token, choice) pair
+        gu = ops.pair_linear_f32(h, w.gate_up, ids, m.num_experts, m.top_k)
+        y = ops.pair_linear_f32(self._activate(gu), w.down, ids, m.num_experts, 1)
+        pair = torch.arange(ids.numel(), dtype=torch.int32, device=h.device).reshape(ids.shape)
+        slot_of = torch.where(ids < m.num_experts, pair, torch.full_like(pair, -1))
+        return ops.RoutedRows(y, slot_of, ids, wts, source, m.num_experts)
 
     def _shared(self, h: torch.Tensor) -> Optional[torch.Tensor]:
         w = self.w
@@ -154,6 +190,10 @@ class MoeFeedForward:
     # ---------------------------------------------------------------------------------- forward
     def __call__(self, h: torch.Tensor, model=None) -> torch.Tensor:
         t = h.shape[0]
+        if self.moe.identity_experts > 0 or self.moe.glu_limit > 0:
+            acc = torch.zeros(t, self.hidden, dtype=torch.float32, device=h.device)
+            ops.residual_norm(acc, self.routed_rows(h), None, None, dim=self.hidden, eps=0.0, layernorm=False, dtype=h.dtype)
+            return acc.to(h.dtype)
         outs = []
         for c0 in range(0, t, _CHUNK):
             hc = h[c0:c0 + _CHUNK]

@@ -50,6 +50,7 @@ class ForwardBatch:
     cross_states: Optional[object] = None           # Mllama: projected vision states [Tv, H] for every row, or a list
                                                     # with one entry (tensor or None) per sequence
     cross_row_mask: Optional[torch.Tensor] = None   # Mllama: [T], 0 for text rows that precede every image
+    state_slots: Optional[torch.Tensor] = None      # [S] int32 recurrent-state slot of every sequence (-1: none)
 
 
 def build_inv_freq(rot: int, theta: float, scaling: RopeScaling, device) -> tuple[torch.Tensor, float]:
@@ -124,8 +125,15 @@ def x_is_cuda(x) -> bool:
 
 class DecoderModel:
     def __init__(self, cfg: TransformerConfig, device: torch.device | str = "cpu", comm: Optional[Comm] = None,
-                 fp8: bool = False, layer_range: Optional[tuple[int, int]] = None, dp_attention: bool = False):
+                 fp8: bool = False, layer_range: Optional[tuple[int, int]] = None, dp_attention: bool = False,
+                 dtype: torch.dtype = torch.bfloat16):
         self.cfg = cfg
+        # activation dtype: bf16, or fp32 (32-bit products and caches) where the layers have that form
+        if dtype != torch.bfloat16 and not (cfg.mixed_layers and dtype == torch.float32):
+            raise ValueError(f"{cfg.arch}: activations run in bfloat16")
+        if cfg.mixed_layers and layer_range is not None and layer_range != (0, cfg.num_layers):
+            raise ValueError(f"{cfg.arch}: models with per-layer mixers are not split into pipeline stages")
+        self.dtype = dtype
         # pipeline stage: this instance holds layers [layer0, layer1) only (all of them by default)
         self.layer0, self.layer1 = layer_range if layer_range is not None else (0, cfg.num_layers)
         self.first_stage, self.last_stage = self.layer0 == 0, self.layer1 == cfg.num_layers
@@ -134,7 +142,7 @@ class DecoderModel:
         self.tp = self.comm.world
         self.tp_rank = self.comm.rank
         cfg.validate_tp(self.tp)
-        self.fp8 = fp8
+        self.fp8 = fp8 and cfg.fp8_linears_ok
         self.hq = cfg.num_heads // self.tp
         self.hkv = max(1, cfg.num_kv_heads // self.tp)
         self.ffn = cfg.ffn_size // self.tp
@@ -153,7 +161,8 @@ class DecoderModel:
         self.embed_norm_w: Optional[torch.Tensor] = None   # LayerNorm on the embedding output (BLOOM)
         self.embed_norm_b: Optional[torch.Tensor] = None
         self.alibi_slopes: Optional[torch.Tensor] = None   # [local heads]
-        self.kv_cache: Optional[torch.Tensor] = None
+        self.kv_cache: Optional[torch.Tensor] = None      # per-layer list for models with per-layer mixers
+        self.mixer_state: list = []                       # per layer: (convolution inputs, recurrent state) by slot, or None
         self.all_reduce: Callable[[torch.Tensor], torch.Tensor] = self.comm.all_reduce
         # hook for the fused GEMM + all-reduce path: (x, weight, residual) -> reduced output
         self.row_parallel_linear: Optional[Callable] = None
@@ -169,8 +178,10 @@ class DecoderModel:
         self.dp_exchange = None
 
     # ------------------------------------------------------------------------------ weights
-    def _lw(self, w: torch.Tensor, bias: Optional[torch.Tensor] = None, allow_fp8: bool = True) -> LinearWeight:
+    def _lw(self, w: torch.Tensor, bias: Optional[torch.Tensor] = None, allow_fp8: bool = True, pad_rows: int = 0) -> LinearWeight:
         w = w.to(self.device)
+        if pad_rows and w.shape[0] % pad_rows:
+            w = torch.cat([w, torch.zeros(pad_rows - w.shape[0] % pad_rows, w.shape[1], dtype=w.dtype, device=w.device)])
         b = None if bias is None else bias.to(self.device)
         return LinearWeight.from_dense(w, b, fp8=self.fp8 and allow_fp8)
 
@@ -196,6 +207,10 @@ class DecoderModel:
                 raise KeyError(f"missing tensor {name}")
             return t
 
+        if cfg.mixed_layers:
+            from .lududra import load_layers
+            load_layers(self, need)
+            return
         emb = need("model.embed_tokens.weight")
         self.embed = emb.to(dt).to(self.device)
         head = get("lm_head.weight")
@@ -404,6 +419,12 @@ class DecoderModel:
         """Synthetic weights generated on the device (no host copy): bf16 N(0, std), or e4m3 bytes
         with constant block scales that reproduce the same distribution."""
         cfg, d, dev = self.cfg, self.cfg.head_dim, self.device
+        if cfg.mixed_layers:
+            from .lududra import load_layers, random_tensor, tensor_shapes
+            shapes = tensor_shapes(cfg)
+            order = {n: i for i, n in enumerate(shapes)}
+            load_layers(self, lambda n: random_tensor(n, shapes[n], dev, seed * 1000003 + 11 * order[n] + 1, std))
+            return
         counter = [seed * 1000003 + self.tp_rank * 7919]
 
         def dense(n, k, s=std):
@@ -580,6 +601,10 @@ class DecoderModel:
 
     # ------------------------------------------------------------------------------ KV cache
     def kv_bytes_per_page(self, page: int) -> int:
+        if self.cfg.mixed_layers:
+            es = torch.finfo(self.dtype).bits // 8
+            return sum(math.prod(lw.attn_module.cache_shape(1, page)) * es for lw in self.layers
+                       if hasattr(lw.attn_module, "cache_shape"))
         if self.cfg.mla is not None:
             return (self.layer1 - self.layer0) * page * (self.cfg.mla.kv_lora_rank + self.cfg.mla.qk_rope_head_dim) * 2
         return (self.layer1 - self.layer0) * 2 * self.hkv * page * self.cfg.head_dim * 2
@@ -587,6 +612,11 @@ class DecoderModel:
     def alloc_kv(self, num_pages: int, page: int = 16) -> torch.Tensor:
         """[layers, 2, pages, hkv_local, page, head_dim] bf16, or with multi-head latent attention
         [layers, pages, page, 576] (latent + rotated shared key, replicated on every rank)."""
+        if self.cfg.mixed_layers:
+            # one pool per attention layer, [planes, pages, kv heads, page, head size] (one plane when values are keys)
+            self.kv_cache = [torch.zeros(lw.attn_module.cache_shape(num_pages, page), dtype=self.dtype, device=self.device)
+                             if hasattr(lw.attn_module, "cache_shape") else None for lw in self.layers]
+            return self.kv_cache
         if self.cfg.mla is not None:
             row = self.cfg.mla.kv_lora_rank + self.cfg.mla.qk_rope_head_dim
             self.kv_cache = torch.zeros(self.layer1 - self.layer0, num_pages, page, row, dtype=torch.bfloat16,
@@ -595,6 +625,25 @@ class DecoderModel:
         self.kv_cache = torch.zeros(self.layer1 - self.layer0, 2, num_pages, self.hkv, page, self.cfg.head_dim,
                                     dtype=torch.bfloat16, device=self.device)
         return self.kv_cache
+
+    def alloc_state(self, slots: int) -> None:
+        """Recurrent state of ``slots`` sequences: per recurrent layer the short convolution's last inputs (in
+        the activation dtype) and the state matrices (fp32)."""
+        self.mixer_state = []
+        for lw in self.layers:
+            st = None
+            if hasattr(lw.attn_module, "state_shapes"):
+                conv, rec = lw.attn_module.state_shapes(slots)
+                st = (torch.zeros(conv, dtype=self.dtype, device=self.device), torch.zeros(rec, dtype=torch.float32, device=self.device))
+            self.mixer_state.append(st)
+
+    def state_bytes_per_slot(self) -> int:
+        es, n = torch.finfo(self.dtype).bits // 8, 0
+        for lw in self.layers:
+            if hasattr(lw.attn_module, "state_shapes"):
+                conv, rec = lw.attn_module.state_shapes(1)
+                n += math.prod(conv) * es + math.prod(rec) * 4
+        return n
 
     # ------------------------------------------------------------------------------ forward
     def _attn_scale(self) -> float:
@@ -810,6 +859,46 @@ class DecoderModel:
             return x, None
         return self._block_norm(x, self.final_norm, self.final_norm_b)
 
+    def _forward_mixers(self, batch: ForwardBatch, capture: Optional[list] = None) -> torch.Tensor:
+        """Layer loop of models with per-layer mixers. ``x`` is the fp32 residual stream, updated in place by
+        the norm kernel that ends one sublayer and starts the next:
+
+            h = norm1(x)                                                   [one launch]
+            mixer -> x += norm1b(y), h = norm2(x)                          [one launch]
+            experts -> x += norm2b(sum of expert rows), h = norm1'(x)      [one launch]
+
+        ``capture`` (a list) receives a copy of the stream after every layer."""
+        cfg = self.cfg
+        kw = dict(dim=cfg.hidden_size, eps=cfg.rms_eps, layernorm=cfg.norm_type == "layernorm", dtype=self.dtype)
+        if batch.embeds is not None:
+            x = torch.nn.functional.pad(batch.embeds.float(), (0, self.embed.shape[1] - batch.embeds.shape[1])).contiguous()
+        else:
+            x = ops.embedding_f32(batch.tokens, self.embed, cfg.embed_scale * cfg.embedding_multiplier, cfg.hidden_size)
+        h = ops.residual_norm(x, None, None, self.layers[0].in_norm if self.layers else self.final_norm, **kw)
+        last = len(self.layers) - 1
+        for li, lw in enumerate(self.layers):
+            after = self.final_norm if li == last else self.layers[li + 1].in_norm
+            y = lw.attn_module(h, batch, li, self)
+            h = ops.residual_norm(x, y, lw.post_attn_norm, lw.post_norm if lw.ffn_module is not None else after, **kw)
+            if lw.ffn_module is not None:
+                h = self._routed_sublayer(lw, x, h, after, kw)
+            if capture is not None:
+                capture.append(x[:, :cfg.hidden_size].clone())
+        return h
+
+    # most rows whose expert inputs and outputs are held at once
+    _ROUTED_ROWS = 8192
+
+    def _routed_sublayer(self, lw: LayerWeights, x: torch.Tensor, h: torch.Tensor, after: torch.Tensor, kw: dict) -> torch.Tensor:
+        t, step = x.shape[0], self._ROUTED_ROWS
+        if t <= step:
+            return ops.residual_norm(x, lw.ffn_module.routed_rows(h), lw.post_ffn_norm, after, **kw)
+        out = torch.empty_like(h)
+        for a in range(0, t, step):
+            b = min(a + step, t)
+            ops.residual_norm(x[a:b], lw.ffn_module.routed_rows(h[a:b]), lw.post_ffn_norm, after, out=out[a:b], **kw)
+        return out
+
     def _fused_tp_ok(self, tokens: int) -> bool:
         """True when the layer loop can run on the fused row-parallel kernel: a plain pre-norm
         RMSNorm decoder with dense gated feed-forward blocks, held completely by this instance."""
@@ -914,6 +1003,8 @@ class DecoderModel:
         cfg = self.cfg
         d = cfg.head_dim
         res: Optional[torch.Tensor] = None
+        if cfg.mixed_layers:
+            return self._forward_mixers(batch)
         if hidden_in is None and self._dp_attention_ok(batch):
             return self._forward_dp_attention(batch)
         if hidden_in is not None:
@@ -975,8 +1066,8 @@ class DecoderModel:
         return out
 
     def logits(self, hidden: torch.Tensor) -> torch.Tensor:
-        """[rows, H] -> local vocabulary shard logits [rows, vocab_local] (bf16)."""
-        y = ops.linear(hidden, self.lm_head)
+        """[rows, H] -> local vocabulary shard logits [rows, vocab_local] (in the activation dtype)."""
+        y = ops.linear_act(hidden, self.lm_head) if self.dtype == torch.float32 else ops.linear(hidden, self.lm_head)
         cfg = self.cfg
         if cfg.logits_scale != 1.0:
             y = (y.float() * cfg.logits_scale).to(y.dtype)
@@ -996,7 +1087,7 @@ class DecoderModel:
         pairs are combined, so only 8 bytes per row and rank cross the wire."""
         y = self.logits(hidden)
         if self.tp == 1:
-            if y.shape[1] > self.cfg.vocab_size:
+            if y.shape[1] > self.cfg.vocab_size:         # rows past the vocabulary pad the weight
                 y = y[:, : self.cfg.vocab_size]
             return ops.argmax(y, out)
         v0 = self.tp_rank * self.vocab_local

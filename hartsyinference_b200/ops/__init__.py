@@ -51,6 +51,19 @@ from .core import (  # noqa: F401
     sample_tokens,
     selective_scan,
 )
+from .mixers import (  # noqa: F401
+    DeltaWeights,
+    RoutedRows,
+    attn_biased,
+    delta_mix,
+    embedding_f32,
+    glu_clamped,
+    kv_store,
+    linear_act,
+    pair_linear_f32,
+    residual_norm,
+    router,
+)
 from . import reference  # noqa: F401
 
 
@@ -61,7 +74,7 @@ from . import reference  # noqa: F401
 def _install_ranges() -> None:
     import sys
     from ..utils.profiling import traced
-    from . import core
+    from . import core, mixers
     mod = sys.modules[__name__]
     for name in ("linear", "norm", "glu", "rope_kv", "attn_decode", "attn_prefill_paged", "attn_paged_biased", "attention",
                  "embedding", "argmax", "quant_fp8_act", "grouped_linear", "grouped_linear_dynamic", "moe_route",
@@ -74,6 +87,8 @@ def _install_ranges() -> None:
         setattr(core, name, wrapped)          # internal calls (core.linear -> core.gguf_linear) are traced too
         if hasattr(mod, name):
             setattr(mod, name, wrapped)
+    for name in ("attn_biased", "delta_mix", "embedding_f32", "glu_clamped", "kv_store", "pair_linear_f32", "residual_norm", "router"):
+        setattr(mod, name, traced(name)(getattr(mixers, name)))
 
 
 _install_ranges()

@@ -50,6 +50,17 @@ _SIGNATURES = {
     "b200_moe_route": (i32, [vp, i32, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, f32, vp]),
     "b200_moe_dispatch": (i32, [vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, i32, vp]),
     "b200_moe_combine": (i32, [vp, vp, vp, vp, i32, i32, i32, i32, vp]),
+    "b200_glu_clamped": (i32, [vp, vp, i64, i32, f32, f32, vp, i32, i32, vp]),
+    "b200_residual_norm": (i32, [vp, vp, vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, i32, i32, f32, i32, vp]),
+    "b200_embedding_f32": (i32, [vp, vp, vp, i32, i32, i32, i32, i32, f32, vp]),
+    "b200_linear_f32": (i32, [vp, i32, vp, vp, vp, i32, i32, i32, i64, i64, i64, vp]),
+    "b200_router": (i32, [vp, i32, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, i32, f32, vp]),
+    "b200_pair_linear_f32": (i32, [vp, vp, vp, vp, i32, i32, i32, i32, i32, i64, i64, vp]),
+    "b200_delta_workspace_bytes": (i64, [i32, i32, i32, i32, i32]),
+    "b200_delta_launches": (i32, [i32, i32, i32, i32]),
+    "b200_delta": (i32, [vp] * 13 + [i32] * 9 + [i64, i32, i64, i32, f32, i32, vp]),
+    "b200_attn_biased": (i32, [vp] * 7 + [i32] * 9 + [vp, f32, f32, i32, vp, i32, vp, vp, i64, i64, i32, i32, vp]),
+    "b200_kv_store": (i32, [vp, vp, vp, vp, vp, i32, i32, i32, i32, i64, i32, vp]),
     "b200_norm": (i32, [vp, vp, vp, vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, f32, i32, i32, i32, vp]),
     "b200_quant_fp8": (i32, [vp, vp, vp, i32, i32, i64, i32, vp]),
     "b200_quant_fp8_weight": (i32, [vp, vp, vp, i32, i32, vp]),
@@ -74,10 +85,12 @@ _SIGNATURES = {
 
 
 def lib_path() -> Path:
-    """The kernels library (flag ``kernels_lib`` points at another build of it)."""
+    """The kernels library (flag ``kernels_lib`` points at another build of it); where only the smaller
+    library of a kernel group has been built (``build.ensure``), that one."""
     from .. import config
     override = config.get("kernels_lib")
-    return Path(override) if override else _LIB_DIR / "libb200_kernels.so"
+    full, group = _LIB_DIR / "libb200_kernels.so", _LIB_DIR / "libb200_kernels_decoder.so"
+    return Path(override) if override else group if group.exists() and not full.exists() else full
 
 
 def available() -> bool:

@@ -161,6 +161,49 @@ def glu(x: torch.Tensor, act: str = "silu") -> torch.Tensor:
     return a * u
 
 
+def glu_clamped(x: torch.Tensor, limit: float, alpha: float) -> torch.Tensor:
+    f = x.shape[-1] // 2
+    g, u = x[..., :f].float().clamp(max=limit), x[..., f:].float().clamp(-limit, limit)
+    return g * torch.sigmoid(alpha * g) * (u + 1.0)
+
+
+def delta_mix(proj, z, w, conv_state, state, positions, cu_q, slots, b_off) -> torch.Tensor:
+    """Gated delta rule with per-channel decay, token by token (see ``ops.delta_mix``)."""
+    t, h, hk, dk, dv, taps, c = proj.shape[0], w.heads, w.kv_heads, w.dk, w.dv, w.conv.shape[1], w.channels
+    bounds = list(range(slots.numel() + 1)) if cu_q is None else cu_q.tolist()
+    out = torch.empty(t, h * dv, dtype=proj.dtype)
+    for i, slot in enumerate(slots.tolist()):
+        a, b = bounds[i], bounds[i + 1]
+        carried = slot >= 0 and int(positions[a]) > 0
+        x = proj[a:b, :c].float()
+        tail = conv_state[slot].float() if carried else torch.zeros(taps - 1, c)
+        seq = torch.cat([tail, x], 0)
+        if slot >= 0 and taps > 1:
+            conv_state[slot] = seq[-(taps - 1):].to(conv_state.dtype)
+        x = torch.nn.functional.silu((seq.unfold(0, taps, 1) * w.conv[None]).sum(-1))
+        q, k, v = x.split([hk * dk, hk * dk, h * dv], -1)
+        unit = lambda u: u * torch.rsqrt(u.pow(2).sum(-1, keepdim=True) + 1e-6)
+        q = (unit(q.reshape(-1, hk, dk)) * w.dk_true ** -0.5).repeat_interleave(h // hk, 1)
+        k = unit(k.reshape(-1, hk, dk)).repeat_interleave(h // hk, 1)
+        v = v.reshape(-1, h, dv)
+        beta = torch.sigmoid(proj[a:b, b_off:b_off + h].float())
+        rate = torch.nn.functional.softplus(z[a:b, :h * dk].float() + w.dt_bias).reshape(-1, h, dk)
+        g = torch.exp(-w.decay_rate[None, :, None] * rate)
+        s = state[slot].clone() if carried else torch.zeros(h, dk, dv)
+        o = torch.empty(b - a, h, dv)
+        for j in range(b - a):
+            s = s * g[j, :, :, None]
+            u = beta[j, :, None] * (v[j] - (s * k[j, :, :, None]).sum(1))
+            s = s + k[j, :, :, None] * u[:, None, :]
+            o[j] = (s * q[j, :, :, None]).sum(1)
+        if slot >= 0:
+            state[slot] = s
+        gate = torch.sigmoid(z[a:b, h * dk:].float()).reshape(-1, h, dv)
+        o = o * torch.rsqrt(o.pow(2).sum(-1, keepdim=True) / w.dv_true + w.eps) * w.norm.float() * gate
+        out[a:b] = o.reshape(b - a, h * dv).to(proj.dtype)
+    return out
+
+
 # --------------------------------------------------------------------------------------------
 # rotary embedding
 # --------------------------------------------------------------------------------------------
@@ -189,10 +232,12 @@ def apply_rope(x: torch.Tensor, positions: torch.Tensor, inv_freq: torch.Tensor,
 # --------------------------------------------------------------------------------------------
 def attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, causal: bool = False,
               scale: Optional[float] = None, softcap: float = 0.0, window: int = 0,
-              alibi: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None) -> torch.Tensor:
+              alibi: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None,
+              dist_bias: Optional[torch.Tensor] = None) -> torch.Tensor:
     """q [Tq, Hq, D], k/v [Tk, Hkv, D] (one sequence). The last query row sits at key position
     Tk - 1 (so a query chunk with a cached prefix is expressed by Tk > Tq). ``alibi`` [Hq] adds
-    slope * key position to the scores; ``sinks`` [Hq] adds one extra logit per head to the softmax
+    slope * key position to the scores; ``dist_bias`` [Hq, n] adds a value by key distance (its last
+    entry also for longer distances); ``sinks`` [Hq] adds one extra logit per head to the softmax
     denominator (it attends to nothing). Returns fp32 [Tq, Hq, D]."""
     tq, hq, d = q.shape
     tk, hkv, _ = k.shape
@@ -212,6 +257,8 @@ def attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, causal: bool = 
         mask &= kpos > qpos - window
     if alibi is not None:
         s = s + alibi.float()[:, None, None] * kpos[None].float()
+    if dist_bias is not None:
+        s = s + dist_bias.float()[:, (qpos - kpos).clamp(0, dist_bias.shape[1] - 1)]
     s = s.masked_fill(~mask[None], float("-inf"))
     if sinks is not None:
         s = torch.cat([s, sinks.float()[:, None, None].expand(hq, tq, 1)], -1)

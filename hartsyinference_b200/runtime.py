@@ -30,6 +30,9 @@ _SIGS = {
     "b200_kv_fork_prefix": (i64, [vp, i64, i64, i64]),
     "b200_kv_seq_len": (i64, [vp, i64]),
     "b200_kv_block_table": (i32, [vp, i64, P(i32), i32]),
+    "b200_kv_set_slots": (None, [vp, i32]),
+    "b200_kv_seq_slot": (i32, [vp, i64]),
+    "b200_kv_num_free_slots": (i32, [vp]),
     "b200_kv_inject_failure": (None, [vp, i32]),
     "b200_sched_create": (vp, [vp, i32, i32, i32]),
     "b200_sched_destroy": (None, [vp]),
@@ -84,14 +87,18 @@ def bind(name: str, restype, argtypes):
 
 
 class KvAllocator:
-    """Fixed-size page pool with per-sequence block tables (C++ core)."""
+    """Fixed-size page pool with per-sequence block tables (C++ core). With ``state_slots`` every
+    sequence also holds one of that many recurrent-state slots while it has pages."""
 
-    def __init__(self, num_blocks: int, block_size: int = 16):
+    def __init__(self, num_blocks: int, block_size: int = 16, state_slots: int = 0):
         self._h = lib().b200_kv_create(num_blocks, block_size)
         if not self._h:
             raise ValueError("bad pool geometry")
         self.num_blocks = num_blocks
         self.block_size = block_size
+        self.state_slots = state_slots
+        if state_slots > 0:
+            lib().b200_kv_set_slots(self._h, state_slots)
 
     def close(self) -> None:
         if self._h:
@@ -129,6 +136,14 @@ class KvAllocator:
 
     def fork_prefix(self, src: int, dst: int, tokens: int) -> int:
         return lib().b200_kv_fork_prefix(self._h, src, dst, tokens)
+
+    def seq_slot(self, seq: int) -> int:
+        """State slot of a sequence, -1 when it holds none."""
+        return lib().b200_kv_seq_slot(self._h, seq)
+
+    @property
+    def num_free_slots(self) -> int:
+        return lib().b200_kv_num_free_slots(self._h)
 
     def seq_len(self, seq: int) -> int:
         return lib().b200_kv_seq_len(self._h, seq)
