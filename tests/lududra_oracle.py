@@ -34,17 +34,17 @@ def distance_bucket(n: int, rows: int, reach: int) -> int:
     return min(rows - 1, int(half + math.floor(math.log(n / half) / math.log(reach / half) * (rows - half))))
 
 
-def attention_weights(q, k, bias_of, scale, cap, window):
-    """[T, T] weights of one head: capped scores + distance bias, window, and 1 added to the
-    denominator (rows sum to less than one)."""
+def attention_weights(q, k, bias_of, scale, cap, window, first=0):
+    """[T - first, T] weights of one head for the queries from ``first`` on: capped scores + distance bias,
+    window, and 1 added to the denominator (rows sum to less than one)."""
     t = q.shape[0]
-    out = torch.zeros(t, t, dtype=q.dtype)
-    for i in range(t):
+    out = torch.zeros(t - first, t, dtype=q.dtype)
+    for i in range(first, t):
         lo = max(0, i - window + 1)
         s = torch.stack([cap * torch.tanh((q[i] @ k[j]) * scale / cap) + bias_of(i - j) for j in range(lo, i + 1)])
         m = torch.clamp(s.max(), min=0.0)
         e = torch.exp(s - m)
-        out[i, lo:i + 1] = e / (torch.exp(-m) + e.sum())
+        out[i - first, lo:i + 1] = e / (torch.exp(-m) + e.sum())
     return out
 
 
