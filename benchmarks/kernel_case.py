@@ -5,6 +5,8 @@
     python benchmarks/kernel_case.py attn_decode 64 8 1 128 2304
     python benchmarks/kernel_case.py mla 64 16 2304
     python benchmarks/kernel_case.py attn_dense 4608 8
+    python benchmarks/kernel_case.py delta 4 2048 16
+    python benchmarks/kernel_case.py attn_window 4 2048 16 2 1024
 
 Inputs are larger than the L2 cache where the op is bandwidth bound but stay far below a few GB,
 so a full-metric capture (dozens of replays per launch) ends in about a minute. The status word is
@@ -102,6 +104,7 @@ def _time_cold(fn, reps=7):
     ts = []
     for i in range(reps + 2):
         flush.zero_()
+        torch.cuda._sleep(600_000)        # the host gets ahead of the device: launch cost stays out
         e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
         e0.record()
         fn()
@@ -285,7 +288,44 @@ def _triplane(argv):
     print(f"triplane {res}^3 = {pts} points: {t:.2f} ms, {flop / t / 1e9:.1f} TFLOP/s fp32, {pts / t / 1e6:.2f} G points/s")
 
 
-CASES = {"mla_proj": _mla_proj, "gemm_ar_large": _gemm_ar_large, "ag_gemm": _ag_gemm, "ulysses": _ulysses, "allreduce": _allreduce, "sample": _sample,
+def _delta(argv):
+    """delta SEQS TOKENS HEADS: the gated delta rule, head size 128 (TOKENS = 1: a decode step)."""
+    seqs, n, h = (int(v) for v in argv[:3])
+    t, d, ch = seqs * n, 128, 3 * 128 * h
+    dev = "cuda"
+    w = ops.DeltaWeights(conv=torch.randn(4, ch, device=dev), decay_rate=torch.ones(h, device=dev), dt_bias=torch.zeros(h * d, device=dev),
+                         norm=torch.ones(d, dtype=torch.bfloat16, device=dev), heads=h, kv_heads=h, dk=d, dv=d, dk_true=d, dv_true=d, eps=1e-6)
+    conv, st = torch.zeros(seqs, 3, ch, dtype=torch.bfloat16, device=dev), torch.zeros(seqs, h, d, d, device=dev)
+    proj, z = torch.randn(t, ch + h, device=dev).to(torch.bfloat16), torch.randn(t, 2 * h * d, device=dev).to(torch.bfloat16)
+    pos = torch.full((t,), 5, dtype=torch.int32, device=dev)
+    cu = None if n == 1 else torch.arange(0, t + 1, n, dtype=torch.int32, device=dev)
+    slots = torch.arange(seqs, dtype=torch.int32, device=dev)
+    ms = _time_cold(lambda: ops.delta_mix(proj, z, w, conv, st, pos, cu, slots, ch))
+    print(f"delta {seqs} x {n} tokens x {h} heads: {ms * 1e3:.1f} us")
+
+
+def _attn_window(argv):
+    """attn_window SEQS TOKENS HEADS KV_HEADS WINDOW [decode]: windowed attention with distance bias, cap, sink,
+    gate and shared keys / values, head size 128, beside the plain kernel."""
+    seqs, n, h, kv, win = (int(v) for v in argv[:5])
+    dec = len(argv) > 5
+    d, per, dev = 128, n // 16, "cuda"
+    kc, vc = (torch.randn(seqs * per, kv, 16, d, device=dev).to(torch.bfloat16) for _ in range(2))
+    table = torch.randperm(seqs * per, device=dev).to(torch.int32).reshape(seqs, per)
+    lens = torch.full((seqs,), n, dtype=torch.int32, device=dev)
+    t, ql = (seqs, 1) if dec else (seqs * n, n)
+    q, gate = (torch.randn(t, h * d, device=dev).to(torch.bfloat16) for _ in range(2))
+    cu = None if dec else torch.arange(0, t + 1, n, dtype=torch.int32, device=dev)
+    dist, sinks = torch.randn(h, 513, device=dev), torch.zeros(h, device=dev)
+    a = _time_cold(lambda: ops.attn_biased(q, kc, None, table, lens, cu, heads=h, max_q_len=ql, max_kv_len=n, scale=0.1, softcap=30.0, window=win,
+                                      dist_bias=dist, sinks=sinks, gate=gate))
+    q3 = q.view(t, h, d)
+    b = _time_cold((lambda: ops.attn_decode(q3, kc, vc, table, lens, window=win, max_kv_len=n)) if dec else
+              (lambda: ops.attn_prefill_paged(q3, kc, vc, table, lens, cu, ql, window=win)))
+    print(f"attn_window: extended {a * 1e3:.1f} us, plain {b * 1e3:.1f} us")
+
+
+CASES = {"delta": _delta, "attn_window": _attn_window, "mla_proj": _mla_proj, "gemm_ar_large": _gemm_ar_large, "ag_gemm": _ag_gemm, "ulysses": _ulysses, "allreduce": _allreduce, "sample": _sample,
          "int8": _int8, "triplane": _triplane,
          "gemm_ar": _gemm_ar, "attn_dense": _attn_dense, "gemm": _gemm, "grouped": _grouped, "attn_decode": _attn_decode, "mla": _mla}
 

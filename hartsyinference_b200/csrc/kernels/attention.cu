@@ -59,8 +59,78 @@ struct AttnParams {
   const __nv_bfloat16* gate;    // [tokens][gate_ld]: out *= sigmoid(gate), or null
   long long q_ld, gate_ld;      // row pitches in elements
   int dist_len, d, shared_kv;   // d: head size as stored; shared_kv: v is k
+  float cap_in, cap_out;        // softcap: cap_out * tanh(score / softcap), exp(2 score / softcap) = 2^(cap_in * q.k)
 };
 constexpr float kLog2e = 1.4426950408889634f;
+constexpr int kDistSmem = 4096;   // longest distance table that prefill blocks keep in shared memory
+
+__device__ __forceinline__ float exp2_approx(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
+// Scores of one warp tile in the extended form, in place (log2 units): scale, cap, distance bias, mask.
+// kMask: some key of the tile may be masked for some row. The bias table is read at fixed offsets from one
+// pointer per row while the tile's distances stay inside it, and only once when they all lie past its end.
+template <int NT, bool kMask>
+__device__ __forceinline__ void ext_scores(float (&s)[NT][4], int key0, const int (&row_limit)[2], const int (&row_start)[2],
+                                           const AttnParams& p, const float* const* row_bias) {
+  int mode = -1;
+  float far[2] = {0.f, 0.f};
+  const float* at[2] = {nullptr, nullptr};
+  if (p.dist_bias) {
+    const int d0 = row_limit[0] - 1 - key0, d1 = row_limit[1] - 1 - key0;       // distances of the first key
+    const int lo = min(d0, d1) - (NT * 8 - 7), hi = max(d0, d1);
+    mode = __all_sync(0xffffffffu, lo >= p.dist_len - 1) ? 2 : __all_sync(0xffffffffu, lo >= 0 && hi < p.dist_len) ? 1 : 0;
+    far[0] = row_bias[0][p.dist_len - 1];
+    far[1] = row_bias[1][p.dist_len - 1];
+    if (mode == 1) {
+      at[0] = row_bias[0] + d0;
+      at[1] = row_bias[1] + d1;
+    }
+  }
+#pragma unroll
+  for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      if (p.softcap > 0.f) {
+        const float e = exp2_approx(fminf(s[nt][j] * p.cap_in, 126.f));
+        s[nt][j] = p.cap_out - __fdividef(2.f * p.cap_out, e + 1.f);
+      } else {
+        s[nt][j] *= p.scale_log2;
+      }
+    }
+  if (mode == 1) {
+#pragma unroll
+    for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) s[nt][j] = fmaf(at[j >> 1][-(nt * 8 + (j & 1))], kLog2e, s[nt][j]);
+  } else if (mode == 2) {
+#pragma unroll
+    for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) s[nt][j] = fmaf(far[j >> 1], kLog2e, s[nt][j]);
+  } else if (mode == 0) {
+#pragma unroll
+    for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int r = j >> 1;
+        const int dist = min(max(row_limit[r] - 1 - (key0 + nt * 8 + (j & 1)), 0), p.dist_len - 1);
+        s[nt][j] = fmaf(row_bias[r][dist], kLog2e, s[nt][j]);
+      }
+  }
+  if (kMask) {
+#pragma unroll
+    for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int key = key0 + nt * 8 + (j & 1);
+        if (key >= row_limit[j >> 1] || key < row_start[j >> 1]) s[nt][j] = -INFINITY;
+      }
+  }
+}
 
 // Shared-memory tile: [64 tokens][D] bf16, row pitch D * 2 bytes, 16-byte chunks XOR-swizzled with
 // (token & 7) so that ldmatrix rows of consecutive tokens hit different banks.
@@ -165,6 +235,12 @@ __device__ __forceinline__ void warp_tile(WarpState<D>& st, const uint32_t (&qf)
   }
   // scale, soft-cap, mask; running max
   float mx[2] = {-INFINITY, -INFINITY};
+  if (kExt) {
+    const int first = tok0 + t_begin, last = first + NG * 16 - 1;
+    const bool open = last < min(row_limit[0], row_limit[1]) && first >= max(row_start[0], row_start[1]);
+    if (__all_sync(0xffffffffu, open)) ext_scores<NG * 2, false>(s, first + tq * 2, row_limit, row_start, p, row_bias);
+    else ext_scores<NG * 2, true>(s, first + tq * 2, row_limit, row_start, p, row_bias);
+  }
 #pragma unroll
   for (int nt = 0; nt < NG * 2; ++nt) {
 #pragma unroll
@@ -172,12 +248,12 @@ __device__ __forceinline__ void warp_tile(WarpState<D>& st, const uint32_t (&qf)
       const int r = j >> 1;
       const int key = tok0 + t_begin + nt * 8 + tq * 2 + (j & 1);
       float x = s[nt][j];
+      if (kExt) {
+        mx[r] = fmaxf(mx[r], x);
+        continue;
+      }
       if (p.softcap > 0.f) x = p.softcap * tanhf(x * p.scale / p.softcap) * (p.scale_log2 / p.scale);
       else x *= p.scale_log2;
-      if (kExt && p.dist_bias) {
-        const int dist = min(max(row_limit[r] - 1 - key, 0), p.dist_len - 1);
-        x = fmaf(row_bias[r][dist], kLog2e, x);
-      }
       if (key >= row_limit[r] || key < row_start[r]) x = -INFINITY;
       s[nt][j] = x;
       mx[r] = fmaxf(mx[r], x);
@@ -203,7 +279,7 @@ __device__ __forceinline__ void warp_tile(WarpState<D>& st, const uint32_t (&qf)
     float e[4];
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
-      e[j] = exp2f(s[nt][j] - msafe[j >> 1]);
+      e[j] = kExt ? exp2_approx(s[nt][j] - msafe[j >> 1]) : exp2f(s[nt][j] - msafe[j >> 1]);
       rs[j >> 1] += e[j];
     }
     // A fragment of P for the 16-token group nt / 2: (a0, a1) from the even n-tile, (a2, a3)
@@ -485,6 +561,7 @@ attn_prefill_kernel(const AttnParams p) {
   const int q_len = p.cu_q ? p.cu_q[seq + 1] - q_off : p.q_len_single;
   const int kv_len = p.kv_lens ? p.kv_lens[seq] : p.kv_len_single;
   if (qt * 64 >= q_len) return;
+  const int stage_bytes = kExt && p.shared_kv ? kTileBytes : 2 * kTileBytes;
   const int ctx = kv_len - q_len;   // keys that precede the first query token
   const uint32_t smem_base = smem_u32(smem);
 
@@ -521,7 +598,14 @@ attn_prefill_kernel(const AttnParams p) {
   }
   const float* row_bias[2] = {nullptr, nullptr};
   if (kExt) {
-    if (p.dist_bias) row_bias[0] = row_bias[1] = p.dist_bias + static_cast<long long>(head) * p.dist_len;
+    if (p.dist_bias) {
+      row_bias[0] = row_bias[1] = p.dist_bias + static_cast<long long>(head) * p.dist_len;
+      if (p.dist_len <= kDistSmem) {
+        float* tab = reinterpret_cast<float*>(smem + 2 * stage_bytes);
+        for (int i = threadIdx.x; i < p.dist_len; i += kAttnThreads) tab[i] = row_bias[0][i];
+        row_bias[0] = row_bias[1] = tab;                // visible after the first barrier of the tile loop
+      }
+    }
     if (p.sinks) {
       st.m[0] = st.m[1] = p.sinks[head] * kLog2e;
       st.l[0] = st.l[1] = 1.f;
@@ -543,7 +627,7 @@ attn_prefill_kernel(const AttnParams p) {
   __shared__ int pg_ring[4][8];
   auto issue = [&](int tile, int stage) {
     if (tile < n_tiles) {
-      const uint32_t kb = smem_base + stage * 2 * kTileBytes;
+      const uint32_t kb = smem_base + stage * stage_bytes;
       if (kExt) {
         load_tile_paged<D, true>(kb, p.k, pg_ring[tile & 3], kvh, p.hkv, p.page_shift, tile * kTileTokens, kv_needed, p.d);
         if (!p.shared_kv)
@@ -572,7 +656,7 @@ attn_prefill_kernel(const AttnParams p) {
     issue(tile + 1, stage ^ 1);
     cp_async_wait<1>();
     __syncthreads();
-    const uint32_t kb = smem_base + stage * 2 * kTileBytes;
+    const uint32_t kb = smem_base + stage * stage_bytes;
     // a warp whose rows all lie before this tile (causal) still runs: masked scores cost nothing
     // in correctness and keep the barrier pattern uniform
     warp_tile<D, 4, kExt>(st, qf, kb, kExt && p.shared_kv ? kb : kb + kTileBytes, 0, tile * kTileTokens, lim, start, p, row_bias);
@@ -894,6 +978,10 @@ B200_API int b200_attn_biased(const void* q, const void* k_cache, const void* v_
   p.scale = scale;
   p.scale_log2 = scale * kLog2e;
   p.softcap = softcap;
+  if (softcap > 0.f) {
+    p.cap_in = 2.f * kLog2e * scale / softcap;
+    p.cap_out = softcap * kLog2e;
+  }
   p.dist_bias = dist_bias; p.dist_len = dist_len; p.sinks = sinks;
   p.gate = static_cast<const __nv_bfloat16*>(gate);
   p.gate_ld = gate_ld; p.q_ld = q_ld; p.d = d;
@@ -902,13 +990,14 @@ B200_API int b200_attn_biased(const void* q, const void* k_cache, const void* v_
   if (cu_q) {
     if (max_q_len <= 0) return 0;
     const dim3 grid((max_q_len + 63) / 64, hq, seqs);
-    const int smem = 2 * 2 * kTileTokens * dd * 2;
+    const int smem = 2 * (p.shared_kv ? 1 : 2) * kTileTokens * dd * 2 + (dist_bias && dist_len <= kDistSmem ? dist_len * 4 : 0);
+    const int most = 2 * 2 * kTileTokens * dd * 2 + kDistSmem * 4;
     static PerDeviceOnce once[2];
     if (dd == 128) {
-      if (once[1].first_time()) cudaFuncSetAttribute(attn_prefill_kernel<128, true, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+      if (once[1].first_time()) cudaFuncSetAttribute(attn_prefill_kernel<128, true, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, most);
       attn_prefill_kernel<128, true, true><<<grid, kAttnThreads, smem, stream>>>(p);
     } else {
-      if (once[0].first_time()) cudaFuncSetAttribute(attn_prefill_kernel<64, true, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+      if (once[0].first_time()) cudaFuncSetAttribute(attn_prefill_kernel<64, true, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, most);
       attn_prefill_kernel<64, true, true><<<grid, kAttnThreads, smem, stream>>>(p);
     }
     const cudaError_t e = cudaGetLastError();

@@ -44,6 +44,11 @@ __device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
   asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
   return r;
 }
+__device__ __forceinline__ f32x2 add2(f32x2 a, f32x2 b) {
+  f32x2 r;
+  asm("add.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
 __device__ __forceinline__ float sum2(f32x2 v) {
   float a, b;
   unpack2(v, a, b);
@@ -94,7 +99,7 @@ __device__ __forceinline__ float decay_of(float y) { return y < 0.5f ? 1.f + exp
 struct DeltaParams {
   const void* proj;          // [T][ldp]: q (hk * dk) | k (hk * dk) | v (h * dv) | ..., beta logits at b_off
   const void* z;             // [T][ldz]: decay logits (h * dk), then output gate logits (h * dv) at gate_off
-  const float* conv_w;       // [channels][taps]
+  const float* conv_w;       // [taps][channels]
   const float* a;            // [h] decay rate exp(A_log)
   const float* dt_bias;      // [h * dk]
   void* conv_state;          // [slots][taps - 1][channels]
@@ -172,8 +177,10 @@ __global__ void __launch_bounds__(256) delta_prep_kernel(const DeltaParams p) {
       else if (carried) ld4(st + static_cast<long long>(tail + src - first) * channels + c0 + e, x);
       // decode: input j becomes row j - 1 of the state (row j has been read already)
       if (shift && j > 0) st4(st + static_cast<long long>(j - 1) * channels + c0 + e, x);
+      float cw[4];
+      ld4(p.conv_w + static_cast<long long>(j) * channels + c0 + e, cw);
 #pragma unroll
-      for (int i = 0; i < 4; ++i) acc[i] += x[i] * p.conv_w[(c0 + e + i) * p.taps + j];
+      for (int i = 0; i < 4; ++i) acc[i] += x[i] * cw[i];
     }
 #pragma unroll
     for (int i = 0; i < 4; ++i) acc[i] = acc[i] * sigmoid_f32(acc[i]);
@@ -204,6 +211,116 @@ __global__ void __launch_bounds__(256) delta_prep_kernel(const DeltaParams p) {
       for (int i = 0; i < 4; ++i) v[i] = keep[n][i] * inv;
       st4(dst + e, v);
     }
+  }
+}
+
+// The same for four taps and q / k heads of at most 128: a warp keeps one slice of up to 128 channels for
+// `run` consecutive tokens, so that the taps' weights and the previous inputs stay in registers.
+// grid: (ceil(T / (8 run)), 2 hk + ceil(h dv / 128) + ceil(h dk / 128))
+template <typename T>
+__global__ void __launch_bounds__(256) delta_prep4_kernel(const DeltaParams p, int run) {
+  pdl_wait();
+  pdl_trigger();
+  const int lane = threadIdx.x & 31;
+  const int t0 = (blockIdx.x * 8 + (threadIdx.x >> 5)) * run, t1 = min(t0 + run, p.tokens);
+  if (t0 >= t1) return;
+  const int vslices = (p.h * p.dv + 127) / 128;
+  int slice = blockIdx.y;
+  if (slice >= 2 * p.hk + vslices) {      // decay, and beta with the first slice
+    slice -= 2 * p.hk + vslices;
+    const int e = slice * 128 + lane * 4;
+    const bool on = e < p.h * p.dk;
+    float b[4] = {0.f, 0.f, 0.f, 0.f};
+    if (on) ld4(p.dt_bias + e, b);
+    const float a = on ? p.a[e / p.dk] : 0.f;
+    for (int t = t0; t < t1; ++t) {
+      if (on) {
+        float z[4];
+        ld4(static_cast<const T*>(p.z) + static_cast<long long>(t) * p.ldz + e, z);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          const float x = z[j] + b[j];
+          z[j] = decay_of(a * (fmaxf(x, 0.f) + log1pf(expf(-fabsf(x)))));
+        }
+        st4(p.g + static_cast<long long>(t) * p.h * p.dk + e, z);
+      }
+      if (slice == 0)
+        for (int hd = lane; hd < p.h; hd += 32)
+          p.beta[static_cast<long long>(t) * p.h + hd] =
+              sigmoid_f32(ld1(static_cast<const T*>(p.proj) + static_cast<long long>(t) * p.ldp + p.b_off + hd));
+    }
+    return;
+  }
+  const bool is_v = slice >= 2 * p.hk;
+  const int channels = 2 * p.hk * p.dk + p.h * p.dv;
+  const int vbase = 2 * p.hk * p.dk;
+  const int c = (is_v ? vbase + (slice - 2 * p.hk) * 128 : slice * p.dk) + lane * 4;
+  const bool on = is_v ? c < channels : lane * 4 < p.dk;
+  float w[4][4];
+#pragma unroll
+  for (int j = 0; j < 4; ++j)
+#pragma unroll
+    for (int i = 0; i < 4; ++i) w[j][i] = 0.f;
+  if (on)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) ld4(p.conv_w + static_cast<long long>(j) * channels + c, w[j]);
+  const T* x = static_cast<const T*>(p.proj) + c;
+  int seq = p.cu_q ? seq_of_token(p.cu_q, p.seqs, t0) : t0;
+  float in[4][4];                          // inputs of the four taps, oldest first
+  bool fresh = true;
+  int next = 0;                            // first token of the following sequence
+  for (int t = t0; t < t1; ++t) {
+    if (fresh || t >= next) {
+      if (!fresh) ++seq;
+      fresh = false;
+      const int first = p.cu_q ? p.cu_q[seq] : t;
+      next = p.cu_q ? p.cu_q[seq + 1] : t + 1;
+      const int slot = p.slots[seq];
+      const bool carried = slot >= 0 && p.positions[first] > 0;
+      T* st = static_cast<T*>(p.conv_state) + static_cast<long long>(slot < 0 ? 0 : slot) * 3 * channels + c;
+#pragma unroll
+      for (int j = 0; j < 3; ++j) {
+#pragma unroll
+        for (int i = 0; i < 4; ++i) in[j][i] = 0.f;
+        const int src = t - 3 + j;
+        if (!on) continue;
+        if (src >= first) ld4(x + static_cast<long long>(src) * p.ldp, in[j]);
+        else if (carried) ld4(st + static_cast<long long>(3 + src - first) * channels, in[j]);
+      }
+      if (p.cu_q == nullptr && slot >= 0 && on) {       // decode: the state moves on by one token
+        float now[4];
+        ld4(x + static_cast<long long>(t) * p.ldp, now);
+        st4(st, in[1]);
+        st4(st + channels, in[2]);
+        st4(st + 2 * channels, now);
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i) in[3][i] = 0.f;
+    if (on) ld4(x + static_cast<long long>(t) * p.ldp, in[3]);
+    float y[4], sq = 0.f;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      float acc = 0.f;
+#pragma unroll
+      for (int j = 0; j < 4; ++j) acc += in[j][i] * w[j][i];
+      y[i] = acc * sigmoid_f32(acc);
+      sq += y[i] * y[i];
+    }
+    if (is_v) {
+      if (on) st4(p.v + static_cast<long long>(t) * p.h * p.dv + (c - vbase), y);
+    } else {
+      sq = warp_sum(sq);
+      const bool is_q = slice < p.hk;
+      const float inv = (is_q ? p.q_scale : 1.f) / sqrtf(sq + 1e-6f);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) y[i] *= inv;
+      if (on) st4((is_q ? p.q + c : p.k + c - p.hk * p.dk) + static_cast<long long>(t) * p.hk * p.dk, y);
+    }
+#pragma unroll
+    for (int j = 0; j < 3; ++j)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) in[j][i] = in[j + 1][i];
   }
 }
 
@@ -304,57 +421,69 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(const DeltaParams p) {
     const int n = min(kScanTokens, len - t0);
     const float* base = sm + buf * kScanTokens * kTok;
     float* op = p.o + (static_cast<long long>(first + t0) * p.h + head) * p.dv + col;
-#pragma unroll 2
-    for (int tk = 0; tk < n; ++tk) {
-      const float* tb = base + tk * kTok;
-      f32x2 kk[NR * 2];
-      f32x2 a0 = 0, a1 = 0, b0 = 0, b1 = 0;
+    for (int tq = 0; tq < n; tq += 4) {
+      float part[8];                       // reads of four tokens x two columns, this lane's rows
 #pragma unroll
-      for (int i = 0; i < NR; ++i) {
-        const ulonglong2 kv = *reinterpret_cast<const ulonglong2*>(tb + i * 32 + rg * 4);
-        const ulonglong2 gv = *reinterpret_cast<const ulonglong2*>(tb + 2 * DK + i * 32 + rg * 4);
-        kk[i * 2] = kv.x;
-        kk[i * 2 + 1] = kv.y;
-        s0[i * 2] = mul2(s0[i * 2], gv.x);
-        s1[i * 2] = mul2(s1[i * 2], gv.x);
-        s0[i * 2 + 1] = mul2(s0[i * 2 + 1], gv.y);
-        s1[i * 2 + 1] = mul2(s1[i * 2 + 1], gv.y);
-        a0 = fma2(s0[i * 2], kv.x, a0);
-        a1 = fma2(s1[i * 2], kv.x, a1);
-        b0 = fma2(s0[i * 2 + 1], kv.y, b0);
-        b1 = fma2(s1[i * 2 + 1], kv.y, b1);
-      }
-      float r0 = sum2(a0) + sum2(b0), r1 = sum2(a1) + sum2(b1);
+      for (int j = 0; j < 4; ++j) {
+        part[2 * j] = part[2 * j + 1] = 0.f;
+        if (tq + j >= n) continue;
+        const float* tb = base + (tq + j) * kTok;
+        f32x2 kk[NR * 2];
+        f32x2 a0 = 0, a1 = 0, b0 = 0, b1 = 0;
 #pragma unroll
-      for (int o = 1; o < 8; o <<= 1) {
-        r0 += __shfl_xor_sync(0xffffffffu, r0, o);
-        r1 += __shfl_xor_sync(0xffffffffu, r1, o);
-      }
-      const float2 v = *reinterpret_cast<const float2*>(tb + 3 * DK + lc);
-      const float beta = tb[3 * DK + kScanCols];
-      const float u0 = beta * (v.x - r0), u1 = beta * (v.y - r1);
-      const f32x2 uu0 = pack2(u0, u0), uu1 = pack2(u1, u1);
-      a0 = a1 = b0 = b1 = 0;
+        for (int i = 0; i < NR; ++i) {
+          const ulonglong2 kv = *reinterpret_cast<const ulonglong2*>(tb + i * 32 + rg * 4);
+          const ulonglong2 gv = *reinterpret_cast<const ulonglong2*>(tb + 2 * DK + i * 32 + rg * 4);
+          kk[i * 2] = kv.x;
+          kk[i * 2 + 1] = kv.y;
+          s0[i * 2] = mul2(s0[i * 2], gv.x);
+          s1[i * 2] = mul2(s1[i * 2], gv.x);
+          s0[i * 2 + 1] = mul2(s0[i * 2 + 1], gv.y);
+          s1[i * 2 + 1] = mul2(s1[i * 2 + 1], gv.y);
+          a0 = fma2(s0[i * 2], kv.x, a0);
+          a1 = fma2(s1[i * 2], kv.x, a1);
+          b0 = fma2(s0[i * 2 + 1], kv.y, b0);
+          b1 = fma2(s1[i * 2 + 1], kv.y, b1);
+        }
+        float r0 = sum2(add2(a0, b0)), r1 = sum2(add2(a1, b1));
 #pragma unroll
-      for (int i = 0; i < NR; ++i) {
-        const ulonglong2 qv = *reinterpret_cast<const ulonglong2*>(tb + DK + i * 32 + rg * 4);
-        s0[i * 2] = fma2(kk[i * 2], uu0, s0[i * 2]);
-        s1[i * 2] = fma2(kk[i * 2], uu1, s1[i * 2]);
-        s0[i * 2 + 1] = fma2(kk[i * 2 + 1], uu0, s0[i * 2 + 1]);
-        s1[i * 2 + 1] = fma2(kk[i * 2 + 1], uu1, s1[i * 2 + 1]);
-        a0 = fma2(s0[i * 2], qv.x, a0);
-        a1 = fma2(s1[i * 2], qv.x, a1);
-        b0 = fma2(s0[i * 2 + 1], qv.y, b0);
-        b1 = fma2(s1[i * 2 + 1], qv.y, b1);
-      }
-      r0 = sum2(a0) + sum2(b0);
-      r1 = sum2(a1) + sum2(b1);
+        for (int o = 1; o < 8; o <<= 1) {
+          r0 += __shfl_xor_sync(0xffffffffu, r0, o);
+          r1 += __shfl_xor_sync(0xffffffffu, r1, o);
+        }
+        const float2 v = *reinterpret_cast<const float2*>(tb + 3 * DK + lc);
+        const float beta = tb[3 * DK + kScanCols];
+        const float u0 = beta * (v.x - r0), u1 = beta * (v.y - r1);
+        const f32x2 uu0 = pack2(u0, u0), uu1 = pack2(u1, u1);
+        a0 = a1 = b0 = b1 = 0;
 #pragma unroll
-      for (int o = 1; o < 8; o <<= 1) {
-        r0 += __shfl_xor_sync(0xffffffffu, r0, o);
-        r1 += __shfl_xor_sync(0xffffffffu, r1, o);
+        for (int i = 0; i < NR; ++i) {
+          const ulonglong2 qv = *reinterpret_cast<const ulonglong2*>(tb + DK + i * 32 + rg * 4);
+          s0[i * 2] = fma2(kk[i * 2], uu0, s0[i * 2]);
+          s1[i * 2] = fma2(kk[i * 2], uu1, s1[i * 2]);
+          s0[i * 2 + 1] = fma2(kk[i * 2 + 1], uu0, s0[i * 2 + 1]);
+          s1[i * 2 + 1] = fma2(kk[i * 2 + 1], uu1, s1[i * 2 + 1]);
+          a0 = fma2(s0[i * 2], qv.x, a0);
+          a1 = fma2(s1[i * 2], qv.x, a1);
+          b0 = fma2(s0[i * 2 + 1], qv.y, b0);
+          b1 = fma2(s1[i * 2 + 1], qv.y, b1);
+        }
+        part[2 * j] = sum2(add2(a0, b0));
+        part[2 * j + 1] = sum2(add2(a1, b1));
       }
-      if (rg == 0 && live) *reinterpret_cast<float2*>(op + static_cast<long long>(tk) * p.h * p.dv) = make_float2(r0, r1);
+      // the eight lanes of a column pair add their parts: every exchange halves the values a lane keeps,
+      // and lane rg ends with token tq + rg / 2, column rg % 2
+#pragma unroll
+      for (int o = 4, cnt = 4; o > 0; o >>= 1, cnt >>= 1) {
+        const bool up = (rg & o) != 0;
+#pragma unroll
+        for (int i = 0; i < cnt; ++i) {
+          const float keep = up ? part[i + cnt] : part[i], give = up ? part[i] : part[i + cnt];
+          part[i] = keep + __shfl_xor_sync(0xffffffffu, give, o);
+        }
+      }
+      const int tk = tq + (rg >> 1);
+      if (live && tk < n) op[static_cast<long long>(tk) * p.h * p.dv + (rg & 1)] = part[0];
     }
     __syncthreads();
   }
@@ -409,8 +538,10 @@ __global__ void __launch_bounds__(256) delta_gate_kernel(const DeltaParams p) {
 // NRT rows. Dynamic shared memory: (3 dk + (rgs + 1) dv + 32) floats.
 constexpr int kStepThreads = 768;   // most threads of a decode block; larger heads are scanned
 
-template <typename T, int NRT>
-__global__ void __launch_bounds__(kStepThreads) delta_step_kernel(const DeltaParams p) {
+// kMax: most threads of this instance (two blocks of up to 512 share an SM, so that one loads while the
+// other computes)
+template <typename T, int NRT, int kMax>
+__global__ void __launch_bounds__(kMax, kMax <= 512 ? 2 : 1) delta_step_kernel(const DeltaParams p) {
   extern __shared__ __align__(16) float sm[];
   const int head = blockIdx.x, seq = blockIdx.y, tid = threadIdx.x;
   const int cgs = p.dv >> 2, cg = tid % cgs, rg = tid / cgs, rgs = blockDim.x / cgs;
@@ -498,19 +629,31 @@ cudaError_t launch_scan(const DeltaParams& p, cudaStream_t stream) {
   return launch_pdl(delta_scan_kernel<NR>, dim3((p.dv + kScanCols - 1) / kScanCols, p.h, p.seqs), dim3(128), smem, stream, p);
 }
 
-template <typename T, int NRT>
-cudaError_t launch_step(const DeltaParams& p, int threads, cudaStream_t stream) {
+template <typename T, int NRT, int kMax>
+cudaError_t launch_step_of(const DeltaParams& p, int threads, cudaStream_t stream) {
   const int rgs = threads / (p.dv / 4);
   const int smem = (3 * p.dk + (rgs + 1) * p.dv + 32) * 4;
   static PerDeviceOnce once;
-  if (once.first_time()) cudaFuncSetAttribute(delta_step_kernel<T, NRT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024);
-  return launch_pdl(delta_step_kernel<T, NRT>, dim3(p.h, p.seqs), dim3(threads), smem, stream, p);
+  if (once.first_time()) cudaFuncSetAttribute(delta_step_kernel<T, NRT, kMax>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024);
+  return launch_pdl(delta_step_kernel<T, NRT, kMax>, dim3(p.h, p.seqs), dim3(threads), smem, stream, p);
+}
+
+template <typename T, int NRT>
+cudaError_t launch_step(const DeltaParams& p, int threads, cudaStream_t stream) {
+  return threads <= 512 ? launch_step_of<T, NRT, 512>(p, threads, stream) : launch_step_of<T, NRT, kStepThreads>(p, threads, stream);
 }
 
 template <typename T>
 int delta_impl(const DeltaParams& p, cudaStream_t stream) {
   const bool decode = p.cu_q == nullptr;
-  cudaError_t e = launch_pdl(delta_prep_kernel<T>, dim3((p.tokens + 7) / 8, 2 * p.hk + 2 * p.h), dim3(256), 0, stream, p);
+  cudaError_t e;
+  if (p.taps == 4 && p.dk <= 128) {
+    const int slices = 2 * p.hk + (p.h * p.dv + 127) / 128 + (p.h * p.dk + 127) / 128;
+    const int run = decode || static_cast<long long>(p.tokens) * slices < 148 * 64 * 8 ? 1 : 8;
+    e = launch_pdl(delta_prep4_kernel<T>, dim3((p.tokens + 8 * run - 1) / (8 * run), slices), dim3(256), 0, stream, p, run);
+  } else {
+    e = launch_pdl(delta_prep_kernel<T>, dim3((p.tokens + 7) / 8, 2 * p.hk + 2 * p.h), dim3(256), 0, stream, p);
+  }
   if (e != cudaSuccess) return -static_cast<int>(e) - 300;
   if (decode) {
     const int cgs = p.dv / 4;

@@ -2,12 +2,14 @@
 //
 //  * b200_linear_f32: x (fp32 or bf16) times a bf16 weight, fp32 accumulation and output: the dense
 //    linears of a model that is run in 32 bits. Plain FMA tiles, no reduced-precision mode.
-//  * b200_router: router logits, scores and top-k of a mixture of experts in one kernel. The token
-//    rows of a block sit in shared memory as fp32, a warp takes four experts at a time, the logits
-//    stay in shared memory, and one warp per token turns them into scores and picks the experts.
+//  * b200_router: router logits, scores and top-k of a mixture of experts in one kernel. The logits of
+//    a block of tokens stay in shared memory as fp32, and one warp per token turns them into scores and
+//    picks the experts. Few tokens: fp32 FMA with the token rows in shared memory, one expert per warp.
+//    Many bf16 tokens: bf16 tensor-core products, which are exact, accumulated in fp32.
 //  * b200_pair_linear_f32: one weight matrix per (token, choice) pair, the expert products of the
 //    32-bit mode.
 #include "common.cuh"
+#include "mma_sync.cuh"
 
 namespace b200 {
 
@@ -79,11 +81,63 @@ struct RouterParams {
   float scale;
 };
 
-constexpr int kRouterExpertsPerWarp = 4;
+// Order-preserving map of a float to an unsigned integer (for warp-wide integer max)
+__device__ __forceinline__ unsigned ordered_bits(float v) {
+  const unsigned u = __float_as_uint(v);
+  return (u >> 31) ? ~u : u | 0x80000000u;
+}
 
-// kTok tokens per block; k is a multiple of 8. Dynamic shared memory: kTok * (k + experts) floats.
+// One warp: logits row [experts] in shared memory -> scores (in place), top-k by score + bias, ties to the
+// lowest index. A chosen expert's score is stored with its sign bit set so that later rounds pass over it
+// (scores are never negative).
+__device__ __forceinline__ void route_row(float* row, const RouterParams& p, int t) {
+  const int lane = threadIdx.x & 31;
+  if (p.sigmoid) {
+    for (int e = lane; e < p.experts; e += 32) row[e] = 1.f / (1.f + expf(-row[e]));
+  } else {
+    float mx = -INFINITY;
+    for (int e = lane; e < p.experts; e += 32) mx = fmaxf(mx, row[e]);
+    mx = warp_max(mx);
+    float s = 0.f;
+    for (int e = lane; e < p.experts; e += 32) {
+      const float v = expf(row[e] - mx);
+      row[e] = v;
+      s += v;
+    }
+    s = warp_sum(s);
+    for (int e = lane; e < p.experts; e += 32) row[e] /= s;
+  }
+  float wsum = 0.f, my_w = 0.f;
+  int my_id = 0;
+  for (int r = 0; r < p.top_k; ++r) {
+    unsigned best = 0;
+    int idx = 0x7fffffff;
+    for (int e = lane; e < p.experts; e += 32) {
+      const float s = row[e];
+      if (__float_as_uint(s) >> 31) continue;
+      const unsigned key = ordered_bits(s + (p.bias ? p.bias[e] : 0.f));
+      if (key > best) { best = key; idx = e; }
+    }
+    const unsigned top = __reduce_max_sync(0xffffffffu, best);
+    idx = __reduce_min_sync(0xffffffffu, best == top ? idx : 0x7fffffff);
+    if (idx >= p.experts) idx = r < p.experts ? r : 0;      // only with scores that are not numbers
+    const float raw = __uint_as_float(__float_as_uint(row[idx]) & 0x7fffffffu);
+    __syncwarp();
+    if (lane == 0) row[idx] = __uint_as_float(__float_as_uint(raw) | 0x80000000u);
+    __syncwarp();
+    if (lane == r) { my_w = raw; my_id = idx; }
+    wsum += raw;
+  }
+  if (lane < p.top_k) {
+    p.ids[static_cast<long long>(t) * p.top_k + lane] = my_id;
+    p.wts[static_cast<long long>(t) * p.top_k + lane] = (p.norm_topk ? my_w / (wsum + 1e-20f) : my_w) * p.scale;
+  }
+}
+
+// Few tokens (and the 32-bit mode): kTok tokens per block in shared memory as fp32, one expert per warp and
+// turn. k is a multiple of 8. Dynamic shared memory: kTok * (k + experts) floats.
 template <typename T, int kTok>
-__global__ void __launch_bounds__(256) router_kernel(const RouterParams p) {
+__global__ void __launch_bounds__(kTok > 2 ? 512 : 1024) router_kernel(const RouterParams p) {
   pdl_wait();
   pdl_trigger();
   extern __shared__ __align__(16) float sm[];
@@ -91,115 +145,148 @@ __global__ void __launch_bounds__(256) router_kernel(const RouterParams p) {
   float* lg = sm + kTok * p.k;          // [kTok][experts]
   const int t0 = blockIdx.x * kTok;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
-  for (int i = threadIdx.x; i < kTok * p.k; i += blockDim.x) {
-    const int r = i / p.k, c = i - r * p.k;
-    xs[i] = t0 + r < p.tokens ? to_f32(static_cast<const T*>(p.x)[static_cast<long long>(t0 + r) * p.ldx + c]) : 0.f;
+#pragma unroll
+  for (int r = 0; r < kTok; ++r) {
+    const T* xr = static_cast<const T*>(p.x) + static_cast<long long>(min(t0 + r, p.tokens - 1)) * p.ldx;
+    for (int c = threadIdx.x; c < p.k; c += blockDim.x) xs[r * p.k + c] = to_f32(xr[c]);
   }
   __syncthreads();
-  for (int e0 = warp * kRouterExpertsPerWarp; e0 < p.experts; e0 += warps * kRouterExpertsPerWarp) {
-    float acc[kRouterExpertsPerWarp][kTok];
+  for (int e = warp; e < p.experts; e += warps) {
+    float acc[kTok];
 #pragma unroll
-    for (int i = 0; i < kRouterExpertsPerWarp; ++i)
-#pragma unroll
-      for (int j = 0; j < kTok; ++j) acc[i][j] = 0.f;
+    for (int j = 0; j < kTok; ++j) acc[j] = 0.f;
+    const __nv_bfloat16* wr = p.w + static_cast<long long>(e) * p.ldw;
+#pragma unroll 4
     for (int c = lane * 8; c < p.k; c += 256) {
-      float wv[kRouterExpertsPerWarp][8];
+      const uint4 raw = *reinterpret_cast<const uint4*>(wr + c);
+      const __nv_bfloat162* b = reinterpret_cast<const __nv_bfloat162*>(&raw);
+      float wv[8];
 #pragma unroll
-      for (int i = 0; i < kRouterExpertsPerWarp; ++i) {
-        const int e = e0 + i < p.experts ? e0 + i : p.experts - 1;
-        const uint4 raw = *reinterpret_cast<const uint4*>(p.w + static_cast<long long>(e) * p.ldw + c);
-        const __nv_bfloat162* b = reinterpret_cast<const __nv_bfloat162*>(&raw);
-#pragma unroll
-        for (int q = 0; q < 4; ++q) {
-          const float2 f = __bfloat1622float2(b[q]);
-          wv[i][2 * q] = f.x;
-          wv[i][2 * q + 1] = f.y;
-        }
+      for (int q = 0; q < 4; ++q) {
+        const float2 f = __bfloat1622float2(b[q]);
+        wv[2 * q] = f.x;
+        wv[2 * q + 1] = f.y;
       }
 #pragma unroll
       for (int j = 0; j < kTok; ++j) {
-        const float4 a = *reinterpret_cast<const float4*>(xs + j * p.k + c);
-        const float4 b = *reinterpret_cast<const float4*>(xs + j * p.k + c + 4);
-#pragma unroll
-        for (int i = 0; i < kRouterExpertsPerWarp; ++i) {
-          acc[i][j] += a.x * wv[i][0] + a.y * wv[i][1] + a.z * wv[i][2] + a.w * wv[i][3];
-          acc[i][j] += b.x * wv[i][4] + b.y * wv[i][5] + b.z * wv[i][6] + b.w * wv[i][7];
-        }
+        const float4 u = *reinterpret_cast<const float4*>(xs + j * p.k + c);
+        const float4 v = *reinterpret_cast<const float4*>(xs + j * p.k + c + 4);
+        acc[j] += u.x * wv[0] + u.y * wv[1] + u.z * wv[2] + u.w * wv[3];
+        acc[j] += v.x * wv[4] + v.y * wv[5] + v.z * wv[6] + v.w * wv[7];
       }
     }
 #pragma unroll
-    for (int i = 0; i < kRouterExpertsPerWarp; ++i)
+    for (int j = 0; j < kTok; ++j) {
+      const float s = warp_sum(acc[j]);
+      if (lane == 0) lg[j * p.experts + e] = s;
+    }
+  }
+  __syncthreads();
+  for (int j = warp; j < kTok; j += warps)
+    if (t0 + j < p.tokens) route_row(lg + j * p.experts, p, t0 + j);
+}
+
+// Many bf16 tokens: 32 tokens per block, bf16 products with fp32 accumulation on the tensor core (m16n8k16),
+// experts in passes of 128. Warp (wm, wn): tokens 16 wm.., experts 64 wn.. of the pass. Dynamic shared memory:
+// 32 * experts floats, then two stages of [32 + 128] rows of 64 values (16-byte chunks XOR-swizzled by row).
+constexpr int kRtTok = 32, kRtExp = 128, kRtK = 64;
+
+__global__ void __launch_bounds__(128) router_tc_kernel(const RouterParams p) {
+  pdl_wait();
+  pdl_trigger();
+  extern __shared__ __align__(128) uint8_t smraw[];
+  constexpr int kStage = (kRtTok + kRtExp) * kRtK * 2;
+  float* lg = reinterpret_cast<float*>(smraw + 2 * kStage);
+  const uint32_t base = smem_u32(smraw);
+  const int t0 = blockIdx.x * kRtTok;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, wm = warp & 1, wn = warp >> 1;
+  const auto* x = static_cast<const __nv_bfloat16*>(p.x);
+  const int nk = (p.k + kRtK - 1) / kRtK;
+  for (int e0 = 0; e0 < p.experts; e0 += kRtExp) {
+    auto load = [&](int kb, int st) {
+      if (kb < nk) {
+        for (int i = threadIdx.x; i < (kRtTok + kRtExp) * 8; i += 128) {
+          const int r = i >> 3, c = i & 7, col = kb * kRtK + c * 8;
+          const __nv_bfloat16* src = x;
+          bool ok = col < p.k;
+          if (r < kRtTok) {
+            ok = ok && t0 + r < p.tokens;
+            if (ok) src = x + static_cast<long long>(t0 + r) * p.ldx + col;
+          } else {
+            const int e = e0 + r - kRtTok;
+            ok = ok && e < p.experts;
+            if (ok) src = p.w + static_cast<long long>(e) * p.ldw + col;
+          }
+          cp_async_16(base + st * kStage + r * (kRtK * 2) + ((c ^ (r & 7)) << 4), src, ok);
+        }
+      }
+      cp_async_commit();
+    };
+    float acc[8][4];
 #pragma unroll
-      for (int j = 0; j < kTok; ++j) {
-        const float s = warp_sum(acc[i][j]);
-        if (lane == 0 && e0 + i < p.experts) lg[j * p.experts + e0 + i] = s;
+    for (int i = 0; i < 8; ++i)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
+    load(0, 0);
+    for (int kb = 0; kb < nk; ++kb) {
+      load(kb + 1, (kb + 1) & 1);
+      cp_async_wait<1>();
+      __syncthreads();
+      const uint32_t st = base + (kb & 1) * kStage;
+#pragma unroll
+      for (int kk = 0; kk < kRtK / 16; ++kk) {
+        uint32_t a[4];
+        const int ar = wm * 16 + (lane & 15), ac = kk * 2 + (lane >> 4);
+        ldmatrix_x4(st + ar * (kRtK * 2) + ((ac ^ (ar & 7)) << 4), a[0], a[1], a[2], a[3]);
+#pragma unroll
+        for (int g = 0; g < 4; ++g) {
+          const int mi = lane >> 3;
+          const int br = kRtTok + wn * 64 + g * 16 + (lane & 7) + 8 * (mi >> 1), bc = kk * 2 + (mi & 1);
+          uint32_t b0, b1, b2, b3;
+          ldmatrix_x4(st + br * (kRtK * 2) + ((bc ^ (br & 7)) << 4), b0, b1, b2, b3);
+          mma_bf16_16816(acc[g * 2], a, b0, b1);
+          mma_bf16_16816(acc[g * 2 + 1], a, b2, b3);
+        }
+      }
+      __syncthreads();
+    }
+    cp_async_wait<0>();
+    const int row = wm * 16 + (lane >> 2);
+#pragma unroll
+    for (int g = 0; g < 8; ++g)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int e = e0 + wn * 64 + g * 8 + (lane & 3) * 2 + (j & 1);
+        if (e < p.experts) lg[(row + 8 * (j >> 1)) * p.experts + e] = acc[g][j];
       }
   }
   __syncthreads();
-  for (int j = warp; j < kTok; j += warps) {
-    const int t = t0 + j;
-    if (t >= p.tokens) continue;
-    float* row = lg + j * p.experts;
-    if (p.sigmoid) {
-      for (int e = lane; e < p.experts; e += 32) row[e] = 1.f / (1.f + expf(-row[e]));
-    } else {
-      float mx = -INFINITY;
-      for (int e = lane; e < p.experts; e += 32) mx = fmaxf(mx, row[e]);
-      mx = warp_max(mx);
-      float s = 0.f;
-      for (int e = lane; e < p.experts; e += 32) {
-        const float v = expf(row[e] - mx);
-        row[e] = v;
-        s += v;
-      }
-      s = warp_sum(s);
-      for (int e = lane; e < p.experts; e += 32) row[e] /= s;
-    }
-    // top-k by score + bias, ties to the lowest index; a chosen expert's score is stored negated so
-    // that later rounds pass over it (scores are never negative)
-    float wsum = 0.f, my_w = 0.f;
-    int my_id = 0;
-    for (int r = 0; r < p.top_k; ++r) {
-      float best = -INFINITY, raw = 0.f;
-      int idx = 0x7fffffff;
-      for (int e = lane; e < p.experts; e += 32) {
-        const float s = row[e];
-        if (__float_as_uint(s) >> 31) continue;
-        const float v = s + (p.bias ? p.bias[e] : 0.f);
-        if (v > best) { best = v; idx = e; raw = s; }
-      }
-      for (int o = 16; o > 0; o >>= 1) {
-        const float ov = __shfl_xor_sync(0xffffffffu, best, o), orw = __shfl_xor_sync(0xffffffffu, raw, o);
-        const int oi = __shfl_xor_sync(0xffffffffu, idx, o);
-        if (ov > best || (ov == best && oi < idx)) { best = ov; idx = oi; raw = orw; }
-      }
-      if (idx >= p.experts) idx = r < p.experts ? r : 0;      // only with scores that are not numbers
-      if ((idx & 31) == lane) row[idx] = __uint_as_float(__float_as_uint(row[idx]) | 0x80000000u);
-      __syncwarp();
-      if (lane == r) { my_w = raw; my_id = idx; }
-      wsum += raw;
-    }
-    if (lane < p.top_k) {
-      p.ids[static_cast<long long>(t) * p.top_k + lane] = my_id;
-      p.wts[static_cast<long long>(t) * p.top_k + lane] = (p.norm_topk ? my_w / (wsum + 1e-20f) : my_w) * p.scale;
-    }
-  }
+  for (int j = warp; j < kRtTok; j += 4)
+    if (t0 + j < p.tokens) route_row(lg + j * p.experts, p, t0 + j);
 }
 
 template <typename T>
-int launch_router(const RouterParams& p, cudaStream_t stream) {
+int launch_router(const RouterParams& p, bool tensor_cores, cudaStream_t stream) {
   const int limit = 200 * 1024;
+  cudaError_t e;
+  const int tc_bytes = 2 * (kRtTok + kRtExp) * kRtK * 2 + kRtTok * p.experts * 4;
+  if (tensor_cores && p.tokens > 4 * 148 && tc_bytes <= limit && p.ldx % 8 == 0) {
+    static PerDeviceOnce once_tc;
+    if (once_tc.first_time()) cudaFuncSetAttribute(router_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, limit);
+    e = launch_pdl(router_tc_kernel, dim3((p.tokens + kRtTok - 1) / kRtTok), dim3(128), tc_bytes, stream, p);
+    return e == cudaSuccess ? 0 : -static_cast<int>(e) - 300;
+  }
   auto bytes = [&](int tok) { return tok * (p.k + p.experts) * 4; };
   // enough blocks to cover the machine first, then as many tokens per read of the weights as fit
-  int tok = p.tokens >= 4 * 148 ? 8 : p.tokens >= 2 * 148 ? 4 : p.tokens >= 148 ? 2 : 1;
+  int tok = p.tokens >= 4 * 148 ? 8 : p.tokens >= 2 * 148 ? 4 : p.tokens > 148 ? 2 : 1;
   while (tok > 1 && bytes(tok) > limit / 2) tok /= 2;
   if (bytes(tok) > limit) return -2;
+  const int threads = p.experts > 16 ? (tok > 2 ? 512 : 1024) : 512;
   auto go = [&](auto kernel, int n, PerDeviceOnce& once) {
     if (once.first_time()) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, limit);
-    return launch_pdl(kernel, dim3((p.tokens + n - 1) / n), dim3(256), bytes(n), stream, p);
+    return launch_pdl(kernel, dim3((p.tokens + n - 1) / n), dim3(threads), bytes(n), stream, p);
   };
   static PerDeviceOnce once[4];
-  cudaError_t e;
   switch (tok) {
     case 8: e = go(router_kernel<T, 8>, 8, once[3]); break;
     case 4: e = go(router_kernel<T, 4>, 4, once[2]); break;
@@ -256,7 +343,7 @@ B200_API int b200_router(const void* x, int x_f32, const void* w, const float* b
   if (k % 8 || ldw % 8 || top_k < 1 || top_k > 32 || top_k > experts) return -2;
   RouterParams p{x, static_cast<const __nv_bfloat16*>(w), bias, ids, wts, tokens, experts, k, ldx, ldw, top_k, sigmoid,
                  norm_topk, scale};
-  return x_f32 ? launch_router<float>(p, stream) : launch_router<__nv_bfloat16>(p, stream);
+  return x_f32 ? launch_router<float>(p, false, stream) : launch_router<__nv_bfloat16>(p, true, stream);
 }
 
 B200_API int b200_pair_linear_f32(const void* x, const void* w, const int* ids, void* out, int pairs, int div, int experts,

@@ -185,6 +185,53 @@ __global__ void moe_plan_kernel(const int* __restrict__ counts, int* __restrict_
     for (int b = s_start[e]; b < s_start[e + 1] && b < max_blocks; ++b) block_group[b] = e;
   }
 }
+// passes 1 and 2 in one block, for lists that one block gets through quickly: counts and block starts stay in
+// shared memory, slots come out directly
+constexpr int kSmallPairs = 4096;
+__global__ void __launch_bounds__(1024) moe_plan_small_kernel(const int* __restrict__ topk_ids, int* __restrict__ slot_of,
+                                                              int* __restrict__ block_group, int* __restrict__ dyn_blocks,
+                                                              int pairs, int e0, int e_local, int cap, int max_blocks) {
+  pdl_wait();
+  pdl_trigger();
+  __shared__ int cnt[1024], start[1024], wsum[32];
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  cnt[tid] = 0;
+  __syncthreads();
+  int e[kSmallPairs / 1024], pos[kSmallPairs / 1024];
+#pragma unroll
+  for (int j = 0; j < kSmallPairs / 1024; ++j) {
+    const int i = tid + j * 1024;
+    e[j] = i < pairs ? topk_ids[i] - e0 : -1;
+    pos[j] = e[j] >= 0 && e[j] < e_local ? atomicAdd(&cnt[e[j]], 1) : -1;
+  }
+  __syncthreads();
+  const int nb = tid < e_local ? (cnt[tid] + cap - 1) / cap : 0;
+  int incl = nb;
+#pragma unroll
+  for (int o = 1; o < 32; o <<= 1) {
+    const int v = __shfl_up_sync(0xffffffffu, incl, o);
+    if (lane >= o) incl += v;
+  }
+  if (lane == 31) wsum[warp] = incl;
+  __syncthreads();
+  int before = 0;
+  for (int i = 0; i < warp; ++i) before += wsum[i];
+  start[tid] = before + incl - nb;
+  for (int b = start[tid]; b < start[tid] + nb && b < max_blocks; ++b) block_group[b] = tid;
+  if (tid == 1023) *dyn_blocks = min(before + incl, max_blocks);
+  __syncthreads();
+#pragma unroll
+  for (int j = 0; j < kSmallPairs / 1024; ++j) {
+    const int i = tid + j * 1024;
+    if (i >= pairs) continue;
+    int slot = -1;
+    if (pos[j] >= 0) {
+      const int blk = start[e[j]] + pos[j] / cap;
+      if (blk < max_blocks) slot = blk * cap + pos[j] % cap;
+    }
+    slot_of[i] = slot;
+  }
+}
 // pass 3: copy rows into their slots
 __global__ void moe_scatter_dynamic_kernel(const __nv_bfloat16* __restrict__ x, __nv_bfloat16* __restrict__ xs,
                                            const int* __restrict__ topk_ids, const int* __restrict__ pos_of,
@@ -208,6 +255,8 @@ __global__ void moe_scatter_dynamic_kernel(const __nv_bfloat16* __restrict__ x, 
 // Copies token rows into their slots (bf16 rows of `dim`, 16-byte vectors). One block per pair.
 __global__ void moe_scatter_kernel(const __nv_bfloat16* __restrict__ x, __nv_bfloat16* __restrict__ xs,
                                    const int* __restrict__ slot_of, int top_k, int dim) {
+  pdl_wait();
+  pdl_trigger();
   const int pair = blockIdx.x;
   const int slot = slot_of[pair];
   if (slot < 0) return;
@@ -253,7 +302,39 @@ __global__ void moe_combine_kernel(const __nv_bfloat16* __restrict__ y, const in
 // Clamped gate of an expert: y = g sigmoid(alpha g) (u + 1), g = min(gate, limit), u = clamp(up, +-limit),
 // for x [rows][2 f] = gate | up. With a block list only the rows of the blocks in use are computed.
 template <typename T>
-__device__ __forceinline__ float glu_ld(const T* p) { return static_cast<float>(*p); }
+struct Vec8;
+template <>
+struct Vec8<__nv_bfloat16> {
+  static __device__ __forceinline__ void load(const __nv_bfloat16* p, float (&v)[8]) {
+    const uint4 raw = *reinterpret_cast<const uint4*>(p);
+    const __nv_bfloat162* b = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const float2 f = __bfloat1622float2(b[i]);
+      v[2 * i] = f.x;
+      v[2 * i + 1] = f.y;
+    }
+  }
+  static __device__ __forceinline__ void store(__nv_bfloat16* p, const float (&v)[8]) {
+    *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]), pack_bf16x2(v[4], v[5]),
+                                              pack_bf16x2(v[6], v[7]));
+  }
+  // bf16 results: the hardware exponential and reciprocal are more than exact enough
+  static __device__ __forceinline__ float gated(float a, float alpha) { return __fdividef(a, 1.f + __expf(-alpha * a)); }
+};
+template <>
+struct Vec8<float> {
+  static __device__ __forceinline__ void load(const float* p, float (&v)[8]) {
+#pragma unroll
+    for (int i = 0; i < 8; ++i) v[i] = p[i];
+  }
+  static __device__ __forceinline__ void store(float* p, const float (&v)[8]) {
+#pragma unroll
+    for (int i = 0; i < 8; ++i) p[i] = v[i];
+  }
+  static __device__ __forceinline__ float gated(float a, float alpha) { return a / (1.f + expf(-alpha * a)); }
+};
+
 template <typename T>
 __global__ void __launch_bounds__(256) glu_clamped_kernel(const T* __restrict__ x, T* __restrict__ y, long long rows, int f,
                                                           float limit, float alpha, const int* __restrict__ dyn_blocks, int cap) {
@@ -263,21 +344,26 @@ __global__ void __launch_bounds__(256) glu_clamped_kernel(const T* __restrict__ 
     const long long used = static_cast<long long>(*dyn_blocks) * cap;
     rows = used < rows ? used : rows;
   }
-  const int pairs = f >> 1;
-  const long long total = rows * pairs;
+  const unsigned vecs = f >> 3;
+  const long long total = rows * vecs;
   for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < total;
        i += static_cast<long long>(gridDim.x) * blockDim.x) {
-    const long long r = i / pairs;
-    const int c = static_cast<int>(i - r * pairs) * 2;
-    const T* g = x + r * 2 * f + c;
-    float o[2];
-#pragma unroll
-    for (int j = 0; j < 2; ++j) {
-      const float a = fminf(glu_ld(g + j), limit), u = fminf(fmaxf(glu_ld(g + f + j), -limit), limit);
-      o[j] = a / (1.f + expf(-alpha * a)) * (u + 1.f);
+    long long r;
+    unsigned c;
+    if (total <= 0xffffffffll) {
+      r = static_cast<unsigned>(i) / vecs;
+      c = static_cast<unsigned>(i) % vecs * 8;
+    } else {
+      r = i / vecs;
+      c = static_cast<unsigned>(i - r * vecs) * 8;
     }
-    y[r * f + c] = static_cast<T>(o[0]);
-    y[r * f + c + 1] = static_cast<T>(o[1]);
+    float g[8], u[8];
+    Vec8<T>::load(x + r * 2 * f + c, g);
+    Vec8<T>::load(x + r * 2 * f + f + c, u);
+#pragma unroll
+    for (int j = 0; j < 8; ++j)
+      g[j] = Vec8<T>::gated(fminf(g[j], limit), alpha) * (fminf(fmaxf(u[j], -limit), limit) + 1.f);
+    Vec8<T>::store(y + r * f + c, g);
   }
 }
 
@@ -285,13 +371,13 @@ __global__ void __launch_bounds__(256) glu_clamped_kernel(const T* __restrict__ 
 
 using namespace b200;
 
-// f even. dyn_blocks (may be null): only the first *dyn_blocks * cap rows are in use.
+// f a multiple of 8. dyn_blocks (may be null): only the first *dyn_blocks * cap rows are in use.
 B200_API int b200_glu_clamped(const void* x, void* y, long long rows, int f, float limit, float alpha, const int* dyn_blocks,
                               int cap, int f32, cudaStream_t stream) {
   if (rows <= 0) return 0;
-  if (f % 2) return -2;
-  long long blocks = (rows * (f / 2) + 255) / 256;
-  if (blocks > 148 * 16) blocks = 148 * 16;
+  if (f % 8) return -2;
+  long long blocks = (rows * (f / 8) + 255) / 256;
+  if (blocks > 148 * 8) blocks = 148 * 8;
   const cudaError_t e =
       f32 ? launch_pdl(glu_clamped_kernel<float>, dim3(static_cast<unsigned>(blocks)), dim3(256), 0, stream,
                        static_cast<const float*>(x), static_cast<float*>(y), rows, f, limit, alpha, dyn_blocks, cap)
@@ -338,6 +424,14 @@ B200_API int b200_moe_dispatch_dynamic(const void* x, void* xs, const int* topk_
   if (tokens <= 0) return 0;
   if (dim % 8 || e_local > 1024 || cap < 1) return -2;
   const int pairs = tokens * top_k;
+  if (pairs <= kSmallPairs) {
+    cudaError_t e = launch_pdl(moe_plan_small_kernel, dim3(1), dim3(1024), 0, stream, topk_ids, slot_of, block_group, dyn_blocks,
+                               pairs, e0, e_local, cap, max_blocks);
+    if (e == cudaSuccess)
+      e = launch_pdl(moe_scatter_kernel, dim3(pairs), dim3(128), 0, stream, static_cast<const __nv_bfloat16*>(x),
+                     static_cast<__nv_bfloat16*>(xs), static_cast<const int*>(slot_of), top_k, dim);
+    return e == cudaSuccess ? 0 : -static_cast<int>(e) - 300;
+  }
   int* counts = scratch;
   int* block_start = scratch + e_local;
   int* pos_of = scratch + 2 * e_local;

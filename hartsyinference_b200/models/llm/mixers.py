@@ -141,7 +141,7 @@ class DeltaMixer:
         self.o = _linear([pad_rows(pad_head_cols(o, h, dv, dvp), wp)], device)
         f32 = lambda t: t.float().to(device).contiguous()
         taps = torch.cat([pad_head_rows(conv[0], hk, d, dp), pad_head_rows(conv[1], hk, d, dp), pad_head_rows(conv[2], h, dv, dvp)])
-        self.w = ops.DeltaWeights(conv=f32(taps), decay_rate=f32(a_log.float().exp()), dt_bias=f32(pad_head_rows(dt_bias, h, d, dp)),
+        self.w = ops.DeltaWeights(conv=f32(taps.t()), decay_rate=f32(a_log.float().exp()), dt_bias=f32(pad_head_rows(dt_bias, h, d, dp)),
                                   norm=torch.nn.functional.pad(norm, (0, dvp - dv)).to(torch.bfloat16).to(device).contiguous(),
                                   heads=h, kv_heads=hk, dk=dp, dv=dvp, dk_true=d, dv_true=dv, eps=eps)
 
@@ -150,7 +150,7 @@ class DeltaMixer:
 
     def state_shapes(self, slots: int) -> tuple[tuple, tuple]:
         w = self.w
-        return (slots, w.conv.shape[1] - 1, w.channels), (slots, w.heads, w.dk, w.dv)
+        return (slots, w.conv.shape[0] - 1, w.channels), (slots, w.heads, w.dk, w.dv)
 
     def __call__(self, h: torch.Tensor, batch, li: int, model) -> torch.Tensor:
         p = ops.linear_act(h, self.proj)

@@ -946,7 +946,7 @@ def moe_dispatch_dynamic(x: torch.Tensor, topk_ids: torch.Tensor, e0: int, e_loc
     dev = x.device
     slot_of = torch.empty(t, k, dtype=torch.int32, device=dev)
     scratch = torch.empty(2 * e_local + t * k, dtype=torch.int32, device=dev)
-    block_group = torch.zeros(max_blocks, dtype=torch.int32, device=dev)
+    block_group = torch.empty(max_blocks, dtype=torch.int32, device=dev)      # entries past the blocks in use are never read
     dyn = torch.empty(1, dtype=torch.int32, device=dev)
     rc = N.lib().b200_moe_dispatch_dynamic(x.data_ptr(), xs.data_ptr(), topk_ids.data_ptr(), slot_of.data_ptr(),
                                            scratch.data_ptr(), block_group.data_ptr(), dyn.data_ptr(), t, k, dim, e0,

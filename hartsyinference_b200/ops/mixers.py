@@ -241,7 +241,7 @@ def attn_biased(q: torch.Tensor, k_cache: torch.Tensor, v_cache: Optional[torch.
 class DeltaWeights:
     """Constants of one delta-rule mixer. ``dk`` / ``dv`` are the head sizes as laid out (padded with zero
     channels), ``dk_true`` / ``dv_true`` the model's."""
-    conv: torch.Tensor         # fp32 [channels, taps], channels = q heads | k heads | v heads
+    conv: torch.Tensor         # fp32 [taps, channels], channels = q heads | k heads | v heads
     decay_rate: torch.Tensor   # fp32 [heads], exp(A_log)
     dt_bias: torch.Tensor      # fp32 [heads * dk]
     norm: torch.Tensor         # bf16 [dv]
@@ -271,7 +271,7 @@ def delta_mix(proj: torch.Tensor, z: torch.Tensor, w: DeltaWeights, conv_state: 
     assert proj.dtype == z.dtype == conv_state.dtype and state.dtype == torch.float32
     assert slots.dtype == torch.int32 and positions.dtype == torch.int32 and proj.stride(1) == 1 and z.stride(1) == 1
     L = N.lib()
-    taps = w.conv.shape[1]
+    taps = w.conv.shape[0]
     ws = torch.empty(L.b200_delta_workspace_bytes(t, w.heads, w.kv_heads, w.dk, w.dv), dtype=torch.uint8, device=proj.device)
     out = torch.empty(t, w.heads * w.dv, dtype=proj.dtype, device=proj.device)
     rc = L.b200_delta(proj.data_ptr(), z.data_ptr(), w.conv.data_ptr(), w.decay_rate.data_ptr(), w.dt_bias.data_ptr(),

@@ -169,7 +169,7 @@ def glu_clamped(x: torch.Tensor, limit: float, alpha: float) -> torch.Tensor:
 
 def delta_mix(proj, z, w, conv_state, state, positions, cu_q, slots, b_off) -> torch.Tensor:
     """Gated delta rule with per-channel decay, token by token (see ``ops.delta_mix``)."""
-    t, h, hk, dk, dv, taps, c = proj.shape[0], w.heads, w.kv_heads, w.dk, w.dv, w.conv.shape[1], w.channels
+    t, h, hk, dk, dv, taps, c = proj.shape[0], w.heads, w.kv_heads, w.dk, w.dv, w.conv.shape[0], w.channels
     bounds = list(range(slots.numel() + 1)) if cu_q is None else cu_q.tolist()
     out = torch.empty(t, h * dv, dtype=proj.dtype)
     for i, slot in enumerate(slots.tolist()):
@@ -180,7 +180,7 @@ def delta_mix(proj, z, w, conv_state, state, positions, cu_q, slots, b_off) -> t
         seq = torch.cat([tail, x], 0)
         if slot >= 0 and taps > 1:
             conv_state[slot] = seq[-(taps - 1):].to(conv_state.dtype)
-        x = torch.nn.functional.silu((seq.unfold(0, taps, 1) * w.conv[None]).sum(-1))
+        x = torch.nn.functional.silu((seq.unfold(0, taps, 1) * w.conv.t()[None]).sum(-1))
         q, k, v = x.split([hk * dk, hk * dk, h * dv], -1)
         unit = lambda u: u * torch.rsqrt(u.pow(2).sum(-1, keepdim=True) + 1e-6)
         q = (unit(q.reshape(-1, hk, dk)) * w.dk_true ** -0.5).repeat_interleave(h // hk, 1)
