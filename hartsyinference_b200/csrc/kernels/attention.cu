@@ -83,8 +83,10 @@ __device__ __forceinline__ void ext_scores(float (&s)[NT][4], int key0, const in
     const int d0 = row_limit[0] - 1 - key0, d1 = row_limit[1] - 1 - key0;       // distances of the first key
     const int lo = min(d0, d1) - (NT * 8 - 7), hi = max(d0, d1);
     mode = __all_sync(0xffffffffu, lo >= p.dist_len - 1) ? 2 : __all_sync(0xffffffffu, lo >= 0 && hi < p.dist_len) ? 1 : 0;
-    far[0] = row_bias[0][p.dist_len - 1];
-    far[1] = row_bias[1][p.dist_len - 1];
+    if (mode == 2) {
+      far[0] = row_bias[0][p.dist_len - 1];
+      far[1] = row_bias[1][p.dist_len - 1];
+    }
     if (mode == 1) {
       at[0] = row_bias[0] + d0;
       at[1] = row_bias[1] + d1;
@@ -160,7 +162,7 @@ __device__ __forceinline__ void load_tile_paged(uint32_t smem_base, const __nv_b
     cp_async_16(smem_base + tile_off<D>(t, c), src, valid);
   }
 }
-// Stages the page ids of tile `tile` into ring slot (tile & 3). Tiles start on page boundaries
+// Stages the page ids of tile `tile` into ring slot (tile & 7). Tiles start on page boundaries
 // because 64 is a multiple of every supported page size.
 __device__ __forceinline__ void stage_pages(int (*ring)[8], const int* table, int tile, int n_tiles,
                                             int page_shift, int kv_len) {
@@ -169,7 +171,7 @@ __device__ __forceinline__ void stage_pages(int (*ring)[8], const int* table, in
     const int first = (tile * kTileTokens) >> page_shift;
     const int idx = first + threadIdx.x;
     const int last_page = (kv_len - 1) >> page_shift;
-    ring[tile & 3][threadIdx.x] = idx <= last_page ? table[idx] : 0;
+    ring[tile & 7][threadIdx.x] = idx <= last_page ? table[idx] : 0;
   }
 }
 template <int D>
@@ -340,6 +342,7 @@ attn_decode_kernel(const AttnParams p) {
   pdl_trigger();
   constexpr int kTileBytes = kTileTokens * D * 2;
   extern __shared__ __align__(128) uint8_t smem[];
+  const int stage_bytes = kExt && p.shared_kv ? kTileBytes : 2 * kTileBytes;
   const int seq = blockIdx.x, kvh = blockIdx.y, split = blockIdx.z;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int g = lane >> 2, tq = lane & 3;
@@ -392,20 +395,20 @@ attn_decode_kernel(const AttnParams p) {
     }
   }
 
-  __shared__ int pg_ring[4][8];
+  __shared__ int pg_ring[8][8];
   auto issue = [&](int tile, int stage) {
     if (tile < tile_end) {
-      const uint32_t kb = smem_base + stage * 2 * kTileBytes;
+      const uint32_t kb = smem_base + stage * stage_bytes;
       if (kExt) {
-        load_tile_paged<D, true>(kb, p.k, pg_ring[tile & 3], kvh, p.hkv, p.page_shift, tile * kTileTokens, kv_len, p.d);
+        load_tile_paged<D, true>(kb, p.k, pg_ring[tile & 7], kvh, p.hkv, p.page_shift, tile * kTileTokens, kv_len, p.d);
         if (!p.shared_kv)
-          load_tile_paged<D, true>(kb + kTileBytes, p.v, pg_ring[tile & 3], kvh, p.hkv, p.page_shift, tile * kTileTokens,
+          load_tile_paged<D, true>(kb + kTileBytes, p.v, pg_ring[tile & 7], kvh, p.hkv, p.page_shift, tile * kTileTokens,
                                    kv_len, p.d);
         cp_async_commit();
         return;
       }
-      load_tile_paged<D>(kb, p.k, pg_ring[tile & 3], kvh, p.hkv, p.page_shift, tile * kTileTokens, kv_len);
-      load_tile_paged<D>(kb + kTileBytes, p.v, pg_ring[tile & 3], kvh, p.hkv, p.page_shift,
+      load_tile_paged<D>(kb, p.k, pg_ring[tile & 7], kvh, p.hkv, p.page_shift, tile * kTileTokens, kv_len);
+      load_tile_paged<D>(kb + kTileBytes, p.v, pg_ring[tile & 7], kvh, p.hkv, p.page_shift,
                          tile * kTileTokens, kv_len);
     }
     cp_async_commit();
@@ -413,17 +416,18 @@ attn_decode_kernel(const AttnParams p) {
   stage_pages(pg_ring, table, tile_begin, tile_end, p.page_shift, kv_len);
   stage_pages(pg_ring, table, tile_begin + 1, tile_end, p.page_shift, kv_len);
   stage_pages(pg_ring, table, tile_begin + 2, tile_end, p.page_shift, kv_len);
+  if (kStages > 3) stage_pages(pg_ring, table, tile_begin + 3, tile_end, p.page_shift, kv_len);
   __syncthreads();
 #pragma unroll
   for (int i = 0; i < kStages - 1; ++i) issue(tile_begin + i, i);
   int stage = 0;
   for (int tile = tile_begin; tile < tile_end; ++tile) {
-    // page ids of tile + 3 are read by issue() in a later iteration, after two barriers
-    stage_pages(pg_ring, table, tile + 3, tile_end, p.page_shift, kv_len);
+    // these page ids are read by issue() in a later iteration, after two barriers
+    stage_pages(pg_ring, table, tile + (kStages > 3 ? kStages : 3), tile_end, p.page_shift, kv_len);
     issue(tile + kStages - 1, (stage + kStages - 1) % kStages);
     cp_async_wait<kStages - 1>();
     __syncthreads();
-    const uint32_t kb = smem_base + stage * 2 * kTileBytes;
+    const uint32_t kb = smem_base + stage * stage_bytes;
     warp_tile<D, 1, kExt>(st, qf, kb, kExt && p.shared_kv ? kb : kb + kTileBytes, warp * 16, tile * kTileTokens, lim, start, p,
                           row_bias);
     __syncthreads();
@@ -624,18 +628,18 @@ attn_prefill_kernel(const AttnParams p) {
   const __nv_bfloat16* kbase = kPaged ? p.k : p.k + (static_cast<long long>(kv_off) * p.hkv + kvh) * D;
   const __nv_bfloat16* vbase = kPaged ? p.v : p.v + (static_cast<long long>(kv_off) * p.hkv + kvh) * D;
 
-  __shared__ int pg_ring[4][8];
+  __shared__ int pg_ring[8][8];
   auto issue = [&](int tile, int stage) {
     if (tile < n_tiles) {
       const uint32_t kb = smem_base + stage * stage_bytes;
       if (kExt) {
-        load_tile_paged<D, true>(kb, p.k, pg_ring[tile & 3], kvh, p.hkv, p.page_shift, tile * kTileTokens, kv_needed, p.d);
+        load_tile_paged<D, true>(kb, p.k, pg_ring[tile & 7], kvh, p.hkv, p.page_shift, tile * kTileTokens, kv_needed, p.d);
         if (!p.shared_kv)
-          load_tile_paged<D, true>(kb + kTileBytes, p.v, pg_ring[tile & 3], kvh, p.hkv, p.page_shift, tile * kTileTokens,
+          load_tile_paged<D, true>(kb + kTileBytes, p.v, pg_ring[tile & 7], kvh, p.hkv, p.page_shift, tile * kTileTokens,
                                    kv_needed, p.d);
       } else if (kPaged) {
-        load_tile_paged<D>(kb, p.k, pg_ring[tile & 3], kvh, p.hkv, p.page_shift, tile * kTileTokens, kv_needed);
-        load_tile_paged<D>(kb + kTileBytes, p.v, pg_ring[tile & 3], kvh, p.hkv, p.page_shift,
+        load_tile_paged<D>(kb, p.k, pg_ring[tile & 7], kvh, p.hkv, p.page_shift, tile * kTileTokens, kv_needed);
+        load_tile_paged<D>(kb + kTileBytes, p.v, pg_ring[tile & 7], kvh, p.hkv, p.page_shift,
                            tile * kTileTokens, kv_needed);
       } else {
         load_tile_linear<D>(kb, kbase, kv_rs, tile * kTileTokens, kv_needed);
@@ -1009,17 +1013,18 @@ B200_API int b200_attn_biased(const void* q, const void* k_cache, const void* v_
     p.ws_ml = p.ws_o + static_cast<long long>(seqs) * hq * p.splits * dd;
   }
   const dim3 grid(seqs, hkv, p.splits);
-  // the ring doubles as the buffer of the four warps' partial results
-  const int ring = 2 * 2 * kTileTokens * dd * 2, merge = 4 * 16 * (dd + 2) * 4, smem = ring > merge ? ring : merge;
-  static PerDeviceOnce once[2];
+  // the ring (two tiles of keys and values, or four tiles of keys that are also the values) doubles as the
+  // buffer of the four warps' partial results
+  const int ring = 4 * kTileTokens * dd * 2, merge = 4 * 16 * (dd + 2) * 4;
+  const int smem = ring > merge ? ring : merge;
+  auto go = [&](auto kernel, PerDeviceOnce& once) {
+    if (once.first_time()) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    return launch_pdl(kernel, grid, dim3(kAttnThreads), smem, stream, p);
+  };
+  static PerDeviceOnce once[4];
   cudaError_t e;
-  if (dd == 128) {
-    if (once[1].first_time()) cudaFuncSetAttribute(attn_decode_kernel<128, 2, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
-    e = launch_pdl(attn_decode_kernel<128, 2, true>, grid, dim3(kAttnThreads), smem, stream, p);
-  } else {
-    if (once[0].first_time()) cudaFuncSetAttribute(attn_decode_kernel<64, 2, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
-    e = launch_pdl(attn_decode_kernel<64, 2, true>, grid, dim3(kAttnThreads), smem, stream, p);
-  }
+  if (dd == 128) e = p.shared_kv ? go(attn_decode_kernel<128, 4, true>, once[0]) : go(attn_decode_kernel<128, 2, true>, once[1]);
+  else e = p.shared_kv ? go(attn_decode_kernel<64, 4, true>, once[2]) : go(attn_decode_kernel<64, 2, true>, once[3]);
   if (e != cudaSuccess) return -static_cast<int>(e) - 300;
   if (p.splits > 1) {
     if (dd == 128) e = launch_pdl(attn_combine_kernel<128, true>, dim3(seqs, hq), dim3(128), 0, stream, p);

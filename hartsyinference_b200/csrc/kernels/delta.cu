@@ -421,6 +421,16 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(const DeltaParams p) {
     const int n = min(kScanTokens, len - t0);
     const float* base = sm + buf * kScanTokens * kTok;
     float* op = p.o + (static_cast<long long>(first + t0) * p.h + head) * p.dv + col;
+    ulonglong2 nk[NR], ng[NR];           // the next token's k and g, read while the current one is computed
+    auto fetch = [&](int tk) {
+      const float* tb = base + tk * kTok;
+#pragma unroll
+      for (int i = 0; i < NR; ++i) {
+        nk[i] = *reinterpret_cast<const ulonglong2*>(tb + i * 32 + rg * 4);
+        ng[i] = *reinterpret_cast<const ulonglong2*>(tb + 2 * DK + i * 32 + rg * 4);
+      }
+    };
+    fetch(0);
     for (int tq = 0; tq < n; tq += 4) {
       float part[8];                       // reads of four tokens x two columns, this lane's rows
 #pragma unroll
@@ -430,43 +440,44 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(const DeltaParams p) {
         const float* tb = base + (tq + j) * kTok;
         f32x2 kk[NR * 2];
         f32x2 a0 = 0, a1 = 0, b0 = 0, b1 = 0;
+        const float2 v = *reinterpret_cast<const float2*>(tb + 3 * DK + lc);
+        const float beta = tb[3 * DK + kScanCols];
 #pragma unroll
         for (int i = 0; i < NR; ++i) {
-          const ulonglong2 kv = *reinterpret_cast<const ulonglong2*>(tb + i * 32 + rg * 4);
-          const ulonglong2 gv = *reinterpret_cast<const ulonglong2*>(tb + 2 * DK + i * 32 + rg * 4);
-          kk[i * 2] = kv.x;
-          kk[i * 2 + 1] = kv.y;
-          s0[i * 2] = mul2(s0[i * 2], gv.x);
-          s1[i * 2] = mul2(s1[i * 2], gv.x);
-          s0[i * 2 + 1] = mul2(s0[i * 2 + 1], gv.y);
-          s1[i * 2 + 1] = mul2(s1[i * 2 + 1], gv.y);
-          a0 = fma2(s0[i * 2], kv.x, a0);
-          a1 = fma2(s1[i * 2], kv.x, a1);
-          b0 = fma2(s0[i * 2 + 1], kv.y, b0);
-          b1 = fma2(s1[i * 2 + 1], kv.y, b1);
+          kk[i * 2] = nk[i].x;
+          kk[i * 2 + 1] = nk[i].y;
+          s0[i * 2] = mul2(s0[i * 2], ng[i].x);
+          s1[i * 2] = mul2(s1[i * 2], ng[i].x);
+          s0[i * 2 + 1] = mul2(s0[i * 2 + 1], ng[i].y);
+          s1[i * 2 + 1] = mul2(s1[i * 2 + 1], ng[i].y);
+          a0 = fma2(s0[i * 2], nk[i].x, a0);
+          a1 = fma2(s1[i * 2], nk[i].x, a1);
+          b0 = fma2(s0[i * 2 + 1], nk[i].y, b0);
+          b1 = fma2(s1[i * 2 + 1], nk[i].y, b1);
         }
+        ulonglong2 qv[NR];
+#pragma unroll
+        for (int i = 0; i < NR; ++i) qv[i] = *reinterpret_cast<const ulonglong2*>(tb + DK + i * 32 + rg * 4);
+        fetch(min(tq + j + 1, n - 1));
         float r0 = sum2(add2(a0, b0)), r1 = sum2(add2(a1, b1));
 #pragma unroll
         for (int o = 1; o < 8; o <<= 1) {
           r0 += __shfl_xor_sync(0xffffffffu, r0, o);
           r1 += __shfl_xor_sync(0xffffffffu, r1, o);
         }
-        const float2 v = *reinterpret_cast<const float2*>(tb + 3 * DK + lc);
-        const float beta = tb[3 * DK + kScanCols];
         const float u0 = beta * (v.x - r0), u1 = beta * (v.y - r1);
         const f32x2 uu0 = pack2(u0, u0), uu1 = pack2(u1, u1);
         a0 = a1 = b0 = b1 = 0;
 #pragma unroll
         for (int i = 0; i < NR; ++i) {
-          const ulonglong2 qv = *reinterpret_cast<const ulonglong2*>(tb + DK + i * 32 + rg * 4);
           s0[i * 2] = fma2(kk[i * 2], uu0, s0[i * 2]);
           s1[i * 2] = fma2(kk[i * 2], uu1, s1[i * 2]);
           s0[i * 2 + 1] = fma2(kk[i * 2 + 1], uu0, s0[i * 2 + 1]);
           s1[i * 2 + 1] = fma2(kk[i * 2 + 1], uu1, s1[i * 2 + 1]);
-          a0 = fma2(s0[i * 2], qv.x, a0);
-          a1 = fma2(s1[i * 2], qv.x, a1);
-          b0 = fma2(s0[i * 2 + 1], qv.y, b0);
-          b1 = fma2(s1[i * 2 + 1], qv.y, b1);
+          a0 = fma2(s0[i * 2], qv[i].x, a0);
+          a1 = fma2(s1[i * 2], qv[i].x, a1);
+          b0 = fma2(s0[i * 2 + 1], qv[i].y, b0);
+          b1 = fma2(s1[i * 2 + 1], qv[i].y, b1);
         }
         part[2 * j] = sum2(add2(a0, b0));
         part[2 * j + 1] = sum2(add2(a1, b1));

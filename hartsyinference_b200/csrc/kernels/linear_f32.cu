@@ -187,16 +187,19 @@ __global__ void __launch_bounds__(kTok > 2 ? 512 : 1024) router_kernel(const Rou
 }
 
 // Many bf16 tokens: 32 tokens per block, bf16 products with fp32 accumulation on the tensor core (m16n8k16),
-// experts in passes of 128. Warp (wm, wn): tokens 16 wm.., experts 64 wn.. of the pass. Dynamic shared memory:
-// 32 * experts floats, then two stages of [32 + 128] rows of 64 values (16-byte chunks XOR-swizzled by row).
-constexpr int kRtTok = 32, kRtExp = 128, kRtK = 64;
+// experts in passes of kRtExp. Warp (wm, wn): tokens 16 wm.., experts kRtExp / 2 wn.. of the pass. Dynamic shared
+// memory: a ring of kRtStages stages of [32 + kRtExp] rows of 64 values (16-byte chunks XOR-swizzled by row),
+// then 32 * experts floats.
+constexpr int kRtTok = 32, kRtK = 64, kRtStages = 5;
 
+template <int kRtExp>
 __global__ void __launch_bounds__(128) router_tc_kernel(const RouterParams p) {
   pdl_wait();
   pdl_trigger();
   extern __shared__ __align__(128) uint8_t smraw[];
   constexpr int kStage = (kRtTok + kRtExp) * kRtK * 2;
-  float* lg = reinterpret_cast<float*>(smraw + 2 * kStage);
+  float* lg = reinterpret_cast<float*>(smraw + kRtStages * kStage);
+  constexpr int kNt = kRtExp / 16;                  // 8-wide expert tiles per warp
   const uint32_t base = smem_u32(smraw);
   const int t0 = blockIdx.x * kRtTok;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, wm = warp & 1, wn = warp >> 1;
@@ -222,41 +225,43 @@ __global__ void __launch_bounds__(128) router_tc_kernel(const RouterParams p) {
       }
       cp_async_commit();
     };
-    float acc[8][4];
+    float acc[kNt][4];
 #pragma unroll
-    for (int i = 0; i < 8; ++i)
+    for (int i = 0; i < kNt; ++i)
 #pragma unroll
       for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
-    load(0, 0);
+    for (int i = 0; i < kRtStages - 1; ++i) load(i, i);
+    int cur = 0;
     for (int kb = 0; kb < nk; ++kb) {
-      load(kb + 1, (kb + 1) & 1);
-      cp_async_wait<1>();
-      __syncthreads();
-      const uint32_t st = base + (kb & 1) * kStage;
+      cp_async_wait<kRtStages - 2>();
+      __syncthreads();                              // stage kb has landed, stage kb - 1 has been read by all
+      load(kb + kRtStages - 1, cur == 0 ? kRtStages - 1 : cur - 1);
+      const uint32_t st = base + cur * kStage;
+      cur = cur + 1 == kRtStages ? 0 : cur + 1;
 #pragma unroll
       for (int kk = 0; kk < kRtK / 16; ++kk) {
         uint32_t a[4];
         const int ar = wm * 16 + (lane & 15), ac = kk * 2 + (lane >> 4);
         ldmatrix_x4(st + ar * (kRtK * 2) + ((ac ^ (ar & 7)) << 4), a[0], a[1], a[2], a[3]);
 #pragma unroll
-        for (int g = 0; g < 4; ++g) {
+        for (int g = 0; g < kNt / 2; ++g) {
           const int mi = lane >> 3;
-          const int br = kRtTok + wn * 64 + g * 16 + (lane & 7) + 8 * (mi >> 1), bc = kk * 2 + (mi & 1);
+          const int br = kRtTok + wn * (kRtExp / 2) + g * 16 + (lane & 7) + 8 * (mi >> 1), bc = kk * 2 + (mi & 1);
           uint32_t b0, b1, b2, b3;
           ldmatrix_x4(st + br * (kRtK * 2) + ((bc ^ (br & 7)) << 4), b0, b1, b2, b3);
           mma_bf16_16816(acc[g * 2], a, b0, b1);
           mma_bf16_16816(acc[g * 2 + 1], a, b2, b3);
         }
       }
-      __syncthreads();
     }
     cp_async_wait<0>();
+    __syncthreads();
     const int row = wm * 16 + (lane >> 2);
 #pragma unroll
-    for (int g = 0; g < 8; ++g)
+    for (int g = 0; g < kNt; ++g)
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
-        const int e = e0 + wn * 64 + g * 8 + (lane & 3) * 2 + (j & 1);
+        const int e = e0 + wn * (kRtExp / 2) + g * 8 + (lane & 3) * 2 + (j & 1);
         if (e < p.experts) lg[(row + 8 * (j >> 1)) * p.experts + e] = acc[g][j];
       }
   }
@@ -269,11 +274,20 @@ template <typename T>
 int launch_router(const RouterParams& p, bool tensor_cores, cudaStream_t stream) {
   const int limit = 200 * 1024;
   cudaError_t e;
-  const int tc_bytes = 2 * (kRtTok + kRtExp) * kRtK * 2 + kRtTok * p.experts * 4;
+  const int tile = p.experts <= 32 ? 32 : p.experts <= 64 ? 64 : p.experts <= 96 ? 96 : 128;
+  const int tc_bytes = kRtStages * (kRtTok + tile) * kRtK * 2 + kRtTok * p.experts * 4;
   if (tensor_cores && p.tokens > 4 * 148 && tc_bytes <= limit && p.ldx % 8 == 0) {
-    static PerDeviceOnce once_tc;
-    if (once_tc.first_time()) cudaFuncSetAttribute(router_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, limit);
-    e = launch_pdl(router_tc_kernel, dim3((p.tokens + kRtTok - 1) / kRtTok), dim3(128), tc_bytes, stream, p);
+    auto tc = [&](auto kernel, PerDeviceOnce& once) {
+      if (once.first_time()) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, limit);
+      return launch_pdl(kernel, dim3((p.tokens + kRtTok - 1) / kRtTok), dim3(128), tc_bytes, stream, p);
+    };
+    static PerDeviceOnce once_tc[4];
+    switch (tile) {
+      case 32: e = tc(router_tc_kernel<32>, once_tc[0]); break;
+      case 64: e = tc(router_tc_kernel<64>, once_tc[1]); break;
+      case 96: e = tc(router_tc_kernel<96>, once_tc[2]); break;
+      default: e = tc(router_tc_kernel<128>, once_tc[3]); break;
+    }
     return e == cudaSuccess ? 0 : -static_cast<int>(e) - 300;
   }
   auto bytes = [&](int tok) { return tok * (p.k + p.experts) * 4; };
