@@ -284,10 +284,34 @@ def test_delta_first_tokens_and_far_write(mode):
     near(y[395:], want[395:], mode, 3e-5, 3e-2)
 
 
+@pytest.mark.parametrize("mode", MODES[1:])
+def test_delta_long_portion_equals_short_ones(mode):
+    """A portion long enough for several tokens per warp, spanning two sequences, against the same tokens in
+    pieces: the recurrence runs the same operations wherever it is cut."""
+    dev, dt = mode
+    g = gen(77)
+    mix, w, t = delta_case(g, 16, 16, 32, 32, 4)
+    hs = rnd(g, 2200, w).to(dt).to(dev)
+    m, state = build_delta(mix, w, t, dev, dt)
+    holder = _Holder()
+    holder.mixer_state = state
+    whole = m(hs, _Batch(dev, list(range(1203)) + list(range(997)), [0, 2], [0, 1203, 2200]), 0, holder)
+    after = [s.clone() for s in state[0]]
+    parts = []
+    for a, b, slot in ((0, 1203, 0), (1203, 2200, 2)):
+        for c in range(a, b, 101):
+            e = min(c + 101, b)
+            parts.append(m(hs[c:e], _Batch(dev, range(c - a, e - a), [slot], [0, e - c]), 0, holder))
+    assert rel_err(torch.cat(parts), whole.cpu()) < (1e-6 if dt == F32 else 2e-3)
+    for x, y in zip(after, state[0]):
+        for slot in (0, 2):
+            assert rel_err(y[slot].float(), x[slot].float().cpu()) < (1e-6 if dt == F32 else 2e-3)
+
+
 # ------------------------------------------------------------------------------------ experts
 @pytest.mark.parametrize("mode", MODES)
 @pytest.mark.parametrize("experts,identity,top,ff,limit,tokens", [(5, 2, 3, 40, 0.7, 37), (3, 0, 1, 64, 1.5, 300), (4, 6, 5, 24, 0.3, 1),
-                                                                  (33, 7, 4, 136, 1.0, 21)])
+                                                                  (33, 7, 4, 136, 1.0, 21), (20, 5, 6, 32, 1.0, 700), (150, 3, 2, 16, 0.8, 650)])
 def test_experts(mode, experts, identity, top, ff, limit, tokens):
     from hartsyinference_b200.models.llm.mixers import build_experts
     from hartsyinference_b200.models.llm.moe import MoeFeedForward
