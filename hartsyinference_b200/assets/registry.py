@@ -59,7 +59,7 @@ def detect(path: str | Path) -> Detected:
         cfg = p / "config.json"
         if cfg.exists():
             d = json.loads(cfg.read_text())
-            mt = d.get("model_type") or (d.get("_class_name") or "").lower()
+            mt = d.get("model_type") or str(d.get("_class_name") or d.get("architecture") or "").lower()
             if mt:
                 fam = "llm"
                 if "flux" in mt:

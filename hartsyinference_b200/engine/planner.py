@@ -156,6 +156,8 @@ def shape_of_checkpoint(path) -> Optional[ModelShape]:
                 break
             except Exception:
                 pass
+    if isinstance(cfg.get("layers"), list):        # layers described one by one: such models are not sharded
+        return None
     heads = int(cfg.get("num_attention_heads") or cfg.get("n_head") or 0)
     experts = int(cfg.get("n_routed_experts") or cfg.get("num_local_experts") or cfg.get("num_experts") or 0)
     cls = str(cfg.get("_class_name", "")).lower()

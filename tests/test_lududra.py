@@ -610,6 +610,31 @@ def test_checkpoint_loads_by_config(checkpoint):
         llm.config.validate_tp(2)
 
 
+def test_checkpoint_is_recognised(checkpoint):
+    from hartsyinference_b200.assets.registry import detect
+    from hartsyinference_b200.engine.planner import shape_of_checkpoint
+    d = detect(checkpoint)
+    assert (d.family, d.arch) == ("llm", "lududra")
+    assert shape_of_checkpoint(checkpoint) is None          # stays on one GPU
+
+
+def test_service_generates_and_embeds(checkpoint):
+    """Through the text service: token ids in, greedy ids out as the engine gives them; embedding a text in
+    between leaves the running requests' pages and states alone."""
+    from hartsyinference_b200.engine.requests import EngineOptions, Modality, ModelSpec, TextRequest
+    from hartsyinference_b200.engine.text_service import TextService
+    svc = TextService(EngineOptions(max_batch=2, max_model_len=64), device="cpu")
+    spec = ModelSpec("m", Modality.TEXT, local_path=str(checkpoint))
+    req = TextRequest(messages=[], prompt_token_ids=prompt("mixed", 20, 5), max_tokens=6, greedy=True, ignore_eos=True)
+    try:
+        a = svc.generate(spec, req).token_ids
+        e = svc.embed(spec, ["abc", "abcd"])
+        assert e.shape == (2, CASES["mixed"]["width"]) and torch.isfinite(e).all()
+        assert svc.generate(spec, req).token_ids == a and len(a) == 6
+    finally:
+        svc.release()
+
+
 @pytest.mark.parametrize("mode", [MODES[0], MODES[1]])
 def test_trace_run(checkpoint, tmp_path, monkeypatch, capsys, mode):
     from hartsyinference_b200.cli import trace
