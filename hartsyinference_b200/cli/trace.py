@@ -1,11 +1,12 @@
-"""``bin/trace_run``: feed given token ids through a served model, step by step, and write logits.
+"""``bin/trace_run``: replay a recorded token stream through a served model and keep the logits.
 
     bin/trace_run --model DIR --dtype bfloat16|float32 --out DIR --max-tokens N  < steps.jsonl
 
-One JSON object per input line: ``{"step": 0, "entries": [{"id": "a", "tokens": [5, 17], "want": [1]}],
-"end": ["a"]}``. ``entries`` are the next tokens of each request and the places among them whose logits are
-wanted; ``end`` lists requests that are finished after the step. A step with wanted places writes
-``<out>/<step>.f32`` (little-endian fp32 [wanted, vocab]); every step prints ``done <step>``.
+Every input line is one engine step as a JSON object, for instance
+``{"step": 7, "entries": [{"id": "req1", "tokens": [901, 44, 2], "want": [2]}], "end": []}``: what each request
+continues with, at which of these tokens (index from 0) logits are to be kept, and which requests leave
+afterwards. Kept logits go to ``<out>/<step>.f32`` (little-endian fp32 [kept, vocab], entry by entry), and
+``done <step>`` is printed when the step is through.
 
 The model is loaded and run by the engine that serves it (``LLMEngine.replay``): its page pool holds
 ``--max-tokens`` tokens, with state slots for ``--max-live`` requests. The kernels library is compiled on
@@ -27,8 +28,8 @@ def parse(argv=None) -> argparse.Namespace:
     ap.add_argument("--dtype", choices=("bfloat16", "float32"), default="bfloat16",
                     help="bfloat16: as served; float32: products and caches in 32 bits")
     ap.add_argument("--out", required=True, help="directory of the logits files")
-    ap.add_argument("--max-tokens", type=int, required=True, help="most tokens that live requests hold at any time")
-    ap.add_argument("--max-live", type=int, default=4, help="most requests that are live at any time")
+    ap.add_argument("--max-tokens", type=int, required=True, help="size of the page pool in tokens (pages of 16)")
+    ap.add_argument("--max-live", type=int, default=4, help="state slots: requests that can be open together")
     ap.add_argument("--device", default="cuda")
     return ap.parse_args(argv)
 

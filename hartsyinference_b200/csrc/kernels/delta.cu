@@ -1,8 +1,8 @@
 // Gated delta-rule mixer with one decay per head and key channel.
 //
-// Per head, with a state S [dk][dv] that is carried in fp32 from token to token of a sequence:
-//   S <- diag(g) S;   u = beta (v - S^T k);   S <- S + k u^T;   o = S^T q
-//   y = o / rms(o) * w * sigmoid(gate)
+// Per head and sequence a matrix S [dk][dv] in fp32, updated by every token t:
+//   S' = Diag(g_t) S_{t-1};   S_t = S' + k_t (beta_t (v_t - S'^T k_t))^T;   o_t = S_t^T q_t
+//   y_t = sigmoid(gate_t) w o_t / rms(o_t)
 // q, k, v come from projections through a short causal convolution and silu; q and k are made unit
 // vectors; g = exp(-A softplus(z + dt_bias)); several heads can share one q / k head.
 //

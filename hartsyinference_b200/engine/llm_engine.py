@@ -7,8 +7,8 @@ Models with per-layer mixers run prompt chunks and decoded tokens of a step as O
 (a decoded token is a chunk of one); a step with decoded tokens only replays a CUDA graph as for every
 other model. Recurrent models hold one state slot per running sequence (``KvAllocator.seq_slot``).
 
-``replay`` drives the same batches from token ids that the caller brings (no scheduler decisions, no
-sampling) and returns logits.
+``replay`` drives the same batches from given token ids (no scheduler decisions, no sampling) and
+returns logits.
 
 Counterpart in the reference: ``DynamicBatchScheduler`` (SubmitAsync:153, RunLoopAsync:162-268,
 AdmitAndPrefill:311-383 prefills each request alone, RunDecodeRound:460-483 gathers pages per
@@ -617,12 +617,12 @@ class LLMEngine:
 
     # ------------------------------------------------------------------------------- replay
     def replay(self, entries: Sequence[tuple], end: Sequence[object] = ()) -> Optional[torch.Tensor]:
-        """One step over token ids brought by the caller: ``entries`` = [(key, tokens, want)] are the next
-        tokens of each keyed sequence (created at its first entry) and the places among them whose logits
-        are asked for. All entries form one batch, run by the step's own functions: single tokens of
-        running sequences replay the decode step, anything else is a ragged batch of runs. Sequences in
-        ``end`` then give back their pages and state slots. Returns fp32 logits [wanted, vocab] in the
-        order of the entries, or None. Raises ``KvPoolExhaustedError`` when pool or slots do not suffice."""
+        """One step over given token ids. ``entries`` = [(key, tokens, want)]: every keyed sequence (opened when
+        its key is new) is extended by ``tokens``, and ``want`` indexes those of them to return logits for.
+        The entries are computed as one batch by the step's own functions: single tokens of running
+        sequences replay the decode step, anything else is a ragged batch of runs. Sequences in ``end``
+        then release their pages and state slots. Returns fp32 logits, one row per wanted token in
+        entry order, or None. Raises ``KvPoolExhaustedError`` when pool or slots do not suffice."""
         self.h2d_bytes_last = 0
         if len(entries) > self.h_kv_lens.numel() or sum(len(e[1]) for e in entries) > self.h_tokens.numel():
             raise ValueError("more entries or tokens in one step than the engine was made for (max_batch, prefill_chunk)")

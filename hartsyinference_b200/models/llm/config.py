@@ -174,7 +174,7 @@ class TransformerConfig:
 
     @property
     def recurrent(self) -> bool:
-        """True when some layer carries a state from token to token (a state slot per sequence)."""
+        """True when some layer is recurrent: its sequences need a state slot."""
         return any(ls.mixer.kind == "channel_delta" for ls in self.layer_specs)
 
     @property

@@ -1,14 +1,13 @@
-"""Lududra: windowed attention and channel-wise gated delta-rule layers over a 32-bit residual stream,
-LayerNorm before and after every sublayer, routed experts with pass-through outputs.
+"""Lududra: windowed attention and channel-wise gated delta-rule layers over a 32-bit residual stream
+with sandwich LayerNorms, and routed experts with pass-through outputs.
 
 This file maps the design's ``config.json`` and tensor names onto the generic pieces: per-layer
 :class:`~.config.LayerSpec` records and the mixers of :mod:`.mixers`. What the design fixes is stated
 here: the attention sink has score 0, keys serve as values, q and k carry biases, the output gate is on,
 router scores are a softmax that is not renormalised after the choice, and the expert gate uses 1.702.
 
-    x   = embed[token] * scale
-    x  += norm1b(mixer(norm1(x)));   x += norm2b(experts(norm2(x)))      per layer
-    out = head . norm(x)
+    per layer, x the stream and N.. its LayerNorms:   x += N1b M(N1 x),   then   x += N2b E(N2 x)
+    with M the layer's mixer and E its experts (a layer can lack E); logits = W_head N_final x
 """
 from __future__ import annotations
 

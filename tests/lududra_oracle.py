@@ -66,7 +66,7 @@ def attention_mixer(h, mix, w, p):
 
 
 def short_conv(x, taps):
-    """Causal per-channel convolution over time, [T, C] with [C, taps]; zeros before the start."""
+    """Per-channel convolution of [T, C] with [C, taps] that looks back only; nothing precedes token 0."""
     n = taps.shape[1]
     out = torch.zeros_like(x)
     for t in range(x.shape[0]):
