@@ -59,6 +59,9 @@ struct AttnParams {
   const __nv_bfloat16* gate;    // [tokens][gate_ld]: out *= sigmoid(gate), or null
   long long q_ld, gate_ld;      // row pitches in elements
   int dist_len, d, shared_kv;   // d: head size as stored; shared_kv: v is k
+  int dv;                       // size of values and output per head (d unless k, v are contiguous)
+  const int* q_lens;            // [seqs] with cu_q = [seqs] starts: the listed runs need not be adjacent; or null
+  long long k_ld, v_ld;         // contiguous k, v: row pitches (head h at h * d, h * dv)
   float cap_in, cap_out;        // softcap: cap_out * tanh(score / softcap), exp(2 score / softcap) = 2^(cap_in * q.k)
 };
 constexpr float kLog2e = 1.4426950408889634f;
@@ -174,14 +177,14 @@ __device__ __forceinline__ void stage_pages(int (*ring)[8], const int* table, in
     ring[tile & 7][threadIdx.x] = idx <= last_page ? table[idx] : 0;
   }
 }
-template <int D>
+template <int D, bool kExt = false>
 __device__ __forceinline__ void load_tile_linear(uint32_t smem_base, const __nv_bfloat16* base,
-                                                 long long row_stride, int tok0, int kv_len) {
+                                                 long long row_stride, int tok0, int kv_len, int d = D) {
   constexpr int kChunks = D / 8;
   for (int i = threadIdx.x; i < kTileTokens * kChunks; i += kAttnThreads) {
     const int t = i / kChunks, c = i % kChunks;
     const int tok = tok0 + t;
-    const bool valid = tok < kv_len;
+    const bool valid = tok < kv_len && (!kExt || c * 8 < d);
     const __nv_bfloat16* src = valid ? base + tok * row_stride + c * 8 : base;
     cp_async_16(smem_base + tile_off<D>(t, c), src, valid);
   }
@@ -329,7 +332,7 @@ __device__ __forceinline__ void warp_tile(WarpState<D>& st, const uint32_t (&qf)
 }
 
 __device__ __forceinline__ float gate_of(const AttnParams& p, long long token, int head, int c) {
-  return p.gate ? 1.f / (1.f + __expf(-__bfloat162float(p.gate[token * p.gate_ld + head * p.d + c]))) : 1.f;
+  return p.gate ? 1.f / (1.f + __expf(-__bfloat162float(p.gate[token * p.gate_ld + head * p.dv + c]))) : 1.f;
 }
 
 // ------------------------------------------------------------------------------------------
@@ -562,7 +565,7 @@ attn_prefill_kernel(const AttnParams p) {
   const int G = p.hq / p.hkv;
   const int kvh = head / G;
   const int q_off = p.cu_q ? p.cu_q[seq] : 0;
-  const int q_len = p.cu_q ? p.cu_q[seq + 1] - q_off : p.q_len_single;
+  const int q_len = kExt && p.q_lens ? p.q_lens[seq] : p.cu_q ? p.cu_q[seq + 1] - q_off : p.q_len_single;
   const int kv_len = p.kv_lens ? p.kv_lens[seq] : p.kv_len_single;
   if (qt * 64 >= q_len) return;
   const int stage_bytes = kExt && p.shared_kv ? kTileBytes : 2 * kTileBytes;
@@ -625,14 +628,17 @@ attn_prefill_kernel(const AttnParams p) {
   const int* table = kPaged ? p.block_table + static_cast<long long>(seq) * p.max_pages : nullptr;
   const int kv_off = (!kPaged && p.cu_kv) ? p.cu_kv[seq] : 0;
   const long long kv_rs = static_cast<long long>(p.hkv) * D;
-  const __nv_bfloat16* kbase = kPaged ? p.k : p.k + (static_cast<long long>(kv_off) * p.hkv + kvh) * D;
-  const __nv_bfloat16* vbase = kPaged ? p.v : p.v + (static_cast<long long>(kv_off) * p.hkv + kvh) * D;
+  const __nv_bfloat16* kbase = kPaged ? p.k : kExt ? p.k + kv_off * p.k_ld + kvh * p.d : p.k + (static_cast<long long>(kv_off) * p.hkv + kvh) * D;
+  const __nv_bfloat16* vbase = kPaged ? p.v : kExt ? p.v + kv_off * p.v_ld + kvh * p.dv : p.v + (static_cast<long long>(kv_off) * p.hkv + kvh) * D;
 
   __shared__ int pg_ring[8][8];
   auto issue = [&](int tile, int stage) {
     if (tile < n_tiles) {
       const uint32_t kb = smem_base + stage * stage_bytes;
-      if (kExt) {
+      if (kExt && !kPaged) {
+        load_tile_linear<D, true>(kb, kbase, p.k_ld, tile * kTileTokens, kv_needed, p.d);
+        load_tile_linear<D, true>(kb + kTileBytes, vbase, p.v_ld, tile * kTileTokens, kv_needed, p.dv);
+      } else if (kExt) {
         load_tile_paged<D, true>(kb, p.k, pg_ring[tile & 7], kvh, p.hkv, p.page_shift, tile * kTileTokens, kv_needed, p.d);
         if (!p.shared_kv)
           load_tile_paged<D, true>(kb + kTileBytes, p.v, pg_ring[tile & 7], kvh, p.hkv, p.page_shift, tile * kTileTokens,
@@ -681,8 +687,8 @@ attn_prefill_kernel(const AttnParams p) {
       for (int i = 0; i < D / 8; ++i) {
         const int c = i * 8 + tq * 2;
         if (kExt) {
-          if (c < p.d)
-            *reinterpret_cast<uint32_t*>(p.out + (static_cast<long long>(q_off + row) * p.hq + head) * p.d + c) =
+          if (c < p.dv)
+            *reinterpret_cast<uint32_t*>(p.out + (static_cast<long long>(q_off + row) * p.hq + head) * p.dv + c) =
                 pack_bf16x2(st.o[i][2 * r] * inv * gate_of(p, q_off + row, head, c),
                             st.o[i][2 * r + 1] * inv * gate_of(p, q_off + row, head, c + 1));
           continue;
@@ -988,7 +994,7 @@ B200_API int b200_attn_biased(const void* q, const void* k_cache, const void* v_
   }
   p.dist_bias = dist_bias; p.dist_len = dist_len; p.sinks = sinks;
   p.gate = static_cast<const __nv_bfloat16*>(gate);
-  p.gate_ld = gate_ld; p.q_ld = q_ld; p.d = d;
+  p.gate_ld = gate_ld; p.q_ld = q_ld; p.d = p.dv = d;
   p.splits = cu_q || splits < 1 ? 1 : splits;
   const int dd = d <= 64 ? 64 : 128;
   if (cu_q) {
@@ -1032,6 +1038,44 @@ B200_API int b200_attn_biased(const void* q, const void* k_cache, const void* v_
     if (e != cudaSuccess) return -static_cast<int>(e) - 400;
   }
   return 0;
+}
+
+// Causal attention of the runs q_start[s] .. + q_lens[s] of q over contiguous keys and values of their whole
+// contexts (rows kv_start[s] .. + kv_lens[s] of k and v; the last key belongs to the run's last query). q, out and
+// gate are indexed by token: q [tokens][q_ld] (head h at h * d), out [tokens][hq * dv]. d, dv <= 128, multiples of 8.
+B200_API int b200_attn_runs(const void* q, const void* k, const void* v, void* out, const void* gate, const int* q_start,
+                            const int* q_lens, const int* kv_start, const int* kv_lens, int seqs, int max_q_len, int hq, int hkv,
+                            int d, int dv, long long q_ld, long long k_ld, long long v_ld, long long gate_ld, float scale,
+                            cudaStream_t stream) {
+  if (seqs <= 0 || max_q_len <= 0) return 0;
+  if (d % 8 || dv % 8 || d < 8 || dv < 8 || d > 128 || dv > 128 || hq % hkv || q_ld % 8 || k_ld % 8 || v_ld % 8 || gate_ld % 8 ||
+      seqs > 65535)
+    return -2;
+  AttnParams p{};
+  p.q = static_cast<const __nv_bfloat16*>(q);
+  p.k = static_cast<const __nv_bfloat16*>(k);
+  p.v = static_cast<const __nv_bfloat16*>(v);
+  p.out = static_cast<__nv_bfloat16*>(out);
+  p.gate = static_cast<const __nv_bfloat16*>(gate);
+  p.cu_q = q_start; p.q_lens = q_lens; p.cu_kv = kv_start; p.kv_lens = kv_lens;
+  p.seqs = seqs; p.hq = hq; p.hkv = hkv; p.splits = 1;
+  p.causal = 1;
+  p.scale = scale;
+  p.scale_log2 = scale * kLog2e;
+  p.d = d; p.dv = dv; p.q_ld = q_ld; p.k_ld = k_ld; p.v_ld = v_ld; p.gate_ld = gate_ld;
+  const dim3 grid((max_q_len + 63) / 64, hq, seqs);
+  static PerDeviceOnce once[2];
+  if (d > 64 || dv > 64) {
+    const int smem = 2 * 2 * kTileTokens * 128 * 2;
+    if (once[1].first_time()) cudaFuncSetAttribute(attn_prefill_kernel<128, false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    attn_prefill_kernel<128, false, true><<<grid, kAttnThreads, smem, stream>>>(p);
+  } else {
+    const int smem = 2 * 2 * kTileTokens * 64 * 2;
+    if (once[0].first_time()) cudaFuncSetAttribute(attn_prefill_kernel<64, false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    attn_prefill_kernel<64, false, true><<<grid, kAttnThreads, smem, stream>>>(p);
+  }
+  const cudaError_t e = cudaGetLastError();
+  return e == cudaSuccess ? 0 : -static_cast<int>(e) - 300;
 }
 
 // k (and v, may be null) rows [tokens][ld] with hkv heads of d values of esz bytes -> page pools

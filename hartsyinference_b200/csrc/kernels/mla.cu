@@ -15,6 +15,11 @@
 //                 tokens of a tile for the scores and the 512 output columns for P.V.
 //  * mla_combine: merges the KV splits.
 //
+// The attention kernel is a template over the latent width (64, 128, 256, 512) and the rotated part (64 or
+// none); rows narrower than the template's width are zero-filled on the way into shared memory. Without a
+// rotated part (latent attention without positions) the probabilities keep 16 bits of mantissa in the PV
+// product (a bf16 head and a bf16 remainder).
+//
 // Every query row carries its own kv length and block-table row, so a prefill chunk runs as rows
 // with causal lengths. Reference behaviour: src/HartsyInference.LLM/Transformer/MlaAttention.cs
 // (expanded K/V per head, contiguous KV cache, scalar attention).
@@ -26,7 +31,6 @@ namespace b200 {
 constexpr int kLat = 512;            // latent width (also the value width)
 constexpr int kRopeDim = 64;
 constexpr int kRow = kLat + kRopeDim;        // 576
-constexpr int kPitch = (kRow + 8) * 2;       // bytes per shared-memory row: 1168 (4-bank skew per row)
 constexpr int kMlaTile = 64;
 constexpr int kMlaThreads = 128;
 constexpr int kPPitch = (kMlaTile + 8) * 2;  // 144 bytes
@@ -105,48 +109,55 @@ __global__ void __launch_bounds__(128) mla_prep_kernel(const MlaPrepParams p) {
 }
 
 struct MlaAttnParams {
-  const __nv_bfloat16* q;       // [rows][heads][576]
-  const __nv_bfloat16* cache;   // [pages][page][576]
-  __nv_bfloat16* out;           // [rows][heads][512]
-  float* part_o;                // [rows][heads][splits][512]
+  const __nv_bfloat16* q;       // [rows][heads][row]
+  const __nv_bfloat16* cache;   // [pages][page][row]
+  __nv_bfloat16* out;           // [rows][heads][lat]
+  float* part_o;                // [rows][heads][splits][template width]
   float* part_ml;               // [rows][heads][splits][2]
   const int* block_table;       // [seqs][table_stride]
   const int* kv_lens;           // [rows]
   const int* row_seq;           // [rows] or null (row r uses block-table row r)
   int rows, heads, page, page_shift, table_stride, splits;
+  int row, lat;                 // values per cached row and per output row (multiples of 8)
   float scale_log2;
 };
 
 // kSets groups of four warps share one CTA and one staged KV tile; each group owns 16 heads of the
 // same query row (with many heads per row, as in the data-parallel attention layout, every tile that
 // is read from memory then serves 32 heads instead of 16, and eight warps hide each other's latencies).
-template <int kSets>
+template <int kL, int kR, int kSets, bool kSplitP>
 struct MlaSmem {
+  static constexpr int kPitch = (kL + kR + 8) * 2;     // bytes per row (4-bank skew per row)
   uint8_t kv[2][kMlaTile * kPitch];
   uint8_t q[kSets][16 * kPitch];
-  uint8_t pmat[kSets][16 * kPPitch];
+  uint8_t pmat[kSets][(kSplitP ? 2 : 1) * 16 * kPPitch];
   float red_max[kSets][4][16];
   float red_sum[kSets][4][16];
   int pages[2][kMaxPagesPerTile];
 };
 
+template <int kL, int kR>
 __device__ __forceinline__ void mla_load_tile(uint32_t dst, const MlaAttnParams& p, const int* pages,
                                               int tok0, int kv_len) {
-  // 64 tokens x 72 chunks of 16 bytes
+  constexpr int kRow = kL + kR, kPitch = (kRow + 8) * 2;
+  // 64 tokens in chunks of 16 bytes
   for (int i = threadIdx.x; i < kMlaTile * (kRow / 8); i += blockDim.x) {
     const int token = i / (kRow / 8), chunk = i - token * (kRow / 8);
     const int pos = tok0 + token;
-    const bool valid = pos < kv_len;
+    const bool valid = pos < kv_len && chunk * 8 < p.row;
     const int pg = valid ? pages[token >> p.page_shift] : 0;
-    const __nv_bfloat16* src = p.cache + (static_cast<long long>(pg) * p.page + (pos & (p.page - 1))) * kRow + chunk * 8;
+    const __nv_bfloat16* src = p.cache + (static_cast<long long>(pg) * p.page + (pos & (p.page - 1))) * p.row + chunk * 8;
     cp_async_16(dst + token * kPitch + chunk * 16, valid ? src : p.cache, valid);
   }
 }
 
-template <int kSets>
+template <int kL, int kR, int kSets, bool kSplitP>
 __global__ void __launch_bounds__(kMlaThreads * kSets) mla_attn_kernel(const MlaAttnParams p) {
+  constexpr int kRow = kL + kR, kCols = kL / 4;       // kCols: output columns per warp
+  using Smem = MlaSmem<kL, kR, kSets, kSplitP>;
+  constexpr int kPitch = Smem::kPitch;
   extern __shared__ __align__(16) uint8_t smem_raw[];
-  MlaSmem<kSets>& sm = *reinterpret_cast<MlaSmem<kSets>*>(smem_raw);
+  Smem& sm = *reinterpret_cast<Smem*>(smem_raw);
   const int row_q = blockIdx.y, split = blockIdx.z;
   const int tid = threadIdx.x, lane = tid & 31;
   const int set = kSets > 1 ? tid >> 7 : 0;      // which group of four warps
@@ -171,8 +182,8 @@ __global__ void __launch_bounds__(kMlaThreads * kSets) mla_attn_kernel(const Mla
   for (int i = tid; i < kSets * 16 * (kRow / 8); i += kMlaThreads * kSets) {
     const int hh = i / (kRow / 8), chunk = i - hh * (kRow / 8);
     const int head = blockIdx.x * kSets * 16 + hh;
-    const bool valid = head < p.heads;
-    const __nv_bfloat16* src = p.q + (static_cast<long long>(row_q) * p.heads + (valid ? head : 0)) * kRow + chunk * 8;
+    const bool valid = head < p.heads && chunk * 8 < p.row;
+    const __nv_bfloat16* src = p.q + (static_cast<long long>(row_q) * p.heads + (valid ? head : 0)) * p.row + (valid ? chunk * 8 : 0);
     cp_async_16(smem_u32(sm.q[0]) + hh * kPitch + chunk * 16, src, valid);
   }
   auto stage_pages = [&](int tile, int buf) {
@@ -185,12 +196,12 @@ __global__ void __launch_bounds__(kMlaThreads * kSets) mla_attn_kernel(const Mla
   };
   if (t0 < t1) stage_pages(t0, 0);
   __syncthreads();
-  if (t0 < t1) mla_load_tile(kv_s[0], p, sm.pages[0], t0 * kMlaTile, kv_len);
+  if (t0 < t1) mla_load_tile<kL, kR>(kv_s[0], p, sm.pages[0], t0 * kMlaTile, kv_len);
   cp_async_commit();
 
-  float o[16][4];
+  float o[kCols / 8][4];
 #pragma unroll
-  for (int i = 0; i < 16; ++i)
+  for (int i = 0; i < kCols / 8; ++i)
 #pragma unroll
     for (int j = 0; j < 4; ++j) o[i][j] = 0.f;
   float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
@@ -201,7 +212,7 @@ __global__ void __launch_bounds__(kMlaThreads * kSets) mla_attn_kernel(const Mla
     if (t + 1 < t1) {
       stage_pages(t + 1, buf ^ 1);
       __syncthreads();
-      mla_load_tile(kv_s[buf ^ 1], p, sm.pages[buf ^ 1], (t + 1) * kMlaTile, kv_len);
+      mla_load_tile<kL, kR>(kv_s[buf ^ 1], p, sm.pages[buf ^ 1], (t + 1) * kMlaTile, kv_len);
       cp_async_commit();
       cp_async_wait<1>();
     } else {
@@ -220,7 +231,7 @@ __global__ void __launch_bounds__(kMlaThreads * kSets) mla_attn_kernel(const Mla
       const int mi = lane >> 3;
       const uint32_t q_lane = q_s + (lane & 15) * kPitch + (lane >> 4) * 16;
       const uint32_t k_lane = kv_s[buf] + (warp * 16 + (lane & 7) + 8 * (mi >> 1)) * kPitch + (mi & 1) * 16;
-#pragma unroll 6
+#pragma unroll (kRow % 96 == 0 ? 6 : 4)
       for (int kk = 0; kk < kRow / 16; kk += 2) {
         uint32_t a[4], a2[4], b0, b1, b2, b3, c0, c1, c2, c3;
         ldmatrix_x4(q_lane + kk * 32, a[0], a[1], a[2], a[3]);
@@ -276,6 +287,12 @@ __global__ void __launch_bounds__(kMlaThreads * kSets) mla_attn_kernel(const Mla
       const int col = warp * 16 + nt * 8 + tq * 2;
       *reinterpret_cast<uint32_t*>(pmat + r0 * kPPitch + col * 2) = pack_bf16x2(e[0], e[1]);
       *reinterpret_cast<uint32_t*>(pmat + (r0 + 8) * kPPitch + col * 2) = pack_bf16x2(e[2], e[3]);
+      if (kSplitP) {
+#pragma unroll
+        for (int j = 0; j < 4; ++j) e[j] -= __bfloat162float(__float2bfloat16(e[j]));
+        *reinterpret_cast<uint32_t*>(pmat + (r0 + 16) * kPPitch + col * 2) = pack_bf16x2(e[0], e[1]);
+        *reinterpret_cast<uint32_t*>(pmat + (r0 + 24) * kPPitch + col * 2) = pack_bf16x2(e[2], e[3]);
+      }
     }
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
@@ -284,7 +301,7 @@ __global__ void __launch_bounds__(kMlaThreads * kSets) mla_attn_kernel(const Mla
     }
     if (tq == 0) { red_sum[warp][r0] = rs[0]; red_sum[warp][r0 + 8] = rs[1]; }
 #pragma unroll
-    for (int i = 0; i < 16; ++i) {
+    for (int i = 0; i < kCols / 8; ++i) {
       o[i][0] *= alpha[0]; o[i][1] *= alpha[0];
       o[i][2] *= alpha[1]; o[i][3] *= alpha[1];
     }
@@ -294,20 +311,26 @@ __global__ void __launch_bounds__(kMlaThreads * kSets) mla_attn_kernel(const Mla
       const int rr = r0 + 8 * r;
       l_run[r] = l_run[r] * alpha[r] + red_sum[0][rr] + red_sum[1][rr] + red_sum[2][rr] + red_sum[3][rr];
     }
-    // ---- O[:, warp * 128 ...] += P V
+    // ---- O[:, warp * kCols ...] += P V
 #pragma unroll
     for (int kk = 0; kk < kMlaTile / 16; ++kk) {
       uint32_t a[4];
       ldmatrix_x4(p_s + (lane & 15) * kPPitch + (kk * 2 + (lane >> 4)) * 16, a[0], a[1], a[2], a[3]);
+      uint32_t al[4];
+      if (kSplitP) ldmatrix_x4(p_s + (16 + (lane & 15)) * kPPitch + (kk * 2 + (lane >> 4)) * 16, al[0], al[1], al[2], al[3]);
 #pragma unroll
-      for (int np = 0; np < 8; ++np) {
+      for (int np = 0; np < kCols / 16; ++np) {
         const int mi = lane >> 3;
         const int token = kk * 16 + (lane & 7) + 8 * (mi & 1);
-        const int chunk = warp * 16 + np * 2 + (mi >> 1);
+        const int chunk = warp * (kCols / 8) + np * 2 + (mi >> 1);
         uint32_t b0, b1, b2, b3;
         ldmatrix_x4_trans(kv_s[buf] + token * kPitch + chunk * 16, b0, b1, b2, b3);
         mma_bf16_16816(o[np * 2], a, b0, b1);
         mma_bf16_16816(o[np * 2 + 1], a, b2, b3);
+        if (kSplitP) {
+          mma_bf16_16816(o[np * 2], al, b0, b1);
+          mma_bf16_16816(o[np * 2 + 1], al, b2, b3);
+        }
       }
     }
     __syncthreads();   // the tile, P and the reduction slots are reused by the next iteration
@@ -322,14 +345,15 @@ __global__ void __launch_bounds__(kMlaThreads * kSets) mla_attn_kernel(const Mla
     const long long rh = static_cast<long long>(row_q) * p.heads + hg * 16 + h;
     if (p.splits == 1) {
       const float inv = l_run[r] > 0.f ? 1.f / l_run[r] : 0.f;
-      __nv_bfloat16* dst = p.out + rh * kLat + warp * 128 + tq * 2;
+      __nv_bfloat16* dst = p.out + rh * p.lat + warp * kCols + tq * 2;
 #pragma unroll
-      for (int nt = 0; nt < 16; ++nt)
-        *reinterpret_cast<uint32_t*>(dst + nt * 8) = pack_bf16x2(o[nt][2 * r] * inv, o[nt][2 * r + 1] * inv);
+      for (int nt = 0; nt < kCols / 8; ++nt)
+        if (warp * kCols + nt * 8 < p.lat)
+          *reinterpret_cast<uint32_t*>(dst + nt * 8) = pack_bf16x2(o[nt][2 * r] * inv, o[nt][2 * r + 1] * inv);
     } else {
-      float* dst = p.part_o + (rh * p.splits + split) * kLat + warp * 128 + tq * 2;
+      float* dst = p.part_o + (rh * p.splits + split) * kL + warp * kCols + tq * 2;
 #pragma unroll
-      for (int nt = 0; nt < 16; ++nt)
+      for (int nt = 0; nt < kCols / 8; ++nt)
         *reinterpret_cast<float2*>(dst + nt * 8) = make_float2(o[nt][2 * r], o[nt][2 * r + 1]);
       if (warp == 0 && tq == 0) {
         p.part_ml[(rh * p.splits + split) * 2] = m_run[r];
@@ -339,7 +363,8 @@ __global__ void __launch_bounds__(kMlaThreads * kSets) mla_attn_kernel(const Mla
   }
 }
 
-// One block of 128 threads per (row, head): out = sum_s 2^(m_s - M) O_s / sum_s 2^(m_s - M) l_s.
+// One block of kL / 4 threads per (row, head): out = sum_s 2^(m_s - M) O_s / sum_s 2^(m_s - M) l_s.
+template <int kL>
 __global__ void mla_combine_kernel(const MlaAttnParams p) {
   const long long rh = blockIdx.x;
   const float* ml = p.part_ml + rh * p.splits * 2;
@@ -352,7 +377,7 @@ __global__ void mla_combine_kernel(const MlaAttnParams p) {
     if (m == -INFINITY) continue;
     const float wgt = exp2f(m - big);
     den += wgt * ml[2 * s + 1];
-    const float4 v = *reinterpret_cast<const float4*>(p.part_o + (rh * p.splits + s) * kLat + threadIdx.x * 4);
+    const float4 v = *reinterpret_cast<const float4*>(p.part_o + (rh * p.splits + s) * kL + threadIdx.x * 4);
     acc[0] += wgt * v.x; acc[1] += wgt * v.y; acc[2] += wgt * v.z; acc[3] += wgt * v.w;
   }
   const float inv = den > 0.f ? 1.f / den : 0.f;
@@ -360,7 +385,7 @@ __global__ void mla_combine_kernel(const MlaAttnParams p) {
   uint32_t* ow = reinterpret_cast<uint32_t*>(&o);
   ow[0] = pack_bf16x2(acc[0] * inv, acc[1] * inv);
   ow[1] = pack_bf16x2(acc[2] * inv, acc[3] * inv);
-  *reinterpret_cast<uint2*>(p.out + rh * kLat + threadIdx.x * 4) = o;
+  if (static_cast<int>(threadIdx.x) * 4 < p.lat) *reinterpret_cast<uint2*>(p.out + rh * p.lat + threadIdx.x * 4) = o;
 }
 
 }  // namespace b200
@@ -399,39 +424,71 @@ B200_API long long b200_mla_workspace_bytes(int rows, int heads, int splits) {
   return static_cast<long long>(rows) * heads * splits * (kLat + 2) * 4;
 }
 
-B200_API int b200_mla_attn(const void* q, const void* cache, void* out, const int* block_table,
-                           const int* kv_lens, const int* row_seq, int rows, int heads, int page,
-                           int table_stride, int splits, void* workspace, float scale, cudaStream_t stream) {
-  if (rows <= 0) return 0;
+template <int kL, int kR, bool kSplitP>
+static int launch_mla(MlaAttnParams p, void* workspace, cudaStream_t stream) {
+  p.part_o = static_cast<float*>(workspace);
+  p.part_ml = p.part_o ? p.part_o + static_cast<long long>(p.rows) * p.heads * p.splits * kL : nullptr;
+  constexpr int smem1 = static_cast<int>(sizeof(MlaSmem<kL, kR, 1, kSplitP>)), smem2 = static_cast<int>(sizeof(MlaSmem<kL, kR, 2, kSplitP>));
+  static PerDeviceOnce configured;
+  if (configured.first_time()) {
+    if (cudaFuncSetAttribute(mla_attn_kernel<kL, kR, 1, kSplitP>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem1) != cudaSuccess ||
+        cudaFuncSetAttribute(mla_attn_kernel<kL, kR, 2, kSplitP>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem2) != cudaSuccess)
+      return -4;
+  }
+  if (mla_sets(p.heads) == 2) {
+    mla_attn_kernel<kL, kR, 2, kSplitP><<<dim3((p.heads + 31) / 32, p.rows, p.splits), kMlaThreads * 2, smem2, stream>>>(p);
+  } else {
+    mla_attn_kernel<kL, kR, 1, kSplitP><<<dim3((p.heads + 15) / 16, p.rows, p.splits), kMlaThreads, smem1, stream>>>(p);
+  }
+  if (p.splits > 1) mla_combine_kernel<kL><<<p.rows * p.heads, kL / 4, 0, stream>>>(p);
+  return cudaGetLastError() == cudaSuccess ? 0 : -300;
+}
+
+static int mla_params(MlaAttnParams& p, const void* q, const void* cache, void* out, const int* block_table, const int* kv_lens,
+                      const int* row_seq, int rows, int heads, int page, int table_stride, int splits, void* workspace,
+                      float scale) {
   int shift = 0;
   while ((1 << shift) < page) ++shift;
-  if ((1 << shift) != page || page < 8 || page > kMlaTile) return -2;
+  if ((1 << shift) != page || page < 8 || page > kMlaTile || rows > 65535) return -2;
   if (splits < 1) splits = 1;
   if (splits > 1 && workspace == nullptr) return -3;
-  MlaAttnParams p{};
   p.q = static_cast<const __nv_bfloat16*>(q);
   p.cache = static_cast<const __nv_bfloat16*>(cache);
   p.out = static_cast<__nv_bfloat16*>(out);
-  p.part_o = static_cast<float*>(workspace);
-  p.part_ml = p.part_o ? p.part_o + static_cast<long long>(rows) * heads * splits * kLat : nullptr;
   p.block_table = block_table;
   p.kv_lens = kv_lens;
   p.row_seq = row_seq;
   p.rows = rows; p.heads = heads; p.page = page; p.page_shift = shift; p.table_stride = table_stride;
   p.splits = splits;
   p.scale_log2 = scale * 1.4426950408889634f;
-  static PerDeviceOnce configured;
-  const int smem1 = static_cast<int>(sizeof(MlaSmem<1>)), smem2 = static_cast<int>(sizeof(MlaSmem<2>));
-  if (configured.first_time()) {
-    if (cudaFuncSetAttribute(mla_attn_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem1) != cudaSuccess ||
-        cudaFuncSetAttribute(mla_attn_kernel<2>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem2) != cudaSuccess)
-      return -4;
-  }
-  if (mla_sets(heads) == 2) {
-    mla_attn_kernel<2><<<dim3((heads + 31) / 32, rows, splits), kMlaThreads * 2, smem2, stream>>>(p);
-  } else {
-    mla_attn_kernel<1><<<dim3((heads + 15) / 16, rows, splits), kMlaThreads, smem1, stream>>>(p);
-  }
-  if (splits > 1) mla_combine_kernel<<<rows * heads, 128, 0, stream>>>(p);
-  return cudaGetLastError() == cudaSuccess ? 0 : -300;
+  return 0;
+}
+
+B200_API int b200_mla_attn(const void* q, const void* cache, void* out, const int* block_table,
+                           const int* kv_lens, const int* row_seq, int rows, int heads, int page,
+                           int table_stride, int splits, void* workspace, float scale, cudaStream_t stream) {
+  if (rows <= 0) return 0;
+  MlaAttnParams p{};
+  const int rc = mla_params(p, q, cache, out, block_table, kv_lens, row_seq, rows, heads, page, table_stride, splits, workspace, scale);
+  if (rc) return rc;
+  p.row = kRow;
+  p.lat = kLat;
+  return launch_mla<kLat, kRopeDim, false>(p, workspace, stream);
+}
+
+// Latent attention without a rotated part: rows of `rank` values (a multiple of 8, at most 512), q
+// [rows][heads][rank], out the same. The workspace is that of b200_mla_workspace_bytes.
+B200_API int b200_latent_attn(const void* q, const void* cache, void* out, const int* block_table, const int* kv_lens,
+                              const int* row_seq, int rows, int heads, int rank, int page, int table_stride, int splits,
+                              void* workspace, float scale, cudaStream_t stream) {
+  if (rows <= 0) return 0;
+  if (rank % 8 || rank < 8 || rank > kLat) return -2;
+  MlaAttnParams p{};
+  const int rc = mla_params(p, q, cache, out, block_table, kv_lens, row_seq, rows, heads, page, table_stride, splits, workspace, scale);
+  if (rc) return rc;
+  p.row = p.lat = rank;
+  if (rank <= 64) return launch_mla<64, 0, true>(p, workspace, stream);
+  if (rank <= 128) return launch_mla<128, 0, true>(p, workspace, stream);
+  if (rank <= 256) return launch_mla<256, 0, true>(p, workspace, stream);
+  return launch_mla<512, 0, true>(p, workspace, stream);
 }

@@ -1,7 +1,7 @@
 // Norms around a 32-bit residual stream, and the embedding that starts it.
 //
-//   x  <- x + norm(y) * w_b                  (sublayer output; left out for the first norm of a stack)
-//   h  <- norm(x) * w_n                      (input of the next sublayer or of the output head)
+//   x  <- x + m * norm(y) * w_b              (sublayer output; left out for the first norm of a stack)
+//   h  <- norm(x) * w_n                      (input of the next sublayer or of the output head; or x itself)
 //
 // in one launch per sublayer: the row stays in registers between the two norms, the stream is read
 // and written once as fp32, y and h are in the activation type (bf16, or fp32 for a model run in
@@ -9,8 +9,10 @@
 //   y[t] = sum_k w[t][k] * (slot_of[t][k] >= 0 ? rows[slot_of[t][k]] : ids[t][k] >= experts ? src[t] : 0)
 // is formed in registers first (an expert index past the last real expert returns its input), so the
 // combine step of a mixture of experts needs no launch and no intermediate rounding of its own.
-// LayerNorm (weight, no bias) or RMSNorm; statistics in two passes over the registers, in fp32.
-#include "common.cuh"
+// LayerNorm (weight, no bias) or RMSNorm; weights as stored or stored around zero (1 + w); statistics in two
+// passes over the registers, in fp32. The embedding can be normed on its way into the stream, and poly_norm is
+// the activation that mixes a row's normed powers.
+#include "mixer_common.cuh"
 
 namespace b200 {
 
@@ -25,60 +27,16 @@ struct ResidualNormParams {
   const float* wts;          //                [rows][top_k]
   const void* src;           //                [rows][ld_src] what a pass-through expert returns
   int dim, ldx, ldy, ldh, ld_src, top_k, experts, layernorm;
-  float eps;
+  int plus_one;              // norms multiply by 1 + w
+  int plain;                 // no w_n: h is the stream itself
+  float eps, mult;           // mult: factor of the (normed) sublayer output
 };
-
-template <typename T>
-__device__ __forceinline__ void load8(const T* p, float (&v)[8]);
-template <>
-__device__ __forceinline__ void load8<__nv_bfloat16>(const __nv_bfloat16* p, float (&v)[8]) {
-  const uint4 raw = *reinterpret_cast<const uint4*>(p);
-  const __nv_bfloat162* b = reinterpret_cast<const __nv_bfloat162*>(&raw);
-#pragma unroll
-  for (int i = 0; i < 4; ++i) {
-    const float2 f = __bfloat1622float2(b[i]);
-    v[2 * i] = f.x;
-    v[2 * i + 1] = f.y;
-  }
-}
-template <>
-__device__ __forceinline__ void load8<float>(const float* p, float (&v)[8]) {
-  const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
-  v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
-  v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
-}
-template <typename T>
-__device__ __forceinline__ void store8(T* p, const float (&v)[8]);
-template <>
-__device__ __forceinline__ void store8<__nv_bfloat16>(__nv_bfloat16* p, const float (&v)[8]) {
-  uint4 o;
-  o.x = pack_bf16x2(v[0], v[1]);
-  o.y = pack_bf16x2(v[2], v[3]);
-  o.z = pack_bf16x2(v[4], v[5]);
-  o.w = pack_bf16x2(v[6], v[7]);
-  *reinterpret_cast<uint4*>(p) = o;
-}
-template <>
-__device__ __forceinline__ void store8<float>(float* p, const float (&v)[8]) {
-  *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
-  *reinterpret_cast<float4*>(p + 4) = make_float4(v[4], v[5], v[6], v[7]);
-}
-
-__device__ __forceinline__ float block_sum(float v, float* red) {
-  v = warp_sum(v);
-  __syncthreads();
-  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
-  __syncthreads();
-  const int n = blockDim.x >> 5;
-  float s = 0.f;
-  for (int i = 0; i < n; ++i) s += red[i];
-  return s;
-}
 
 // v <- norm(v) * w over the row's first `dim` values (values past them are zero on entry and exit)
 template <int kIters>
 __device__ __forceinline__ void norm_row(float (&v)[kIters][8], const __nv_bfloat16* w, int dim, int layernorm,
-                                         float eps, float* red) {
+                                         int plus_one, float eps, float* red) {
+  const float one = plus_one ? 1.f : 0.f;
   float mean = 0.f;
   if (layernorm) {
     float s = 0.f;
@@ -106,10 +64,10 @@ __device__ __forceinline__ void norm_row(float (&v)[kIters][8], const __nv_bfloa
       float wv[8];
       load8(w + c, wv);
 #pragma unroll
-      for (int j = 0; j < 8; ++j) v[i][j] = (v[i][j] - mean) * inv * wv[j];
+      for (int j = 0; j < 8; ++j) v[i][j] = (v[i][j] - mean) * inv * (one + wv[j]);
     } else {
 #pragma unroll
-      for (int j = 0; j < 8; ++j) v[i][j] = c + j < dim ? (v[i][j] - mean) * inv * __bfloat162float(w[c + j]) : 0.f;
+      for (int j = 0; j < 8; ++j) v[i][j] = c + j < dim ? (v[i][j] - mean) * inv * (one + __bfloat162float(w[c + j])) : 0.f;
     }
   }
 }
@@ -163,7 +121,7 @@ __global__ void __launch_bounds__(1024) residual_norm_kernel(const ResidualNormP
       for (int j = 0; j < 8; ++j)
         if (c + j >= p.dim) yv[i][j] = 0.f;
     }
-    if (p.w_b != nullptr) norm_row<kIters>(yv, p.w_b, p.dim, p.layernorm, p.eps, red);
+    if (p.w_b != nullptr) norm_row<kIters>(yv, p.w_b, p.dim, p.layernorm, p.plus_one, p.eps, red);
 #pragma unroll
     for (int i = 0; i < kIters; ++i) {
       const int c = (threadIdx.x + i * blockDim.x) * 8;
@@ -172,7 +130,7 @@ __global__ void __launch_bounds__(1024) residual_norm_kernel(const ResidualNormP
       if (c < p.dim) {
         load8(xr + c, xv[i]);
 #pragma unroll
-        for (int j = 0; j < 8; ++j) xv[i][j] += yv[i][j];
+        for (int j = 0; j < 8; ++j) xv[i][j] = fmaf(p.mult, yv[i][j], xv[i][j]);
         store8(xr + c, xv[i]);
       }
     }
@@ -185,8 +143,8 @@ __global__ void __launch_bounds__(1024) residual_norm_kernel(const ResidualNormP
       if (c < p.dim) load8(xr + c, xv[i]);
     }
   }
-  if (p.w_n == nullptr) return;
-  norm_row<kIters>(xv, p.w_n, p.dim, p.layernorm, p.eps, red);
+  if (p.w_n == nullptr && !p.plain) return;
+  if (p.w_n != nullptr) norm_row<kIters>(xv, p.w_n, p.dim, p.layernorm, p.plus_one, p.eps, red);
   T* hr = static_cast<T*>(p.h) + row * p.ldh;
 #pragma unroll
   for (int i = 0; i < kIters; ++i) {
@@ -212,13 +170,118 @@ __global__ void embedding_f32_kernel(const int* __restrict__ ids, const __nv_bfl
   }
 }
 
+// x[t] = norm(table[id]) * w in fp32 (the stream) and h[t] = x[t] in the activation type. ids null: the rows of
+// `table` in order.
+struct EmbeddingNormParams {
+  const int* ids;
+  const __nv_bfloat16* table;
+  const __nv_bfloat16* w;
+  float* x;
+  void* h;
+  int dim, ldx, ldt, vocab, layernorm, plus_one;
+  float scale, eps;
+};
+
+template <typename T, int kIters>
+__global__ void __launch_bounds__(1024) embedding_norm_kernel(const EmbeddingNormParams p) {
+  pdl_wait();
+  pdl_trigger();
+  __shared__ float red[32];
+  const long long t = blockIdx.x;
+  long long id = t;
+  if (p.ids) id = min(max(p.ids[t], 0), p.vocab - 1);
+  const __nv_bfloat16* src = p.table + id * p.ldt;
+  float v[kIters][8];
+#pragma unroll
+  for (int i = 0; i < kIters; ++i) {
+    const int c = (threadIdx.x + i * blockDim.x) * 8;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) v[i][j] = 0.f;
+    if (c < p.dim) load8(src + c, v[i]);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) v[i][j] = c + j < p.dim ? v[i][j] * p.scale : 0.f;
+  }
+  norm_row<kIters>(v, p.w, p.dim, p.layernorm, p.plus_one, p.eps, red);
+#pragma unroll
+  for (int i = 0; i < kIters; ++i) {
+    const int c = (threadIdx.x + i * blockDim.x) * 8;
+    if (c < p.ldx) {
+      store8(p.x + t * p.ldx + c, v[i]);
+      store8(static_cast<T*>(p.h) + t * p.ldx + c, v[i]);
+    }
+  }
+}
+
+// y = a z / rms(z) + b z^2 / rms(z^2) + c z^3 / rms(z^3) + e over a row of `dim` values (powers element by
+// element); columns past dim are zeroed. The row stays in registers between the two passes.
+template <typename T, int kIters>
+__global__ void __launch_bounds__(1024) poly_norm_kernel(const T* __restrict__ z, T* __restrict__ y,
+                                                         const float* __restrict__ coef, int dim, int ldz, int ldy, float eps) {
+  pdl_wait();
+  pdl_trigger();
+  __shared__ float red[3][32];
+  const long long row = blockIdx.x;
+  float v[kIters][8];
+  float q1 = 0.f, q2 = 0.f, q3 = 0.f;
+#pragma unroll
+  for (int i = 0; i < kIters; ++i) {
+    const int c = (threadIdx.x + i * blockDim.x) * 8;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) v[i][j] = 0.f;
+    if (c < dim) load8(z + row * ldz + c, v[i]);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      if (c + j >= dim) v[i][j] = 0.f;
+      const float s = v[i][j] * v[i][j];
+      q1 += s;
+      q2 = fmaf(s, s, q2);
+      q3 = fmaf(s * s, s, q3);
+    }
+  }
+  q1 = warp_sum(q1);
+  q2 = warp_sum(q2);
+  q3 = warp_sum(q3);
+  if ((threadIdx.x & 31) == 0) {
+    red[0][threadIdx.x >> 5] = q1;
+    red[1][threadIdx.x >> 5] = q2;
+    red[2][threadIdx.x >> 5] = q3;
+  }
+  __syncthreads();
+  q1 = q2 = q3 = 0.f;
+  for (int i = 0; i < static_cast<int>(blockDim.x >> 5); ++i) {
+    q1 += red[0][i];
+    q2 += red[1][i];
+    q3 += red[2][i];
+  }
+  const float a = coef[0] / sqrtf(q1 / dim + eps), b = coef[1] / sqrtf(q2 / dim + eps), c3 = coef[2] / sqrtf(q3 / dim + eps);
+  const float e = coef[3];
+#pragma unroll
+  for (int i = 0; i < kIters; ++i) {
+    const int c = (threadIdx.x + i * blockDim.x) * 8;
+    if (c >= ldy) continue;
+    float o[8];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      const float u = v[i][j];
+      o[j] = c + j < dim ? fmaf(u, fmaf(u, fmaf(u, c3, b), a), e) : 0.f;
+    }
+    store8(y + row * ldy + c, o);
+  }
+}
+
+// Rows of up to 16384 values, eight per thread and vector: two vectors per thread for long rows, and when there
+// are many rows (more bytes in flight per thread).
+inline bool row_shape(int dim, int rows, int& iters, int& threads) {
+  const int vecs = (dim + 7) / 8;
+  iters = vecs > 1024 || (rows >= 1024 && vecs >= 128) ? 2 : 1;
+  threads = ((vecs + iters - 1) / iters + 31) / 32 * 32;
+  return threads <= 1024;
+}
+
 template <typename T>
 int launch_residual_norm(const ResidualNormParams& p, int rows, cudaStream_t stream) {
-  const int vecs = (p.dim + 7) / 8;
-  // two vectors per thread for long rows, and when there are many rows (more bytes in flight per thread)
-  const int iters = vecs > 1024 || (rows >= 1024 && vecs >= 128) ? 2 : 1;
-  int threads = ((vecs + iters - 1) / iters + 31) / 32 * 32;
-  if (threads > 1024) return -2;
+  int iters, threads;
+  if (!row_shape(p.dim, rows, iters, threads)) return -2;
   cudaError_t e;
   switch (iters) {
     case 1: e = launch_pdl(residual_norm_kernel<T, 1>, dim3(rows), dim3(threads), 0, stream, p); break;
@@ -235,16 +298,16 @@ using namespace b200;
 // multiples of 8. Rows of at most 16384 values.
 B200_API int b200_residual_norm(void* x, const void* y, void* h, const void* w_b, const void* w_n, const int* slot_of,
                                 const int* ids, const float* wts, const void* src, int rows, int dim, int ldx, int ldy,
-                                int ldh, int ld_src, int top_k, int experts, int layernorm, float eps, int f32,
-                                cudaStream_t stream) {
+                                int ldh, int ld_src, int top_k, int experts, int layernorm, int plus_one, int plain, float eps,
+                                float mult, int f32, cudaStream_t stream) {
   if (rows <= 0) return 0;
   const int dim8 = (dim + 7) / 8 * 8;
-  if (dim < 1 || dim > 16384 || ldx < dim8 || ldx % 8 || (w_n && (ldh != dim8 || !h))) return -2;
+  if (dim < 1 || dim > 16384 || ldx < dim8 || ldx % 8 || ((w_n || plain) && (ldh != dim8 || !h))) return -2;
   if (y && (ldy < dim8 || ldy % 8)) return -2;
   if (slot_of && (!ids || !wts || top_k < 1 || (src && (ld_src < dim8 || ld_src % 8)))) return -2;
   ResidualNormParams p{static_cast<float*>(x), y, h, static_cast<const __nv_bfloat16*>(w_b),
                        static_cast<const __nv_bfloat16*>(w_n), slot_of, ids, wts, src, dim, ldx, ldy, ldh, ld_src, top_k,
-                       experts, layernorm, eps};
+                       experts, layernorm, plus_one, plain, eps, mult};
   return f32 ? launch_residual_norm<float>(p, rows, stream) : launch_residual_norm<__nv_bfloat16>(p, rows, stream);
 }
 
@@ -257,4 +320,38 @@ B200_API int b200_embedding_f32(const int* ids, const void* table, void* x, int 
   embedding_f32_kernel<<<tokens, threads, 0, stream>>>(ids, static_cast<const __nv_bfloat16*>(table), static_cast<float*>(x),
                                                        dim, ldx, ldt, vocab, scale);
   return cudaGetLastError() == cudaSuccess ? 0 : -300;
+}
+
+// x fp32 and h (activation type) [tokens][ldx] = norm(table[ids] * scale) * w
+B200_API int b200_embedding_norm(const int* ids, const void* table, const void* w, void* x, void* h, int tokens, int dim,
+                                 int ldx, int ldt, int vocab, float scale, int layernorm, int plus_one, float eps, int f32,
+                                 cudaStream_t stream) {
+  if (tokens <= 0) return 0;
+  int iters, threads;
+  if (ldx % 8 || ldt % 8 || ldx != (dim + 7) / 8 * 8 || ldt < ldx || !row_shape(dim, tokens, iters, threads)) return -2;
+  EmbeddingNormParams p{ids, static_cast<const __nv_bfloat16*>(table), static_cast<const __nv_bfloat16*>(w),
+                        static_cast<float*>(x), h, dim, ldx, ldt, vocab, layernorm, plus_one, scale, eps};
+  cudaError_t e;
+  if (f32) e = iters == 1 ? launch_pdl(embedding_norm_kernel<float, 1>, dim3(tokens), dim3(threads), 0, stream, p)
+                          : launch_pdl(embedding_norm_kernel<float, 2>, dim3(tokens), dim3(threads), 0, stream, p);
+  else e = iters == 1 ? launch_pdl(embedding_norm_kernel<__nv_bfloat16, 1>, dim3(tokens), dim3(threads), 0, stream, p)
+                      : launch_pdl(embedding_norm_kernel<__nv_bfloat16, 2>, dim3(tokens), dim3(threads), 0, stream, p);
+  return e == cudaSuccess ? 0 : -static_cast<int>(e) - 300;
+}
+
+// y [rows][ldy] from z [rows][ldz]; coef: the four numbers a, b, c, e (fp32, device)
+B200_API int b200_poly_norm(const void* z, void* y, const float* coef, int rows, int dim, int ldz, int ldy, float eps, int f32,
+                            cudaStream_t stream) {
+  if (rows <= 0) return 0;
+  int iters, threads;
+  if (ldz % 8 || ldy != (dim + 7) / 8 * 8 || ldz < ldy || !row_shape(dim, rows, iters, threads)) return -2;
+  auto go = [&](auto kernel, auto tag) {
+    using T = decltype(tag);
+    return launch_pdl(kernel, dim3(rows), dim3(threads), 0, stream, static_cast<const T*>(z), static_cast<T*>(y), coef, dim, ldz,
+                      ldy, eps);
+  };
+  cudaError_t e;
+  if (f32) e = iters == 1 ? go(poly_norm_kernel<float, 1>, float()) : go(poly_norm_kernel<float, 2>, float());
+  else e = iters == 1 ? go(poly_norm_kernel<__nv_bfloat16, 1>, __nv_bfloat16()) : go(poly_norm_kernel<__nv_bfloat16, 2>, __nv_bfloat16());
+  return e == cudaSuccess ? 0 : -static_cast<int>(e) - 300;
 }

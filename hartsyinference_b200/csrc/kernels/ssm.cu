@@ -7,7 +7,25 @@
 // Decode runs with T = 1. The state is fp32 and updated in place.
 //
 // Reference: the scan of src/HartsyInference.LLM/Ssm/ (CPU loop / per-op GPU kernels).
-#include "common.cuh"
+//
+// The rest of this file is the batched form that the serving engine runs: ragged batches of portions of
+// sequences (cu_q), states in slots, bf16 or fp32 activations. A sequence whose portion starts at position 0
+// starts from zeros whatever its slot held before; a negative slot is computed from zeros and stored nowhere.
+//
+//  * short_conv     causal convolution per channel + bias + silu over any column range of a projection; its
+//                   last taps - 1 inputs are state too. short_conv_tail saves them after a portion.
+//  * channel_scan   one decay per channel and state value (the recurrence above). Four lanes share a channel
+//                   and walk over the tokens with their part of its state in registers; everything that does
+//                   not depend on the state (step size, dt x, D x, silu(z)) is formed once per element while a
+//                   tile of tokens is staged in shared memory, and the sums of four tokens are reduced over the
+//                   four lanes in one transposed exchange.
+//  * head_scan      one decay per head, state N x P: S = a S + B (dt x)^T, y = S^T C + D x. A thread keeps 8 rows
+//                   x 4 columns of S as packed pairs; otherwise like channel_scan.
+//  * channel_step, head_step   the same for one token per sequence (decode): the state is read once, updated,
+//                   written back.
+//  * gated_norm     y silu(z), RMS-normed in equal parts of the row.
+// The scans perform the same operations in the same order wherever a prompt is cut.
+#include "mixer_common.cuh"
 
 namespace b200 {
 
@@ -72,6 +90,736 @@ __global__ void __launch_bounds__(128) selective_scan_kernel(const ScanParams p)
   }
 }
 
+// ---------------------------------------------------------------------------------------------------------
+// short convolution
+// ---------------------------------------------------------------------------------------------------------
+struct ShortConvParams {
+  const void* x;             // [T][ldx], the channels start here
+  const float* w;            // [taps][channels], last row: the current token
+  const float* bias;         // [channels] or null
+  void* state;               // [slots][taps - 1][channels]
+  const int* positions;      // [T]
+  const int* cu_q;           // [seqs + 1]; null: one token per sequence
+  const int* slots;          // [seqs]
+  void* out;                 // [T][channels]
+  long long ldx;
+  int tokens, seqs, channels, taps, run;
+};
+
+__device__ __forceinline__ float silu_f32(float x) { return x * sigmoid_f32(x); }
+
+// kTaps inputs of eight channels in registers for `run` consecutive tokens. kTaps 0: any number of taps, inputs
+// are read again for every token. grid (ceil(channels / 256), ceil(T / (4 run))), 128 threads.
+template <typename T, int kTaps>
+__global__ void __launch_bounds__(128) short_conv_kernel(const ShortConvParams p) {
+  pdl_wait();
+  pdl_trigger();
+  const int lane = threadIdx.x & 31;
+  const int c = (blockIdx.x * 32 + lane) * 8;
+  const int t0 = (blockIdx.y * 4 + (threadIdx.x >> 5)) * p.run, t1 = min(t0 + p.run, p.tokens);
+  if (c >= p.channels || t0 >= t1) return;
+  const int taps = kTaps > 0 ? kTaps : p.taps, tail = taps - 1;
+  const T* x = static_cast<const T*>(p.x) + c;
+  T* out = static_cast<T*>(p.out) + c;
+  float bias[8];
+#pragma unroll
+  for (int i = 0; i < 8; ++i) bias[i] = 0.f;
+  if (p.bias) load8(p.bias + c, bias);
+  float w[kTaps > 0 ? kTaps : 1][8], in[kTaps > 0 ? kTaps : 1][8];
+  if (kTaps > 0)
+#pragma unroll
+    for (int j = 0; j < kTaps; ++j) load8(p.w + static_cast<long long>(j) * p.channels + c, w[kTaps > 0 ? j : 0]);
+  int seq = p.cu_q ? seq_of_token(p.cu_q, p.seqs, t0) : t0;
+  int first = 0, next = 0;
+  bool fresh = true, carried = false;
+  T* st = nullptr;
+  for (int t = t0; t < t1; ++t) {
+    if (fresh || t >= next) {
+      if (!fresh) ++seq;
+      if (p.cu_q) while (p.cu_q[seq + 1] <= t) ++seq;      // empty runs
+      fresh = false;
+      first = p.cu_q ? p.cu_q[seq] : t;
+      next = p.cu_q ? p.cu_q[seq + 1] : t + 1;
+      const int slot = p.slots[seq];
+      carried = slot >= 0 && p.positions[first] > 0;
+      st = slot >= 0 ? static_cast<T*>(p.state) + static_cast<long long>(slot) * tail * p.channels + c : nullptr;
+      if (kTaps > 0)
+#pragma unroll
+        for (int j = 0; j < kTaps - 1; ++j) {
+          float (&v)[8] = in[kTaps > 0 ? j : 0];
+#pragma unroll
+          for (int i = 0; i < 8; ++i) v[i] = 0.f;
+          const int src = t - tail + j;
+          if (src >= first) load8(x + src * p.ldx, v);
+          else if (carried) load8(st + static_cast<long long>(tail + src - first) * p.channels, v);
+        }
+    }
+    float y[8];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) y[i] = bias[i];
+    if (kTaps > 0) {
+      load8(x + t * p.ldx, in[kTaps > 0 ? kTaps - 1 : 0]);
+#pragma unroll
+      for (int j = 0; j < kTaps; ++j)
+#pragma unroll
+        for (int i = 0; i < 8; ++i) y[i] = fmaf(in[kTaps > 0 ? j : 0][i], w[kTaps > 0 ? j : 0][i], y[i]);
+      if (p.cu_q == nullptr && st != nullptr)
+#pragma unroll
+        for (int j = 1; j < kTaps; ++j) store8(st + static_cast<long long>(j - 1) * p.channels, in[kTaps > 0 ? j : 0]);
+#pragma unroll
+      for (int j = 0; j + 1 < kTaps; ++j)
+#pragma unroll
+        for (int i = 0; i < 8; ++i) in[kTaps > 0 ? j : 0][i] = in[kTaps > 0 ? j + 1 : 0][i];
+    } else {
+      for (int j = 0; j < taps; ++j) {
+        const int src = t - tail + j;
+        float v[8], wj[8];
+#pragma unroll
+        for (int i = 0; i < 8; ++i) v[i] = 0.f;
+        if (src >= first) load8(x + src * p.ldx, v);
+        else if (carried) load8(st + static_cast<long long>(tail + src - first) * p.channels, v);
+        if (p.cu_q == nullptr && st != nullptr && j > 0) store8(st + static_cast<long long>(j - 1) * p.channels, v);
+        load8(p.w + static_cast<long long>(j) * p.channels + c, wj);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) y[i] = fmaf(v[i], wj[i], y[i]);
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < 8; ++i) y[i] = silu_f32(y[i]);
+    store8(out + static_cast<long long>(t) * p.channels, y);
+  }
+}
+
+// The last taps - 1 inputs after a portion. grid (ceil(channels / 1024), seqs), 128 threads.
+template <typename T>
+__global__ void __launch_bounds__(128) short_conv_tail_kernel(const ShortConvParams p) {
+  pdl_wait();
+  pdl_trigger();
+  const int c = (blockIdx.x * 128 + threadIdx.x) * 8, seq = blockIdx.y;
+  const int slot = p.slots[seq], first = p.cu_q[seq], len = p.cu_q[seq + 1] - first;
+  if (c >= p.channels || slot < 0 || len <= 0) return;
+  const int tail = p.taps - 1;
+  const bool carried = p.positions[first] > 0;
+  T* st = static_cast<T*>(p.state) + static_cast<long long>(slot) * tail * p.channels + c;
+  const T* x = static_cast<const T*>(p.x) + c;
+  for (int j = 0; j < tail; ++j) {           // row j comes from row j + len of (old state | portion)
+    const int rel = len - tail + j;
+    float v[8];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) v[i] = 0.f;
+    if (rel >= 0) load8(x + (first + rel) * p.ldx, v);
+    else if (carried) load8(st + static_cast<long long>(rel + tail) * p.channels, v);
+    store8(st + static_cast<long long>(j) * p.channels, v);
+  }
+}
+
+// ---------------------------------------------------------------------------------------------------------
+// scan with one decay per channel and state value
+// ---------------------------------------------------------------------------------------------------------
+struct ChannelScanParams {
+  const void* x;             // [T][ldx] convolved inputs
+  const void* dt;            // [T][ld_dt] step-size logits (without bias)
+  const void* bc;            // [T][ld_bc]: B at b_off, C at c_off
+  const void* z;             // [T][ldz] gate
+  const float* dt_bias;      // [channels]
+  const float* a;            // [channels][n], -exp(A_log)
+  const float* d;            // [channels]
+  float* state;              // [slots][channels][n]
+  const int* positions;
+  const int* cu_q;           // null: one token per sequence
+  const int* slots;
+  void* y;                   // [T][ldy] gated outputs
+  long long ldx, ld_dt, ld_bc, ldz, ldy;
+  int channels, n, b_off, c_off, seqs;
+};
+
+__device__ __forceinline__ float softplus_f32(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
+
+// exp(y) for y <= 0 with a in log2 units already applied (bf16 activations), or from the plain exponent
+// with a single unbiased rounding near 1 (fp32 runs)
+template <typename T>
+struct DecayFn;
+template <>
+struct DecayFn<__nv_bfloat16> {
+  static constexpr float kPre = 1.4426950408889634f;
+  __device__ __forceinline__ static float of(float y) {
+    float r;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(y));
+    return r;
+  }
+};
+template <>
+struct DecayFn<float> {
+  static constexpr float kPre = 1.f;
+  __device__ __forceinline__ static float of(float y) { return decay_of(-y); }
+};
+
+constexpr int kCsLanes = 4;                  // lanes per channel
+constexpr int kCsChannels = 32;              // channels per block of 128 threads
+
+// grid (ceil(channels / 32), seqs), 128 threads; kPer states per lane, n = 4 kPer
+template <typename T, int kPer>
+__global__ void __launch_bounds__(128) channel_scan_kernel(const ChannelScanParams p) {
+  constexpr int N = kPer * kCsLanes;
+  constexpr int TT = N >= 128 ? 16 : 32;     // tokens per staged tile
+  constexpr int kBcVecs = (TT * 2 * N / 8 + 127) / 128;
+  __shared__ __align__(16) float s_dt[TT][kCsChannels], s_dx[TT][kCsChannels], s_e[TT][kCsChannels], s_g[TT][kCsChannels];
+  __shared__ __align__(16) float s_bc[TT][2 * N];
+  pdl_wait();
+  pdl_trigger();
+  const int seq = blockIdx.y, slot = p.slots[seq];
+  const int first = p.cu_q[seq], len = p.cu_q[seq + 1] - first;
+  if (len <= 0) return;
+  const int tid = threadIdx.x, sub = tid & 3, cl = tid >> 2;
+  const int ch0 = blockIdx.x * kCsChannels, ch = ch0 + cl;
+  const bool active = ch < p.channels;
+  const bool carried = slot >= 0 && p.positions[first] > 0;
+  float S[kPer], A[kPer];
+  float* sp = p.state + (static_cast<long long>(slot < 0 ? 0 : slot) * p.channels + ch) * N + sub * kPer;
+#pragma unroll
+  for (int i = 0; i < kPer; ++i) {
+    A[i] = active ? p.a[static_cast<long long>(ch) * N + sub * kPer + i] * DecayFn<T>::kPre : 0.f;
+    S[i] = active && carried ? sp[i] : 0.f;
+  }
+  // staging: one vector of eight channels of one token per thread, plus its share of B | C
+  const int st_t = tid >> 2, st_c = (tid & 3) * 8;
+  const bool st_on = st_t < TT && ch0 + st_c < p.channels;
+  float bias[8], dsk[8];
+#pragma unroll
+  for (int i = 0; i < 8; ++i) bias[i] = dsk[i] = 0.f;
+  if (st_on) {
+    load8(p.dt_bias + ch0 + st_c, bias);
+    load8(p.d + ch0 + st_c, dsk);
+  }
+  float rx[8], rdt[8], rz[8], rbc[kBcVecs][8];
+  auto fetch = [&](int t0) {
+    const bool on = st_on && t0 + st_t < len;
+    const long long t = first + t0 + st_t;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) rx[i] = rdt[i] = rz[i] = 0.f;
+    if (on) {
+      load8(static_cast<const T*>(p.x) + t * p.ldx + ch0 + st_c, rx);
+      load8(static_cast<const T*>(p.dt) + t * p.ld_dt + ch0 + st_c, rdt);
+      load8(static_cast<const T*>(p.z) + t * p.ldz + ch0 + st_c, rz);
+    }
+#pragma unroll
+    for (int k = 0; k < kBcVecs; ++k) {
+#pragma unroll
+      for (int i = 0; i < 8; ++i) rbc[k][i] = 0.f;
+      const int v = tid + k * 128, tt = v / (2 * N / 8), c = v % (2 * N / 8) * 8;
+      if (tt < TT && t0 + tt < len)
+        load8(static_cast<const T*>(p.bc) + (first + t0 + tt) * p.ld_bc + (c < N ? p.b_off + c : p.c_off + c - N), rbc[k]);
+    }
+  };
+  auto stage = [&](int t0) {                 // tokens past the end: dt = 0, which leaves the state as it is
+    if (st_t < TT) {
+      const bool on = st_on && t0 + st_t < len;
+      float dt[8], dx[8], e[8], g[8];
+#pragma unroll
+      for (int i = 0; i < 8; ++i) {
+        dt[i] = on ? softplus_f32(rdt[i] + bias[i]) : 0.f;
+        dx[i] = dt[i] * rx[i];
+        e[i] = dsk[i] * rx[i];
+        g[i] = silu_f32(rz[i]);
+      }
+      store8(&s_dt[st_t][st_c], dt);
+      store8(&s_dx[st_t][st_c], dx);
+      store8(&s_e[st_t][st_c], e);
+      store8(&s_g[st_t][st_c], g);
+    }
+#pragma unroll
+    for (int k = 0; k < kBcVecs; ++k) {
+      const int v = tid + k * 128, tt = v / (2 * N / 8), c = v % (2 * N / 8) * 8;
+      if (tt < TT) store8(&s_bc[tt][c], rbc[k]);
+    }
+  };
+  fetch(0);
+  for (int t0 = 0; t0 < len; t0 += TT) {
+    stage(t0);
+    __syncthreads();
+    if (t0 + TT < len) fetch(t0 + TT);
+    for (int t = 0; t < TT; t += 4) {
+      if (t0 + t >= len) break;
+      float part[4];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const float dt = s_dt[t + j][cl], dx = s_dx[t + j][cl];
+        const float* b = &s_bc[t + j][sub * kPer];
+        float acc = 0.f;
+#pragma unroll
+        for (int i = 0; i < kPer; ++i) {
+          S[i] = fmaf(DecayFn<T>::of(dt * A[i]), S[i], dx * b[i]);
+          acc = fmaf(S[i], b[N + i], acc);
+        }
+        part[j] = acc;
+      }
+      // token (sub) of the four ends up in lane sub
+      const bool hi = sub & 1, top = sub & 2;
+      float k0 = hi ? part[1] : part[0], k1 = hi ? part[3] : part[2];
+      k0 += __shfl_xor_sync(0xffffffffu, hi ? part[0] : part[1], 1);
+      k1 += __shfl_xor_sync(0xffffffffu, hi ? part[2] : part[3], 1);
+      float r = top ? k1 : k0;
+      r += __shfl_xor_sync(0xffffffffu, top ? k0 : k1, 2);
+      s_g[t + sub][cl] *= r + s_e[t + sub][cl];
+    }
+    __syncthreads();
+    if (st_on && t0 + st_t < len) {
+      float o[8];
+      load8(&s_g[st_t][st_c], o);
+      store8(static_cast<T*>(p.y) + (first + t0 + st_t) * p.ldy + ch0 + st_c, o);
+    }
+    // the next stage() writes s_g rows that only this thread has read since the barrier
+  }
+  if (active && slot >= 0)
+#pragma unroll
+    for (int i = 0; i < kPer; ++i) sp[i] = S[i];
+}
+
+// Decode: grid (ceil(channels / 64), seqs), 256 threads
+template <typename T, int kPer>
+__global__ void __launch_bounds__(256) channel_step_kernel(const ChannelScanParams p) {
+  constexpr int N = kPer * kCsLanes;
+  pdl_wait();
+  pdl_trigger();
+  const int seq = blockIdx.y, slot = p.slots[seq];
+  const int sub = threadIdx.x & 3, ch = blockIdx.x * 64 + (threadIdx.x >> 2);
+  const bool active = ch < p.channels;
+  const bool carried = slot >= 0 && p.positions[seq] > 0;
+  float* sp = p.state + (static_cast<long long>(slot < 0 ? 0 : slot) * p.channels + ch) * N + sub * kPer;
+  float acc = 0.f, x = 0.f;
+  if (active) {
+    float S[kPer];
+#pragma unroll
+    for (int i = 0; i < kPer; i += 2) {
+      const float2 v = carried ? *reinterpret_cast<const float2*>(sp + i) : make_float2(0.f, 0.f);
+      S[i] = v.x;
+      S[i + 1] = v.y;
+    }
+    x = ld1(static_cast<const T*>(p.x) + seq * p.ldx + ch);
+    const float dt = softplus_f32(ld1(static_cast<const T*>(p.dt) + seq * p.ld_dt + ch) + p.dt_bias[ch]);
+    const float dx = dt * x;
+    const T* bc = static_cast<const T*>(p.bc) + seq * p.ld_bc + sub * kPer;
+    const float* a = p.a + static_cast<long long>(ch) * N + sub * kPer;
+#pragma unroll
+    for (int i = 0; i < kPer; ++i) {
+      S[i] = fmaf(DecayFn<T>::of(dt * (a[i] * DecayFn<T>::kPre)), S[i], dx * ld1(bc + p.b_off + i));
+      acc = fmaf(S[i], ld1(bc + p.c_off + i), acc);
+    }
+    if (slot >= 0)
+#pragma unroll
+      for (int i = 0; i < kPer; i += 2) *reinterpret_cast<float2*>(sp + i) = make_float2(S[i], S[i + 1]);
+  }
+  acc += __shfl_xor_sync(0xffffffffu, acc, 1);
+  acc += __shfl_xor_sync(0xffffffffu, acc, 2);
+  if (active && sub == 0) {
+    const float z = ld1(static_cast<const T*>(p.z) + seq * p.ldz + ch);
+    static_cast<T*>(p.y)[seq * p.ldy + ch] = static_cast<T>((acc + p.d[ch] * x) * silu_f32(z));
+  }
+}
+
+// ---------------------------------------------------------------------------------------------------------
+// scan with one decay per head
+// ---------------------------------------------------------------------------------------------------------
+struct HeadScanParams {
+  const void* x;             // [T][ldx] convolved inputs: x (heads * p), B at b_off, C at c_off (groups * n each)
+  const void* dt;            // [T][ld_dt] step-size logits, one per head (without bias)
+  const float* dt_bias;      // [heads]
+  const float* rate;         // [heads] exp(A_log)
+  const float* d;            // [heads]
+  float* state;              // [slots][heads][n][p]
+  const int* positions;
+  const int* cu_q;           // null: one token per sequence
+  const int* slots;
+  void* y;                   // [T][ldy]
+  long long ldx, ld_dt, ldy;
+  int heads, groups, n, p, b_off, c_off, seqs, slices;
+};
+
+constexpr int kHsTile = 16;                  // tokens per staged tile
+
+// grid (heads * slices, seqs). n = 8 kNl; thread = (column group of 4, lane of kNl); lane l owns rows 4l..4l+3 and
+// n/2 + 4l .. n/2 + 4l + 3. Dynamic shared memory: [16][2n] B | C, [16][cols] u, [16][cols] D x -> y, [16] decays.
+template <typename T, int kNl>
+__global__ void __launch_bounds__(128) head_scan_kernel(const HeadScanParams p) {
+  constexpr int N = 8 * kNl;
+  constexpr int kBcVecs = kNl <= 8 ? kNl : kNl / 4, kXVecs = kNl >= 8 ? 1 : 8 / kNl;
+  extern __shared__ __align__(16) float sm[];
+  pdl_wait();
+  pdl_trigger();
+  const int head = blockIdx.x / p.slices, slice = blockIdx.x - head * p.slices, seq = blockIdx.y;
+  const int slot = p.slots[seq], first = p.cu_q[seq], len = p.cu_q[seq + 1] - first;
+  if (len <= 0) return;
+  const int tid = threadIdx.x, threads = blockDim.x, nl = tid % kNl, cg = tid / kNl;
+  const int cols = threads / kNl * 4, col0 = slice * cols, col = col0 + cg * 4;
+  float* s_bc = sm;
+  float* s_u = s_bc + kHsTile * 2 * N;
+  float* s_y = s_u + kHsTile * cols;
+  float* s_a = s_y + kHsTile * cols;
+  const bool active = col < p.p;
+  const bool carried = slot >= 0 && p.positions[first] > 0;
+  const int group = head / (p.heads / p.groups);
+  const float rate = p.rate[head], dt_bias = p.dt_bias[head], dsk = p.d[head];
+  float* sp = p.state + (static_cast<long long>(slot < 0 ? 0 : slot) * p.heads + head) * N * p.p + col;
+  auto row_of = [&](int r) { return (r >> 2) * (N / 2) + nl * 4 + (r & 3); };
+  f32x2 S[4][4];                             // [row pair][column]
+#pragma unroll
+  for (int r = 0; r < 4; ++r) {
+    float4 v0 = make_float4(0.f, 0.f, 0.f, 0.f), v1 = v0;
+    if (active && carried) {
+      v0 = *reinterpret_cast<const float4*>(sp + static_cast<long long>(row_of(2 * r)) * p.p);
+      v1 = *reinterpret_cast<const float4*>(sp + static_cast<long long>(row_of(2 * r + 1)) * p.p);
+    }
+    S[r][0] = pack2(v0.x, v1.x);
+    S[r][1] = pack2(v0.y, v1.y);
+    S[r][2] = pack2(v0.z, v1.z);
+    S[r][3] = pack2(v0.w, v1.w);
+  }
+  const int xv = cols / 8;                   // vectors of x per token
+  float rbc[kBcVecs][8], rx[kXVecs][8], rdt[kXVecs], rda = 0.f;
+  auto fetch = [&](int t0) {
+#pragma unroll
+    for (int k = 0; k < kBcVecs; ++k) {
+      const int v = tid + k * threads, tt = v / (2 * N / 8), c = v % (2 * N / 8) * 8;
+#pragma unroll
+      for (int i = 0; i < 8; ++i) rbc[k][i] = 0.f;
+      if (tt < kHsTile && t0 + tt < len)
+        load8(static_cast<const T*>(p.x) + (first + t0 + tt) * p.ldx + (c < N ? p.b_off + c : p.c_off + c - N) + group * N, rbc[k]);
+    }
+#pragma unroll
+    for (int k = 0; k < kXVecs; ++k) {
+      const int v = tid + k * threads, tt = v / xv, c = col0 + v % xv * 8;
+#pragma unroll
+      for (int i = 0; i < 8; ++i) rx[k][i] = 0.f;
+      rdt[k] = 0.f;
+      if (tt < kHsTile && t0 + tt < len && c < p.p) {
+        load8(static_cast<const T*>(p.x) + (first + t0 + tt) * p.ldx + head * p.p + c, rx[k]);
+        rdt[k] = ld1(static_cast<const T*>(p.dt) + (first + t0 + tt) * p.ld_dt + head);
+      }
+    }
+    if (tid < kHsTile && t0 + tid < len) rda = ld1(static_cast<const T*>(p.dt) + (first + t0 + tid) * p.ld_dt + head);
+  };
+  auto stage = [&](int t0) {                 // tokens past the end: decay 1, nothing added
+#pragma unroll
+    for (int k = 0; k < kBcVecs; ++k) {
+      const int v = tid + k * threads, tt = v / (2 * N / 8), c = v % (2 * N / 8) * 8;
+      if (tt < kHsTile) store8(s_bc + tt * 2 * N + c, rbc[k]);
+    }
+#pragma unroll
+    for (int k = 0; k < kXVecs; ++k) {
+      const int v = tid + k * threads, tt = v / xv, c = v % xv * 8;
+      if (tt < kHsTile) {
+        const float dt = softplus_f32(rdt[k] + dt_bias);
+        float u[8], e[8];
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+          u[i] = dt * rx[k][i];
+          e[i] = dsk * rx[k][i];
+        }
+        store8(s_u + tt * cols + c, u);
+        store8(s_y + tt * cols + c, e);
+      }
+    }
+    if (tid < kHsTile) s_a[tid] = t0 + tid < len ? decay_of(rate * softplus_f32(rda + dt_bias)) : 1.f;
+  };
+  fetch(0);
+  for (int t0 = 0; t0 < len; t0 += kHsTile) {
+    stage(t0);
+    __syncthreads();
+    if (t0 + kHsTile < len) fetch(t0 + kHsTile);
+    for (int t = 0; t < kHsTile; t += 4) {
+      if (t0 + t >= len) break;
+      float v[16];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const float a = s_a[t + j];
+        const f32x2 aa = pack2(a, a);
+        const float4 u = *reinterpret_cast<const float4*>(s_u + (t + j) * cols + cg * 4);
+        const float* row = s_bc + (t + j) * 2 * N + nl * 4;
+        const ulonglong2 b0 = *reinterpret_cast<const ulonglong2*>(row), b1 = *reinterpret_cast<const ulonglong2*>(row + N / 2);
+        const ulonglong2 c0 = *reinterpret_cast<const ulonglong2*>(row + N), c1 = *reinterpret_cast<const ulonglong2*>(row + N + N / 2);
+        const f32x2 bb[4] = {b0.x, b0.y, b1.x, b1.y}, cc[4] = {c0.x, c0.y, c1.x, c1.y};
+        const f32x2 uu[4] = {pack2(u.x, u.x), pack2(u.y, u.y), pack2(u.z, u.z), pack2(u.w, u.w)};
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+          f32x2 acc = pack2(0.f, 0.f);
+#pragma unroll
+          for (int r = 0; r < 4; ++r) {
+            S[r][c] = fma2(aa, S[r][c], mul2(bb[r], uu[c]));
+            acc = fma2(S[r][c], cc[r], acc);
+          }
+          v[j * 4 + c] = sum2(acc);
+        }
+      }
+      // sixteen sums (token, column) over the kNl lanes: every step halves what a lane keeps
+      int at = 0, cnt = 16;
+#pragma unroll
+      for (int m = 1; m < kNl; m *= 2) {
+        if (cnt > 1) {
+          const bool hi = nl & m;
+#pragma unroll
+          for (int i = 0; i < 8; ++i)
+            if (i < cnt / 2) {
+              const float keep = hi ? v[i + cnt / 2] : v[i], send = hi ? v[i] : v[i + cnt / 2];
+              v[i] = keep + __shfl_xor_sync(0xffffffffu, send, m);
+            }
+          cnt /= 2;
+          at += hi ? cnt : 0;
+        } else {
+          v[0] += __shfl_xor_sync(0xffffffffu, v[0], m);
+        }
+      }
+      constexpr int kKeep = kNl >= 16 ? 1 : 16 / kNl;
+      if (kNl <= 16 || nl < 16)
+#pragma unroll
+        for (int i = 0; i < kKeep; ++i) s_y[(t + ((at + i) >> 2)) * cols + cg * 4 + ((at + i) & 3)] += v[i];
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < kXVecs; ++k) {
+      const int v = tid + k * threads, tt = v / xv, c = v % xv * 8;
+      if (tt < kHsTile && t0 + tt < len && col0 + c < p.p) {
+        float o[8];
+        load8(s_y + tt * cols + c, o);
+        store8(static_cast<T*>(p.y) + (first + t0 + tt) * p.ldy + head * p.p + col0 + c, o);
+      }
+    }
+    // stage() writes the s_y vectors that this same thread has just read
+  }
+  if (active && slot >= 0)
+#pragma unroll
+    for (int r = 0; r < 4; ++r) {
+      float4 v0, v1;
+      unpack2(S[r][0], v0.x, v1.x);
+      unpack2(S[r][1], v0.y, v1.y);
+      unpack2(S[r][2], v0.z, v1.z);
+      unpack2(S[r][3], v0.w, v1.w);
+      *reinterpret_cast<float4*>(sp + static_cast<long long>(row_of(2 * r)) * p.p) = v0;
+      *reinterpret_cast<float4*>(sp + static_cast<long long>(row_of(2 * r + 1)) * p.p) = v1;
+    }
+}
+
+// Decode: grid (heads, seqs), 256 threads; thread = (4 columns, every rg-th row). Dynamic shared memory:
+// [2n] B | C, [p] x, [row groups][p] partial sums.
+template <typename T>
+__global__ void __launch_bounds__(256) head_step_kernel(const HeadScanParams p) {
+  extern __shared__ __align__(16) float sm[];
+  pdl_wait();
+  pdl_trigger();
+  const int head = blockIdx.x, seq = blockIdx.y, slot = p.slots[seq];
+  const int tid = threadIdx.x, cgs = p.p / 4, rgs = 256 / cgs, cg = tid % cgs, rg = tid / cgs;
+  const bool carried = slot >= 0 && p.positions[seq] > 0;
+  const int group = head / (p.heads / p.groups);
+  float *s_b = sm, *s_c = sm + p.n, *s_x = sm + 2 * p.n, *s_p = s_x + p.p;
+  float* sp = p.state + (static_cast<long long>(slot < 0 ? 0 : slot) * p.heads + head) * p.n * p.p + cg * 4;
+  constexpr int kRows = 8;                   // rows in flight per thread
+  float4 S[kRows];
+  auto load = [&](int n0) {
+#pragma unroll
+    for (int i = 0; i < kRows; ++i) {
+      const int n = n0 + i * rgs;
+      S[i] = rg < rgs && n < p.n && carried ? *reinterpret_cast<const float4*>(sp + static_cast<long long>(n) * p.p)
+                                            : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+  };
+  load(rg);
+  const T* xr = static_cast<const T*>(p.x) + seq * p.ldx;
+  for (int i = tid; i < 2 * p.n + p.p; i += 256)
+    sm[i] = ld1(xr + (i < p.n ? p.b_off + group * p.n + i : i < 2 * p.n ? p.c_off + group * p.n + i - p.n : head * p.p + i - 2 * p.n));
+  const float dt = softplus_f32(ld1(static_cast<const T*>(p.dt) + seq * p.ld_dt + head) + p.dt_bias[head]);
+  const float a = decay_of(p.rate[head] * dt);
+  __syncthreads();
+  if (rg < rgs) {
+    float4 u = *reinterpret_cast<const float4*>(s_x + cg * 4);
+    u.x *= dt; u.y *= dt; u.z *= dt; u.w *= dt;
+    float4 y = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int n0 = rg; n0 < p.n; n0 += kRows * rgs) {
+      if (n0 != rg) load(n0);
+#pragma unroll
+      for (int i = 0; i < kRows; ++i) {
+        const int n = n0 + i * rgs;
+        if (n < p.n) {
+          const float b = s_b[n], c = s_c[n];
+          S[i].x = fmaf(a, S[i].x, b * u.x);
+          S[i].y = fmaf(a, S[i].y, b * u.y);
+          S[i].z = fmaf(a, S[i].z, b * u.z);
+          S[i].w = fmaf(a, S[i].w, b * u.w);
+          y.x = fmaf(S[i].x, c, y.x);
+          y.y = fmaf(S[i].y, c, y.y);
+          y.z = fmaf(S[i].z, c, y.z);
+          y.w = fmaf(S[i].w, c, y.w);
+          if (slot >= 0) *reinterpret_cast<float4*>(sp + static_cast<long long>(n) * p.p) = S[i];
+        }
+      }
+    }
+    *reinterpret_cast<float4*>(s_p + rg * p.p + cg * 4) = y;
+  }
+  __syncthreads();
+  for (int c = tid; c < p.p; c += 256) {
+    float y = p.d[head] * s_x[c];
+    for (int r = 0; r < rgs; ++r) y += s_p[r * p.p + c];
+    static_cast<T*>(p.y)[seq * p.ldy + head * p.p + c] = static_cast<T>(y);
+  }
+}
+
+// ---------------------------------------------------------------------------------------------------------
+// out = norm(y silu(z)) w in `groups` equal parts of the row
+// ---------------------------------------------------------------------------------------------------------
+struct GatedNormParams {
+  const void* y;             // [T][ldy], head h at h * pp
+  const void* z;             // [T][ldz]
+  const __nv_bfloat16* w;    // [heads * pp]
+  void* out;                 // [T][ldo]
+  long long ldy, ldz, ldo;
+  int part, p, pp;           // values per part; true and laid-out head size
+  float eps;
+};
+
+// kVec: heads are laid out without gaps and parts are whole vectors; the part stays in registers.
+// grid (T, parts)
+template <typename T, bool kVec, int kIters>
+__global__ void __launch_bounds__(1024) gated_norm_kernel(const GatedNormParams p) {
+  pdl_wait();
+  pdl_trigger();
+  __shared__ float red[32];
+  const long long t = blockIdx.x;
+  const T* y = static_cast<const T*>(p.y) + t * p.ldy;
+  const T* z = static_cast<const T*>(p.z) + t * p.ldz;
+  T* out = static_cast<T*>(p.out) + t * p.ldo;
+  const int lo = blockIdx.y * p.part;
+  float q = 0.f;
+  if (kVec) {
+    float v[kIters][8];
+#pragma unroll
+    for (int k = 0; k < kIters; ++k) {
+      const int c = (threadIdx.x + k * blockDim.x) * 8;
+      float g[8];
+#pragma unroll
+      for (int i = 0; i < 8; ++i) v[k][i] = g[i] = 0.f;
+      if (c < p.part) {
+        load8(y + lo + c, v[k]);
+        load8(z + lo + c, g);
+      }
+#pragma unroll
+      for (int i = 0; i < 8; ++i) {
+        v[k][i] *= silu_f32(g[i]);
+        q = fmaf(v[k][i], v[k][i], q);
+      }
+    }
+    const float inv = 1.f / sqrtf(block_sum(q, red) / p.part + p.eps);
+#pragma unroll
+    for (int k = 0; k < kIters; ++k) {
+      const int c = (threadIdx.x + k * blockDim.x) * 8;
+      if (c < p.part) {
+        float w[8];
+        load8(p.w + lo + c, w);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) v[k][i] *= inv * w[i];
+        store8(out + lo + c, v[k]);
+      }
+    }
+    return;
+  }
+  for (int i = threadIdx.x; i < p.part; i += blockDim.x) {
+    const int at = (lo + i) / p.p * p.pp + (lo + i) % p.p;
+    const float v = ld1(y + at) * silu_f32(ld1(z + at));
+    q = fmaf(v, v, q);
+  }
+  const float inv = 1.f / sqrtf(block_sum(q, red) / p.part + p.eps);
+  for (int i = threadIdx.x; i < p.part; i += blockDim.x) {
+    const int at = (lo + i) / p.p * p.pp + (lo + i) % p.p;
+    out[at] = static_cast<T>(ld1(y + at) * silu_f32(ld1(z + at)) * inv * ld1(p.w + at));
+  }
+}
+
+template <typename T>
+int launch_short_conv(ShortConvParams p, cudaStream_t stream) {
+  const int vecs = (p.channels / 8 + 31) / 32;
+  // enough warps to cover the machine, then as many tokens per warp as that leaves
+  int run = 1;
+  if (p.cu_q) while (run < 32 && static_cast<long long>(p.tokens) * vecs / (2 * run) >= 148 * 16) run *= 2;
+  p.run = run;
+  const dim3 grid(vecs, (p.tokens + 4 * run - 1) / (4 * run));
+  if (grid.y > 65535) return -2;
+  cudaError_t e;
+  switch (p.taps) {
+    case 1: e = launch_pdl(short_conv_kernel<T, 1>, grid, dim3(128), 0, stream, p); break;
+    case 2: e = launch_pdl(short_conv_kernel<T, 2>, grid, dim3(128), 0, stream, p); break;
+    case 3: e = launch_pdl(short_conv_kernel<T, 3>, grid, dim3(128), 0, stream, p); break;
+    case 4: e = launch_pdl(short_conv_kernel<T, 4>, grid, dim3(128), 0, stream, p); break;
+    default: e = launch_pdl(short_conv_kernel<T, 0>, grid, dim3(128), 0, stream, p); break;
+  }
+  if (e == cudaSuccess && p.cu_q && p.taps > 1)
+    e = launch_pdl(short_conv_tail_kernel<T>, dim3((p.channels / 8 + 127) / 128, p.seqs), dim3(128), 0, stream, p);
+  return e == cudaSuccess ? 0 : -static_cast<int>(e) - 300;
+}
+
+template <typename T, int kPer>
+int launch_channel_scan(const ChannelScanParams& p, cudaStream_t stream) {
+  const cudaError_t e =
+      p.cu_q ? launch_pdl(channel_scan_kernel<T, kPer>, dim3((p.channels + kCsChannels - 1) / kCsChannels, p.seqs), dim3(128), 0, stream, p)
+             : launch_pdl(channel_step_kernel<T, kPer>, dim3((p.channels + 63) / 64, p.seqs), dim3(256), 0, stream, p);
+  return e == cudaSuccess ? 0 : -static_cast<int>(e) - 300;
+}
+template <typename T>
+int dispatch_channel_scan(const ChannelScanParams& p, cudaStream_t stream) {
+  switch (p.n) {
+    case 8: return launch_channel_scan<T, 2>(p, stream);
+    case 16: return launch_channel_scan<T, 4>(p, stream);
+    case 32: return launch_channel_scan<T, 8>(p, stream);
+    case 64: return launch_channel_scan<T, 16>(p, stream);
+    case 128: return launch_channel_scan<T, 32>(p, stream);
+    default: return -2;
+  }
+}
+
+template <typename T, int kNl>
+int launch_head_scan(HeadScanParams p, cudaStream_t stream) {
+  int threads = (kNl * (p.p / 4) + 31) / 32 * 32;
+  if (threads > 128) threads = 128;
+  if (kNl >= 16) threads = 128;
+  const int cols = threads / kNl * 4;
+  p.slices = (p.p + cols - 1) / cols;
+  const int smem = (kHsTile * (2 * p.n + 2 * cols) + kHsTile) * 4;
+  static PerDeviceOnce once;
+  if (once.first_time()) cudaFuncSetAttribute(head_scan_kernel<T, kNl>, cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024);
+  const cudaError_t e = launch_pdl(head_scan_kernel<T, kNl>, dim3(p.heads * p.slices, p.seqs), dim3(threads), smem, stream, p);
+  return e == cudaSuccess ? 0 : -static_cast<int>(e) - 300;
+}
+template <typename T>
+int dispatch_head_scan(const HeadScanParams& p, cudaStream_t stream) {
+  if (!p.cu_q) {
+    const int rgs = 256 / (p.p / 4);
+    const int smem = (2 * p.n + p.p + rgs * p.p) * 4;
+    const cudaError_t e = launch_pdl(head_step_kernel<T>, dim3(p.heads, p.seqs), dim3(256), smem, stream, p);
+    return e == cudaSuccess ? 0 : -static_cast<int>(e) - 300;
+  }
+  switch (p.n) {
+    case 8: return launch_head_scan<T, 1>(p, stream);
+    case 16: return launch_head_scan<T, 2>(p, stream);
+    case 32: return launch_head_scan<T, 4>(p, stream);
+    case 64: return launch_head_scan<T, 8>(p, stream);
+    case 128: return launch_head_scan<T, 16>(p, stream);
+    case 256: return launch_head_scan<T, 32>(p, stream);
+    default: return -2;
+  }
+}
+
+template <typename T>
+int launch_gated_norm(const GatedNormParams& p, int tokens, int parts, cudaStream_t stream) {
+  const bool vec = p.p == p.pp && p.part % 8 == 0;
+  const int vecs = vec ? p.part / 8 : (p.part + 3) / 4;
+  const int iters = vec && (vecs > 1024 || (vecs >= 128 && tokens >= 1024)) ? 2 : 1;
+  int threads = ((vecs + iters - 1) / iters + 31) / 32 * 32;
+  if (vec && threads > 1024) return -2;
+  if (threads > 1024) threads = 1024;
+  const dim3 grid(tokens, parts);
+  cudaError_t e;
+  if (!vec) e = launch_pdl(gated_norm_kernel<T, false, 1>, grid, dim3(threads), 0, stream, p);
+  else if (iters == 1) e = launch_pdl(gated_norm_kernel<T, true, 1>, grid, dim3(threads), 0, stream, p);
+  else e = launch_pdl(gated_norm_kernel<T, true, 2>, grid, dim3(threads), 0, stream, p);
+  return e == cudaSuccess ? 0 : -static_cast<int>(e) - 300;
+}
+
 }  // namespace b200
 
 using namespace b200;
@@ -85,4 +833,49 @@ B200_API int b200_selective_scan(const void* x, const float* dt, const float* a,
                static_cast<const __nv_bfloat16*>(c), d, state, static_cast<__nv_bfloat16*>(y), tokens, channels, n};
   selective_scan_kernel<<<(channels + 127) / 128, 128, 0, stream>>>(p);
   return cudaGetLastError() == cudaSuccess ? 0 : -300;
+}
+
+// x [tokens][ldx] -> out [tokens][channels] (see short_conv_kernel); channels and ldx multiples of 8
+B200_API int b200_short_conv(const void* x, const float* w, const float* bias, void* state, const int* positions,
+                             const int* cu_q, const int* slots, void* out, int tokens, int seqs, int channels, int taps,
+                             long long ldx, int f32, cudaStream_t stream) {
+  if (tokens <= 0 || seqs <= 0) return 0;
+  if (channels % 8 || ldx % 8 || taps < 1 || seqs > 65535 || (!cu_q && seqs != tokens)) return -2;
+  ShortConvParams p{x, w, bias, state, positions, cu_q, slots, out, ldx, tokens, seqs, channels, taps, 1};
+  return f32 ? launch_short_conv<float>(p, stream) : launch_short_conv<__nv_bfloat16>(p, stream);
+}
+
+// n in {8, 16, 32, 64, 128}; channels, offsets and row pitches multiples of 8
+B200_API int b200_channel_scan(const void* x, const void* dt, const void* bc, const void* z, const float* dt_bias, const float* a,
+                               const float* d, float* state, const int* positions, const int* cu_q, const int* slots, void* y,
+                               int seqs, int channels, int n, int b_off, int c_off, long long ldx, long long ld_dt,
+                               long long ld_bc, long long ldz, long long ldy, int f32, cudaStream_t stream) {
+  if (seqs <= 0) return 0;
+  if (channels % 8 || b_off % 8 || c_off % 8 || ldx % 8 || ld_dt % 8 || ld_bc % 8 || ldz % 8 || ldy % 8 || seqs > 65535) return -2;
+  ChannelScanParams p{x, dt, bc, z, dt_bias, a, d, state, positions, cu_q, slots, y, ldx, ld_dt, ld_bc, ldz, ldy,
+                      channels, n, b_off, c_off, seqs};
+  return f32 ? dispatch_channel_scan<float>(p, stream) : dispatch_channel_scan<__nv_bfloat16>(p, stream);
+}
+
+// n in {8, 16, ..., 256}, hp (values per head) a multiple of 8 up to 512; offsets and row pitches (but ld_dt)
+// multiples of 8
+B200_API int b200_head_scan(const void* x, const void* dt, const float* dt_bias, const float* rate, const float* d, float* state,
+                            const int* positions, const int* cu_q, const int* slots, void* y, int seqs, int heads, int groups,
+                            int n, int hp, int b_off, int c_off, long long ldx, long long ld_dt, long long ldy, int f32,
+                            cudaStream_t stream) {
+  if (seqs <= 0) return 0;
+  if (hp % 8 || hp > 512 || n % 8 || n > 256 || heads % groups || b_off % 8 || c_off % 8 || ldx % 8 || ldy % 8 || seqs > 65535)
+    return -2;
+  HeadScanParams p{x, dt, dt_bias, rate, d, state, positions, cu_q, slots, y, ldx, ld_dt, ldy, heads, groups, n, hp, b_off,
+                   c_off, seqs, 1};
+  return f32 ? dispatch_head_scan<float>(p, stream) : dispatch_head_scan<__nv_bfloat16>(p, stream);
+}
+
+// y, z, out [tokens][...] with heads of hp values laid out hpp apart; parts * part = heads * hp
+B200_API int b200_gated_norm(const void* y, const void* z, const void* w, void* out, int tokens, int parts, int part, int hp,
+                             int hpp, long long ldy, long long ldz, long long ldo, float eps, int f32, cudaStream_t stream) {
+  if (tokens <= 0 || parts <= 0) return 0;
+  if (part < 1 || hp < 1 || hpp < hp || ldy % 8 || ldz % 8 || ldo % 8 || parts > 65535) return -2;
+  GatedNormParams p{y, z, static_cast<const __nv_bfloat16*>(w), out, ldy, ldz, ldo, part, hp, hpp, eps};
+  return f32 ? launch_gated_norm<float>(p, tokens, parts, stream) : launch_gated_norm<__nv_bfloat16>(p, tokens, parts, stream);
 }

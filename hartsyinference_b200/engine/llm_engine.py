@@ -265,6 +265,7 @@ class LLMEngine:
                              cu_q=self._to_device(self.h_cu_q, n + 1), max_q_len=max_q, max_kv_len=max_kv,
                              embeds=embeds, cross_states=self._cross_states([self.requests[rid] for rid, _, _ in chunks]),
                              positions3=self._positions3(chunks), deepstack=self._deepstack(chunks, t),
+                             runs=[(count, start + count) for _, start, count in chunks],
                              state_slots=self._to_device(self.h_state, n) if self.kv.state_slots else None)
         return self.model.forward_hidden(batch), ends
 

@@ -574,7 +574,7 @@ class TextService:
                                  slot_mapping=torch.arange(n, dtype=torch.int64, device=dev),
                                  block_table=torch.arange(max(pages, 1), dtype=torch.int32, device=dev)[None],
                                  kv_lens=torch.tensor([n], dtype=torch.int32, device=dev), is_decode=False,
-                                 cu_q=torch.tensor([0, n], dtype=torch.int32, device=dev), max_q_len=n, max_kv_len=n,
+                                 cu_q=torch.tensor([0, n], dtype=torch.int32, device=dev), max_q_len=n, max_kv_len=n, runs=[(n, n)],
                                  state_slots=torch.zeros(1, dtype=torch.int32, device=dev) if recurrent else None)
                 hid = m.forward_hidden(b)[:, :m.cfg.hidden_size].float().mean(0)
                 m.kv_cache = saved

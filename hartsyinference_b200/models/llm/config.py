@@ -51,7 +51,7 @@ class MlaConfig:
 @dataclass(frozen=True)
 class MixerSpec:
     """Token mixer of one layer of a model whose layers differ (``TransformerConfig.layer_specs``)."""
-    kind: str = "attention"             # attention | channel_delta
+    kind: str = "attention"             # attention | channel_delta | latent_attention | channel_scan | head_scan
     heads: int = 1
     kv_heads: int = 1
     dim: int = 64                       # query / key size per head
@@ -66,15 +66,36 @@ class MixerSpec:
     qk_bias: bool = False
     out_gate: bool = False              # output * sigmoid(W_g h)
     sink: Optional[float] = None        # score of a key without a value
-    # channel_delta
+    # latent_attention (dim / vdim: query-key and value size per head, out_gate as above)
+    q_rank: int = 0                     # size of the query latent
+    kv_rank: int = 0                    # size of the cached key / value latent
+    # recurrent kinds
     conv: int = 0                       # taps of the short convolution
-    rank: int = 0                       # low-rank size of decay and gate in synthetic weights (0 = dim)
+    rank: int = 0                       # low-rank size: channel_delta decay and gate in synthetic weights (0 = dim); channel_scan step size
+    state: int = 0                      # channel_scan: state values per channel; head_scan: state rows per head (columns: vdim)
+    inner: int = 0                      # channel_scan: channels
+    groups: int = 1                     # head_scan: groups of heads that share B and C
+    norm_groups: int = 1                # head_scan: equal parts of the gated output norm
+
+    @property
+    def recurrent(self) -> bool:
+        """The mixer carries a state: its sequences need a slot."""
+        return self.kind in ("channel_delta", "channel_scan", "head_scan")
+
+
+@dataclass(frozen=True)
+class DenseSpec:
+    """Ungated dense feed-forward of one layer: down(act(up h))."""
+    ffn: int
+    act: str = "poly_norm"
 
 
 @dataclass(frozen=True)
 class LayerSpec:
     mixer: MixerSpec
-    moe: Optional[MoeConfig] = None     # None: no feed-forward in this layer
+    moe: Optional[MoeConfig] = None     # routed experts
+    dense: Optional[DenseSpec] = None   # or a dense feed-forward; neither: no feed-forward in this layer
+    weights_of: Optional[int] = None    # index of the layer whose weights this one uses (its cache and state are its own)
 
 
 @dataclass(frozen=True)
@@ -175,7 +196,7 @@ class TransformerConfig:
     @property
     def recurrent(self) -> bool:
         """True when some layer is recurrent: its sequences need a state slot."""
-        return any(ls.mixer.kind == "channel_delta" for ls in self.layer_specs)
+        return any(ls.mixer.recurrent for ls in self.layer_specs)
 
     @property
     def general_path(self) -> bool:
@@ -210,7 +231,8 @@ class TransformerConfig:
         h, l = self.hidden_size, self.num_layers
         if self.layer_specs:
             from .mixers import spec_param_count
-            return sum(spec_param_count(ls, h) for ls in self.layer_specs) + 2 * self.vocab_size * h + h
+            own = sum(spec_param_count(ls, h) for ls in self.layer_specs if ls.weights_of is None)
+            return own + (1 if self.tie_embeddings else 2) * self.vocab_size * h + h
         attn = h * (self.q_size + 2 * self.kv_size) + self.q_size * h
         if self.mla is not None:
             m = self.mla
@@ -281,13 +303,23 @@ def tiny(base: str = "qwen2.5-0.5b", **over: Any) -> TransformerConfig:
     return replace(cfg, **small)
 
 
+# designs whose layers are described one by one; each is a module of this package with ``config_from``,
+# ``load_layers``, ``tensor_shapes`` and ``random_tensor``
+MIXED_DESIGNS = ("lududra", "salopel")
+
+
+def mixed_design(arch: str):
+    import importlib
+    return importlib.import_module(f"{__package__}.{arch}")
+
+
 def from_hf_config(d: dict) -> TransformerConfig:
     """Map a Hugging Face ``config.json`` (llama / mistral / qwen2 / qwen3 / gemma 1-3 / granite / olmo2 /
     phi3 / glm / glm4 / starcoder2 / stablelm / cohere / cohere2 / nemotron / gpt_neox / gpt2 / granitemoe / mllama (text) / qwen2_vl - qwen2_5_vl - qwen3_vl (text) / hunyuan_v1_dense / apertus / bloom / gpt_oss / gptj / opt / phi / olmo3 / exaone4 / helium / ernie4_5 / arcee / smollm3 / ministral / seed_oss / minicpm / internlm2 / deepseek_v2-v3 / glm4_moe / dots1 / ernie4_5_moe / hunyuan_v1_moe / cwm / gpt_bigcode / falcon / mixtral /
-    olmoe / qwen2_moe / qwen3_moe families, and lududra) onto :class:`TransformerConfig`."""
-    if str(d.get("architecture", "")).lower() == "lududra":
-        from .lududra import lududra_config
-        return lududra_config(d)
+    olmoe / qwen2_moe / qwen3_moe families, and the designs of :data:`MIXED_DESIGNS`) onto :class:`TransformerConfig`."""
+    name = str(d.get("architecture", "")).lower()
+    if name in MIXED_DESIGNS:
+        return mixed_design(name).config_from(d)
     mt = d.get("model_type", "llama")
     if mt == "opt":
         d = {**d, "intermediate_size": d.get("ffn_dim") or 4 * d["hidden_size"], "hidden_act": d.get("activation_function", "relu"),

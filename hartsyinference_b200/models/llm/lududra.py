@@ -59,6 +59,9 @@ def lududra_config(d: dict) -> TransformerConfig:
                              bos_token_id=int(d.get("bos_token_id") or 0), eos_token_ids=eos)
 
 
+config_from = lududra_config
+
+
 def load_layers(model, need: Callable[[str], torch.Tensor]) -> None:
     """Checkpoint tensors (``embed``, ``l<i>.norm1``, ``l<i>.mix.*``, ``l<i>.mlp.*``, ``final.norm``, ``head``)
     -> the decoder's layers. ``need(name)`` returns a tensor on any device."""

@@ -18,7 +18,7 @@ import torch
 
 from ... import ops
 from ...ops import LinearWeight
-from .config import LayerSpec, MixerSpec, MoeConfig
+from .config import DenseSpec, LayerSpec, MixerSpec, MoeConfig
 
 
 def pad_to(n: int, m: int) -> int:
@@ -161,6 +161,226 @@ class DeltaMixer:
         return ops.linear_act(y, self.o)
 
 
+class ChannelScanMixer:
+    """Selective scan (one decay per channel and state value): projection, short convolution, a second projection
+    of the convolved inputs for step size, B and C, scan with the output gate in its epilogue."""
+
+    def __init__(self, spec: MixerSpec, width: int, device, *, w_in, conv, conv_bias, x, dt, dt_bias, a_log, d, o):
+        self.spec = spec
+        c, n, r = spec.inner, spec.state, spec.rank
+        self.n = next((s for s in (8, 16, 32, 64, 128) if s >= n), 0)
+        if not self.n:
+            raise ValueError(f"channel_scan with {n} state values per channel is not supported (at most 128)")
+        cp, wp, self.rp = pad_to(c, 8), pad_to(width, 8), pad_to(r, 8)
+        self.c = cp
+        f32 = lambda t: t.float().to(device).contiguous()
+        self.proj = _linear([pad_cols(pad_head_rows(w_in, 2, c, cp), wp)], device)
+        self.low = _linear([pad_cols(pad_rows(p, k), cp) for p, k in ((x[:r], self.rp), (x[r:r + n], self.n), (x[r + n:], self.n))], device)
+        self.dt = _linear([pad_cols(pad_rows(dt, cp), self.rp)], device)
+        self.o = _linear([pad_rows(pad_cols(o, cp), wp)], device)
+        self.conv, self.conv_bias = f32(pad_rows(conv, cp).t()), f32(pad_rows(conv_bias, cp))
+        a = torch.zeros(cp, self.n, device=device)
+        a[:c, :n] = -torch.exp(a_log.float().to(device))
+        self.w = ops.ChannelScanWeights(a=a, dt_bias=f32(pad_rows(dt_bias, cp)), d=f32(pad_rows(d, cp)))
+
+    def nbytes(self) -> int:
+        return sum(w.nbytes() for w in (self.proj, self.low, self.dt, self.o))
+
+    def state_shapes(self, slots: int) -> tuple[tuple, tuple]:
+        return (slots, self.conv.shape[0] - 1, self.c), (slots, self.c, self.n)
+
+    def __call__(self, h: torch.Tensor, batch, li: int, model) -> torch.Tensor:
+        p = ops.linear_act(h, self.proj)
+        conv, state = model.mixer_state[li]
+        cu = None if batch.is_decode else batch.cu_q
+        x = ops.short_conv(p[:, :self.c], self.conv, self.conv_bias, conv, batch.positions, cu, batch.state_slots)
+        low = ops.linear_act(x, self.low)
+        dt = ops.linear_act(low[:, :self.rp], self.dt)
+        y = ops.channel_scan(x, dt, low, self.rp, self.rp + self.n, p[:, self.c:], self.w, state, batch.positions, cu, batch.state_slots)
+        return ops.linear_act(y, self.o)
+
+
+class HeadScanMixer:
+    """State-space mixer with one decay per head and a matrix state: projection (z | x | B | C | step size), short
+    convolution over x | B | C, scan, gate, RMS norm in equal parts."""
+
+    def __init__(self, spec: MixerSpec, width: int, eps: float, device, *, w_in, conv, conv_bias, dt_bias, a_log, d, norm, o):
+        self.spec, self.eps = spec, eps
+        h, v, n, g = spec.heads, spec.vdim, spec.state, spec.groups
+        np_ = next((s for s in (8, 16, 32, 64, 128, 256) if s >= n), 0)
+        vp, wp = pad_to(v, 8), pad_to(width, 8)
+        if not np_ or vp > 512:
+            raise ValueError(f"head_scan states of {n} x {v} are not supported (at most 256 x 512)")
+        if h % g or h * v % spec.norm_groups:
+            raise ValueError(f"head_scan: {h} heads do not divide over {g} groups, or {h * v} channels over {spec.norm_groups} norm groups")
+        f32 = lambda t: t.float().to(device).contiguous()
+        inner, gn = h * v, g * n
+        z, x, b, c, dt = w_in.split([inner, inner, gn, gn, h])
+        head, grp = (lambda t: pad_head_rows(t, h, v, vp)), (lambda t: pad_head_rows(t, g, n, np_))
+        self.proj = _linear([pad_cols(p, wp) for p in (head(z), head(x), grp(b), grp(c), pad_rows(dt, pad_to(h, 8)))], device)
+        self.inner, self.channels = h * vp, h * vp + 2 * g * np_
+        xbc = lambda t: torch.cat([head(t[:inner]), grp(t[inner:inner + gn]), grp(t[inner + gn:])])
+        self.conv, self.conv_bias = f32(xbc(conv).t()), f32(xbc(conv_bias))
+        self.norm = head(norm).to(torch.bfloat16).to(device).contiguous()
+        self.o = _linear([pad_rows(pad_head_cols(o, h, v, vp), wp)], device)
+        self.w = ops.HeadScanWeights(rate=f32(a_log.float().exp()), dt_bias=f32(dt_bias), d=f32(d), heads=h, groups=g, n=np_, p=vp)
+
+    def nbytes(self) -> int:
+        return self.proj.nbytes() + self.o.nbytes()
+
+    def state_shapes(self, slots: int) -> tuple[tuple, tuple]:
+        return (slots, self.conv.shape[0] - 1, self.channels), (slots, self.w.heads, self.w.n, self.w.p)
+
+    def __call__(self, h: torch.Tensor, batch, li: int, model) -> torch.Tensor:
+        p = ops.linear_act(h, self.proj)
+        conv, state = model.mixer_state[li]
+        cu = None if batch.is_decode else batch.cu_q
+        i, s = self.inner, self.spec
+        x = ops.short_conv(p[:, i:i + self.channels], self.conv, self.conv_bias, conv, batch.positions, cu, batch.state_slots)
+        y = ops.head_scan(x, p[:, i + self.channels:i + self.channels + s.heads], self.w, state, batch.positions, cu, batch.state_slots)
+        y = ops.gated_norm(y, p[:, :i], self.norm, s.norm_groups, self.eps, s.heads, s.vdim)
+        return ops.linear_act(y, self.o)
+
+
+# ragged batches: runs of at least this many query tokens expand keys and values of their context once; shorter
+# ones attend in latent space
+_EXPAND_RUN = 48
+# most context tokens whose keys and values are held at once
+_EXPAND_TOKENS = 65536
+
+
+class LatentPlan:
+    """How a ragged batch is split for latent attention: groups of long runs, and the rows of the short ones.
+    The index arrays go to the device in one copy."""
+
+    def __init__(self, batch, expand: bool):
+        runs = batch.runs
+        if runs is None:
+            cu, kv = batch.cu_q.tolist(), batch.kv_lens.tolist()
+            runs = [(b - a, n) for a, b, n in zip(cu, cu[1:], kv)]
+        starts, t = [], 0
+        for q, _ in runs:
+            starts.append(t)
+            t += q
+        long = [i for i, (q, _) in enumerate(runs) if expand and q >= _EXPAND_RUN]
+        groups: list[list[int]] = []
+        for i in long:
+            if not groups or sum(runs[j][1] for j in groups[-1]) + runs[i][1] > _EXPAND_TOKENS:
+                groups.append([])
+            groups[-1].append(i)
+        flat: list[int] = []
+
+        def put(values) -> slice:
+            a = len(flat)
+            flat.extend(values)
+            flat.extend([0] * (-len(flat) % 4))          # every array starts on 16 bytes
+            return slice(a, a + len(values))
+
+        rows: list[tuple[int, int, int]] = []
+        skip = set(long)
+        for i, (q, kv) in enumerate(runs):
+            if i not in skip:
+                rows += [(starts[i] + j, i, kv - q + j + 1) for j in range(q)]
+        at = []
+        for g in groups:
+            off = [0]
+            for i in g:
+                off.append(off[-1] + runs[i][1])
+            at.append((put(g), put(off), put([starts[i] for i in g]), put([runs[i][0] for i in g]), put([runs[i][1] for i in g])))
+        r = [put([x[k] for x in rows]) for k in range(3)]
+        dev = torch.tensor(flat, dtype=torch.int32).to(batch.tokens.device)
+        self.groups = [dict(seqs=dev[a], offsets=dev[b], q_start=dev[c], q_lens=dev[d], kv_lens=dev[e],
+                            total=sum(runs[i][1] for i in g), max_kv=max(runs[i][1] for i in g), max_q=max(runs[i][0] for i in g))
+                       for g, (a, b, c, d, e) in zip(groups, at)]
+        # rows None: every row of the batch, in order
+        self.short = len(rows)
+        self.rows = dev[r[0]] if groups else None
+        self.row_seq, self.row_len = dev[r[1]], dev[r[2]]
+
+
+class LatentAttention:
+    """Attention whose keys and values are per-head maps of one cached latent; queries through a latent of their
+    own, sigmoid output gate, no positions. One projection GEMM (query latent | latent | gate)."""
+
+    def __init__(self, spec: MixerSpec, width: int, eps: float, device, *, dq, dq_norm, uq, dkv, dkv_norm, uk, uv, g, o):
+        self.spec, self.eps = spec, eps
+        h, d, v = spec.heads, spec.dim, spec.vdim
+        if spec.kv_rank > 512:
+            raise ValueError(f"latent_attention with a latent of {spec.kv_rank} values is not supported (at most 512)")
+        wp = pad_to(width, 8)
+        self.d, self.v = dp, vp = pad_to(d, 8), pad_to(v, 8)
+        self.qr, self.r = qr, r = pad_to(spec.q_rank, 8), pad_to(spec.kv_rank, 8)
+        head = lambda t, k, kp: pad_head_rows(t, h, k, kp)
+        self.proj = _linear([pad_cols(p, wp) for p in (pad_rows(dq, qr), pad_rows(dkv, r), head(g, v, vp))], device)
+        vec = lambda t, n: pad_rows(t, n).to(torch.bfloat16).to(device).contiguous()
+        self.q_norm, self.kv_norm = vec(dq_norm, qr), vec(dkv_norm, r)
+        self.uq = _linear([pad_cols(head(uq, d, dp), qr)], device)
+        uk, uv = pad_cols(head(uk, d, dp), r), pad_cols(head(uv, v, vp), r)
+        self.kv_up = _linear([uk, uv], device)
+        self.uv = LinearWeight(self.kv_up.weight[h * dp:])
+        self.uk_t = _linear([uk.reshape(h, dp, r).transpose(1, 2).reshape(h * r, dp)], device)     # the query's side of W_uk
+        self.o = _linear([pad_rows(pad_head_cols(o, h, v, vp), wp)], device)
+        self.scale = spec.scale or d ** -0.5
+
+    def nbytes(self) -> int:
+        return sum(w.nbytes() for w in (self.proj, self.uq, self.kv_up, self.uk_t, self.o))
+
+    def cache_shape(self, pages: int, page: int) -> tuple:
+        return (1, pages, 1, page, self.r)
+
+    def _plan(self, batch, h: torch.Tensor) -> LatentPlan:
+        expand = h.is_cuda and h.dtype == torch.bfloat16 and max(self.d, self.v) <= 128
+        if batch.plan is None:
+            batch.plan = {}
+        if expand not in batch.plan:
+            batch.plan[expand] = LatentPlan(batch, expand)
+        return batch.plan[expand]
+
+    def __call__(self, h: torch.Tensor, batch, li: int, model) -> torch.Tensor:
+        heads = self.spec.heads
+        p = ops.linear_act(h, self.proj)
+        gate = p[:, self.qr + self.r:]
+        cache = model.kv_cache[li][0]
+        cq = ops.latent_prep(p, 0, self.spec.q_rank, self.q_norm, self.qr, self.spec.kv_rank, self.kv_norm, cache, batch.slot_mapping, self.eps)
+        q = ops.linear_act(cq, self.uq)
+        if batch.is_decode:
+            a = ops.latent_attn(ops.head_linear(q, self.uk_t, heads), cache, batch.block_table, batch.kv_lens, heads, self.scale,
+                                max_kv_len=batch.max_kv_len)
+            return ops.linear_act(ops.head_linear(a, self.uv, heads, gate=gate), self.o)
+        plan = self._plan(batch, h)
+        y = torch.empty(h.shape[0], heads * self.v, dtype=h.dtype, device=h.device)
+        for g in plan.groups:
+            c = ops.latent_gather(cache, batch.block_table, g["seqs"], g["offsets"], g["total"], g["max_kv"])
+            kv = ops.linear_act(c, self.kv_up)
+            ops.attn_runs(q, kv[:, :heads * self.d], kv[:, heads * self.d:], y, g["q_start"], g["q_lens"], g["offsets"], g["kv_lens"],
+                          heads=heads, max_q_len=g["max_q"], scale=self.scale, gate=gate)
+        if plan.short:
+            ql = ops.head_linear(q, self.uk_t, heads, in_rows=plan.rows)
+            a = ops.latent_attn(ql, cache, batch.block_table, plan.row_len, heads, self.scale, row_seq=plan.row_seq,
+                                max_kv_len=batch.max_kv_len)
+            ops.head_linear(a, self.uv, heads, gate=gate, out=y, out_rows=plan.rows)
+        return ops.linear_act(y, self.o)
+
+
+class DenseFeedForward:
+    """Ungated feed-forward ``down(act(up h))``; ``coef``: the activation's numbers."""
+
+    def __init__(self, spec: DenseSpec, width: int, eps: float, device, *, up, down, coef):
+        if spec.act != "poly_norm":
+            raise ValueError(f"unknown activation '{spec.act}'")
+        self.spec, self.eps = spec, eps
+        fp, wp = pad_to(spec.ffn, 8), pad_to(width, 8)
+        self.up = _linear([pad_rows(pad_cols(up, wp), fp)], device)
+        self.down = _linear([pad_rows(pad_cols(down, fp), wp)], device)
+        self.coef = coef.float().to(device).contiguous()
+
+    def nbytes(self) -> int:
+        return self.up.nbytes() + self.down.nbytes()
+
+    def __call__(self, h: torch.Tensor, model=None) -> torch.Tensor:
+        return ops.linear_act(ops.poly_norm(ops.linear_act(h, self.up), self.coef, self.spec.ffn, self.eps), self.down)
+
+
 def build_experts(moe: MoeConfig, width: int, device, router: torch.Tensor, correction: Optional[torch.Tensor], experts):
     """Stacked expert weights for the grouped GEMMs: per expert gate | up [2F, W] and down [W, F] with F padded
     to 64 and W (as output) to 128. ``experts`` yields (gate, up, down)."""
@@ -179,11 +399,19 @@ def build_experts(moe: MoeConfig, width: int, device, router: torch.Tensor, corr
 
 def spec_param_count(ls: LayerSpec, width: int) -> int:
     m = ls.mixer
-    if m.kind == "attention":
+    if m.kind == "latent_attention":
+        n = width * (m.q_rank + m.kv_rank + 2 * m.heads * m.vdim) + m.heads * (m.q_rank * m.dim + m.kv_rank * (m.dim + m.vdim))
+    elif m.kind == "channel_scan":
+        n = m.inner * (3 * width + 2 * m.rank + 3 * m.state + m.conv)
+    elif m.kind == "head_scan":
+        n = width * (3 * m.heads * m.vdim + 2 * m.groups * m.state + m.heads) + m.conv * (m.heads * m.vdim + 2 * m.groups * m.state)
+    elif m.kind == "attention":
         n = width * m.dim * (m.heads * (2 + m.out_gate) + m.kv_heads * (1 if m.shared_kv else 2))
     else:
         r = m.rank or m.dim
         n = width * (2 * m.kv_heads * m.dim + 2 * m.heads * m.vdim + m.heads + 2 * r) + r * m.heads * (m.dim + m.vdim)
     if ls.moe is not None:
         n += 3 * width * ls.moe.expert_ffn * ls.moe.num_experts + width * ls.moe.choices
+    if ls.dense is not None:
+        n += 2 * width * ls.dense.ffn
     return n + 4 * width

@@ -28,7 +28,7 @@ import torch
 from ... import config, ops
 from ...ops import LinearWeight
 from ...parallel.comm import Comm, SingleComm
-from .config import RopeScaling, TransformerConfig
+from .config import RopeScaling, TransformerConfig, mixed_design
 
 
 @dataclass
@@ -51,6 +51,8 @@ class ForwardBatch:
                                                     # with one entry (tensor or None) per sequence
     cross_row_mask: Optional[torch.Tensor] = None   # Mllama: [T], 0 for text rows that precede every image
     state_slots: Optional[torch.Tensor] = None      # [S] int32 recurrent-state slot of every sequence (-1: none)
+    runs: Optional[list] = None                     # ragged batch, host copy: (query tokens, keys) of every sequence
+    plan: Optional[object] = None                   # what a mixer works out once per batch for all its layers
 
 
 def build_inv_freq(rot: int, theta: float, scaling: RopeScaling, device) -> tuple[torch.Tensor, float]:
@@ -208,8 +210,7 @@ class DecoderModel:
             return t
 
         if cfg.mixed_layers:
-            from .lududra import load_layers
-            load_layers(self, need)
+            mixed_design(cfg.arch).load_layers(self, need)
             return
         emb = need("model.embed_tokens.weight")
         self.embed = emb.to(dt).to(self.device)
@@ -420,10 +421,10 @@ class DecoderModel:
         with constant block scales that reproduce the same distribution."""
         cfg, d, dev = self.cfg, self.cfg.head_dim, self.device
         if cfg.mixed_layers:
-            from .lududra import load_layers, random_tensor, tensor_shapes
-            shapes = tensor_shapes(cfg)
+            design = mixed_design(cfg.arch)
+            shapes = design.tensor_shapes(cfg)
             order = {n: i for i, n in enumerate(shapes)}
-            load_layers(self, lambda n: random_tensor(n, shapes[n], dev, seed * 1000003 + 11 * order[n] + 1, std))
+            design.load_layers(self, lambda n: design.random_tensor(n, shapes[n], dev, seed * 1000003 + 11 * order[n] + 1, std))
             return
         counter = [seed * 1000003 + self.tp_rank * 7919]
 
@@ -585,7 +586,7 @@ class DecoderModel:
         n = self.embed.numel() * 2 + self.final_norm.numel() * 2
         if self.lm_head.weight.data_ptr() != self.embed.data_ptr():
             n += self.lm_head.nbytes()
-        for lw in self.layers:
+        for lw in {id(lw): lw for lw in self.layers}.values():      # layers can share weights
             for w in (lw.qkv, lw.o, lw.gate_up, lw.down):
                 if w is not None:
                     n += w.nbytes()
@@ -867,21 +868,34 @@ class DecoderModel:
             mixer -> x += norm1b(y), h = norm2(x)                          [one launch]
             experts -> x += norm2b(sum of expert rows), h = norm1'(x)      [one launch]
 
-        ``capture`` (a list) receives a copy of the stream after every layer."""
+        Without norms ahead of the sublayers (``pre_norm`` off) h is x itself in the activation type. ``capture`` (a list) receives a copy of the stream after every layer."""
         cfg = self.cfg
-        kw = dict(dim=cfg.hidden_size, eps=cfg.rms_eps, layernorm=cfg.norm_type == "layernorm", dtype=self.dtype)
-        if batch.embeds is not None:
+        kw = dict(dim=cfg.hidden_size, eps=cfg.rms_eps, layernorm=cfg.norm_type == "layernorm", dtype=self.dtype,
+                  plus_one=cfg.norm_plus_one, mult=cfg.residual_multiplier, plain=not cfg.pre_norm)
+        if self.embed_norm_w is not None:
+            ids, table = batch.tokens, self.embed
+            if batch.embeds is not None:
+                e = batch.embeds.to(table.dtype)
+                ids, table = None, torch.nn.functional.pad(e, (0, table.shape[1] - e.shape[1]))
+            scale = 1.0 if ids is None else cfg.embed_scale * cfg.embedding_multiplier
+            x, h = ops.embedding_norm(ids, table, self.embed_norm_w, dim=cfg.hidden_size, eps=cfg.rms_eps, layernorm=kw["layernorm"],
+                                      plus_one=cfg.norm_plus_one, scale=scale, dtype=self.dtype)
+        elif batch.embeds is not None:
             x = torch.nn.functional.pad(batch.embeds.float(), (0, self.embed.shape[1] - batch.embeds.shape[1])).contiguous()
         else:
             x = ops.embedding_f32(batch.tokens, self.embed, cfg.embed_scale * cfg.embedding_multiplier, cfg.hidden_size)
-        h = ops.residual_norm(x, None, None, self.layers[0].in_norm if self.layers else self.final_norm, **kw)
+        first = self.layers[0].in_norm if self.layers else self.final_norm
+        if first is not None or self.embed_norm_w is None:
+            h = ops.residual_norm(x, None, None, first, **kw)
         last = len(self.layers) - 1
         for li, lw in enumerate(self.layers):
             after = self.final_norm if li == last else self.layers[li + 1].in_norm
             y = lw.attn_module(h, batch, li, self)
             h = ops.residual_norm(x, y, lw.post_attn_norm, lw.post_norm if lw.ffn_module is not None else after, **kw)
-            if lw.ffn_module is not None:
+            if hasattr(lw.ffn_module, "routed_rows"):
                 h = self._routed_sublayer(lw, x, h, after, kw)
+            elif lw.ffn_module is not None:
+                h = ops.residual_norm(x, lw.ffn_module(h), lw.post_ffn_norm, after, **kw)
             if capture is not None:
                 capture.append(x[:, :cfg.hidden_size].clone())
         return h

@@ -52,17 +52,30 @@ from .core import (  # noqa: F401
     selective_scan,
 )
 from .mixers import (  # noqa: F401
+    ChannelScanWeights,
     DeltaWeights,
+    HeadScanWeights,
     RoutedRows,
     attn_biased,
+    attn_runs,
+    channel_scan,
     delta_mix,
     embedding_f32,
+    embedding_norm,
+    gated_norm,
     glu_clamped,
+    head_linear,
+    head_scan,
     kv_store,
+    latent_attn,
+    latent_gather,
+    latent_prep,
     linear_act,
     pair_linear_f32,
+    poly_norm,
     residual_norm,
     router,
+    short_conv,
 )
 from . import reference  # noqa: F401
 
@@ -87,7 +100,9 @@ def _install_ranges() -> None:
         setattr(core, name, wrapped)          # internal calls (core.linear -> core.gguf_linear) are traced too
         if hasattr(mod, name):
             setattr(mod, name, wrapped)
-    for name in ("attn_biased", "delta_mix", "embedding_f32", "glu_clamped", "kv_store", "pair_linear_f32", "residual_norm", "router"):
+    for name in ("attn_biased", "attn_runs", "channel_scan", "delta_mix", "embedding_f32", "embedding_norm", "gated_norm", "glu_clamped",
+                 "head_linear", "head_scan", "kv_store", "latent_attn", "latent_gather", "latent_prep", "pair_linear_f32", "poly_norm",
+                 "residual_norm", "router", "short_conv"):
         setattr(mod, name, traced(name)(getattr(mixers, name)))
 
 

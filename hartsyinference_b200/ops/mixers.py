@@ -1,5 +1,5 @@
 """Ops of layers around a 32-bit residual stream: the stream's norms, attention with a distance bias and
-sinks, the gated delta rule, and routed experts with pass-through outputs.
+sinks, latent attention, the gated delta rule, state-space scans, and routed experts with pass-through outputs.
 
 Activations are bf16 (tensor-core products) or fp32 (a model run in 32 bits: plain FMA products); the
 dtype of the input tensor picks the form. Same dispatch rule as the other ops: CUDA tensors go to the
@@ -79,27 +79,29 @@ class RoutedRows:
 
 
 def residual_norm(x: torch.Tensor, y, w_b: Optional[torch.Tensor], w_n: Optional[torch.Tensor], *, dim: int, eps: float,
-                  layernorm: bool, dtype: torch.dtype, out: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
-    """In place on the fp32 stream ``x`` [T, ld]: ``x += norm(y) * w_b`` (``y`` a tensor, :class:`RoutedRows`
-    or None), then returns ``norm(x) * w_n`` in ``dtype`` (None without ``w_n``). One launch."""
+                  layernorm: bool, dtype: torch.dtype, out: Optional[torch.Tensor] = None, plus_one: bool = False, mult: float = 1.0,
+                  plain: bool = False) -> Optional[torch.Tensor]:
+    """In place on the fp32 stream ``x`` [T, ld]: ``x += mult * norm(y) * w_b`` (``y`` a tensor, :class:`RoutedRows`
+    or None), then returns ``norm(x) * w_n`` in ``dtype`` (without ``w_n``: the stream itself if ``plain``, else
+    None). ``plus_one``: the norms multiply by 1 + w. One launch."""
     rows, ld = x.shape
     routed = y if isinstance(y, RoutedRows) else None
     if not x.is_cuda:
         def nrm(v, w):
             v = v[:, :dim]
-            r, _ = R.norm(v, w, eps=eps, layernorm=layernorm)
+            r, _ = R.norm(v, w.float() + 1 if plus_one else w, eps=eps, layernorm=layernorm)
             return r
         if y is not None:
             v = routed.combined() if routed is not None else y.float()
-            x[:, :dim] += nrm(v, w_b) if w_b is not None else v[:, :dim]
-        if w_n is None:
+            x[:, :dim] += mult * (nrm(v, w_b) if w_b is not None else v[:, :dim])
+        if w_n is None and not plain:
             return None
         h = torch.zeros(rows, ld, dtype=dtype) if out is None else out
-        h[:, :dim] = nrm(x, w_n).to(dtype)
+        h[:, :dim] = (nrm(x, w_n) if w_n is not None else x[:, :dim]).to(dtype)
         return h
     assert x.dtype == torch.float32 and x.stride(1) == 1
     h = None
-    if w_n is not None:
+    if w_n is not None or plain:
         h = torch.empty(rows, ld, dtype=dtype, device=x.device) if out is None else out
         assert h.dtype == dtype and h.is_contiguous()
     yt = routed.rows if routed is not None else y
@@ -111,7 +113,7 @@ def residual_norm(x: torch.Tensor, y, w_b: Optional[torch.Tensor], w_n: Optional
         N.ptr(routed.weights) if routed is not None else None, N.ptr(src), rows, dim, x.stride(0),
         yt.stride(0) if yt is not None else 0, ld, src.stride(0) if src is not None else 0,
         routed.ids.shape[1] if routed is not None else 0, routed.experts if routed is not None else 0, int(layernorm),
-        float(eps), 1 if dtype == torch.float32 else 0, N.stream())
+        int(plus_one), int(plain), float(eps), float(mult), 1 if dtype == torch.float32 else 0, N.stream())
     N.check(rc, "b200_residual_norm")
     return h
 
@@ -280,3 +282,247 @@ def delta_mix(proj: torch.Tensor, z: torch.Tensor, w: DeltaWeights, conv_state: 
                       w.dv_true, taps, proj.stride(0), b_off, z.stride(0), w.heads * w.dk, float(w.eps), _f32(proj), N.stream())
     N.check(rc, "b200_delta", L.b200_delta_launches(1 if cu_q is None else 0, taps, w.dk, w.dv))
     return out
+
+
+def embedding_norm(ids: Optional[torch.Tensor], table: torch.Tensor, w: torch.Tensor, *, dim: int, eps: float, layernorm: bool = False,
+                   plus_one: bool = False, scale: float = 1.0, dtype: torch.dtype = torch.bfloat16) -> tuple[torch.Tensor, torch.Tensor]:
+    """(x, h): the fp32 stream ``norm(table[ids] * scale) * w`` and the same rows in ``dtype``. ``ids`` None: all
+    rows of ``table`` in order. Columns from ``dim`` on (row padding) are zero."""
+    ld = (dim + 7) // 8 * 8
+    t = table.shape[0] if ids is None else ids.numel()
+    if not table.is_cuda:
+        rows = (table if ids is None else table[ids.long()])[:, :dim].float() * scale
+        x = torch.zeros(t, ld)
+        x[:, :dim] = R.norm(rows, w.float() + 1 if plus_one else w, eps=eps, layernorm=layernorm)[0]
+        return x, x.to(dtype)
+    assert table.dtype == torch.bfloat16 and table.stride(1) == 1
+    x = torch.empty(t, ld, dtype=torch.float32, device=table.device)
+    h = torch.empty(t, ld, dtype=dtype, device=table.device)
+    N.check(N.lib().b200_embedding_norm(N.ptr(ids), table.data_ptr(), w.data_ptr(), x.data_ptr(), h.data_ptr(), t, dim, ld,
+                                        table.stride(0), table.shape[0], float(scale), int(layernorm), int(plus_one), float(eps),
+                                        1 if dtype == torch.float32 else 0, N.stream()), "b200_embedding_norm")
+    return x, h
+
+
+def poly_norm(z: torch.Tensor, coef: torch.Tensor, dim: int, eps: float) -> torch.Tensor:
+    """``a N(z) + b N(z^2) + c N(z^3) + e`` per row with ``coef`` = (a, b, c, e) fp32 and N the division by the root
+    mean square of the row's first ``dim`` values; columns past ``dim`` are zero."""
+    rows, ld = z.shape
+    if not z.is_cuda:
+        return R.poly_norm(z, coef, dim, eps).to(z.dtype)
+    assert z.stride(1) == 1 and coef.dtype == torch.float32
+    y = torch.empty(rows, (dim + 7) // 8 * 8, dtype=z.dtype, device=z.device)
+    N.check(N.lib().b200_poly_norm(z.data_ptr(), y.data_ptr(), coef.data_ptr(), rows, dim, z.stride(0), y.stride(0), float(eps), _f32(z),
+                                   N.stream()), "b200_poly_norm")
+    return y
+
+
+# ------------------------------------------------------------------------------------------ state-space mixers
+def short_conv(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], state: torch.Tensor, positions: torch.Tensor,
+               cu_q: Optional[torch.Tensor], slots: torch.Tensor) -> torch.Tensor:
+    """silu of a causal convolution per channel: ``x`` [T, C] (any row pitch), ``w`` fp32 [taps, C] (last row: the
+    current token). ``state`` [slots, taps - 1, C] holds the inputs before each sequence's portion and is updated in
+    place; a sequence whose first position is 0 starts from zeros, slot -1 is not stored."""
+    t, c = x.shape
+    if not x.is_cuda:
+        return R.short_conv(x, w, bias, state, positions, cu_q, slots)
+    assert x.stride(1) == 1 and w.dtype == torch.float32 and w.is_contiguous() and state.dtype == x.dtype and state.is_contiguous()
+    assert slots.dtype == torch.int32 and positions.dtype == torch.int32
+    out = torch.empty(t, c, dtype=x.dtype, device=x.device)
+    taps = w.shape[0]
+    N.check(N.lib().b200_short_conv(x.data_ptr(), w.data_ptr(), N.ptr(bias), state.data_ptr(), positions.data_ptr(), N.ptr(cu_q),
+                                    slots.data_ptr(), out.data_ptr(), t, slots.numel(), c, taps, x.stride(0), _f32(x), N.stream()),
+            "b200_short_conv", 2 if cu_q is not None and taps > 1 else 1)
+    return out
+
+
+@dataclass
+class ChannelScanWeights:
+    """Constants of a selective scan: ``a`` fp32 [C, N] (negative), ``dt_bias``, ``d`` fp32 [C]. N is one of 8, 16, 32,
+    64, 128 (padded with zero columns)."""
+    a: torch.Tensor
+    dt_bias: torch.Tensor
+    d: torch.Tensor
+
+
+def channel_scan(x: torch.Tensor, dt: torch.Tensor, bc: torch.Tensor, b_off: int, c_off: int, z: torch.Tensor, w: ChannelScanWeights,
+                 state: torch.Tensor, positions: torch.Tensor, cu_q: Optional[torch.Tensor], slots: torch.Tensor) -> torch.Tensor:
+    """Scan with one decay per channel c and state value n, gated:
+    ``S = exp(dt a[c, n]) S + dt x B[n]``, ``y = (sum_n S C[n] + d x) silu(z)``, ``dt = softplus(logit + bias)``.
+    ``x``, ``dt`` (logits), ``z`` [T, C]; B and C are columns ``b_off``.. and ``c_off``.. of ``bc``. ``state`` fp32
+    [slots, C, N] is updated in place (slots and first positions as in :func:`short_conv`)."""
+    t, c = x.shape
+    if not x.is_cuda:
+        return R.channel_scan(x, dt, bc, b_off, c_off, z, w, state, positions, cu_q, slots)
+    assert x.dtype == dt.dtype == bc.dtype == z.dtype and x.stride(1) == dt.stride(1) == bc.stride(1) == z.stride(1) == 1
+    assert state.dtype == torch.float32 and state.is_contiguous() and slots.dtype == torch.int32 and positions.dtype == torch.int32
+    y = torch.empty(t, c, dtype=x.dtype, device=x.device)
+    rc = N.lib().b200_channel_scan(x.data_ptr(), dt.data_ptr(), bc.data_ptr(), z.data_ptr(), w.dt_bias.data_ptr(), w.a.data_ptr(),
+                                   w.d.data_ptr(), state.data_ptr(), positions.data_ptr(), N.ptr(cu_q), slots.data_ptr(), y.data_ptr(),
+                                   slots.numel(), c, w.a.shape[1], b_off, c_off, x.stride(0), dt.stride(0), bc.stride(0), z.stride(0),
+                                   y.stride(0), _f32(x), N.stream())
+    N.check(rc, "b200_channel_scan")
+    return y
+
+
+@dataclass
+class HeadScanWeights:
+    """Constants of a scan with one decay per head: fp32 [heads] ``rate`` = exp(A_log), ``dt_bias``, ``d``. ``n``
+    (8, 16, ..., 256) and ``p`` (a multiple of 8) are the state's sizes as laid out (padded with zeros)."""
+    rate: torch.Tensor
+    dt_bias: torch.Tensor
+    d: torch.Tensor
+    heads: int
+    groups: int
+    n: int
+    p: int
+
+
+def head_scan(x: torch.Tensor, dt: torch.Tensor, w: HeadScanWeights, state: torch.Tensor, positions: torch.Tensor,
+              cu_q: Optional[torch.Tensor], slots: torch.Tensor) -> torch.Tensor:
+    """Scan with a matrix state [n, p] per head: ``S = exp(-rate dt) S + B (dt x)^T``, ``y = S^T C + d x``,
+    ``dt = softplus(logit + bias)``. ``x`` [T, heads p + 2 groups n] = x | B | C (head h reads group
+    h // (heads / groups)), ``dt`` logits [T, heads]. ``state`` fp32 [slots, heads, n, p] is updated in place.
+    Returns [T, heads p]."""
+    t = x.shape[0]
+    if not x.is_cuda:
+        return R.head_scan(x, dt, w, state, positions, cu_q, slots)
+    assert x.dtype == dt.dtype and x.stride(1) == 1 and dt.stride(1) == 1 and state.dtype == torch.float32 and state.is_contiguous()
+    assert slots.dtype == torch.int32 and positions.dtype == torch.int32
+    hp = w.heads * w.p
+    y = torch.empty(t, hp, dtype=x.dtype, device=x.device)
+    rc = N.lib().b200_head_scan(x.data_ptr(), dt.data_ptr(), w.dt_bias.data_ptr(), w.rate.data_ptr(), w.d.data_ptr(), state.data_ptr(),
+                                positions.data_ptr(), N.ptr(cu_q), slots.data_ptr(), y.data_ptr(), slots.numel(), w.heads, w.groups, w.n,
+                                w.p, hp, hp + w.groups * w.n, x.stride(0), dt.stride(0), y.stride(0), _f32(x), N.stream())
+    N.check(rc, "b200_head_scan")
+    return y
+
+
+def gated_norm(y: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, parts: int, eps: float, heads: int, p_true: int) -> torch.Tensor:
+    """``norm(y silu(z)) weight`` with the norm taken over ``parts`` equal parts of the heads * p_true values of a row
+    (heads may be laid out with zero columns behind them; those stay zero)."""
+    t, cols = y.shape
+    pp = cols // heads
+    part = heads * p_true // parts
+    if not y.is_cuda:
+        return R.gated_norm(y, z, weight, parts, eps, heads, p_true).to(y.dtype)
+    assert y.stride(1) == 1 and z.stride(1) == 1 and y.dtype == z.dtype and weight.dtype == torch.bfloat16
+    out = (torch.empty if pp == p_true else torch.zeros)(t, cols, dtype=y.dtype, device=y.device)
+    N.check(N.lib().b200_gated_norm(y.data_ptr(), z.data_ptr(), weight.data_ptr(), out.data_ptr(), t, parts, part, p_true, pp,
+                                    y.stride(0), z.stride(0), out.stride(0), float(eps), _f32(y), N.stream()), "b200_gated_norm")
+    return out
+
+
+# ------------------------------------------------------------------------------------------ latent attention
+def latent_prep(x: torch.Tensor, q_off: int, q_dim: int, wq: torch.Tensor, kv_off: int, kv_dim: int, wkv: torch.Tensor,
+                cache: torch.Tensor, slots: torch.Tensor, eps: float) -> torch.Tensor:
+    """RMS norms of the two latents in a projection's columns ``q_off``.. and ``kv_off``..: the query's is returned
+    [T, len(wq)], the key / value one is written to ``cache`` [pages, 1, page, len(wkv)]. The weights are padded to
+    the laid-out widths, ``q_dim`` / ``kv_dim`` are the true ones."""
+    t = x.shape[0]
+    if not x.is_cuda:
+        def rms(v, w, dim):
+            v = v[:, :dim].float()
+            out = torch.zeros(t, w.numel())
+            out[:, :dim] = v / torch.sqrt((v * v).mean(-1, keepdim=True) + eps) * w[:dim].float()
+            return out.to(x.dtype)
+        kv_store(rms(x[:, kv_off:], wkv, kv_dim), cache, slots)
+        return rms(x[:, q_off:], wq, q_dim)
+    assert x.stride(1) == 1 and cache.dtype == x.dtype and cache.is_contiguous() and slots.dtype == torch.int64
+    cq = torch.empty(t, wq.numel(), dtype=x.dtype, device=x.device)
+    N.check(N.lib().b200_latent_prep(x.data_ptr(), wq.data_ptr(), wkv.data_ptr(), cq.data_ptr(), cache.data_ptr(), slots.data_ptr(), t,
+                                     x.stride(0), q_off, q_dim, wq.numel(), kv_off, kv_dim, wkv.numel(), float(eps), _f32(x), N.stream()),
+            "b200_latent_prep")
+    return cq
+
+
+def head_linear(x: torch.Tensor, w: LinearWeight, heads: int, *, gate: Optional[torch.Tensor] = None,
+                in_rows: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None,
+                out_rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """One product per head: ``out[r, h] = W[h] x[r, h]`` with ``w`` stacked [heads * n, k], ``x`` [rows, heads * k] and
+    ``out`` [rows, heads * n], optionally times ``sigmoid(gate)``. ``in_rows`` / ``out_rows`` (int32) select the rows of
+    ``x`` and of ``out`` and ``gate`` that the product's rows stand for."""
+    n, k = w.weight.shape[0] // heads, w.weight.shape[1]
+    rows = x.shape[0] if in_rows is None else in_rows.numel()
+    rows = rows if out_rows is None else out_rows.numel()
+    if out is None:
+        out = torch.empty(rows, heads * n, dtype=x.dtype, device=x.device)
+    if not x.is_cuda:
+        xi = (x if in_rows is None else x[in_rows.long()]).float().reshape(rows, heads, -1)[:, :, :k]
+        y = torch.einsum("rhk,hnk->rhn", xi, w.host_f32().reshape(heads, n, k)).reshape(rows, heads * n)
+        at = slice(None) if out_rows is None else out_rows.long()
+        if gate is not None:
+            y = y * torch.sigmoid(gate[at].float())
+        out[at] = y.to(out.dtype)
+        return out
+    assert x.stride(1) == 1 and out.stride(1) == 1 and w.weight.is_contiguous() and out.dtype == x.dtype
+    assert x.shape[1] == heads * k and out.shape[1] == heads * n and (gate is None or gate.stride(1) == 1)
+    assert all(i is None or i.dtype == torch.int32 for i in (in_rows, out_rows))
+    N.check(N.lib().b200_head_linear(x.data_ptr(), w.weight.data_ptr(), out.data_ptr(), N.ptr(gate), N.ptr(in_rows), N.ptr(out_rows), rows,
+                                     heads, n, k, x.stride(0), k, out.stride(0), n, gate.stride(0) if gate is not None else 0, _f32(x),
+                                     N.stream()), "b200_head_linear")
+    return out
+
+
+def latent_attn(q: torch.Tensor, cache: torch.Tensor, block_table: torch.Tensor, kv_lens: torch.Tensor, heads: int, scale: float,
+                row_seq: Optional[torch.Tensor] = None, max_kv_len: int = 0) -> torch.Tensor:
+    """Attention of queries in latent space [rows, heads * rank] over cached latents [pages, 1, page, rank], which are
+    keys and values of every head: row r sees the first ``kv_lens[r]`` tokens of block-table row ``row_seq[r]`` (r when
+    None). bf16 rows of at most 512 values run on the tensor cores, fp32 and wider ones as plain 32-bit arithmetic.
+    Returns [rows, heads * rank]."""
+    rows, rank, page = q.shape[0], cache.shape[3], cache.shape[2]
+    table = block_table
+    if not q.is_cuda or q.dtype == torch.float32 or rank > 512:
+        if row_seq is not None:
+            table = block_table[row_seq.long()].contiguous()
+        return attn_biased(q, cache, None, table, kv_lens, None, heads=heads, scale=scale)
+    assert q.is_contiguous() and cache.is_contiguous() and kv_lens.dtype == torch.int32 and kv_lens.numel() == rows
+    assert block_table.dtype == torch.int32 and (row_seq is None or row_seq.dtype == torch.int32)
+    L = N.lib()
+    out = torch.empty_like(q)
+    step = 32768                            # rows are the grid's second dimension
+    for a in range(0, rows, step):
+        b = min(a + step, rows)
+        splits = L.b200_mla_pick_splits(b - a, heads, int(max_kv_len or table.shape[1] * page))
+        ws = None
+        if splits > 1:
+            ws = torch.empty(L.b200_mla_workspace_bytes(b - a, heads, splits), dtype=torch.uint8, device=q.device)
+        tab = table if row_seq is not None else table[a:b]
+        rc = L.b200_latent_attn(q[a:b].data_ptr(), cache.data_ptr(), out[a:b].data_ptr(), tab.data_ptr(), kv_lens[a:b].data_ptr(),
+                                N.ptr(None if row_seq is None else row_seq[a:b]), b - a, heads, rank, page, table.stride(0), splits,
+                                N.ptr(ws), float(scale), N.stream())
+        N.check(rc, "b200_latent_attn", 2 if splits > 1 else 1)
+    return out
+
+
+def latent_gather(cache: torch.Tensor, block_table: torch.Tensor, seq_ids: torch.Tensor, offsets: torch.Tensor, total: int,
+                  max_len: int) -> torch.Tensor:
+    """Cached latents of the sequences in ``seq_ids``, one after another: rows ``offsets[s] .. offsets[s + 1]`` of the
+    result [total, rank] are the tokens of block-table row ``seq_ids[s]``."""
+    page, rank = cache.shape[2], cache.shape[3]
+    out = torch.empty(total, rank, dtype=cache.dtype, device=cache.device)
+    if not cache.is_cuda:
+        for i, s in enumerate(seq_ids.tolist()):
+            a, b = int(offsets[i]), int(offsets[i + 1])
+            out[a:b] = R.gather_paged(cache, block_table[s], b - a).reshape(b - a, rank)
+        return out
+    N.check(N.lib().b200_latent_gather(cache.data_ptr(), out.data_ptr(), block_table.data_ptr(), seq_ids.data_ptr(), offsets.data_ptr(),
+                                       seq_ids.numel(), max_len, rank * cache.element_size(), page, block_table.stride(0), N.stream()),
+            "b200_latent_gather")
+    return out
+
+
+def attn_runs(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, out: torch.Tensor, q_start: torch.Tensor, q_lens: torch.Tensor,
+              kv_start: torch.Tensor, kv_lens: torch.Tensor, *, heads: int, max_q_len: int, scale: float,
+              gate: Optional[torch.Tensor] = None) -> None:
+    """Causal attention of runs of query rows over contiguous keys and values of their contexts: run s is rows
+    ``q_start[s]`` .. + ``q_lens[s]`` of ``q`` [T, heads * d], its context rows ``kv_start[s]`` .. + ``kv_lens[s]`` of ``k``
+    [.., heads * d] and ``v`` [.., heads * dv]; the last key belongs to the last query. Rows of the runs are written to
+    ``out`` [T, heads * dv], times ``sigmoid(gate)``. bf16, d and dv up to 128."""
+    d, dv = k.shape[1] // heads, v.shape[1] // heads
+    assert q.is_cuda and q.dtype == torch.bfloat16 and out.is_contiguous() and q.stride(1) == k.stride(1) == v.stride(1) == 1
+    assert out.shape[1] == heads * dv and (gate is None or gate.stride(1) == 1)
+    N.check(N.lib().b200_attn_runs(q.data_ptr(), k.data_ptr(), v.data_ptr(), out.data_ptr(), N.ptr(gate), q_start.data_ptr(),
+                                   q_lens.data_ptr(), kv_start.data_ptr(), kv_lens.data_ptr(), q_lens.numel(), max_q_len, heads, heads, d,
+                                   dv, q.stride(0), k.stride(0), v.stride(0), gate.stride(0) if gate is not None else 0, float(scale),
+                                   N.stream()), "b200_attn_runs")

@@ -204,6 +204,82 @@ def delta_mix(proj, z, w, conv_state, state, positions, cu_q, slots, b_off) -> t
     return out
 
 
+def short_conv(x, w, bias, state, positions, cu_q, slots) -> torch.Tensor:
+    """Causal convolution per channel + silu over a ragged batch (see ``ops.short_conv``)."""
+    taps, c = w.shape
+    bounds = list(range(slots.numel() + 1)) if cu_q is None else cu_q.tolist()
+    out = torch.empty_like(x)
+    for i, slot in enumerate(slots.tolist()):
+        a, b = bounds[i], bounds[i + 1]
+        if b == a:
+            continue
+        carried = slot >= 0 and int(positions[a]) > 0
+        seq = torch.cat([state[slot].float() if carried else torch.zeros(taps - 1, c), x[a:b].float()], 0)
+        if slot >= 0 and taps > 1:
+            state[slot] = seq[-(taps - 1):].to(state.dtype)
+        y = (seq.unfold(0, taps, 1) * w.t()[None]).sum(-1)
+        out[a:b] = torch.nn.functional.silu(y if bias is None else y + bias).to(x.dtype)
+    return out
+
+
+def channel_scan(x, dt, bc, b_off, c_off, z, w, state, positions, cu_q, slots) -> torch.Tensor:
+    """Selective scan over a ragged batch, token by token (see ``ops.channel_scan``)."""
+    n = w.a.shape[1]
+    bounds = list(range(slots.numel() + 1)) if cu_q is None else cu_q.tolist()
+    out = torch.empty(x.shape, dtype=x.dtype)
+    for i, slot in enumerate(slots.tolist()):
+        a, b = bounds[i], bounds[i + 1]
+        if b == a:
+            continue
+        s = state[slot].clone() if slot >= 0 and int(positions[a]) > 0 else torch.zeros(w.a.shape)
+        for t in range(a, b):
+            xt, step = x[t].float(), torch.nn.functional.softplus(dt[t].float() + w.dt_bias, threshold=60.0)
+            s = torch.exp(step[:, None] * w.a) * s + (step * xt)[:, None] * bc[t, b_off:b_off + n].float()[None]
+            y = (s * bc[t, c_off:c_off + n].float()[None]).sum(1) + w.d * xt
+            out[t] = (y * torch.nn.functional.silu(z[t].float())).to(x.dtype)
+        if slot >= 0:
+            state[slot] = s
+    return out
+
+
+def head_scan(x, dt, w, state, positions, cu_q, slots) -> torch.Tensor:
+    """Scan with a matrix state per head over a ragged batch, token by token (see ``ops.head_scan``)."""
+    h, g, n, p = w.heads, w.groups, w.n, w.p
+    bounds = list(range(slots.numel() + 1)) if cu_q is None else cu_q.tolist()
+    out = torch.empty(x.shape[0], h * p, dtype=x.dtype)
+    for i, slot in enumerate(slots.tolist()):
+        a, b = bounds[i], bounds[i + 1]
+        if b == a:
+            continue
+        s = state[slot].clone() if slot >= 0 and int(positions[a]) > 0 else torch.zeros(h, n, p)
+        for t in range(a, b):
+            step = torch.nn.functional.softplus(dt[t].float() + w.dt_bias, threshold=60.0)
+            xt, bt, ct = x[t].float().split([h * p, g * n, g * n])
+            xt = xt.reshape(h, p)
+            bt, ct = (v.reshape(g, n).repeat_interleave(h // g, 0) for v in (bt, ct))
+            s = torch.exp(-w.rate * step)[:, None, None] * s + bt[:, :, None] * (step[:, None] * xt)[:, None, :]
+            out[t] = ((s * ct[:, :, None]).sum(1) + w.d[:, None] * xt).reshape(-1).to(x.dtype)
+        if slot >= 0:
+            state[slot] = s
+    return out
+
+
+def gated_norm(y, z, weight, parts, eps, heads, p_true) -> torch.Tensor:
+    """Gate, then an RMS norm over equal parts of a row (see ``ops.gated_norm``)."""
+    t, cols = y.shape
+    v = (y.float() * torch.nn.functional.silu(z.float())).reshape(t, heads, -1)[:, :, :p_true].reshape(t, parts, -1)
+    v = (v * torch.rsqrt(v.pow(2).mean(-1, keepdim=True) + eps)).reshape(t, heads, p_true)
+    return torch.nn.functional.pad(v, (0, cols // heads - p_true)).reshape(t, cols) * weight.float()
+
+
+def poly_norm(z, coef, dim, eps) -> torch.Tensor:
+    """Weighted sum of a row's normed powers (see ``ops.poly_norm``)."""
+    v = z[:, :dim].float()
+    rms = lambda u: u * torch.rsqrt(u.pow(2).mean(-1, keepdim=True) + eps)
+    y = coef[0] * rms(v) + coef[1] * rms(v * v) + coef[2] * rms(v * v * v) + coef[3]
+    return torch.nn.functional.pad(y, (0, (dim + 7) // 8 * 8 - dim))
+
+
 # --------------------------------------------------------------------------------------------
 # rotary embedding
 # --------------------------------------------------------------------------------------------
