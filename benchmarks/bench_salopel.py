@@ -87,6 +87,7 @@ def kernels(s: dict, dev) -> dict:
         cu = None if phase == "decode" else torch.arange(0, t + 1, t // 4, dtype=torch.int32, device=dev)
         slots = torch.arange(nseq, dtype=torch.int32, device=dev)
         pos = torch.full((t,), 5, dtype=torch.int32, device=dev)
+        runs = None if phase == "decode" else [(t // 4, t // 4)] * 4
         # ---- norms and activation
         x, y = torch.randn(t, w, device=dev), bf(t, w)
         kw = dict(dim=w, eps=1e-6, layernorm=False, dtype=torch.bfloat16, plus_one=True, mult=0.5, plain=True)
@@ -124,7 +125,7 @@ def kernels(s: dict, dev) -> dict:
         hw = ops.HeadScanWeights(rate=f32(heads2), dt_bias=f32(heads2) - 4, d=f32(heads2), heads=heads2, groups=1, n=STATE2, p=P)
         st2 = torch.zeros(nseq, heads2, STATE2, P, device=dev)
         xbc, dth = bf(t, ch), bf(t, heads2)
-        new = tm.row(lambda: ops.head_scan(xbc, dth, hw, st2, pos, cu, slots), t * (ch + inner) * 2 + nseq * heads2 * STATE2 * P * 8)
+        new = tm.row(lambda: ops.head_scan(xbc, dth, hw, st2, pos, cu, slots, runs), t * (ch + inner) * 2 + nseq * heads2 * STATE2 * P * 8)
         # the same count of state values through the Mamba-2 model's kernel (32 rows per channel, one sequence)
         c32 = inner * STATE2 // 32
         xs, ds, b32, a32, d32 = bf(one, c32), f32(one, c32), bf(one, 32), -f32(c32, 32), f32(c32)
@@ -139,7 +140,7 @@ def kernels(s: dict, dev) -> dict:
         dp, dz = bf(t, dch + dh), bf(t, 2 * dh * 128)
 
         def head_mixer():
-            return ops.gated_norm(ops.head_scan(conv(), dth, hw, st2, pos, cu, slots), zi, ones[:inner], 1, 1e-6, heads2, P)
+            return ops.gated_norm(ops.head_scan(conv(), dth, hw, st2, pos, cu, slots, runs), zi, ones[:inner], 1, 1e-6, heads2, P)
         put("conv + head_scan + gated_norm / delta_mix", phase,
             tm.row(head_mixer, t * (ch + 2 * inner) * 2 + nseq * heads2 * STATE2 * P * 8),
             tm.row(lambda: ops.delta_mix(dp, dz, dw, dcs, dst, pos, cu, slots, dch), t * (dch + 3 * dh * 128) * 2 + nseq * dh * 128 * 128 * 8))

@@ -215,24 +215,27 @@ __global__ void __launch_bounds__(1024) embedding_norm_kernel(const EmbeddingNor
 // y = a z / rms(z) + b z^2 / rms(z^2) + c z^3 / rms(z^3) + e over a row of `dim` values (powers element by
 // element); columns past dim are zeroed. The row stays in registers between the two passes.
 template <typename T, int kIters>
-__global__ void __launch_bounds__(1024) poly_norm_kernel(const T* __restrict__ z, T* __restrict__ y,
-                                                         const float* __restrict__ coef, int dim, int ldz, int ldy, float eps) {
+__global__ void __launch_bounds__(512) poly_norm_kernel(const T* __restrict__ z, T* __restrict__ y,
+                                                        const float* __restrict__ coef, int dim, int ldz, int ldy, float eps) {
   pdl_wait();
   pdl_trigger();
-  __shared__ float red[3][32];
+  __shared__ float red[3][16];
+  struct alignas(16) Vec { T v[8]; };
   const long long row = blockIdx.x;
-  float v[kIters][8];
+  Vec raw[kIters];                           // as stored: half the registers for bf16
+#pragma unroll
+  for (int i = 0; i < kIters; ++i) {
+    const int c = (threadIdx.x + i * blockDim.x) * 8;
+    raw[i] = Vec{};
+    if (c < dim) raw[i] = *reinterpret_cast<const Vec*>(z + row * ldz + c);
+  }
   float q1 = 0.f, q2 = 0.f, q3 = 0.f;
 #pragma unroll
   for (int i = 0; i < kIters; ++i) {
     const int c = (threadIdx.x + i * blockDim.x) * 8;
 #pragma unroll
-    for (int j = 0; j < 8; ++j) v[i][j] = 0.f;
-    if (c < dim) load8(z + row * ldz + c, v[i]);
-#pragma unroll
     for (int j = 0; j < 8; ++j) {
-      if (c + j >= dim) v[i][j] = 0.f;
-      const float s = v[i][j] * v[i][j];
+      const float u = c + j < dim ? ld1(&raw[i].v[j]) : 0.f, s = u * u;
       q1 += s;
       q2 = fmaf(s, s, q2);
       q3 = fmaf(s * s, s, q3);
@@ -262,7 +265,7 @@ __global__ void __launch_bounds__(1024) poly_norm_kernel(const T* __restrict__ z
     float o[8];
 #pragma unroll
     for (int j = 0; j < 8; ++j) {
-      const float u = v[i][j];
+      const float u = ld1(&raw[i].v[j]);
       o[j] = c + j < dim ? fmaf(u, fmaf(u, fmaf(u, c3, b), a), e) : 0.f;
     }
     store8(y + row * ldy + c, o);
@@ -339,19 +342,23 @@ B200_API int b200_embedding_norm(const int* ids, const void* table, const void* 
   return e == cudaSuccess ? 0 : -static_cast<int>(e) - 300;
 }
 
-// y [rows][ldy] from z [rows][ldz]; coef: the four numbers a, b, c, e (fp32, device)
+// y [rows][ldy] from z [rows][ldz]; coef: the four numbers a, b, c, e (fp32, device). Rows of up to 16384 values: one,
+// two or four vectors of eight per thread.
 B200_API int b200_poly_norm(const void* z, void* y, const float* coef, int rows, int dim, int ldz, int ldy, float eps, int f32,
                             cudaStream_t stream) {
   if (rows <= 0) return 0;
-  int iters, threads;
-  if (ldz % 8 || ldy != (dim + 7) / 8 * 8 || ldz < ldy || !row_shape(dim, rows, iters, threads)) return -2;
+  if (dim < 1 || dim > 16384 || ldz % 8 || ldy != (dim + 7) / 8 * 8 || ldz < ldy) return -2;
+  const int vecs = ldy / 8;
+  const int iters = vecs > 1024 || (rows >= 1024 && vecs >= 512) ? 4 : vecs > 512 || (rows >= 1024 && vecs >= 128) ? 2 : 1;
+  const int threads = ((vecs + iters - 1) / iters + 31) / 32 * 32;
   auto go = [&](auto kernel, auto tag) {
     using T = decltype(tag);
     return launch_pdl(kernel, dim3(rows), dim3(threads), 0, stream, static_cast<const T*>(z), static_cast<T*>(y), coef, dim, ldz,
                       ldy, eps);
   };
   cudaError_t e;
-  if (f32) e = iters == 1 ? go(poly_norm_kernel<float, 1>, float()) : go(poly_norm_kernel<float, 2>, float());
-  else e = iters == 1 ? go(poly_norm_kernel<__nv_bfloat16, 1>, __nv_bfloat16()) : go(poly_norm_kernel<__nv_bfloat16, 2>, __nv_bfloat16());
+  if (f32) e = iters == 1 ? go(poly_norm_kernel<float, 1>, float()) : iters == 2 ? go(poly_norm_kernel<float, 2>, float()) : go(poly_norm_kernel<float, 4>, float());
+  else e = iters == 1 ? go(poly_norm_kernel<__nv_bfloat16, 1>, __nv_bfloat16()) : iters == 2 ? go(poly_norm_kernel<__nv_bfloat16, 2>, __nv_bfloat16())
+                                                                                       : go(poly_norm_kernel<__nv_bfloat16, 4>, __nv_bfloat16());
   return e == cudaSuccess ? 0 : -static_cast<int>(e) - 300;
 }

@@ -23,9 +23,11 @@
 //                   x 4 columns of S as packed pairs; otherwise like channel_scan.
 //  * channel_step, head_step   the same for one token per sequence (decode): the state is read once, updated,
 //                   written back.
+//  * head_chunk     head_scan for long runs in bf16: chunks of 64 tokens as tensor-core products (see there).
 //  * gated_norm     y silu(z), RMS-normed in equal parts of the row.
-// The scans perform the same operations in the same order wherever a prompt is cut.
+// channel_scan and head_scan perform the same operations in the same order wherever a prompt is cut.
 #include "mixer_common.cuh"
+#include "mma_sync.cuh"
 
 namespace b200 {
 
@@ -107,6 +109,11 @@ struct ShortConvParams {
 };
 
 __device__ __forceinline__ float silu_f32(float x) { return x * sigmoid_f32(x); }
+// silu of a value that is stored in the activation type: for bf16 a hardware exponential and division do
+template <typename T>
+__device__ __forceinline__ float silu_act(float x) { return silu_f32(x); }
+template <>
+__device__ __forceinline__ float silu_act<__nv_bfloat16>(float x) { return __fdividef(x, 1.f + __expf(fminf(-x, 80.f))); }
 
 // kTaps inputs of eight channels in registers for `run` consecutive tokens. kTaps 0: any number of taps, inputs
 // are read again for every token. grid (ceil(channels / 256), ceil(T / (4 run))), 128 threads.
@@ -154,6 +161,35 @@ __global__ void __launch_bounds__(128) short_conv_kernel(const ShortConvParams p
           else if (carried) load8(st + static_cast<long long>(tail + src - first) * p.channels, v);
         }
     }
+    if (kTaps > 0 && t + 4 <= min(t1, next)) {          // four tokens of the same sequence, loads first
+      float nw[4][8];
+#pragma unroll
+      for (int u = 0; u < 4; ++u) load8(x + (t + u) * p.ldx, nw[u]);
+#pragma unroll
+      for (int u = 0; u < 4; ++u) {
+        float y[8];
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+          y[i] = bias[i];
+#pragma unroll
+          for (int j = 0; j < kTaps; ++j) {
+            // tap j of token u: one of the four new inputs, or an earlier one
+            const int at = u - (kTaps - 1) + j;
+            y[i] = fmaf(at >= 0 ? nw[at >= 0 ? at : 0][i] : in[kTaps > 0 ? kTaps - 1 + (at < 0 ? at : -1) : 0][i], w[kTaps > 0 ? j : 0][i], y[i]);
+          }
+          y[i] = silu_act<T>(y[i]);
+        }
+        store8(out + static_cast<long long>(t + u) * p.channels, y);
+      }
+#pragma unroll
+      for (int j = 0; j + 1 < kTaps; ++j) {              // the last kTaps - 1 inputs stay (taps are at most four)
+        const int at = 4 - (kTaps - 1) + j;
+#pragma unroll
+        for (int i = 0; i < 8; ++i) in[kTaps > 0 ? j : 0][i] = nw[at & 3][i];
+      }
+      t += 3;
+      continue;
+    }
     float y[8];
 #pragma unroll
     for (int i = 0; i < 8; ++i) y[i] = bias[i];
@@ -185,7 +221,7 @@ __global__ void __launch_bounds__(128) short_conv_kernel(const ShortConvParams p
       }
     }
 #pragma unroll
-    for (int i = 0; i < 8; ++i) y[i] = silu_f32(y[i]);
+    for (int i = 0; i < 8; ++i) y[i] = silu_act<T>(y[i]);
     store8(out + static_cast<long long>(t) * p.channels, y);
   }
 }
@@ -274,12 +310,13 @@ __global__ void __launch_bounds__(128) channel_scan_kernel(const ChannelScanPara
   const int ch0 = blockIdx.x * kCsChannels, ch = ch0 + cl;
   const bool active = ch < p.channels;
   const bool carried = slot >= 0 && p.positions[first] > 0;
-  float S[kPer], A[kPer];
+  f32x2 S[kPer / 2], A[kPer / 2];            // pairs of states
   float* sp = p.state + (static_cast<long long>(slot < 0 ? 0 : slot) * p.channels + ch) * N + sub * kPer;
 #pragma unroll
-  for (int i = 0; i < kPer; ++i) {
-    A[i] = active ? p.a[static_cast<long long>(ch) * N + sub * kPer + i] * DecayFn<T>::kPre : 0.f;
-    S[i] = active && carried ? sp[i] : 0.f;
+  for (int i = 0; i < kPer; i += 2) {
+    const float* a = p.a + static_cast<long long>(ch) * N + sub * kPer + i;
+    A[i / 2] = active ? pack2(a[0] * DecayFn<T>::kPre, a[1] * DecayFn<T>::kPre) : pack2(0.f, 0.f);
+    S[i / 2] = active && carried ? pack2(sp[i], sp[i + 1]) : pack2(0.f, 0.f);
   }
   // staging: one vector of eight channels of one token per thread, plus its share of B | C
   const int st_t = tid >> 2, st_c = (tid & 3) * 8;
@@ -320,7 +357,7 @@ __global__ void __launch_bounds__(128) channel_scan_kernel(const ChannelScanPara
         dt[i] = on ? softplus_f32(rdt[i] + bias[i]) : 0.f;
         dx[i] = dt[i] * rx[i];
         e[i] = dsk[i] * rx[i];
-        g[i] = silu_f32(rz[i]);
+        g[i] = silu_act<T>(rz[i]);
       }
       store8(&s_dt[st_t][st_c], dt);
       store8(&s_dx[st_t][st_c], dx);
@@ -344,14 +381,17 @@ __global__ void __launch_bounds__(128) channel_scan_kernel(const ChannelScanPara
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         const float dt = s_dt[t + j][cl], dx = s_dx[t + j][cl];
-        const float* b = &s_bc[t + j][sub * kPer];
-        float acc = 0.f;
+        const f32x2* b = reinterpret_cast<const f32x2*>(&s_bc[t + j][sub * kPer]);
+        const f32x2 dt2 = pack2(dt, dt), dx2 = pack2(dx, dx);
+        f32x2 acc = pack2(0.f, 0.f);
 #pragma unroll
-        for (int i = 0; i < kPer; ++i) {
-          S[i] = fmaf(DecayFn<T>::of(dt * A[i]), S[i], dx * b[i]);
-          acc = fmaf(S[i], b[N + i], acc);
+        for (int i = 0; i < kPer / 2; ++i) {
+          float e0, e1;
+          unpack2(mul2(dt2, A[i]), e0, e1);
+          S[i] = fma2(pack2(DecayFn<T>::of(e0), DecayFn<T>::of(e1)), S[i], mul2(dx2, b[i]));
+          acc = fma2(S[i], b[N / 2 + i], acc);
         }
-        part[j] = acc;
+        part[j] = sum2(acc);
       }
       // token (sub) of the four ends up in lane sub
       const bool hi = sub & 1, top = sub & 2;
@@ -372,7 +412,11 @@ __global__ void __launch_bounds__(128) channel_scan_kernel(const ChannelScanPara
   }
   if (active && slot >= 0)
 #pragma unroll
-    for (int i = 0; i < kPer; ++i) sp[i] = S[i];
+    for (int i = 0; i < kPer; i += 2) {
+      float a, b;
+      unpack2(S[i / 2], a, b);
+      *reinterpret_cast<float2*>(sp + i) = make_float2(a, b);
+    }
 }
 
 // Decode: grid (ceil(channels / 64), seqs), 256 threads
@@ -413,7 +457,7 @@ __global__ void __launch_bounds__(256) channel_step_kernel(const ChannelScanPara
   acc += __shfl_xor_sync(0xffffffffu, acc, 2);
   if (active && sub == 0) {
     const float z = ld1(static_cast<const T*>(p.z) + seq * p.ldz + ch);
-    static_cast<T*>(p.y)[seq * p.ldy + ch] = static_cast<T>((acc + p.d[ch] * x) * silu_f32(z));
+    static_cast<T*>(p.y)[seq * p.ldy + ch] = static_cast<T>((acc + p.d[ch] * x) * silu_act<T>(z));
   }
 }
 
@@ -433,6 +477,7 @@ struct HeadScanParams {
   void* y;                   // [T][ldy]
   long long ldx, ld_dt, ldy;
   int heads, groups, n, p, b_off, c_off, seqs, slices;
+  int min_len, max_len;      // runs of other lengths are another kernel's
 };
 
 constexpr int kHsTile = 16;                  // tokens per staged tile
@@ -448,7 +493,7 @@ __global__ void __launch_bounds__(128) head_scan_kernel(const HeadScanParams p) 
   pdl_trigger();
   const int head = blockIdx.x / p.slices, slice = blockIdx.x - head * p.slices, seq = blockIdx.y;
   const int slot = p.slots[seq], first = p.cu_q[seq], len = p.cu_q[seq + 1] - first;
-  if (len <= 0) return;
+  if (len <= 0 || len < p.min_len || len > p.max_len) return;
   const int tid = threadIdx.x, threads = blockDim.x, nl = tid % kNl, cg = tid / kNl;
   const int cols = threads / kNl * 4, col0 = slice * cols, col = col0 + cg * 4;
   float* s_bc = sm;
@@ -598,6 +643,251 @@ __global__ void __launch_bounds__(128) head_scan_kernel(const HeadScanParams p) 
     }
 }
 
+// Long runs, bf16. With l_t the running sum of the log decays inside a chunk of 64 tokens, S the state before it and
+// dt_s the step sizes:
+//   y_t = sum_{s <= t} (C_t . B_s) e^(l_t - l_s) dt_s x_s  +  e^(l_t) C_t S  +  D x_t
+//   S   = e^(l_end) S + sum_s (e^(l_end - l_s) dt_s B_s) x_s^T
+// Four products per chunk on the warp-level tensor cores, accumulated in fp32. B, C and x are bf16 as they come from
+// the convolution; what is computed in 32 bits (the weights of the first sum, the state, the weighted B) enters as a
+// bf16 head plus a bf16 remainder. The state itself stays in fp32 accumulators, transposed: warp w owns columns 16 w ..
+// of the slice, and its accumulator layout is the operand layout that the product with C wants.
+// grid (heads * slices of 64 columns, seqs), 128 threads.
+constexpr int kHcTok = 64, kHcCols = 64;
+
+template <int N>
+struct HeadChunkSmem {
+  static constexpr int kPitch = N * 2 + 16, kXPitch = kHcCols * 2 + 16;    // rows 16 bytes apart modulo 128
+  uint8_t b[kHcTok * kPitch], c[kHcTok * kPitch], wh[kHcTok * kPitch], wl[kHcTok * kPitch];
+  uint8_t x[kHcTok * kXPitch];
+  float y[kHcTok][kHcCols + 4];
+  float l[kHcTok], dt[kHcTok];
+};
+
+__device__ __forceinline__ uint32_t split_bf16x2(float a, float b, uint32_t& rest) {
+  const uint32_t h = pack_bf16x2(a, b);
+  const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&h));
+  rest = pack_bf16x2(a - f.x, b - f.y);
+  return h;
+}
+
+template <int N>
+__global__ void __launch_bounds__(128, 2) head_chunk_kernel(const HeadScanParams p) {
+  using Smem = HeadChunkSmem<N>;
+  constexpr int kPitch = Smem::kPitch, kXPitch = Smem::kXPitch, kK = N / 16;
+  extern __shared__ __align__(16) uint8_t raw[];
+  Smem& sm = *reinterpret_cast<Smem*>(raw);
+  pdl_wait();
+  const int head = blockIdx.x / p.slices, col0 = (blockIdx.x - head * p.slices) * kHcCols, seq = blockIdx.y;
+  const int slot = p.slots[seq], first = p.cu_q[seq], len = p.cu_q[seq + 1] - first;
+  if (len < p.min_len || len > p.max_len) {
+    pdl_trigger();
+    return;
+  }
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, tq = lane & 3, mi = lane >> 3;
+  const bool carried = slot >= 0 && p.positions[first] > 0;
+  const int group = head / (p.heads / p.groups);
+  const float rate = p.rate[head], dt_bias = p.dt_bias[head], dsk = p.d[head];
+  const auto* xp = static_cast<const __nv_bfloat16*>(p.x);
+  const auto* dtp = static_cast<const __nv_bfloat16*>(p.dt);
+  auto* yp = static_cast<__nv_bfloat16*>(p.y);
+  float* sp = p.state + (static_cast<long long>(slot < 0 ? 0 : slot) * p.heads + head) * N * p.p;
+  const int pc = col0 + warp * 16 + g;       // this thread's state columns: pc and pc + 8
+  float S[N / 8][4];                         // S^T: [8 n][column pc: n, n + 1; column pc + 8: n, n + 1]
+#pragma unroll
+  for (int j = 0; j < N / 8; ++j)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int n = j * 8 + tq * 2 + (e & 1), c = pc + 8 * (e >> 1);
+      S[j][e] = carried && c < p.p ? sp[static_cast<long long>(n) * p.p + c] : 0.f;
+    }
+  const uint32_t sb = smem_u32(sm.b), sc = smem_u32(sm.c), swh = smem_u32(sm.wh), swl = smem_u32(sm.wl), sx = smem_u32(sm.x);
+
+  for (int t0 = 0; t0 < len; t0 += kHcTok) {
+    const int nt = min(kHcTok, len - t0);
+    const long long row0 = first + t0;
+    for (int i = tid; i < kHcTok * (N / 8); i += 128) {
+      const int t = i / (N / 8), c = i % (N / 8);
+      const bool on = t < nt;
+      const __nv_bfloat16* src = xp + (on ? row0 + t : row0) * p.ldx + group * N + c * 8;
+      cp_async_16(sb + t * kPitch + c * 16, src + p.b_off, on);
+      cp_async_16(sc + t * kPitch + c * 16, src + p.c_off, on);
+    }
+    for (int i = tid; i < kHcTok * (kHcCols / 8); i += 128) {
+      const int t = i / (kHcCols / 8), c = i % (kHcCols / 8);
+      const bool on = t < nt && col0 + c * 8 < p.p;
+      cp_async_16(sx + t * kXPitch + c * 16, on ? xp + (row0 + t) * p.ldx + head * p.p + col0 + c * 8 : xp, on);
+    }
+    cp_async_commit();
+    if (warp == 0) {                         // step sizes and the running sum of log decays, two tokens per lane
+      float dt[2], l[2];
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int t = lane * 2 + e;
+        dt[e] = t < nt ? softplus_f32(ld1(dtp + (row0 + t) * p.ld_dt + head) + dt_bias) : 0.f;
+        l[e] = -rate * dt[e];
+      }
+      l[1] += l[0];
+      float sum = l[1];
+#pragma unroll
+      for (int o = 1; o < 32; o *= 2) {
+        const float u = __shfl_up_sync(0xffffffffu, sum, o);
+        if (lane >= o) sum += u;
+      }
+      const float before = sum - l[1];
+      sm.dt[lane * 2] = dt[0];
+      sm.dt[lane * 2 + 1] = dt[1];
+      sm.l[lane * 2] = before + l[0];
+      sm.l[lane * 2 + 1] = sum;
+    }
+    cp_async_wait<0>();
+    __syncthreads();
+    const float l_end = sm.l[kHcTok - 1];
+    // weighted B for the state's update
+    for (int i = tid; i < kHcTok * (N / 8); i += 128) {
+      const int t = i / (N / 8), c = i % (N / 8);
+      float v[8];
+      load8(reinterpret_cast<const __nv_bfloat16*>(sm.b + t * kPitch) + c * 8, v);
+      const float w = expf(l_end - sm.l[t]) * sm.dt[t];
+      uint4 h, r;
+      h.x = split_bf16x2(v[0] * w, v[1] * w, r.x);
+      h.y = split_bf16x2(v[2] * w, v[3] * w, r.y);
+      h.z = split_bf16x2(v[4] * w, v[5] * w, r.z);
+      h.w = split_bf16x2(v[6] * w, v[7] * w, r.w);
+      *reinterpret_cast<uint4*>(sm.wh + t * kPitch + c * 16) = h;
+      *reinterpret_cast<uint4*>(sm.wl + t * kPitch + c * 16) = r;
+    }
+    // tokens of the chunk on each other: rows 16 warp .., sixteen source tokens at a time
+    {
+      float y1[kHcCols / 8][4];
+#pragma unroll
+      for (int i = 0; i < kHcCols / 8; ++i)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) y1[i][e] = 0.f;
+      const int r0 = warp * 16 + g;
+      const float lt[2] = {sm.l[r0], sm.l[r0 + 8]};
+      for (int j = 0; j <= warp; ++j) {
+        float q[2][4];
+#pragma unroll
+        for (int i = 0; i < 2; ++i)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) q[i][e] = 0.f;
+#pragma unroll
+        for (int kk = 0; kk < kK; ++kk) {
+          uint32_t a[4], b0, b1, b2, b3;
+          ldmatrix_x4(sc + (warp * 16 + (lane & 15)) * kPitch + (kk * 2 + (lane >> 4)) * 16, a[0], a[1], a[2], a[3]);
+          ldmatrix_x4(sb + (j * 16 + (lane & 7) + 8 * (mi >> 1)) * kPitch + (kk * 2 + (mi & 1)) * 16, b0, b1, b2, b3);
+          mma_bf16_16816(q[0], a, b0, b1);
+          mma_bf16_16816(q[1], a, b2, b3);
+        }
+        uint32_t ah[4], al[4];
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          const int s0 = j * 16 + i * 8 + tq * 2;
+          const float ls[2] = {sm.l[s0], sm.l[s0 + 1]}, ds[2] = {sm.dt[s0], sm.dt[s0 + 1]};
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const int r = e >> 1, o = e & 1;
+            q[i][e] = s0 + o <= r0 + 8 * r ? q[i][e] * (expf(lt[r] - ls[o]) * ds[o]) : 0.f;
+          }
+          ah[i * 2] = split_bf16x2(q[i][0], q[i][1], al[i * 2]);
+          ah[i * 2 + 1] = split_bf16x2(q[i][2], q[i][3], al[i * 2 + 1]);
+        }
+#pragma unroll
+        for (int np = 0; np < kHcCols / 16; ++np) {
+          uint32_t b0, b1, b2, b3;
+          ldmatrix_x4_trans(sx + (j * 16 + (lane & 7) + 8 * (mi & 1)) * kXPitch + (np * 2 + (mi >> 1)) * 16, b0, b1, b2, b3);
+          mma_bf16_16816(y1[np * 2], ah, b0, b1);
+          mma_bf16_16816(y1[np * 2 + 1], ah, b2, b3);
+          mma_bf16_16816(y1[np * 2], al, b0, b1);
+          mma_bf16_16816(y1[np * 2 + 1], al, b2, b3);
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < kHcCols / 8; ++i)
+#pragma unroll
+        for (int r = 0; r < 2; ++r)
+          *reinterpret_cast<float2*>(&sm.y[r0 + 8 * r][i * 8 + tq * 2]) = make_float2(y1[i][2 * r], y1[i][2 * r + 1]);
+    }
+    __syncthreads();
+    // the state's contribution, columns 16 warp .. of every token
+    {
+      float y2[4][2][4];
+#pragma unroll
+      for (int m = 0; m < 4; ++m)
+#pragma unroll
+        for (int i = 0; i < 2; ++i)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) y2[m][i][e] = 0.f;
+#pragma unroll
+      for (int kk = 0; kk < kK; ++kk) {
+        uint32_t bh[2][2], bl[2][2];         // [column tile][k half]
+#pragma unroll
+        for (int i = 0; i < 2; ++i)
+#pragma unroll
+          for (int k = 0; k < 2; ++k) bh[i][k] = split_bf16x2(S[kk * 2 + k][i * 2], S[kk * 2 + k][i * 2 + 1], bl[i][k]);
+#pragma unroll
+        for (int m = 0; m < 4; ++m) {
+          uint32_t a[4];
+          ldmatrix_x4(sc + (m * 16 + (lane & 15)) * kPitch + (kk * 2 + (lane >> 4)) * 16, a[0], a[1], a[2], a[3]);
+#pragma unroll
+          for (int i = 0; i < 2; ++i) {
+            mma_bf16_16816(y2[m][i], a, bh[i][0], bh[i][1]);
+            mma_bf16_16816(y2[m][i], a, bl[i][0], bl[i][1]);
+          }
+        }
+      }
+#pragma unroll
+      for (int m = 0; m < 4; ++m)
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+          const int t = m * 16 + g + 8 * r;
+          const float e = expf(sm.l[t]);
+#pragma unroll
+          for (int i = 0; i < 2; ++i) {
+            const int c = warp * 16 + i * 8 + tq * 2;
+            if (t >= nt || col0 + c >= p.p) continue;
+            const float2 y1 = *reinterpret_cast<const float2*>(&sm.y[t][c]);
+            const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(sm.x + t * kXPitch + c * 2));
+            *reinterpret_cast<uint32_t*>(yp + (row0 + t) * p.ldy + head * p.p + col0 + c) =
+                pack_bf16x2(fmaf(e, y2[m][i][2 * r], y1.x) + dsk * x.x, fmaf(e, y2[m][i][2 * r + 1], y1.y) + dsk * x.y);
+          }
+        }
+    }
+    // the state after the chunk
+    const float keep = decay_of(-l_end);
+#pragma unroll
+    for (int j = 0; j < N / 8; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) S[j][e] *= keep;
+#pragma unroll
+    for (int kk = 0; kk < kHcTok / 16; ++kk) {
+      uint32_t a[4];
+      ldmatrix_x4_trans(sx + (kk * 16 + 8 * (mi >> 1) + (lane & 7)) * kXPitch + (warp * 2 + (mi & 1)) * 16, a[0], a[1], a[2], a[3]);
+      const uint32_t off = (kk * 16 + (lane & 7) + 8 * (mi & 1)) * kPitch + (mi >> 1) * 16;
+#pragma unroll
+      for (int np = 0; np < N / 16; ++np) {
+        uint32_t b0, b1, b2, b3;
+        ldmatrix_x4_trans(swh + off + np * 32, b0, b1, b2, b3);
+        mma_bf16_16816(S[np * 2], a, b0, b1);
+        mma_bf16_16816(S[np * 2 + 1], a, b2, b3);
+        ldmatrix_x4_trans(swl + off + np * 32, b0, b1, b2, b3);
+        mma_bf16_16816(S[np * 2], a, b0, b1);
+        mma_bf16_16816(S[np * 2 + 1], a, b2, b3);
+      }
+    }
+    __syncthreads();
+  }
+  pdl_trigger();
+  if (slot >= 0)
+#pragma unroll
+    for (int j = 0; j < N / 8; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int n = j * 8 + tq * 2 + (e & 1), c = pc + 8 * (e >> 1);
+        if (c < p.p) sp[static_cast<long long>(n) * p.p + c] = S[j][e];
+      }
+}
+
 // Decode: grid (heads, seqs), 256 threads; thread = (4 columns, every rg-th row). Dynamic shared memory:
 // [2n] B | C, [p] x, [row groups][p] partial sums.
 template <typename T>
@@ -701,7 +991,7 @@ __global__ void __launch_bounds__(1024) gated_norm_kernel(const GatedNormParams 
       }
 #pragma unroll
       for (int i = 0; i < 8; ++i) {
-        v[k][i] *= silu_f32(g[i]);
+        v[k][i] *= silu_act<T>(g[i]);
         q = fmaf(v[k][i], v[k][i], q);
       }
     }
@@ -721,13 +1011,13 @@ __global__ void __launch_bounds__(1024) gated_norm_kernel(const GatedNormParams 
   }
   for (int i = threadIdx.x; i < p.part; i += blockDim.x) {
     const int at = (lo + i) / p.p * p.pp + (lo + i) % p.p;
-    const float v = ld1(y + at) * silu_f32(ld1(z + at));
+    const float v = ld1(y + at) * silu_act<T>(ld1(z + at));
     q = fmaf(v, v, q);
   }
   const float inv = 1.f / sqrtf(block_sum(q, red) / p.part + p.eps);
   for (int i = threadIdx.x; i < p.part; i += blockDim.x) {
     const int at = (lo + i) / p.p * p.pp + (lo + i) % p.p;
-    out[at] = static_cast<T>(ld1(y + at) * silu_f32(ld1(z + at)) * inv * ld1(p.w + at));
+    out[at] = static_cast<T>(ld1(y + at) * silu_act<T>(ld1(z + at)) * inv * ld1(p.w + at));
   }
 }
 
@@ -785,13 +1075,41 @@ int launch_head_scan(HeadScanParams p, cudaStream_t stream) {
   const cudaError_t e = launch_pdl(head_scan_kernel<T, kNl>, dim3(p.heads * p.slices, p.seqs), dim3(threads), smem, stream, p);
   return e == cudaSuccess ? 0 : -static_cast<int>(e) - 300;
 }
+constexpr int kChunkRun = 48;                // shortest run that goes to head_chunk
+
+template <int N>
+int launch_head_chunk(HeadScanParams p, cudaStream_t stream) {
+  p.slices = (p.p + kHcCols - 1) / kHcCols;
+  p.min_len = kChunkRun;
+  p.max_len = 0x7fffffff;
+  const int smem = static_cast<int>(sizeof(HeadChunkSmem<N>));
+  static PerDeviceOnce once;
+  if (once.first_time()) cudaFuncSetAttribute(head_chunk_kernel<N>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+  const cudaError_t e = launch_pdl(head_chunk_kernel<N>, dim3(p.heads * p.slices, p.seqs), dim3(128), smem, stream, p);
+  return e == cudaSuccess ? 0 : -static_cast<int>(e) - 300;
+}
+
 template <typename T>
-int dispatch_head_scan(const HeadScanParams& p, cudaStream_t stream) {
+int dispatch_head_scan(HeadScanParams p, int longest, int shortest, cudaStream_t stream) {
   if (!p.cu_q) {
     const int rgs = 256 / (p.p / 4);
     const int smem = (2 * p.n + p.p + rgs * p.p) * 4;
     const cudaError_t e = launch_pdl(head_step_kernel<T>, dim3(p.heads, p.seqs), dim3(256), smem, stream, p);
     return e == cudaSuccess ? 0 : -static_cast<int>(e) - 300;
+  }
+  p.min_len = 0;
+  p.max_len = 0x7fffffff;
+  if (sizeof(T) == 2 && longest >= kChunkRun && p.n >= 16 && p.n <= 128) {      // long runs as chunks, the others here
+    int rc = -2;
+    switch (p.n) {
+      case 16: rc = launch_head_chunk<16>(p, stream); break;
+      case 32: rc = launch_head_chunk<32>(p, stream); break;
+      case 64: rc = launch_head_chunk<64>(p, stream); break;
+      case 128: rc = launch_head_chunk<128>(p, stream); break;
+      default: break;
+    }
+    if (rc || shortest >= kChunkRun) return rc;
+    p.max_len = kChunkRun - 1;
   }
   switch (p.n) {
     case 8: return launch_head_scan<T, 1>(p, stream);
@@ -858,17 +1176,17 @@ B200_API int b200_channel_scan(const void* x, const void* dt, const void* bc, co
 }
 
 // n in {8, 16, ..., 256}, hp (values per head) a multiple of 8 up to 512; offsets and row pitches (but ld_dt)
-// multiples of 8
+// multiples of 8. longest, shortest: bounds on the tokens of a run, 0 when not known (all runs are scanned)
 B200_API int b200_head_scan(const void* x, const void* dt, const float* dt_bias, const float* rate, const float* d, float* state,
                             const int* positions, const int* cu_q, const int* slots, void* y, int seqs, int heads, int groups,
-                            int n, int hp, int b_off, int c_off, long long ldx, long long ld_dt, long long ldy, int f32,
-                            cudaStream_t stream) {
+                            int n, int hp, int b_off, int c_off, long long ldx, long long ld_dt, long long ldy, int longest,
+                            int shortest, int f32, cudaStream_t stream) {
   if (seqs <= 0) return 0;
   if (hp % 8 || hp > 512 || n % 8 || n > 256 || heads % groups || b_off % 8 || c_off % 8 || ldx % 8 || ldy % 8 || seqs > 65535)
     return -2;
   HeadScanParams p{x, dt, dt_bias, rate, d, state, positions, cu_q, slots, y, ldx, ld_dt, ldy, heads, groups, n, hp, b_off,
-                   c_off, seqs, 1};
-  return f32 ? dispatch_head_scan<float>(p, stream) : dispatch_head_scan<__nv_bfloat16>(p, stream);
+                   c_off, seqs, 1, 0, 0};
+  return f32 ? dispatch_head_scan<float>(p, longest, shortest, stream) : dispatch_head_scan<__nv_bfloat16>(p, longest, shortest, stream);
 }
 
 // y, z, out [tokens][...] with heads of hp values laid out hpp apart; parts * part = heads * hp

@@ -237,7 +237,8 @@ class HeadScanMixer:
         cu = None if batch.is_decode else batch.cu_q
         i, s = self.inner, self.spec
         x = ops.short_conv(p[:, i:i + self.channels], self.conv, self.conv_bias, conv, batch.positions, cu, batch.state_slots)
-        y = ops.head_scan(x, p[:, i + self.channels:i + self.channels + s.heads], self.w, state, batch.positions, cu, batch.state_slots)
+        y = ops.head_scan(x, p[:, i + self.channels:i + self.channels + s.heads], self.w, state, batch.positions, cu, batch.state_slots,
+                          batch.runs if cu is not None else None)
         y = ops.gated_norm(y, p[:, :i], self.norm, s.norm_groups, self.eps, s.heads, s.vdim)
         return ops.linear_act(y, self.o)
 

@@ -56,7 +56,7 @@ _SIGNATURES = {
     "b200_poly_norm": (i32, [vp, vp, vp, i32, i32, i32, i32, f32, i32, vp]),
     "b200_short_conv": (i32, [vp] * 8 + [i32] * 4 + [i64, i32, vp]),
     "b200_channel_scan": (i32, [vp] * 12 + [i32] * 5 + [i64] * 5 + [i32, vp]),
-    "b200_head_scan": (i32, [vp] * 10 + [i32] * 7 + [i64] * 3 + [i32, vp]),
+    "b200_head_scan": (i32, [vp] * 10 + [i32] * 7 + [i64] * 3 + [i32, i32, i32, vp]),
     "b200_gated_norm": (i32, [vp] * 4 + [i32] * 5 + [i64] * 3 + [f32, i32, vp]),
     "b200_latent_prep": (i32, [vp] * 6 + [i32, i64] + [i32] * 6 + [f32, i32, vp]),
     "b200_latent_gather": (i32, [vp] * 5 + [i32] * 5 + [vp]),

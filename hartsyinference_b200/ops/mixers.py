@@ -379,10 +379,11 @@ class HeadScanWeights:
 
 
 def head_scan(x: torch.Tensor, dt: torch.Tensor, w: HeadScanWeights, state: torch.Tensor, positions: torch.Tensor,
-              cu_q: Optional[torch.Tensor], slots: torch.Tensor) -> torch.Tensor:
+              cu_q: Optional[torch.Tensor], slots: torch.Tensor, runs: Optional[list] = None) -> torch.Tensor:
     """Scan with a matrix state [n, p] per head: ``S = exp(-rate dt) S + B (dt x)^T``, ``y = S^T C + d x``,
     ``dt = softplus(logit + bias)``. ``x`` [T, heads p + 2 groups n] = x | B | C (head h reads group
     h // (heads / groups)), ``dt`` logits [T, heads]. ``state`` fp32 [slots, heads, n, p] is updated in place.
+    ``runs`` (host list of (tokens, ..) per sequence of a ragged batch) lets long bf16 runs go through the tensor cores.
     Returns [T, heads p]."""
     t = x.shape[0]
     if not x.is_cuda:
@@ -393,7 +394,8 @@ def head_scan(x: torch.Tensor, dt: torch.Tensor, w: HeadScanWeights, state: torc
     y = torch.empty(t, hp, dtype=x.dtype, device=x.device)
     rc = N.lib().b200_head_scan(x.data_ptr(), dt.data_ptr(), w.dt_bias.data_ptr(), w.rate.data_ptr(), w.d.data_ptr(), state.data_ptr(),
                                 positions.data_ptr(), N.ptr(cu_q), slots.data_ptr(), y.data_ptr(), slots.numel(), w.heads, w.groups, w.n,
-                                w.p, hp, hp + w.groups * w.n, x.stride(0), dt.stride(0), y.stride(0), _f32(x), N.stream())
+                                w.p, hp, hp + w.groups * w.n, x.stride(0), dt.stride(0), y.stride(0), max((r[0] for r in runs or ()), default=0),
+                                min((r[0] for r in runs or ()), default=0), _f32(x), N.stream())
     N.check(rc, "b200_head_scan")
     return y
 

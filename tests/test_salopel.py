@@ -12,7 +12,8 @@ import torch
 
 sys.path.insert(0, os.path.dirname(os.path.abspath(__file__)))
 import salopel_oracle as O  # noqa: E402
-from test_lududra import BF, F32, MODES, Pages, _Batch, _Holder, gen, logits_near, near, rel_err, rnd  # noqa: E402
+from test_lududra import BF, F32, MODES, Pages, _Holder, gen, logits_near, near, rel_err, rnd  # noqa: E402
+from test_lududra import _Batch as _PlainBatch  # noqa: E402
 
 from hartsyinference_b200 import ops  # noqa: E402
 from hartsyinference_b200.engine import LLMEngine, SamplingParams  # noqa: E402
@@ -22,6 +23,12 @@ from hartsyinference_b200.models.llm import mixers as M  # noqa: E402
 from hartsyinference_b200.models.llm.loader import load_llm, save_hf_checkpoint  # noqa: E402
 from hartsyinference_b200.models.llm.salopel import config_from, tensor_shapes  # noqa: E402
 from hartsyinference_b200.models.llm.transformer import DecoderModel  # noqa: E402
+
+
+class _Batch(_PlainBatch):
+    def __init__(self, dev, positions, slots, cu=None):
+        super().__init__(dev, positions, slots, cu)
+        self.runs = None if cu is None else [(b - a, None) for a, b in zip(cu, cu[1:])]
 
 
 # ------------------------------------------------------------------------------------ norms and stream
@@ -147,7 +154,7 @@ def run_cuts(m, state, hs, slots, cuts, dt, dev):
     return got
 
 
-CUTS = ((17, 0), (2, 5), (1, 2), (16, 1), (3, 9), (0, 2))
+CUTS = ((17, 0), (2, 5), (1, 2), (16, 1), (3, 9), (0, 2), (64, 3), (65, 1), (48, 0), (130, 2))
 CHANNEL_SIZES = [(32, 16, 4, 4), (20, 5, 1, 1), (72, 32, 9, 3), (40, 8, 16, 2), (33, 64, 3, 6), (8, 100, 2, 4), (100, 12, 5, 5)]
 HEAD_SIZES = [(4, 2, 16, 16, 2, 4), (3, 1, 32, 20, 1, 3), (6, 3, 8, 8, 4, 2), (2, 2, 128, 64, 2, 4), (5, 1, 40, 12, 3, 1), (2, 1, 200, 136, 1, 6),
               (1, 1, 64, 256, 1, 4), (8, 4, 12, 24, 8, 5), (6, 2, 20, 40, 6, 4)]
@@ -161,7 +168,7 @@ def test_channel_scan_mixer(mode, sizes):
     dev, dt = mode
     g = gen(sum(sizes))
     mix, t = channel_case(g, *sizes)
-    hs = [rnd(g, 45, WIDTH), rnd(g, 23, WIDTH)]
+    hs = [rnd(g, 352, WIDTH), rnd(g, 29, WIDTH)]
     wd = {"mix." + n: v.double() for n, v in t.items()}
     m = build_channel(mix, t, dev)
     state = used_slots(m, dt, dev)
@@ -177,7 +184,7 @@ def test_head_scan_mixer(mode, sizes):
     dev, dt = mode
     g = gen(sum(sizes))
     mix, t = head_case(g, *sizes)
-    hs = [rnd(g, 45, WIDTH), rnd(g, 23, WIDTH)]
+    hs = [rnd(g, 352, WIDTH), rnd(g, 29, WIDTH)]
     wd = {"mix." + n: v.double() for n, v in t.items()}
     m = build_head(mix, t, dev)
     state = used_slots(m, dt, dev)
