@@ -7,6 +7,9 @@
     python benchmarks/kernel_case.py attn_dense 4608 8
     python benchmarks/kernel_case.py delta 4 2048 16
     python benchmarks/kernel_case.py attn_window 4 2048 16 2 1024
+    python benchmarks/kernel_case.py channel_scan 4 2048 4096
+    python benchmarks/kernel_case.py head_scan 4 2048 64
+    python benchmarks/kernel_case.py latent 64 2048 16
 
 Inputs are larger than the L2 cache where the op is bandwidth bound but stay far below a few GB,
 so a full-metric capture (dozens of replays per launch) ends in about a minute. The status word is
@@ -325,7 +328,57 @@ def _attn_window(argv):
     print(f"attn_window: extended {a * 1e3:.1f} us, plain {b * 1e3:.1f} us")
 
 
-CASES = {"delta": _delta, "attn_window": _attn_window, "mla_proj": _mla_proj, "gemm_ar_large": _gemm_ar_large, "ag_gemm": _ag_gemm, "ulysses": _ulysses, "allreduce": _allreduce, "sample": _sample,
+def _scan_batch(seqs, n):
+    t, dev = seqs * n, "cuda"
+    cu = None if n == 1 else torch.arange(0, t + 1, n, dtype=torch.int32, device=dev)
+    return t, torch.full((t,), 5, dtype=torch.int32, device=dev), cu, torch.arange(seqs, dtype=torch.int32, device=dev)
+
+
+def _channel_scan(argv):
+    """channel_scan SEQS TOKENS CHANNELS: selective scan, 16 states per channel (TOKENS = 1: a decode step)."""
+    seqs, n, c = (int(v) for v in argv[:3])
+    t, pos, cu, slots = _scan_batch(seqs, n)
+    x, dt, z, bc = (torch.randn(t, w, device="cuda").to(torch.bfloat16) for w in (c, c, c, 32))
+    w = ops.ChannelScanWeights(a=-torch.rand(c, 16, device="cuda"), dt_bias=torch.full((c,), -4.0, device="cuda"), d=torch.ones(c, device="cuda"))
+    st = torch.zeros(seqs, c, 16, device="cuda")
+    ms = _time_cold(lambda: ops.channel_scan(x, dt, bc, 0, 16, z, w, st, pos, cu, slots))
+    print(f"channel_scan {seqs} x {n} tokens x {c} channels: {ms * 1e3:.1f} us")
+
+
+def _head_scan(argv):
+    """head_scan SEQS TOKENS HEADS [scan]: scan with one decay per head, state 128 x 64 (TOKENS = 1: a decode step;
+    "scan": token by token instead of chunks)."""
+    seqs, n, h = (int(v) for v in argv[:3])
+    t, pos, cu, slots = _scan_batch(seqs, n)
+    x, dt = torch.randn(t, h * 64 + 256, device="cuda").to(torch.bfloat16), torch.randn(t, h, device="cuda").to(torch.bfloat16)
+    w = ops.HeadScanWeights(rate=torch.rand(h, device="cuda"), dt_bias=torch.full((h,), -4.0, device="cuda"), d=torch.ones(h, device="cuda"),
+                            heads=h, groups=1, n=128, p=64)
+    st = torch.zeros(seqs, h, 128, 64, device="cuda")
+    runs = None if n == 1 or len(argv) > 3 else [(n, n)] * seqs
+    ms = _time_cold(lambda: ops.head_scan(x, dt, w, st, pos, cu, slots, runs))
+    print(f"head_scan {seqs} x {n} tokens x {h} heads: {ms * 1e3:.1f} us")
+
+
+def _latent(argv):
+    """latent SEQS CONTEXT HEADS [runs]: decode attention over cached latents of 512 values, or with "runs" the
+    attention of whole prompts over expanded keys and values."""
+    seqs, n, h = (int(v) for v in argv[:3])
+    dev, d, per = "cuda", 128, n // 16
+    lens = torch.full((seqs,), n, dtype=torch.int32, device=dev)
+    if len(argv) > 3:
+        t = seqs * n
+        q, kv, gate = (torch.randn(t, w * h * d, device=dev).to(torch.bfloat16) for w in (1, 2, 1))
+        out, at = torch.empty_like(q), torch.arange(0, t + 1, n, dtype=torch.int32, device=dev)
+        fn = lambda: ops.attn_runs(q, kv[:, :h * d], kv[:, h * d:], out, at[:-1], lens, at, lens, heads=h, max_q_len=n, scale=0.1, gate=gate)
+    else:
+        cache = torch.randn(seqs * per, 1, 16, 512, device=dev).to(torch.bfloat16)
+        table = torch.randperm(seqs * per, device=dev).to(torch.int32).reshape(seqs, per)
+        q = torch.randn(seqs, h * 512, device=dev).to(torch.bfloat16)
+        fn = lambda: ops.latent_attn(q, cache, table, lens, h, 0.05, max_kv_len=n)
+    print(f"latent {argv}: {_time_cold(fn) * 1e3:.1f} us")
+
+
+CASES = {"channel_scan": _channel_scan, "head_scan": _head_scan, "latent": _latent, "delta": _delta, "attn_window": _attn_window, "mla_proj": _mla_proj, "gemm_ar_large": _gemm_ar_large, "ag_gemm": _ag_gemm, "ulysses": _ulysses, "allreduce": _allreduce, "sample": _sample,
          "int8": _int8, "triplane": _triplane,
          "gemm_ar": _gemm_ar, "attn_dense": _attn_dense, "gemm": _gemm, "grouped": _grouped, "attn_decode": _attn_decode, "mla": _mla}
 
