@@ -15,8 +15,10 @@
 // (src/HartsyInference.Core/Backends/AttentionReference.cs): GQA, causal, sliding window,
 // logit soft-cap. The extended form of both kernels (template flag kExt) adds, each optional: a bias
 // by key distance from a per-head table, a per-head sink score that only enters the denominator,
-// values that are the keys themselves (one page plane), a sigmoid gate on the output, any head size
-// up to 128 that is a multiple of 8, and a row pitch for q. There the probabilities keep 16 bits of
+// values that are the keys themselves (one page plane), a sigmoid gate on the output, first tokens that
+// stay visible outside the window, key and value sizes up to 128 that are multiples of 8, and a row pitch
+// for q; over contiguous keys also a part of the key that all heads share, with the rotation of its query
+// side. There the probabilities keep 16 bits of
 // mantissa in the PV product (a bf16 head and a bf16 remainder). `attn_rows_kernel` computes the same
 // with plain fp32 arithmetic for models run in 32 bits and for shapes the tensor-core form leaves out.
 //
@@ -59,9 +61,16 @@ struct AttnParams {
   const __nv_bfloat16* gate;    // [tokens][gate_ld]: out *= sigmoid(gate), or null
   long long q_ld, gate_ld;      // row pitches in elements
   int dist_len, d, shared_kv;   // d: head size as stored; shared_kv: v is k
-  int dv;                       // size of values and output per head (d unless k, v are contiguous)
+  int dv;                       // size of values and output per head
   const int* q_lens;            // [seqs] with cu_q = [seqs] starts: the listed runs need not be adjacent; or null
   long long k_ld, v_ld;         // contiguous k, v: row pitches (head h at h * d, h * dv)
+  int keep;                     // window > 0: keys before this position are visible whatever the window
+  // contiguous k: columns from d_own on are the same for all heads, row pitch k2_ld (d_own = d: none). With
+  // rot_table [tokens][(d - d_own) / 2] (cos, sin) those columns of q are turned on the way in, pairs (2i, 2i + 1)
+  const __nv_bfloat16* k2;
+  const float2* rot_table;
+  long long k2_ld;
+  int d_own, rot_pairs;
   float cap_in, cap_out;        // softcap: cap_out * tanh(score / softcap), exp(2 score / softcap) = 2^(cap_in * q.k)
 };
 constexpr float kLog2e = 1.4426950408889634f;
@@ -132,10 +141,17 @@ __device__ __forceinline__ void ext_scores(float (&s)[NT][4], int key0, const in
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         const int key = key0 + nt * 8 + (j & 1);
-        if (key >= row_limit[j >> 1] || key < row_start[j >> 1]) s[nt][j] = -INFINITY;
+        if (key >= row_limit[j >> 1] || (key < row_start[j >> 1] && key >= p.keep)) s[nt][j] = -INFINITY;
       }
   }
 }
+
+// Tiles that a window leaves: [0, kept) of the first tokens, then [tile0, n). They are walked as one range that starts
+// at tile0 - kept; tile_at gives the tile of a step.
+__device__ __forceinline__ int kept_tiles(const AttnParams& p, int tile0) {
+  return min((p.keep + kTileTokens - 1) / kTileTokens, tile0);
+}
+__device__ __forceinline__ int tile_at(int step, int tile0, int kept) { return step < tile0 ? step - (tile0 - kept) : step; }
 
 // Shared-memory tile: [64 tokens][D] bf16, row pitch D * 2 bytes, 16-byte chunks XOR-swizzled with
 // (token & 7) so that ldmatrix rows of consecutive tokens hit different banks.
@@ -165,27 +181,29 @@ __device__ __forceinline__ void load_tile_paged(uint32_t smem_base, const __nv_b
     cp_async_16(smem_base + tile_off<D>(t, c), src, valid);
   }
 }
-// Stages the page ids of tile `tile` into ring slot (tile & 7). Tiles start on page boundaries
+// Stages the page ids of step `step` (tile `tile`) into ring slot (step & 7). Tiles start on page boundaries
 // because 64 is a multiple of every supported page size.
-__device__ __forceinline__ void stage_pages(int (*ring)[8], const int* table, int tile, int n_tiles,
+__device__ __forceinline__ void stage_pages(int (*ring)[8], const int* table, int step, int n_steps, int tile,
                                             int page_shift, int kv_len) {
   const int per_tile = kTileTokens >> page_shift;
-  if (tile < n_tiles && threadIdx.x < per_tile) {
+  if (step < n_steps && threadIdx.x < per_tile) {
     const int first = (tile * kTileTokens) >> page_shift;
     const int idx = first + threadIdx.x;
     const int last_page = (kv_len - 1) >> page_shift;
-    ring[tile & 7][threadIdx.x] = idx <= last_page ? table[idx] : 0;
+    ring[step & 7][threadIdx.x] = idx <= last_page ? table[idx] : 0;
   }
 }
 template <int D, bool kExt = false>
 __device__ __forceinline__ void load_tile_linear(uint32_t smem_base, const __nv_bfloat16* base,
-                                                 long long row_stride, int tok0, int kv_len, int d = D) {
+                                                 long long row_stride, int tok0, int kv_len, int d = D,
+                                                 const __nv_bfloat16* base2 = nullptr, long long stride2 = 0, int d_own = D) {
   constexpr int kChunks = D / 8;
   for (int i = threadIdx.x; i < kTileTokens * kChunks; i += kAttnThreads) {
     const int t = i / kChunks, c = i % kChunks;
     const int tok = tok0 + t;
     const bool valid = tok < kv_len && (!kExt || c * 8 < d);
     const __nv_bfloat16* src = valid ? base + tok * row_stride + c * 8 : base;
+    if (kExt && valid && c * 8 >= d_own) src = base2 + tok * stride2 + (c * 8 - d_own);
     cp_async_16(smem_base + tile_off<D>(t, c), src, valid);
   }
 }
@@ -242,7 +260,7 @@ __device__ __forceinline__ void warp_tile(WarpState<D>& st, const uint32_t (&qf)
   float mx[2] = {-INFINITY, -INFINITY};
   if (kExt) {
     const int first = tok0 + t_begin, last = first + NG * 16 - 1;
-    const bool open = last < min(row_limit[0], row_limit[1]) && first >= max(row_start[0], row_start[1]);
+    const bool open = last < min(row_limit[0], row_limit[1]) && (first >= max(row_start[0], row_start[1]) || last < p.keep);
     if (__all_sync(0xffffffffu, open)) ext_scores<NG * 2, false>(s, first + tq * 2, row_limit, row_start, p, row_bias);
     else ext_scores<NG * 2, true>(s, first + tq * 2, row_limit, row_start, p, row_bias);
   }
@@ -354,8 +372,9 @@ attn_decode_kernel(const AttnParams p) {
   const int n_tiles = (kv_len + kTileTokens - 1) / kTileTokens;
   const int start_key = p.window > 0 ? max(0, kv_len - p.window) : 0;
   const int tile0 = start_key / kTileTokens;                    // tiles before the window are not read
-  const int tiles_per_split = (n_tiles - tile0 + p.splits - 1) / p.splits;
-  const int tile_begin = tile0 + split * tiles_per_split;
+  const int kept = kExt ? kept_tiles(p, tile0) : 0;             // except those of the kept first tokens
+  const int tiles_per_split = (n_tiles - tile0 + kept + p.splits - 1) / p.splits;
+  const int tile_begin = tile0 - kept + split * tiles_per_split;
   const int tile_end = min(n_tiles, tile_begin + tiles_per_split);
   const int* table = p.block_table + static_cast<long long>(seq) * p.max_pages;
   const uint32_t smem_base = smem_u32(smem);
@@ -399,42 +418,43 @@ attn_decode_kernel(const AttnParams p) {
   }
 
   __shared__ int pg_ring[8][8];
-  auto issue = [&](int tile, int stage) {
-    if (tile < tile_end) {
-      const uint32_t kb = smem_base + stage * stage_bytes;
+  auto tile_of = [&](int step) { return kExt ? tile_at(step, tile0, kept) : step; };
+  auto stage = [&](int step) { stage_pages(pg_ring, table, step, tile_end, tile_of(step), p.page_shift, kv_len); };
+  auto issue = [&](int step, int slot) {
+    if (step < tile_end) {
+      const uint32_t kb = smem_base + slot * stage_bytes;
+      const int* pages = pg_ring[step & 7];
+      const int tok0 = tile_of(step) * kTileTokens;
       if (kExt) {
-        load_tile_paged<D, true>(kb, p.k, pg_ring[tile & 7], kvh, p.hkv, p.page_shift, tile * kTileTokens, kv_len, p.d);
-        if (!p.shared_kv)
-          load_tile_paged<D, true>(kb + kTileBytes, p.v, pg_ring[tile & 7], kvh, p.hkv, p.page_shift, tile * kTileTokens,
-                                   kv_len, p.d);
+        load_tile_paged<D, true>(kb, p.k, pages, kvh, p.hkv, p.page_shift, tok0, kv_len, p.d);
+        if (!p.shared_kv) load_tile_paged<D, true>(kb + kTileBytes, p.v, pages, kvh, p.hkv, p.page_shift, tok0, kv_len, p.dv);
         cp_async_commit();
         return;
       }
-      load_tile_paged<D>(kb, p.k, pg_ring[tile & 7], kvh, p.hkv, p.page_shift, tile * kTileTokens, kv_len);
-      load_tile_paged<D>(kb + kTileBytes, p.v, pg_ring[tile & 7], kvh, p.hkv, p.page_shift,
-                         tile * kTileTokens, kv_len);
+      load_tile_paged<D>(kb, p.k, pages, kvh, p.hkv, p.page_shift, tok0, kv_len);
+      load_tile_paged<D>(kb + kTileBytes, p.v, pages, kvh, p.hkv, p.page_shift, tok0, kv_len);
     }
     cp_async_commit();
   };
-  stage_pages(pg_ring, table, tile_begin, tile_end, p.page_shift, kv_len);
-  stage_pages(pg_ring, table, tile_begin + 1, tile_end, p.page_shift, kv_len);
-  stage_pages(pg_ring, table, tile_begin + 2, tile_end, p.page_shift, kv_len);
-  if (kStages > 3) stage_pages(pg_ring, table, tile_begin + 3, tile_end, p.page_shift, kv_len);
+  stage(tile_begin);
+  stage(tile_begin + 1);
+  stage(tile_begin + 2);
+  if (kStages > 3) stage(tile_begin + 3);
   __syncthreads();
 #pragma unroll
   for (int i = 0; i < kStages - 1; ++i) issue(tile_begin + i, i);
-  int stage = 0;
-  for (int tile = tile_begin; tile < tile_end; ++tile) {
+  int slot = 0;
+  for (int step = tile_begin; step < tile_end; ++step) {
     // these page ids are read by issue() in a later iteration, after two barriers
-    stage_pages(pg_ring, table, tile + (kStages > 3 ? kStages : 3), tile_end, p.page_shift, kv_len);
-    issue(tile + kStages - 1, (stage + kStages - 1) % kStages);
+    stage(step + (kStages > 3 ? kStages : 3));
+    issue(step + kStages - 1, (slot + kStages - 1) % kStages);
     cp_async_wait<kStages - 1>();
     __syncthreads();
-    const uint32_t kb = smem_base + stage * stage_bytes;
-    warp_tile<D, 1, kExt>(st, qf, kb, kExt && p.shared_kv ? kb : kb + kTileBytes, warp * 16, tile * kTileTokens, lim, start, p,
-                          row_bias);
+    const uint32_t kb = smem_base + slot * stage_bytes;
+    warp_tile<D, 1, kExt>(st, qf, kb, kExt && p.shared_kv ? kb : kb + kTileBytes, warp * 16, tile_of(step) * kTileTokens, lim, start,
+                          p, row_bias);
     __syncthreads();
-    stage = (stage + 1) % kStages;
+    slot = (slot + 1) % kStages;
   }
   cp_async_wait<0>();
   __syncthreads();
@@ -472,8 +492,8 @@ attn_decode_kernel(const AttnParams p) {
     }
     const int head = kvh * G + r;
     if (kExt && p.splits == 1) {
-      if (c < p.d)
-        p.out[(static_cast<long long>(seq) * p.hq + head) * p.d + c] =
+      if (c < p.dv)
+        p.out[(static_cast<long long>(seq) * p.hq + head) * p.dv + c] =
             __float2bfloat16((ll > 0.f ? acc / ll : 0.f) * gate_of(p, seq, head, c));
     } else if (p.splits == 1) {
       p.out[(static_cast<long long>(seq) * p.hq + head) * D + c] =
@@ -506,8 +526,8 @@ __global__ void attn_combine_kernel(const AttnParams p) {
       ll += p.ws_ml[(base + s) * 2 + 1] * f;
     }
     if (kExt) {
-      if (c < p.d)
-        p.out[(static_cast<long long>(seq) * p.hq + head) * p.d + c] =
+      if (c < p.dv)
+        p.out[(static_cast<long long>(seq) * p.hq + head) * p.dv + c] =
             __float2bfloat16((ll > 0.f ? acc / ll : 0.f) * gate_of(p, seq, head, c));
       continue;
     }
@@ -594,6 +614,20 @@ attn_prefill_kernel(const AttnParams p) {
       qf[kk][3] = row0 + 8 < q_len ? *reinterpret_cast<const uint32_t*>(qb + (row0 + 8) * rs + c0 + 8) : 0u;
     }
   }
+  if (kExt && !kPaged && p.rot_table) {
+    // a thread's values come in pairs of neighbours: turn those of the shared part
+#pragma unroll
+    for (int kk = 0; kk < D / 16; ++kk)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const int pair = (kk * 16 + tq * 2 + 8 * (i >> 1) - p.d_own) >> 1, row = row0 + 8 * (i & 1);
+        if (pair >= 0 && pair < p.rot_pairs && row < q_len) {
+          const float2 cs = p.rot_table[static_cast<long long>(q_off + row) * p.rot_pairs + pair];
+          const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&qf[kk][i]));
+          qf[kk][i] = pack_bf16x2(v.x * cs.x - v.y * cs.y, v.y * cs.x + v.x * cs.y);
+        }
+      }
+  }
   WarpState<D> st;
   st.init();
   int lim[2], start[2];
@@ -624,54 +658,59 @@ attn_prefill_kernel(const AttnParams p) {
   const int n_tiles = (kv_needed + kTileTokens - 1) / kTileTokens;
   int tile0 = 0;
   if (p.window > 0) tile0 = max(0, ctx + qt * 64 + 1 - p.window) / kTileTokens;
+  const int kept = kExt ? kept_tiles(p, tile0) : 0;
 
   const int* table = kPaged ? p.block_table + static_cast<long long>(seq) * p.max_pages : nullptr;
   const int kv_off = (!kPaged && p.cu_kv) ? p.cu_kv[seq] : 0;
   const long long kv_rs = static_cast<long long>(p.hkv) * D;
-  const __nv_bfloat16* kbase = kPaged ? p.k : kExt ? p.k + kv_off * p.k_ld + kvh * p.d : p.k + (static_cast<long long>(kv_off) * p.hkv + kvh) * D;
+  const __nv_bfloat16* kbase = kPaged ? p.k : kExt ? p.k + kv_off * p.k_ld + kvh * p.d_own : p.k + (static_cast<long long>(kv_off) * p.hkv + kvh) * D;
+  const __nv_bfloat16* k2base = kExt && !kPaged && p.k2 ? p.k2 + kv_off * p.k2_ld : nullptr;
   const __nv_bfloat16* vbase = kPaged ? p.v : kExt ? p.v + kv_off * p.v_ld + kvh * p.dv : p.v + (static_cast<long long>(kv_off) * p.hkv + kvh) * D;
 
   __shared__ int pg_ring[8][8];
-  auto issue = [&](int tile, int stage) {
-    if (tile < n_tiles) {
-      const uint32_t kb = smem_base + stage * stage_bytes;
+  auto tile_of = [&](int step) { return kExt ? tile_at(step, tile0, kept) : step; };
+  auto stage = [&](int step) { stage_pages(pg_ring, table, step, n_tiles, tile_of(step), p.page_shift, kv_needed); };
+  auto issue = [&](int step, int slot) {
+    if (step < n_tiles) {
+      const uint32_t kb = smem_base + slot * stage_bytes;
+      const int* pages = pg_ring[step & 7];
+      const int tok0 = tile_of(step) * kTileTokens;
       if (kExt && !kPaged) {
-        load_tile_linear<D, true>(kb, kbase, p.k_ld, tile * kTileTokens, kv_needed, p.d);
-        load_tile_linear<D, true>(kb + kTileBytes, vbase, p.v_ld, tile * kTileTokens, kv_needed, p.dv);
+        load_tile_linear<D, true>(kb, kbase, p.k_ld, tok0, kv_needed, p.d, k2base, p.k2_ld, p.d_own);
+        load_tile_linear<D, true>(kb + kTileBytes, vbase, p.v_ld, tok0, kv_needed, p.dv);
       } else if (kExt) {
-        load_tile_paged<D, true>(kb, p.k, pg_ring[tile & 7], kvh, p.hkv, p.page_shift, tile * kTileTokens, kv_needed, p.d);
-        if (!p.shared_kv)
-          load_tile_paged<D, true>(kb + kTileBytes, p.v, pg_ring[tile & 7], kvh, p.hkv, p.page_shift, tile * kTileTokens,
-                                   kv_needed, p.d);
+        load_tile_paged<D, true>(kb, p.k, pages, kvh, p.hkv, p.page_shift, tok0, kv_needed, p.d);
+        if (!p.shared_kv) load_tile_paged<D, true>(kb + kTileBytes, p.v, pages, kvh, p.hkv, p.page_shift, tok0, kv_needed, p.dv);
       } else if (kPaged) {
-        load_tile_paged<D>(kb, p.k, pg_ring[tile & 7], kvh, p.hkv, p.page_shift, tile * kTileTokens, kv_needed);
-        load_tile_paged<D>(kb + kTileBytes, p.v, pg_ring[tile & 7], kvh, p.hkv, p.page_shift,
-                           tile * kTileTokens, kv_needed);
+        load_tile_paged<D>(kb, p.k, pages, kvh, p.hkv, p.page_shift, tok0, kv_needed);
+        load_tile_paged<D>(kb + kTileBytes, p.v, pages, kvh, p.hkv, p.page_shift, tok0, kv_needed);
       } else {
-        load_tile_linear<D>(kb, kbase, kv_rs, tile * kTileTokens, kv_needed);
-        load_tile_linear<D>(kb + kTileBytes, vbase, kv_rs, tile * kTileTokens, kv_needed);
+        load_tile_linear<D>(kb, kbase, kv_rs, tok0, kv_needed);
+        load_tile_linear<D>(kb + kTileBytes, vbase, kv_rs, tok0, kv_needed);
       }
     }
     cp_async_commit();
   };
+  const int first = tile0 - kept;
   if (kPaged) {
-    stage_pages(pg_ring, table, tile0, n_tiles, p.page_shift, kv_needed);
-    stage_pages(pg_ring, table, tile0 + 1, n_tiles, p.page_shift, kv_needed);
+    stage(first);
+    stage(first + 1);
     __syncthreads();
   }
-  issue(tile0, 0);
-  int stage = 0;
-  for (int tile = tile0; tile < n_tiles; ++tile) {
-    if (kPaged) stage_pages(pg_ring, table, tile + 2, n_tiles, p.page_shift, kv_needed);
-    issue(tile + 1, stage ^ 1);
+  issue(first, 0);
+  int slot = 0;
+  for (int step = first; step < n_tiles; ++step) {
+    if (kPaged) stage(step + 2);
+    issue(step + 1, slot ^ 1);
     cp_async_wait<1>();
     __syncthreads();
-    const uint32_t kb = smem_base + stage * stage_bytes;
+    const uint32_t kb = smem_base + slot * stage_bytes;
     // a warp whose rows all lie before this tile (causal) still runs: masked scores cost nothing
     // in correctness and keep the barrier pattern uniform
-    warp_tile<D, 4, kExt>(st, qf, kb, kExt && p.shared_kv ? kb : kb + kTileBytes, 0, tile * kTileTokens, lim, start, p, row_bias);
+    warp_tile<D, 4, kExt>(st, qf, kb, kExt && p.shared_kv ? kb : kb + kTileBytes, 0, tile_of(step) * kTileTokens, lim, start, p,
+                          row_bias);
     __syncthreads();
-    stage ^= 1;
+    slot ^= 1;
   }
   cp_async_wait<0>();
   static_assert(kStages == 2, "double buffered");
@@ -711,8 +750,9 @@ struct AttnRowsParams {
   long long q_ld, gate_ld;
   int tokens, seqs, hq, hkv, d, page, max_pages, window, dist_len;
   float scale, softcap;
+  int keep, dv, v_row;         // kept first tokens; value size, and values per row of the value pages
 };
-constexpr int kRowsMaxD = 512;
+constexpr int kRowsMaxD = 1024, kRowsMaxV = 512;   // query-key and value size
 
 __device__ __forceinline__ float as_f32(float v) { return v; }
 __device__ __forceinline__ float as_f32(__nv_bfloat16 v) { return __bfloat162float(v); }
@@ -738,22 +778,23 @@ __global__ void __launch_bounds__(128) attn_rows_kernel(const AttnRowsParams p) 
   }
   const int pos = p.kv_lens[seq] - q_len + (t - first);      // -1 for an empty sequence: no keys
   const int begin = p.window > 0 ? max(0, pos + 1 - p.window) : 0;
+  const int kept = min(p.keep, begin), keys = kept + pos + 1 - begin;       // [0, kept) and [begin, pos]
   const int kvh = head / (p.hq / p.hkv);
   const int* table = p.block_table + static_cast<long long>(seq) * p.max_pages;
   const T* q = static_cast<const T*>(p.q) + t * p.q_ld + head * p.d;
   for (int c = lane; c < p.d; c += 32) qs[warp][c] = as_f32(q[c]);
   __syncwarp();
   float m = p.sinks ? p.sinks[head] : -INFINITY, l = p.sinks ? 1.f : 0.f;
-  float o[kRowsMaxD / 32];
+  float o[kRowsMaxV / 32];
 #pragma unroll
-  for (int i = 0; i < kRowsMaxD / 32; ++i) o[i] = 0.f;
-  for (int j0 = begin; j0 <= pos; j0 += 32) {
-    const int j = j0 + lane;
+  for (int i = 0; i < kRowsMaxV / 32; ++i) o[i] = 0.f;
+  for (int j0 = 0; j0 < keys; j0 += 32) {
+    const int j = j0 + lane < kept ? j0 + lane : begin + j0 + lane - kept;
     long long at = 0;
     float s = -INFINITY;
-    if (j <= pos) {
-      at = ((static_cast<long long>(table[j / p.page]) * p.hkv + kvh) * p.page + j % p.page) * p.d;
-      const T* kr = static_cast<const T*>(p.k) + at;
+    if (j0 + lane < keys) {
+      at = (static_cast<long long>(table[j / p.page]) * p.hkv + kvh) * p.page + j % p.page;
+      const T* kr = static_cast<const T*>(p.k) + at * p.d;
       float a = 0.f;
       for (int c = 0; c < p.d; ++c) a += qs[warp][c] * as_f32(kr[c]);
       s = a * p.scale;
@@ -766,22 +807,22 @@ __global__ void __launch_bounds__(128) attn_rows_kernel(const AttnRowsParams p) 
     l = l * f + warp_sum(e);
     m = mn;
 #pragma unroll
-    for (int i = 0; i < kRowsMaxD / 32; ++i) o[i] *= f;
-    const int n = min(32, pos - j0 + 1);
+    for (int i = 0; i < kRowsMaxV / 32; ++i) o[i] *= f;
+    const int n = min(32, keys - j0);
     for (int jj = 0; jj < n; ++jj) {
       const float w = __shfl_sync(0xffffffffu, e, jj);
-      const T* vr = static_cast<const T*>(p.v) + __shfl_sync(0xffffffffu, at, jj);
+      const T* vr = static_cast<const T*>(p.v) + __shfl_sync(0xffffffffu, at, jj) * p.v_row;
 #pragma unroll
-      for (int i = 0; i < kRowsMaxD / 32; ++i)
-        if (lane + i * 32 < p.d) o[i] += w * as_f32(vr[lane + i * 32]);
+      for (int i = 0; i < kRowsMaxV / 32; ++i)
+        if (lane + i * 32 < p.dv) o[i] += w * as_f32(vr[lane + i * 32]);
     }
   }
-  T* out = static_cast<T*>(p.out) + (static_cast<long long>(t) * p.hq + head) * p.d;
-  const T* gate = p.gate ? static_cast<const T*>(p.gate) + t * p.gate_ld + head * p.d : nullptr;
+  T* out = static_cast<T*>(p.out) + (static_cast<long long>(t) * p.hq + head) * p.dv;
+  const T* gate = p.gate ? static_cast<const T*>(p.gate) + t * p.gate_ld + head * p.dv : nullptr;
 #pragma unroll
-  for (int i = 0; i < kRowsMaxD / 32; ++i) {
+  for (int i = 0; i < kRowsMaxV / 32; ++i) {
     const int c = lane + i * 32;
-    if (c < p.d) {
+    if (c < p.dv) {
       float y = l > 0.f ? o[i] / l : 0.f;
       if (gate) y *= 1.f / (1.f + expf(-as_f32(gate[c])));
       out[c] = static_cast<T>(y);
@@ -949,28 +990,31 @@ B200_API int b200_attn_prefill(const void* q, const void* k, const void* v, void
 }
 
 // Extended attention over pages (see the header comment). cu_q null: one query token per sequence.
-// q [tokens][q_ld] (head h at h * d), out [tokens][hq * d]. v_cache null: the values are the keys.
+// q [tokens][q_ld] (head h at h * d), out [tokens][hq * dv]. v_cache null: the values are the keys (with exact, their
+// first dv columns). window > 0: the last `window` keys and the first keep_first of the sequence.
 // exact != 0: plain fp32 kernel, tensors are fp32 when f32 is set and bf16 otherwise; exact == 0: the
-// tensor-core kernels (bf16, d <= 128, at most 16 query heads per key head at decode; returns -6 for
+// tensor-core kernels (bf16, d, dv <= 128, at most 16 query heads per key head at decode; returns -6 for
 // what they do not take). splits / workspace: decode only, as in b200_attn_decode (with the head size
 // rounded up to 64 or 128).
 B200_API int b200_attn_biased(const void* q, const void* k_cache, const void* v_cache, void* out, const int* block_table,
                               const int* kv_lens, const int* cu_q, int tokens, int seqs, int max_q_len, int hq, int hkv, int d,
-                              int page, int max_pages, int splits, void* workspace, float scale, float softcap, int window,
+                              int dv, int page, int max_pages, int splits, void* workspace, float scale, float softcap, int window, int keep_first,
                               const float* dist_bias, int dist_len, const float* sinks, const void* gate, long long gate_ld,
                               long long q_ld, int exact, int f32, cudaStream_t stream) {
   if (tokens <= 0 || seqs <= 0) return 0;
-  if (d % 8 || d < 8 || d > kRowsMaxD || hq % hkv || q_ld % 8 || (gate && gate_ld % 8) || (dist_bias && dist_len < 1)) return -2;
+  if (d % 8 || d < 8 || d > kRowsMaxD || dv % 8 || dv < 8 || dv > kRowsMaxV || (!v_cache && dv > d) || keep_first < 0 || hq % hkv || q_ld % 8 || (gate && gate_ld % 8) || (dist_bias && dist_len < 1)) return -2;
   if (f32 && !exact) return -6;
+  if (window <= 0) keep_first = 0;
   if (exact) {
     AttnRowsParams p{q, k_cache, v_cache ? v_cache : k_cache, gate, out, block_table, kv_lens, cu_q, dist_bias, sinks,
-                     q_ld, gate_ld, tokens, seqs, hq, hkv, d, page, max_pages, window, dist_len, scale, softcap};
+                     q_ld, gate_ld, tokens, seqs, hq, hkv, d, page, max_pages, window, dist_len, scale, softcap,
+                     keep_first, dv, v_cache ? dv : d};
     const dim3 grid((tokens + 3) / 4, hq);
     const cudaError_t e = f32 ? launch_pdl(attn_rows_kernel<float>, grid, dim3(128), 0, stream, p)
                               : launch_pdl(attn_rows_kernel<__nv_bfloat16>, grid, dim3(128), 0, stream, p);
     return e == cudaSuccess ? 0 : -static_cast<int>(e) - 300;
   }
-  if (d > 128 || (!cu_q && hq / hkv > 16)) return -6;
+  if (d > 128 || dv > 128 || (!v_cache && dv != d) || (!cu_q && hq / hkv > 16)) return -6;
   AttnParams p{};
   p.q = static_cast<const __nv_bfloat16*>(q);
   p.k = static_cast<const __nv_bfloat16*>(k_cache);
@@ -994,9 +1038,9 @@ B200_API int b200_attn_biased(const void* q, const void* k_cache, const void* v_
   }
   p.dist_bias = dist_bias; p.dist_len = dist_len; p.sinks = sinks;
   p.gate = static_cast<const __nv_bfloat16*>(gate);
-  p.gate_ld = gate_ld; p.q_ld = q_ld; p.d = p.dv = d;
+  p.gate_ld = gate_ld; p.q_ld = q_ld; p.d = p.d_own = d; p.dv = dv; p.keep = keep_first;
   p.splits = cu_q || splits < 1 ? 1 : splits;
-  const int dd = d <= 64 ? 64 : 128;
+  const int dd = d <= 64 && dv <= 64 ? 64 : 128;
   if (cu_q) {
     if (max_q_len <= 0) return 0;
     const dim3 grid((max_q_len + 63) / 64, hq, seqs);
@@ -1041,16 +1085,19 @@ B200_API int b200_attn_biased(const void* q, const void* k_cache, const void* v_
 }
 
 // Causal attention of the runs q_start[s] .. + q_lens[s] of q over contiguous keys and values of their whole
-// contexts (rows kv_start[s] .. + kv_lens[s] of k and v; the last key belongs to the run's last query). q, out and
-// gate are indexed by token: q [tokens][q_ld] (head h at h * d), out [tokens][hq * dv]. d, dv <= 128, multiples of 8.
+// contexts (rows kv_start[s] .. + kv_lens[s] of k and v; the last key belongs to the run's last query; window > 0: the
+// last `window` keys of every query). q, out and gate are indexed by token: q [tokens][q_ld] (head h at h * d), out
+// [tokens][hq * dv]. d, dv <= 128, multiples of 8. The keys' columns from d_own on are rows of k2 for every head
+// (d_own = d: none); with rot_table [tokens][rot_pairs] (cos, sin) those columns of q are turned.
 B200_API int b200_attn_runs(const void* q, const void* k, const void* v, void* out, const void* gate, const int* q_start,
                             const int* q_lens, const int* kv_start, const int* kv_lens, int seqs, int max_q_len, int hq, int hkv,
-                            int d, int dv, long long q_ld, long long k_ld, long long v_ld, long long gate_ld, float scale,
-                            cudaStream_t stream) {
+                            int d, int dv, long long q_ld, long long k_ld, long long v_ld, long long gate_ld, float scale, int window,
+                            const void* k2, int d_own, long long k2_ld, const void* rot_table, int rot_pairs, cudaStream_t stream) {
   if (seqs <= 0 || max_q_len <= 0) return 0;
   if (d % 8 || dv % 8 || d < 8 || dv < 8 || d > 128 || dv > 128 || hq % hkv || q_ld % 8 || k_ld % 8 || v_ld % 8 || gate_ld % 8 ||
       seqs > 65535)
     return -2;
+  if (d_own % 8 || d_own > d || k2_ld % 8 || (d_own < d && !k2) || (rot_table && 2 * rot_pairs > d - d_own)) return -2;
   AttnParams p{};
   p.q = static_cast<const __nv_bfloat16*>(q);
   p.k = static_cast<const __nv_bfloat16*>(k);
@@ -1060,20 +1107,21 @@ B200_API int b200_attn_runs(const void* q, const void* k, const void* v, void* o
   p.cu_q = q_start; p.q_lens = q_lens; p.cu_kv = kv_start; p.kv_lens = kv_lens;
   p.seqs = seqs; p.hq = hq; p.hkv = hkv; p.splits = 1;
   p.causal = 1;
+  p.window = window;
   p.scale = scale;
   p.scale_log2 = scale * kLog2e;
   p.d = d; p.dv = dv; p.q_ld = q_ld; p.k_ld = k_ld; p.v_ld = v_ld; p.gate_ld = gate_ld;
+  p.k2 = static_cast<const __nv_bfloat16*>(k2); p.d_own = d_own; p.k2_ld = k2_ld;
+  p.rot_table = static_cast<const float2*>(rot_table); p.rot_pairs = rot_pairs;
   const dim3 grid((max_q_len + 63) / 64, hq, seqs);
+  auto go = [&](auto kernel, int dd, PerDeviceOnce& once) {
+    const int smem = 2 * 2 * kTileTokens * dd * 2;
+    if (once.first_time()) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    kernel<<<grid, kAttnThreads, smem, stream>>>(p);
+  };
   static PerDeviceOnce once[2];
-  if (d > 64 || dv > 64) {
-    const int smem = 2 * 2 * kTileTokens * 128 * 2;
-    if (once[1].first_time()) cudaFuncSetAttribute(attn_prefill_kernel<128, false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
-    attn_prefill_kernel<128, false, true><<<grid, kAttnThreads, smem, stream>>>(p);
-  } else {
-    const int smem = 2 * 2 * kTileTokens * 64 * 2;
-    if (once[0].first_time()) cudaFuncSetAttribute(attn_prefill_kernel<64, false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
-    attn_prefill_kernel<64, false, true><<<grid, kAttnThreads, smem, stream>>>(p);
-  }
+  if (d > 64 || dv > 64) go(attn_prefill_kernel<128, false, true>, 128, once[1]);
+  else go(attn_prefill_kernel<64, false, true>, 64, once[0]);
   const cudaError_t e = cudaGetLastError();
   return e == cudaSuccess ? 0 : -static_cast<int>(e) - 300;
 }

@@ -484,5 +484,9 @@ __device__ __forceinline__ float gelu_tanh(float x) {
   return 0.5f * x * (1.f + tanhf(k0 * (x + k1 * x * x * x)));
 }
 __device__ __forceinline__ float silu(float x) { return x / (1.f + __expf(-x)); }
+__device__ __forceinline__ float relu2(float x) {
+  const float r = fmaxf(x, 0.f);
+  return r * r;
+}
 
 }  // namespace b200

@@ -191,7 +191,7 @@ struct GemmParams {
   const __nv_bfloat16* bias;      // per output feature (column of C), may be null
   const __nv_bfloat16* gate;      // per output feature multiplicative gate, may be null
   const __nv_bfloat16* residual;  // same layout as C, may be null
-  int act;                        // 0 none, 1 gelu-tanh, 2 silu
+  int act;                        // 0 none, 1 gelu-tanh, 2 silu, 3 relu squared
   // fp8 block scales, K-contiguous: scale(row, kb) = s[(row / gran) * ld + kb], ld = K / 128.
   // A thread walks one row's scales along K, so consecutive k-blocks hit the same cache line.
   const float* scale_a;
@@ -303,6 +303,7 @@ __device__ __forceinline__ float apply_epilogue(const GemmParams& p, float v, lo
   if (p.bias) v += __bfloat162float(p.bias[col]);
   if (p.act == 1) v = gelu_tanh(v);
   else if (p.act == 2) v = silu(v);
+  else if (p.act == 3) v = relu2(v);
   if (p.gate) v *= __bfloat162float(p.gate[col]);
   if (p.residual) v += __bfloat162float(p.residual[row * p.ldc + col]);
   return v;

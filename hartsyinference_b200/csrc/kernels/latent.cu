@@ -1,15 +1,17 @@
-// Pieces of latent attention without positions (no rotated part), any head count and sizes.
+// Pieces of latent attention, with or without a rotated part, any head count and sizes.
 //
-// Per token the cache holds one RMS-normed latent c; per head k = W_uk c and v = W_uv c. Queries come through a
+// Per token the cache holds one RMS-normed latent c; per head k = W_uk c and v = W_uv c. With a rotated part the row
+// goes on with one rotated key vector that all heads share, and each head's query has a part of that size. Queries come through a
 // normed latent of their own. Decoding and short runs attend over the cached latents with W_uk moved to the query
 // side and W_uv behind the softmax (mla.cu); long runs of a prompt expand keys and values of their context once
 // (attention.cu, the contiguous form).
 //
-//  * latent_prep    both latents' RMS norms in one launch: the query latent to a dense matrix, the key / value
-//                   latent straight into its page.
-//  * latent_gather  cached latents of whole sequences, in order, for the expansion.
+//  * latent_prep    both latents' RMS norms and the key's rotation in one launch: the query latent to a dense
+//                   matrix, the key / value latent and the rotated key straight into their page.
+//  * latent_gather  cached rows of sequences (from a given token on), in order, for the expansion.
 //  * head_linear    one small product per head, out[t][h] = W[h] x[t][h], optionally times sigmoid(gate): the
-//                   query-side W_uk, and W_uv with the output gate in its epilogue. Warp-level mma.sync: with at
+//                   query-side W_uk (its first column block also turns the query's rotated part and moves it behind
+//                   the product), and W_uv with the output gate in its epilogue. Warp-level mma.sync: with at
 //                   most a few hundred rows per head it is bound by reading the weights.
 #include "mixer_common.cuh"
 #include "mma_sync.cuh"
@@ -25,6 +27,8 @@ struct LatentPrepParams {
   long long ld;
   int tokens, q_off, q_dim, q_cols, kv_off, kv_dim, kv_cols;    // dims: true sizes; cols: laid out (rest zero)
   float eps;
+  const float2* table;       // [T][rot / 2] (cos, sin) of the key's rotated part behind the latent, pairs (2i, 2i + 1)
+  int rot, rot_cols;         // its true and laid-out size (0: none); cache rows are kv_cols + rot_cols long
 };
 
 // One warp per (token, latent): even warps the query's, odd warps the cached one. 256 threads.
@@ -41,7 +45,19 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const LatentPrepParams
   if (kv) {
     const long long slot = p.slots[t];
     if (slot < 0) return;
-    dst = static_cast<T*>(p.cache) + slot * cols;
+    dst = static_cast<T*>(p.cache) + slot * (cols + p.rot_cols);
+    const T* rs = static_cast<const T*>(p.p) + t * p.ld + p.kv_off + cols;
+    for (int i = lane; i < p.rot_cols / 2; i += 32) {
+      float a = 0.f, b = 0.f;
+      if (2 * i < p.rot) {
+        const float2 cs = p.table[t * (p.rot / 2) + i];
+        const float u = ld1(rs + 2 * i), v = ld1(rs + 2 * i + 1);
+        a = u * cs.x - v * cs.y;
+        b = v * cs.x + u * cs.y;
+      }
+      dst[cols + 2 * i] = static_cast<T>(a);
+      dst[cols + 2 * i + 1] = static_cast<T>(b);
+    }
   }
   const T* src = static_cast<const T*>(p.p) + t * p.ld + (kv ? p.kv_off : p.q_off);
   const __nv_bfloat16* w = kv ? p.wkv : p.wq;
@@ -77,18 +93,20 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const LatentPrepParams
   }
 }
 
-// out[off[s] + i] = cache row of token i of sequence seq_ids[s]; 16 bytes per thread. grid (blocks, seqs)
+// out[off[s] + i] = cache row of token starts[s] + i of sequence seq_ids[s]; 16 bytes per thread. grid (blocks, seqs)
 __global__ void __launch_bounds__(256) latent_gather_kernel(const uint8_t* __restrict__ cache, uint8_t* __restrict__ out,
                                                             const int* __restrict__ block_table, const int* __restrict__ seq_ids,
-                                                            const int* __restrict__ offsets, int vecs, int page, int max_pages) {
+                                                            const int* __restrict__ offsets, const int* __restrict__ starts, int vecs,
+                                                            int page, int max_pages) {
   pdl_wait();
   pdl_trigger();
-  const int s = blockIdx.y, off = offsets[s], n = offsets[s + 1] - off;
+  const int s = blockIdx.y, off = offsets[s], n = offsets[s + 1] - off, first = starts ? starts[s] : 0;
   const int* table = block_table + static_cast<long long>(seq_ids[s]) * max_pages;
   for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < static_cast<long long>(n) * vecs;
        i += static_cast<long long>(gridDim.x) * blockDim.x) {
     const int t = static_cast<int>(i / vecs), c = static_cast<int>(i % vecs);
-    const long long row = static_cast<long long>(table[t / page]) * page + t % page;
+    const int at = first + t;
+    const long long row = static_cast<long long>(table[at / page]) * page + at % page;
     reinterpret_cast<uint4*>(out)[(off + t) * static_cast<long long>(vecs) + c] = reinterpret_cast<const uint4*>(cache)[row * vecs + c];
   }
 }
@@ -102,7 +120,33 @@ struct HeadLinearParams {
   const int* out_rows;       // row of out and gate for product row i, or null
   long long ldx, ldo, ldg;
   int rows, n, k, x_stride, o_stride;
+  // tail > 0: the tail values behind a head's k are turned by table [token][rot / 2] (cos, sin) of their row of x, pairs
+  // (2i, 2i + 1), zero from rot on, and stored behind the head's n
+  const float2* table;
+  int rot, tail;
 };
+
+// The tail of the rows m0 .. m0 + count of one head.
+template <typename T>
+__device__ __forceinline__ void head_tail(const HeadLinearParams& p, int m0, int count, int head) {
+  const int pairs = p.tail / 2;
+  for (int u = threadIdx.x; u < count * pairs; u += blockDim.x) {
+    const int i = m0 + u / pairs, j = u % pairs;
+    if (i >= p.rows) break;
+    const long long src = p.in_rows ? p.in_rows[i] : i, dst = p.out_rows ? p.out_rows[i] : i;
+    float a = 0.f, b = 0.f;
+    if (2 * j < p.rot) {
+      const float2 cs = p.table[src * (p.rot / 2) + j];
+      const T* x = static_cast<const T*>(p.x) + src * p.ldx + static_cast<long long>(head) * p.x_stride + p.k + 2 * j;
+      const float s = ld1(x), t = ld1(x + 1);
+      a = s * cs.x - t * cs.y;
+      b = t * cs.x + s * cs.y;
+    }
+    T* o = static_cast<T*>(p.out) + dst * p.ldo + static_cast<long long>(head) * p.o_stride + p.n + 2 * j;
+    o[0] = static_cast<T>(a);
+    o[1] = static_cast<T>(b);
+  }
+}
 
 constexpr int kHlM = 64, kHlK = 64, kHlStages = 3;
 
@@ -172,6 +216,7 @@ __global__ void __launch_bounds__(128) head_linear_kernel(const HeadLinearParams
     }
   }
   cp_async_wait<0>();
+  if (p.tail && blockIdx.y == 0) head_tail<__nv_bfloat16>(p, m0, kHlM, head);
 #pragma unroll
   for (int m = 0; m < 2; ++m)
 #pragma unroll
@@ -217,6 +262,7 @@ __global__ void __launch_bounds__(256) head_linear_f32_kernel(const HeadLinearPa
       for (int q = 0; q < 4; ++q) acc[q] = fmaf(xs[r0 + 8 * q][kk], ws[c][kk], acc[q]);
     __syncthreads();
   }
+  if (p.tail && blockIdx.y == 0) head_tail<float>(p, m0, 32, head);
 #pragma unroll
   for (int q = 0; q < 4; ++q) {
     const int i = m0 + r0 + 8 * q, j = n0 + c;
@@ -232,23 +278,26 @@ __global__ void __launch_bounds__(256) head_linear_f32_kernel(const HeadLinearPa
 
 using namespace b200;
 
-// Offsets, columns and ld are multiples of 8; weights have `cols` entries (padded).
+// Offsets, columns and ld are multiples of 8; weights have `cols` entries (padded). rot > 0 (even): the rot_cols columns
+// behind the key / value latent are a rotated key, turned by table [tokens][rot / 2] (cos, sin).
 B200_API int b200_latent_prep(const void* x, const void* wq, const void* wkv, void* cq, void* cache, const long long* slots,
                               int tokens, long long ld, int q_off, int q_dim, int q_cols, int kv_off, int kv_dim, int kv_cols,
-                              float eps, int f32, cudaStream_t stream) {
+                              float eps, const void* table, int rot, int rot_cols, int f32, cudaStream_t stream) {
   if (tokens <= 0) return 0;
+  if (rot % 2 || rot > rot_cols || rot_cols % 8 || (rot && !table)) return -2;
   if (ld % 8 || q_off % 8 || kv_off % 8 || q_cols % 8 || kv_cols % 8 || q_dim > q_cols || kv_dim > kv_cols) return -2;
   LatentPrepParams p{x, static_cast<const __nv_bfloat16*>(wq), static_cast<const __nv_bfloat16*>(wkv), cq, cache, slots, ld,
-                     tokens, q_off, q_dim, q_cols, kv_off, kv_dim, kv_cols, eps};
+                     tokens, q_off, q_dim, q_cols, kv_off, kv_dim, kv_cols, eps, static_cast<const float2*>(table), rot, rot_cols};
   const dim3 grid((tokens + 3) / 4);
   const cudaError_t e = f32 ? launch_pdl(latent_prep_kernel<float>, grid, dim3(256), 0, stream, p)
                             : launch_pdl(latent_prep_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, p);
   return e == cudaSuccess ? 0 : -static_cast<int>(e) - 300;
 }
 
-// Rows of row_bytes (a multiple of 16); offsets [seqs + 1] rows of out; max_len the longest sequence.
+// Rows of row_bytes (a multiple of 16); offsets [seqs + 1] rows of out; max_len the longest sequence; starts [seqs]
+// first token of each (null: 0).
 B200_API int b200_latent_gather(const void* cache, void* out, const int* block_table, const int* seq_ids, const int* offsets,
-                                int seqs, int max_len, int row_bytes, int page, int max_pages, cudaStream_t stream) {
+                                const int* starts, int seqs, int max_len, int row_bytes, int page, int max_pages, cudaStream_t stream) {
   if (seqs <= 0 || max_len <= 0) return 0;
   if (row_bytes % 16 || seqs > 65535) return -2;
   const int vecs = row_bytes / 16;
@@ -256,17 +305,19 @@ B200_API int b200_latent_gather(const void* cache, void* out, const int* block_t
   if (blocks > 1024) blocks = 1024;
   const cudaError_t e = launch_pdl(latent_gather_kernel, dim3(static_cast<unsigned>(blocks), seqs), dim3(256), 0, stream,
                                    static_cast<const uint8_t*>(cache), static_cast<uint8_t*>(out), block_table, seq_ids, offsets,
-                                   vecs, page, max_pages);
+                                   starts, vecs, page, max_pages);
   return e == cudaSuccess ? 0 : -static_cast<int>(e) - 300;
 }
 
-// n, k, strides and row pitches multiples of 8
+// n, k, strides and row pitches multiples of 8; tail > 0: see HeadLinearParams
 B200_API int b200_head_linear(const void* x, const void* w, void* out, const void* gate, const int* in_rows, const int* out_rows,
                               int rows, int heads, int n, int k, long long ldx, int x_stride, long long ldo, int o_stride,
-                              long long ldg, int f32, cudaStream_t stream) {
+                              long long ldg, const void* table, int rot, int tail, int f32, cudaStream_t stream) {
   if (rows <= 0 || heads <= 0) return 0;
+  if (tail && (tail % 8 || rot % 2 || rot > tail || !table || x_stride < k + tail || o_stride < n + tail)) return -2;
   if (n % 8 || k % 8 || ldx % 8 || x_stride % 8 || ldo % 8 || o_stride % 8 || ldg % 8 || heads > 65535) return -2;
-  HeadLinearParams p{x, static_cast<const __nv_bfloat16*>(w), out, gate, in_rows, out_rows, ldx, ldo, ldg, rows, n, k, x_stride, o_stride};
+  HeadLinearParams p{x, static_cast<const __nv_bfloat16*>(w), out, gate, in_rows, out_rows, ldx, ldo, ldg, rows, n, k, x_stride, o_stride,
+                     static_cast<const float2*>(table), rot, tail};
   if (f32) {
     head_linear_f32_kernel<<<dim3((rows + 31) / 32, (n + 31) / 32, heads), 256, 0, stream>>>(p);
     return cudaGetLastError() == cudaSuccess ? 0 : -300;

@@ -6,6 +6,8 @@
 //    a block of tokens stay in shared memory as fp32, and one warp per token turns them into scores and
 //    picks the experts. Few tokens: fp32 FMA with the token rows in shared memory, one expert per warp.
 //    Many bf16 tokens: bf16 tensor-core products, which are exact, accumulated in fp32.
+//    Group-limited choice (the best groups by the sum of their two best experts) happens in the same warp, and
+//    a further weight row can give the sigmoid gate of a shared expert.
 //  * b200_pair_linear_f32: one weight matrix per (token, choice) pair, the expert products of the
 //    32-bit mode.
 #include "common.cuh"
@@ -28,7 +30,7 @@ constexpr int kLT = 64, kLK = 16;
 template <typename T>
 __global__ void __launch_bounds__(256)
 linear_f32_kernel(const T* __restrict__ x, const __nv_bfloat16* __restrict__ w, const __nv_bfloat16* __restrict__ bias,
-                  float* __restrict__ out, int m, int n, int k, long long ldx, long long ldw, long long ldo) {
+                  float* __restrict__ out, int m, int n, int k, long long ldx, long long ldw, long long ldo, int act) {
   __shared__ float xs[kLK][kLT + 4], ws[kLK][kLT + 4];
   const int m0 = blockIdx.y * kLT, n0 = blockIdx.x * kLT;
   const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
@@ -63,7 +65,10 @@ linear_f32_kernel(const T* __restrict__ x, const __nv_bfloat16* __restrict__ w, 
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int c = n0 + tx * 4 + j;
-      if (c < n) out[r * ldo + c] = acc[i][j] + (bias ? __bfloat162float(bias[c]) : 0.f);
+      if (c < n) {
+        const float v = acc[i][j] + (bias ? __bfloat162float(bias[c]) : 0.f);
+        out[r * ldo + c] = act == 3 ? relu2(v) : v;
+      }
     }
   }
 }
@@ -79,6 +84,9 @@ struct RouterParams {
   float* wts;                  // [tokens][top_k]
   int tokens, experts, k, ldx, ldw, top_k, sigmoid, norm_topk;
   float scale;
+  int n_group, topk_group;     // n_group > 1: only experts of the best topk_group groups of neighbours
+  int rows;                    // weight rows: experts, and one more when gate is given
+  float* gate;                 // [tokens] sigmoid of the last row's logit (may be null)
 };
 
 // Order-preserving map of a float to an unsigned integer (for warp-wide integer max)
@@ -92,6 +100,7 @@ __device__ __forceinline__ unsigned ordered_bits(float v) {
 // (scores are never negative).
 __device__ __forceinline__ void route_row(float* row, const RouterParams& p, int t) {
   const int lane = threadIdx.x & 31;
+  if (p.gate && lane == 0) p.gate[t] = 1.f / (1.f + expf(-row[p.experts]));
   if (p.sigmoid) {
     for (int e = lane; e < p.experts; e += 32) row[e] = 1.f / (1.f + expf(-row[e]));
   } else {
@@ -106,6 +115,30 @@ __device__ __forceinline__ void route_row(float* row, const RouterParams& p, int
     }
     s = warp_sum(s);
     for (int e = lane; e < p.experts; e += 32) row[e] /= s;
+  }
+  if (p.n_group > 1 && p.topk_group < p.n_group) {
+    // lane g ranks group g; experts of the other groups are passed over like chosen ones
+    __syncwarp();
+    const int size = p.experts / p.n_group;
+    unsigned value = 0;
+    if (lane < p.n_group) {
+      float b1 = -INFINITY, b2 = -INFINITY;
+      for (int e = lane * size; e < (lane + 1) * size; ++e) {
+        const float s = row[e] + (p.bias ? p.bias[e] : 0.f);
+        b2 = fmaxf(b2, fminf(b1, s));
+        b1 = fmaxf(b1, s);
+      }
+      value = ordered_bits(size > 1 ? b1 + b2 : b1);
+    }
+    unsigned kept = 0;
+    for (int r = 0; r < p.topk_group; ++r) {
+      const unsigned v = (kept >> lane) & 1 ? 0u : value;
+      const unsigned top = __reduce_max_sync(0xffffffffu, v);
+      kept |= 1u << (__ffs(__ballot_sync(0xffffffffu, v == top)) - 1);
+    }
+    for (int e = lane; e < p.experts; e += 32)
+      if (!((kept >> (e / size)) & 1)) row[e] = __uint_as_float(__float_as_uint(row[e]) | 0x80000000u);
+    __syncwarp();
   }
   float wsum = 0.f, my_w = 0.f;
   int my_id = 0;
@@ -135,14 +168,14 @@ __device__ __forceinline__ void route_row(float* row, const RouterParams& p, int
 }
 
 // Few tokens (and the 32-bit mode): kTok tokens per block in shared memory as fp32, one expert per warp and
-// turn. k is a multiple of 8. Dynamic shared memory: kTok * (k + experts) floats.
+// turn. k is a multiple of 8. Dynamic shared memory: kTok * (k + rows) floats.
 template <typename T, int kTok>
 __global__ void __launch_bounds__(kTok > 2 ? 512 : 1024) router_kernel(const RouterParams p) {
   pdl_wait();
   pdl_trigger();
   extern __shared__ __align__(16) float sm[];
   float* xs = sm;                       // [kTok][k]
-  float* lg = sm + kTok * p.k;          // [kTok][experts]
+  float* lg = sm + kTok * p.k;          // [kTok][rows]
   const int t0 = blockIdx.x * kTok;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
 #pragma unroll
@@ -151,7 +184,7 @@ __global__ void __launch_bounds__(kTok > 2 ? 512 : 1024) router_kernel(const Rou
     for (int c = threadIdx.x; c < p.k; c += blockDim.x) xs[r * p.k + c] = to_f32(xr[c]);
   }
   __syncthreads();
-  for (int e = warp; e < p.experts; e += warps) {
+  for (int e = warp; e < p.rows; e += warps) {
     float acc[kTok];
 #pragma unroll
     for (int j = 0; j < kTok; ++j) acc[j] = 0.f;
@@ -178,18 +211,18 @@ __global__ void __launch_bounds__(kTok > 2 ? 512 : 1024) router_kernel(const Rou
 #pragma unroll
     for (int j = 0; j < kTok; ++j) {
       const float s = warp_sum(acc[j]);
-      if (lane == 0) lg[j * p.experts + e] = s;
+      if (lane == 0) lg[j * p.rows + e] = s;
     }
   }
   __syncthreads();
   for (int j = warp; j < kTok; j += warps)
-    if (t0 + j < p.tokens) route_row(lg + j * p.experts, p, t0 + j);
+    if (t0 + j < p.tokens) route_row(lg + j * p.rows, p, t0 + j);
 }
 
 // Many bf16 tokens: 32 tokens per block, bf16 products with fp32 accumulation on the tensor core (m16n8k16),
 // experts in passes of kRtExp. Warp (wm, wn): tokens 16 wm.., experts kRtExp / 2 wn.. of the pass. Dynamic shared
 // memory: a ring of kRtStages stages of [32 + kRtExp] rows of 64 values (16-byte chunks XOR-swizzled by row),
-// then 32 * experts floats.
+// then 32 * rows floats.
 constexpr int kRtTok = 32, kRtK = 64, kRtStages = 5;
 
 template <int kRtExp>
@@ -205,7 +238,7 @@ __global__ void __launch_bounds__(128) router_tc_kernel(const RouterParams p) {
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, wm = warp & 1, wn = warp >> 1;
   const auto* x = static_cast<const __nv_bfloat16*>(p.x);
   const int nk = (p.k + kRtK - 1) / kRtK;
-  for (int e0 = 0; e0 < p.experts; e0 += kRtExp) {
+  for (int e0 = 0; e0 < p.rows; e0 += kRtExp) {
     auto load = [&](int kb, int st) {
       if (kb < nk) {
         for (int i = threadIdx.x; i < (kRtTok + kRtExp) * 8; i += 128) {
@@ -217,7 +250,7 @@ __global__ void __launch_bounds__(128) router_tc_kernel(const RouterParams p) {
             if (ok) src = x + static_cast<long long>(t0 + r) * p.ldx + col;
           } else {
             const int e = e0 + r - kRtTok;
-            ok = ok && e < p.experts;
+            ok = ok && e < p.rows;
             if (ok) src = p.w + static_cast<long long>(e) * p.ldw + col;
           }
           cp_async_16(base + st * kStage + r * (kRtK * 2) + ((c ^ (r & 7)) << 4), src, ok);
@@ -262,20 +295,20 @@ __global__ void __launch_bounds__(128) router_tc_kernel(const RouterParams p) {
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         const int e = e0 + wn * (kRtExp / 2) + g * 8 + (lane & 3) * 2 + (j & 1);
-        if (e < p.experts) lg[(row + 8 * (j >> 1)) * p.experts + e] = acc[g][j];
+        if (e < p.rows) lg[(row + 8 * (j >> 1)) * p.rows + e] = acc[g][j];
       }
   }
   __syncthreads();
   for (int j = warp; j < kRtTok; j += 4)
-    if (t0 + j < p.tokens) route_row(lg + j * p.experts, p, t0 + j);
+    if (t0 + j < p.tokens) route_row(lg + j * p.rows, p, t0 + j);
 }
 
 template <typename T>
 int launch_router(const RouterParams& p, bool tensor_cores, cudaStream_t stream) {
   const int limit = 200 * 1024;
   cudaError_t e;
-  const int tile = p.experts <= 32 ? 32 : p.experts <= 64 ? 64 : p.experts <= 96 ? 96 : 128;
-  const int tc_bytes = kRtStages * (kRtTok + tile) * kRtK * 2 + kRtTok * p.experts * 4;
+  const int tile = p.rows <= 32 ? 32 : p.rows <= 64 ? 64 : p.rows <= 96 ? 96 : 128;
+  const int tc_bytes = kRtStages * (kRtTok + tile) * kRtK * 2 + kRtTok * p.rows * 4;
   if (tensor_cores && p.tokens > 4 * 148 && tc_bytes <= limit && p.ldx % 8 == 0) {
     auto tc = [&](auto kernel, PerDeviceOnce& once) {
       if (once.first_time()) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, limit);
@@ -290,7 +323,7 @@ int launch_router(const RouterParams& p, bool tensor_cores, cudaStream_t stream)
     }
     return e == cudaSuccess ? 0 : -static_cast<int>(e) - 300;
   }
-  auto bytes = [&](int tok) { return tok * (p.k + p.experts) * 4; };
+  auto bytes = [&](int tok) { return tok * (p.k + p.rows) * 4; };
   // enough blocks to cover the machine first, then as many tokens per read of the weights as fit
   int tok = p.tokens >= 4 * 148 ? 8 : p.tokens >= 2 * 148 ? 4 : p.tokens > 148 ? 2 : 1;
   while (tok > 1 && bytes(tok) > limit / 2) tok /= 2;
@@ -314,7 +347,7 @@ int launch_router(const RouterParams& p, bool tensor_cores, cudaStream_t stream)
 // One warp per output feature, eight features per block.
 __global__ void __launch_bounds__(256)
 pair_linear_f32_kernel(const float* __restrict__ x, const __nv_bfloat16* __restrict__ w, const int* __restrict__ ids,
-                       float* __restrict__ out, int div, int experts, int n, int k, long long ldx, long long ldo) {
+                       float* __restrict__ out, int div, int experts, int n, int k, long long ldx, long long ldo, int act) {
   const int pair = blockIdx.y, e = ids[pair];
   if (e < 0 || e >= experts) return;
   const int j = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
@@ -324,15 +357,17 @@ pair_linear_f32_kernel(const float* __restrict__ x, const __nv_bfloat16* __restr
   float s = 0.f;
   for (int c = lane; c < k; c += 32) s += xr[c] * __bfloat162float(wr[c]);
   s = warp_sum(s);
-  if (lane == 0) out[static_cast<long long>(pair) * ldo + j] = s;
+  if (lane == 0) out[static_cast<long long>(pair) * ldo + j] = act == 3 ? relu2(s) : s;
 }
 
 }  // namespace b200
 
 using namespace b200;
 
+// act: 0 none, 3 relu squared
 B200_API int b200_linear_f32(const void* x, int x_f32, const void* w, const void* bias, void* out, int m, int n, int k,
-                             long long ldx, long long ldw, long long ldo, cudaStream_t stream) {
+                             long long ldx, long long ldw, long long ldo, int act, cudaStream_t stream) {
+  if (act != 0 && act != 3) return -2;
   if (m <= 0 || n <= 0) return 0;
   const dim3 grid((n + kLT - 1) / kLT, (m + kLT - 1) / kLT);
   if (grid.y > 65535) return -2;
@@ -340,28 +375,31 @@ B200_API int b200_linear_f32(const void* x, int x_f32, const void* w, const void
   const auto* bp = static_cast<const __nv_bfloat16*>(bias);
   if (x_f32)
     linear_f32_kernel<float><<<grid, 256, 0, stream>>>(static_cast<const float*>(x), wp, bp, static_cast<float*>(out), m, n, k,
-                                                       ldx, ldw, ldo);
+                                                       ldx, ldw, ldo, act);
   else
     linear_f32_kernel<__nv_bfloat16><<<grid, 256, 0, stream>>>(static_cast<const __nv_bfloat16*>(x), wp, bp,
-                                                               static_cast<float*>(out), m, n, k, ldx, ldw, ldo);
+                                                               static_cast<float*>(out), m, n, k, ldx, ldw, ldo, act);
   return cudaGetLastError() == cudaSuccess ? 0 : -300;
 }
 
 // ids / wts [tokens][top_k] from x [tokens][k] (fp32 or bf16) and the router weight [experts][k] bf16:
 // softmax or sigmoid scores in 32 bits, top-k by score + bias, weights = scores (optionally
-// renormalised) * scale. k a multiple of 8, top_k <= 32.
+// renormalised) * scale. k a multiple of 8, top_k <= 32. n_group > 1 (at most 32): group-limited choice. gate
+// (may be null) [tokens]: sigmoid of the logit of one more weight row behind the experts'.
 B200_API int b200_router(const void* x, int x_f32, const void* w, const float* bias, int* ids, float* wts, int tokens,
                          int experts, int k, int ldx, int ldw, int top_k, int sigmoid, int norm_topk, float scale,
-                         cudaStream_t stream) {
+                         int n_group, int topk_group, float* gate, cudaStream_t stream) {
   if (tokens <= 0) return 0;
   if (k % 8 || ldw % 8 || top_k < 1 || top_k > 32 || top_k > experts) return -2;
+  if (n_group > 1 && (n_group > 32 || experts % n_group || topk_group < 1 || topk_group > n_group)) return -2;
   RouterParams p{x, static_cast<const __nv_bfloat16*>(w), bias, ids, wts, tokens, experts, k, ldx, ldw, top_k, sigmoid,
-                 norm_topk, scale};
+                 norm_topk, scale, n_group, topk_group, experts + (gate ? 1 : 0), gate};
   return x_f32 ? launch_router<float>(p, false, stream) : launch_router<__nv_bfloat16>(p, true, stream);
 }
 
 B200_API int b200_pair_linear_f32(const void* x, const void* w, const int* ids, void* out, int pairs, int div, int experts,
-                                  int n, int k, long long ldx, long long ldo, cudaStream_t stream) {
+                                  int n, int k, long long ldx, long long ldo, int act, cudaStream_t stream) {
+  if (act != 0 && act != 3) return -2;
   if (pairs <= 0 || n <= 0) return 0;
   // the pair index is the grid's second dimension: run longer lists in slices (slices start on a token)
   const int step = 65535 / div * div;
@@ -369,7 +407,7 @@ B200_API int b200_pair_linear_f32(const void* x, const void* w, const int* ids, 
     const int cnt = pairs - p0 < step ? pairs - p0 : step;
     pair_linear_f32_kernel<<<dim3((n + 7) / 8, cnt), 256, 0, stream>>>(
         static_cast<const float*>(x) + static_cast<long long>(p0 / div) * ldx, static_cast<const __nv_bfloat16*>(w), ids + p0,
-        static_cast<float*>(out) + static_cast<long long>(p0) * ldo, div, experts, n, k, ldx, ldo);
+        static_cast<float*>(out) + static_cast<long long>(p0) * ldo, div, experts, n, k, ldx, ldo, act);
   }
   return cudaGetLastError() == cudaSuccess ? 0 : -300;
 }

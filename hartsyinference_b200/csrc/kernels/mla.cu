@@ -16,9 +16,9 @@
 //  * mla_combine: merges the KV splits.
 //
 // The attention kernel is a template over the latent width (64, 128, 256, 512) and the rotated part (64 or
-// none); rows narrower than the template's width are zero-filled on the way into shared memory. Without a
-// rotated part (latent attention without positions) the probabilities keep 16 bits of mantissa in the PV
-// product (a bf16 head and a bf16 remainder).
+// none); rows narrower than the template's width are zero-filled on the way into shared memory, output columns past
+// the latent are not stored. `b200_latent_attn` takes any latent and rotated size that fits, a sliding window, and
+// keeps 16 bits of the probabilities' mantissa in the PV product (a bf16 head and a bf16 remainder).
 //
 // Every query row carries its own kv length and block-table row, so a prefill chunk runs as rows
 // with causal lengths. Reference behaviour: src/HartsyInference.LLM/Transformer/MlaAttention.cs
@@ -120,6 +120,7 @@ struct MlaAttnParams {
   int rows, heads, page, page_shift, table_stride, splits;
   int row, lat;                 // values per cached row and per output row (multiples of 8)
   float scale_log2;
+  int window;                   // > 0: only the last `window` tokens of each row's context
 };
 
 // kSets groups of four warps share one CTA and one staged KV tile; each group owns 16 heads of the
@@ -167,8 +168,9 @@ __global__ void __launch_bounds__(kMlaThreads * kSets) mla_attn_kernel(const Mla
   const int seq = p.row_seq ? p.row_seq[row_q] : row_q;
   const int* table = p.block_table + static_cast<long long>(seq) * p.table_stride;
   const int n_tiles = (kv_len + kMlaTile - 1) / kMlaTile;
-  const int per = (n_tiles + p.splits - 1) / p.splits;
-  const int t0 = split * per, t1 = min(n_tiles, t0 + per);
+  const int start = p.window > 0 ? max(0, kv_len - p.window) : 0, tile0 = start / kMlaTile;
+  const int per = (n_tiles - tile0 + p.splits - 1) / p.splits;
+  const int t0 = tile0 + split * per, t1 = min(n_tiles, t0 + per);
   const int heads_here = max(0, min(16, p.heads - hg * 16));
   const int pages_per_tile = kMlaTile >> p.page_shift;
 
@@ -254,7 +256,7 @@ __global__ void __launch_bounds__(kMlaThreads * kSets) mla_attn_kernel(const Mla
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         const int key = t * kMlaTile + warp * 16 + nt * 8 + tq * 2 + (j & 1);
-        const float x = key < kv_len ? s[nt][j] * p.scale_log2 : -INFINITY;
+        const float x = key < kv_len && key >= start ? s[nt][j] * p.scale_log2 : -INFINITY;
         s[nt][j] = x;
         mx[j >> 1] = fmaxf(mx[j >> 1], x);
       }
@@ -476,19 +478,26 @@ B200_API int b200_mla_attn(const void* q, const void* cache, void* out, const in
   return launch_mla<kLat, kRopeDim, false>(p, workspace, stream);
 }
 
-// Latent attention without a rotated part: rows of `rank` values (a multiple of 8, at most 512), q
-// [rows][heads][rank], out the same. The workspace is that of b200_mla_workspace_bytes.
+// Latent attention of any size: cached rows of `row` values, the first `lat` of which are the values (multiples of 8,
+// lat <= 512, row <= 576), q [rows][heads][row], out
+// [rows][heads][lat]. window > 0: the last `window` tokens. The workspace is that of b200_mla_workspace_bytes.
 B200_API int b200_latent_attn(const void* q, const void* cache, void* out, const int* block_table, const int* kv_lens,
-                              const int* row_seq, int rows, int heads, int rank, int page, int table_stride, int splits,
-                              void* workspace, float scale, cudaStream_t stream) {
+                              const int* row_seq, int rows, int heads, int row, int lat, int page, int table_stride, int splits,
+                              void* workspace, float scale, int window, cudaStream_t stream) {
   if (rows <= 0) return 0;
-  if (rank % 8 || rank < 8 || rank > kLat) return -2;
+  if (lat % 8 || lat < 8 || lat > kLat || row % 8 || row < lat) return -2;
   MlaAttnParams p{};
   const int rc = mla_params(p, q, cache, out, block_table, kv_lens, row_seq, rows, heads, page, table_stride, splits, workspace, scale);
   if (rc) return rc;
-  p.row = p.lat = rank;
-  if (rank <= 64) return launch_mla<64, 0, true>(p, workspace, stream);
-  if (rank <= 128) return launch_mla<128, 0, true>(p, workspace, stream);
-  if (rank <= 256) return launch_mla<256, 0, true>(p, workspace, stream);
-  return launch_mla<512, 0, true>(p, workspace, stream);
+  p.row = row;
+  p.lat = lat;
+  p.window = window;
+  if (row <= 64) return launch_mla<64, 0, true>(p, workspace, stream);
+  if (row <= 128) return lat <= 64 ? launch_mla<64, 64, true>(p, workspace, stream) : launch_mla<128, 0, true>(p, workspace, stream);
+  if (row <= 192 && lat <= 128) return launch_mla<128, 64, true>(p, workspace, stream);
+  if (row <= 256) return launch_mla<256, 0, true>(p, workspace, stream);
+  if (row <= 320 && lat <= 256) return launch_mla<256, 64, true>(p, workspace, stream);
+  if (row <= 512) return launch_mla<512, 0, true>(p, workspace, stream);
+  if (row <= 576) return launch_mla<512, 64, true>(p, workspace, stream);
+  return -2;
 }

@@ -337,7 +337,7 @@ struct Vec8<float> {
 
 template <typename T>
 __global__ void __launch_bounds__(256) glu_clamped_kernel(const T* __restrict__ x, T* __restrict__ y, long long rows, int f,
-                                                          float limit, float alpha, const int* __restrict__ dyn_blocks, int cap) {
+                                                          float limit, float alpha, float shift, const int* __restrict__ dyn_blocks, int cap) {
   pdl_wait();
   pdl_trigger();
   if (dyn_blocks) {
@@ -362,7 +362,7 @@ __global__ void __launch_bounds__(256) glu_clamped_kernel(const T* __restrict__ 
     Vec8<T>::load(x + r * 2 * f + f + c, u);
 #pragma unroll
     for (int j = 0; j < 8; ++j)
-      g[j] = Vec8<T>::gated(fminf(g[j], limit), alpha) * (fminf(fmaxf(u[j], -limit), limit) + 1.f);
+      g[j] = Vec8<T>::gated(fminf(g[j], limit), alpha) * (fminf(fmaxf(u[j], -limit), limit) + shift);
     Vec8<T>::store(y + r * f + c, g);
   }
 }
@@ -372,7 +372,7 @@ __global__ void __launch_bounds__(256) glu_clamped_kernel(const T* __restrict__ 
 using namespace b200;
 
 // f a multiple of 8. dyn_blocks (may be null): only the first *dyn_blocks * cap rows are in use.
-B200_API int b200_glu_clamped(const void* x, void* y, long long rows, int f, float limit, float alpha, const int* dyn_blocks,
+B200_API int b200_glu_clamped(const void* x, void* y, long long rows, int f, float limit, float alpha, float shift, const int* dyn_blocks,
                               int cap, int f32, cudaStream_t stream) {
   if (rows <= 0) return 0;
   if (f % 8) return -2;
@@ -380,9 +380,9 @@ B200_API int b200_glu_clamped(const void* x, void* y, long long rows, int f, flo
   if (blocks > 148 * 8) blocks = 148 * 8;
   const cudaError_t e =
       f32 ? launch_pdl(glu_clamped_kernel<float>, dim3(static_cast<unsigned>(blocks)), dim3(256), 0, stream,
-                       static_cast<const float*>(x), static_cast<float*>(y), rows, f, limit, alpha, dyn_blocks, cap)
+                       static_cast<const float*>(x), static_cast<float*>(y), rows, f, limit, alpha, shift, dyn_blocks, cap)
           : launch_pdl(glu_clamped_kernel<__nv_bfloat16>, dim3(static_cast<unsigned>(blocks)), dim3(256), 0, stream,
-                       static_cast<const __nv_bfloat16*>(x), static_cast<__nv_bfloat16*>(y), rows, f, limit, alpha, dyn_blocks,
+                       static_cast<const __nv_bfloat16*>(x), static_cast<__nv_bfloat16*>(y), rows, f, limit, alpha, shift, dyn_blocks,
                        cap);
   return e == cudaSuccess ? 0 : -static_cast<int>(e) - 300;
 }

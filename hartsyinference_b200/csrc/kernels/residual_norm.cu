@@ -8,9 +8,11 @@
 // 32 bits). y can also be given as routed expert rows: the weighted sum over the chosen experts
 //   y[t] = sum_k w[t][k] * (slot_of[t][k] >= 0 ? rows[slot_of[t][k]] : ids[t][k] >= experts ? src[t] : 0)
 // is formed in registers first (an expert index past the last real expert returns its input), so the
-// combine step of a mixture of experts needs no launch and no intermediate rounding of its own.
+// combine step of a mixture of experts needs no launch and no intermediate rounding of its own; a shared expert's
+// rows join the sum with one weight per token.
 // LayerNorm (weight, no bias) or RMSNorm; weights as stored or stored around zero (1 + w); statistics in two
-// passes over the registers, in fp32. The embedding can be normed on its way into the stream, and poly_norm is
+// passes over the registers, in fp32. The norm on x can also be tanh(alpha x) w + b, which has no statistics.
+// side_gate is the elementwise step of a second embedding that enters every layer. The embedding can be normed on its way into the stream, and poly_norm is
 // the activation that mixes a row's normed powers.
 #include "mixer_common.cuh"
 
@@ -30,6 +32,11 @@ struct ResidualNormParams {
   int plus_one;              // norms multiply by 1 + w
   int plain;                 // no w_n: h is the stream itself
   float eps, mult;           // mult: factor of the (normed) sublayer output
+  const __nv_bfloat16* b_n;  // not null: h = tanh(alpha x) w_n + b_n
+  float alpha;
+  const void* extra;         // routed source: [rows][ld_extra] added with weight extra_w[row] (null: none)
+  const float* extra_w;
+  int ld_extra;
 };
 
 // v <- norm(v) * w over the row's first `dim` values (values past them are zero on entry and exit)
@@ -72,6 +79,26 @@ __device__ __forceinline__ void norm_row(float (&v)[kIters][8], const __nv_bfloa
   }
 }
 
+// v <- tanh(alpha v) * w + b over the row's first `dim` values, zero past them
+template <int kIters>
+__device__ __forceinline__ void tanh_row(float (&v)[kIters][8], const __nv_bfloat16* w, const __nv_bfloat16* b, float alpha, int dim) {
+#pragma unroll
+  for (int i = 0; i < kIters; ++i) {
+    const int c = (threadIdx.x + i * blockDim.x) * 8;
+    if (c + 8 <= dim) {
+      float wv[8], bv[8];
+      load8(w + c, wv);
+      load8(b + c, bv);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) v[i][j] = fmaf(tanhf(alpha * v[i][j]), wv[j], bv[j]);
+    } else {
+#pragma unroll
+      for (int j = 0; j < 8; ++j)
+        v[i][j] = c + j < dim ? fmaf(tanhf(alpha * v[i][j]), __bfloat162float(w[c + j]), __bfloat162float(b[c + j])) : 0.f;
+    }
+  }
+}
+
 // One block per row; every leading dimension is a multiple of 8 and covers dim rounded up to 8.
 template <typename T, int kIters>
 __global__ void __launch_bounds__(1024) residual_norm_kernel(const ResidualNormParams p) {
@@ -95,6 +122,20 @@ __global__ void __launch_bounds__(1024) residual_norm_kernel(const ResidualNormP
         else if (p.src != nullptr && p.ids[row * p.top_k + k] >= p.experts) sp = static_cast<const T*>(p.src) + row * p.ld_src;
         if (sp == nullptr) continue;
         const float w = p.wts[row * p.top_k + k];
+#pragma unroll
+        for (int i = 0; i < kIters; ++i) {
+          const int c = (threadIdx.x + i * blockDim.x) * 8;
+          if (c < p.dim) {
+            float t[8];
+            load8(sp + c, t);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) yv[i][j] += w * t[j];
+          }
+        }
+      }
+      if (p.extra != nullptr) {
+        const T* sp = static_cast<const T*>(p.extra) + row * p.ld_extra;
+        const float w = p.extra_w[row];
 #pragma unroll
         for (int i = 0; i < kIters; ++i) {
           const int c = (threadIdx.x + i * blockDim.x) * 8;
@@ -144,7 +185,8 @@ __global__ void __launch_bounds__(1024) residual_norm_kernel(const ResidualNormP
     }
   }
   if (p.w_n == nullptr && !p.plain) return;
-  if (p.w_n != nullptr) norm_row<kIters>(xv, p.w_n, p.dim, p.layernorm, p.plus_one, p.eps, red);
+  if (p.b_n != nullptr) tanh_row<kIters>(xv, p.w_n, p.b_n, p.alpha, p.dim);
+  else if (p.w_n != nullptr) norm_row<kIters>(xv, p.w_n, p.dim, p.layernorm, p.plus_one, p.eps, red);
   T* hr = static_cast<T*>(p.h) + row * p.ldh;
 #pragma unroll
   for (int i = 0; i < kIters; ++i) {
@@ -210,6 +252,26 @@ __global__ void __launch_bounds__(1024) embedding_norm_kernel(const EmbeddingNor
       store8(static_cast<T*>(p.h) + t * p.ldx + c, v[i]);
     }
   }
+}
+
+// y[t][c] = gelu_tanh(u[t][c]) * table[ids[t]][off + c], eight values per thread
+template <typename T>
+__global__ void __launch_bounds__(256) side_gate_kernel(const T* __restrict__ u, const int* __restrict__ ids,
+                                                        const __nv_bfloat16* __restrict__ table, T* __restrict__ y, long long n,
+                                                        int vecs, int ldu, int ldt, int vocab) {
+  pdl_wait();
+  pdl_trigger();
+  const long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x;
+  if (i >= n) return;
+  const long long t = i / vecs;
+  const int c = static_cast<int>(i % vecs) * 8;
+  const int id = min(max(ids[t], 0), vocab - 1);
+  float a[8], e[8];
+  load8(u + t * ldu + c, a);
+  load8(table + static_cast<long long>(id) * ldt + c, e);
+#pragma unroll
+  for (int j = 0; j < 8; ++j) a[j] = gelu_tanh(a[j]) * e[j];
+  store8(y + t * vecs * 8 + c, a);
 }
 
 // y = a z / rms(z) + b z^2 / rms(z^2) + c z^3 / rms(z^3) + e over a row of `dim` values (powers element by
@@ -297,21 +359,41 @@ int launch_residual_norm(const ResidualNormParams& p, int rows, cudaStream_t str
 
 using namespace b200;
 
-// See the header comment. f32 != 0: y / src / h are fp32 instead of bf16. ldy etc. in elements,
+// See the header comment. f32 != 0: y / src / extra / h are fp32 instead of bf16. ldy etc. in elements,
 // multiples of 8. Rows of at most 16384 values.
 B200_API int b200_residual_norm(void* x, const void* y, void* h, const void* w_b, const void* w_n, const int* slot_of,
                                 const int* ids, const float* wts, const void* src, int rows, int dim, int ldx, int ldy,
                                 int ldh, int ld_src, int top_k, int experts, int layernorm, int plus_one, int plain, float eps,
-                                float mult, int f32, cudaStream_t stream) {
+                                float mult, int f32, const void* b_n, float alpha, const void* extra, const float* extra_w,
+                                int ld_extra, cudaStream_t stream) {
   if (rows <= 0) return 0;
   const int dim8 = (dim + 7) / 8 * 8;
   if (dim < 1 || dim > 16384 || ldx < dim8 || ldx % 8 || ((w_n || plain) && (ldh != dim8 || !h))) return -2;
   if (y && (ldy < dim8 || ldy % 8)) return -2;
   if (slot_of && (!ids || !wts || top_k < 1 || (src && (ld_src < dim8 || ld_src % 8)))) return -2;
+  if ((b_n && !w_n) || (extra && (!slot_of || !extra_w || ld_extra < dim8 || ld_extra % 8))) return -2;
   ResidualNormParams p{static_cast<float*>(x), y, h, static_cast<const __nv_bfloat16*>(w_b),
                        static_cast<const __nv_bfloat16*>(w_n), slot_of, ids, wts, src, dim, ldx, ldy, ldh, ld_src, top_k,
-                       experts, layernorm, plus_one, plain, eps, mult};
+                       experts, layernorm, plus_one, plain, eps, mult, static_cast<const __nv_bfloat16*>(b_n), alpha, extra, extra_w,
+                       ld_extra};
   return f32 ? launch_residual_norm<float>(p, rows, stream) : launch_residual_norm<__nv_bfloat16>(p, rows, stream);
+}
+
+// y [tokens][dim] from u [tokens][ldu] and rows of table [vocab][ldt] (already moved to the layer's columns); dim and
+// both pitches multiples of 8
+B200_API int b200_side_gate(const void* u, const int* ids, const void* table, void* y, int tokens, int dim, int ldu, int ldt,
+                            int vocab, int f32, cudaStream_t stream) {
+  if (tokens <= 0) return 0;
+  if (dim < 8 || dim % 8 || ldu % 8 || ldt % 8) return -2;
+  const long long n = static_cast<long long>(tokens) * (dim / 8);
+  const dim3 grid(static_cast<unsigned>((n + 255) / 256));
+  const auto* tab = static_cast<const __nv_bfloat16*>(table);
+  const cudaError_t e =
+      f32 ? launch_pdl(side_gate_kernel<float>, grid, dim3(256), 0, stream, static_cast<const float*>(u), ids, tab,
+                       static_cast<float*>(y), n, dim / 8, ldu, ldt, vocab)
+          : launch_pdl(side_gate_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, static_cast<const __nv_bfloat16*>(u), ids, tab,
+                       static_cast<__nv_bfloat16*>(y), n, dim / 8, ldu, ldt, vocab);
+  return e == cudaSuccess ? 0 : -static_cast<int>(e) - 300;
 }
 
 B200_API int b200_embedding_f32(const int* ids, const void* table, void* x, int tokens, int dim, int ldx, int ldt,

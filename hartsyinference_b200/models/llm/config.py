@@ -31,6 +31,7 @@ class MoeConfig:
     exact_router: bool = False          # router logits and scores in 32 bits
     glu_limit: float = 0.0              # > 0: clamped expert activation g sigmoid(alpha g) (u + 1), g <= limit, |u| <= limit
     glu_alpha: float = 1.702
+    expert_act: str = "glu"             # glu: gated experts (gate | up); relu2: down(relu(up h)^2), shared expert alike
 
     @property
     def choices(self) -> int:
@@ -49,6 +50,28 @@ class MlaConfig:
 
 
 @dataclass(frozen=True)
+class RopeScaling:
+    kind: str = "none"                  # none | linear | llama3 | yarn
+    factor: float = 1.0
+    low_freq_factor: float = 1.0
+    high_freq_factor: float = 4.0
+    original_max_position: float = 8192
+    beta_fast: float = 32.0
+    beta_slow: float = 1.0
+    attn_factor: float = 1.0
+    truncate: bool = True               # YaRN: round the correction range to whole dimensions (gpt-oss does not)
+
+
+@dataclass(frozen=True)
+class RotarySpec:
+    """Rotation of one mixer's queries and keys."""
+    dims: int                           # leading values of a head (or of its rotated part) that turn
+    base: float = 10000.0
+    interleaved: bool = False           # pairs (2i, 2i + 1) instead of (i, i + dims / 2)
+    scaling: RopeScaling = field(default_factory=RopeScaling)
+
+
+@dataclass(frozen=True)
 class MixerSpec:
     """Token mixer of one layer of a model whose layers differ (``TransformerConfig.layer_specs``)."""
     kind: str = "attention"             # attention | channel_delta | latent_attention | channel_scan | head_scan
@@ -60,15 +83,19 @@ class MixerSpec:
     scale: float = 0.0                  # 0 = 1/sqrt(dim)
     softcap: float = 0.0
     window: int = 0                     # 0 = unlimited
+    keep_first: int = 0                 # first tokens of the sequence that stay visible outside the window
+    rot: Optional[RotarySpec] = None
+    qk_norm: bool = False               # RMS norm of q and of k over all their heads at once, before the rotation
     bias_reach: int = 0                 # distance at which the logarithmic bias buckets end (0: no distance bias)
     bias_rows: int = 32                 # bias table rows of synthetic weights (a checkpoint's table gives its own)
     shared_kv: bool = False             # the values are the keys
     qk_bias: bool = False
     out_gate: bool = False              # output * sigmoid(W_g h)
     sink: Optional[float] = None        # score of a key without a value
-    # latent_attention (dim / vdim: query-key and value size per head, out_gate as above)
+    # latent_attention (dim / vdim: unrotated query-key and value size per head; window, rot and out_gate as above)
     q_rank: int = 0                     # size of the query latent
     kv_rank: int = 0                    # size of the cached key / value latent
+    rot_dim: int = 0                    # rotated query-key size per head; the keys share one rotated part
     # recurrent kinds
     conv: int = 0                       # taps of the short convolution
     rank: int = 0                       # low-rank size: channel_delta decay and gate in synthetic weights (0 = dim); channel_scan step size
@@ -85,9 +112,9 @@ class MixerSpec:
 
 @dataclass(frozen=True)
 class DenseSpec:
-    """Ungated dense feed-forward of one layer: down(act(up h))."""
+    """Dense feed-forward of one layer: ungated down(act(up h)), or down(silu(gate h) * up h)."""
     ffn: int
-    act: str = "poly_norm"
+    act: str = "poly_norm"              # poly_norm (ungated) | silu (gated)
 
 
 @dataclass(frozen=True)
@@ -96,19 +123,6 @@ class LayerSpec:
     moe: Optional[MoeConfig] = None     # routed experts
     dense: Optional[DenseSpec] = None   # or a dense feed-forward; neither: no feed-forward in this layer
     weights_of: Optional[int] = None    # index of the layer whose weights this one uses (its cache and state are its own)
-
-
-@dataclass(frozen=True)
-class RopeScaling:
-    kind: str = "none"                  # none | linear | llama3 | yarn
-    factor: float = 1.0
-    low_freq_factor: float = 1.0
-    high_freq_factor: float = 4.0
-    original_max_position: int = 8192
-    beta_fast: float = 32.0
-    beta_slow: float = 1.0
-    attn_factor: float = 1.0
-    truncate: bool = True               # YaRN: round the correction range to whole dimensions (gpt-oss does not)
 
 
 @dataclass(frozen=True)
@@ -149,7 +163,7 @@ class TransformerConfig:
     qk_norm_full: bool = False          # q/k RMSNorm over the whole projection instead of per head (OLMo 2, OLMoE)
     rope_local_theta: float = 0.0       # rotary base of the sliding-window layers when it differs (Gemma 3)
     layer_types: tuple = ()             # explicit per-layer "sliding_attention" / "full_attention"
-    norm_type: str = "rms"              # rms | layernorm
+    norm_type: str = "rms"              # rms | layernorm | tanh (no statistics: tanh(alpha x) w + b)
     norm_bias: bool = False
     parallel_residual: bool = False     # x + attn(n1(x)) + ffn(n2(x)) (GPT-NeoX, Cohere)
     shared_parallel_norm: bool = False  # the parallel branches share one norm (Cohere)
@@ -169,7 +183,8 @@ class TransformerConfig:
     moe: Optional[MoeConfig] = None
     mla: Optional[MlaConfig] = None
     layer_specs: tuple = ()             # one LayerSpec per layer: mixers of different kinds and sizes around a 32-bit
-                                        # residual stream, norms before and after every sublayer
+                                        # residual stream, norms before and / or after every sublayer
+    token_side: int = 0                 # > 0: every layer adds a gated map of its part (this many values) of a second token embedding
     bos_token_id: int = 1
     eos_token_ids: tuple = (2,)
 
@@ -232,6 +247,8 @@ class TransformerConfig:
         if self.layer_specs:
             from .mixers import spec_param_count
             own = sum(spec_param_count(ls, h) for ls in self.layer_specs if ls.weights_of is None)
+            if self.token_side:
+                own += l * (self.token_side * (self.vocab_size + 2 * h) + h)
             return own + (1 if self.tie_embeddings else 2) * self.vocab_size * h + h
         attn = h * (self.q_size + 2 * self.kv_size) + self.q_size * h
         if self.mla is not None:
@@ -305,7 +322,7 @@ def tiny(base: str = "qwen2.5-0.5b", **over: Any) -> TransformerConfig:
 
 # designs whose layers are described one by one; each is a module of this package with ``config_from``,
 # ``load_layers``, ``tensor_shapes`` and ``random_tensor``
-MIXED_DESIGNS = ("lududra", "salopel")
+MIXED_DESIGNS = ("lududra", "salopel", "zovudra")
 
 
 def mixed_design(arch: str):

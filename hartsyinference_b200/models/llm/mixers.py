@@ -19,6 +19,7 @@ import torch
 from ... import ops
 from ...ops import LinearWeight
 from .config import DenseSpec, LayerSpec, MixerSpec, MoeConfig
+from .rope import Rotary
 
 
 def pad_to(n: int, m: int) -> int:
@@ -73,26 +74,36 @@ def distance_bias_table(rel: torch.Tensor, reach: int, window: int) -> torch.Ten
 
 
 class BiasedAttention:
-    """Grouped-query attention over the page pool with a distance bias, a window, a score cap, a sink and an
-    output gate, each as the spec says. One projection GEMM (q | k | v | gate)."""
+    """Grouped-query attention over the page pool with a norm over all heads of q and of k, a rotation, a distance
+    bias, a window with kept first tokens, a score cap, a sink and an output gate, each as the spec says. One projection
+    GEMM (q | k | v | gate)."""
 
     def __init__(self, spec: MixerSpec, width: int, device, *, q: torch.Tensor, k: torch.Tensor, v: Optional[torch.Tensor],
                  o: torch.Tensor, q_bias: Optional[torch.Tensor] = None, k_bias: Optional[torch.Tensor] = None,
-                 gate: Optional[torch.Tensor] = None, rel: Optional[torch.Tensor] = None):
-        self.spec = spec
-        hq, hk, d = spec.heads, spec.kv_heads, spec.dim
-        self.d = dp = pad_to(d, 8)
+                 gate: Optional[torch.Tensor] = None, rel: Optional[torch.Tensor] = None, q_norm: Optional[torch.Tensor] = None,
+                 k_norm: Optional[torch.Tensor] = None, eps: float = 0.0):
+        self.spec, self.eps = spec, eps
+        hq, hk, d, dv = spec.heads, spec.kv_heads, spec.dim, spec.dim if v is None else spec.vdim
+        if max(d, dv) > 512:
+            raise ValueError(f"attention heads of {d} / {dv} values are not supported (at most 512)")
+        self.d, self.dv = dp, vp = pad_to(d, 8), pad_to(dv, 8)
         wp = pad_to(width, 8)
         head = lambda t, n: pad_head_rows(t, n, d, dp)
-        parts = [head(q, hq), head(k, hk)] + ([head(v, hk)] if v is not None else []) + ([head(gate, hq)] if gate is not None else [])
+        vhead = lambda t, n: pad_head_rows(t, n, dv, vp)
+        parts = [head(q, hq), head(k, hk)] + ([vhead(v, hk)] if v is not None else []) + ([vhead(gate, hq)] if gate is not None else [])
         bias = None
         if q_bias is not None:
             rest = sum(p.shape[0] for p in parts[2:])
             bias = torch.cat([head(q_bias, hq), head(k_bias, hk), torch.zeros(rest, dtype=q_bias.dtype, device=q_bias.device)])
         self.proj = _linear([pad_cols(p, wp) for p in parts], device, bias)
-        self.o = _linear([pad_rows(pad_head_cols(o, hq, d, dp), wp)], device)
-        self.nq, self.nk = hq * dp, hk * dp
+        self.o = _linear([pad_rows(pad_head_cols(o, hq, dv, vp), wp)], device)
+        self.nq, self.nk, self.nv = hq * dp, hk * dp, hk * vp
         self.shared_kv, self.gated = v is None, gate is not None
+        norm = lambda t, n: None if t is None else head(t, n).to(torch.bfloat16).to(device).contiguous()
+        self.q_norm, self.k_norm = norm(q_norm, hq), norm(k_norm, hk)
+        self.rotary = None if spec.rot is None else Rotary(spec.rot, device)
+        if self.shared_kv and (self.rotary is not None or q_norm is not None):
+            raise ValueError("attention: keys that are values are neither normed nor turned")
         self.bias = distance_bias_table(rel, spec.bias_reach, spec.window).to(device) if rel is not None and spec.bias_reach > 0 else None
         self.sinks = None if spec.sink is None else torch.full((hq,), float(spec.sink), dtype=torch.float32, device=device)
         self.scale = spec.scale or d ** -0.5
@@ -101,19 +112,43 @@ class BiasedAttention:
         return self.proj.nbytes() + self.o.nbytes()
 
     def cache_shape(self, pages: int, page: int) -> tuple:
-        return ((1 if self.shared_kv else 2), pages, self.spec.kv_heads, page, self.d)
+        """[planes, pages, kv heads, page, head size], or, with values of another size than the keys, all key pages and
+        then all value pages in one row."""
+        hk = self.spec.kv_heads
+        if self.shared_kv or self.d == self.dv:
+            return ((1 if self.shared_kv else 2), pages, hk, page, self.d)
+        return (pages, hk * page * (self.d + self.dv))
+
+    def _planes(self, cache: torch.Tensor) -> tuple[torch.Tensor, Optional[torch.Tensor]]:
+        if cache.dim() > 2:
+            return cache[0], None if self.shared_kv else cache[1]
+        pages, hk = cache.shape[0], self.spec.kv_heads
+        page = cache.shape[1] // (hk * (self.d + self.dv))
+        n = pages * hk * page * self.d
+        flat = cache.view(-1)
+        return flat[:n].view(pages, hk, page, self.d), flat[n:].view(pages, hk, page, self.dv)
 
     def __call__(self, h: torch.Tensor, batch, li: int, model) -> torch.Tensor:
         p = ops.linear_act(h, self.proj)
         k0, v0 = self.nq, self.nq + self.nk
-        g0 = v0 if self.shared_kv else v0 + self.nk
+        g0 = v0 if self.shared_kv else v0 + self.nv
         cache = model.kv_cache[li]
-        kc, vc = cache[0], None if self.shared_kv else cache[1]
-        ops.kv_store(p[:, k0:v0], kc, batch.slot_mapping, None if self.shared_kv else p[:, v0:g0], vc)
-        a = ops.attn_biased(p[:, :k0], kc, vc, batch.block_table, batch.kv_lens, None if batch.is_decode else batch.cu_q,
+        kc, vc = self._planes(cache)
+        if self.rotary is not None or self.q_norm is not None:
+            q = ops.qk_rope_store(p, self.spec.heads, kc, vc, batch.slot_mapping, table=None if self.rotary is None else self.rotary.table(batch),
+                                  interleaved=self.rotary is not None and self.rotary.spec.interleaved, q_norm=self.q_norm, k_norm=self.k_norm,
+                                  d_true=self.spec.dim, eps=self.eps)
+        else:
+            q = p[:, :k0]
+            if self.shared_kv or self.d == self.dv:
+                ops.kv_store(p[:, k0:v0], kc, batch.slot_mapping, None if self.shared_kv else p[:, v0:g0], vc)
+            else:
+                ops.kv_store(p[:, k0:v0], kc, batch.slot_mapping)
+                ops.kv_store(p[:, v0:g0], vc, batch.slot_mapping)
+        a = ops.attn_biased(q, kc, vc, batch.block_table, batch.kv_lens, None if batch.is_decode else batch.cu_q,
                             heads=self.spec.heads, max_q_len=batch.max_q_len, max_kv_len=batch.max_kv_len, scale=self.scale,
                             softcap=self.spec.softcap, window=self.spec.window, dist_bias=self.bias, sinks=self.sinks,
-                            gate=p[:, g0:] if self.gated else None)
+                            gate=p[:, g0:] if self.gated else None, keep_first=self.spec.keep_first)
         return ops.linear_act(a, self.o)
 
 
@@ -251,10 +286,10 @@ _EXPAND_TOKENS = 65536
 
 
 class LatentPlan:
-    """How a ragged batch is split for latent attention: groups of long runs, and the rows of the short ones.
-    The index arrays go to the device in one copy."""
+    """How a ragged batch is split for latent attention: groups of long runs with the part of their contexts that a
+    window leaves, and the rows of the short ones. The index arrays go to the device in one copy."""
 
-    def __init__(self, batch, expand: bool):
+    def __init__(self, batch, expand: bool, window: int = 0):
         runs = batch.runs
         if runs is None:
             cu, kv = batch.cu_q.tolist(), batch.kv_lens.tolist()
@@ -263,10 +298,13 @@ class LatentPlan:
         for q, _ in runs:
             starts.append(t)
             t += q
+        # first key that a run's first query sees, and keys from there on
+        first = [max(0, kv - q - window + 1) if window > 0 else 0 for q, kv in runs]
+        keys = [kv - f for (_, kv), f in zip(runs, first)]
         long = [i for i, (q, _) in enumerate(runs) if expand and q >= _EXPAND_RUN]
         groups: list[list[int]] = []
         for i in long:
-            if not groups or sum(runs[j][1] for j in groups[-1]) + runs[i][1] > _EXPAND_TOKENS:
+            if not groups or sum(keys[j] for j in groups[-1]) + keys[i] > _EXPAND_TOKENS:
                 groups.append([])
             groups[-1].append(i)
         flat: list[int] = []
@@ -286,13 +324,14 @@ class LatentPlan:
         for g in groups:
             off = [0]
             for i in g:
-                off.append(off[-1] + runs[i][1])
-            at.append((put(g), put(off), put([starts[i] for i in g]), put([runs[i][0] for i in g]), put([runs[i][1] for i in g])))
+                off.append(off[-1] + keys[i])
+            at.append((put(g), put(off), put([starts[i] for i in g]), put([runs[i][0] for i in g]), put([keys[i] for i in g]),
+                       put([first[i] for i in g])))
         r = [put([x[k] for x in rows]) for k in range(3)]
         dev = torch.tensor(flat, dtype=torch.int32).to(batch.tokens.device)
-        self.groups = [dict(seqs=dev[a], offsets=dev[b], q_start=dev[c], q_lens=dev[d], kv_lens=dev[e],
-                            total=sum(runs[i][1] for i in g), max_kv=max(runs[i][1] for i in g), max_q=max(runs[i][0] for i in g))
-                       for g, (a, b, c, d, e) in zip(groups, at)]
+        self.groups = [dict(seqs=dev[a], offsets=dev[b], q_start=dev[c], q_lens=dev[d], kv_lens=dev[e], first=dev[f],
+                            total=sum(keys[i] for i in g), max_kv=max(keys[i] for i in g), max_q=max(runs[i][0] for i in g))
+                       for g, (a, b, c, d, e, f) in zip(groups, at)]
         # rows None: every row of the batch, in order
         self.short = len(rows)
         self.rows = dev[r[0]] if groups else None
@@ -301,118 +340,177 @@ class LatentPlan:
 
 class LatentAttention:
     """Attention whose keys and values are per-head maps of one cached latent; queries through a latent of their
-    own, sigmoid output gate, no positions. One projection GEMM (query latent | latent | gate)."""
+    own. Optional: a rotated part of queries and keys (one rotated key for all heads, cached behind the latent), a
+    window, a sigmoid output gate. One projection GEMM (query latent | latent | rotated key | gate)."""
 
-    def __init__(self, spec: MixerSpec, width: int, eps: float, device, *, dq, dq_norm, uq, dkv, dkv_norm, uk, uv, g, o):
+    def __init__(self, spec: MixerSpec, width: int, eps: float, device, *, dq, dq_norm, uq, dkv, dkv_norm, uk, uv, o, g=None):
         self.spec, self.eps = spec, eps
-        h, d, v = spec.heads, spec.dim, spec.vdim
+        h, d, v, t = spec.heads, spec.dim, spec.vdim, spec.rot_dim
         if spec.kv_rank > 512:
             raise ValueError(f"latent_attention with a latent of {spec.kv_rank} values is not supported (at most 512)")
+        if t % 2 or t > 512 or bool(t) != (spec.rot is not None):
+            raise ValueError(f"latent_attention with a rotated part of {t} values is not supported (even, at most 512, with its rotation)")
         wp = pad_to(width, 8)
-        self.d, self.v = dp, vp = pad_to(d, 8), pad_to(v, 8)
+        self.d, self.v, self.t = dp, vp, tp = pad_to(d, 8), pad_to(v, 8), pad_to(t, 8)
         self.qr, self.r = qr, r = pad_to(spec.q_rank, 8), pad_to(spec.kv_rank, 8)
-        head = lambda t, k, kp: pad_head_rows(t, h, k, kp)
-        self.proj = _linear([pad_cols(p, wp) for p in (pad_rows(dq, qr), pad_rows(dkv, r), head(g, v, vp))], device)
-        vec = lambda t, n: pad_rows(t, n).to(torch.bfloat16).to(device).contiguous()
+        head = lambda m, k, kp: pad_head_rows(m, h, k, kp)
+        parts = [pad_rows(dq, qr), pad_rows(dkv[:spec.kv_rank], r)] + ([pad_rows(dkv[spec.kv_rank:], tp)] if t else [])
+        self.proj = _linear([pad_cols(p, wp) for p in parts + ([] if g is None else [head(g, v, vp)])], device)
+        self.gated = g is not None
+        vec = lambda m, n: pad_rows(m, n).to(torch.bfloat16).to(device).contiguous()
         self.q_norm, self.kv_norm = vec(dq_norm, qr), vec(dkv_norm, r)
-        self.uq = _linear([pad_cols(head(uq, d, dp), qr)], device)
+        if t:                                    # both parts of every head padded on their own
+            uq = uq.reshape(h, d + t, -1)
+            uq = torch.cat([pad_head_rows(uq[:, :d].reshape(h * d, -1), h, d, dp).reshape(h, dp, -1),
+                            pad_head_rows(uq[:, d:].reshape(h * t, -1), h, t, tp).reshape(h, tp, -1)], 1).reshape(h * (dp + tp), -1)
+        else:
+            uq = head(uq, d, dp)
+        self.uq = _linear([pad_cols(uq, qr)], device)
         uk, uv = pad_cols(head(uk, d, dp), r), pad_cols(head(uv, v, vp), r)
         self.kv_up = _linear([uk, uv], device)
         self.uv = LinearWeight(self.kv_up.weight[h * dp:])
         self.uk_t = _linear([uk.reshape(h, dp, r).transpose(1, 2).reshape(h * r, dp)], device)     # the query's side of W_uk
         self.o = _linear([pad_rows(pad_head_cols(o, h, v, vp), wp)], device)
-        self.scale = spec.scale or d ** -0.5
+        self.scale = spec.scale or (d + t) ** -0.5
+        self.rotary = None if spec.rot is None else Rotary(spec.rot, device)
+        if self.rotary is not None and (not spec.rot.interleaved or spec.rot.dims != t):
+            raise ValueError("latent_attention turns the whole rotated part in pairs of neighbours")
 
     def nbytes(self) -> int:
         return sum(w.nbytes() for w in (self.proj, self.uq, self.kv_up, self.uk_t, self.o))
 
     def cache_shape(self, pages: int, page: int) -> tuple:
-        return (1, pages, 1, page, self.r)
+        return (1, pages, 1, page, self.r + self.t)
 
     def _plan(self, batch, h: torch.Tensor) -> LatentPlan:
-        expand = h.is_cuda and h.dtype == torch.bfloat16 and max(self.d, self.v) <= 128
+        expand = h.is_cuda and h.dtype == torch.bfloat16 and max(self.d + self.t, self.v) <= 128
         if batch.plan is None:
             batch.plan = {}
-        if expand not in batch.plan:
-            batch.plan[expand] = LatentPlan(batch, expand)
-        return batch.plan[expand]
+        key = (expand, self.spec.window)
+        if key not in batch.plan:
+            batch.plan[key] = LatentPlan(batch, *key)
+        return batch.plan[key]
 
     def __call__(self, h: torch.Tensor, batch, li: int, model) -> torch.Tensor:
-        heads = self.spec.heads
+        heads, window, r = self.spec.heads, self.spec.window, self.r
+        table = None if self.rotary is None else self.rotary.table(batch)
         p = ops.linear_act(h, self.proj)
-        gate = p[:, self.qr + self.r:]
+        gate = p[:, self.qr + r + self.t:] if self.gated else None
         cache = model.kv_cache[li][0]
-        cq = ops.latent_prep(p, 0, self.spec.q_rank, self.q_norm, self.qr, self.spec.kv_rank, self.kv_norm, cache, batch.slot_mapping, self.eps)
+        cq = ops.latent_prep(p, 0, self.spec.q_rank, self.q_norm, self.qr, self.spec.kv_rank, self.kv_norm, cache, batch.slot_mapping, self.eps,
+                             table)
         q = ops.linear_act(cq, self.uq)
         if batch.is_decode:
-            a = ops.latent_attn(ops.head_linear(q, self.uk_t, heads), cache, batch.block_table, batch.kv_lens, heads, self.scale,
-                                max_kv_len=batch.max_kv_len)
+            a = ops.latent_attn(ops.head_linear(q, self.uk_t, heads, tail=self.t, table=table), cache, batch.block_table, batch.kv_lens, heads,
+                                self.scale, max_kv_len=batch.max_kv_len, v_dim=r, window=window)
             return ops.linear_act(ops.head_linear(a, self.uv, heads, gate=gate), self.o)
         plan = self._plan(batch, h)
         y = torch.empty(h.shape[0], heads * self.v, dtype=h.dtype, device=h.device)
         for g in plan.groups:
-            c = ops.latent_gather(cache, batch.block_table, g["seqs"], g["offsets"], g["total"], g["max_kv"])
-            kv = ops.linear_act(c, self.kv_up)
+            c = ops.latent_gather(cache, batch.block_table, g["seqs"], g["offsets"], g["total"], g["max_kv"], g["first"])
+            kv = ops.linear_act(c[:, :r], self.kv_up)
             ops.attn_runs(q, kv[:, :heads * self.d], kv[:, heads * self.d:], y, g["q_start"], g["q_lens"], g["offsets"], g["kv_lens"],
-                          heads=heads, max_q_len=g["max_q"], scale=self.scale, gate=gate)
+                          heads=heads, max_q_len=g["max_q"], scale=self.scale, gate=gate, window=window,
+                          k_shared=c[:, r:] if self.t else None, table=table)
         if plan.short:
-            ql = ops.head_linear(q, self.uk_t, heads, in_rows=plan.rows)
+            ql = ops.head_linear(q, self.uk_t, heads, in_rows=plan.rows, tail=self.t, table=table)
             a = ops.latent_attn(ql, cache, batch.block_table, plan.row_len, heads, self.scale, row_seq=plan.row_seq,
-                                max_kv_len=batch.max_kv_len)
+                                max_kv_len=batch.max_kv_len, v_dim=r, window=window)
             ops.head_linear(a, self.uv, heads, gate=gate, out=y, out_rows=plan.rows)
         return ops.linear_act(y, self.o)
 
 
 class DenseFeedForward:
-    """Ungated feed-forward ``down(act(up h))``; ``coef``: the activation's numbers."""
+    """Feed-forward ``down(act(up h))`` (``coef``: the activation's numbers), or gated: ``down(silu(gate h) * up h)``."""
 
-    def __init__(self, spec: DenseSpec, width: int, eps: float, device, *, up, down, coef):
-        if spec.act != "poly_norm":
+    def __init__(self, spec: DenseSpec, width: int, eps: float, device, *, up, down, coef=None, gate=None):
+        if spec.act not in ("poly_norm", "silu"):
             raise ValueError(f"unknown activation '{spec.act}'")
         self.spec, self.eps = spec, eps
         fp, wp = pad_to(spec.ffn, 8), pad_to(width, 8)
-        self.up = _linear([pad_rows(pad_cols(up, wp), fp)], device)
+        rows = [pad_rows(pad_cols(t, wp), fp) for t in (gate, up) if t is not None]
+        if len(rows) != (2 if spec.act == "silu" else 1):
+            raise ValueError(f"a feed-forward with activation '{spec.act}' has {'a' if spec.act == 'silu' else 'no'} gate")
+        self.up = _linear(rows, device)
         self.down = _linear([pad_rows(pad_cols(down, fp), wp)], device)
-        self.coef = coef.float().to(device).contiguous()
+        self.coef = None if coef is None else coef.float().to(device).contiguous()
 
     def nbytes(self) -> int:
         return self.up.nbytes() + self.down.nbytes()
 
     def __call__(self, h: torch.Tensor, model=None) -> torch.Tensor:
-        return ops.linear_act(ops.poly_norm(ops.linear_act(h, self.up), self.coef, self.spec.ffn, self.eps), self.down)
+        if self.spec.act == "poly_norm":
+            return ops.linear_act(ops.poly_norm(ops.linear_act(h, self.up), self.coef, self.spec.ffn, self.eps), self.down)
+        if h.dtype == torch.float32:
+            a = ops.glu_clamped(ops.linear_act(h, self.up), math.inf, 1.0, shift=0.0)
+        else:
+            a, _ = ops.glu(ops.linear(h, self.up, defer=h.is_cuda and h.shape[0] <= 128))
+        return ops.linear_act(a, self.down)
 
 
-def build_experts(moe: MoeConfig, width: int, device, router: torch.Tensor, correction: Optional[torch.Tensor], experts):
-    """Stacked expert weights for the grouped GEMMs: per expert gate | up [2F, W] and down [W, F] with F padded
-    to 64 and W (as output) to 128. ``experts`` yields (gate, up, down)."""
+class TokenInput:
+    """What a layer adds from its part of a second token embedding: ``proj(gelu_tanh(gate x) * table[token])``; the
+    norm of the sum's new term is the caller's. ``table`` [vocab, dim] is the layer's columns, padded to 8."""
+
+    def __init__(self, dim: int, width: int, device, *, table: torch.Tensor, gate: torch.Tensor, proj: torch.Tensor):
+        dp, wp = pad_to(dim, 8), pad_to(width, 8)
+        self.table = table
+        self.gate = _linear([pad_rows(pad_cols(gate, wp), dp)], device)
+        self.proj = _linear([pad_rows(pad_cols(proj, dp), wp)], device)
+
+    def nbytes(self) -> int:
+        return self.gate.nbytes() + self.proj.nbytes() + self.table.numel() * self.table.element_size()
+
+    def __call__(self, x: torch.Tensor, tokens: torch.Tensor) -> torch.Tensor:
+        return ops.linear_act(ops.side_gate(ops.linear_act(x, self.gate), tokens, self.table), self.proj)
+
+
+def build_experts(moe: MoeConfig, width: int, device, router: torch.Tensor, correction: Optional[torch.Tensor], experts, shared=None):
+    """Stacked expert weights for the grouped GEMMs: per expert gate | up [2F, W] (up [F, W] for experts without a gate)
+    and down [W, F] with F padded to 64 and W (as output) to 128. ``experts`` yields (gate or None, up, down);
+    ``shared``: (up, down, sigmoid gate [1, W]) of an ungated shared expert, whose gate becomes the router's last row."""
     from .moe import MoeWeights
     wp, f, fp, wo = pad_to(width, 8), moe.expert_ffn, pad_to(moe.expert_ffn, 64), pad_to(width, 128)
-    gu = torch.zeros(moe.num_experts, 2, fp, wp, dtype=torch.bfloat16, device=device)
+    halves = 1 if moe.expert_act == "relu2" else 2
+    if halves == 1:
+        fp = pad_to(f, 128)                    # the up product's own rows are tiles of 128
+    gu = torch.zeros(moe.num_experts, halves, fp, wp, dtype=torch.bfloat16, device=device)
     dn = torch.zeros(moe.num_experts, wo, fp, dtype=torch.bfloat16, device=device)
     for i, (g, u, d) in enumerate(experts):
-        gu[i, 0, :f, :width] = g.to(gu)
-        gu[i, 1, :f, :width] = u.to(gu)
+        if halves == 2:
+            gu[i, 0, :f, :width] = g.to(gu)
+        gu[i, halves - 1, :f, :width] = u.to(gu)
         dn[i, :width, :f] = d.to(dn)
-    return MoeWeights(router=LinearWeight(pad_cols(router, wp).to(torch.bfloat16).to(device).contiguous()),
-                      router_bias=None if correction is None else correction.float().to(device).contiguous(),
-                      gate_up=LinearWeight(gu.reshape(moe.num_experts * 2 * fp, wp)), down=LinearWeight(dn.reshape(moe.num_experts * wo, fp)))
+    w = MoeWeights(router=_linear([pad_cols(router, wp)] + ([] if shared is None else [pad_cols(shared[2], wp)]), device),
+                   router_bias=None if correction is None else correction.float().to(device).contiguous(),
+                   gate_up=LinearWeight(gu.reshape(moe.num_experts * halves * fp, wp)), down=LinearWeight(dn.reshape(moe.num_experts * wo, fp)))
+    if shared is not None:
+        sp = pad_to(shared[0].shape[0], 8)
+        w.shared_gate_up = _linear([pad_rows(pad_cols(shared[0], wp), sp)], device)
+        w.shared_down = _linear([pad_rows(pad_cols(shared[1], sp), wp)], device)
+        w.gate_in_router = True
+    return w
 
 
 def spec_param_count(ls: LayerSpec, width: int) -> int:
     m = ls.mixer
     if m.kind == "latent_attention":
-        n = width * (m.q_rank + m.kv_rank + 2 * m.heads * m.vdim) + m.heads * (m.q_rank * m.dim + m.kv_rank * (m.dim + m.vdim))
+        n = width * (m.q_rank + m.kv_rank + m.rot_dim + (1 + m.out_gate) * m.heads * m.vdim)
+        n += m.heads * (m.q_rank * (m.dim + m.rot_dim) + m.kv_rank * (m.dim + m.vdim))
     elif m.kind == "channel_scan":
         n = m.inner * (3 * width + 2 * m.rank + 3 * m.state + m.conv)
     elif m.kind == "head_scan":
         n = width * (3 * m.heads * m.vdim + 2 * m.groups * m.state + m.heads) + m.conv * (m.heads * m.vdim + 2 * m.groups * m.state)
     elif m.kind == "attention":
-        n = width * m.dim * (m.heads * (2 + m.out_gate) + m.kv_heads * (1 if m.shared_kv else 2))
+        v = m.dim if m.shared_kv else m.vdim
+        n = width * (m.heads * (m.dim + (1 + m.out_gate) * v) + m.kv_heads * (m.dim + (0 if m.shared_kv else v)))
     else:
         r = m.rank or m.dim
         n = width * (2 * m.kv_heads * m.dim + 2 * m.heads * m.vdim + m.heads + 2 * r) + r * m.heads * (m.dim + m.vdim)
     if ls.moe is not None:
-        n += 3 * width * ls.moe.expert_ffn * ls.moe.num_experts + width * ls.moe.choices
+        mats = 2 if ls.moe.expert_act == "relu2" else 3
+        n += mats * width * (ls.moe.expert_ffn * ls.moe.num_experts + ls.moe.shared_ffn * ls.moe.num_shared_experts)
+        n += width * (ls.moe.choices + ls.moe.shared_gate)
     if ls.dense is not None:
-        n += 2 * width * ls.dense.ffn
+        n += (3 if ls.dense.act == "silu" else 2) * width * ls.dense.ffn
     return n + 4 * width

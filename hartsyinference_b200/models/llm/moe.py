@@ -45,6 +45,7 @@ class MoeWeights:
     shared_gate_up: Optional[LinearWeight] = None   # [2 * Fs / W, H]
     shared_down: Optional[LinearWeight] = None      # [H, Fs / W]
     shared_gate: Optional[LinearWeight] = None      # [1, H] sigmoid gate of the shared expert (Qwen2-MoE)
+    gate_in_router: bool = False                    # that gate is the router weight's last row (32-bit routing)
 
 
 class MoeFeedForward:
@@ -73,11 +74,12 @@ class MoeFeedForward:
         return n
 
     # ---------------------------------------------------------------------------------- pieces
-    def route(self, h: torch.Tensor) -> tuple[torch.Tensor, torch.Tensor]:
+    def route(self, h: torch.Tensor) -> tuple:
         m = self.moe
         if m.exact_router:
             return ops.router(h, self.w.router, self.w.router_bias, m.top_k, sigmoid=m.scoring == "sigmoid",
-                              norm_topk=m.norm_topk_prob, scale=m.routed_scaling_factor)
+                              norm_topk=m.norm_topk_prob, scale=m.routed_scaling_factor, n_group=m.n_group, topk_group=m.topk_group,
+                              gate=self.w.gate_in_router)
         logits = ops.linear(h, self.w.router)
         if not logits.is_cuda:
             logits = logits.float()
@@ -86,32 +88,39 @@ class MoeFeedForward:
                              scale=m.routed_scaling_factor)
 
     def _activate(self, gu: torch.Tensor, plan=None) -> torch.Tensor:
+        if self.moe.expert_act == "relu2":       # in the epilogue of the product before it
+            return gu
         if self.moe.glu_limit > 0:
             return ops.glu_clamped(gu, self.moe.glu_limit, self.moe.glu_alpha, plan)
         return ops.glu(gu, self.cfg.activation)[0]
 
     def routed_rows(self, h: torch.Tensor) -> "ops.RoutedRows":
         """Expert outputs of every row of ``h`` (bf16 or fp32) with their slots and weights, for a consumer
-        that combines them (``ops.residual_norm``). Single rank, no shared expert, no token limit."""
+        that combines them (``ops.residual_norm``); the shared expert's rows and gates go with them. Single rank, no
+        token limit."""
         m, w = self.moe, self.w
-        assert self.world == 1 and w.shared_gate_up is None
-        ids, wts = self.route(h)
+        assert self.world == 1 and (w.shared_gate_up is None or w.gate_in_router)
+        act = m.expert_act if m.expert_act == "relu2" else None
+        ids, wts, *gate = self.route(h)
         source = h if m.identity_experts > 0 else None
+        extra = {}
+        if w.shared_gate_up is not None:
+            extra = dict(extra=ops.linear_act(ops.linear_act(h, w.shared_gate_up, act), w.shared_down), extra_weight=gate[0])
         if h.is_cuda and h.dtype == torch.bfloat16:
             cap = ops.moe_block_capacity(h.shape[0], m.top_k, m.choices)
             blocks = (h.shape[0] * m.top_k + cap - 1) // cap + self.e_local
             # rows of slots without a token are computed and never read: they need no value
             xs = torch.empty(blocks * cap, self.hidden, dtype=h.dtype, device=h.device)
             plan = ops.moe_dispatch_dynamic(h, ids, 0, self.e_local, cap, xs)
-            gu = ops.grouped_linear_dynamic(xs, w.gate_up, self.e_local, plan)
+            gu = ops.grouped_linear_dynamic(xs, w.gate_up, self.e_local, plan, act=act)
             y = ops.grouped_linear_dynamic(self._activate(gu, plan), w.down, self.e_local, plan)
-            return ops.RoutedRows(y, plan.slot_of, ids, wts, source, m.num_experts)
+            return ops.RoutedRows(y, plan.slot_of, ids, wts, source, m.num_experts, **extra)
         # 32-bit products (and CPU tensors): one product per (token, choice) pair
-        gu = ops.pair_linear_f32(h, w.gate_up, ids, m.num_experts, m.top_k)
+        gu = ops.pair_linear_f32(h, w.gate_up, ids, m.num_experts, m.top_k, act)
         y = ops.pair_linear_f32(self._activate(gu), w.down, ids, m.num_experts, 1)
         pair = torch.arange(ids.numel(), dtype=torch.int32, device=h.device).reshape(ids.shape)
         slot_of = torch.where(ids < m.num_experts, pair, torch.full_like(pair, -1))
-        return ops.RoutedRows(y, slot_of, ids, wts, source, m.num_experts)
+        return ops.RoutedRows(y, slot_of, ids, wts, source, m.num_experts, **extra)
 
     def _shared(self, h: torch.Tensor) -> Optional[torch.Tensor]:
         w = self.w
@@ -190,7 +199,7 @@ class MoeFeedForward:
     # ---------------------------------------------------------------------------------- forward
     def __call__(self, h: torch.Tensor, model=None) -> torch.Tensor:
         t = h.shape[0]
-        if self.moe.identity_experts > 0 or self.moe.glu_limit > 0:
+        if self.moe.identity_experts > 0 or self.moe.glu_limit > 0 or self.moe.expert_act != "glu":
             acc = torch.zeros(t, self.hidden, dtype=torch.float32, device=h.device)
             ops.residual_norm(acc, self.routed_rows(h), None, None, dim=self.hidden, eps=0.0, layernorm=False, dtype=h.dtype)
             return acc.to(h.dtype)

@@ -21,7 +21,7 @@ from __future__ import annotations
 
 import math
 from dataclasses import dataclass
-from typing import Callable, Optional
+from typing import Callable, Optional, Union
 
 import torch
 
@@ -29,6 +29,7 @@ from ... import config, ops
 from ...ops import LinearWeight
 from ...parallel.comm import Comm, SingleComm
 from .config import RopeScaling, TransformerConfig, mixed_design
+from .rope import build_inv_freq
 
 
 @dataclass
@@ -55,37 +56,6 @@ class ForwardBatch:
     plan: Optional[object] = None                   # what a mixer works out once per batch for all its layers
 
 
-def build_inv_freq(rot: int, theta: float, scaling: RopeScaling, device) -> tuple[torch.Tensor, float]:
-    """Inverse rotary frequencies with linear / llama3 / YaRN scaling, and the attention factor.
-    (Reference: src/HartsyInference.Core/Rope/RopeFrequencyBuilder.cs, RopeScaling.cs.)"""
-    inv = theta ** (-torch.arange(0, rot, 2, dtype=torch.float64) / rot)
-    attn_factor = 1.0
-    if scaling.kind == "linear":
-        inv = inv / scaling.factor
-    elif scaling.kind == "llama3":
-        low = scaling.original_max_position / scaling.low_freq_factor
-        high = scaling.original_max_position / scaling.high_freq_factor
-        wavelen = 2 * math.pi / inv
-        smooth = ((scaling.original_max_position / wavelen) - scaling.low_freq_factor) / (
-            scaling.high_freq_factor - scaling.low_freq_factor)
-        scaled = torch.where(wavelen > low, inv / scaling.factor, inv)
-        mid = (wavelen <= low) & (wavelen >= high)
-        scaled = torch.where(mid, (1 - smooth) * inv / scaling.factor + smooth * inv, scaled)
-        inv = scaled
-    elif scaling.kind == "yarn":
-        def corr_dim(n_rot):
-            return (rot * math.log(scaling.original_max_position / (n_rot * 2 * math.pi))) / (2 * math.log(theta))
-        lo, hi = corr_dim(scaling.beta_fast), corr_dim(scaling.beta_slow)
-        if scaling.truncate:
-            lo, hi = math.floor(lo), math.ceil(hi)
-        lo, hi = max(lo, 0), min(hi, rot // 2 - 1)
-        ramp = ((torch.arange(rot // 2, dtype=torch.float64) - lo) / max(hi - lo, 1e-3)).clamp(0, 1)
-        mask = 1 - ramp
-        inv = inv / scaling.factor * (1 - mask) + inv * mask
-        attn_factor = scaling.attn_factor * (0.1 * math.log(scaling.factor) + 1.0) if scaling.factor > 1 else 1.0
-    return inv.to(torch.float32).to(device), attn_factor
-
-
 def alibi_slopes(heads: int) -> torch.Tensor:
     """ALiBi head slopes: a geometric sequence for the largest power of two <= heads, then every
     other term of the sequence for twice that count to fill the remainder."""
@@ -100,10 +70,10 @@ def alibi_slopes(heads: int) -> torch.Tensor:
 
 @dataclass
 class LayerWeights:
-    in_norm: torch.Tensor
+    in_norm: Union[torch.Tensor, ops.TanhNorm, None]
     qkv: LinearWeight
     o: LinearWeight
-    post_norm: torch.Tensor
+    post_norm: Union[torch.Tensor, ops.TanhNorm, None]
     gate_up: Optional[LinearWeight] = None
     down: Optional[LinearWeight] = None
     q_norm: Optional[torch.Tensor] = None
@@ -119,6 +89,8 @@ class LayerWeights:
     cross: Optional[object] = None                    # cross-attention layer over vision states (Mllama) instead of a block
     act_params: Optional[tuple] = None                # xIELU: (alpha_p, alpha_n, beta, eps) as floats (Apertus)
     sinks: Optional[torch.Tensor] = None              # per-head sink logit in the attention softmax (gpt-oss)
+    side_module: Optional[object] = None              # callable (x, tokens) -> [T, W] added after the feed-forward: token input
+    side_norm: Optional[torch.Tensor] = None          # RMS norm of what it adds
 
 
 def x_is_cuda(x) -> bool:
@@ -583,7 +555,8 @@ class DecoderModel:
         return MlaAttention(cfg, shard, hl)
 
     def weight_bytes(self) -> int:
-        n = self.embed.numel() * 2 + self.final_norm.numel() * 2
+        fn = self.final_norm
+        n = self.embed.numel() * 2 + (2 * fn.weight.numel() if isinstance(fn, ops.TanhNorm) else fn.numel()) * 2
         if self.lm_head.weight.data_ptr() != self.embed.data_ptr():
             n += self.lm_head.nbytes()
         for lw in {id(lw): lw for lw in self.layers}.values():      # layers can share weights
@@ -596,6 +569,8 @@ class DecoderModel:
                 n += lw.ffn_module.nbytes()
             if lw.attn_module is not None and hasattr(lw.attn_module, "nbytes"):
                 n += lw.attn_module.nbytes()
+            if lw.side_module is not None:
+                n += lw.side_module.nbytes()
             if lw.attn_dp is not None:      # the all-head copy (its head shard above may share storage with it)
                 n += lw.attn_dp.nbytes()
         return n
@@ -868,7 +843,8 @@ class DecoderModel:
             mixer -> x += norm1b(y), h = norm2(x)                          [one launch]
             experts -> x += norm2b(sum of expert rows), h = norm1'(x)      [one launch]
 
-        Without norms ahead of the sublayers (``pre_norm`` off) h is x itself in the activation type. ``capture`` (a list) receives a copy of the stream after every layer."""
+        With a token input behind the feed-forward, h in the last line is x itself in the activation type, and
+        side(h, tokens) -> x += rms(y), h = norm1'(x) is one more. Without norms ahead of the sublayers (``pre_norm`` off) h is x itself in the activation type. ``capture`` (a list) receives a copy of the stream after every layer."""
         cfg = self.cfg
         kw = dict(dim=cfg.hidden_size, eps=cfg.rms_eps, layernorm=cfg.norm_type == "layernorm", dtype=self.dtype,
                   plus_one=cfg.norm_plus_one, mult=cfg.residual_multiplier, plain=not cfg.pre_norm)
@@ -891,11 +867,18 @@ class DecoderModel:
         for li, lw in enumerate(self.layers):
             after = self.final_norm if li == last else self.layers[li + 1].in_norm
             y = lw.attn_module(h, batch, li, self)
-            h = ops.residual_norm(x, y, lw.post_attn_norm, lw.post_norm if lw.ffn_module is not None else after, **kw)
-            if hasattr(lw.ffn_module, "routed_rows"):
-                h = self._routed_sublayer(lw, x, h, after, kw)
-            elif lw.ffn_module is not None:
-                h = ops.residual_norm(x, lw.ffn_module(h), lw.post_ffn_norm, after, **kw)
+            # the stream goes to the token input as it is
+            end, kwe = (after, kw) if lw.side_module is None else (None, {**kw, "plain": True})
+            if lw.ffn_module is None:
+                h = ops.residual_norm(x, y, lw.post_attn_norm, end, **kwe)
+            else:
+                h = ops.residual_norm(x, y, lw.post_attn_norm, lw.post_norm, **kw)
+                if hasattr(lw.ffn_module, "routed_rows"):
+                    h = self._routed_sublayer(lw, x, h, end, kwe)
+                else:
+                    h = ops.residual_norm(x, lw.ffn_module(h), lw.post_ffn_norm, end, **kwe)
+            if lw.side_module is not None:
+                h = ops.residual_norm(x, lw.side_module(h, batch.tokens), lw.side_norm, after, **kw)
             if capture is not None:
                 capture.append(x[:, :cfg.hidden_size].clone())
         return h

@@ -56,6 +56,7 @@ from .mixers import (  # noqa: F401
     DeltaWeights,
     HeadScanWeights,
     RoutedRows,
+    TanhNorm,
     attn_biased,
     attn_runs,
     channel_scan,
@@ -73,9 +74,12 @@ from .mixers import (  # noqa: F401
     linear_act,
     pair_linear_f32,
     poly_norm,
+    qk_rope_store,
     residual_norm,
+    rope_table,
     router,
     short_conv,
+    side_gate,
 )
 from . import reference  # noqa: F401
 
@@ -102,7 +106,7 @@ def _install_ranges() -> None:
             setattr(mod, name, wrapped)
     for name in ("attn_biased", "attn_runs", "channel_scan", "delta_mix", "embedding_f32", "embedding_norm", "gated_norm", "glu_clamped",
                  "head_linear", "head_scan", "kv_store", "latent_attn", "latent_gather", "latent_prep", "pair_linear_f32", "poly_norm",
-                 "residual_norm", "router", "short_conv"):
+                 "qk_rope_store", "residual_norm", "rope_table", "router", "short_conv", "side_gate"):
         setattr(mod, name, traced(name)(getattr(mixers, name)))
 
 

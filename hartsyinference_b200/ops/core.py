@@ -11,7 +11,7 @@ import torch
 from . import _native as N
 from . import reference as R
 
-_ACT = {None: 0, "none": 0, "gelu_tanh": 1, "silu": 2}
+_ACT = {None: 0, "none": 0, "gelu_tanh": 1, "silu": 2, "relu2": 3}
 
 
 def fp8_mx() -> bool:

@@ -111,6 +111,8 @@ def linear(x: torch.Tensor, w: torch.Tensor, w_scale: Optional[torch.Tensor] = N
         y = gelu_tanh(y)
     elif act == "silu":
         y = torch.nn.functional.silu(y)
+    elif act == "relu2":
+        y = torch.relu(y) ** 2
     if gate is not None:
         y = y * gate.float()
     if residual is not None:
@@ -161,10 +163,10 @@ def glu(x: torch.Tensor, act: str = "silu") -> torch.Tensor:
     return a * u
 
 
-def glu_clamped(x: torch.Tensor, limit: float, alpha: float) -> torch.Tensor:
+def glu_clamped(x: torch.Tensor, limit: float, alpha: float, shift: float = 1.0) -> torch.Tensor:
     f = x.shape[-1] // 2
     g, u = x[..., :f].float().clamp(max=limit), x[..., f:].float().clamp(-limit, limit)
-    return g * torch.sigmoid(alpha * g) * (u + 1.0)
+    return g * torch.sigmoid(alpha * g) * (u + shift)
 
 
 def delta_mix(proj, z, w, conv_state, state, positions, cu_q, slots, b_off) -> torch.Tensor:
@@ -303,18 +305,36 @@ def apply_rope(x: torch.Tensor, positions: torch.Tensor, inv_freq: torch.Tensor,
     return torch.cat([out, rest], dim=-1)
 
 
+def rope_table(positions: torch.Tensor, hi: torch.Tensor, lo: torch.Tensor) -> torch.Tensor:
+    """fp32 [T, n, 2] cosines and sines of position * (hi + lo)."""
+    ang = positions.double()[:, None] * (hi.double() + lo.double())[None]
+    return torch.stack([ang.cos(), ang.sin()], -1).float()
+
+
+def turn(x: torch.Tensor, table: torch.Tensor, interleaved: bool) -> torch.Tensor:
+    """x [T, H, D] with its first 2 n values turned by ``table`` [T, n, 2]; fp32."""
+    n = table.shape[1]
+    c, s = table[:, None, :, 0], table[:, None, :, 1]
+    xf = x.float()
+    r = xf[..., :2 * n]
+    u, v = (r[..., 0::2], r[..., 1::2]) if interleaved else (r[..., :n], r[..., n:])
+    a, b = u * c - v * s, v * c + u * s
+    return torch.cat([torch.stack([a, b], -1).flatten(-2) if interleaved else torch.cat([a, b], -1), xf[..., 2 * n:]], -1)
+
+
 # --------------------------------------------------------------------------------------------
 # attention
 # --------------------------------------------------------------------------------------------
 def attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, causal: bool = False,
               scale: Optional[float] = None, softcap: float = 0.0, window: int = 0,
               alibi: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None,
-              dist_bias: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """q [Tq, Hq, D], k/v [Tk, Hkv, D] (one sequence). The last query row sits at key position
+              dist_bias: Optional[torch.Tensor] = None, keep_first: int = 0) -> torch.Tensor:
+    """q [Tq, Hq, D], k [Tk, Hkv, D], v [Tk, Hkv, Dv] (one sequence). The last query row sits at key position
     Tk - 1 (so a query chunk with a cached prefix is expressed by Tk > Tq). ``alibi`` [Hq] adds
     slope * key position to the scores; ``dist_bias`` [Hq, n] adds a value by key distance (its last
     entry also for longer distances); ``sinks`` [Hq] adds one extra logit per head to the softmax
-    denominator (it attends to nothing). Returns fp32 [Tq, Hq, D]."""
+    denominator (it attends to nothing). The ``keep_first`` first keys stay visible outside the window. Returns fp32
+    [Tq, Hq, Dv]."""
     tq, hq, d = q.shape
     tk, hkv, _ = k.shape
     g = hq // hkv
@@ -330,7 +350,7 @@ def attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, causal: bool = 
     if causal:
         mask &= kpos <= qpos
     if window > 0:
-        mask &= kpos > qpos - window
+        mask &= (kpos > qpos - window) | (kpos < keep_first)
     if alibi is not None:
         s = s + alibi.float()[:, None, None] * kpos[None].float()
     if dist_bias is not None:
