@@ -72,10 +72,10 @@ def visible(i, mask):
     return [j for j in range(i + 1) if size <= 0 or i - j < size or j < first]
 
 
-def masked_attention(q, k, v, scale, mask):
-    """One head, q, k [T, D], v [T, V]."""
+def masked_attention(q, k, v, scale, mask, first=0):
+    """One head, q, k [T, D], v [T, V]; outputs from position ``first`` on."""
     out = []
-    for i in range(q.shape[0]):
+    for i in range(first, q.shape[0]):
         at = visible(i, mask)
         s = (k[at] @ q[i]) * scale
         e = torch.exp(s - s.max())
