@@ -229,8 +229,8 @@ struct WarpState {
 //   (keys >= limit are masked), row_start[r]: first visible key (sliding window).
 //   Extended form: row_bias[r] is the row's distance-bias table (the distance of a key is counted back
 //   from row_limit[r] - 1).
-template <int D, int NG, bool kExt = false>
-__device__ __forceinline__ void warp_tile(WarpState<D>& st, const uint32_t (&qf)[D / 16][4],
+template <int D, int NG, bool kExt = false, int DV = D>
+__device__ __forceinline__ void warp_tile(WarpState<DV>& st, const uint32_t (&qf)[D / 16][4],
                                           uint32_t k_smem, uint32_t v_smem, int t_begin,
                                           int tok0, const int (&row_limit)[2],
                                           const int (&row_start)[2], const AttnParams& p,
@@ -323,7 +323,7 @@ __device__ __forceinline__ void warp_tile(WarpState<D>& st, const uint32_t (&qf)
     st.l[r] = st.l[r] * alpha[r] + rs[r];
   }
 #pragma unroll
-  for (int i = 0; i < D / 8; ++i) {
+  for (int i = 0; i < DV / 8; ++i) {
     st.o[i][0] *= alpha[0];
     st.o[i][1] *= alpha[0];
     st.o[i][2] *= alpha[1];
@@ -333,12 +333,12 @@ __device__ __forceinline__ void warp_tile(WarpState<D>& st, const uint32_t (&qf)
 #pragma unroll
   for (int gi = 0; gi < NG; ++gi) {
 #pragma unroll
-    for (int np = 0; np < D / 16; ++np) {
+    for (int np = 0; np < DV / 16; ++np) {
       const int mi = lane >> 3;
       const int token = t_begin + gi * 16 + (lane & 7) + 8 * (mi & 1);
       const int chunk = np * 2 + (mi >> 1);
       uint32_t b0, b1, b2, b3;
-      ldmatrix_x4_trans(v_smem + tile_off<D>(token, chunk), b0, b1, b2, b3);
+      ldmatrix_x4_trans(v_smem + tile_off<DV>(token, chunk), b0, b1, b2, b3);
       mma_bf16_16816(st.o[np * 2], pf[gi], b0, b1);
       mma_bf16_16816(st.o[np * 2 + 1], pf[gi], b2, b3);
       if (kExt) {
@@ -573,7 +573,8 @@ __global__ void attn_combine_kernel(const AttnParams p) {
 // ------------------------------------------------------------------------------------------
 // prefill / full attention
 // ------------------------------------------------------------------------------------------
-template <int D, bool kPaged, bool kExt = false>
+// DV: width of the value tiles (D but for keys of 192, which come with values of at most 128)
+template <int D, bool kPaged, bool kExt = false, int DV = D>
 __global__ void __launch_bounds__(kAttnThreads)
 attn_prefill_kernel(const AttnParams p) {
   constexpr int kStages = 2;
@@ -588,7 +589,7 @@ attn_prefill_kernel(const AttnParams p) {
   const int q_len = kExt && p.q_lens ? p.q_lens[seq] : p.cu_q ? p.cu_q[seq + 1] - q_off : p.q_len_single;
   const int kv_len = p.kv_lens ? p.kv_lens[seq] : p.kv_len_single;
   if (qt * 64 >= q_len) return;
-  const int stage_bytes = kExt && p.shared_kv ? kTileBytes : 2 * kTileBytes;
+  const int stage_bytes = kExt && p.shared_kv ? kTileBytes : kTileBytes + kTileTokens * DV * 2;
   const int ctx = kv_len - q_len;   // keys that precede the first query token
   const uint32_t smem_base = smem_u32(smem);
 
@@ -628,7 +629,7 @@ attn_prefill_kernel(const AttnParams p) {
         }
       }
   }
-  WarpState<D> st;
+  WarpState<DV> st;
   st.init();
   int lim[2], start[2];
 #pragma unroll
@@ -677,7 +678,7 @@ attn_prefill_kernel(const AttnParams p) {
       const int tok0 = tile_of(step) * kTileTokens;
       if (kExt && !kPaged) {
         load_tile_linear<D, true>(kb, kbase, p.k_ld, tok0, kv_needed, p.d, k2base, p.k2_ld, p.d_own);
-        load_tile_linear<D, true>(kb + kTileBytes, vbase, p.v_ld, tok0, kv_needed, p.dv);
+        load_tile_linear<DV, true>(kb + kTileBytes, vbase, p.v_ld, tok0, kv_needed, p.dv);
       } else if (kExt) {
         load_tile_paged<D, true>(kb, p.k, pages, kvh, p.hkv, p.page_shift, tok0, kv_needed, p.d);
         if (!p.shared_kv) load_tile_paged<D, true>(kb + kTileBytes, p.v, pages, kvh, p.hkv, p.page_shift, tok0, kv_needed, p.dv);
@@ -707,7 +708,7 @@ attn_prefill_kernel(const AttnParams p) {
     const uint32_t kb = smem_base + slot * stage_bytes;
     // a warp whose rows all lie before this tile (causal) still runs: masked scores cost nothing
     // in correctness and keep the barrier pattern uniform
-    warp_tile<D, 4, kExt>(st, qf, kb, kExt && p.shared_kv ? kb : kb + kTileBytes, 0, tile_of(step) * kTileTokens, lim, start, p,
+    warp_tile<D, 4, kExt, DV>(st, qf, kb, kExt && p.shared_kv ? kb : kb + kTileBytes, 0, tile_of(step) * kTileTokens, lim, start, p,
                           row_bias);
     __syncthreads();
     slot ^= 1;
@@ -723,7 +724,7 @@ attn_prefill_kernel(const AttnParams p) {
     if (row < q_len) {
       const float inv = st.l[r] > 0.f ? 1.f / st.l[r] : 0.f;
 #pragma unroll
-      for (int i = 0; i < D / 8; ++i) {
+      for (int i = 0; i < DV / 8; ++i) {
         const int c = i * 8 + tq * 2;
         if (kExt) {
           if (c < p.dv)
@@ -1087,14 +1088,14 @@ B200_API int b200_attn_biased(const void* q, const void* k_cache, const void* v_
 // Causal attention of the runs q_start[s] .. + q_lens[s] of q over contiguous keys and values of their whole
 // contexts (rows kv_start[s] .. + kv_lens[s] of k and v; the last key belongs to the run's last query; window > 0: the
 // last `window` keys of every query). q, out and gate are indexed by token: q [tokens][q_ld] (head h at h * d), out
-// [tokens][hq * dv]. d, dv <= 128, multiples of 8. The keys' columns from d_own on are rows of k2 for every head
+// [tokens][hq * dv]. d <= 192, dv <= 128, multiples of 8. The keys' columns from d_own on are rows of k2 for every head
 // (d_own = d: none); with rot_table [tokens][rot_pairs] (cos, sin) those columns of q are turned.
 B200_API int b200_attn_runs(const void* q, const void* k, const void* v, void* out, const void* gate, const int* q_start,
                             const int* q_lens, const int* kv_start, const int* kv_lens, int seqs, int max_q_len, int hq, int hkv,
                             int d, int dv, long long q_ld, long long k_ld, long long v_ld, long long gate_ld, float scale, int window,
                             const void* k2, int d_own, long long k2_ld, const void* rot_table, int rot_pairs, cudaStream_t stream) {
   if (seqs <= 0 || max_q_len <= 0) return 0;
-  if (d % 8 || dv % 8 || d < 8 || dv < 8 || d > 128 || dv > 128 || hq % hkv || q_ld % 8 || k_ld % 8 || v_ld % 8 || gate_ld % 8 ||
+  if (d % 8 || dv % 8 || d < 8 || dv < 8 || d > 192 || dv > 128 || hq % hkv || q_ld % 8 || k_ld % 8 || v_ld % 8 || gate_ld % 8 ||
       seqs > 65535)
     return -2;
   if (d_own % 8 || d_own > d || k2_ld % 8 || (d_own < d && !k2) || (rot_table && 2 * rot_pairs > d - d_own)) return -2;
@@ -1115,12 +1116,13 @@ B200_API int b200_attn_runs(const void* q, const void* k, const void* v, void* o
   p.rot_table = static_cast<const float2*>(rot_table); p.rot_pairs = rot_pairs;
   const dim3 grid((max_q_len + 63) / 64, hq, seqs);
   auto go = [&](auto kernel, int dd, PerDeviceOnce& once) {
-    const int smem = 2 * 2 * kTileTokens * dd * 2;
+    const int smem = 2 * kTileTokens * (dd + (dd > 128 ? 128 : dd)) * 2;
     if (once.first_time()) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     kernel<<<grid, kAttnThreads, smem, stream>>>(p);
   };
-  static PerDeviceOnce once[2];
-  if (d > 64 || dv > 64) go(attn_prefill_kernel<128, false, true>, 128, once[1]);
+  static PerDeviceOnce once[3];
+  if (d > 128) go(attn_prefill_kernel<192, false, true, 128>, 192, once[2]);
+  else if (d > 64 || dv > 64) go(attn_prefill_kernel<128, false, true>, 128, once[1]);
   else go(attn_prefill_kernel<64, false, true>, 64, once[0]);
   const cudaError_t e = cudaGetLastError();
   return e == cudaSuccess ? 0 : -static_cast<int>(e) - 300;

@@ -21,9 +21,10 @@ __global__ void __launch_bounds__(256) rope_table_kernel(const int* __restrict__
   const int j = static_cast<int>(i - t * pairs);
   const float pos = static_cast<float>(positions[t]);
   const float a = pos * hi[j], rest = fmaf(pos, hi[j], -a) + pos * lo[j];
-  float s, c;
+  float s, c, rs, rc;
   sincosf(a, &s, &c);
-  out[i] = make_float2(fmaf(-s, rest, c), fmaf(c, rest, s));
+  sincosf(rest, &rs, &rc);
+  out[i] = make_float2(c * rc - s * rs, s * rc + c * rs);
 }
 
 struct QkRopeParams {

@@ -383,7 +383,7 @@ class LatentAttention:
         return (1, pages, 1, page, self.r + self.t)
 
     def _plan(self, batch, h: torch.Tensor) -> LatentPlan:
-        expand = h.is_cuda and h.dtype == torch.bfloat16 and max(self.d + self.t, self.v) <= 128
+        expand = h.is_cuda and h.dtype == torch.bfloat16 and self.d + self.t <= 192 and self.v <= 128
         if batch.plan is None:
             batch.plan = {}
         key = (expand, self.spec.window)

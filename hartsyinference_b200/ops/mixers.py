@@ -629,7 +629,7 @@ def attn_runs(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, out: torch.Tens
     [.., heads * d] and ``v`` [.., heads * dv]; the last key belongs to the last query, and with a ``window`` a query sees the
     last ``window`` keys up to its own. ``k_shared`` [.., n]: the last n values of every key head, the same for all heads
     (heads of ``k`` are then d - n wide), the query's side of which is turned by ``table`` [T, pairs, 2]. Rows of the runs are
-    written to ``out`` [T, heads * dv], times ``sigmoid(gate)``. bf16, d and dv up to 128."""
+    written to ``out`` [T, heads * dv], times ``sigmoid(gate)``. bf16, d up to 192 and dv up to 128."""
     own, dv = k.shape[1] // heads, v.shape[1] // heads
     d = own + (0 if k_shared is None else k_shared.shape[1])
     assert q.is_cuda and q.dtype == torch.bfloat16 and out.is_contiguous() and q.stride(1) == k.stride(1) == v.stride(1) == 1

@@ -533,11 +533,26 @@ def built(case, mode):
     return _BUILT[case, mode]
 
 
-def expected(case, tokens):
+def _expected(case, tokens):
     key = (case, tuple(tokens))
     if key not in _WANT:
-        _WANT[key] = O.forward(tokens, CASES[case], rand_weights(CASES[case]))
+        clear = []
+        y = O.forward(tokens, CASES[case], rand_weights(CASES[case]), clear=clear)
+        _WANT[key] = y, torch.tensor(clear).amin(0) if clear else torch.ones(len(tokens))
     return _WANT[key]
+
+
+def expected(case, tokens):
+    return _expected(case, tokens)[0]
+
+
+def check(got, case, tokens, mode):
+    """Logits of all positions. In bf16 a token for which two experts or groups are as good as tied may take the other
+    one: such positions are left out there."""
+    want, clear = _expected(case, tokens)
+    sure = clear > (0.0 if mode[1] == F32 else 0.005)
+    assert int(sure.sum()) >= 0.6 * len(tokens) or len(tokens) < 10
+    logits_near(got.cpu()[sure], want[sure], mode)
 
 
 def prompt(case, n, seed):
@@ -550,10 +565,9 @@ def test_model_cuts(mode, case):
     """Whole prompt, token by token, and portions: the same logits at every position."""
     _, _, model = built(case, mode)
     toks = prompt(case, 110, 1)
-    want = expected(case, toks)
     eng = engine(model)
     for cuts in ([110], [1] * 110, [2] * 55, [16, 1, 1, 15, 2, 75], [3, 5, 7, 11, 13, 17, 54], [50, 48] + [1] * 12):
-        logits_near(play(eng, toks, cuts), want, mode)
+        check(play(eng, toks, cuts), case, toks, mode)
         assert eng.kv.num_free == eng.num_pages
 
 
@@ -582,7 +596,7 @@ def test_model_mixed_batches(mode, case):
             y = y[n:]
     assert all(at[k] == len(seqs[k]) for k in seqs) and eng.kv.num_free == eng.num_pages
     for k in seqs:
-        logits_near(torch.cat(got[k]), expected(case, seqs[k]), mode)
+        check(torch.cat(got[k]), case, seqs[k], mode)
 
 
 @pytest.mark.parametrize("mode", MODES)
@@ -607,7 +621,7 @@ def test_model_stream_per_layer(mode):
 def test_long_decode(mode):
     _, _, model = built("mixed", mode)
     toks = prompt("mixed", 150, 4)
-    logits_near(play(engine(model), toks, [4] + [1] * 146), expected("mixed", toks), mode)
+    check(play(engine(model), toks, [4] + [1] * 146), "mixed", toks, mode)
 
 
 @pytest.mark.parametrize("mode", MODES)

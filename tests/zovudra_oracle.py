@@ -134,9 +134,27 @@ def choose(scores, router):
     return sorted(allowed, key=lambda e: (-scores[e], e))[:router["top"]]
 
 
-def moe_ff(h, mlp, w, p):
+def clearance(scores, router):
+    """How far one token's choice is from another one: the smallest gap between what was taken and what was left."""
+    n, out = len(scores), []
+    grp = router.get("groups")
+    allowed = list(range(n))
+    if grp:
+        size = n // grp["count"]
+        value = [sum(sorted(scores[g * size:(g + 1) * size], reverse=True)[:2]) for g in range(grp["count"])]
+        best = sorted(range(grp["count"]), key=lambda g: -value[g])
+        out += [value[a] - value[b] for a, b in zip(best[grp["keep"] - 1:], best[grp["keep"]:][:1])]
+        allowed = [e for e in allowed if e // size in best[:grp["keep"]]]
+    rest = sorted((scores[e] for e in allowed), reverse=True)
+    out += [a - b for a, b in zip(rest[router["top"] - 1:], rest[router["top"]:][:1])]
+    return min(out, default=1.0)
+
+
+def moe_ff(h, mlp, w, p, clear=None):
     r = mlp["router"]
     scores = sigmoid(h @ w[p + "router"].T)
+    if clear is not None:
+        clear.append([clearance(row, r) for row in scores.tolist()])
     out = torch.zeros_like(h)
     for t in range(h.shape[0]):
         ids = choose(scores[t].tolist(), r)
@@ -154,8 +172,9 @@ def side_input(x, e, w, p, eps):
     return rms(y, w[p + "norm"], eps)
 
 
-def forward(tokens, cfg, weights, dtype=torch.float64, layers_out=None):
-    """Logits [T, vocab]; ``layers_out`` (a list) receives the stream after every layer."""
+def forward(tokens, cfg, weights, dtype=torch.float64, layers_out=None, clear=None):
+    """Logits [T, vocab]; ``layers_out`` (a list) receives the stream after every layer, ``clear`` the tokens'
+    :func:`clearance` in every routed layer."""
     w = {n: t.to(dtype) for n, t in weights.items()}
     eps, ids = cfg["norm"]["eps"], torch.as_tensor(tokens)
     norm = lambda v, name: tanh_norm(v, w[name + ".alpha"], w[name], w[name + ".b"])
@@ -166,7 +185,7 @@ def forward(tokens, cfg, weights, dtype=torch.float64, layers_out=None):
         x = x + mixer(norm(x, p + "norm1"), mix, w, p + "mix.", eps)
         if mlp is not None:
             h = norm(x, p + "norm2")
-            x = x + (dense_ff(h, w, p + "mlp.") if mlp["kind"] == "dense" else moe_ff(h, mlp, w, p + "mlp."))
+            x = x + (dense_ff(h, w, p + "mlp.") if mlp["kind"] == "dense" else moe_ff(h, mlp, w, p + "mlp.", clear))
         if cfg.get("token_side"):
             n = cfg["token_side"]["dim"]
             x = x + side_input(x, w["side.embed"][ids, i * n:(i + 1) * n], w, p + "side.", eps)
