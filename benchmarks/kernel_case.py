@@ -10,6 +10,8 @@
     python benchmarks/kernel_case.py channel_scan 4 2048 4096
     python benchmarks/kernel_case.py head_scan 4 2048 64
     python benchmarks/kernel_case.py latent 64 2048 16
+    python benchmarks/kernel_case.py latent_rot 4 2048 16 1024 runs
+    python benchmarks/kernel_case.py qk_rope 8192 16 4
 
 Inputs are larger than the L2 cache where the op is bandwidth bound but stay far below a few GB,
 so a full-metric capture (dozens of replays per launch) ends in about a minute. The status word is
@@ -378,7 +380,45 @@ def _latent(argv):
     print(f"latent {argv}: {_time_cold(fn) * 1e3:.1f} us")
 
 
-CASES = {"channel_scan": _channel_scan, "head_scan": _head_scan, "latent": _latent, "delta": _delta, "attn_window": _attn_window, "mla_proj": _mla_proj, "gemm_ar_large": _gemm_ar_large, "ag_gemm": _ag_gemm, "ulysses": _ulysses, "allreduce": _allreduce, "sample": _sample,
+def _turns(pos, dims, interleaved):
+    f = 1e6 ** (-torch.arange(0, dims, 2, device="cuda", dtype=torch.float32) / dims)
+    return ops.rope_table(pos, f, torch.zeros_like(f))
+
+
+def _latent_rot(argv):
+    """latent_rot SEQS CONTEXT HEADS WINDOW [runs]: decode attention over cached latents of 512 values and a rotated key
+    of 64, or with "runs" the attention of whole prompts over expanded keys of 128 + 64."""
+    seqs, n, h, win = (int(v) for v in argv[:4])
+    dev, d, per = "cuda", 128, n // 16
+    bf = lambda *sh: torch.randn(*sh, device=dev).to(torch.bfloat16)
+    lens = torch.full((seqs,), n, dtype=torch.int32, device=dev)
+    if len(argv) > 4:
+        t = seqs * n
+        q, kv, c, out = bf(t, h * (d + 64)), bf(t, 2 * h * d), bf(t, 576), torch.empty(t, h * d, dtype=torch.bfloat16, device=dev)
+        at = torch.arange(0, t + 1, n, dtype=torch.int32, device=dev)
+        table = _turns(torch.arange(t, dtype=torch.int32, device=dev) % n, 64, True)
+        fn = lambda: ops.attn_runs(q, kv[:, :h * d], kv[:, h * d:], out, at[:-1], lens, at, lens, heads=h, max_q_len=n, scale=0.07, window=win,
+                                   k_shared=c[:, 512:], table=table)
+    else:
+        cache, q = bf(seqs * per, 1, 16, 576), bf(seqs, h * 576)
+        pages = torch.randperm(seqs * per, device=dev).to(torch.int32).reshape(seqs, per)
+        fn = lambda: ops.latent_attn(q, cache, pages, lens, h, 0.05, max_kv_len=n, v_dim=512, window=win)
+    print(f"latent_rot {argv}: {_time_cold(fn) * 1e3:.1f} us")
+
+
+def _qk_rope(argv):
+    """qk_rope TOKENS HEADS KV_HEADS: norms over all heads, rotation and page store of a q | k | v projection, heads of 128."""
+    t, h, kv = (int(v) for v in argv[:3])
+    dev = "cuda"
+    p, ones = torch.randn(t, (h + 2 * kv) * 128, device=dev).to(torch.bfloat16), torch.ones(h * 128, device=dev, dtype=torch.bfloat16)
+    kc, vc = (torch.zeros((t + 15) // 16, kv, 16, 128, device=dev, dtype=torch.bfloat16) for _ in range(2))
+    table = _turns(torch.arange(t, dtype=torch.int32, device=dev), 128, False)
+    slots = torch.randperm(t, device=dev)
+    fn = lambda: ops.qk_rope_store(p, h, kc, vc, slots, table=table, q_norm=ones, k_norm=ones[:kv * 128], eps=1e-6)
+    print(f"qk_rope {argv}: {_time_cold(fn) * 1e3:.1f} us")
+
+
+CASES = {"qk_rope": _qk_rope, "latent_rot": _latent_rot, "channel_scan": _channel_scan, "head_scan": _head_scan, "latent": _latent, "delta": _delta, "attn_window": _attn_window, "mla_proj": _mla_proj, "gemm_ar_large": _gemm_ar_large, "ag_gemm": _ag_gemm, "ulysses": _ulysses, "allreduce": _allreduce, "sample": _sample,
          "int8": _int8, "triplane": _triplane,
          "gemm_ar": _gemm_ar, "attn_dense": _attn_dense, "gemm": _gemm, "grouped": _grouped, "attn_decode": _attn_decode, "mla": _mla}
 
