@@ -178,7 +178,7 @@ def plant(q, k, rows, spots, head, group, gain=4.0):
 
 @pytest.mark.parametrize("mode", MODES)
 @pytest.mark.parametrize("hq,hkv,d,dv,page,window,keep,tail", [
-    (4, 2, 64, 64, 16, 40, 6, 1), (4, 2, 64, 64, 16, 40, 6, 70), (6, 2, 40, 24, 8, 17, 1, 3), (8, 8, 128, 64, 16, 65, 70, 130), (3, 1, 16, 104, 64, 1, 3, 5),
+    (6, 2, 64, 64, 16, 50, 7, 1), (6, 2, 64, 64, 16, 50, 7, 70), (6, 2, 40, 24, 8, 17, 1, 3), (8, 8, 128, 64, 16, 65, 70, 130), (3, 1, 16, 104, 64, 1, 3, 5),
     (20, 1, 24, 24, 16, 130, 65, 1), (2, 1, 160, 32, 16, 33, 9, 9), (16, 1, 96, 128, 32, 64, 64, 1), (4, 4, 8, 8, 16, 1000, 5, 2), (2, 1, 32, 32, 16, 20, 0, 40),
     (4, 1, 64, 64, 16, 0, 9, 50), (2, 2, 64, 128, 16, 16, 200, 40), (2, 1, 48, 200, 16, 70, 2, 33)])
 def test_window_with_kept_tokens(mode, hq, hkv, d, dv, page, window, keep, tail):
@@ -212,7 +212,7 @@ def test_window_with_kept_tokens(mode, hq, hkv, d, dv, page, window, keep, tail)
 
 
 @pytest.mark.parametrize("mode", MODES)
-@pytest.mark.parametrize("heads,rank,rot,page,window", [(4, 64, 32, 16, 40), (6, 40, 8, 8, 0), (17, 128, 64, 16, 70), (1, 96, 32, 64, 1), (33, 24, 104, 16, 130),
+@pytest.mark.parametrize("heads,rank,rot,page,window", [(5, 64, 48, 16, 40), (6, 40, 8, 8, 0), (17, 128, 64, 16, 70), (1, 96, 32, 64, 1), (33, 24, 104, 16, 130),
                                                         (3, 512, 64, 32, 65), (20, 264, 16, 16, 9), (2, 200, 56, 16, 64), (2, 160, 200, 16, 33), (2, 448, 64, 16, 50)])
 def test_latent_rows_with_rotated_part(mode, heads, rank, rot, page, window):
     """Queries in latent space: rows of the cache are keys, their first part the values; keys at the window's edge stand
@@ -248,7 +248,7 @@ def test_latent_rows_with_rotated_part(mode, heads, rank, rot, page, window):
 
 
 @pytest.mark.parametrize("mode", MODES)
-@pytest.mark.parametrize("heads,n,k,tail,rot,rows", [(3, 40, 24, 8, 6, 5), (6, 64, 64, 32, 32, 130), (2, 512, 128, 64, 64, 64), (16, 8, 200, 16, 10, 1)])
+@pytest.mark.parametrize("heads,n,k,tail,rot,rows", [(3, 40, 24, 8, 6, 5), (6, 72, 64, 32, 32, 130), (2, 512, 128, 64, 64, 64), (16, 8, 200, 16, 10, 1)])
 def test_head_linear_with_turned_tail(mode, heads, n, k, tail, rot, rows):
     dev, dt = mode
     g = gen(n + k)
@@ -267,7 +267,7 @@ def test_head_linear_with_turned_tail(mode, heads, n, k, tail, rot, rows):
 
 
 @pytest.mark.gpu
-@pytest.mark.parametrize("heads,own,rot,dv,window", [(4, 64, 32, 80, 136), (3, 40, 16, 24, 1), (2, 64, 64, 128, 64), (5, 16, 8, 104, 65), (2, 32, 32, 32, 0),
+@pytest.mark.parametrize("heads,own,rot,dv,window", [(3, 64, 48, 72, 130), (3, 40, 16, 24, 1), (2, 64, 64, 128, 64), (5, 16, 8, 104, 65), (2, 32, 32, 32, 0),
                                                      (3, 128, 64, 128, 70), (2, 104, 40, 64, 0)])
 def test_runs_with_shared_rotated_keys(heads, own, rot, dv, window):
     """Runs that are not adjacent, contexts cut at the first visible key, keys at the window's edges stand out."""
@@ -413,7 +413,7 @@ def test_relu_squared_product(mode, m, n, k):
 
 
 @pytest.mark.parametrize("mode", MODES)
-@pytest.mark.parametrize("experts,groups,keep,top,width,rows", [(16, 4, 3, 3, 40, 9), (12, 6, 2, 2, 64, 30), (8, 8, 3, 2, 24, 7), (10, 1, 1, 4, 32, 700), (64, 8, 2, 6, 136, 700),
+@pytest.mark.parametrize("experts,groups,keep,top,width,rows", [(20, 4, 3, 4, 40, 9), (12, 6, 2, 2, 64, 30), (8, 8, 3, 2, 24, 7), (10, 1, 1, 4, 32, 700), (64, 8, 2, 6, 136, 700),
                                                                 (40, 5, 5, 5, 72, 20), (160, 4, 1, 8, 64, 650), (96, 32, 4, 1, 64, 3)])
 def test_router_in_groups(mode, experts, groups, keep, top, width, rows):
     """Groups whose single best expert is not in the best groups, against the choice token by token; the shared gate."""
