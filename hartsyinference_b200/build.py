@@ -47,7 +47,7 @@ NVCC_FLAGS = [
 # sources that make a smaller library for one kind of model; no source refers to a symbol of another one
 # except the launch switch that gemm_tcgen05.cu defines
 KERNEL_GROUPS = {
-    "decoder": ("gemm_tcgen05", "attention", "delta", "fused_ops", "latent", "linear_f32", "mla", "moe", "residual_norm", "rotary", "sampling", "ssm"),
+    "decoder": ("gemm_tcgen05", "attention", "delta", "delta_general", "fused_ops", "latent", "linear_f32", "mla", "moe", "residual_norm", "rotary", "sampling", "ssm"),
 }
 CXX_FLAGS = ["-O2", "-std=c++17", "-fPIC", "-Wall", "-Wno-unused-function", "-pthread"]
 

@@ -14,8 +14,9 @@
 // flash_attn_v2_tf32.cu). Supported per-call options follow the reference's attention oracle
 // (src/HartsyInference.Core/Backends/AttentionReference.cs): GQA, causal, sliding window,
 // logit soft-cap. The extended form of both kernels (template flag kExt) adds, each optional: a bias
-// by key distance from a per-head table, a per-head sink score that only enters the denominator,
-// values that are the keys themselves (one page plane), a sigmoid gate on the output, first tokens that
+// by key distance from a per-head table or linear in the distance, a per-head sink score that only enters the
+// denominator, values that are the keys themselves (one page plane), a sigmoid gate on the output (per value or per
+// head), an output row pitch, first tokens that
 // stay visible outside the window, key and value sizes up to 128 that are multiples of 8, and a row pitch
 // for q; over contiguous keys also a part of the key that all heads share, with the rotation of its query
 // side. There the probabilities keep 16 bits of
@@ -71,6 +72,9 @@ struct AttnParams {
   const float2* rot_table;
   long long k2_ld;
   int d_own, rot_pairs;
+  const float* slopes;          // [hq] slope * distance is taken off the score, or null
+  int head_gate;                // gate [tokens][gate_ld] holds one column per head
+  long long out_ld;             // output row pitch (head h at h * dv)
   float cap_in, cap_out;        // softcap: cap_out * tanh(score / softcap), exp(2 score / softcap) = 2^(cap_in * q.k)
 };
 constexpr float kLog2e = 1.4426950408889634f;
@@ -87,7 +91,7 @@ __device__ __forceinline__ float exp2_approx(float x) {
 // pointer per row while the tile's distances stay inside it, and only once when they all lie past its end.
 template <int NT, bool kMask>
 __device__ __forceinline__ void ext_scores(float (&s)[NT][4], int key0, const int (&row_limit)[2], const int (&row_start)[2],
-                                           const AttnParams& p, const float* const* row_bias) {
+                                           const AttnParams& p, const float* const* row_bias, const float* row_slope) {
   int mode = -1;
   float far[2] = {0.f, 0.f};
   const float* at[2] = {nullptr, nullptr};
@@ -134,6 +138,13 @@ __device__ __forceinline__ void ext_scores(float (&s)[NT][4], int key0, const in
         const int dist = min(max(row_limit[r] - 1 - (key0 + nt * 8 + (j & 1)), 0), p.dist_len - 1);
         s[nt][j] = fmaf(row_bias[r][dist], kLog2e, s[nt][j]);
       }
+  }
+  if (p.slopes) {
+    const float back[2] = {static_cast<float>(key0 + 1 - row_limit[0]), static_cast<float>(key0 + 1 - row_limit[1])};   // minus the distance
+#pragma unroll
+    for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) s[nt][j] = fmaf(row_slope[j >> 1], back[j >> 1] + (nt * 8 + (j & 1)), s[nt][j]);
   }
   if (kMask) {
 #pragma unroll
@@ -228,13 +239,13 @@ struct WarpState {
 //   qf: Q fragments [D/16][4]; row_limit[r]: first masked key position for the thread's row r
 //   (keys >= limit are masked), row_start[r]: first visible key (sliding window).
 //   Extended form: row_bias[r] is the row's distance-bias table (the distance of a key is counted back
-//   from row_limit[r] - 1).
+//   from row_limit[r] - 1), row_slope[r] its slope times log2(e).
 template <int D, int NG, bool kExt = false, int DV = D>
 __device__ __forceinline__ void warp_tile(WarpState<DV>& st, const uint32_t (&qf)[D / 16][4],
                                           uint32_t k_smem, uint32_t v_smem, int t_begin,
                                           int tok0, const int (&row_limit)[2],
                                           const int (&row_start)[2], const AttnParams& p,
-                                          const float* const* row_bias = nullptr) {
+                                          const float* const* row_bias = nullptr, const float* row_slope = nullptr) {
   const int lane = threadIdx.x & 31;
   const int tq = lane & 3;
   float s[NG * 2][4];
@@ -261,8 +272,8 @@ __device__ __forceinline__ void warp_tile(WarpState<DV>& st, const uint32_t (&qf
   if (kExt) {
     const int first = tok0 + t_begin, last = first + NG * 16 - 1;
     const bool open = last < min(row_limit[0], row_limit[1]) && (first >= max(row_start[0], row_start[1]) || last < p.keep);
-    if (__all_sync(0xffffffffu, open)) ext_scores<NG * 2, false>(s, first + tq * 2, row_limit, row_start, p, row_bias);
-    else ext_scores<NG * 2, true>(s, first + tq * 2, row_limit, row_start, p, row_bias);
+    if (__all_sync(0xffffffffu, open)) ext_scores<NG * 2, false>(s, first + tq * 2, row_limit, row_start, p, row_bias, row_slope);
+    else ext_scores<NG * 2, true>(s, first + tq * 2, row_limit, row_start, p, row_bias, row_slope);
   }
 #pragma unroll
   for (int nt = 0; nt < NG * 2; ++nt) {
@@ -350,7 +361,7 @@ __device__ __forceinline__ void warp_tile(WarpState<DV>& st, const uint32_t (&qf
 }
 
 __device__ __forceinline__ float gate_of(const AttnParams& p, long long token, int head, int c) {
-  return p.gate ? 1.f / (1.f + __expf(-__bfloat162float(p.gate[token * p.gate_ld + head * p.dv + c]))) : 1.f;
+  return p.gate ? 1.f / (1.f + __expf(-__bfloat162float(p.gate[token * p.gate_ld + (p.head_gate ? head : head * p.dv + c)]))) : 1.f;
 }
 
 // ------------------------------------------------------------------------------------------
@@ -405,10 +416,12 @@ attn_decode_kernel(const AttnParams p) {
   const int lim[2] = {kv_len, kv_len};
   const int start[2] = {start_key, start_key};
   const float* row_bias[2] = {nullptr, nullptr};
+  float row_slope[2] = {0.f, 0.f};
   if (kExt) {
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
       const int head = kvh * G + min(g + 8 * r, G - 1);
+      if (p.slopes) row_slope[r] = p.slopes[head] * kLog2e;
       if (p.dist_bias) row_bias[r] = p.dist_bias + static_cast<long long>(head) * p.dist_len;
       if (p.sinks && split == 0 && warp == 0) {       // the sink enters the running sums once
         st.m[r] = p.sinks[head] * kLog2e;
@@ -452,7 +465,7 @@ attn_decode_kernel(const AttnParams p) {
     __syncthreads();
     const uint32_t kb = smem_base + slot * stage_bytes;
     warp_tile<D, 1, kExt>(st, qf, kb, kExt && p.shared_kv ? kb : kb + kTileBytes, warp * 16, tile_of(step) * kTileTokens, lim, start,
-                          p, row_bias);
+                          p, row_bias, row_slope);
     __syncthreads();
     slot = (slot + 1) % kStages;
   }
@@ -493,8 +506,7 @@ attn_decode_kernel(const AttnParams p) {
     const int head = kvh * G + r;
     if (kExt && p.splits == 1) {
       if (c < p.dv)
-        p.out[(static_cast<long long>(seq) * p.hq + head) * p.dv + c] =
-            __float2bfloat16((ll > 0.f ? acc / ll : 0.f) * gate_of(p, seq, head, c));
+        p.out[seq * p.out_ld + head * p.dv + c] = __float2bfloat16((ll > 0.f ? acc / ll : 0.f) * gate_of(p, seq, head, c));
     } else if (p.splits == 1) {
       p.out[(static_cast<long long>(seq) * p.hq + head) * D + c] =
           __float2bfloat16(ll > 0.f ? acc / ll : 0.f);
@@ -527,8 +539,7 @@ __global__ void attn_combine_kernel(const AttnParams p) {
     }
     if (kExt) {
       if (c < p.dv)
-        p.out[(static_cast<long long>(seq) * p.hq + head) * p.dv + c] =
-            __float2bfloat16((ll > 0.f ? acc / ll : 0.f) * gate_of(p, seq, head, c));
+        p.out[seq * p.out_ld + head * p.dv + c] = __float2bfloat16((ll > 0.f ? acc / ll : 0.f) * gate_of(p, seq, head, c));
       continue;
     }
     const __nv_bfloat16 o = __float2bfloat16(ll > 0.f ? acc / ll : 0.f);
@@ -639,7 +650,9 @@ attn_prefill_kernel(const AttnParams p) {
     start[r] = p.window > 0 ? max(0, pos + 1 - p.window) : 0;
   }
   const float* row_bias[2] = {nullptr, nullptr};
+  float row_slope[2] = {0.f, 0.f};
   if (kExt) {
+    if (p.slopes) row_slope[0] = row_slope[1] = p.slopes[head] * kLog2e;
     if (p.dist_bias) {
       row_bias[0] = row_bias[1] = p.dist_bias + static_cast<long long>(head) * p.dist_len;
       if (p.dist_len <= kDistSmem) {
@@ -709,7 +722,7 @@ attn_prefill_kernel(const AttnParams p) {
     // a warp whose rows all lie before this tile (causal) still runs: masked scores cost nothing
     // in correctness and keep the barrier pattern uniform
     warp_tile<D, 4, kExt, DV>(st, qf, kb, kExt && p.shared_kv ? kb : kb + kTileBytes, 0, tile_of(step) * kTileTokens, lim, start, p,
-                          row_bias);
+                          row_bias, row_slope);
     __syncthreads();
     slot ^= 1;
   }
@@ -722,15 +735,19 @@ attn_prefill_kernel(const AttnParams p) {
   for (int r = 0; r < 2; ++r) {
     const int row = row0 + 8 * r;
     if (row < q_len) {
-      const float inv = st.l[r] > 0.f ? 1.f / st.l[r] : 0.f;
+      float inv = st.l[r] > 0.f ? 1.f / st.l[r] : 0.f;
+      if (kExt && p.head_gate) inv *= gate_of(p, q_off + row, head, 0);
 #pragma unroll
       for (int i = 0; i < DV / 8; ++i) {
         const int c = i * 8 + tq * 2;
         if (kExt) {
-          if (c < p.dv)
-            *reinterpret_cast<uint32_t*>(p.out + (static_cast<long long>(q_off + row) * p.hq + head) * p.dv + c) =
-                pack_bf16x2(st.o[i][2 * r] * inv * gate_of(p, q_off + row, head, c),
-                            st.o[i][2 * r + 1] * inv * gate_of(p, q_off + row, head, c + 1));
+          float a = st.o[i][2 * r] * inv, b = st.o[i][2 * r + 1] * inv;
+          if (c >= p.dv) continue;
+          if (!p.head_gate) {
+            a *= gate_of(p, q_off + row, head, c);
+            b *= gate_of(p, q_off + row, head, c + 1);
+          }
+          *reinterpret_cast<uint32_t*>(p.out + (q_off + row) * p.out_ld + head * p.dv + c) = pack_bf16x2(a, b);
           continue;
         }
         *reinterpret_cast<uint32_t*>(ob + row * rs + c) =
@@ -752,6 +769,9 @@ struct AttnRowsParams {
   int tokens, seqs, hq, hkv, d, page, max_pages, window, dist_len;
   float scale, softcap;
   int keep, dv, v_row;         // kept first tokens; value size, and values per row of the value pages
+  const float* slopes;         // as in AttnParams
+  int head_gate;
+  long long out_ld;
 };
 constexpr int kRowsMaxD = 1024, kRowsMaxV = 512;   // query-key and value size
 
@@ -801,6 +821,7 @@ __global__ void __launch_bounds__(128) attn_rows_kernel(const AttnRowsParams p) 
       s = a * p.scale;
       if (p.softcap > 0.f) s = p.softcap * tanhf(s / p.softcap);
       if (p.dist_bias) s += p.dist_bias[static_cast<long long>(head) * p.dist_len + min(pos - j, p.dist_len - 1)];
+      if (p.slopes) s -= p.slopes[head] * static_cast<float>(pos - j);
     }
     const float mn = fmaxf(m, warp_max(s));
     const float f = m == -INFINITY ? 0.f : expf(m - mn);
@@ -818,14 +839,14 @@ __global__ void __launch_bounds__(128) attn_rows_kernel(const AttnRowsParams p) 
         if (lane + i * 32 < p.dv) o[i] += w * as_f32(vr[lane + i * 32]);
     }
   }
-  T* out = static_cast<T*>(p.out) + (static_cast<long long>(t) * p.hq + head) * p.dv;
-  const T* gate = p.gate ? static_cast<const T*>(p.gate) + t * p.gate_ld + head * p.dv : nullptr;
+  T* out = static_cast<T*>(p.out) + t * p.out_ld + head * p.dv;
+  const T* gate = p.gate ? static_cast<const T*>(p.gate) + t * p.gate_ld + (p.head_gate ? head : head * p.dv) : nullptr;
 #pragma unroll
   for (int i = 0; i < kRowsMaxV / 32; ++i) {
     const int c = lane + i * 32;
     if (c < p.dv) {
       float y = l > 0.f ? o[i] / l : 0.f;
-      if (gate) y *= 1.f / (1.f + expf(-as_f32(gate[c])));
+      if (gate) y *= 1.f / (1.f + expf(-as_f32(gate[p.head_gate ? 0 : c])));
       out[c] = static_cast<T>(y);
     }
   }
@@ -991,25 +1012,26 @@ B200_API int b200_attn_prefill(const void* q, const void* k, const void* v, void
 }
 
 // Extended attention over pages (see the header comment). cu_q null: one query token per sequence.
-// q [tokens][q_ld] (head h at h * d), out [tokens][hq * dv]. v_cache null: the values are the keys (with exact, their
+// q [tokens][q_ld] (head h at h * d), out [tokens][out_ld] (head h at h * dv). v_cache null: the values are the keys (with exact, their
 // first dv columns). window > 0: the last `window` keys and the first keep_first of the sequence.
 // exact != 0: plain fp32 kernel, tensors are fp32 when f32 is set and bf16 otherwise; exact == 0: the
 // tensor-core kernels (bf16, d, dv <= 128, at most 16 query heads per key head at decode; returns -6 for
 // what they do not take). splits / workspace: decode only, as in b200_attn_decode (with the head size
-// rounded up to 64 or 128).
+// rounded up to 64 or 128). slopes: a bias linear in the distance; head_gate: one gate column per head.
 B200_API int b200_attn_biased(const void* q, const void* k_cache, const void* v_cache, void* out, const int* block_table,
                               const int* kv_lens, const int* cu_q, int tokens, int seqs, int max_q_len, int hq, int hkv, int d,
                               int dv, int page, int max_pages, int splits, void* workspace, float scale, float softcap, int window, int keep_first,
                               const float* dist_bias, int dist_len, const float* sinks, const void* gate, long long gate_ld,
-                              long long q_ld, int exact, int f32, cudaStream_t stream) {
+                              long long q_ld, int exact, int f32, const float* slopes, int head_gate, long long out_ld,
+                              cudaStream_t stream) {
   if (tokens <= 0 || seqs <= 0) return 0;
-  if (d % 8 || d < 8 || d > kRowsMaxD || dv % 8 || dv < 8 || dv > kRowsMaxV || (!v_cache && dv > d) || keep_first < 0 || hq % hkv || q_ld % 8 || (gate && gate_ld % 8) || (dist_bias && dist_len < 1)) return -2;
+  if (d % 8 || d < 8 || d > kRowsMaxD || dv % 8 || dv < 8 || dv > kRowsMaxV || (!v_cache && dv > d) || keep_first < 0 || hq % hkv || q_ld % 8 || (gate && gate_ld % 8) || (dist_bias && dist_len < 1) || out_ld < static_cast<long long>(hq) * dv || out_ld % 8) return -2;
   if (f32 && !exact) return -6;
   if (window <= 0) keep_first = 0;
   if (exact) {
     AttnRowsParams p{q, k_cache, v_cache ? v_cache : k_cache, gate, out, block_table, kv_lens, cu_q, dist_bias, sinks,
                      q_ld, gate_ld, tokens, seqs, hq, hkv, d, page, max_pages, window, dist_len, scale, softcap,
-                     keep_first, dv, v_cache ? dv : d};
+                     keep_first, dv, v_cache ? dv : d, slopes, head_gate, out_ld};
     const dim3 grid((tokens + 3) / 4, hq);
     const cudaError_t e = f32 ? launch_pdl(attn_rows_kernel<float>, grid, dim3(128), 0, stream, p)
                               : launch_pdl(attn_rows_kernel<__nv_bfloat16>, grid, dim3(128), 0, stream, p);
@@ -1037,7 +1059,7 @@ B200_API int b200_attn_biased(const void* q, const void* k_cache, const void* v_
     p.cap_in = 2.f * kLog2e * scale / softcap;
     p.cap_out = softcap * kLog2e;
   }
-  p.dist_bias = dist_bias; p.dist_len = dist_len; p.sinks = sinks;
+  p.dist_bias = dist_bias; p.dist_len = dist_len; p.sinks = sinks; p.slopes = slopes; p.head_gate = head_gate; p.out_ld = out_ld;
   p.gate = static_cast<const __nv_bfloat16*>(gate);
   p.gate_ld = gate_ld; p.q_ld = q_ld; p.d = p.d_own = d; p.dv = dv; p.keep = keep_first;
   p.splits = cu_q || splits < 1 ? 1 : splits;
@@ -1088,16 +1110,18 @@ B200_API int b200_attn_biased(const void* q, const void* k_cache, const void* v_
 // Causal attention of the runs q_start[s] .. + q_lens[s] of q over contiguous keys and values of their whole
 // contexts (rows kv_start[s] .. + kv_lens[s] of k and v; the last key belongs to the run's last query; window > 0: the
 // last `window` keys of every query). q, out and gate are indexed by token: q [tokens][q_ld] (head h at h * d), out
-// [tokens][hq * dv]. d <= 192, dv <= 128, multiples of 8. The keys' columns from d_own on are rows of k2 for every head
+// [tokens][out_ld] (head h at h * dv); head_gate: one gate column per head. d <= 192, dv <= 128, multiples of 8. The keys' columns from d_own on are rows of k2 for every head
 // (d_own = d: none); with rot_table [tokens][rot_pairs] (cos, sin) those columns of q are turned.
 B200_API int b200_attn_runs(const void* q, const void* k, const void* v, void* out, const void* gate, const int* q_start,
                             const int* q_lens, const int* kv_start, const int* kv_lens, int seqs, int max_q_len, int hq, int hkv,
                             int d, int dv, long long q_ld, long long k_ld, long long v_ld, long long gate_ld, float scale, int window,
-                            const void* k2, int d_own, long long k2_ld, const void* rot_table, int rot_pairs, cudaStream_t stream) {
+                            const void* k2, int d_own, long long k2_ld, const void* rot_table, int rot_pairs, const float* sinks, int head_gate,
+                            long long out_ld, cudaStream_t stream) {
   if (seqs <= 0 || max_q_len <= 0) return 0;
   if (d % 8 || dv % 8 || d < 8 || dv < 8 || d > 192 || dv > 128 || hq % hkv || q_ld % 8 || k_ld % 8 || v_ld % 8 || gate_ld % 8 ||
       seqs > 65535)
     return -2;
+  if (out_ld % 8 || out_ld < static_cast<long long>(hq) * dv) return -2;
   if (d_own % 8 || d_own > d || k2_ld % 8 || (d_own < d && !k2) || (rot_table && 2 * rot_pairs > d - d_own)) return -2;
   AttnParams p{};
   p.q = static_cast<const __nv_bfloat16*>(q);
@@ -1114,6 +1138,7 @@ B200_API int b200_attn_runs(const void* q, const void* k, const void* v, void* o
   p.d = d; p.dv = dv; p.q_ld = q_ld; p.k_ld = k_ld; p.v_ld = v_ld; p.gate_ld = gate_ld;
   p.k2 = static_cast<const __nv_bfloat16*>(k2); p.d_own = d_own; p.k2_ld = k2_ld;
   p.rot_table = static_cast<const float2*>(rot_table); p.rot_pairs = rot_pairs;
+  p.sinks = sinks; p.head_gate = head_gate; p.out_ld = out_ld;
   const dim3 grid((max_q_len + 63) / 64, hq, seqs);
   auto go = [&](auto kernel, int dd, PerDeviceOnce& once) {
     const int smem = 2 * kTileTokens * (dd + (dd > 128 ? 128 : dd)) * 2;

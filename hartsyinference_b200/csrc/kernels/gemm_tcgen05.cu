@@ -191,7 +191,8 @@ struct GemmParams {
   const __nv_bfloat16* bias;      // per output feature (column of C), may be null
   const __nv_bfloat16* gate;      // per output feature multiplicative gate, may be null
   const __nv_bfloat16* residual;  // same layout as C, may be null
-  int act;                        // 0 none, 1 gelu-tanh, 2 silu, 3 relu squared
+  int act;                        // 0 none, 1 gelu-tanh, 2 silu, 3 relu squared, 4 tanh
+  int act_col;                    // first output feature that the activation applies to
   // fp8 block scales, K-contiguous: scale(row, kb) = s[(row / gran) * ld + kb], ld = K / 128.
   // A thread walks one row's scales along K, so consecutive k-blocks hit the same cache line.
   const float* scale_a;
@@ -304,6 +305,7 @@ __device__ __forceinline__ float apply_epilogue(const GemmParams& p, float v, lo
   if (p.act == 1) v = gelu_tanh(v);
   else if (p.act == 2) v = silu(v);
   else if (p.act == 3) v = relu2(v);
+  else if (p.act == 4 && col >= p.act_col) v = tanhf(v);
   if (p.gate) v *= __bfloat162float(p.gate[col]);
   if (p.residual) v += __bfloat162float(p.residual[row * p.ldc + col]);
   return v;
@@ -1516,7 +1518,9 @@ int gemm_impl(const void* x, const void* w, void* out, int m, int n, int k, long
   p.bias = static_cast<const __nv_bfloat16*>(bias);
   p.gate = static_cast<const __nv_bfloat16*>(gate);
   p.residual = static_cast<const __nv_bfloat16*>(residual);
-  p.act = act;
+  p.act = act & 255;
+  p.act_col = act >> 8;
+  if (p.act_col > 0 && p.act != 4) return -6;
   p.status = static_cast<DeviceStatus*>(status);
   p.swap_out = swap ? 1 : 0;
   if (ar != nullptr) {
@@ -1758,6 +1762,8 @@ B200_API long long b200_gemm_workspace_bytes() {
 //   x_scale: [m][k/128] fp32 (per token, per 128-wide K group); w_scale: [ceil(n/128)][k/128] fp32
 //   splits: 0 = automatic (split only the tiles of a partial last wave), 1 = never, > 1 = split
 //           every tile that many ways
+//   act: 0 none, 1 gelu-tanh, 2 silu, 3 relu squared, 4 tanh; tanh can be limited to the output features from
+//           act >> 8 on
 //   workspace: zero-initialised scratch (see b200_gemm_workspace_bytes), may be null (no splitting)
 // Returns 0 on success, negative on a launch-time error.
 B200_API int b200_gemm(const void* x, const void* w, void* out, int m, int n, int k, long long ldx,

@@ -115,7 +115,7 @@ struct HeadLinearParams {
   const void* x;             // row r, head h: x + r * ldx + h * x_stride, k values
   const __nv_bfloat16* w;    // [heads * n][k]
   void* out;                 // row r, head h: out + r * ldo + h * o_stride, n values
-  const void* gate;          // row r, head h: gate + r * ldg + h * o_stride, or null
+  const void* gate;          // row r, head h: gate + r * ldg + h * o_stride (head_gate: one value at h), or null
   const int* in_rows;        // row of x for product row i, or null
   const int* out_rows;       // row of out and gate for product row i, or null
   long long ldx, ldo, ldg;
@@ -124,6 +124,7 @@ struct HeadLinearParams {
   // (2i, 2i + 1), zero from rot on, and stored behind the head's n
   const float2* table;
   int rot, tail;
+  int head_gate;
 };
 
 // The tail of the rows m0 .. m0 + count of one head.
@@ -225,12 +226,15 @@ __global__ void __launch_bounds__(128) head_linear_kernel(const HeadLinearParams
       if (i >= p.rows) continue;
       const long long row = p.out_rows ? p.out_rows[i] : i;
       __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out) + row * p.ldo + head * p.o_stride;
-      const __nv_bfloat16* gate = p.gate ? static_cast<const __nv_bfloat16*>(p.gate) + row * p.ldg + head * p.o_stride : nullptr;
+      const __nv_bfloat16* gate = nullptr;
+      float scale = 1.f;
+      if (p.gate && p.head_gate) scale = sigmoid_f32(ld1(static_cast<const __nv_bfloat16*>(p.gate) + row * p.ldg + head));
+      else if (p.gate) gate = static_cast<const __nv_bfloat16*>(p.gate) + row * p.ldg + head * p.o_stride;
 #pragma unroll
       for (int g = 0; g < kNt; ++g) {
         const int j = n0 + wn * (kN / 2) + g * 8 + (lane & 3) * 2;
         if (j >= p.n) continue;
-        float u = acc[m][g][2 * r], v = acc[m][g][2 * r + 1];
+        float u = acc[m][g][2 * r] * scale, v = acc[m][g][2 * r + 1] * scale;
         if (gate) {
           const float2 s = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(gate + j));
           u *= sigmoid_f32(s.x);
@@ -269,7 +273,7 @@ __global__ void __launch_bounds__(256) head_linear_f32_kernel(const HeadLinearPa
     if (i >= p.rows || j >= p.n) continue;
     const long long row = p.out_rows ? p.out_rows[i] : i;
     float v = acc[q];
-    if (p.gate) v *= sigmoid_f32(static_cast<const float*>(p.gate)[row * p.ldg + head * p.o_stride + j]);
+    if (p.gate) v *= sigmoid_f32(static_cast<const float*>(p.gate)[row * p.ldg + (p.head_gate ? head : head * p.o_stride + j)]);
     static_cast<float*>(p.out)[row * p.ldo + head * p.o_stride + j] = v;
   }
 }
@@ -309,15 +313,15 @@ B200_API int b200_latent_gather(const void* cache, void* out, const int* block_t
   return e == cudaSuccess ? 0 : -static_cast<int>(e) - 300;
 }
 
-// n, k, strides and row pitches multiples of 8; tail > 0: see HeadLinearParams
+// n, k, strides and row pitches multiples of 8; head_gate: one gate column per head; tail > 0: see HeadLinearParams
 B200_API int b200_head_linear(const void* x, const void* w, void* out, const void* gate, const int* in_rows, const int* out_rows,
                               int rows, int heads, int n, int k, long long ldx, int x_stride, long long ldo, int o_stride,
-                              long long ldg, const void* table, int rot, int tail, int f32, cudaStream_t stream) {
+                              long long ldg, const void* table, int rot, int tail, int head_gate, int f32, cudaStream_t stream) {
   if (rows <= 0 || heads <= 0) return 0;
   if (tail && (tail % 8 || rot % 2 || rot > tail || !table || x_stride < k + tail || o_stride < n + tail)) return -2;
   if (n % 8 || k % 8 || ldx % 8 || x_stride % 8 || ldo % 8 || o_stride % 8 || ldg % 8 || heads > 65535) return -2;
   HeadLinearParams p{x, static_cast<const __nv_bfloat16*>(w), out, gate, in_rows, out_rows, ldx, ldo, ldg, rows, n, k, x_stride, o_stride,
-                     static_cast<const float2*>(table), rot, tail};
+                     static_cast<const float2*>(table), rot, tail, head_gate};
   if (f32) {
     head_linear_f32_kernel<<<dim3((rows + 31) / 32, (n + 31) / 32, heads), 256, 0, stream>>>(p);
     return cudaGetLastError() == cudaSuccess ? 0 : -300;

@@ -67,7 +67,7 @@ linear_f32_kernel(const T* __restrict__ x, const __nv_bfloat16* __restrict__ w, 
       const int c = n0 + tx * 4 + j;
       if (c < n) {
         const float v = acc[i][j] + (bias ? __bfloat162float(bias[c]) : 0.f);
-        out[r * ldo + c] = act == 3 ? relu2(v) : v;
+        out[r * ldo + c] = act == 3 ? relu2(v) : (act & 255) == 4 && c >= act >> 8 ? tanhf(v) : v;
       }
     }
   }
@@ -364,10 +364,10 @@ pair_linear_f32_kernel(const float* __restrict__ x, const __nv_bfloat16* __restr
 
 using namespace b200;
 
-// act: 0 none, 3 relu squared
+// act: 0 none, 3 relu squared, 4 tanh of the output features from act >> 8 on
 B200_API int b200_linear_f32(const void* x, int x_f32, const void* w, const void* bias, void* out, int m, int n, int k,
                              long long ldx, long long ldw, long long ldo, int act, cudaStream_t stream) {
-  if (act != 0 && act != 3) return -2;
+  if (act != 0 && act != 3 && (act & 255) != 4) return -2;
   if (m <= 0 || n <= 0) return 0;
   const dim3 grid((n + kLT - 1) / kLT, (m + kLT - 1) / kLT);
   if (grid.y > 65535) return -2;

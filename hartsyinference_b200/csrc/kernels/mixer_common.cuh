@@ -71,6 +71,11 @@ __device__ __forceinline__ void st4<__nv_bfloat16>(__nv_bfloat16* p, const float
 }
 __device__ __forceinline__ float ld1(const float* p) { return *p; }
 __device__ __forceinline__ float ld1(const __nv_bfloat16* p) { return __bfloat162float(*p); }
+// a value as the activation type holds it
+template <typename T>
+__device__ __forceinline__ float ld1_of(float v) { return v; }
+template <>
+__device__ __forceinline__ float ld1_of<__nv_bfloat16>(float v) { return __bfloat162float(__float2bfloat16(v)); }
 __device__ __forceinline__ float sigmoid_f32(float x) { return 1.f / (1.f + expf(-x)); }
 
 // exp(-y). The decays of a sequence multiply up over thousands of tokens, so near 1 the value is formed from

@@ -121,6 +121,7 @@ struct MlaAttnParams {
   int row, lat;                 // values per cached row and per output row (multiples of 8)
   float scale_log2;
   int window;                   // > 0: only the last `window` tokens of each row's context
+  const float* sinks;           // [heads] scores that only enter the denominators, or null
 };
 
 // kSets groups of four warps share one CTA and one staged KV tile; each group owns 16 heads of the
@@ -208,6 +209,14 @@ __global__ void __launch_bounds__(kMlaThreads * kSets) mla_attn_kernel(const Mla
     for (int j = 0; j < 4; ++j) o[i][j] = 0.f;
   float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
   const int r0 = lane >> 2, tq = lane & 3;
+  if (p.sinks != nullptr && split == 0) {          // once per row: the first split starts with it
+#pragma unroll
+    for (int r = 0; r < 2; ++r)
+      if (r0 + 8 * r < heads_here) {
+        m_run[r] = p.sinks[hg * 16 + r0 + 8 * r] * 1.4426950408889634f;
+        l_run[r] = 1.f;
+      }
+  }
 
   for (int t = t0; t < t1; ++t) {
     const int buf = (t - t0) & 1;
@@ -480,10 +489,10 @@ B200_API int b200_mla_attn(const void* q, const void* cache, void* out, const in
 
 // Latent attention of any size: cached rows of `row` values, the first `lat` of which are the values (multiples of 8,
 // lat <= 512, row <= 576), q [rows][heads][row], out
-// [rows][heads][lat]. window > 0: the last `window` tokens. The workspace is that of b200_mla_workspace_bytes.
+// [rows][heads][lat]. window > 0: the last `window` tokens. sinks: [heads] fp32 or null. The workspace is that of b200_mla_workspace_bytes.
 B200_API int b200_latent_attn(const void* q, const void* cache, void* out, const int* block_table, const int* kv_lens,
                               const int* row_seq, int rows, int heads, int row, int lat, int page, int table_stride, int splits,
-                              void* workspace, float scale, int window, cudaStream_t stream) {
+                              void* workspace, float scale, int window, const float* sinks, cudaStream_t stream) {
   if (rows <= 0) return 0;
   if (lat % 8 || lat < 8 || lat > kLat || row % 8 || row < lat) return -2;
   MlaAttnParams p{};
@@ -492,6 +501,7 @@ B200_API int b200_latent_attn(const void* q, const void* cache, void* out, const
   p.row = row;
   p.lat = lat;
   p.window = window;
+  p.sinks = sinks;
   if (row <= 64) return launch_mla<64, 0, true>(p, workspace, stream);
   if (row <= 128) return lat <= 64 ? launch_mla<64, 64, true>(p, workspace, stream) : launch_mla<128, 0, true>(p, workspace, stream);
   if (row <= 192 && lat <= 128) return launch_mla<128, 64, true>(p, workspace, stream);

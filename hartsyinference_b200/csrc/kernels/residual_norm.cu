@@ -11,8 +11,10 @@
 // combine step of a mixture of experts needs no launch and no intermediate rounding of its own; a shared expert's
 // rows join the sum with one weight per token.
 // LayerNorm (weight, no bias) or RMSNorm; weights as stored or stored around zero (1 + w); statistics in two
-// passes over the registers, in fp32. The norm on x can also be tanh(alpha x) w + b, which has no statistics.
-// side_gate is the elementwise step of a second embedding that enters every layer. The embedding can be normed on its way into the stream, and poly_norm is
+// passes over the registers, in fp32. An RMS norm on x can also be taken over equal parts of the row, each on its own,
+// and at one token per sequence h can go through the convolutions over time that the next sublayers read
+// (h + conv_i(h), see ssm.cu for prompts) in the same launch. The norm on x can also be tanh(alpha x) w + b, which has no statistics.
+// cap_logits scales and caps the output logits; side_gate is the elementwise step of a second embedding that enters every layer. The embedding can be normed on its way into the stream, and poly_norm is
 // the activation that mixes a row's normed powers.
 #include "mixer_common.cuh"
 
@@ -37,6 +39,12 @@ struct ResidualNormParams {
   const void* extra;         // routed source: [rows][ld_extra] added with weight extra_w[row] (null: none)
   const float* extra_w;
   int ld_extra;
+  int groups;                // > 1: w_n's norm is an RMS norm of this many equal parts
+  const float* conv_w;       // not null: [conv_n][taps][ldh]; h is [conv_n][rows][ldh]
+  int conv_n, taps;
+  void* conv_state;          // [slots][taps - 1][ldh] earlier h, oldest first; moved on by one
+  const int* positions;      // [rows], 0: the sequence starts
+  const int* slots;          // [rows]
 };
 
 // v <- norm(v) * w over the row's first `dim` values (values past them are zero on entry and exit)
@@ -76,6 +84,84 @@ __device__ __forceinline__ void norm_row(float (&v)[kIters][8], const __nv_bfloa
 #pragma unroll
       for (int j = 0; j < 8; ++j) v[i][j] = c + j < dim ? (v[i][j] - mean) * inv * (one + __bfloat162float(w[c + j])) : 0.f;
     }
+  }
+}
+
+// v <- norm of each of `groups` equal parts of the row, times w. xr: the row as stored (this block's stores of it are
+// done); sm: dim / 8 + groups floats of shared memory
+template <int kIters>
+__device__ __forceinline__ void group_norm_row(float (&v)[kIters][8], const float* xr, const __nv_bfloat16* w, int dim, int groups,
+                                               int plus_one, float eps, float* sm) {
+  const float one = plus_one ? 1.f : 0.f;
+  const int n = dim / groups, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+  const bool whole = (n & 7) == 0;                 // parts consist of whole vectors
+  float* inv = sm + (dim + 7) / 8;
+  if (whole) {
+#pragma unroll
+    for (int i = 0; i < kIters; ++i) {
+      const int vec = threadIdx.x + i * blockDim.x;
+      float q = 0.f;
+#pragma unroll
+      for (int j = 0; j < 8; ++j) q = fmaf(v[i][j], v[i][j], q);
+      if (vec * 8 < dim) sm[vec] = q;
+    }
+  }
+  __syncthreads();
+  for (int g = warp; g < groups; g += warps) {
+    float q = 0.f;
+    if (whole) for (int e = lane; e < n / 8; e += 32) q += sm[g * (n / 8) + e];
+    else for (int e = lane; e < n; e += 32) q = fmaf(xr[g * n + e], xr[g * n + e], q);
+    q = warp_sum(q);
+    if (lane == 0) inv[g] = 1.f / sqrtf(q / n + eps);
+  }
+  __syncthreads();
+#pragma unroll
+  for (int i = 0; i < kIters; ++i) {
+    const int c = (threadIdx.x + i * blockDim.x) * 8;
+    if (c + 8 <= dim && whole) {
+      float wv[8];
+      load8(w + c, wv);
+      const float f = inv[c / n];
+#pragma unroll
+      for (int j = 0; j < 8; ++j) v[i][j] = v[i][j] * f * (one + wv[j]);
+    } else {
+#pragma unroll
+      for (int j = 0; j < 8; ++j) v[i][j] = c + j < dim ? v[i][j] * inv[(c + j) / n] * (one + __bfloat162float(w[c + j])) : 0.f;
+    }
+  }
+}
+
+// One token per sequence: h[i][row] = v + sum over the taps, the state moves on by one token.
+template <typename T, int kIters>
+__device__ __forceinline__ void conv_row(const ResidualNormParams& p, long long row, const float (&v)[kIters][8]) {
+  const int slot = p.slots[row], tail = p.taps - 1;
+  const bool carried = slot >= 0 && p.positions[row] > 0;
+  T* state = static_cast<T*>(p.conv_state) + static_cast<long long>(slot < 0 ? 0 : slot) * tail * p.ldh;
+#pragma unroll
+  for (int i = 0; i < kIters; ++i) {
+    const int c = (threadIdx.x + i * blockDim.x) * 8;
+    if (c >= p.ldh) continue;
+    float now[8], y[2][8];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) now[j] = y[0][j] = y[1][j] = ld1_of<T>(v[i][j]);
+    for (int k = 0; k < p.taps; ++k) {
+      float in[8];
+#pragma unroll
+      for (int j = 0; j < 8; ++j) in[j] = k == tail ? now[j] : 0.f;
+      if (k < tail && carried) load8(state + static_cast<long long>(k) * p.ldh + c, in);
+      if (k > 0 && slot >= 0) store8(state + static_cast<long long>(k - 1) * p.ldh + c, in);
+#pragma unroll
+      for (int o = 0; o < 2; ++o)
+        if (o < p.conv_n) {
+          float w[8];
+          load8(p.conv_w + (static_cast<long long>(o) * p.taps + k) * p.ldh + c, w);
+#pragma unroll
+          for (int j = 0; j < 8; ++j) y[o][j] = fmaf(in[j], w[j], y[o][j]);
+        }
+    }
+#pragma unroll
+    for (int o = 0; o < 2; ++o)
+      if (o < p.conv_n) store8(static_cast<T*>(p.h) + (static_cast<long long>(o) * gridDim.x + row) * p.ldh + c, y[o]);
   }
 }
 
@@ -186,7 +272,14 @@ __global__ void __launch_bounds__(1024) residual_norm_kernel(const ResidualNormP
   }
   if (p.w_n == nullptr && !p.plain) return;
   if (p.b_n != nullptr) tanh_row<kIters>(xv, p.w_n, p.b_n, p.alpha, p.dim);
-  else if (p.w_n != nullptr) norm_row<kIters>(xv, p.w_n, p.dim, p.layernorm, p.plus_one, p.eps, red);
+  else if (p.w_n != nullptr && p.groups > 1) {
+    extern __shared__ float parts[];
+    group_norm_row<kIters>(xv, xr, p.w_n, p.dim, p.groups, p.plus_one, p.eps, parts);
+  } else if (p.w_n != nullptr) norm_row<kIters>(xv, p.w_n, p.dim, p.layernorm, p.plus_one, p.eps, red);
+  if (p.conv_w != nullptr) {
+    conv_row<T, kIters>(p, row, xv);
+    return;
+  }
   T* hr = static_cast<T*>(p.h) + row * p.ldh;
 #pragma unroll
   for (int i = 0; i < kIters; ++i) {
@@ -274,6 +367,25 @@ __global__ void __launch_bounds__(256) side_gate_kernel(const T* __restrict__ u,
   store8(y + t * vecs * 8 + c, a);
 }
 
+// out = cap * tanh(scale y / cap), or scale y without a cap: logits in 32 bits. Eight values per thread.
+template <typename T>
+__global__ void __launch_bounds__(256) cap_logits_kernel(const T* __restrict__ y, float* __restrict__ out, long long n, float scale, float cap) {
+  pdl_wait();
+  pdl_trigger();
+  const long long i = (static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x) * 8;
+  if (i >= n) return;
+  const float inner = cap > 0.f ? scale / cap : scale;
+  float v[8];
+  if (i + 8 <= n) {
+    load8(y + i, v);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) v[j] = cap > 0.f ? cap * tanhf(v[j] * inner) : v[j] * inner;
+    store8(out + i, v);
+  } else {
+    for (long long j = i; j < n; ++j) out[j] = cap > 0.f ? cap * tanhf(ld1(y + j) * inner) : ld1(y + j) * inner;
+  }
+}
+
 // y = a z / rms(z) + b z^2 / rms(z^2) + c z^3 / rms(z^3) + e over a row of `dim` values (powers element by
 // element); columns past dim are zeroed. The row stays in registers between the two passes.
 template <typename T, int kIters>
@@ -347,10 +459,11 @@ template <typename T>
 int launch_residual_norm(const ResidualNormParams& p, int rows, cudaStream_t stream) {
   int iters, threads;
   if (!row_shape(p.dim, rows, iters, threads)) return -2;
+  const int smem = p.groups > 1 ? ((p.dim + 7) / 8 + p.groups) * 4 : 0;
   cudaError_t e;
   switch (iters) {
-    case 1: e = launch_pdl(residual_norm_kernel<T, 1>, dim3(rows), dim3(threads), 0, stream, p); break;
-    default: e = launch_pdl(residual_norm_kernel<T, 2>, dim3(rows), dim3(threads), 0, stream, p); break;
+    case 1: e = launch_pdl(residual_norm_kernel<T, 1>, dim3(rows), dim3(threads), smem, stream, p); break;
+    default: e = launch_pdl(residual_norm_kernel<T, 2>, dim3(rows), dim3(threads), smem, stream, p); break;
   }
   return e == cudaSuccess ? 0 : -static_cast<int>(e) - 300;
 }
@@ -360,22 +473,26 @@ int launch_residual_norm(const ResidualNormParams& p, int rows, cudaStream_t str
 using namespace b200;
 
 // See the header comment. f32 != 0: y / src / extra / h are fp32 instead of bf16. ldy etc. in elements,
-// multiples of 8. Rows of at most 16384 values.
+// multiples of 8. Rows of at most 16384 values, norms of at most 2048 parts. conv_w (may be null): one or two sets of
+// taps for h, one token per sequence.
 B200_API int b200_residual_norm(void* x, const void* y, void* h, const void* w_b, const void* w_n, const int* slot_of,
                                 const int* ids, const float* wts, const void* src, int rows, int dim, int ldx, int ldy,
                                 int ldh, int ld_src, int top_k, int experts, int layernorm, int plus_one, int plain, float eps,
                                 float mult, int f32, const void* b_n, float alpha, const void* extra, const float* extra_w,
-                                int ld_extra, cudaStream_t stream) {
+                                int ld_extra, int groups, const float* conv_w, int conv_n, int taps, void* conv_state,
+                                const int* positions, const int* slots, cudaStream_t stream) {
   if (rows <= 0) return 0;
   const int dim8 = (dim + 7) / 8 * 8;
   if (dim < 1 || dim > 16384 || ldx < dim8 || ldx % 8 || ((w_n || plain) && (ldh != dim8 || !h))) return -2;
   if (y && (ldy < dim8 || ldy % 8)) return -2;
   if (slot_of && (!ids || !wts || top_k < 1 || (src && (ld_src < dim8 || ld_src % 8)))) return -2;
   if ((b_n && !w_n) || (extra && (!slot_of || !extra_w || ld_extra < dim8 || ld_extra % 8))) return -2;
+  if (groups > 1 && (groups > 2048 || dim % groups || layernorm || b_n)) return -2;
+  if (conv_w && (conv_n < 1 || conv_n > 2 || taps < 1 || (taps > 1 && !conv_state) || !positions || !slots || !h)) return -2;
   ResidualNormParams p{static_cast<float*>(x), y, h, static_cast<const __nv_bfloat16*>(w_b),
                        static_cast<const __nv_bfloat16*>(w_n), slot_of, ids, wts, src, dim, ldx, ldy, ldh, ld_src, top_k,
                        experts, layernorm, plus_one, plain, eps, mult, static_cast<const __nv_bfloat16*>(b_n), alpha, extra, extra_w,
-                       ld_extra};
+                       ld_extra, groups, conv_w, conv_n, taps, conv_state, positions, slots};
   return f32 ? launch_residual_norm<float>(p, rows, stream) : launch_residual_norm<__nv_bfloat16>(p, rows, stream);
 }
 
@@ -393,6 +510,17 @@ B200_API int b200_side_gate(const void* u, const int* ids, const void* table, vo
                        static_cast<float*>(y), n, dim / 8, ldu, ldt, vocab)
           : launch_pdl(side_gate_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, static_cast<const __nv_bfloat16*>(u), ids, tab,
                        static_cast<__nv_bfloat16*>(y), n, dim / 8, ldu, ldt, vocab);
+  return e == cudaSuccess ? 0 : -static_cast<int>(e) - 300;
+}
+
+// out [n] fp32 from y [n] (fp32 or bf16); cap 0: scale only
+B200_API int b200_cap_logits(const void* y, void* out, long long n, float scale, float cap, int f32, cudaStream_t stream) {
+  if (n <= 0) return 0;
+  const dim3 grid(static_cast<unsigned>((n + 2047) / 2048));
+  const cudaError_t e = f32 ? launch_pdl(cap_logits_kernel<float>, grid, dim3(256), 0, stream, static_cast<const float*>(y),
+                                         static_cast<float*>(out), n, scale, cap)
+                            : launch_pdl(cap_logits_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, static_cast<const __nv_bfloat16*>(y),
+                                         static_cast<float*>(out), n, scale, cap);
   return e == cudaSuccess ? 0 : -static_cast<int>(e) - 300;
 }
 

@@ -7,6 +7,8 @@
 //                     at once (optional), rotation of the leading values of each head (optional, either pairing), q to a
 //                     dense matrix, k and v straight into their pages. One block per token; the row is read twice, the
 //                     second time from L1.
+//  * head_norm_store  the same with a norm of every head on its own; k and v can be left out (a layer that reads another
+//                     one's pages).
 #include "mixer_common.cuh"
 
 namespace b200 {
@@ -148,6 +150,51 @@ __global__ void __launch_bounds__(512) qk_rope_store_kernel(const QkRopeParams p
   }
 }
 
+// kLanes neighbouring lanes per head. p.inv_q: 1 / true head size; p.hkv 0: no keys and values.
+template <typename T, int kLanes>
+__global__ void __launch_bounds__(512) head_norm_store_kernel(const QkRopeParams p) {
+  pdl_wait();
+  pdl_trigger();
+  const long long t = blockIdx.x;
+  const T* row = static_cast<const T*>(p.p) + t * p.ld;
+  const float2* cs = p.table ? p.table + t * (p.rot >> 1) : nullptr;
+  const long long slot = p.slots[t];
+  const long long page = slot >= 0 ? slot / p.page : 0, off = slot >= 0 ? slot % p.page : 0;
+  const int g = threadIdx.x / kLanes, lane = threadIdx.x % kLanes, all = p.heads + p.hkv;
+  for (int h0 = 0; h0 < all; h0 += blockDim.x / kLanes) {
+    const int h = h0 + g;
+    const bool is_q = h < p.heads, on = is_q || (h < all && slot >= 0);
+    const T* x = row + (is_q ? h * p.d : p.k_off + (h - p.heads) * p.d);
+    float s = 0.f;
+    if (on)
+      for (int c = lane * 8; c < p.d; c += kLanes * 8) {
+        float v[8];
+        load8(x + c, v);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) s = fmaf(v[j], v[j], s);
+      }
+#pragma unroll
+    for (int o = kLanes / 2; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+    if (!on) continue;
+    const float inv = 1.f / sqrtf(s * p.inv_q + p.eps);
+    T* dst = is_q ? static_cast<T*>(p.q_out) + (t * p.heads + h) * p.d
+                  : static_cast<T*>(p.k_cache) + ((page * p.hkv + h - p.heads) * p.page + off) * p.d;
+    for (int c = lane * 8; c < p.d; c += kLanes * 8) {
+      float v[8];
+      turned8(p, x, is_q ? p.wq : p.wk, inv, cs, c, v);
+      store8(dst + c, v);
+    }
+  }
+  if (slot < 0) return;
+  const int vvec = p.dv >> 3;
+  for (int i = threadIdx.x; i < p.hkv * vvec; i += blockDim.x) {
+    const int h = i / vvec, c = (i - h * vvec) * 8;
+    float v[8];
+    load8(row + p.v_off + h * p.dv + c, v);
+    store8(static_cast<T*>(p.v_cache) + ((page * p.hkv + h) * p.page + off) * p.dv + c, v);
+  }
+}
+
 }  // namespace b200
 
 using namespace b200;
@@ -176,5 +223,26 @@ B200_API int b200_qk_rope_store(const void* p, const void* wq, const void* wk, c
   if (threads > 512) threads = 512;
   const cudaError_t e = f32 ? launch_pdl(qk_rope_store_kernel<float>, dim3(tokens), dim3(threads), 0, stream, a)
                             : launch_pdl(qk_rope_store_kernel<__nv_bfloat16>, dim3(tokens), dim3(threads), 0, stream, a);
+  return e == cudaSuccess ? 0 : -static_cast<int>(e) - 300;
+}
+
+// See the header comment: as b200_qk_rope_store with weights [d] that all heads share and a norm per head of its d_true
+// values. hkv 0: q only (wk and the caches are not used).
+B200_API int b200_head_norm_store(const void* p, const void* wq, const void* wk, const void* table, void* q_out, void* k_cache, void* v_cache,
+                                  const long long* slots, int tokens, long long ld, int heads, int hkv, int d, int dv, int k_off, int v_off,
+                                  int page, int rot, int interleaved, int d_true, float eps, int f32, cudaStream_t stream) {
+  if (tokens <= 0) return 0;
+  if (ld % 8 || d % 8 || dv % 8 || k_off % 8 || v_off % 8 || rot % 2 || rot > d || page < 1 || d_true < 1 || !wq || (hkv && !wk)) return -2;
+  QkRopeParams a{p, static_cast<const __nv_bfloat16*>(wq), static_cast<const __nv_bfloat16*>(wk),
+                 rot > 0 ? static_cast<const float2*>(table) : nullptr, q_out, k_cache, v_cache, slots, ld, heads, hkv, d, dv, k_off, v_off,
+                 page, rot, interleaved, 1.f / d_true, 1.f / d_true, eps};
+  const int lanes = d <= 64 ? 8 : d <= 128 ? 16 : 32;
+  int threads = ((heads + hkv) * lanes + 31) / 32 * 32;
+  if (threads > 512) threads = 512;
+  auto go = [&](auto kernel) { return launch_pdl(kernel, dim3(tokens), dim3(threads), 0, stream, a); };
+  cudaError_t e;
+  if (f32) e = lanes == 8 ? go(head_norm_store_kernel<float, 8>) : lanes == 16 ? go(head_norm_store_kernel<float, 16>) : go(head_norm_store_kernel<float, 32>);
+  else e = lanes == 8 ? go(head_norm_store_kernel<__nv_bfloat16, 8>) : lanes == 16 ? go(head_norm_store_kernel<__nv_bfloat16, 16>)
+                                                                            : go(head_norm_store_kernel<__nv_bfloat16, 32>);
   return e == cudaSuccess ? 0 : -static_cast<int>(e) - 300;
 }

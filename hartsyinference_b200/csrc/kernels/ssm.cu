@@ -14,6 +14,8 @@
 //
 //  * short_conv     causal convolution per channel + bias + silu over any column range of a projection; its
 //                   last taps - 1 inputs are state too. short_conv_tail saves them after a portion.
+//  * input_conv     the input plus one or two such convolutions of it, without bias and activation: what the sublayers
+//                   of a layer read.
 //  * channel_scan   one decay per channel and state value (the recurrence above). Four lanes share a channel
 //                   and walk over the tokens with their part of its state in registers; everything that does
 //                   not depend on the state (step size, dt x, D x, silu(z)) is formed once per element while a
@@ -246,6 +248,121 @@ __global__ void __launch_bounds__(128) short_conv_tail_kernel(const ShortConvPar
     if (rel >= 0) load8(x + (first + rel) * p.ldx, v);
     else if (carried) load8(st + static_cast<long long>(rel + tail) * p.channels, v);
     store8(st + static_cast<long long>(j) * p.channels, v);
+  }
+}
+
+// out[o][t] = x[t] + sum over the taps of w[o] for one or two sets of taps (no bias, no activation), as short_conv_kernel
+// otherwise: the same grid, kTaps 0 for any number of taps.
+template <typename T, int kTaps, int kOut>
+__global__ void __launch_bounds__(128) input_conv_kernel(const ShortConvParams p) {
+  pdl_wait();
+  pdl_trigger();
+  constexpr int kT = kTaps > 0 ? kTaps : 1;
+  const int c = (blockIdx.x * 32 + (threadIdx.x & 31)) * 8;
+  const int t0 = (blockIdx.y * 4 + (threadIdx.x >> 5)) * p.run, t1 = min(t0 + p.run, p.tokens);
+  if (c >= p.channels || t0 >= t1) return;
+  const int taps = kTaps > 0 ? kTaps : p.taps, tail = taps - 1;
+  const T* x = static_cast<const T*>(p.x) + c;
+  T* out = static_cast<T*>(p.out) + c;
+  const long long plane = static_cast<long long>(p.tokens) * p.channels;
+  float w[kOut][kT][8], in[kT][8];
+  if (kTaps > 0)
+#pragma unroll
+    for (int o = 0; o < kOut; ++o)
+#pragma unroll
+      for (int j = 0; j < kT; ++j) load8(p.w + static_cast<long long>(o * kT + j) * p.channels + c, w[o][j]);
+  int seq = p.cu_q ? seq_of_token(p.cu_q, p.seqs, t0) : t0;
+  int first = 0, next = 0;
+  bool fresh = true, carried = false;
+  T* st = nullptr;
+  for (int t = t0; t < t1; ++t) {
+    if (fresh || t >= next) {
+      if (!fresh) ++seq;
+      if (p.cu_q) while (p.cu_q[seq + 1] <= t) ++seq;      // empty runs
+      fresh = false;
+      first = p.cu_q ? p.cu_q[seq] : t;
+      next = p.cu_q ? p.cu_q[seq + 1] : t + 1;
+      const int slot = p.slots[seq];
+      carried = slot >= 0 && p.positions[first] > 0;
+      st = slot >= 0 ? static_cast<T*>(p.state) + static_cast<long long>(slot) * tail * p.channels + c : nullptr;
+      if (kTaps > 0)
+#pragma unroll
+        for (int j = 0; j < kT - 1; ++j) {
+#pragma unroll
+          for (int i = 0; i < 8; ++i) in[j][i] = 0.f;
+          const int src = t - tail + j;
+          if (src >= first) load8(x + src * p.ldx, in[j]);
+          else if (carried) load8(st + static_cast<long long>(tail + src - first) * p.channels, in[j]);
+        }
+    }
+    if (kTaps > 0 && t + 4 <= min(t1, next)) {          // four tokens of the same sequence, loads first
+      float nw[4][8];
+#pragma unroll
+      for (int u = 0; u < 4; ++u) load8(x + (t + u) * p.ldx, nw[u]);
+#pragma unroll
+      for (int u = 0; u < 4; ++u)
+#pragma unroll
+        for (int o = 0; o < kOut; ++o) {
+          float y[8];
+#pragma unroll
+          for (int i = 0; i < 8; ++i) {
+            y[i] = nw[u][i];
+#pragma unroll
+            for (int j = 0; j < kT; ++j) {
+              const int at = u - (kT - 1) + j;           // one of the four new inputs, or an earlier one
+              y[i] = fmaf(at >= 0 ? nw[at >= 0 ? at : 0][i] : in[at < 0 ? kT - 1 + at : 0][i], w[o][j][i], y[i]);
+            }
+          }
+          store8(out + o * plane + static_cast<long long>(t + u) * p.channels, y);
+        }
+#pragma unroll
+      for (int j = 0; j + 1 < kT; ++j)
+#pragma unroll
+        for (int i = 0; i < 8; ++i) in[j][i] = nw[(4 - (kT - 1) + j) & 3][i];    // taps are at most four
+      t += 3;
+      continue;
+    }
+    float now[8], y[kOut][8];
+    load8(x + t * p.ldx, now);
+#pragma unroll
+    for (int o = 0; o < kOut; ++o)
+#pragma unroll
+      for (int i = 0; i < 8; ++i) y[o][i] = now[i];
+    if (kTaps > 0) {
+#pragma unroll
+      for (int i = 0; i < 8; ++i) in[kT - 1][i] = now[i];
+#pragma unroll
+      for (int o = 0; o < kOut; ++o)
+#pragma unroll
+        for (int j = 0; j < kT; ++j)
+#pragma unroll
+          for (int i = 0; i < 8; ++i) y[o][i] = fmaf(in[j][i], w[o][j][i], y[o][i]);
+      if (p.cu_q == nullptr && st != nullptr)
+#pragma unroll
+        for (int j = 1; j < kT; ++j) store8(st + static_cast<long long>(j - 1) * p.channels, in[j]);
+#pragma unroll
+      for (int j = 0; j + 1 < kT; ++j)
+#pragma unroll
+        for (int i = 0; i < 8; ++i) in[j][i] = in[j + 1][i];
+    } else {
+      for (int j = 0; j < taps; ++j) {
+        const int src = t - tail + j;
+        float v[8], wj[8];
+#pragma unroll
+        for (int i = 0; i < 8; ++i) v[i] = 0.f;
+        if (src >= first) load8(x + src * p.ldx, v);
+        else if (carried) load8(st + static_cast<long long>(tail + src - first) * p.channels, v);
+        if (p.cu_q == nullptr && st != nullptr && j > 0) store8(st + static_cast<long long>(j - 1) * p.channels, v);
+#pragma unroll
+        for (int o = 0; o < kOut; ++o) {
+          load8(p.w + (static_cast<long long>(o) * taps + j) * p.channels + c, wj);
+#pragma unroll
+          for (int i = 0; i < 8; ++i) y[o][i] = fmaf(v[i], wj[i], y[o][i]);
+        }
+      }
+    }
+#pragma unroll
+    for (int o = 0; o < kOut; ++o) store8(out + o * plane + static_cast<long long>(t) * p.channels, y[o]);
   }
 }
 
@@ -1021,14 +1138,34 @@ __global__ void __launch_bounds__(1024) gated_norm_kernel(const GatedNormParams 
   }
 }
 
+// Grid of the convolutions: enough warps to cover the machine, then as many tokens per warp as that leaves
+inline dim3 conv_grid(ShortConvParams& p) {
+  const int vecs = (p.channels / 8 + 31) / 32;
+  p.run = 1;
+  if (p.cu_q) while (p.run < 32 && static_cast<long long>(p.tokens) * vecs / (2 * p.run) >= 148 * 16) p.run *= 2;
+  return dim3(vecs, (p.tokens + 4 * p.run - 1) / (4 * p.run));
+}
+
+template <typename T, int kOut>
+int launch_input_conv(ShortConvParams p, cudaStream_t stream) {
+  const dim3 grid = conv_grid(p);
+  if (grid.y > 65535) return -2;
+  cudaError_t e;
+  switch (p.taps) {
+    case 1: e = launch_pdl(input_conv_kernel<T, 1, kOut>, grid, dim3(128), 0, stream, p); break;
+    case 2: e = launch_pdl(input_conv_kernel<T, 2, kOut>, grid, dim3(128), 0, stream, p); break;
+    case 3: e = launch_pdl(input_conv_kernel<T, 3, kOut>, grid, dim3(128), 0, stream, p); break;
+    case 4: e = launch_pdl(input_conv_kernel<T, 4, kOut>, grid, dim3(128), 0, stream, p); break;
+    default: e = launch_pdl(input_conv_kernel<T, 0, kOut>, grid, dim3(128), 0, stream, p); break;
+  }
+  if (e == cudaSuccess && p.cu_q && p.taps > 1)
+    e = launch_pdl(short_conv_tail_kernel<T>, dim3((p.channels / 8 + 127) / 128, p.seqs), dim3(128), 0, stream, p);
+  return e == cudaSuccess ? 0 : -static_cast<int>(e) - 300;
+}
+
 template <typename T>
 int launch_short_conv(ShortConvParams p, cudaStream_t stream) {
-  const int vecs = (p.channels / 8 + 31) / 32;
-  // enough warps to cover the machine, then as many tokens per warp as that leaves
-  int run = 1;
-  if (p.cu_q) while (run < 32 && static_cast<long long>(p.tokens) * vecs / (2 * run) >= 148 * 16) run *= 2;
-  p.run = run;
-  const dim3 grid(vecs, (p.tokens + 4 * run - 1) / (4 * run));
+  const dim3 grid = conv_grid(p);
   if (grid.y > 65535) return -2;
   cudaError_t e;
   switch (p.taps) {
@@ -1161,6 +1298,18 @@ B200_API int b200_short_conv(const void* x, const float* w, const float* bias, v
   if (channels % 8 || ldx % 8 || taps < 1 || seqs > 65535 || (!cu_q && seqs != tokens)) return -2;
   ShortConvParams p{x, w, bias, state, positions, cu_q, slots, out, ldx, tokens, seqs, channels, taps, 1};
   return f32 ? launch_short_conv<float>(p, stream) : launch_short_conv<__nv_bfloat16>(p, stream);
+}
+
+// h [tokens][ldx] -> out [n][tokens][channels] (see input_conv_kernel) with w [n][taps][channels], n 1 or 2; channels
+// and ldx multiples of 8
+B200_API int b200_input_conv(const void* h, const float* w, void* state, const int* positions, const int* cu_q, const int* slots,
+                             void* out, int tokens, int seqs, int channels, int taps, int n, long long ldx, int f32,
+                             cudaStream_t stream) {
+  if (tokens <= 0 || seqs <= 0) return 0;
+  if (channels % 8 || ldx % 8 || taps < 1 || n < 1 || n > 2 || seqs > 65535 || (!cu_q && seqs != tokens)) return -2;
+  ShortConvParams p{h, w, nullptr, state, positions, cu_q, slots, out, ldx, tokens, seqs, channels, taps, 1};
+  if (f32) return n == 1 ? launch_input_conv<float, 1>(p, stream) : launch_input_conv<float, 2>(p, stream);
+  return n == 1 ? launch_input_conv<__nv_bfloat16, 1>(p, stream) : launch_input_conv<__nv_bfloat16, 2>(p, stream);
 }
 
 // n in {8, 16, 32, 64, 128}; channels, offsets and row pitches multiples of 8

@@ -74,7 +74,7 @@ class RotarySpec:
 @dataclass(frozen=True)
 class MixerSpec:
     """Token mixer of one layer of a model whose layers differ (``TransformerConfig.layer_specs``)."""
-    kind: str = "attention"             # attention | channel_delta | latent_attention | channel_scan | head_scan
+    kind: str = "attention"             # attention | channel_delta | general_delta | latent_attention | channel_scan | head_scan
     heads: int = 1
     kv_heads: int = 1
     dim: int = 64                       # query / key size per head
@@ -86,19 +86,24 @@ class MixerSpec:
     keep_first: int = 0                 # first tokens of the sequence that stay visible outside the window
     rot: Optional[RotarySpec] = None
     qk_norm: bool = False               # RMS norm of q and of k over all their heads at once, before the rotation
+    head_norm: bool = False             # or of every head of q and k on its own (one weight for all heads)
+    slope_bias: bool = False            # score - 2^(-8 (h + 1) / heads) * distance for head h
+    kv_from: Optional[int] = None       # layer whose keys and values this one reads (it has none of its own)
     bias_reach: int = 0                 # distance at which the logarithmic bias buckets end (0: no distance bias)
     bias_rows: int = 32                 # bias table rows of synthetic weights (a checkpoint's table gives its own)
     shared_kv: bool = False             # the values are the keys
     qk_bias: bool = False
     out_gate: bool = False              # output * sigmoid(W_g h)
-    sink: Optional[float] = None        # score of a key without a value
+    head_gate: bool = False             # the same with one number per head
+    sink: Optional[float] = None        # score of a key without a value (latent_attention: per head, from the checkpoint)
     # latent_attention (dim / vdim: unrotated query-key and value size per head; window, rot and out_gate as above)
     q_rank: int = 0                     # size of the query latent
     kv_rank: int = 0                    # size of the cached key / value latent
     rot_dim: int = 0                    # rotated query-key size per head; the keys share one rotated part
     # recurrent kinds
     conv: int = 0                       # taps of the short convolution
-    rank: int = 0                       # low-rank size: channel_delta decay and gate in synthetic weights (0 = dim); channel_scan step size
+    rank: int = 0                       # low-rank size: channel_delta decay and gate, general_delta decay in synthetic weights (0 = dim);
+                                        # channel_scan step size
     state: int = 0                      # channel_scan: state values per channel; head_scan: state rows per head (columns: vdim)
     inner: int = 0                      # channel_scan: channels
     groups: int = 1                     # head_scan: groups of heads that share B and C
@@ -107,14 +112,14 @@ class MixerSpec:
     @property
     def recurrent(self) -> bool:
         """The mixer carries a state: its sequences need a slot."""
-        return self.kind in ("channel_delta", "channel_scan", "head_scan")
+        return self.kind in ("channel_delta", "general_delta", "channel_scan", "head_scan")
 
 
 @dataclass(frozen=True)
 class DenseSpec:
     """Dense feed-forward of one layer: ungated down(act(up h)), or down(silu(gate h) * up h)."""
     ffn: int
-    act: str = "poly_norm"              # poly_norm (ungated) | silu (gated)
+    act: str = "poly_norm"              # poly_norm | relu2 (ungated) | silu (gated)
 
 
 @dataclass(frozen=True)
@@ -164,6 +169,7 @@ class TransformerConfig:
     rope_local_theta: float = 0.0       # rotary base of the sliding-window layers when it differs (Gemma 3)
     layer_types: tuple = ()             # explicit per-layer "sliding_attention" / "full_attention"
     norm_type: str = "rms"              # rms | layernorm | tanh (no statistics: tanh(alpha x) w + b)
+    norm_groups: int = 1                # models with per-layer mixers: equal parts of a row, each normed on its own
     norm_bias: bool = False
     parallel_residual: bool = False     # x + attn(n1(x)) + ffn(n2(x)) (GPT-NeoX, Cohere)
     shared_parallel_norm: bool = False  # the parallel branches share one norm (Cohere)
@@ -184,6 +190,8 @@ class TransformerConfig:
     mla: Optional[MlaConfig] = None
     layer_specs: tuple = ()             # one LayerSpec per layer: mixers of different kinds and sizes around a 32-bit
                                         # residual stream, norms before and / or after every sublayer
+    input_conv: int = 0                 # > 0: every sublayer reads h + a causal convolution of h with this many taps; its last
+                                        # inputs are part of a sequence's state
     token_side: int = 0                 # > 0: every layer adds a gated map of its part (this many values) of a second token embedding
     bos_token_id: int = 1
     eos_token_ids: tuple = (2,)
@@ -210,8 +218,8 @@ class TransformerConfig:
 
     @property
     def recurrent(self) -> bool:
-        """True when some layer is recurrent: its sequences need a state slot."""
-        return any(ls.mixer.recurrent for ls in self.layer_specs)
+        """True when some layer is recurrent, or keeps inputs of a convolution: sequences need a state slot."""
+        return self.input_conv > 1 or any(ls.mixer.recurrent for ls in self.layer_specs)
 
     @property
     def general_path(self) -> bool:
@@ -247,6 +255,8 @@ class TransformerConfig:
         if self.layer_specs:
             from .mixers import spec_param_count
             own = sum(spec_param_count(ls, h) for ls in self.layer_specs if ls.weights_of is None)
+            if self.input_conv:
+                own += sum(1 + (ls.dense is not None or ls.moe is not None) for ls in self.layer_specs) * h * self.input_conv
             if self.token_side:
                 own += l * (self.token_side * (self.vocab_size + 2 * h) + h)
             return own + (1 if self.tie_embeddings else 2) * self.vocab_size * h + h
@@ -322,7 +332,7 @@ def tiny(base: str = "qwen2.5-0.5b", **over: Any) -> TransformerConfig:
 
 # designs whose layers are described one by one; each is a module of this package with ``config_from``,
 # ``load_layers``, ``tensor_shapes`` and ``random_tensor``
-MIXED_DESIGNS = ("lududra", "salopel", "zovudra")
+MIXED_DESIGNS = ("ginodra", "lududra", "salopel", "zovudra")
 
 
 def mixed_design(arch: str):

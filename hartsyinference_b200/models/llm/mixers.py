@@ -54,6 +54,11 @@ def _linear(parts: Iterable[torch.Tensor], device, bias: Optional[torch.Tensor] 
     return LinearWeight(w, None, None if bias is None else bias.to(torch.bfloat16).to(device).contiguous())
 
 
+def out_matrix(o: Optional[torch.Tensor], heads: int, v: int, vp: int, width: int, device) -> Optional[LinearWeight]:
+    """A mixer's output matrix in its laid-out sizes; None when the layer holds it (:class:`ParallelBlock`)."""
+    return None if o is None else _linear([pad_rows(pad_head_cols(o, heads, v, vp), pad_to(width, 8))], device)
+
+
 def distance_bias_table(rel: torch.Tensor, reach: int, window: int) -> torch.Tensor:
     """Per-head bias by key distance, fp32 [heads, n]: distances below half of the table's rows have a row of
     their own, longer ones share rows on a logarithmic scale that ends at ``reach``. The table stops where
@@ -74,44 +79,56 @@ def distance_bias_table(rel: torch.Tensor, reach: int, window: int) -> torch.Ten
 
 
 class BiasedAttention:
-    """Grouped-query attention over the page pool with a norm over all heads of q and of k, a rotation, a distance
-    bias, a window with kept first tokens, a score cap, a sink and an output gate, each as the spec says. One projection
-    GEMM (q | k | v | gate)."""
+    """Grouped-query attention over the page pool with a norm of q and of k (over all heads at once or per head), a rotation,
+    a distance bias (a table or a slope per head), a window with kept first tokens, a score cap, a sink and an output gate (per
+    value or per head), each as the spec says. One projection GEMM (q | k | v | gate). Without ``k`` and ``v`` it reads the
+    pages of another layer (``spec.kv_from``), which come before it in the same pass."""
 
-    def __init__(self, spec: MixerSpec, width: int, device, *, q: torch.Tensor, k: torch.Tensor, v: Optional[torch.Tensor],
-                 o: torch.Tensor, q_bias: Optional[torch.Tensor] = None, k_bias: Optional[torch.Tensor] = None,
+    def __init__(self, spec: MixerSpec, width: int, device, *, q: torch.Tensor, k: Optional[torch.Tensor] = None, v: Optional[torch.Tensor] = None,
+                 o: Optional[torch.Tensor], q_bias: Optional[torch.Tensor] = None, k_bias: Optional[torch.Tensor] = None,
                  gate: Optional[torch.Tensor] = None, rel: Optional[torch.Tensor] = None, q_norm: Optional[torch.Tensor] = None,
                  k_norm: Optional[torch.Tensor] = None, eps: float = 0.0):
         self.spec, self.eps = spec, eps
-        hq, hk, d, dv = spec.heads, spec.kv_heads, spec.dim, spec.dim if v is None else spec.vdim
+        borrowed = spec.kv_from is not None
+        self.shared_kv, self.gated = v is None and not borrowed, gate is not None
+        hq, hk, d, dv = spec.heads, spec.kv_heads, spec.dim, spec.dim if self.shared_kv else spec.vdim
         if max(d, dv) > 512:
             raise ValueError(f"attention heads of {d} / {dv} values are not supported (at most 512)")
+        if borrowed != (k is None) or (borrowed and (v is not None or k_norm is not None)):
+            raise ValueError("attention: keys and values are a layer's own or another layer's")
         self.d, self.dv = dp, vp = pad_to(d, 8), pad_to(dv, 8)
         wp = pad_to(width, 8)
         head = lambda t, n: pad_head_rows(t, n, d, dp)
         vhead = lambda t, n: pad_head_rows(t, n, dv, vp)
-        parts = [head(q, hq), head(k, hk)] + ([vhead(v, hk)] if v is not None else []) + ([vhead(gate, hq)] if gate is not None else [])
+        parts = [head(q, hq)] + ([head(k, hk)] if k is not None else []) + ([vhead(v, hk)] if v is not None else [])
+        if gate is not None:
+            parts.append(pad_rows(gate, pad_to(hq, 8)) if spec.head_gate else vhead(gate, hq))
         bias = None
         if q_bias is not None:
             rest = sum(p.shape[0] for p in parts[2:])
             bias = torch.cat([head(q_bias, hq), head(k_bias, hk), torch.zeros(rest, dtype=q_bias.dtype, device=q_bias.device)])
         self.proj = _linear([pad_cols(p, wp) for p in parts], device, bias)
-        self.o = _linear([pad_rows(pad_head_cols(o, hq, dv, vp), wp)], device)
-        self.nq, self.nk, self.nv = hq * dp, hk * dp, hk * vp
-        self.shared_kv, self.gated = v is None, gate is not None
+        self.o = out_matrix(o, hq, dv, vp, width, device)
+        self.nq, self.nk, self.nv = hq * dp, 0 if borrowed else hk * dp, 0 if borrowed or self.shared_kv else hk * vp
+        self.inner = hq * vp
         norm = lambda t, n: None if t is None else head(t, n).to(torch.bfloat16).to(device).contiguous()
-        self.q_norm, self.k_norm = norm(q_norm, hq), norm(k_norm, hk)
+        self.q_norm, self.k_norm = (norm(t, 1 if spec.head_norm else n) for t, n in ((q_norm, hq), (k_norm, hk)))
         self.rotary = None if spec.rot is None else Rotary(spec.rot, device)
         if self.shared_kv and (self.rotary is not None or q_norm is not None):
             raise ValueError("attention: keys that are values are neither normed nor turned")
         self.bias = distance_bias_table(rel, spec.bias_reach, spec.window).to(device) if rel is not None and spec.bias_reach > 0 else None
+        self.slopes = None
+        if spec.slope_bias:
+            self.slopes = torch.tensor([2.0 ** (-8.0 * (h + 1) / hq) for h in range(hq)], dtype=torch.float32, device=device)
         self.sinks = None if spec.sink is None else torch.full((hq,), float(spec.sink), dtype=torch.float32, device=device)
         self.scale = spec.scale or d ** -0.5
+        if not borrowed:
+            self.cache_shape = self._cache_shape
 
     def nbytes(self) -> int:
-        return self.proj.nbytes() + self.o.nbytes()
+        return self.proj.nbytes() + (0 if self.o is None else self.o.nbytes())
 
-    def cache_shape(self, pages: int, page: int) -> tuple:
+    def _cache_shape(self, pages: int, page: int) -> tuple:
         """[planes, pages, kv heads, page, head size], or, with values of another size than the keys, all key pages and
         then all value pages in one row."""
         hk = self.spec.kv_heads
@@ -128,16 +145,17 @@ class BiasedAttention:
         flat = cache.view(-1)
         return flat[:n].view(pages, hk, page, self.d), flat[n:].view(pages, hk, page, self.dv)
 
-    def __call__(self, h: torch.Tensor, batch, li: int, model) -> torch.Tensor:
+    def values(self, h: torch.Tensor, batch, li: int, model, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """Gated head outputs [T, heads * value size], before the output product."""
+        spec = self.spec
         p = ops.linear_act(h, self.proj)
         k0, v0 = self.nq, self.nq + self.nk
-        g0 = v0 if self.shared_kv else v0 + self.nv
-        cache = model.kv_cache[li]
-        kc, vc = self._planes(cache)
+        g0 = v0 + self.nv
+        kc, vc = self._planes(model.kv_cache[li if spec.kv_from is None else spec.kv_from])
         if self.rotary is not None or self.q_norm is not None:
-            q = ops.qk_rope_store(p, self.spec.heads, kc, vc, batch.slot_mapping, table=None if self.rotary is None else self.rotary.table(batch),
+            q = ops.qk_rope_store(p, spec.heads, kc, vc, batch.slot_mapping, table=None if self.rotary is None else self.rotary.table(batch),
                                   interleaved=self.rotary is not None and self.rotary.spec.interleaved, q_norm=self.q_norm, k_norm=self.k_norm,
-                                  d_true=self.spec.dim, eps=self.eps)
+                                  d_true=spec.dim, eps=self.eps, per_head=spec.head_norm, store=spec.kv_from is None)
         else:
             q = p[:, :k0]
             if self.shared_kv or self.d == self.dv:
@@ -145,11 +163,14 @@ class BiasedAttention:
             else:
                 ops.kv_store(p[:, k0:v0], kc, batch.slot_mapping)
                 ops.kv_store(p[:, v0:g0], vc, batch.slot_mapping)
-        a = ops.attn_biased(q, kc, vc, batch.block_table, batch.kv_lens, None if batch.is_decode else batch.cu_q,
-                            heads=self.spec.heads, max_q_len=batch.max_q_len, max_kv_len=batch.max_kv_len, scale=self.scale,
-                            softcap=self.spec.softcap, window=self.spec.window, dist_bias=self.bias, sinks=self.sinks,
-                            gate=p[:, g0:] if self.gated else None, keep_first=self.spec.keep_first)
-        return ops.linear_act(a, self.o)
+        return ops.attn_biased(q, kc, vc, batch.block_table, batch.kv_lens, None if batch.is_decode else batch.cu_q,
+                               heads=spec.heads, max_q_len=batch.max_q_len, max_kv_len=batch.max_kv_len, scale=self.scale,
+                               softcap=spec.softcap, window=spec.window, dist_bias=self.bias, sinks=self.sinks,
+                               gate=p[:, g0:] if self.gated else None, keep_first=spec.keep_first, slopes=self.slopes,
+                               head_gate=spec.head_gate, out=out)
+
+    def __call__(self, h: torch.Tensor, batch, li: int, model) -> torch.Tensor:
+        return ops.linear_act(self.values(h, batch, li, model), self.o)
 
 
 class DeltaMixer:
@@ -194,6 +215,45 @@ class DeltaMixer:
         y = ops.delta_mix(p, z, self.w, conv, state, batch.positions, None if batch.is_decode else batch.cu_q, batch.state_slots,
                           self.b_off)
         return ops.linear_act(y, self.o)
+
+
+class GeneralDeltaMixer:
+    """Delta rule whose removal has a rate of its own per key channel: ``S = diag(w) S - (a u)(u^T S) + k v^T`` with the unit
+    key u, read by r, normed per head, weighted and gated. Two GEMMs before the recurrence: every projection of h at once
+    (r | k | removal rate | v | gate | low-rank decay, the last with tanh in its epilogue), then the decay's expansion."""
+
+    def __init__(self, spec: MixerSpec, width: int, eps: float, device, *, r, k, v, a, a_bias, g, w1, w2, w0, norm, o):
+        self.spec = spec
+        h, d = spec.heads, spec.dim
+        if d > 256:
+            raise ValueError(f"general_delta heads of {d} values are not supported (at most 256)")
+        dp, vp, wp = pad_to(d, 32), pad_to(d, 8), pad_to(width, 8)
+        rank = pad_to(w1.shape[0], 8)
+        key, val = (lambda t: pad_head_rows(t, h, d, dp)), (lambda t: pad_head_rows(t, h, d, vp))
+        self.low = 3 * h * dp + 2 * h * vp
+        self.proj = _linear([pad_cols(p, wp) for p in (key(r), key(k), key(a), val(v), val(g), pad_rows(w1, rank))], device)
+        self.up = _linear([pad_cols(key(w2), rank)], device)
+        self.o = out_matrix(o, h, d, vp, width, device)
+        self.inner = h * vp
+        f32 = lambda t: t.float().to(device).contiguous()
+        self.w = ops.GeneralDeltaWeights(decay_bias=f32(key(w0)), rate_bias=f32(key(a_bias)), norm=val(norm).to(torch.bfloat16).to(device).contiguous(),
+                                         heads=h, dk=dp, dv=vp, d_true=d, eps=eps)
+
+    def nbytes(self) -> int:
+        return self.proj.nbytes() + self.up.nbytes() + (0 if self.o is None else self.o.nbytes())
+
+    def state_shapes(self, slots: int) -> tuple[Optional[tuple], tuple]:
+        w = self.w
+        return None, (slots, w.heads, w.dk, w.dv)
+
+    def values(self, h: torch.Tensor, batch, li: int, model, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+        p = ops.linear_act(h, self.proj, "tanh", act_from=self.low)
+        z = ops.linear_act(p[:, self.low:], self.up)
+        return ops.general_delta(p, z, self.w, model.mixer_state[li][1], batch.positions, None if batch.is_decode else batch.cu_q,
+                                 batch.state_slots, out=out)
+
+    def __call__(self, h: torch.Tensor, batch, li: int, model) -> torch.Tensor:
+        return ops.linear_act(self.values(h, batch, li, model), self.o)
 
 
 class ChannelScanMixer:
@@ -341,22 +401,31 @@ class LatentPlan:
 class LatentAttention:
     """Attention whose keys and values are per-head maps of one cached latent; queries through a latent of their
     own. Optional: a rotated part of queries and keys (one rotated key for all heads, cached behind the latent), a
-    window, a sigmoid output gate. One projection GEMM (query latent | latent | rotated key | gate)."""
+    window, a sink per head, a sigmoid output gate (per value or per head). One projection GEMM (query latent | latent |
+    rotated key | gate). The kernels turn pairs of neighbours; for a rotation of split halves the rotated rows of both
+    projections are put in that order, which leaves the scores as they are."""
 
-    def __init__(self, spec: MixerSpec, width: int, eps: float, device, *, dq, dq_norm, uq, dkv, dkv_norm, uk, uv, o, g=None):
+    def __init__(self, spec: MixerSpec, width: int, eps: float, device, *, dq, dq_norm, uq, dkv, dkv_norm, uk, uv, o, g=None, sinks=None):
         self.spec, self.eps = spec, eps
         h, d, v, t = spec.heads, spec.dim, spec.vdim, spec.rot_dim
         if spec.kv_rank > 512:
             raise ValueError(f"latent_attention with a latent of {spec.kv_rank} values is not supported (at most 512)")
         if t % 2 or t > 512 or bool(t) != (spec.rot is not None):
             raise ValueError(f"latent_attention with a rotated part of {t} values is not supported (even, at most 512, with its rotation)")
+        if t and not spec.rot.interleaved:
+            pairs = torch.arange(t).reshape(2, t // 2).t().reshape(-1).to(uq.device)
+            uq = torch.cat([uq.reshape(h, d + t, -1)[:, :d], uq.reshape(h, d + t, -1)[:, d:][:, pairs]], 1).reshape(h * (d + t), -1)
+            dkv = torch.cat([dkv[:spec.kv_rank], dkv[spec.kv_rank:][pairs.to(dkv.device)]])
         wp = pad_to(width, 8)
         self.d, self.v, self.t = dp, vp, tp = pad_to(d, 8), pad_to(v, 8), pad_to(t, 8)
         self.qr, self.r = qr, r = pad_to(spec.q_rank, 8), pad_to(spec.kv_rank, 8)
         head = lambda m, k, kp: pad_head_rows(m, h, k, kp)
         parts = [pad_rows(dq, qr), pad_rows(dkv[:spec.kv_rank], r)] + ([pad_rows(dkv[spec.kv_rank:], tp)] if t else [])
-        self.proj = _linear([pad_cols(p, wp) for p in parts + ([] if g is None else [head(g, v, vp)])], device)
+        if g is not None:
+            parts.append(pad_rows(g, pad_to(h, 8)) if spec.head_gate else head(g, v, vp))
+        self.proj = _linear([pad_cols(p, wp) for p in parts], device)
         self.gated = g is not None
+        self.sinks = None if sinks is None else sinks.float().to(device).contiguous()
         vec = lambda m, n: pad_rows(m, n).to(torch.bfloat16).to(device).contiguous()
         self.q_norm, self.kv_norm = vec(dq_norm, qr), vec(dkv_norm, r)
         if t:                                    # both parts of every head padded on their own
@@ -370,14 +439,15 @@ class LatentAttention:
         self.kv_up = _linear([uk, uv], device)
         self.uv = LinearWeight(self.kv_up.weight[h * dp:])
         self.uk_t = _linear([uk.reshape(h, dp, r).transpose(1, 2).reshape(h * r, dp)], device)     # the query's side of W_uk
-        self.o = _linear([pad_rows(pad_head_cols(o, h, v, vp), wp)], device)
+        self.o = out_matrix(o, h, v, vp, width, device)
+        self.inner = h * vp
         self.scale = spec.scale or (d + t) ** -0.5
         self.rotary = None if spec.rot is None else Rotary(spec.rot, device)
-        if self.rotary is not None and (not spec.rot.interleaved or spec.rot.dims != t):
-            raise ValueError("latent_attention turns the whole rotated part in pairs of neighbours")
+        if self.rotary is not None and spec.rot.dims != t:
+            raise ValueError("latent_attention turns the whole rotated part")
 
     def nbytes(self) -> int:
-        return sum(w.nbytes() for w in (self.proj, self.uq, self.kv_up, self.uk_t, self.o))
+        return sum(w.nbytes() for w in (self.proj, self.uq, self.kv_up, self.uk_t, self.o) if w is not None)
 
     def cache_shape(self, pages: int, page: int) -> tuple:
         return (1, pages, 1, page, self.r + self.t)
@@ -391,8 +461,9 @@ class LatentAttention:
             batch.plan[key] = LatentPlan(batch, *key)
         return batch.plan[key]
 
-    def __call__(self, h: torch.Tensor, batch, li: int, model) -> torch.Tensor:
-        heads, window, r = self.spec.heads, self.spec.window, self.r
+    def values(self, h: torch.Tensor, batch, li: int, model, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """Gated head outputs [T, heads * value size], before the output product."""
+        heads, window, r, head_gate = self.spec.heads, self.spec.window, self.r, self.spec.head_gate
         table = None if self.rotary is None else self.rotary.table(batch)
         p = ops.linear_act(h, self.proj)
         gate = p[:, self.qr + r + self.t:] if self.gated else None
@@ -402,50 +473,91 @@ class LatentAttention:
         q = ops.linear_act(cq, self.uq)
         if batch.is_decode:
             a = ops.latent_attn(ops.head_linear(q, self.uk_t, heads, tail=self.t, table=table), cache, batch.block_table, batch.kv_lens, heads,
-                                self.scale, max_kv_len=batch.max_kv_len, v_dim=r, window=window)
-            return ops.linear_act(ops.head_linear(a, self.uv, heads, gate=gate), self.o)
+                                self.scale, max_kv_len=batch.max_kv_len, v_dim=r, window=window, sinks=self.sinks)
+            return ops.head_linear(a, self.uv, heads, gate=gate, head_gate=head_gate, out=out)
         plan = self._plan(batch, h)
-        y = torch.empty(h.shape[0], heads * self.v, dtype=h.dtype, device=h.device)
+        y = torch.empty(h.shape[0], heads * self.v, dtype=h.dtype, device=h.device) if out is None else out
         for g in plan.groups:
             c = ops.latent_gather(cache, batch.block_table, g["seqs"], g["offsets"], g["total"], g["max_kv"], g["first"])
             kv = ops.linear_act(c[:, :r], self.kv_up)
             ops.attn_runs(q, kv[:, :heads * self.d], kv[:, heads * self.d:], y, g["q_start"], g["q_lens"], g["offsets"], g["kv_lens"],
                           heads=heads, max_q_len=g["max_q"], scale=self.scale, gate=gate, window=window,
-                          k_shared=c[:, r:] if self.t else None, table=table)
+                          k_shared=c[:, r:] if self.t else None, table=table, sinks=self.sinks, head_gate=head_gate)
         if plan.short:
             ql = ops.head_linear(q, self.uk_t, heads, in_rows=plan.rows, tail=self.t, table=table)
             a = ops.latent_attn(ql, cache, batch.block_table, plan.row_len, heads, self.scale, row_seq=plan.row_seq,
-                                max_kv_len=batch.max_kv_len, v_dim=r, window=window)
-            ops.head_linear(a, self.uv, heads, gate=gate, out=y, out_rows=plan.rows)
-        return ops.linear_act(y, self.o)
+                                max_kv_len=batch.max_kv_len, v_dim=r, window=window, sinks=self.sinks)
+            ops.head_linear(a, self.uv, heads, gate=gate, head_gate=head_gate, out=y, out_rows=plan.rows)
+        return y
+
+    def __call__(self, h: torch.Tensor, batch, li: int, model) -> torch.Tensor:
+        return ops.linear_act(self.values(h, batch, li, model), self.o)
 
 
 class DenseFeedForward:
-    """Feed-forward ``down(act(up h))`` (``coef``: the activation's numbers), or gated: ``down(silu(gate h) * up h)``."""
+    """Feed-forward ``down(act(up h))`` (``coef``: the activation's numbers), or gated: ``down(silu(gate h) * up h)``.
+    ``down`` None: the layer holds it (:class:`ParallelBlock`)."""
 
     def __init__(self, spec: DenseSpec, width: int, eps: float, device, *, up, down, coef=None, gate=None):
-        if spec.act not in ("poly_norm", "silu"):
+        if spec.act not in ("poly_norm", "relu2", "silu"):
             raise ValueError(f"unknown activation '{spec.act}'")
         self.spec, self.eps = spec, eps
-        fp, wp = pad_to(spec.ffn, 8), pad_to(width, 8)
+        self.inner = fp = pad_to(spec.ffn, 8)
+        wp = pad_to(width, 8)
         rows = [pad_rows(pad_cols(t, wp), fp) for t in (gate, up) if t is not None]
         if len(rows) != (2 if spec.act == "silu" else 1):
             raise ValueError(f"a feed-forward with activation '{spec.act}' has {'a' if spec.act == 'silu' else 'no'} gate")
         self.up = _linear(rows, device)
-        self.down = _linear([pad_rows(pad_cols(down, fp), wp)], device)
+        self.down = None if down is None else _linear([pad_rows(pad_cols(down, fp), wp)], device)
         self.coef = None if coef is None else coef.float().to(device).contiguous()
 
     def nbytes(self) -> int:
-        return self.up.nbytes() + self.down.nbytes()
+        return self.up.nbytes() + (0 if self.down is None else self.down.nbytes())
 
-    def __call__(self, h: torch.Tensor, model=None) -> torch.Tensor:
+    def values(self, h: torch.Tensor, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """The activation's output [T, inner], before the down product."""
+        if self.spec.act == "relu2":
+            return ops.linear_act(h, self.up, "relu2", out=out)
         if self.spec.act == "poly_norm":
-            return ops.linear_act(ops.poly_norm(ops.linear_act(h, self.up), self.coef, self.spec.ffn, self.eps), self.down)
-        if h.dtype == torch.float32:
+            a = ops.poly_norm(ops.linear_act(h, self.up), self.coef, self.spec.ffn, self.eps)
+        elif h.dtype == torch.float32:
             a = ops.glu_clamped(ops.linear_act(h, self.up), math.inf, 1.0, shift=0.0)
         else:
             a, _ = ops.glu(ops.linear(h, self.up, defer=h.is_cuda and h.shape[0] <= 128))
-        return ops.linear_act(a, self.down)
+        return a if out is None else out.copy_(a)
+
+    def __call__(self, h: torch.Tensor, model=None) -> torch.Tensor:
+        return ops.linear_act(self.values(h), self.down)
+
+
+class ParallelBlock:
+    """Mixer and feed-forward of a layer that read the same norm and whose outputs are summed: both write what precedes
+    their output product side by side into one buffer, and one product with the two output matrices side by side gives
+    the sum, accumulated in 32 bits and rounded once."""
+
+    def __init__(self, mixer, ffn: Optional[DenseFeedForward], width: int, device, *, o: torch.Tensor, down: Optional[torch.Tensor]):
+        self.mixer, self.ffn = mixer, ffn
+        heads = mixer.spec.heads
+        vp = mixer.inner // heads
+        parts = [pad_head_cols(o, heads, o.shape[1] // heads, vp).to(o.device)]
+        if ffn is not None:
+            parts.append(pad_cols(down.to(o.device), ffn.inner))
+        self.out = _linear([pad_rows(torch.cat(parts, 1), pad_to(width, 8))], device)
+        for name in ("cache_shape", "state_shapes"):       # what the cache and the state manager ask a layer for
+            if hasattr(mixer, name):
+                setattr(self, name, getattr(mixer, name))
+
+    def nbytes(self) -> int:
+        return self.mixer.nbytes() + self.out.nbytes() + (0 if self.ffn is None else self.ffn.nbytes())
+
+    def __call__(self, h: torch.Tensor, hf: Optional[torch.Tensor], batch, li: int, model) -> torch.Tensor:
+        """``h`` goes to the mixer, ``hf`` to the feed-forward."""
+        n = self.mixer.inner
+        buf = torch.empty(h.shape[0], self.out.weight.shape[1], dtype=h.dtype, device=h.device)
+        self.mixer.values(h, batch, li, model, out=buf[:, :n])
+        if self.ffn is not None:
+            self.ffn.values(hf, out=buf[:, n:])
+        return ops.linear_act(buf, self.out)
 
 
 class TokenInput:
@@ -495,7 +607,7 @@ def build_experts(moe: MoeConfig, width: int, device, router: torch.Tensor, corr
 def spec_param_count(ls: LayerSpec, width: int) -> int:
     m = ls.mixer
     if m.kind == "latent_attention":
-        n = width * (m.q_rank + m.kv_rank + m.rot_dim + (1 + m.out_gate) * m.heads * m.vdim)
+        n = width * (m.q_rank + m.kv_rank + m.rot_dim + m.heads * ((1 + m.out_gate) * m.vdim + m.head_gate))
         n += m.heads * (m.q_rank * (m.dim + m.rot_dim) + m.kv_rank * (m.dim + m.vdim))
     elif m.kind == "channel_scan":
         n = m.inner * (3 * width + 2 * m.rank + 3 * m.state + m.conv)
@@ -503,7 +615,10 @@ def spec_param_count(ls: LayerSpec, width: int) -> int:
         n = width * (3 * m.heads * m.vdim + 2 * m.groups * m.state + m.heads) + m.conv * (m.heads * m.vdim + 2 * m.groups * m.state)
     elif m.kind == "attention":
         v = m.dim if m.shared_kv else m.vdim
-        n = width * (m.heads * (m.dim + (1 + m.out_gate) * v) + m.kv_heads * (m.dim + (0 if m.shared_kv else v)))
+        own = 0 if m.kv_from is not None else m.kv_heads * (m.dim + (0 if m.shared_kv else v))
+        n = width * (m.heads * (m.dim + (1 + m.out_gate) * v + m.head_gate) + own)
+    elif m.kind == "general_delta":
+        n = m.heads * m.dim * (6 * width + (m.rank or m.dim)) + (m.rank or m.dim) * width
     else:
         r = m.rank or m.dim
         n = width * (2 * m.kv_heads * m.dim + 2 * m.heads * m.vdim + m.heads + 2 * r) + r * m.heads * (m.dim + m.vdim)

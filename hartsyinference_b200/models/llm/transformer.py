@@ -91,6 +91,7 @@ class LayerWeights:
     sinks: Optional[torch.Tensor] = None              # per-head sink logit in the attention softmax (gpt-oss)
     side_module: Optional[object] = None              # callable (x, tokens) -> [T, W] added after the feed-forward: token input
     side_norm: Optional[torch.Tensor] = None          # RMS norm of what it adds
+    input_conv: Optional[torch.Tensor] = None         # fp32 [sublayers, taps, W]: h + conv(h) is what each sublayer reads
 
 
 def x_is_cuda(x) -> bool:
@@ -137,6 +138,7 @@ class DecoderModel:
         self.alibi_slopes: Optional[torch.Tensor] = None   # [local heads]
         self.kv_cache: Optional[torch.Tensor] = None      # per-layer list for models with per-layer mixers
         self.mixer_state: list = []                       # per layer: (convolution inputs, recurrent state) by slot, or None
+        self.input_state: list = []                       # per layer: last inputs of the convolution ahead of its sublayers by slot, or None
         self.all_reduce: Callable[[torch.Tensor], torch.Tensor] = self.comm.all_reduce
         # hook for the fused GEMM + all-reduce path: (x, weight, residual) -> reduced output
         self.row_parallel_linear: Optional[Callable] = None
@@ -604,21 +606,29 @@ class DecoderModel:
 
     def alloc_state(self, slots: int) -> None:
         """Recurrent state of ``slots`` sequences: per recurrent layer the short convolution's last inputs (in
-        the activation dtype) and the state matrices (fp32)."""
-        self.mixer_state = []
+        the activation dtype; None without one) and the state matrices (fp32); per layer with a convolution ahead of its
+        sublayers the last inputs of that."""
+        zeros = lambda shape, dtype: None if shape is None else torch.zeros(shape, dtype=dtype, device=self.device)
+        self.mixer_state, self.input_state = [], []
         for lw in self.layers:
             st = None
             if hasattr(lw.attn_module, "state_shapes"):
                 conv, rec = lw.attn_module.state_shapes(slots)
-                st = (torch.zeros(conv, dtype=self.dtype, device=self.device), torch.zeros(rec, dtype=torch.float32, device=self.device))
+                st = (zeros(conv, self.dtype), zeros(rec, torch.float32))
             self.mixer_state.append(st)
+            self.input_state.append(zeros(self._input_state_shape(lw, slots), self.dtype))
+
+    @staticmethod
+    def _input_state_shape(lw: LayerWeights, slots: int) -> Optional[tuple]:
+        return None if lw.input_conv is None else (slots, lw.input_conv.shape[1] - 1, lw.input_conv.shape[2])
 
     def state_bytes_per_slot(self) -> int:
         es, n = torch.finfo(self.dtype).bits // 8, 0
         for lw in self.layers:
             if hasattr(lw.attn_module, "state_shapes"):
                 conv, rec = lw.attn_module.state_shapes(1)
-                n += math.prod(conv) * es + math.prod(rec) * 4
+                n += (0 if conv is None else math.prod(conv) * es) + math.prod(rec) * 4
+            n += math.prod(self._input_state_shape(lw, 1) or (0,)) * es
         return n
 
     # ------------------------------------------------------------------------------ forward
@@ -847,7 +857,7 @@ class DecoderModel:
         side(h, tokens) -> x += rms(y), h = norm1'(x) is one more. Without norms ahead of the sublayers (``pre_norm`` off) h is x itself in the activation type. ``capture`` (a list) receives a copy of the stream after every layer."""
         cfg = self.cfg
         kw = dict(dim=cfg.hidden_size, eps=cfg.rms_eps, layernorm=cfg.norm_type == "layernorm", dtype=self.dtype,
-                  plus_one=cfg.norm_plus_one, mult=cfg.residual_multiplier, plain=not cfg.pre_norm)
+                  plus_one=cfg.norm_plus_one, mult=cfg.residual_multiplier, plain=not cfg.pre_norm, groups=cfg.norm_groups)
         if self.embed_norm_w is not None:
             ids, table = batch.tokens, self.embed
             if batch.embeds is not None:
@@ -860,6 +870,8 @@ class DecoderModel:
             x = torch.nn.functional.pad(batch.embeds.float(), (0, self.embed.shape[1] - batch.embeds.shape[1])).contiguous()
         else:
             x = ops.embedding_f32(batch.tokens, self.embed, cfg.embed_scale * cfg.embedding_multiplier, cfg.hidden_size)
+        if cfg.parallel_residual:
+            return self._parallel_layers(batch, x, kw, capture)
         first = self.layers[0].in_norm if self.layers else self.final_norm
         if first is not None or self.embed_norm_w is None:
             h = ops.residual_norm(x, None, None, first, **kw)
@@ -881,6 +893,36 @@ class DecoderModel:
                 h = ops.residual_norm(x, lw.side_module(h, batch.tokens), lw.side_norm, after, **kw)
             if capture is not None:
                 capture.append(x[:, :cfg.hidden_size].clone())
+        return h
+
+    def _parallel_layers(self, batch: ForwardBatch, x: torch.Tensor, kw: dict, capture: Optional[list]) -> torch.Tensor:
+        """Layers whose mixer and feed-forward read one norm, each through its own convolution over time:
+
+            x += m y, h = norm(x), (h + conv1(h), h + conv2(h))            [one launch at decode, two and the state's else]
+            mixer and feed-forward side by side, one output product        -> y
+        """
+        def inputs(y, li: int) -> tuple:
+            lw = self.layers[li]
+            if lw.input_conv is None:
+                h = ops.residual_norm(x, y, None, lw.in_norm, **kw)
+                return h, h
+            state = self.input_state[li]
+            if batch.is_decode:
+                both = ops.residual_norm(x, y, None, lw.in_norm, conv=(lw.input_conv, state, batch.positions, batch.state_slots), **kw)
+            else:
+                both = ops.input_conv(ops.residual_norm(x, y, None, lw.in_norm, **kw), lw.input_conv, state, batch.positions, batch.cu_q,
+                                      batch.state_slots)
+            return both[0], both[-1]
+
+        y = None
+        for li, lw in enumerate(self.layers):
+            h, hf = inputs(y, li)
+            if capture is not None and li:
+                capture.append(x[:, :self.cfg.hidden_size].clone())
+            y = lw.attn_module(h, hf, batch, li, self)
+        h = ops.residual_norm(x, y, None, self.final_norm, **kw)
+        if capture is not None:
+            capture.append(x[:, :self.cfg.hidden_size].clone())
         return h
 
     # most rows whose expert inputs and outputs are held at once
@@ -1064,13 +1106,18 @@ class DecoderModel:
 
     def logits(self, hidden: torch.Tensor) -> torch.Tensor:
         """[rows, H] -> local vocabulary shard logits [rows, vocab_local] (in the activation dtype)."""
-        y = ops.linear_act(hidden, self.lm_head) if self.dtype == torch.float32 else ops.linear(hidden, self.lm_head)
+        y = self._raw_logits(hidden)
         cfg = self.cfg
+        if cfg.mixed_layers:             # fp32, one launch: a cap rounded to bf16 would tie the largest logits
+            return ops.cap_logits(y, cfg.logits_scale, cfg.logit_softcap) if cfg.logits_scale != 1.0 or cfg.logit_softcap > 0 else y
         if cfg.logits_scale != 1.0:
             y = (y.float() * cfg.logits_scale).to(y.dtype)
         if cfg.logit_softcap > 0:
             y = (torch.tanh(y.float() / cfg.logit_softcap) * cfg.logit_softcap).to(y.dtype)
         return y
+
+    def _raw_logits(self, hidden: torch.Tensor) -> torch.Tensor:
+        return ops.linear_act(hidden, self.lm_head) if self.dtype == torch.float32 else ops.linear(hidden, self.lm_head)
 
     def full_logits(self, hidden: torch.Tensor) -> torch.Tensor:
         """Logits over the whole vocabulary (gathers the shards when tensor parallel)."""
@@ -1082,7 +1129,8 @@ class DecoderModel:
     def greedy_tokens(self, hidden: torch.Tensor, out: Optional[torch.Tensor] = None) -> torch.Tensor:
         """argmax over the vocabulary; with TP each rank reduces its shard and the (value, index)
         pairs are combined, so only 8 bytes per row and rank cross the wire."""
-        y = self.logits(hidden)
+        # scale and cap keep the order of the logits: designs with per-layer mixers leave them out here
+        y = self._raw_logits(hidden) if self.cfg.mixed_layers and self.cfg.logits_scale > 0 else self.logits(hidden)
         if self.tp == 1:
             if y.shape[1] > self.cfg.vocab_size:         # rows past the vocabulary pad the weight
                 y = y[:, : self.cfg.vocab_size]

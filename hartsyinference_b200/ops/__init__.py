@@ -54,10 +54,14 @@ from .core import (  # noqa: F401
 from .mixers import (  # noqa: F401
     ChannelScanWeights,
     DeltaWeights,
+    GeneralDeltaWeights,
     HeadScanWeights,
     RoutedRows,
     TanhNorm,
     attn_biased,
+    cap_logits,
+    general_delta,
+    input_conv,
     attn_runs,
     channel_scan,
     delta_mix,

@@ -51,7 +51,13 @@ _SIGNATURES = {
     "b200_moe_dispatch": (i32, [vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, i32, vp]),
     "b200_moe_combine": (i32, [vp, vp, vp, vp, i32, i32, i32, i32, vp]),
     "b200_glu_clamped": (i32, [vp, vp, i64, i32, f32, f32, f32, vp, i32, i32, vp]),
-    "b200_residual_norm": (i32, [vp] * 9 + [i32] * 11 + [f32, f32, i32, vp, f32, vp, vp, i32, vp]),
+    "b200_residual_norm": (i32, [vp] * 9 + [i32] * 11 + [f32, f32, i32, vp, f32, vp, vp, i32, i32, vp, i32, i32, vp, vp, vp, vp]),
+    "b200_input_conv": (i32, [vp] * 7 + [i32] * 5 + [i64, i32, vp]),
+    "b200_cap_logits": (i32, [vp, vp, i64, f32, f32, i32, vp]),
+    "b200_head_norm_store": (i32, [vp] * 8 + [i32, i64] + [i32] * 10 + [f32, i32, vp]),
+    "b200_general_delta_workspace_bytes": (i64, [i32, i32, i32, i32]),
+    "b200_general_delta_launches": (i32, [i32, i32, i32]),
+    "b200_general_delta": (i32, [vp] * 11 + [i32] * 6 + [i64, i64, i64, f32, i32, vp]),
     "b200_side_gate": (i32, [vp] * 4 + [i32] * 6 + [vp]),
     "b200_rope_table": (i32, [vp] * 4 + [i32] * 2 + [vp]),
     "b200_qk_rope_store": (i32, [vp] * 8 + [i32, i64] + [i32] * 11 + [f32, i32, vp]),
@@ -63,9 +69,9 @@ _SIGNATURES = {
     "b200_gated_norm": (i32, [vp] * 4 + [i32] * 5 + [i64] * 3 + [f32, i32, vp]),
     "b200_latent_prep": (i32, [vp] * 6 + [i32, i64] + [i32] * 6 + [f32, vp, i32, i32, i32, vp]),
     "b200_latent_gather": (i32, [vp] * 6 + [i32] * 5 + [vp]),
-    "b200_latent_attn": (i32, [vp] * 6 + [i32] * 7 + [vp, f32, i32, vp]),
-    "b200_head_linear": (i32, [vp] * 6 + [i32] * 4 + [i64, i32, i64, i32, i64, vp, i32, i32, i32, vp]),
-    "b200_attn_runs": (i32, [vp] * 9 + [i32] * 6 + [i64] * 4 + [f32, i32, vp, i32, i64, vp, i32, vp]),
+    "b200_latent_attn": (i32, [vp] * 6 + [i32] * 7 + [vp, f32, i32, vp, vp]),
+    "b200_head_linear": (i32, [vp] * 6 + [i32] * 4 + [i64, i32, i64, i32, i64, vp, i32, i32, i32, i32, vp]),
+    "b200_attn_runs": (i32, [vp] * 9 + [i32] * 6 + [i64] * 4 + [f32, i32, vp, i32, i64, vp, i32, vp, i32, i64, vp]),
     "b200_embedding_f32": (i32, [vp, vp, vp, i32, i32, i32, i32, i32, f32, vp]),
     "b200_linear_f32": (i32, [vp, i32, vp, vp, vp, i32, i32, i32, i64, i64, i64, i32, vp]),
     "b200_router": (i32, [vp, i32, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, i32, f32, i32, i32, vp, vp]),
@@ -73,7 +79,7 @@ _SIGNATURES = {
     "b200_delta_workspace_bytes": (i64, [i32, i32, i32, i32, i32]),
     "b200_delta_launches": (i32, [i32, i32, i32, i32]),
     "b200_delta": (i32, [vp] * 13 + [i32] * 9 + [i64, i32, i64, i32, f32, i32, vp]),
-    "b200_attn_biased": (i32, [vp] * 7 + [i32] * 10 + [vp, f32, f32, i32, i32, vp, i32, vp, vp, i64, i64, i32, i32, vp]),
+    "b200_attn_biased": (i32, [vp] * 7 + [i32] * 10 + [vp, f32, f32, i32, i32, vp, i32, vp, vp, i64, i64, i32, i32, vp, i32, i64, vp]),
     "b200_kv_store": (i32, [vp, vp, vp, vp, vp, i32, i32, i32, i32, i64, i32, vp]),
     "b200_norm": (i32, [vp, vp, vp, vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, f32, i32, i32, i32, vp]),
     "b200_quant_fp8": (i32, [vp, vp, vp, i32, i32, i64, i32, vp]),

@@ -11,7 +11,12 @@ import torch
 from . import _native as N
 from . import reference as R
 
-_ACT = {None: 0, "none": 0, "gelu_tanh": 1, "silu": 2, "relu2": 3}
+_ACT = {None: 0, "none": 0, "gelu_tanh": 1, "silu": 2, "relu2": 3, "tanh": 4}
+
+
+def act_code(act: Optional[str], act_from: int) -> int:
+    """Activation argument of a product: the low byte names the function, the rest the first feature it applies to."""
+    return _ACT[act] | act_from << 8
 
 
 def fp8_mx() -> bool:
@@ -270,8 +275,9 @@ def _scale_ptrs(x, w: LinearWeight):
 
 def linear(x, w: LinearWeight, act: Optional[str] = None, gate: Optional[torch.Tensor] = None,
            residual: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None,
-           splits: Optional[int] = None, defer: bool = False):
-    """y = residual + gate * act(x @ W^T + bias), bf16 output [M, N].
+           splits: Optional[int] = None, defer: bool = False, act_from: int = 0):
+    """y = residual + gate * act(x @ W^T + bias), bf16 output [M, N]. ``act`` applies to the output features from
+    ``act_from`` on.
 
     ``x`` is a bf16 tensor [M, K] or an :class:`Fp8Act`. With an fp8 weight a bf16 ``x`` is
     quantised on the fly (1x128 groups). ``gate`` is a per-output-feature vector [N].
@@ -294,7 +300,7 @@ def linear(x, w: LinearWeight, act: Optional[str] = None, gate: Optional[torch.T
             q, s = R.quant_fp8_act(x, pow2=fp8_mx())
             y = R.linear(q, w.weight, w.scale, s, w.bias, act, gate, residual)
         else:
-            y = R.linear(x, w.host_f32(), None, None, w.bias, act, gate, residual)
+            y = R.linear(x, w.host_f32(), None, None, w.bias, act, gate, residual, act_from=act_from)
         if out is not None:
             out.copy_(y)
             return out
@@ -328,7 +334,7 @@ def linear(x, w: LinearWeight, act: Optional[str] = None, gate: Optional[torch.T
     rc = L.b200_gemm(xd.data_ptr(), w.weight.data_ptr(), out.data_ptr(), m, n, k,
                      xd.stride(0), w.weight.stride(0), out.stride(0), _gemm_dtype(w),
                      xs_ptr, ws_ptr,
-                     N.ptr(w.bias), N.ptr(gate), N.ptr(residual), _ACT[act], 0 if splits is None else splits,
+                     N.ptr(w.bias), N.ptr(gate), N.ptr(residual), act_code(act, act_from), 0 if splits is None else splits,
                      ws.data_ptr(), ws.numel(), st.status.data_ptr(), N.stream())
     N.check(rc, "b200_gemm")
     return out

@@ -15,7 +15,7 @@ import torch
 
 from . import _native as N
 from . import reference as R
-from .core import _ACT, LinearWeight, linear
+from .core import _ACT, LinearWeight, act_code, linear
 
 
 def _f32(t: torch.Tensor) -> int:
@@ -23,19 +23,24 @@ def _f32(t: torch.Tensor) -> int:
     return 1 if t.dtype == torch.float32 else 0
 
 
-def linear_act(x: torch.Tensor, w: LinearWeight, act: Optional[str] = None) -> torch.Tensor:
+def linear_act(x: torch.Tensor, w: LinearWeight, act: Optional[str] = None, act_from: int = 0,
+               out: Optional[torch.Tensor] = None) -> torch.Tensor:
     """act(x @ W^T (+ bias)) in the dtype of ``x``: bf16 through the tensor-core GEMM, fp32 through 32-bit
-    FMA tiles (the weight itself is bf16 in both). ``act``: None or "relu2" (relu squared)."""
+    FMA tiles (the weight itself is bf16 in both). ``act``: None, "relu2" (relu squared) or "tanh", for the output features
+    from ``act_from`` on. ``out``: [M, N] of any row pitch."""
     if x.dtype != torch.float32:
-        return linear(x, w, act)
+        return linear(x, w, act, act_from=act_from, out=out)
     if not x.is_cuda:
-        return R.linear(x, w.host_f32(), bias=w.bias, act=act, out_dtype=torch.float32)
+        y = R.linear(x, w.host_f32(), bias=w.bias, act=act, out_dtype=torch.float32, act_from=act_from)
+        return y if out is None else out.copy_(y)
     m, k = x.shape
     n = w.weight.shape[0]
     assert w.weight.shape[1] == k and x.stride(1) == 1 and w.weight.stride(1) == 1 and not w.is_fp8
-    out = torch.empty(m, n, dtype=torch.float32, device=x.device)
+    if out is None:
+        out = torch.empty(m, n, dtype=torch.float32, device=x.device)
+    assert out.shape == (m, n) and out.stride(1) == 1 and out.dtype == torch.float32
     N.check(N.lib().b200_linear_f32(x.data_ptr(), 1, w.weight.data_ptr(), N.ptr(w.bias), out.data_ptr(), m, n, k, x.stride(0),
-                                    w.weight.stride(0), n, _ACT[act], N.stream()), "b200_linear_f32")
+                                    w.weight.stride(0), out.stride(0), act_code(act, act_from), N.stream()), "b200_linear_f32")
     return out
 
 
@@ -95,10 +100,12 @@ class TanhNorm:
 
 def residual_norm(x: torch.Tensor, y, w_b: Optional[torch.Tensor], w_n, *, dim: int, eps: float,
                   layernorm: bool, dtype: torch.dtype, out: Optional[torch.Tensor] = None, plus_one: bool = False, mult: float = 1.0,
-                  plain: bool = False) -> Optional[torch.Tensor]:
+                  plain: bool = False, groups: int = 1, conv: Optional[tuple] = None) -> Optional[torch.Tensor]:
     """In place on the fp32 stream ``x`` [T, ld]: ``x += mult * norm(y) * w_b`` (``y`` a tensor, :class:`RoutedRows`
     or None), then returns ``norm(x) * w_n`` in ``dtype``, or :class:`TanhNorm` ``w_n`` of x (without ``w_n``: the
-    stream itself if ``plain``, else None). ``plus_one``: the norms multiply by 1 + w. One launch."""
+    stream itself if ``plain``, else None). ``plus_one``: the norms multiply by 1 + w. ``groups``: the norm on x is an RMS norm
+    of that many equal parts, each on its own. ``conv`` = (w, state, positions, slots), one token per sequence: the result goes
+    through :func:`input_conv` and is [n, T, ld]. One launch."""
     rows, ld = x.shape
     routed = y if isinstance(y, RoutedRows) else None
     tanh = w_n if isinstance(w_n, TanhNorm) else None
@@ -115,12 +122,23 @@ def residual_norm(x: torch.Tensor, y, w_b: Optional[torch.Tensor], w_n, *, dim: 
         h = torch.zeros(rows, ld, dtype=dtype) if out is None else out
         if tanh is not None:
             h[:, :dim] = (torch.tanh(tanh.alpha * x[:, :dim]) * tanh.weight.float() + tanh.bias.float()).to(dtype)
+        elif w_n is not None and groups > 1:
+            part = x[:, :dim].reshape(rows * groups, dim // groups)
+            part = part * torch.rsqrt(part.pow(2).mean(-1, keepdim=True) + eps)
+            h[:, :dim] = (part.reshape(rows, dim) * (w_n.float() + 1 if plus_one else w_n.float())).to(dtype)
         else:
             h[:, :dim] = (nrm(x, w_n) if w_n is not None else x[:, :dim]).to(dtype)
-        return h
+        return h if conv is None else R.input_conv(h, conv[0], conv[1], conv[2], None, conv[3])
     assert x.dtype == torch.float32 and x.stride(1) == 1
     h = None
-    if w_n is not None or plain:
+    if conv is not None:
+        cw, cst, positions, slots = conv
+        n, taps = cw.shape[:2]
+        assert out is None and cw.dtype == torch.float32 and cw.is_contiguous() and cw.shape[2] == ld and cst.dtype == dtype
+        assert cst.is_contiguous() and cst.shape[1:] == (taps - 1, ld) and slots.numel() == rows
+        assert slots.dtype == torch.int32 and positions.dtype == torch.int32
+        h = torch.empty(n, rows, ld, dtype=dtype, device=x.device)
+    elif w_n is not None or plain:
         h = torch.empty(rows, ld, dtype=dtype, device=x.device) if out is None else out
         assert h.dtype == dtype and h.is_contiguous()
     yt = routed.rows if routed is not None else y
@@ -136,9 +154,41 @@ def residual_norm(x: torch.Tensor, y, w_b: Optional[torch.Tensor], w_n, *, dim: 
         routed.ids.shape[1] if routed is not None else 0, routed.experts if routed is not None else 0, int(layernorm),
         int(plus_one), int(plain), float(eps), float(mult), 1 if dtype == torch.float32 else 0,
         N.ptr(None if tanh is None else tanh.bias), 0.0 if tanh is None else float(tanh.alpha), N.ptr(extra),
-        N.ptr(routed.extra_weight) if extra is not None else None, extra.stride(0) if extra is not None else 0, N.stream())
+        N.ptr(routed.extra_weight) if extra is not None else None, extra.stride(0) if extra is not None else 0, int(groups),
+        *((cw.data_ptr(), n, taps, cst.data_ptr(), positions.data_ptr(), slots.data_ptr()) if conv is not None else (None, 0, 0, None, None, None)),
+        N.stream())
     N.check(rc, "b200_residual_norm")
     return h
+
+
+def input_conv(h: torch.Tensor, w: torch.Tensor, state: torch.Tensor, positions: torch.Tensor, cu_q: Optional[torch.Tensor],
+               slots: torch.Tensor) -> torch.Tensor:
+    """``h + conv_i(h)`` for every i: [n, T, C] from ``h`` [T, C] (any row pitch) and ``w`` fp32 [n, taps, C] (last row: the
+    current token), causal over time per channel. ``state`` [slots, taps - 1, C] holds the inputs before each sequence's
+    portion and is updated in place; a sequence whose first position is 0 starts from zeros, slot -1 is not stored."""
+    t, c = h.shape
+    if not h.is_cuda:
+        return R.input_conv(h, w, state, positions, cu_q, slots)
+    n, taps, _ = w.shape
+    assert h.stride(1) == 1 and w.dtype == torch.float32 and w.is_contiguous() and w.shape[2] == c and state.dtype == h.dtype
+    assert state.is_contiguous() and state.shape[1:] == (taps - 1, c) and slots.dtype == torch.int32 and positions.dtype == torch.int32
+    out = torch.empty(n, t, c, dtype=h.dtype, device=h.device)
+    N.check(N.lib().b200_input_conv(h.data_ptr(), w.data_ptr(), state.data_ptr(), positions.data_ptr(), N.ptr(cu_q), slots.data_ptr(),
+                                    out.data_ptr(), t, slots.numel(), c, taps, n, h.stride(0), _f32(h), N.stream()),
+            "b200_input_conv", 2 if cu_q is not None and taps > 1 else 1)
+    return out
+
+
+def cap_logits(y: torch.Tensor, scale: float, cap: float) -> torch.Tensor:
+    """fp32 ``cap * tanh(y * scale / cap)`` (``cap`` 0: ``y * scale``)."""
+    if not y.is_cuda:
+        z = y.float() * scale
+        return cap * torch.tanh(z / cap) if cap > 0 else z
+    rows, n = y.shape
+    assert y.is_contiguous()
+    out = torch.empty(rows, n, dtype=torch.float32, device=y.device)
+    N.check(N.lib().b200_cap_logits(y.data_ptr(), out.data_ptr(), y.numel(), float(scale), float(cap), _f32(y), N.stream()), "b200_cap_logits")
+    return out
 
 
 def side_gate(u: torch.Tensor, ids: torch.Tensor, table: torch.Tensor) -> torch.Tensor:
@@ -213,6 +263,12 @@ def pair_linear_f32(x: torch.Tensor, w: LinearWeight, ids: torch.Tensor, experts
     return out
 
 
+def _gate_of(gate: torch.Tensor, heads: int, dv: int, head_gate: bool) -> torch.Tensor:
+    """fp32 sigmoid of gate logits, one per value or (``head_gate``) the first ``heads`` columns, one per head."""
+    g = torch.sigmoid(gate.float())
+    return g[:, :heads].repeat_interleave(dv, 1) if head_gate else g
+
+
 def kv_store(k: torch.Tensor, k_cache: torch.Tensor, slots: torch.Tensor, v: Optional[torch.Tensor] = None,
              v_cache: Optional[torch.Tensor] = None) -> None:
     """Write key (and value) rows [T, hkv * d] (any row pitch) into pages [pages, hkv, page, d]; slot =
@@ -237,33 +293,36 @@ def attn_biased(q: torch.Tensor, k_cache: torch.Tensor, v_cache: Optional[torch.
                 kv_lens: torch.Tensor, cu_q: Optional[torch.Tensor], *, heads: int, max_q_len: int = 1, max_kv_len: int = 0,
                 scale: float = 1.0, softcap: float = 0.0, window: int = 0, dist_bias: Optional[torch.Tensor] = None,
                 sinks: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, keep_first: int = 0,
-                v_dim: int = 0) -> torch.Tensor:
+                v_dim: int = 0, slopes: Optional[torch.Tensor] = None, head_gate: bool = False,
+                out: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal attention over pages (with a ``window``: over the last ``window`` tokens and the ``keep_first`` first
     ones of the sequence) with, each optional, a per-head bias by key distance (``dist_bias``
-    [heads, n], its last entry also stands for longer distances), a sink score per head that only enters
-    the softmax denominator, and a sigmoid ``gate`` [T, heads * dv] on the output. ``q`` [T, heads * d] (any
+    [heads, n], its last entry also stands for longer distances) or linear in it (``slopes`` fp32 [heads], taken off), a sink
+    score per head that only enters the softmax denominator, and a sigmoid ``gate`` [T, heads * dv] (``head_gate``: one column
+    per head) on the output. ``q`` [T, heads * d] (any
     row pitch); ``v_cache`` None: the values are the keys (their first ``v_dim`` columns when given); ``cu_q`` None:
-    one query token per sequence. Returns [T, heads * dv]."""
+    one query token per sequence. Returns [T, heads * dv] (``out`` when given, any row pitch)."""
     t = q.shape[0]
     _, hkv, page, d = k_cache.shape
     dv = v_cache.shape[3] if v_cache is not None else v_dim or d
     seqs = kv_lens.numel()
     if not q.is_cuda:
-        out = torch.empty(t, heads * dv, dtype=q.dtype)
+        out = torch.empty(t, heads * dv, dtype=q.dtype) if out is None else out
         bounds = list(range(seqs + 1)) if cu_q is None else cu_q.tolist()
         for i in range(seqs):
             a, b, ln = bounds[i], bounds[i + 1], int(kv_lens[i])
             kk = R.gather_paged(k_cache, block_table[i], ln)
             vv = kk[..., :dv] if v_cache is None else R.gather_paged(v_cache, block_table[i], ln)
             o = R.attention(q[a:b].reshape(b - a, heads, d), kk, vv, causal=True, scale=scale, softcap=softcap, window=window,
-                            sinks=sinks, dist_bias=dist_bias, keep_first=keep_first).reshape(b - a, heads * dv)
+                            sinks=sinks, dist_bias=dist_bias, keep_first=keep_first, slopes=slopes).reshape(b - a, heads * dv)
             if gate is not None:
-                o = o * torch.sigmoid(gate[a:b].float())
+                o = o * _gate_of(gate[a:b], heads, dv, head_gate)
             out[a:b] = o.to(q.dtype)
         return out
     assert block_table.dtype == torch.int32 and kv_lens.dtype == torch.int32 and q.stride(1) == 1
     assert dist_bias is None or (dist_bias.dtype == torch.float32 and dist_bias.is_contiguous())
     assert gate is None or gate.stride(1) == 1
+    assert slopes is None or (slopes.dtype == torch.float32 and dist_bias is None)
     L = N.lib()
     f32 = _f32(q)
     exact = 1 if f32 or max(d, dv) > 128 or (v_cache is None and dv != d) or page > 64 or (cu_q is None and heads // hkv > 16) else 0
@@ -276,12 +335,15 @@ def attn_biased(q: torch.Tensor, k_cache: torch.Tensor, v_cache: Optional[torch.
         splits = L.b200_attn_decode_pick_splits(seqs, hkv, mk)
         if splits > 1:
             ws = N.state(q.device).scratch(L.b200_attn_decode_workspace_bytes(seqs, heads, dd, splits)).data_ptr()
-    out = torch.empty(t, heads * dv, dtype=q.dtype, device=q.device)
+    if out is None:
+        out = torch.empty(t, heads * dv, dtype=q.dtype, device=q.device)
+    assert out.shape == (t, heads * dv) and out.stride(1) == 1 and out.dtype == q.dtype
     rc = L.b200_attn_biased(q.data_ptr(), k_cache.data_ptr(), N.ptr(v_cache), out.data_ptr(), block_table.data_ptr(),
                             kv_lens.data_ptr(), N.ptr(cu_q), t, seqs, max_q_len, heads, hkv, d, dv, page, block_table.shape[1],
                             splits, ws, float(scale), float(softcap), int(window), int(keep_first), N.ptr(dist_bias),
                             dist_bias.shape[1] if dist_bias is not None else 0, N.ptr(sinks), N.ptr(gate),
-                            gate.stride(0) if gate is not None else 0, q.stride(0), exact, f32, N.stream())
+                            gate.stride(0) if gate is not None else 0, q.stride(0), exact, f32, N.ptr(slopes), int(head_gate), out.stride(0),
+                            N.stream())
     N.check(rc, "b200_attn_biased", 2 if splits > 1 else 1)
     return out
 
@@ -300,11 +362,14 @@ def rope_table(positions: torch.Tensor, hi: torch.Tensor, lo: torch.Tensor) -> t
 
 def qk_rope_store(p: torch.Tensor, heads: int, k_cache: torch.Tensor, v_cache: torch.Tensor, slots: torch.Tensor, *,
                   table: Optional[torch.Tensor] = None, interleaved: bool = False, q_norm: Optional[torch.Tensor] = None,
-                  k_norm: Optional[torch.Tensor] = None, d_true: int = 0, eps: float = 0.0) -> torch.Tensor:
+                  k_norm: Optional[torch.Tensor] = None, d_true: int = 0, eps: float = 0.0, per_head: bool = False,
+                  store: bool = True) -> torch.Tensor:
     """From a projection ``p`` [T, q | k | v] (any row pitch) to attention's inputs: RMS norm of q and of k over all their
-    heads at once (``q_norm`` [heads * d], ``k_norm`` [hkv * d], or None), rotation of the first values of every q and k head
+    heads at once (``q_norm`` [heads * d], ``k_norm`` [hkv * d], or None) or, ``per_head``, of each head on its own (weights
+    [d]), rotation of the first values of every q and k head
     by ``table`` (:func:`rope_table`, or None), k and v into the pages [pages, hkv, page, d] and [pages, hkv, page, dv].
-    ``d_true``: the model's head size where heads are padded with zeros. Returns q [T, heads * d]."""
+    ``d_true``: the model's head size where heads are padded with zeros. ``store`` off: q only, ``p`` has no k and v.
+    Returns q [T, heads * d]."""
     _, hkv, page, d = k_cache.shape
     dv = v_cache.shape[3]
     t, nq, nk = p.shape[0], heads * d, hkv * d
@@ -312,16 +377,28 @@ def qk_rope_store(p: torch.Tensor, heads: int, k_cache: torch.Tensor, v_cache: t
     if not p.is_cuda:
         def part(x, w, n):
             x = x.float()
-            if w is not None:
+            if w is not None and not per_head:
                 x = x / torch.sqrt((x * x).sum(-1, keepdim=True) / (n * dt) + eps) * w.float()
             x = x.reshape(t, n, d)
+            if w is not None and per_head:
+                x = x / torch.sqrt((x * x).sum(-1, keepdim=True) / dt + eps) * w.float()
             return (x if table is None else R.turn(x, table, interleaved)).reshape(t, n * d).to(p.dtype)
-        kv_store(part(p[:, nq:nq + nk], k_norm, hkv), k_cache, slots)
-        kv_store(p[:, nq + nk:nq + nk + hkv * dv], v_cache, slots)
+        if store:
+            kv_store(part(p[:, nq:nq + nk], k_norm, hkv), k_cache, slots)
+            kv_store(p[:, nq + nk:nq + nk + hkv * dv], v_cache, slots)
         return part(p[:, :nq], q_norm, heads)
     assert p.stride(1) == 1 and slots.dtype == torch.int64 and k_cache.dtype == v_cache.dtype == p.dtype
-    assert (q_norm is None) == (k_norm is None) and (q_norm is None or (q_norm.numel() == nq and k_norm.numel() == nk))
+    if per_head:
+        assert q_norm.numel() == d and (not store or k_norm.numel() == d)
+    else:
+        assert store and (q_norm is None) == (k_norm is None) and (q_norm is None or (q_norm.numel() == nq and k_norm.numel() == nk))
     q = torch.empty(t, nq, dtype=p.dtype, device=p.device)
+    if per_head:
+        N.check(N.lib().b200_head_norm_store(p.data_ptr(), q_norm.data_ptr(), N.ptr(k_norm if store else None), N.ptr(table), q.data_ptr(),
+                                             k_cache.data_ptr(), v_cache.data_ptr(), slots.data_ptr(), t, p.stride(0), heads, hkv if store else 0,
+                                             d, dv, nq, nq + nk, page, 0 if table is None else 2 * table.shape[1], int(interleaved), dt,
+                                             float(eps), _f32(p), N.stream()), "b200_head_norm_store")
+        return q
     N.check(N.lib().b200_qk_rope_store(p.data_ptr(), N.ptr(q_norm), N.ptr(k_norm), N.ptr(table), q.data_ptr(), k_cache.data_ptr(),
                                        v_cache.data_ptr(), slots.data_ptr(), t, p.stride(0), heads, hkv, d, dv, nq, nq + nk, page,
                                        0 if table is None else 2 * table.shape[1], int(interleaved), heads * dt, hkv * dt, float(eps),
@@ -371,6 +448,46 @@ def delta_mix(proj: torch.Tensor, z: torch.Tensor, w: DeltaWeights, conv_state: 
                       slots.data_ptr(), ws.data_ptr(), out.data_ptr(), t, seqs, w.heads, w.kv_heads, w.dk, w.dv, w.dk_true,
                       w.dv_true, taps, proj.stride(0), b_off, z.stride(0), w.heads * w.dk, float(w.eps), _f32(proj), N.stream())
     N.check(rc, "b200_delta", L.b200_delta_launches(1 if cu_q is None else 0, taps, w.dk, w.dv))
+    return out
+
+
+@dataclass
+class GeneralDeltaWeights:
+    """Constants of one general delta mixer. ``dk`` / ``dv`` are the head sizes as laid out (padded with zero channels),
+    ``d_true`` the model's."""
+    decay_bias: torch.Tensor   # fp32 [heads * dk]
+    rate_bias: torch.Tensor    # fp32 [heads * dk]
+    norm: torch.Tensor         # bf16 [heads * dv]
+    heads: int
+    dk: int
+    dv: int
+    d_true: int
+    eps: float
+
+
+def general_delta(proj: torch.Tensor, z: torch.Tensor, w: GeneralDeltaWeights, state: torch.Tensor, positions: torch.Tensor,
+                  cu_q: Optional[torch.Tensor], slots: torch.Tensor, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Per head ``S = diag(e) S - (a u)(u^T S) + k v^T``, ``y = norm(S^T r) * weight * sigmoid(gate)`` with the unit key
+    ``u = k / sqrt(k^2 + 1e-6)``, the decay ``e = exp(-exp(-1/2) sigmoid(z + decay_bias))`` and the removal rate
+    ``a = sigmoid(logit + rate_bias)``, both per key channel. ``proj`` [T, ld] = r | k | a logits [heads * dk] | v | gate logits
+    [heads * dv]; ``z`` [T, heads * dk] decay logits. ``state`` fp32 [slots, heads, dk, dv] is updated in place; a sequence
+    whose first position is 0 starts from zeros, slot -1 is not stored. Returns [T, heads * dv] (``out`` when given)."""
+    t = proj.shape[0]
+    if not proj.is_cuda:
+        y = R.general_delta(proj, z, w, state, positions, cu_q, slots)
+        return y if out is None else out.copy_(y)
+    assert proj.dtype == z.dtype and state.dtype == torch.float32 and state.is_contiguous()
+    assert slots.dtype == torch.int32 and positions.dtype == torch.int32 and proj.stride(1) == 1 and z.stride(1) == 1
+    L = N.lib()
+    if out is None:
+        out = torch.empty(t, w.heads * w.dv, dtype=proj.dtype, device=proj.device)
+    assert out.shape == (t, w.heads * w.dv) and out.stride(1) == 1 and out.dtype == proj.dtype
+    decode = cu_q is None
+    ws = torch.empty(L.b200_general_delta_workspace_bytes(t, w.heads, w.dk, w.dv), dtype=torch.uint8, device=proj.device)
+    rc = L.b200_general_delta(proj.data_ptr(), z.data_ptr(), w.decay_bias.data_ptr(), w.rate_bias.data_ptr(), w.norm.data_ptr(), state.data_ptr(),
+                              positions.data_ptr(), N.ptr(cu_q), slots.data_ptr(), ws.data_ptr(), out.data_ptr(), t, slots.numel(), w.heads, w.dk,
+                              w.dv, w.d_true, proj.stride(0), z.stride(0), out.stride(0), float(w.eps), _f32(proj), N.stream())
+    N.check(rc, "b200_general_delta", L.b200_general_delta_launches(int(decode), w.dk, w.dv))
     return out
 
 
@@ -536,9 +653,10 @@ def latent_prep(x: torch.Tensor, q_off: int, q_dim: int, wq: torch.Tensor, kv_of
 
 def head_linear(x: torch.Tensor, w: LinearWeight, heads: int, *, gate: Optional[torch.Tensor] = None,
                 in_rows: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None,
-                out_rows: Optional[torch.Tensor] = None, tail: int = 0, table: Optional[torch.Tensor] = None) -> torch.Tensor:
+                out_rows: Optional[torch.Tensor] = None, tail: int = 0, table: Optional[torch.Tensor] = None,
+                head_gate: bool = False) -> torch.Tensor:
     """One product per head: ``out[r, h] = W[h] x[r, h]`` with ``w`` stacked [heads * n, k], ``x`` [rows, heads * k] and
-    ``out`` [rows, heads * n], optionally times ``sigmoid(gate)``. ``in_rows`` / ``out_rows`` (int32) select the rows of
+    ``out`` [rows, heads * n], optionally times ``sigmoid(gate)`` (``head_gate``: one column per head). ``in_rows`` / ``out_rows`` (int32) select the rows of
     ``x`` and of ``out`` and ``gate`` that the product's rows stand for. ``tail`` > 0: heads of ``x`` are k + tail wide and
     heads of ``out`` n + tail; the tail is turned by the row of x in ``table`` (pairs of neighbours; zero past it)."""
     n, k = w.weight.shape[0] // heads, w.weight.shape[1]
@@ -555,7 +673,7 @@ def head_linear(x: torch.Tensor, w: LinearWeight, heads: int, *, gate: Optional[
         y = y.reshape(rows, heads * (n + tail))
         at = slice(None) if out_rows is None else out_rows.long()
         if gate is not None:
-            y = y * torch.sigmoid(gate[at].float())
+            y = y * _gate_of(gate[at], heads, n, head_gate)
         out[at] = y.to(out.dtype)
         return out
     assert x.stride(1) == 1 and out.stride(1) == 1 and w.weight.is_contiguous() and out.dtype == x.dtype
@@ -563,16 +681,18 @@ def head_linear(x: torch.Tensor, w: LinearWeight, heads: int, *, gate: Optional[
     assert all(i is None or i.dtype == torch.int32 for i in (in_rows, out_rows)) and (tail == 0 or gate is None)
     N.check(N.lib().b200_head_linear(x.data_ptr(), w.weight.data_ptr(), out.data_ptr(), N.ptr(gate), N.ptr(in_rows), N.ptr(out_rows), rows,
                                      heads, n, k, x.stride(0), k + tail, out.stride(0), n + tail, gate.stride(0) if gate is not None else 0,
-                                     N.ptr(table if tail else None), 2 * table.shape[1] if tail else 0, tail, _f32(x), N.stream()),
+                                     N.ptr(table if tail else None), 2 * table.shape[1] if tail else 0, tail, int(head_gate), _f32(x), N.stream()),
             "b200_head_linear")
     return out
 
 
 def latent_attn(q: torch.Tensor, cache: torch.Tensor, block_table: torch.Tensor, kv_lens: torch.Tensor, heads: int, scale: float,
-                row_seq: Optional[torch.Tensor] = None, max_kv_len: int = 0, v_dim: int = 0, window: int = 0) -> torch.Tensor:
+                row_seq: Optional[torch.Tensor] = None, max_kv_len: int = 0, v_dim: int = 0, window: int = 0,
+                sinks: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Attention of queries in latent space [rows, heads * row] over cached rows [pages, 1, page, row], which are keys of every
     head and, in their first ``v_dim`` values (0: all), its values: row r sees the first ``kv_lens[r]`` tokens of block-table
-    row ``row_seq[r]`` (r when None), with a ``window`` the last ``window`` of them. bf16 rows of at most 512 + 64 values run on
+    row ``row_seq[r]`` (r when None), with a ``window`` the last ``window`` of them; ``sinks`` fp32 [heads] are scores that only enter
+    the denominators. bf16 rows of at most 512 + 64 values run on
     the tensor cores, fp32 and wider ones as plain 32-bit arithmetic. Returns [rows, heads * v_dim]."""
     rows, row, page = q.shape[0], cache.shape[3], cache.shape[2]
     lat = v_dim or row
@@ -580,7 +700,7 @@ def latent_attn(q: torch.Tensor, cache: torch.Tensor, block_table: torch.Tensor,
     if not q.is_cuda or q.dtype == torch.float32 or lat > 512 or row > 576:
         if row_seq is not None:
             table = block_table[row_seq.long()].contiguous()
-        return attn_biased(q, cache, None, table, kv_lens, None, heads=heads, scale=scale, window=window, v_dim=lat)
+        return attn_biased(q, cache, None, table, kv_lens, None, heads=heads, scale=scale, window=window, v_dim=lat, sinks=sinks)
     assert q.is_contiguous() and cache.is_contiguous() and kv_lens.dtype == torch.int32 and kv_lens.numel() == rows
     assert block_table.dtype == torch.int32 and (row_seq is None or row_seq.dtype == torch.int32)
     L = N.lib()
@@ -598,7 +718,7 @@ def latent_attn(q: torch.Tensor, cache: torch.Tensor, block_table: torch.Tensor,
         tab = table if row_seq is not None else table[a:b]
         rc = L.b200_latent_attn(q[a:b].data_ptr(), cache.data_ptr(), out[a:b].data_ptr(), tab.data_ptr(), kv_lens[a:b].data_ptr(),
                                 N.ptr(None if row_seq is None else row_seq[a:b]), b - a, heads, row, lat, page, table.stride(0), splits,
-                                N.ptr(ws), float(scale), int(window), N.stream())
+                                N.ptr(ws), float(scale), int(window), N.ptr(sinks), N.stream())
         N.check(rc, "b200_latent_attn", 2 if splits > 1 else 1)
     return out
 
@@ -623,20 +743,22 @@ def latent_gather(cache: torch.Tensor, block_table: torch.Tensor, seq_ids: torch
 def attn_runs(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, out: torch.Tensor, q_start: torch.Tensor, q_lens: torch.Tensor,
               kv_start: torch.Tensor, kv_lens: torch.Tensor, *, heads: int, max_q_len: int, scale: float,
               gate: Optional[torch.Tensor] = None, window: int = 0, k_shared: Optional[torch.Tensor] = None,
-              table: Optional[torch.Tensor] = None) -> None:
+              table: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None, head_gate: bool = False) -> None:
     """Causal attention of runs of query rows over contiguous keys and values of their contexts: run s is rows
     ``q_start[s]`` .. + ``q_lens[s]`` of ``q`` [T, heads * d], its context rows ``kv_start[s]`` .. + ``kv_lens[s]`` of ``k``
     [.., heads * d] and ``v`` [.., heads * dv]; the last key belongs to the last query, and with a ``window`` a query sees the
     last ``window`` keys up to its own. ``k_shared`` [.., n]: the last n values of every key head, the same for all heads
     (heads of ``k`` are then d - n wide), the query's side of which is turned by ``table`` [T, pairs, 2]. Rows of the runs are
-    written to ``out`` [T, heads * dv], times ``sigmoid(gate)``. bf16, d up to 192 and dv up to 128."""
+    written to ``out`` [T, heads * dv] (any row pitch), times ``sigmoid(gate)`` (``head_gate``: one column per head); ``sinks``
+    fp32 [heads] are scores that only enter the denominators. bf16, d up to 192 and dv up to 128."""
     own, dv = k.shape[1] // heads, v.shape[1] // heads
     d = own + (0 if k_shared is None else k_shared.shape[1])
-    assert q.is_cuda and q.dtype == torch.bfloat16 and out.is_contiguous() and q.stride(1) == k.stride(1) == v.stride(1) == 1
+    assert q.is_cuda and q.dtype == torch.bfloat16 and out.stride(1) == q.stride(1) == k.stride(1) == v.stride(1) == 1
     assert q.shape[1] == heads * d and out.shape[1] == heads * dv and (gate is None or gate.stride(1) == 1)
     assert k_shared is None or (k_shared.stride(1) == 1 and k_shared.dtype == q.dtype)
     N.check(N.lib().b200_attn_runs(q.data_ptr(), k.data_ptr(), v.data_ptr(), out.data_ptr(), N.ptr(gate), q_start.data_ptr(),
                                    q_lens.data_ptr(), kv_start.data_ptr(), kv_lens.data_ptr(), q_lens.numel(), max_q_len, heads, heads, d,
                                    dv, q.stride(0), k.stride(0), v.stride(0), gate.stride(0) if gate is not None else 0, float(scale),
                                    int(window), N.ptr(k_shared), own, k_shared.stride(0) if k_shared is not None else 0, N.ptr(table),
-                                   table.shape[1] if table is not None else 0, N.stream()), "b200_attn_runs")
+                                   table.shape[1] if table is not None else 0, N.ptr(sinks), int(head_gate), out.stride(0), N.stream()),
+            "b200_attn_runs")

@@ -100,19 +100,24 @@ def gelu_tanh(x: torch.Tensor) -> torch.Tensor:
 def linear(x: torch.Tensor, w: torch.Tensor, w_scale: Optional[torch.Tensor] = None,
            x_scale: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None,
            act: Optional[str] = None, gate: Optional[torch.Tensor] = None,
-           residual: Optional[torch.Tensor] = None, out_dtype: torch.dtype = torch.bfloat16) -> torch.Tensor:
-    """y = residual + gate * act(x @ w^T + bias); fp8 operands are dequantised first."""
+           residual: Optional[torch.Tensor] = None, out_dtype: torch.dtype = torch.bfloat16, act_from: int = 0) -> torch.Tensor:
+    """y = residual + gate * act(x @ w^T + bias); fp8 operands are dequantised first. ``act`` applies from feature ``act_from`` on."""
     xf = dequant_fp8_act(x, x_scale) if x_scale is not None else x.float()
     wf = dequant_fp8_weight(w, w_scale) if w_scale is not None else w.float()
     y = xf @ wf.t()
     if bias is not None:
         y = y + bias.float()
+    plain, y = y[..., :act_from], y[..., act_from:]
     if act == "gelu_tanh":
         y = gelu_tanh(y)
     elif act == "silu":
         y = torch.nn.functional.silu(y)
     elif act == "relu2":
         y = torch.relu(y) ** 2
+    elif act == "tanh":
+        y = torch.tanh(y)
+    if act_from:
+        y = torch.cat([plain, y], -1)
     if gate is not None:
         y = y * gate.float()
     if residual is not None:
@@ -203,6 +208,52 @@ def delta_mix(proj, z, w, conv_state, state, positions, cu_q, slots, b_off) -> t
         gate = torch.sigmoid(z[a:b, h * dk:].float()).reshape(-1, h, dv)
         o = o * torch.rsqrt(o.pow(2).sum(-1, keepdim=True) / w.dv_true + w.eps) * w.norm.float() * gate
         out[a:b] = o.reshape(b - a, h * dv).to(proj.dtype)
+    return out
+
+
+def general_delta(proj, z, w, state, positions, cu_q, slots) -> torch.Tensor:
+    """Delta rule with a removal rate per key channel, token by token (see ``ops.general_delta``)."""
+    t, h, dk, dv = proj.shape[0], w.heads, w.dk, w.dv
+    n, m = h * dk, h * dv
+    bounds = list(range(slots.numel() + 1)) if cu_q is None else cu_q.tolist()
+    p = proj[:, :3 * n + 2 * m].float()
+    r, k = (p[:, i * n:(i + 1) * n].reshape(t, h, dk) for i in range(2))
+    a = torch.sigmoid(p[:, 2 * n:3 * n] + w.rate_bias).reshape(t, h, dk)
+    v, gate = p[:, 3 * n:3 * n + m].reshape(t, h, dv), torch.sigmoid(p[:, 3 * n + m:])
+    decay = torch.exp(-math.exp(-0.5) * torch.sigmoid(z.float() + w.decay_bias)).reshape(t, h, dk)
+    u = k * torch.rsqrt(k.pow(2).sum(-1, keepdim=True) + 1e-6)
+    o = torch.zeros(t, h, dv)
+    for i, slot in enumerate(slots.tolist()):
+        first, last = bounds[i], bounds[i + 1]
+        if first == last:
+            continue
+        s = state[slot].clone() if slot >= 0 and int(positions[first]) > 0 else torch.zeros(h, dk, dv)
+        for j in range(first, last):
+            read = (s * u[j, :, :, None]).sum(1)
+            s = decay[j, :, :, None] * s - (a[j] * u[j])[:, :, None] * read[:, None] + k[j, :, :, None] * v[j, :, None]
+            o[j] = (s * r[j, :, :, None]).sum(1)
+        if slot >= 0:
+            state[slot] = s
+    o = o * torch.rsqrt(o.pow(2).sum(-1, keepdim=True) / w.d_true + w.eps)
+    return (o.reshape(t, m) * w.norm.float() * gate).to(proj.dtype)
+
+
+def input_conv(h, w, state, positions, cu_q, slots) -> torch.Tensor:
+    """``h`` plus causal convolutions of it over a ragged batch (see ``ops.input_conv``)."""
+    n, taps, c = w.shape
+    bounds = list(range(slots.numel() + 1)) if cu_q is None else cu_q.tolist()
+    out = torch.empty(n, *h.shape, dtype=h.dtype)
+    for i, slot in enumerate(slots.tolist()):
+        a, b = bounds[i], bounds[i + 1]
+        if b == a:
+            continue
+        carried = slot >= 0 and int(positions[a]) > 0
+        seq = torch.cat([state[slot].float() if carried else torch.zeros(taps - 1, c), h[a:b].float()], 0)
+        if slot >= 0 and taps > 1:
+            state[slot] = seq[-(taps - 1):].to(state.dtype)
+        win = seq.unfold(0, taps, 1)
+        for j in range(n):
+            out[j, a:b] = (h[a:b].float() + (win * w[j].t()[None]).sum(-1)).to(h.dtype)
     return out
 
 
@@ -328,11 +379,11 @@ def turn(x: torch.Tensor, table: torch.Tensor, interleaved: bool) -> torch.Tenso
 def attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, causal: bool = False,
               scale: Optional[float] = None, softcap: float = 0.0, window: int = 0,
               alibi: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None,
-              dist_bias: Optional[torch.Tensor] = None, keep_first: int = 0) -> torch.Tensor:
+              dist_bias: Optional[torch.Tensor] = None, keep_first: int = 0, slopes: Optional[torch.Tensor] = None) -> torch.Tensor:
     """q [Tq, Hq, D], k [Tk, Hkv, D], v [Tk, Hkv, Dv] (one sequence). The last query row sits at key position
     Tk - 1 (so a query chunk with a cached prefix is expressed by Tk > Tq). ``alibi`` [Hq] adds
     slope * key position to the scores; ``dist_bias`` [Hq, n] adds a value by key distance (its last
-    entry also for longer distances); ``sinks`` [Hq] adds one extra logit per head to the softmax
+    entry also for longer distances), ``slopes`` [Hq] takes off slope * distance; ``sinks`` [Hq] adds one extra logit per head to the softmax
     denominator (it attends to nothing). The ``keep_first`` first keys stay visible outside the window. Returns fp32
     [Tq, Hq, Dv]."""
     tq, hq, d = q.shape
@@ -355,6 +406,8 @@ def attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, causal: bool = 
         s = s + alibi.float()[:, None, None] * kpos[None].float()
     if dist_bias is not None:
         s = s + dist_bias.float()[:, (qpos - kpos).clamp(0, dist_bias.shape[1] - 1)]
+    if slopes is not None:
+        s = s - slopes.float()[:, None, None] * (qpos - kpos)[None].float()
     s = s.masked_fill(~mask[None], float("-inf"))
     if sinks is not None:
         s = torch.cat([s, sinks.float()[:, None, None].expand(hq, tq, 1)], -1)
