@@ -9,8 +9,8 @@ The other headline workloads run through ``--preset``: ``deepseek-v3`` (DeepSeek
 fp8, 256 x (1024 + 128), experts sharded over N = 8 GPUs; decode tok/s), ``flux-dev`` (Flux-Dev
 1024 x 1024, TP = N; s/step) and ``wan-14b`` (Wan2.1-14B, 81 frames x 720 x 1280, sequence parallel
 + CFG-parallel over N GPUs; s/step), see ``benchmarks/headline_dit.py``. ``--preset lududra``,
-``--preset salopel`` and ``--preset zovudra`` time layers of these designs beside existing models (one GPU,
-``benchmarks/bench_mixers.py``, ``benchmarks/bench_salopel.py``, ``benchmarks/bench_zovudra.py``). On more than one GPU every
+``salopel``, ``zovudra`` and ``ginodra`` time layers of these designs beside existing models (one GPU,
+``benchmarks/bench_mixers.py``, ``bench_salopel.py``, ``bench_zovudra.py``, ``bench_ginodra.py``). On more than one GPU every
 preset first checks a two-layer slice of its model in the parallel layout against one rank alone
 and reports it as ``parity``.
 
@@ -50,7 +50,7 @@ def parse_args():
     ap.add_argument("--warmup", type=int, default=4)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--preset", default="llama-3-70b",
-                    choices=["llama-3-70b", "deepseek-v3", "flux-dev", "wan-14b", "llama-3-8b", "qwen2.5-0.5b", "lududra", "salopel", "zovudra"],
+                    choices=["llama-3-70b", "deepseek-v3", "flux-dev", "wan-14b", "llama-3-8b", "qwen2.5-0.5b", "lududra", "salopel", "zovudra", "ginodra"],
                     help="workload (the headline is llama-3-70b)")
     ap.add_argument("--batch", type=int, default=0, help="requests (default: 64; deepseek-v3: 256)")
     ap.add_argument("--prompt-len", type=int, default=0, help="prompt tokens (default: 2048; deepseek-v3: 1024)")
@@ -177,9 +177,9 @@ def main() -> int:
         import logging
         log.logger.setLevel(logging.WARNING)
     sys.path.insert(0, os.path.join(ROOT, "benchmarks"))
-    if args.preset in ("lududra", "salopel", "zovudra"):
+    if args.preset in ("lududra", "salopel", "zovudra", "ginodra"):
         import importlib
-        bench = importlib.import_module({"lududra": "bench_mixers", "salopel": "bench_salopel", "zovudra": "bench_zovudra"}[args.preset])
+        bench = importlib.import_module({"lududra": "bench_mixers", "salopel": "bench_salopel", "zovudra": "bench_zovudra", "ginodra": "bench_ginodra"}[args.preset])
         if rank == 0:
             print(json.dumps(bench.run(args, device, ClockSampler(local_rank))))
         return _leave(comm, world)

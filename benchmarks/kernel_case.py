@@ -12,6 +12,8 @@
     python benchmarks/kernel_case.py latent 64 2048 16
     python benchmarks/kernel_case.py latent_rot 4 2048 16 1024 runs
     python benchmarks/kernel_case.py qk_rope 8192 16 4
+    python benchmarks/kernel_case.py general_delta 4 2048 16
+    python benchmarks/kernel_case.py input_conv 8192 2048
 
 Inputs are larger than the L2 cache where the op is bandwidth bound but stay far below a few GB,
 so a full-metric capture (dozens of replays per launch) ends in about a minute. The status word is
@@ -418,7 +420,31 @@ def _qk_rope(argv):
     print(f"qk_rope {argv}: {_time_cold(fn) * 1e3:.1f} us")
 
 
-CASES = {"qk_rope": _qk_rope, "latent_rot": _latent_rot, "channel_scan": _channel_scan, "head_scan": _head_scan, "latent": _latent, "delta": _delta, "attn_window": _attn_window, "mla_proj": _mla_proj, "gemm_ar_large": _gemm_ar_large, "ag_gemm": _ag_gemm, "ulysses": _ulysses, "allreduce": _allreduce, "sample": _sample,
+def _general_delta(argv):
+    """general_delta SEQS TOKENS HEADS: the delta rule with removal rates per channel, head size 128 (TOKENS = 1: a decode step)."""
+    seqs, n, h = (int(v) for v in argv[:3])
+    t, pos, cu, slots = _scan_batch(seqs, n)
+    c, dev = h * 128, "cuda"
+    w = ops.GeneralDeltaWeights(decay_bias=torch.full((c,), -4.0, device=dev), rate_bias=torch.zeros(c, device=dev),
+                                norm=torch.ones(c, dtype=torch.bfloat16, device=dev), heads=h, dk=128, dv=128, d_true=128, eps=1e-6)
+    st = torch.zeros(seqs, h, 128, 128, device=dev)
+    proj, z = torch.randn(t, 5 * c + 128, device=dev).to(torch.bfloat16), torch.randn(t, c, device=dev).to(torch.bfloat16)
+    ms = _time_cold(lambda: ops.general_delta(proj, z, w, st, pos, cu, slots))
+    print(f"general_delta {seqs} x {n} tokens x {h} heads: {ms * 1e3:.1f} us")
+
+
+def _input_conv(argv):
+    """input_conv TOKENS WIDTH: both convolutions of a layer's normed input, four taps, four prompts."""
+    t, w = (int(v) for v in argv[:2])
+    dev = "cuda"
+    h, taps = torch.randn(t, w, device=dev).to(torch.bfloat16), torch.randn(2, 4, w, device=dev)
+    st, cu = torch.zeros(4, 3, w, dtype=torch.bfloat16, device=dev), torch.arange(0, t + 1, t // 4, dtype=torch.int32, device=dev)
+    pos, slots = torch.full((t,), 5, dtype=torch.int32, device=dev), torch.arange(4, dtype=torch.int32, device=dev)
+    ms = _time_cold(lambda: ops.input_conv(h, taps, st, pos, cu, slots))
+    print(f"input_conv {argv}: {ms * 1e3:.1f} us")
+
+
+CASES = {"general_delta": _general_delta, "input_conv": _input_conv, "qk_rope": _qk_rope, "latent_rot": _latent_rot, "channel_scan": _channel_scan, "head_scan": _head_scan, "latent": _latent, "delta": _delta, "attn_window": _attn_window, "mla_proj": _mla_proj, "gemm_ar_large": _gemm_ar_large, "ag_gemm": _ag_gemm, "ulysses": _ulysses, "allreduce": _allreduce, "sample": _sample,
          "int8": _int8, "triplane": _triplane,
          "gemm_ar": _gemm_ar, "attn_dense": _attn_dense, "gemm": _gemm, "grouped": _grouped, "attn_decode": _attn_decode, "mla": _mla}
 
