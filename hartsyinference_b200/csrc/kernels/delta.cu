@@ -556,7 +556,10 @@ cudaError_t launch_scan(const DeltaParams& p, cudaStream_t stream) {
   const int smem = 2 * kScanTokens * (3 * NR * 32 + kScanCols + 4) * 4;
   static PerDeviceOnce once;
   if (once.first_time()) cudaFuncSetAttribute(delta_scan_kernel<NR>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
-  return launch_pdl(delta_scan_kernel<NR>, dim3((p.dv + kScanCols - 1) / kScanCols, p.h, p.seqs), dim3(128), smem, stream, p);
+  // an ordinary launch: blocks that were started while the last blocks of the kernel before still run would crowd the
+  // processors that are free first, and there are few blocks
+  delta_scan_kernel<NR><<<dim3((p.dv + kScanCols - 1) / kScanCols, p.h, p.seqs), 128, smem, stream>>>(p);
+  return cudaGetLastError();
 }
 
 template <typename T, int NRT, int kMax>

@@ -10,7 +10,7 @@
 //
 //  * general_prep   one warp per (token, head): unit key, decay, removal and read vectors and both dot products as one
 //                   fp32 record.
-//  * general_scan   portions of prompts: the columns of S are independent, a block takes 32 of them (a thread keeps two
+//  * general_scan   portions of prompts: the columns of S are independent, a block takes 32 of them (a thread keeps four
 //                   columns of an eighth of the rows in registers) and walks over the tokens, whose records are staged
 //                   through shared memory. The operations do not depend on where a prompt is cut.
 //  * general_gate   the output norm and gate of a scanned portion, one warp per (token, head).
@@ -114,19 +114,19 @@ __global__ void __launch_bounds__(256) general_prep_kernel(const GeneralDeltaPar
 
 constexpr int kGenTokens = 8;      // tokens per staging buffer
 constexpr int kGenCols = 32;       // columns of S per block
+constexpr int kGenFew = 1200;      // fewer blocks than this: more lanes per column
 
-// grid: (ceil(dv / 32), h, seqs), 128 threads. dk = 32 * NR. Lane: rows i * 32 + (lane % 8) * 4 + 0..3 of columns
-// 2 * (lane / 8), + 1 of the warp's eight.
-template <int NR>
-__global__ void __launch_bounds__(128) general_scan_kernel(const GeneralDeltaParams p) {
-  pdl_wait();
-  pdl_trigger();
-  constexpr int DK = NR * 32;
+// grid: (ceil(dv / 32), h, seqs), 8 RL threads. dk = 4 RL NV. A column's rows are dealt over RL lanes (8, or 16 for more
+// warps when there are few columns). Lane: rows 4 (i RL + lane % RL) + 0..3 of columns 4 (lane / RL) + 0..3 of the warp's:
+// four columns share what a lane reads from shared memory.
+template <int NV, int RL>
+__global__ void __launch_bounds__(8 * RL) general_scan_kernel(const GeneralDeltaParams p) {
+  constexpr int DK = NV * RL * 4, NR = NV, kStep = 4 * RL, kThreads = 8 * RL;
   constexpr int kTok = 4 + 4 * DK + kGenCols;       // floats per staged token
   extern __shared__ __align__(16) float sm[];
   const int head = blockIdx.y, seq = blockIdx.z, tid = threadIdx.x;
-  const int warp = tid >> 5, lane = tid & 31, rg = lane & 7;
-  const int col0 = blockIdx.x * kGenCols, lc = warp * 8 + (lane >> 3) * 2, col = col0 + lc;
+  const int rg = tid % RL;
+  const int col0 = blockIdx.x * kGenCols, lc = tid / RL * 4, col = col0 + lc;
   const int first = p.cu_q ? p.cu_q[seq] : seq;
   const int len = p.cu_q ? p.cu_q[seq + 1] - first : 1;
   if (len <= 0) return;
@@ -136,26 +136,26 @@ __global__ void __launch_bounds__(128) general_scan_kernel(const GeneralDeltaPar
   float* sp = p.state + (static_cast<long long>(slot < 0 ? 0 : slot) * p.h + head) * DK * p.dv + col;
   const int rec = record_floats(DK, p.dv);
 
-  f32x2 s0[NR * 2], s1[NR * 2];       // two columns, row pairs
+  f32x2 s[4][NR * 2];                 // four columns, row pairs
 #pragma unroll
   for (int i = 0; i < NR; ++i)
 #pragma unroll
     for (int j = 0; j < 2; ++j) {
-      float2 a = make_float2(0.f, 0.f), b = a;
+      float a[4] = {0.f, 0.f, 0.f, 0.f}, b[4] = {0.f, 0.f, 0.f, 0.f};
       if (carried && live) {
-        const float* rp = sp + static_cast<long long>(i * 32 + rg * 4 + j * 2) * p.dv;
-        a = *reinterpret_cast<const float2*>(rp);
-        b = *reinterpret_cast<const float2*>(rp + p.dv);
+        const float* rp = sp + static_cast<long long>(i * kStep + rg * 4 + j * 2) * p.dv;
+        ld4(rp, a);
+        ld4(rp + p.dv, b);
       }
-      s0[i * 2 + j] = pack2(a.x, b.x);
-      s1[i * 2 + j] = pack2(a.y, b.y);
+#pragma unroll
+      for (int c = 0; c < 4; ++c) s[c][i * 2 + j] = pack2(a[c], b[c]);
     }
 
   auto stage = [&](int t0, int buf) {
     float* base = sm + buf * kGenTokens * kTok;
     const int n = min(kGenTokens, len - t0);
     constexpr int kVec = kTok / 4;
-    for (int i = tid; i < n * kVec; i += 128) {
+    for (int i = tid; i < n * kVec; i += kThreads) {
       const int tk = i / kVec, c = (i - tk * kVec) * 4;
       const float* src = p.rec + (static_cast<long long>(first + t0 + tk) * p.h + head) * rec;
       const bool value = c >= 4 + 4 * DK;
@@ -176,58 +176,87 @@ __global__ void __launch_bounds__(128) general_scan_kernel(const GeneralDeltaPar
     const int n = min(kGenTokens, len - t0);
     const float* base = sm + buf * kGenTokens * kTok;
     float* op = p.o + (static_cast<long long>(first + t0) * p.h + head) * p.dv + col;
+    ulonglong2 nu[NR], ner[NR];            // the next token's u and e r, read while the current one is computed
+    auto fetch = [&](int tk) {
+      const float* rows = base + tk * kTok + 4 + rg * 4;
+#pragma unroll
+      for (int i = 0; i < NR; ++i) {
+        nu[i] = *reinterpret_cast<const ulonglong2*>(rows + i * kStep);
+        ner[i] = *reinterpret_cast<const ulonglong2*>(rows + 3 * DK + i * kStep);
+      }
+    };
+    fetch(0);
     for (int tq = 0; tq < n; tq += 4) {
-      float part[8];                       // outputs of four tokens x two columns, this lane's rows
+      float part[16];                      // outputs of four tokens x four columns, this lane's rows
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
-        part[2 * j] = part[2 * j + 1] = 0.f;
+#pragma unroll
+        for (int c = 0; c < 4; ++c) part[4 * j + c] = 0.f;
         if (tq + j >= n) continue;
         const float* tb = base + (tq + j) * kTok;
         const float* rows = tb + 4 + rg * 4;
-        f32x2 p0 = 0, p1 = 0, q0 = 0, q1 = 0, x0 = 0, x1 = 0, y0 = 0, y1 = 0;
         ulonglong2 uu[NR];
+        f32x2 a[4], b[4], x[4], y[4];
+#pragma unroll
+        for (int c = 0; c < 4; ++c) a[c] = b[c] = x[c] = y[c] = 0;
 #pragma unroll
         for (int i = 0; i < NR; ++i) {
-          uu[i] = *reinterpret_cast<const ulonglong2*>(rows + i * 32);
-          const ulonglong2 er = *reinterpret_cast<const ulonglong2*>(rows + 3 * DK + i * 32);
-          p0 = fma2(s0[i * 2], uu[i].x, p0);
-          p1 = fma2(s1[i * 2], uu[i].x, p1);
-          q0 = fma2(s0[i * 2 + 1], uu[i].y, q0);
-          q1 = fma2(s1[i * 2 + 1], uu[i].y, q1);
-          x0 = fma2(s0[i * 2], er.x, x0);
-          x1 = fma2(s1[i * 2], er.x, x1);
-          y0 = fma2(s0[i * 2 + 1], er.y, y0);
-          y1 = fma2(s1[i * 2 + 1], er.y, y1);
-        }
-        float r0 = sum2(add2(p0, q0)), r1 = sum2(add2(p1, q1));
+          uu[i] = nu[i];
 #pragma unroll
-        for (int o = 1; o < 8; o <<= 1) {
-          r0 += __shfl_xor_sync(0xffffffffu, r0, o);
-          r1 += __shfl_xor_sync(0xffffffffu, r1, o);
+          for (int c = 0; c < 4; ++c) {
+            a[c] = fma2(s[c][i * 2], uu[i].x, a[c]);
+            b[c] = fma2(s[c][i * 2 + 1], uu[i].y, b[c]);
+          }
         }
-        const float2 c = *reinterpret_cast<const float2*>(tb);
-        const float2 v = *reinterpret_cast<const float2*>(tb + 4 + 4 * DK + lc);
-        part[2 * j] = sum2(add2(x0, y0));
-        part[2 * j + 1] = sum2(add2(x1, y1));
-        if (rg == 0) {                     // what the token itself adds, once per column
-          part[2 * j] += v.x * c.y - r0 * c.x;
-          part[2 * j + 1] += v.y * c.y - r1 * c.x;
+        float r[4];
+#pragma unroll
+        for (int c = 0; c < 4; ++c) r[c] = sum2(add2(a[c], b[c]));
+#pragma unroll
+        for (int o = 1; o < RL; o <<= 1)
+#pragma unroll
+          for (int c = 0; c < 4; ++c) r[c] += __shfl_xor_sync(0xffffffffu, r[c], o);
+#pragma unroll
+        for (int i = 0; i < NR; ++i)
+#pragma unroll
+          for (int c = 0; c < 4; ++c) {
+            x[c] = fma2(s[c][i * 2], ner[i].x, x[c]);
+            y[c] = fma2(s[c][i * 2 + 1], ner[i].y, y[c]);
+          }
+        fetch(min(tq + j + 1, n - 1));
+        const float2 k = *reinterpret_cast<const float2*>(tb);
+        float v[4];
+        ld4(tb + 4 + 4 * DK + lc, v);
+#pragma unroll
+        for (int i = 0; i < NR; ++i) {     // what does not need the reads: decay and the new value
+          const ulonglong2 e = *reinterpret_cast<const ulonglong2*>(rows + DK + i * kStep);
+#pragma unroll
+          for (int c = 0; c < 4; ++c) {
+            const f32x2 vc = pack2(v[c], v[c]);
+            s[c][i * 2] = fma2(uu[i].x, vc, mul2(e.x, s[c][i * 2]));
+            s[c][i * 2 + 1] = fma2(uu[i].y, vc, mul2(e.y, s[c][i * 2 + 1]));
+          }
         }
-        const f32x2 n0 = pack2(-r0, -r0), n1 = pack2(-r1, -r1), v0 = pack2(v.x, v.x), v1 = pack2(v.y, v.y);
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+          part[4 * j + c] = sum2(add2(x[c], y[c]));
+          if (rg == 0) part[4 * j + c] += v[c] * k.y - r[c] * k.x;     // what the token itself adds, once per column
+          r[c] = -r[c];
+        }
 #pragma unroll
         for (int i = 0; i < NR; ++i) {
-          const ulonglong2 e = *reinterpret_cast<const ulonglong2*>(rows + DK + i * 32);
-          const ulonglong2 au = *reinterpret_cast<const ulonglong2*>(rows + 2 * DK + i * 32);
-          s0[i * 2] = fma2(au.x, n0, fma2(uu[i].x, v0, mul2(e.x, s0[i * 2])));
-          s1[i * 2] = fma2(au.x, n1, fma2(uu[i].x, v1, mul2(e.x, s1[i * 2])));
-          s0[i * 2 + 1] = fma2(au.y, n0, fma2(uu[i].y, v0, mul2(e.y, s0[i * 2 + 1])));
-          s1[i * 2 + 1] = fma2(au.y, n1, fma2(uu[i].y, v1, mul2(e.y, s1[i * 2 + 1])));
+          const ulonglong2 au = *reinterpret_cast<const ulonglong2*>(rows + 2 * DK + i * kStep);
+#pragma unroll
+          for (int c = 0; c < 4; ++c) {
+            const f32x2 rc = pack2(r[c], r[c]);
+            s[c][i * 2] = fma2(au.x, rc, s[c][i * 2]);
+            s[c][i * 2 + 1] = fma2(au.y, rc, s[c][i * 2 + 1]);
+          }
         }
       }
-      // the eight lanes of a column pair add their parts: every exchange halves the values a lane keeps,
-      // and lane rg ends with token tq + rg / 2, column rg % 2
+      // the lanes of four columns add their parts: every exchange halves the values a lane keeps, and lane rg ends with
+      // one of the sixteen, or two neighbours
 #pragma unroll
-      for (int o = 4, cnt = 4; o > 0; o >>= 1, cnt >>= 1) {
+      for (int o = RL / 2, cnt = 8; o > 0; o >>= 1, cnt >>= 1) {
         const bool up = (rg & o) != 0;
 #pragma unroll
         for (int i = 0; i < cnt; ++i) {
@@ -235,8 +264,12 @@ __global__ void __launch_bounds__(128) general_scan_kernel(const GeneralDeltaPar
           part[i] = keep + __shfl_xor_sync(0xffffffffu, give, o);
         }
       }
-      const int tk = tq + (rg >> 1);
-      if (live && tk < n) op[static_cast<long long>(tk) * p.h * p.dv + (rg & 1)] = part[0];
+      const int at = rg * (16 / RL), tk = tq + (at >> 2);
+      if (live && tk < n) {
+        float* dst = op + static_cast<long long>(tk) * p.h * p.dv + (at & 3);
+        if (RL == 8) *reinterpret_cast<float2*>(dst) = make_float2(part[0], part[1]);
+        else *dst = part[0];
+      }
     }
     __syncthreads();
   }
@@ -245,12 +278,12 @@ __global__ void __launch_bounds__(128) general_scan_kernel(const GeneralDeltaPar
     for (int i = 0; i < NR; ++i)
 #pragma unroll
       for (int j = 0; j < 2; ++j) {
-        float2 a, b;
-        unpack2(s0[i * 2 + j], a.x, b.x);
-        unpack2(s1[i * 2 + j], a.y, b.y);
-        float* rp = sp + static_cast<long long>(i * 32 + rg * 4 + j * 2) * p.dv;
-        *reinterpret_cast<float2*>(rp) = a;
-        *reinterpret_cast<float2*>(rp + p.dv) = b;
+        float a[4], b[4];
+#pragma unroll
+        for (int c = 0; c < 4; ++c) unpack2(s[c][i * 2 + j], a[c], b[c]);
+        float* rp = sp + static_cast<long long>(i * kStep + rg * 4 + j * 2) * p.dv;
+        st4(rp, a);
+        st4(rp + p.dv, b);
       }
   }
 }
@@ -401,12 +434,15 @@ __global__ void __launch_bounds__(kMax, kMax <= 512 ? 2 : 1) general_step_kernel
   }
 }
 
-template <int NR>
+// An ordinary launch: blocks that were started while the last blocks of the kernel before still run would crowd the
+// processors that are free first, and there are few blocks.
+template <int NV, int RL>
 cudaError_t launch_general_scan(const GeneralDeltaParams& p, cudaStream_t stream) {
-  const int smem = 2 * kGenTokens * (4 + 4 * NR * 32 + kGenCols) * 4;
+  const int smem = 2 * kGenTokens * (4 + 16 * NV * RL + kGenCols) * 4;
   static PerDeviceOnce once;
-  if (once.first_time()) cudaFuncSetAttribute(general_scan_kernel<NR>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
-  return launch_pdl(general_scan_kernel<NR>, dim3((p.dv + kGenCols - 1) / kGenCols, p.h, p.seqs), dim3(128), smem, stream, p);
+  if (once.first_time()) cudaFuncSetAttribute(general_scan_kernel<NV, RL>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+  general_scan_kernel<NV, RL><<<dim3((p.dv + kGenCols - 1) / kGenCols, p.h, p.seqs), 8 * RL, smem, stream>>>(p);
+  return cudaGetLastError();
 }
 
 template <typename T, int NRT, int kMax>
@@ -446,15 +482,16 @@ int general_delta_impl(const GeneralDeltaParams& p, cudaStream_t stream) {
   const dim3 warps(static_cast<unsigned>((static_cast<long long>(p.tokens) * p.h + 7) / 8));
   e = launch_pdl(general_prep_kernel<T>, warps, dim3(256), 0, stream, p);
   if (e != cudaSuccess) return -static_cast<int>(e) - 300;
+  const bool few = static_cast<long long>((p.dv + kGenCols - 1) / kGenCols) * p.h * p.seqs < kGenFew;
   switch (p.dk / 32) {
-    case 1: e = launch_general_scan<1>(p, stream); break;
-    case 2: e = launch_general_scan<2>(p, stream); break;
-    case 3: e = launch_general_scan<3>(p, stream); break;
-    case 4: e = launch_general_scan<4>(p, stream); break;
-    case 5: e = launch_general_scan<5>(p, stream); break;
-    case 6: e = launch_general_scan<6>(p, stream); break;
-    case 7: e = launch_general_scan<7>(p, stream); break;
-    default: e = launch_general_scan<8>(p, stream); break;
+    case 1: e = launch_general_scan<1, 8>(p, stream); break;
+    case 2: e = few ? launch_general_scan<1, 16>(p, stream) : launch_general_scan<2, 8>(p, stream); break;
+    case 3: e = launch_general_scan<3, 8>(p, stream); break;
+    case 4: e = few ? launch_general_scan<2, 16>(p, stream) : launch_general_scan<4, 8>(p, stream); break;
+    case 5: e = launch_general_scan<5, 8>(p, stream); break;
+    case 6: e = few ? launch_general_scan<3, 16>(p, stream) : launch_general_scan<6, 8>(p, stream); break;
+    case 7: e = launch_general_scan<7, 8>(p, stream); break;
+    default: e = launch_general_scan<4, 16>(p, stream); break;
   }
   if (e != cudaSuccess) return -static_cast<int>(e) - 300;
   e = launch_pdl(general_gate_kernel<T>, warps, dim3(256), 0, stream, p);

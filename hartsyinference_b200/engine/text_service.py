@@ -564,7 +564,7 @@ class TextService:
                 n = len(ids)
                 dev = m.device
                 pages = (n + 15) // 16
-                saved, saved_state = m.kv_cache, getattr(m, "mixer_state", None)
+                saved, saved_state = m.kv_cache, (getattr(m, "mixer_state", None), getattr(m, "input_state", None))
                 m.alloc_kv(max(pages, 1), 16)
                 recurrent = getattr(m.cfg, "recurrent", False)
                 if recurrent:
@@ -579,6 +579,6 @@ class TextService:
                 hid = m.forward_hidden(b)[:, :m.cfg.hidden_size].float().mean(0)
                 m.kv_cache = saved
                 if recurrent:
-                    m.mixer_state = saved_state
+                    m.mixer_state, m.input_state = saved_state
                 outs.append(torch.nn.functional.normalize(hid, dim=0).cpu())
         return torch.stack(outs)
