@@ -36,6 +36,7 @@ struct GeneralDeltaParams {
   void* out;                 // [T][ldo]
   long long ldp, ldz, ldo;
   int tokens, seqs, h, dk, dv, d_true;
+  int longest;               // tokens of the longest portion (0: not known)
   float eps;
 };
 
@@ -482,7 +483,9 @@ int general_delta_impl(const GeneralDeltaParams& p, cudaStream_t stream) {
   const dim3 warps(static_cast<unsigned>((static_cast<long long>(p.tokens) * p.h + 7) / 8));
   e = launch_pdl(general_prep_kernel<T>, warps, dim3(256), 0, stream, p);
   if (e != cudaSuccess) return -static_cast<int>(e) - 300;
-  const bool few = static_cast<long long>((p.dv + kGenCols - 1) / kGenCols) * p.h * p.seqs < kGenFew;
+  // single tokens beside long portions are done soon: count the portions as if all were as long as the longest
+  const int portions = p.longest > 0 ? (p.tokens + p.longest - 1) / p.longest : p.seqs;
+  const bool few = static_cast<long long>((p.dv + kGenCols - 1) / kGenCols) * p.h * portions < kGenFew;
   switch (p.dk / 32) {
     case 1: e = launch_general_scan<1, 8>(p, stream); break;
     case 2: e = few ? launch_general_scan<1, 16>(p, stream) : launch_general_scan<2, 8>(p, stream); break;
@@ -514,10 +517,11 @@ B200_API int b200_general_delta_launches(int decode, int dk, int dv) {
 
 // See the header comment and GeneralDeltaParams. dk (<= 256) a multiple of 32, dv (<= 256) a multiple of 8; d_true is the
 // head size before padding (the output norm uses it; padded channels carry zeros). cu_q null: one token per sequence.
+// longest: tokens of the longest portion, 0 when not known.
 B200_API int b200_general_delta(const void* proj, const void* z, const float* decay_bias, const float* rate_bias, const void* norm_w,
                                 void* state, const int* positions, const int* cu_q, const int* slots, void* workspace, void* out,
                                 int tokens, int seqs, int h, int dk, int dv, int d_true, long long ldp, long long ldz, long long ldo,
-                                float eps, int f32, cudaStream_t stream) {
+                                float eps, int longest, int f32, cudaStream_t stream) {
   if (tokens <= 0 || seqs <= 0) return 0;
   if (dk % 32 || dk < 32 || dk > kGenMaxD || dv % 8 || dv < 8 || dv > kGenMaxD || h < 1 || h > 65535 || seqs > 65535) return -2;
   if (ldp % 8 || ldz % 8 || ldo % 8 || ldp < 3ll * h * dk + 2ll * h * dv || (!cu_q && tokens != seqs)) return -2;
@@ -530,5 +534,6 @@ B200_API int b200_general_delta(const void* proj, const void* z, const float* de
   p.o = p.rec + static_cast<long long>(tokens) * h * record_floats(dk, dv);
   p.out = out; p.ldp = ldp; p.ldz = ldz; p.ldo = ldo;
   p.tokens = tokens; p.seqs = seqs; p.h = h; p.dk = dk; p.dv = dv; p.d_true = d_true; p.eps = eps;
+  p.longest = longest;
   return f32 ? general_delta_impl<float>(p, stream) : general_delta_impl<__nv_bfloat16>(p, stream);
 }

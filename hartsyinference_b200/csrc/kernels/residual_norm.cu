@@ -131,9 +131,35 @@ __device__ __forceinline__ void group_norm_row(float (&v)[kIters][8], const floa
   }
 }
 
-// One token per sequence: h[i][row] = v + sum over the taps, the state moves on by one token.
+// One token per sequence: h[i][row] = v + sum over the taps, the state moves on by one token. The state was last written
+// by an earlier step, not by the kernel right before this one: up to three rows of it are read ahead of the wait.
+constexpr int kConvAhead = 3;
+
 template <typename T, int kIters>
-__device__ __forceinline__ void conv_row(const ResidualNormParams& p, long long row, const float (&v)[kIters][8]) {
+struct ConvAhead {
+  struct alignas(16) Vec { T v[8]; };       // as stored: half the registers for bf16
+  Vec in[kIters][kConvAhead];
+  __device__ __forceinline__ void load(const ResidualNormParams& p, long long row) {
+    const int slot = p.slots[row], tail = p.taps - 1;
+    const bool carried = slot >= 0 && p.positions[row] > 0;
+    const T* state = static_cast<const T*>(p.conv_state) + static_cast<long long>(slot < 0 ? 0 : slot) * tail * p.ldh;
+#pragma unroll
+    for (int i = 0; i < kIters; ++i) {
+      const int c = (threadIdx.x + i * blockDim.x) * 8;
+#pragma unroll
+      for (int k = 0; k < kConvAhead; ++k) {
+        in[i][k] = Vec{};
+        if (carried && k < tail && c < p.ldh) in[i][k] = *reinterpret_cast<const Vec*>(state + static_cast<long long>(k) * p.ldh + c);
+      }
+      if (c < p.ldh)                          // weights on their way into L2
+        for (int k = 0; k < p.conv_n * p.taps; ++k) asm volatile("prefetch.global.L2 [%0];" ::"l"(p.conv_w + static_cast<long long>(k) * p.ldh + c));
+      if (p.w_n != nullptr && c < p.dim) asm volatile("prefetch.global.L2 [%0];" ::"l"(p.w_n + c));
+    }
+  }
+};
+
+template <typename T, int kIters>
+__device__ __forceinline__ void conv_row(const ResidualNormParams& p, long long row, const float (&v)[kIters][8], const ConvAhead<T, kIters>& ahead) {
   const int slot = p.slots[row], tail = p.taps - 1;
   const bool carried = slot >= 0 && p.positions[row] > 0;
   T* state = static_cast<T*>(p.conv_state) + static_cast<long long>(slot < 0 ? 0 : slot) * tail * p.ldh;
@@ -144,11 +170,7 @@ __device__ __forceinline__ void conv_row(const ResidualNormParams& p, long long 
     float now[8], y[2][8];
 #pragma unroll
     for (int j = 0; j < 8; ++j) now[j] = y[0][j] = y[1][j] = ld1_of<T>(v[i][j]);
-    for (int k = 0; k < p.taps; ++k) {
-      float in[8];
-#pragma unroll
-      for (int j = 0; j < 8; ++j) in[j] = k == tail ? now[j] : 0.f;
-      if (k < tail && carried) load8(state + static_cast<long long>(k) * p.ldh + c, in);
+    auto tap = [&](int k, const float (&in)[8]) {
       if (k > 0 && slot >= 0) store8(state + static_cast<long long>(k - 1) * p.ldh + c, in);
 #pragma unroll
       for (int o = 0; o < 2; ++o)
@@ -158,7 +180,23 @@ __device__ __forceinline__ void conv_row(const ResidualNormParams& p, long long 
 #pragma unroll
           for (int j = 0; j < 8; ++j) y[o][j] = fmaf(in[j], w[j], y[o][j]);
         }
+    };
+#pragma unroll
+    for (int k = 0; k < kConvAhead; ++k)
+      if (k < tail) {
+        float in[8];
+#pragma unroll
+        for (int j = 0; j < 8; ++j) in[j] = ld1(&ahead.in[i][k].v[j]);
+        tap(k, in);
+      }
+    for (int k = kConvAhead; k < tail; ++k) {
+      float in[8];
+#pragma unroll
+      for (int j = 0; j < 8; ++j) in[j] = 0.f;
+      if (carried) load8(state + static_cast<long long>(k) * p.ldh + c, in);
+      tap(k, in);
     }
+    tap(tail, now);
 #pragma unroll
     for (int o = 0; o < 2; ++o)
       if (o < p.conv_n) store8(static_cast<T*>(p.h) + (static_cast<long long>(o) * gridDim.x + row) * p.ldh + c, y[o]);
@@ -186,12 +224,15 @@ __device__ __forceinline__ void tanh_row(float (&v)[kIters][8], const __nv_bfloa
 }
 
 // One block per row; every leading dimension is a multiple of 8 and covers dim rounded up to 8.
-template <typename T, int kIters>
+// kConv: conv_w is given (rows come one per sequence, so they are few and two vectors per thread mean long ones).
+template <typename T, int kIters, bool kConv>
 __global__ void __launch_bounds__(1024) residual_norm_kernel(const ResidualNormParams p) {
+  const long long row = blockIdx.x;
+  ConvAhead<T, kConv ? kIters : 1> ahead;
+  if (kConv) ahead.load(p, row);
   pdl_wait();
   pdl_trigger();
   __shared__ float red[32];
-  const long long row = blockIdx.x;
   float* xr = p.x + row * p.ldx;
   float xv[kIters][8];
   if (p.y != nullptr) {
@@ -276,8 +317,8 @@ __global__ void __launch_bounds__(1024) residual_norm_kernel(const ResidualNormP
     extern __shared__ float parts[];
     group_norm_row<kIters>(xv, xr, p.w_n, p.dim, p.groups, p.plus_one, p.eps, parts);
   } else if (p.w_n != nullptr) norm_row<kIters>(xv, p.w_n, p.dim, p.layernorm, p.plus_one, p.eps, red);
-  if (p.conv_w != nullptr) {
-    conv_row<T, kIters>(p, row, xv);
+  if constexpr (kConv) {
+    conv_row<T, kIters>(p, row, xv, ahead);
     return;
   }
   T* hr = static_cast<T*>(p.h) + row * p.ldh;
@@ -460,11 +501,9 @@ int launch_residual_norm(const ResidualNormParams& p, int rows, cudaStream_t str
   int iters, threads;
   if (!row_shape(p.dim, rows, iters, threads)) return -2;
   const int smem = p.groups > 1 ? ((p.dim + 7) / 8 + p.groups) * 4 : 0;
-  cudaError_t e;
-  switch (iters) {
-    case 1: e = launch_pdl(residual_norm_kernel<T, 1>, dim3(rows), dim3(threads), smem, stream, p); break;
-    default: e = launch_pdl(residual_norm_kernel<T, 2>, dim3(rows), dim3(threads), smem, stream, p); break;
-  }
+  auto go = [&](auto kernel) { return launch_pdl(kernel, dim3(rows), dim3(threads), smem, stream, p); };
+  const cudaError_t e = p.conv_w ? (iters == 1 ? go(residual_norm_kernel<T, 1, true>) : go(residual_norm_kernel<T, 2, true>))
+                                 : (iters == 1 ? go(residual_norm_kernel<T, 1, false>) : go(residual_norm_kernel<T, 2, false>));
   return e == cudaSuccess ? 0 : -static_cast<int>(e) - 300;
 }
 

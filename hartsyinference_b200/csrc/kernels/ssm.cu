@@ -108,6 +108,7 @@ struct ShortConvParams {
   void* out;                 // [T][channels]
   long long ldx;
   int tokens, seqs, channels, taps, run;
+  long long plane;           // input_conv: values between the outputs of two sets of taps
 };
 
 __device__ __forceinline__ float silu_f32(float x) { return x * sigmoid_f32(x); }
@@ -264,7 +265,6 @@ __global__ void __launch_bounds__(128) input_conv_kernel(const ShortConvParams p
   const int taps = kTaps > 0 ? kTaps : p.taps, tail = taps - 1;
   const T* x = static_cast<const T*>(p.x) + c;
   T* out = static_cast<T*>(p.out) + c;
-  const long long plane = static_cast<long long>(p.tokens) * p.channels;
   float w[kOut][kT][8], in[kT][8];
   if (kTaps > 0)
 #pragma unroll
@@ -313,7 +313,7 @@ __global__ void __launch_bounds__(128) input_conv_kernel(const ShortConvParams p
               y[i] = fmaf(at >= 0 ? nw[at >= 0 ? at : 0][i] : in[at < 0 ? kT - 1 + at : 0][i], w[o][j][i], y[i]);
             }
           }
-          store8(out + o * plane + static_cast<long long>(t + u) * p.channels, y);
+          store8(out + o * p.plane + static_cast<long long>(t + u) * p.channels, y);
         }
 #pragma unroll
       for (int j = 0; j + 1 < kT; ++j)
@@ -362,7 +362,7 @@ __global__ void __launch_bounds__(128) input_conv_kernel(const ShortConvParams p
       }
     }
 #pragma unroll
-    for (int o = 0; o < kOut; ++o) store8(out + o * plane + static_cast<long long>(t) * p.channels, y[o]);
+    for (int o = 0; o < kOut; ++o) store8(out + o * p.plane + static_cast<long long>(t) * p.channels, y[o]);
   }
 }
 
@@ -1300,14 +1300,14 @@ B200_API int b200_short_conv(const void* x, const float* w, const float* bias, v
   return f32 ? launch_short_conv<float>(p, stream) : launch_short_conv<__nv_bfloat16>(p, stream);
 }
 
-// h [tokens][ldx] -> out [n][tokens][channels] (see input_conv_kernel) with w [n][taps][channels], n 1 or 2; channels
-// and ldx multiples of 8
+// h [tokens][ldx] -> out [n][tokens][channels], matrices `plane` values apart (see input_conv_kernel), with w
+// [n][taps][channels], n 1 or 2; channels, ldx and plane multiples of 8
 B200_API int b200_input_conv(const void* h, const float* w, void* state, const int* positions, const int* cu_q, const int* slots,
-                             void* out, int tokens, int seqs, int channels, int taps, int n, long long ldx, int f32,
+                             void* out, int tokens, int seqs, int channels, int taps, int n, long long ldx, long long plane, int f32,
                              cudaStream_t stream) {
   if (tokens <= 0 || seqs <= 0) return 0;
-  if (channels % 8 || ldx % 8 || taps < 1 || n < 1 || n > 2 || seqs > 65535 || (!cu_q && seqs != tokens)) return -2;
-  ShortConvParams p{h, w, nullptr, state, positions, cu_q, slots, out, ldx, tokens, seqs, channels, taps, 1};
+  if (channels % 8 || ldx % 8 || taps < 1 || n < 1 || n > 2 || plane % 8 || seqs > 65535 || (!cu_q && seqs != tokens)) return -2;
+  ShortConvParams p{h, w, nullptr, state, positions, cu_q, slots, out, ldx, tokens, seqs, channels, taps, 1, plane};
   if (f32) return n == 1 ? launch_input_conv<float, 1>(p, stream) : launch_input_conv<float, 2>(p, stream);
   return n == 1 ? launch_input_conv<__nv_bfloat16, 1>(p, stream) : launch_input_conv<__nv_bfloat16, 2>(p, stream);
 }

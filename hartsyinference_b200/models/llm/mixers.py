@@ -54,6 +54,22 @@ def _linear(parts: Iterable[torch.Tensor], device, bias: Optional[torch.Tensor] 
     return LinearWeight(w, None, None if bias is None else bias.to(torch.bfloat16).to(device).contiguous())
 
 
+def batch_parts(batch) -> list[tuple]:
+    """A batch as parts that one kernel form each takes best: (rows, sequences, their ``cu_q`` or None), the runs ahead of the
+    one-token runs that end a ragged batch (decoded tokens beside prompts), and those as a decode batch."""
+    whole = slice(None)
+    runs = None if batch.is_decode else getattr(batch, "runs", None)
+    if not runs:
+        return [(whole, whole, None if batch.is_decode else batch.cu_q)]
+    n = len(runs)
+    while n and runs[n - 1][0] == 1:
+        n -= 1
+    if n == len(runs):
+        return [(whole, whole, batch.cu_q)]
+    t = sum(r[0] for r in runs[:n])
+    return ([(slice(0, t), slice(0, n), batch.cu_q[:n + 1])] if n else []) + [(slice(t, None), slice(n, None), None)]
+
+
 def out_matrix(o: Optional[torch.Tensor], heads: int, v: int, vp: int, width: int, device) -> Optional[LinearWeight]:
     """A mixer's output matrix in its laid-out sizes; None when the layer holds it (:class:`ParallelBlock`)."""
     return None if o is None else _linear([pad_rows(pad_head_cols(o, heads, v, vp), pad_to(width, 8))], device)
@@ -110,7 +126,7 @@ class BiasedAttention:
         self.proj = _linear([pad_cols(p, wp) for p in parts], device, bias)
         self.o = out_matrix(o, hq, dv, vp, width, device)
         self.nq, self.nk, self.nv = hq * dp, 0 if borrowed else hk * dp, 0 if borrowed or self.shared_kv else hk * vp
-        self.inner = hq * vp
+        self.inner = hq * vp                       # columns of what :meth:`values` returns
         norm = lambda t, n: None if t is None else head(t, n).to(torch.bfloat16).to(device).contiguous()
         self.q_norm, self.k_norm = (norm(t, 1 if spec.head_norm else n) for t, n in ((q_norm, hq), (k_norm, hk)))
         self.rotary = None if spec.rot is None else Rotary(spec.rot, device)
@@ -163,11 +179,14 @@ class BiasedAttention:
             else:
                 ops.kv_store(p[:, k0:v0], kc, batch.slot_mapping)
                 ops.kv_store(p[:, v0:g0], vc, batch.slot_mapping)
-        return ops.attn_biased(q, kc, vc, batch.block_table, batch.kv_lens, None if batch.is_decode else batch.cu_q,
-                               heads=spec.heads, max_q_len=batch.max_q_len, max_kv_len=batch.max_kv_len, scale=self.scale,
-                               softcap=spec.softcap, window=spec.window, dist_bias=self.bias, sinks=self.sinks,
-                               gate=p[:, g0:] if self.gated else None, keep_first=spec.keep_first, slopes=self.slopes,
-                               head_gate=spec.head_gate, out=out)
+        if out is None:
+            out = torch.empty(h.shape[0], self.inner, dtype=h.dtype, device=h.device)
+        for rows, seqs, cu in batch_parts(batch):
+            ops.attn_biased(q[rows], kc, vc, batch.block_table[seqs], batch.kv_lens[seqs], cu, heads=spec.heads, max_q_len=batch.max_q_len,
+                            max_kv_len=batch.max_kv_len, scale=self.scale, softcap=spec.softcap, window=spec.window, dist_bias=self.bias,
+                            sinks=self.sinks, gate=p[rows, g0:] if self.gated else None, keep_first=spec.keep_first, slopes=self.slopes,
+                            head_gate=spec.head_gate, out=out[rows])
+        return out
 
     def __call__(self, h: torch.Tensor, batch, li: int, model) -> torch.Tensor:
         return ops.linear_act(self.values(h, batch, li, model), self.o)
@@ -249,8 +268,12 @@ class GeneralDeltaMixer:
     def values(self, h: torch.Tensor, batch, li: int, model, out: Optional[torch.Tensor] = None) -> torch.Tensor:
         p = ops.linear_act(h, self.proj, "tanh", act_from=self.low)
         z = ops.linear_act(p[:, self.low:], self.up)
-        return ops.general_delta(p, z, self.w, model.mixer_state[li][1], batch.positions, None if batch.is_decode else batch.cu_q,
-                                 batch.state_slots, out=out)
+        if out is None:
+            out = torch.empty(h.shape[0], self.inner, dtype=h.dtype, device=h.device)
+        for rows, seqs, cu in batch_parts(batch):
+            ops.general_delta(p[rows], z[rows], self.w, model.mixer_state[li][1], batch.positions[rows], cu, batch.state_slots[seqs], out=out[rows],
+                              runs=batch.runs[seqs] if cu is not None and batch.runs else None)
+        return out
 
     def __call__(self, h: torch.Tensor, batch, li: int, model) -> torch.Tensor:
         return ops.linear_act(self.values(h, batch, li, model), self.o)

@@ -901,6 +901,9 @@ class DecoderModel:
             x += m y, h = norm(x), (h + conv1(h), h + conv2(h))            [one launch at decode, two and the state's else]
             mixer and feed-forward side by side, one output product        -> y
         """
+        from .mixers import batch_parts
+        parts = batch_parts(batch)
+
         def inputs(y, li: int) -> tuple:
             lw = self.layers[li]
             if lw.input_conv is None:
@@ -910,8 +913,10 @@ class DecoderModel:
             if batch.is_decode:
                 both = ops.residual_norm(x, y, None, lw.in_norm, conv=(lw.input_conv, state, batch.positions, batch.state_slots), **kw)
             else:
-                both = ops.input_conv(ops.residual_norm(x, y, None, lw.in_norm, **kw), lw.input_conv, state, batch.positions, batch.cu_q,
-                                      batch.state_slots)
+                h = ops.residual_norm(x, y, None, lw.in_norm, **kw)
+                both = torch.empty(lw.input_conv.shape[0], *h.shape, dtype=h.dtype, device=h.device)
+                for rows, seqs, cu in parts:
+                    ops.input_conv(h[rows], lw.input_conv, state, batch.positions[rows], cu, batch.state_slots[seqs], out=both[:, rows])
             return both[0], both[-1]
 
         y = None

@@ -52,12 +52,12 @@ _SIGNATURES = {
     "b200_moe_combine": (i32, [vp, vp, vp, vp, i32, i32, i32, i32, vp]),
     "b200_glu_clamped": (i32, [vp, vp, i64, i32, f32, f32, f32, vp, i32, i32, vp]),
     "b200_residual_norm": (i32, [vp] * 9 + [i32] * 11 + [f32, f32, i32, vp, f32, vp, vp, i32, i32, vp, i32, i32, vp, vp, vp, vp]),
-    "b200_input_conv": (i32, [vp] * 7 + [i32] * 5 + [i64, i32, vp]),
+    "b200_input_conv": (i32, [vp] * 7 + [i32] * 5 + [i64, i64, i32, vp]),
     "b200_cap_logits": (i32, [vp, vp, i64, f32, f32, i32, vp]),
     "b200_head_norm_store": (i32, [vp] * 8 + [i32, i64] + [i32] * 10 + [f32, i32, vp]),
     "b200_general_delta_workspace_bytes": (i64, [i32, i32, i32, i32]),
     "b200_general_delta_launches": (i32, [i32, i32, i32]),
-    "b200_general_delta": (i32, [vp] * 11 + [i32] * 6 + [i64, i64, i64, f32, i32, vp]),
+    "b200_general_delta": (i32, [vp] * 11 + [i32] * 6 + [i64, i64, i64, f32, i32, i32, vp]),
     "b200_side_gate": (i32, [vp] * 4 + [i32] * 6 + [vp]),
     "b200_rope_table": (i32, [vp] * 4 + [i32] * 2 + [vp]),
     "b200_qk_rope_store": (i32, [vp] * 8 + [i32, i64] + [i32] * 11 + [f32, i32, vp]),

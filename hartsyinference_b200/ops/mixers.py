@@ -162,19 +162,22 @@ def residual_norm(x: torch.Tensor, y, w_b: Optional[torch.Tensor], w_n, *, dim: 
 
 
 def input_conv(h: torch.Tensor, w: torch.Tensor, state: torch.Tensor, positions: torch.Tensor, cu_q: Optional[torch.Tensor],
-               slots: torch.Tensor) -> torch.Tensor:
-    """``h + conv_i(h)`` for every i: [n, T, C] from ``h`` [T, C] (any row pitch) and ``w`` fp32 [n, taps, C] (last row: the
+               slots: torch.Tensor, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``h + conv_i(h)`` for every i: [n, T, C] (``out`` when given, any distance between its n matrices) from ``h`` [T, C] (any row pitch) and ``w`` fp32 [n, taps, C] (last row: the
     current token), causal over time per channel. ``state`` [slots, taps - 1, C] holds the inputs before each sequence's
     portion and is updated in place; a sequence whose first position is 0 starts from zeros, slot -1 is not stored."""
     t, c = h.shape
     if not h.is_cuda:
-        return R.input_conv(h, w, state, positions, cu_q, slots)
+        y = R.input_conv(h, w, state, positions, cu_q, slots)
+        return y if out is None else out.copy_(y)
     n, taps, _ = w.shape
     assert h.stride(1) == 1 and w.dtype == torch.float32 and w.is_contiguous() and w.shape[2] == c and state.dtype == h.dtype
     assert state.is_contiguous() and state.shape[1:] == (taps - 1, c) and slots.dtype == torch.int32 and positions.dtype == torch.int32
-    out = torch.empty(n, t, c, dtype=h.dtype, device=h.device)
+    if out is None:
+        out = torch.empty(n, t, c, dtype=h.dtype, device=h.device)
+    assert out.shape == (n, t, c) and out.stride(1) == c and out.stride(2) == 1 and out.dtype == h.dtype
     N.check(N.lib().b200_input_conv(h.data_ptr(), w.data_ptr(), state.data_ptr(), positions.data_ptr(), N.ptr(cu_q), slots.data_ptr(),
-                                    out.data_ptr(), t, slots.numel(), c, taps, n, h.stride(0), _f32(h), N.stream()),
+                                    out.data_ptr(), t, slots.numel(), c, taps, n, h.stride(0), out.stride(0), _f32(h), N.stream()),
             "b200_input_conv", 2 if cu_q is not None and taps > 1 else 1)
     return out
 
@@ -466,12 +469,14 @@ class GeneralDeltaWeights:
 
 
 def general_delta(proj: torch.Tensor, z: torch.Tensor, w: GeneralDeltaWeights, state: torch.Tensor, positions: torch.Tensor,
-                  cu_q: Optional[torch.Tensor], slots: torch.Tensor, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+                  cu_q: Optional[torch.Tensor], slots: torch.Tensor, out: Optional[torch.Tensor] = None,
+                  runs: Optional[list] = None) -> torch.Tensor:
     """Per head ``S = diag(e) S - (a u)(u^T S) + k v^T``, ``y = norm(S^T r) * weight * sigmoid(gate)`` with the unit key
     ``u = k / sqrt(k^2 + 1e-6)``, the decay ``e = exp(-exp(-1/2) sigmoid(z + decay_bias))`` and the removal rate
     ``a = sigmoid(logit + rate_bias)``, both per key channel. ``proj`` [T, ld] = r | k | a logits [heads * dk] | v | gate logits
     [heads * dv]; ``z`` [T, heads * dk] decay logits. ``state`` fp32 [slots, heads, dk, dv] is updated in place; a sequence
-    whose first position is 0 starts from zeros, slot -1 is not stored. Returns [T, heads * dv] (``out`` when given)."""
+    whose first position is 0 starts from zeros, slot -1 is not stored. ``runs`` (host list of (tokens, ..) per sequence of a ragged
+    batch) tells how the work is spread. Returns [T, heads * dv] (``out`` when given)."""
     t = proj.shape[0]
     if not proj.is_cuda:
         y = R.general_delta(proj, z, w, state, positions, cu_q, slots)
@@ -486,7 +491,8 @@ def general_delta(proj: torch.Tensor, z: torch.Tensor, w: GeneralDeltaWeights, s
     ws = torch.empty(L.b200_general_delta_workspace_bytes(t, w.heads, w.dk, w.dv), dtype=torch.uint8, device=proj.device)
     rc = L.b200_general_delta(proj.data_ptr(), z.data_ptr(), w.decay_bias.data_ptr(), w.rate_bias.data_ptr(), w.norm.data_ptr(), state.data_ptr(),
                               positions.data_ptr(), N.ptr(cu_q), slots.data_ptr(), ws.data_ptr(), out.data_ptr(), t, slots.numel(), w.heads, w.dk,
-                              w.dv, w.d_true, proj.stride(0), z.stride(0), out.stride(0), float(w.eps), _f32(proj), N.stream())
+                              w.dv, w.d_true, proj.stride(0), z.stride(0), out.stride(0), float(w.eps),
+                              max((r[0] for r in runs or ()), default=0), _f32(proj), N.stream())
     N.check(rc, "b200_general_delta", L.b200_general_delta_launches(int(decode), w.dk, w.dv))
     return out
 

@@ -476,7 +476,7 @@ def test_delta_far_write(mode):
 
 
 @pytest.mark.parametrize("mode", MODES[1:])
-@pytest.mark.parametrize("heads,dim", [(16, 32), (20, 64), (8, 96), (40, 128)])
+@pytest.mark.parametrize("heads,dim", [(16, 32), (60, 64), (40, 128), (20, 192)])
 def test_delta_long_portion_equals_short_ones(mode, heads, dim):
     """Many columns, so that a column's rows lie in fewer lanes, against pieces with few columns; two sequences and an empty
     run between them."""
@@ -525,6 +525,21 @@ def test_parallel_block(mode, width, ff, dim, rows):
     holder.mixer_state = [(None, torch.zeros(mixer.state_shapes(1)[1], device=dev))]
     y = b(h.to(dt).to(dev), hf.to(dt).to(dev), _Batch(dev, range(rows), [0], [0, rows]), 0, holder)
     near(y[:, :width], want, mode, 3e-5, 1.5e-2)
+
+
+def test_one_token_runs_at_the_end_are_a_part_of_their_own():
+    b = _Holder()
+    b.is_decode, b.cu_q = False, torch.tensor([0, 3, 4, 9, 10, 11])
+    b.runs = [(3, 3), (1, 8), (5, 9), (1, 2), (1, 40)]
+    (r1, s1, c1), (r2, s2, c2) = M.batch_parts(b)
+    assert (r1, s1, c1.tolist()) == (slice(0, 9), slice(0, 3), [0, 3, 4, 9]) and (r2, s2, c2) == (slice(9, None), slice(3, None), None)
+    b.runs = [(1, 3), (1, 1)]
+    assert M.batch_parts(b) == [(slice(0, None), slice(0, None), None)]
+    for runs in ([(1, 1), (2, 5)], None):
+        b.runs = runs
+        assert M.batch_parts(b) == [(slice(None), slice(None), b.cu_q)]
+    b.is_decode = True
+    assert M.batch_parts(b) == [(slice(None), slice(None), None)]
 
 
 # ------------------------------------------------------------------------------------ whole models
